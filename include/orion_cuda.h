@@ -122,6 +122,38 @@ typedef struct OrionModelDesc {
 int orion_cuda_model_create(OrionBackend *backend, const OrionModelDesc *desc, OrionModel **out);
 void orion_cuda_model_destroy(OrionModel *model);
 
+/* ---- layer-list models (no reference counterpart) ----
+ * Decoders whose layers are listed one by one, each with a token mixer of its own sizes and an
+ * optional feed-forward. A layer is parallel: h = RMSNorm(x); the mixer and the feed-forward each read
+ * h plus a causal per-channel convolution of h over `conv_taps` tokens, and both results are added to
+ * x. The logits are the final norm's output times the embedding table. Metapel is the one design
+ * of this kind. */
+enum { ORION_MIXER_MIN_GRU = 0, ORION_MIXER_LATENT_ATTENTION = 1 };
+typedef struct OrionLayerDesc {
+  uint32_t mixer;    /* ORION_MIXER_* */
+  uint32_t ffn_dim;  /* width of the dense GELU feed-forward; 0 = the layer has none */
+  uint32_t width;    /* min_gru: channels of the recurrence */
+  /* latent_attention: query heads, unrotated and rotated query/key dimensions and value size per head,
+   * latent size, sliding window in tokens (0 = every earlier token is seen), rotated pairs' dimensions
+   * and base, score scale */
+  uint32_t heads, dim, rot_dim, value_dim, kv_rank, window, rope_dims;
+  double rope_base, scale;
+} OrionLayerDesc;
+typedef struct OrionLayeredDesc {
+  uint32_t hidden_size, vocab_size, num_layers;
+  const OrionLayerDesc *layers; /* [num_layers], read during the call only */
+  double norm_eps;
+  uint32_t conv_taps;           /* 1 or more; conv_taps - 1 rows of h per layer are a sequence's state */
+  uint32_t max_position_embeddings; /* positions the rotation tables cover */
+  uint32_t num_blocks, block_size;  /* paged latent cache */
+  uint32_t num_state_slots;         /* sequences whose state is held at any time */
+  uint32_t compute_dtype;           /* ORION_DTYPE_F32 or ORION_DTYPE_BF16 */
+  uint32_t max_batch_tokens, max_batch_sequences;
+} OrionLayeredDesc;
+int orion_cuda_model_create_layered(OrionBackend *backend, const OrionLayeredDesc *desc, OrionModel **out);
+/* State slots of the model: 0 for models that carry nothing but the KV cache from step to step. */
+int orion_cuda_model_num_state_slots(const OrionModel *model, uint32_t *slots);
+
 /* Failure-detection self-test (no reference counterpart): every device-side wait of this library
  * gives up after a time limit, records an error word and lets its kernel finish, which the host
  * reports as EngineError::Backend. This entry point runs the same bounded wait on a barrier that
@@ -197,6 +229,22 @@ int orion_cuda_model_forward_greedy(OrionModel *model, const uint32_t *tokens,
                                     uint64_t num_block_tables, uint64_t num_sequences,
                                     int has_prefill, uint32_t *token_ids_out, float *logits_out,
                                     uint64_t logits_capacity);
+/* The general form of the two calls above. `state_slots` names the state slot of every sequence (models
+ * with state slots require it, null otherwise): a sequence that starts at position 0 takes its slot over,
+ * a later portion must continue at the position where the slot's last step ended. `logit_rows` lists the
+ * batch rows whose logits are wanted, in order (null: the last row of every sequence; an empty list: none);
+ * logits_out and token_ids_out then hold one entry per listed row. */
+int orion_cuda_model_forward_rows(OrionModel *model, const uint32_t *tokens,
+                                  uint64_t num_tokens, const uint32_t *positions,
+                                  uint64_t num_positions, const uint64_t *slot_token_counts,
+                                  uint64_t num_slot_token_counts, const uint64_t *context_lens,
+                                  uint64_t num_context_lens, const uint32_t *block_tables_flat,
+                                  const uint64_t *block_table_offsets,
+                                  uint64_t num_block_tables, uint64_t num_sequences,
+                                  int has_prefill, const uint32_t *state_slots,
+                                  uint64_t num_state_slots, const uint32_t *logit_rows,
+                                  uint64_t num_logit_rows, uint32_t *token_ids_out,
+                                  float *logits_out, uint64_t logits_capacity);
 
 /* Replays the previous successful forward on the device without any host<->
  * device copy (inputs and block tables stay resident). Used to time the

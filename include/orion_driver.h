@@ -42,7 +42,10 @@ typedef struct OrionCacheStats {
  * whose blocks came from the prefix cache. 0 = the reference's behaviour.
  * logical_decode_positions has none either: non-zero feeds a decode token at position
  * total_len - 1, its logical place, instead of the reference's total_len (scheduler.rs:283), so
- * that no cache slot is skipped and no step is refused. 0 = the reference's behaviour. */
+ * that no cache slot is skipped and no step is refused. 0 = the reference's behaviour.
+ * recompute_on_preempt: non-zero prefills a preempted sequence's generated tokens again after its prompt
+ * (the reference leaves them out of the cache). An engine around a model with state slots sets this and
+ * logical_decode_positions itself, and refuses skip_cached_prefix. */
 typedef struct OrionSchedulerConfig {
   uint64_t max_num_seqs, max_num_batched_tokens, max_model_len;
   uint32_t enable_chunked_prefill;
@@ -50,6 +53,7 @@ typedef struct OrionSchedulerConfig {
   uint32_t prioritize_decode;
   uint32_t skip_cached_prefix;
   uint32_t logical_decode_positions;
+  uint32_t recompute_on_preempt;
 } OrionSchedulerConfig;
 
 /* SamplingParams (crates/orion-core/src/sampling.rs:25-70), the fields the driver reads. */
@@ -95,6 +99,14 @@ uint64_t orion_sequence_id_peek(void);
 
 /* ---- KvCacheManager (crates/orion-kv-cache/src/manager.rs:85-425) ---- */
 OrionKvManager *orion_kv_manager_create(uint64_t num_blocks, uint64_t block_size, int prefix_caching_enabled);
+/* The same with state slots for models that carry recurrent state (no reference counterpart): allocate takes
+ * a slot (and fails with CacheExhausted when none is free), free gives it back. */
+OrionKvManager *orion_kv_manager_create_with_state(uint64_t num_blocks, uint64_t block_size, int prefix_caching_enabled,
+                                                   uint64_t num_state_slots);
+/* 1 and the sequence's slot, or 0 when it holds none. */
+int orion_kv_manager_state_slot(const OrionKvManager *m, uint64_t seq, uint32_t *slot);
+/* append_token for `count` tokens, all of them or none. */
+int orion_kv_manager_extend(OrionKvManager *m, uint64_t seq, uint64_t count);
 void orion_kv_manager_destroy(OrionKvManager *m);
 int orion_kv_manager_allocate(OrionKvManager *m, uint64_t seq, const uint32_t *prompt, uint64_t num_tokens,
                               OrionAllocationOutcome *outcome);                       /* :163-250 */

@@ -13,7 +13,9 @@ from .errors import (BackendError, CacheExhausted, ContextLengthExceeded, CudaUn
                      InternalError, InvalidRequest, ModelError, QueueFull)
 from .types import DType, Device, ForwardBatch, ForwardOutput, ModelMetadata
 from .backend import CudaBackend, device_count, is_available
-from .model import CudaTransformerModel, HfConfig, read_safetensors, write_safetensors
+from .model import CudaModel, CudaTransformerModel, HfConfig, read_safetensors, write_safetensors
+from .layered import CudaLayeredModel, LayeredMetadata, LayerSpec
+from .registry import load_model, model_class
 from .validate import Tolerance, ValidationReport, validate
 from .distributed import (Collective, CommunicationEstimate, NcclCollective, NcclCollectiveId, ParallelLayout, Rank,
                           Shard, ShardStrategy, SingleRank, shard_dimension)
@@ -24,7 +26,8 @@ from .attn_bench import PagedAttentionBench
 __all__ = [
     "BackendError", "CudaUnavailable", "EngineError", "InternalError", "InvalidRequest", "ModelError",
     "DType", "Device", "ForwardBatch", "ForwardOutput", "ModelMetadata", "CudaBackend",
-    "device_count", "is_available", "CudaTransformerModel", "HfConfig", "read_safetensors",
+    "device_count", "is_available", "CudaTransformerModel", "CudaModel", "CudaLayeredModel", "LayeredMetadata",
+    "LayerSpec", "load_model", "model_class", "HfConfig", "read_safetensors",
     "write_safetensors", "Tolerance", "ValidationReport", "validate", "Collective",
     "CommunicationEstimate", "NcclCollective", "NcclCollectiveId", "ParallelLayout", "Rank", "Shard", "ShardStrategy",
     "SingleRank", "shard_dimension", "ops", "PagedAttentionBench", "CacheExhausted", "ContextLengthExceeded",

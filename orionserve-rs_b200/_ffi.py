@@ -38,6 +38,21 @@ class OrionModelDesc(C.Structure):
     ]
 
 
+class OrionLayerDesc(C.Structure):
+    _fields_ = [(n, C.c_uint32) for n in ("mixer", "ffn_dim", "width", "heads", "dim", "rot_dim", "value_dim", "kv_rank",
+                                          "window", "rope_dims")] + [("rope_base", C.c_double), ("scale", C.c_double)]
+
+
+class OrionLayeredDesc(C.Structure):
+    _fields_ = [("hidden_size", C.c_uint32), ("vocab_size", C.c_uint32), ("num_layers", C.c_uint32),
+                ("layers", C.POINTER(OrionLayerDesc)), ("norm_eps", C.c_double), ("conv_taps", C.c_uint32),
+                ("max_position_embeddings", C.c_uint32), ("num_blocks", C.c_uint32), ("block_size", C.c_uint32),
+                ("num_state_slots", C.c_uint32), ("compute_dtype", C.c_uint32), ("max_batch_tokens", C.c_uint32),
+                ("max_batch_sequences", C.c_uint32)]
+
+
+MIXER_MIN_GRU, MIXER_LATENT_ATTENTION = 0, 1
+
 _lib = None
 
 _f32p, _u32p, _u64p, _u8p = (C.POINTER(C.c_float), C.POINTER(C.c_uint32), C.POINTER(C.c_uint64),
@@ -61,11 +76,14 @@ SIGNATURES = {
     "orion_cuda_backend_supports_dtype": (_int, [_vp, _int]),
     "orion_cuda_model_create": (_int, [_vp, C.POINTER(OrionModelDesc), C.POINTER(_vp)]),
     "orion_cuda_model_destroy": (None, [_vp]),
+    "orion_cuda_model_create_layered": (_int, [_vp, C.POINTER(OrionLayeredDesc), C.POINTER(_vp)]),
+    "orion_cuda_model_num_state_slots": (_int, [_vp, _u32p]),
     "orion_cuda_model_load_tensor": (_int, [_vp, C.c_char_p, _int, _u64p, _int, _vp]),
     "orion_cuda_model_finalize": (_int, [_vp]),
     "orion_cuda_model_init_random": (_int, [_vp, _u64, C.c_float]),
     "orion_cuda_model_forward": (_int, [_vp, *_BATCH, _vp, _u64]),
     "orion_cuda_model_forward_greedy": (_int, [_vp, *_BATCH, _u32p, _vp, _u64]),
+    "orion_cuda_model_forward_rows": (_int, [_vp, *_BATCH, _u32p, _u64, _u32p, _u64, _u32p, _vp, _u64]),
     "orion_cuda_model_load_checkpoint": (_int, [_vp, C.c_char_p, C.POINTER(C.c_uint64)]),
     "orion_cuda_poll_wait_timeouts": (_int, [_vp, C.POINTER(C.c_uint32)]),
     "orion_cuda_selftest_peer_wait": (_int, [_vp, C.c_uint64, C.POINTER(C.c_uint32), C.POINTER(C.c_uint32)]),
@@ -126,7 +144,8 @@ class OrionSchedulerConfig(C.Structure):
     _fields_ = [("max_num_seqs", C.c_uint64), ("max_num_batched_tokens", C.c_uint64), ("max_model_len", C.c_uint64),
                 ("enable_chunked_prefill", C.c_uint32), ("max_waiting_requests", C.c_uint64),
                 ("request_timeout_secs", C.c_uint64), ("prioritize_decode", C.c_uint32),
-                ("skip_cached_prefix", C.c_uint32), ("logical_decode_positions", C.c_uint32)]
+                ("skip_cached_prefix", C.c_uint32), ("logical_decode_positions", C.c_uint32),
+                ("recompute_on_preempt", C.c_uint32)]
 
 
 class OrionSamplingParams(C.Structure):
@@ -161,6 +180,9 @@ DRIVER_SIGNATURES = {
     "orion_hash_block": (_u64, [C.c_int, _u64, _u32p, _u64]),
     "orion_sequence_id_peek": (_u64, []),
     "orion_kv_manager_create": (C.c_void_p, [_u64, _u64, C.c_int]),
+    "orion_kv_manager_create_with_state": (C.c_void_p, [_u64, _u64, C.c_int, _u64]),
+    "orion_kv_manager_state_slot": (C.c_int, [C.c_void_p, _u64, _u32p]),
+    "orion_kv_manager_extend": (C.c_int, [C.c_void_p, _u64, _u64]),
     "orion_kv_manager_destroy": (None, [C.c_void_p]),
     "orion_kv_manager_allocate": (C.c_int, [C.c_void_p, _u64, _u32p, _u64, C.POINTER(OrionAllocationOutcome)]),
     "orion_kv_manager_commit_prefill": (None, [C.c_void_p, _u64, _u32p, _u64]),

@@ -396,6 +396,27 @@ int orion_cuda_model_create(OrionBackend *backend, const OrionModelDesc *desc, O
 
 void orion_cuda_model_destroy(OrionModel *model) { delete model; }
 
+int orion_cuda_model_create_layered(OrionBackend *backend, const OrionLayeredDesc *desc, OrionModel **out) {
+  clear_error();
+  if (!out || !desc) return set_error(ORION_ERR_INVALID_REQUEST, "null pointer argument");
+  *out = nullptr;
+  ORION_TRY(check_backend(backend));
+  ModelBase *impl = nullptr;
+  ORION_TRY(create_layered_model(backend, desc, &impl));
+  auto *m = new (std::nothrow) OrionModel();
+  if (!m) { delete impl; return set_error(ORION_ERR_INTERNAL, "out of host memory"); }
+  m->impl.reset(impl);
+  *out = m;
+  return ORION_OK;
+}
+
+int orion_cuda_model_num_state_slots(const OrionModel *model, uint32_t *slots) {
+  clear_error();
+  if (!model || !slots) return set_error(ORION_ERR_INVALID_REQUEST, "null pointer argument");
+  *slots = model->impl->num_state_slots();
+  return ORION_OK;
+}
+
 int orion_cuda_model_load_tensor(OrionModel *model, const char *name, int dtype, const uint64_t *shape, int ndim,
                                  const void *data) {
   clear_error();
@@ -426,7 +447,24 @@ int orion_cuda_model_forward_greedy(OrionModel *model, const uint32_t *tokens, u
   if (!model) return set_error(ORION_ERR_INVALID_REQUEST, "null model handle");
   BatchView b{tokens, num_tokens, positions, num_positions, slot_token_counts, num_slot_token_counts,
               context_lens, num_context_lens, block_tables_flat, block_table_offsets, num_block_tables,
-              num_sequences, has_prefill};
+              num_sequences, has_prefill, nullptr, 0, nullptr, 0};
+  return model->impl->forward(b, logits_out, logits_capacity, token_ids_out);
+}
+
+int orion_cuda_model_forward_rows(OrionModel *model, const uint32_t *tokens, uint64_t num_tokens,
+                                  const uint32_t *positions, uint64_t num_positions,
+                                  const uint64_t *slot_token_counts, uint64_t num_slot_token_counts,
+                                  const uint64_t *context_lens, uint64_t num_context_lens,
+                                  const uint32_t *block_tables_flat, const uint64_t *block_table_offsets,
+                                  uint64_t num_block_tables, uint64_t num_sequences, int has_prefill,
+                                  const uint32_t *state_slots, uint64_t num_state_slots,
+                                  const uint32_t *logit_rows, uint64_t num_logit_rows, uint32_t *token_ids_out,
+                                  float *logits_out, uint64_t logits_capacity) {
+  clear_error();
+  if (!model) return set_error(ORION_ERR_INVALID_REQUEST, "null model handle");
+  BatchView b{tokens, num_tokens, positions, num_positions, slot_token_counts, num_slot_token_counts,
+              context_lens, num_context_lens, block_tables_flat, block_table_offsets, num_block_tables,
+              num_sequences, has_prefill, logit_rows, num_logit_rows, state_slots, num_state_slots};
   return model->impl->forward(b, logits_out, logits_capacity, token_ids_out);
 }
 

@@ -188,28 +188,6 @@ struct Mapping {
   }
 };
 
-// Names ModelWeights::load asks for (transformer.rs:12-18, 73-118).
-bool model_uses(const std::string &name, uint32_t num_layers) {
-  if (name == "model.embed_tokens.weight" || name == "model.norm.weight" || name == "lm_head.weight") return true;
-  static const char prefix[] = "model.layers.";
-  if (name.compare(0, sizeof prefix - 1, prefix) != 0) return false;
-  size_t i = sizeof prefix - 1, digits = 0;
-  uint64_t layer = 0;
-  while (i < name.size() && name[i] >= '0' && name[i] <= '9' && digits < 9) {
-    layer = layer * 10 + (uint64_t)(name[i] - '0');
-    ++i;
-    ++digits;
-  }
-  if (digits == 0 || i >= name.size() || name[i] != '.' || layer >= num_layers) return false;
-  static const char *rest[] = {"input_layernorm.weight", "post_attention_layernorm.weight", "self_attn.q_proj.weight",
-                               "self_attn.k_proj.weight", "self_attn.v_proj.weight", "self_attn.o_proj.weight",
-                               "self_attn.q_proj.bias", "self_attn.k_proj.bias", "self_attn.v_proj.bias",
-                               "mlp.gate_proj.weight", "mlp.up_proj.weight", "mlp.down_proj.weight"};
-  for (const char *r : rest)
-    if (name.compare(i + 1, std::string::npos, r) == 0) return true;
-  return false;
-}
-
 }  // namespace
 
 int load_checkpoint(ModelBase *model, const char *directory, uint64_t *tensors_loaded) {
@@ -227,7 +205,6 @@ int load_checkpoint(ModelBase *model, const char *directory, uint64_t *tensors_l
   std::sort(files.begin(), files.end());  // loader.rs:128-130: a duplicated name always resolves the same way
   if (files.empty()) return set_error(ORION_ERR_MODEL, "missing file: %s/*.safetensors", directory);
 
-  const uint32_t num_layers = model->desc().num_layers;
   std::set<std::string> seen;
   uint64_t loaded = 0;
   for (const std::string &f : files) {
@@ -257,7 +234,7 @@ int load_checkpoint(ModelBase *model, const char *directory, uint64_t *tensors_l
     const uint64_t data_size = m.size - 8 - hlen;
     for (const TensorInfo &t : tensors) {
       if (!seen.insert(t.name).second) continue;  // an earlier file already provided it
-      if (!model_uses(t.name, num_layers)) continue;
+      if (!model->uses_tensor(t.name.c_str())) continue;
       int dtype;
       size_t es;
       if (t.dtype == "F32") { dtype = ORION_DTYPE_F32; es = 4; }

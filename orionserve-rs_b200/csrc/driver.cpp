@@ -138,8 +138,15 @@ void PrefixCache::remove(BlockHash hash, BlockId block) {  // prefix.rs:123-129
 
 // ---- KvCacheManager --------------------------------------------------------------------------
 
-KvCacheManager::KvCacheManager(size_t num_blocks, size_t block_size, bool prefix_caching_enabled)
-    : pool_(num_blocks, block_size), prefix_caching_enabled_(prefix_caching_enabled) {}
+KvCacheManager::KvCacheManager(size_t num_blocks, size_t block_size, bool prefix_caching_enabled, size_t num_state_slots)
+    : pool_(num_blocks, block_size), prefix_caching_enabled_(prefix_caching_enabled), num_state_slots_(num_state_slots) {
+  for (size_t i = 0; i < num_state_slots; ++i) free_slots_.push_back((uint32_t)i);
+}
+
+std::optional<uint32_t> KvCacheManager::state_slot(SequenceId seq) const {
+  auto it = slots_.find(seq);
+  return it == slots_.end() ? std::nullopt : std::optional<uint32_t>(it->second);
+}
 
 CacheStats KvCacheManager::stats() const {  // manager.rs:110-121
   return CacheStats{pool_.total_blocks(), pool_.num_used(),      pool_.num_free(),      pool_.block_size(),
@@ -161,6 +168,8 @@ int KvCacheManager::allocate(SequenceId seq, const TokenId *prompt, size_t n, Al
   const size_t bs = pool_.block_size();
   const size_t needed = BlockTable::blocks_required(n, bs);
   if (needed > pool_.num_free()) return cache_exhausted(needed, pool_.num_free());
+  if (!has_free_state_slot())
+    return set_error(ORION_ERR_CACHE_EXHAUSTED, "all %zu state slots are taken", num_state_slots_);
 
   BlockTable table;
   AllocationOutcome out;
@@ -199,6 +208,10 @@ int KvCacheManager::allocate(SequenceId seq, const TokenId *prompt, size_t n, Al
   }
   table.num_tokens = n;
   tables_.emplace(seq, std::move(table));
+  if (num_state_slots_ > 0) {
+    slots_.emplace(seq, free_slots_.front());
+    free_slots_.pop_front();
+  }
   if (outcome) *outcome = out;
   return ORION_OK;
 }
@@ -247,8 +260,22 @@ int KvCacheManager::append_token(SequenceId seq) {  // manager.rs:290-335
   return pool_.set_contents(table.blocks.back(), filled, std::nullopt);
 }
 
+int KvCacheManager::extend(SequenceId seq, size_t count) {
+  auto it = tables_.find(seq);
+  if (it == tables_.end()) return set_error(ORION_ERR_INTERNAL, "seq-%llu has no block table", (unsigned long long)seq);
+  const size_t need = BlockTable::blocks_required(it->second.num_tokens + count, pool_.block_size()), have = it->second.blocks.size();
+  if (need > have && need - have > pool_.num_free()) return cache_exhausted(need - have, pool_.num_free());
+  for (size_t i = 0; i < count; ++i) ORION_TRY(append_token(seq));
+  return ORION_OK;
+}
+
 void KvCacheManager::free(SequenceId seq) {  // manager.rs:341-359
   chain_tips_.erase(seq);
+  auto slot = slots_.find(seq);
+  if (slot != slots_.end()) {
+    free_slots_.push_back(slot->second);
+    slots_.erase(slot);
+  }
   auto it = tables_.find(seq);
   if (it == tables_.end()) return;
   BlockTable table = std::move(it->second);

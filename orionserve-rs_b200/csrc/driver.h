@@ -107,7 +107,9 @@ struct CacheStats {  // manager.rs:46-56
 
 class KvCacheManager {  // manager.rs:73-425
  public:
-  KvCacheManager(size_t num_blocks, size_t block_size, bool prefix_caching_enabled);
+  // `num_state_slots` (not in the reference): models that carry recurrent state keep it in one of this many
+  // slots per sequence, taken with the block table and given back with it. 0 = no slots are handed out.
+  KvCacheManager(size_t num_blocks, size_t block_size, bool prefix_caching_enabled, size_t num_state_slots = 0);
   size_t block_size() const { return pool_.block_size(); }
   size_t total_blocks() const { return pool_.total_blocks(); }
   size_t free_blocks() const { return pool_.num_free(); }
@@ -119,7 +121,12 @@ class KvCacheManager {  // manager.rs:73-425
   int allocate(SequenceId seq, const TokenId *prompt, size_t n, AllocationOutcome *outcome);
   void commit_prefill(SequenceId seq, const TokenId *prompt, size_t n);
   int append_token(SequenceId seq);
+  // append_token for `count` tokens at once, or for none of them (not in the reference).
+  int extend(SequenceId seq, size_t count);
   void free(SequenceId seq);
+  size_t num_state_slots() const { return num_state_slots_; }
+  bool has_free_state_slot() const { return num_state_slots_ == 0 || !free_slots_.empty(); }
+  std::optional<uint32_t> state_slot(SequenceId seq) const;
   size_t preempt(SequenceId seq);
   size_t evict_cached(size_t count);
   void clear_prefix_cache();
@@ -137,6 +144,9 @@ class KvCacheManager {  // manager.rs:73-425
   PrefixCache prefix_cache_;
   bool prefix_caching_enabled_;
   std::unordered_map<SequenceId, BlockHash> chain_tips_;
+  size_t num_state_slots_;
+  std::deque<uint32_t> free_slots_;  // oldest first
+  std::unordered_map<SequenceId, uint32_t> slots_;
   bool fail_next_append_ = false, fail_next_allocate_ = false;
 };
 
@@ -162,16 +172,21 @@ class Sequence {  // sequence.rs:158-330
   size_t output_len() const { return output_.size(); }
   size_t total_len() const { return prompt_.size() + output_.size(); }
   size_t computed_prefix_len() const { return computed_prefix_len_; }
-  size_t remaining_prefill() const { return prompt_.size() > computed_prefix_len_ ? prompt_.size() - computed_prefix_len_ : 0; }
-  bool is_prefill_complete() const { return computed_prefix_len_ >= prompt_.size(); }
+  // Tokens the prefill has to run: the prompt, or after a preemption with recomputation the tokens generated
+  // so far as well.
+  size_t prefill_len() const { return prompt_.size() + recompute_; }
+  std::vector<TokenId> prefill_tokens() const;
+  size_t remaining_prefill() const { return prefill_len() > computed_prefix_len_ ? prefill_len() - computed_prefix_len_ : 0; }
+  bool is_prefill_complete() const { return computed_prefix_len_ >= prefill_len(); }
   bool is_finished() const { return state_ == SequenceState::Finished; }
   FinishReason finish_reason() const { return finish_reason_; }
   std::chrono::steady_clock::time_point arrived_at() const { return arrived_at_; }
   bool transition_to(SequenceState next);
   void advance_prefill(size_t n);
+  void rewind_prefill(size_t position);  // a step that carried the prompt from here on did not run
   void push_token(TokenId t) { output_.push_back(t); }
   void finish(FinishReason reason);
-  bool preempt();
+  bool preempt(bool recompute_output = false);
   bool reached_max_tokens() const { return output_.size() >= params_.max_tokens; }
   bool may_stop_on_eos() const { return output_.size() >= params_.min_tokens; }
   static bool can_transition(SequenceState from, SequenceState to);
@@ -179,7 +194,7 @@ class Sequence {  // sequence.rs:158-330
  private:
   SequenceId id_;
   std::vector<TokenId> prompt_, output_;
-  size_t computed_prefix_len_ = 0;
+  size_t computed_prefix_len_ = 0, recompute_ = 0;
   SequenceState state_ = SequenceState::Waiting;
   FinishReason finish_reason_ = FinishReason::None;
   SamplingParams params_;
@@ -201,6 +216,11 @@ struct SchedulerConfig {  // crates/orion-core/src/config.rs:107-156
   // instead of total_len (scheduler.rs:283 counts the token that was just sampled), so no cache
   // slot is skipped and no step is refused for a block the table does not hold yet.
   bool logical_decode_positions = false;
+  // Not in the reference either: a preempted sequence that has generated tokens prefills them again after
+  // its prompt (the reference drops them from the cache and goes on behind them), so that what it carries
+  // is complete when it decodes on. Needed by models with recurrent state, which set it and
+  // logical_decode_positions themselves.
+  bool recompute_on_preempt = false;
 };
 
 struct ScheduledSequence {  // scheduler.rs:36-50
@@ -239,7 +259,8 @@ class Scheduler {  // scheduler.rs:127-580
   std::vector<SequenceId> expire_timeouts();
   const Sequence *running_sequence(SequenceId id) const;
   void commit_prefill(SequenceId id);
-  // Only with skip_cached_prefix: the forward of a step failed, so the prefill chunks it carried
+  // With recompute_on_preempt the prefill goes back to where the failed step found it. With
+  // skip_cached_prefix: the forward of a step failed, so the prefill chunks it carried
   // wrote no keys or values although their progress was recorded at schedule time. The prompts
   // of these sequences are not published to the prefix cache (a later request would adopt blocks
   // that were never written and skip their computation); they stay usable for their own sequence
@@ -270,6 +291,7 @@ struct HostBatch {
   std::vector<uint64_t> slot_token_counts, context_lens;
   std::vector<uint32_t> block_tables_flat;
   std::vector<uint64_t> block_table_offsets;  // [sequences + 1]
+  std::vector<uint32_t> state_slots;          // one per sequence if the cache manager hands out slots, else empty
   bool has_prefill = false;
   void clear();
 };

@@ -38,6 +38,7 @@ SchedulerConfig to_config(const OrionSchedulerConfig *c) {
   out.prioritize_decode = c->prioritize_decode != 0;
   out.skip_cached_prefix = c->skip_cached_prefix != 0;
   out.logical_decode_positions = c->logical_decode_positions != 0;
+  out.recompute_on_preempt = c->recompute_on_preempt != 0;
   return out;
 }
 
@@ -68,13 +69,17 @@ uint64_t orion_sequence_id_peek(void) { return peek_sequence_id(); }
 // ---- manager -----------------------------------------------------------------------------------
 
 OrionKvManager *orion_kv_manager_create(uint64_t num_blocks, uint64_t block_size, int prefix_caching_enabled) {
+  return orion_kv_manager_create_with_state(num_blocks, block_size, prefix_caching_enabled, 0);
+}
+OrionKvManager *orion_kv_manager_create_with_state(uint64_t num_blocks, uint64_t block_size, int prefix_caching_enabled,
+                                                   uint64_t num_state_slots) {
   clear_error();
   if (block_size == 0) {
     set_error(ORION_ERR_INVALID_REQUEST, "block_size must be non-zero");
     return nullptr;
   }
   auto *h = new OrionKvManager;
-  h->owned.reset(new KvCacheManager(num_blocks, block_size, prefix_caching_enabled != 0));
+  h->owned.reset(new KvCacheManager(num_blocks, block_size, prefix_caching_enabled != 0, num_state_slots));
   h->p = h->owned.get();
   return h;
 }
@@ -96,6 +101,15 @@ void orion_kv_manager_commit_prefill(OrionKvManager *m, uint64_t seq, const uint
 int orion_kv_manager_append_token(OrionKvManager *m, uint64_t seq) {
   clear_error();
   return m ? m->p->append_token(seq) : null_handle();
+}
+int orion_kv_manager_extend(OrionKvManager *m, uint64_t seq, uint64_t count) {
+  clear_error();
+  return m ? m->p->extend(seq, count) : null_handle();
+}
+int orion_kv_manager_state_slot(const OrionKvManager *m, uint64_t seq, uint32_t *slot) {
+  const auto s = m ? m->p->state_slot(seq) : std::nullopt;
+  if (s && slot) *slot = *s;
+  return s.has_value() ? 1 : 0;
 }
 void orion_kv_manager_free(OrionKvManager *m, uint64_t seq) {
   if (m) m->p->free(seq);
@@ -246,6 +260,17 @@ OrionEngine *orion_engine_create(OrionModel *model, OrionForwardFn forward, void
     return nullptr;
   }
   ForwardFn fn;
+  SchedulerConfig cfg = to_config(config);
+  size_t state_slots = 0;
+  if (model && (state_slots = model->impl->num_state_slots()) > 0) {
+    // State is carried from token to token: positions follow one another without a gap, and nothing of a
+    // sequence can be skipped because another one has cached it.
+    if (cfg.skip_cached_prefix) {
+      set_error(ORION_ERR_INVALID_REQUEST, "skip_cached_prefix: a model with recurrent state computes every token of a sequence");
+      return nullptr;
+    }
+    cfg.logical_decode_positions = cfg.recompute_on_preempt = true;
+  }
   if (model) {
     ModelBase *impl = model->impl.get();
     fn = [impl](const HostBatch &b, uint32_t *token_ids) -> int {
@@ -263,6 +288,7 @@ OrionEngine *orion_engine_create(OrionModel *model, OrionForwardFn forward, void
       v.num_block_tables = b.sequence_ids.size();
       v.num_sequences = b.sequence_ids.size();
       v.has_prefill = b.has_prefill ? 1 : 0;
+      if (!b.state_slots.empty()) v.state_slots = b.state_slots.data(), v.num_state_slots = b.state_slots.size();
       return impl->forward(v, nullptr, 0, token_ids);
     };
   } else {
@@ -273,7 +299,7 @@ OrionEngine *orion_engine_create(OrionModel *model, OrionForwardFn forward, void
     };
   }
   auto *h = new OrionEngine;
-  h->impl.reset(new Engine(Scheduler(to_config(config), KvCacheManager(num_blocks, block_size, prefix_caching_enabled != 0)),
+  h->impl.reset(new Engine(Scheduler(cfg, KvCacheManager(num_blocks, block_size, prefix_caching_enabled != 0, state_slots)),
                            std::move(fn), std::vector<TokenId>(eos_ids, eos_ids + (eos_ids ? num_eos : 0))));
   h->sched.p = &h->impl->scheduler();
   h->sched.cache.p = &h->sched.p->cache();

@@ -48,7 +48,19 @@ bool Sequence::transition_to(SequenceState next) {  // sequence.rs:255-264
 }
 
 void Sequence::advance_prefill(size_t n) {  // sequence.rs:270-272
-  computed_prefix_len_ = std::min(computed_prefix_len_ + n, prompt_.size());
+  computed_prefix_len_ = std::min(computed_prefix_len_ + n, prefill_len());
+}
+
+void Sequence::rewind_prefill(size_t position) {
+  if (state_ == SequenceState::Finished) return;
+  computed_prefix_len_ = std::min(computed_prefix_len_, position);
+  state_ = SequenceState::Prefilling;
+}
+
+std::vector<TokenId> Sequence::prefill_tokens() const {
+  std::vector<TokenId> t(prompt_);
+  t.insert(t.end(), output_.begin(), output_.begin() + (ptrdiff_t)recompute_);
+  return t;
 }
 
 void Sequence::finish(FinishReason reason) {  // sequence.rs:286-293: the first reason wins
@@ -57,10 +69,11 @@ void Sequence::finish(FinishReason reason) {  // sequence.rs:286-293: the first 
   finish_reason_ = reason;
 }
 
-bool Sequence::preempt() {  // sequence.rs:303-310: prefill progress is dropped, generated tokens are kept
+bool Sequence::preempt(bool recompute_output) {  // sequence.rs:303-310: prefill progress is dropped, generated tokens are kept
   if (!can_transition(state_, SequenceState::Waiting)) return false;
   state_ = SequenceState::Waiting;
   computed_prefix_len_ = 0;
+  recompute_ = recompute_output ? output_.size() : 0;
   return true;
 }
 
@@ -177,9 +190,12 @@ bool Scheduler::preempt_one(SchedulerOutput &out) {  // scheduler.rs:317-330
   running_.pop_back();
   const SequenceId id = victim.id();
   cache_.free(id);
-  victim.preempt();
+  victim.preempt(config_.recompute_on_preempt);
   unwritten_prefill_.erase(id);  // its prefill starts over, every chunk will be computed again
   waiting_.push_front(std::move(victim));
+  if (config_.recompute_on_preempt)  // it starts over; what this step had already planned for it does not run
+    out.scheduled.erase(std::remove_if(out.scheduled.begin(), out.scheduled.end(), [&](const ScheduledSequence &s) { return s.id == id; }),
+                        out.scheduled.end());
   out.preempted.push_back(id);
   stats_.total_preempted += 1;
   return true;
@@ -214,7 +230,7 @@ void Scheduler::schedule_prefills(SchedulerOutput &out, size_t budget, size_t &u
     if (running_.size() >= config_.max_num_seqs || used >= budget) break;
     if (waiting_.empty()) break;
     const Sequence &next = waiting_.front();
-    const size_t prompt_len = next.prompt_len();
+    const size_t prompt_len = next.prefill_len();
     const size_t already = next.computed_prefix_len();
     const size_t remaining = prompt_len - already;
     const size_t room = budget - used;
@@ -225,6 +241,7 @@ void Scheduler::schedule_prefills(SchedulerOutput &out, size_t budget, size_t &u
     if (chunk == 0) break;
 
     const bool is_first_chunk = already == 0;  // only the first chunk allocates
+    if (is_first_chunk && !cache_.has_free_state_slot()) break;  // a slot comes free when a sequence ends
     if (is_first_chunk && !cache_.can_allocate(prompt_len)) {
       if (!preempt_one(out)) break;
       continue;
@@ -235,8 +252,9 @@ void Scheduler::schedule_prefills(SchedulerOutput &out, size_t budget, size_t &u
     size_t start_position = already;
     if (is_first_chunk) {
       AllocationOutcome outcome;
-      if (cache_.allocate(id, seq.prompt().data(), seq.prompt().size(), &outcome) != ORION_OK) {
-        seq.preempt();
+      const std::vector<TokenId> tokens = seq.prefill_tokens();
+      if (cache_.allocate(id, tokens.data(), tokens.size(), &outcome) != ORION_OK) {
+        seq.preempt(config_.recompute_on_preempt);
         waiting_.push_front(std::move(seq));
         break;
       }
@@ -320,6 +338,9 @@ void Scheduler::commit_prefill(SequenceId id) {  // scheduler.rs:557-564
 }
 
 void Scheduler::note_failed_step(const SchedulerOutput &out) {
+  if (config_.recompute_on_preempt)  // what the step was to prefill is prefilled by the next one
+    for (const ScheduledSequence &s : out.scheduled)
+      if (Sequence *seq = s.is_prefill ? running_mut(s.id) : nullptr) seq->rewind_prefill(s.start_position);
   if (!config_.skip_cached_prefix) return;
   for (const ScheduledSequence &s : out.scheduled)
     if (s.is_prefill) unwritten_prefill_.insert(s.id);
@@ -335,6 +356,7 @@ void HostBatch::clear() {
   context_lens.clear();
   block_tables_flat.clear();
   block_table_offsets.assign(1, 0);
+  state_slots.clear();
   has_prefill = false;
 }
 
@@ -446,8 +468,10 @@ int Engine::build_batch(const SchedulerOutput &output) {  // engine.rs:429-487
     size_t count = 0;
     if (sched.is_prefill) {  // the prompt slice this chunk covers
       const size_t start = sched.start_position;
-      const size_t end = std::min(start + sched.num_tokens, seq->prompt_len());
-      for (size_t i = start; i < end; ++i) batch_.tokens.push_back(seq->prompt()[i]);
+      const size_t end = std::min(start + sched.num_tokens, seq->prefill_len());
+      const size_t prompt_len = seq->prompt_len();
+      for (size_t i = start; i < end; ++i)
+        batch_.tokens.push_back(i < prompt_len ? seq->prompt()[i] : seq->output()[i - prompt_len]);
       count = end > start ? end - start : 0;
     } else if (!seq->output().empty()) {  // decode: the most recent token
       batch_.tokens.push_back(seq->output().back());
@@ -463,6 +487,7 @@ int Engine::build_batch(const SchedulerOutput &output) {  // engine.rs:429-487
     batch_.context_lens.push_back(sched.start_position + count);
     batch_.block_tables_flat.insert(batch_.block_tables_flat.end(), table->blocks.begin(), table->blocks.end());
     batch_.block_table_offsets.push_back(batch_.block_tables_flat.size());
+    if (const auto slot = scheduler_.cache().state_slot(sched.id)) batch_.state_slots.push_back(*slot);
     batch_.has_prefill = batch_.has_prefill || sched.is_prefill;
   }
   return ORION_OK;

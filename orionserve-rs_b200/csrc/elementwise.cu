@@ -635,6 +635,34 @@ int launch_swiglu(const float *partial, uint32_t splits, size_t split_stride, T 
   return after_launch("swiglu");
 }
 
+template <typename T>
+__device__ __forceinline__ float gelu_f(float x) {  // the tanh form
+  return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+gelu_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, T *__restrict__ out, uint32_t ldo, uint32_t rows,
+            uint32_t cols) {
+  pdl_trigger();
+  pdl_wait();
+  const size_t total = (size_t)rows * cols;
+  for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
+    float v = partial[idx];
+    for (uint32_t s = 1; s < splits; ++s) v += partial[s * split_stride + idx];
+    out[(idx / cols) * ldo + idx % cols] = from_f32<T>(gelu_f<T>(v));
+  }
+}
+
+template <typename T>
+int launch_gelu(const float *partial, uint32_t splits, size_t split_stride, T *out, uint32_t ldo, uint32_t rows, uint32_t cols,
+                cudaStream_t stream) {
+  if (rows == 0 || cols == 0) return ORION_OK;
+  ORION_CUDA_CHECK("gelu", launch_pdl(gelu_kernel<T>, dim3(grid_for((size_t)rows * cols, 256)), dim3(256), 0, stream, partial, splits,
+                                      split_stride, out, ldo, rows, cols));
+  return after_launch("gelu");
+}
+
 // dst[r * dst_stride + c] = src[r * cols + c]: spreads the rows of a contiguous matrix over a
 // strided destination (the gate and up projections are stored row-interleaved).
 template <typename T>
@@ -758,6 +786,7 @@ int launch_fill_normal(T *dst, size_t n, uint64_t seed, cudaStream_t stream) {
   template int launch_copy_rows_strided<T>(const T *, T *, size_t, size_t, size_t, cudaStream_t);   \
   template int launch_swiglu<T>(const float *, uint32_t, size_t, T *, uint32_t, uint32_t,         \
                                 cudaStream_t, bool);                                              \
+  template int launch_gelu<T>(const float *, uint32_t, size_t, T *, uint32_t, uint32_t, uint32_t, cudaStream_t); \
   template int launch_convert_from_f32<T>(const float *, T *, size_t, cudaStream_t);              \
   template int launch_convert_to_f32<T>(const T *, float *, size_t, cudaStream_t);                \
   template int launch_arena_to_reference_order<T>(const T *, KvLayout, float *, cudaStream_t);    \

@@ -81,6 +81,11 @@ int launch_swiglu(const float *partial, uint32_t splits, size_t split_stride, T 
 template <typename T>
 int launch_copy_rows_strided(const T *src, T *dst, size_t rows, size_t cols, size_t dst_stride, cudaStream_t stream);
 
+// out[r * ldo + c] = gelu(sum_s partial[s][r][c]), the tanh form.
+template <typename T>
+int launch_gelu(const float *partial, uint32_t splits, size_t split_stride, T *out, uint32_t ldo, uint32_t rows, uint32_t cols,
+                cudaStream_t stream);
+
 // out[r][n] = sum_s partial[s][r][n] + bias[n]  (finishes tensor::linear, tensor.rs:126).
 int launch_finish_linear(const float *partial, uint32_t splits, size_t split_stride,
                          const float *bias, float *out, uint32_t rows, uint32_t n,
@@ -211,6 +216,72 @@ int launch_paged_attention_decode(const bf16 *q, const bf16 *arena, KvLayout kv,
 void decode_set_tuning(int stages, uint32_t cta_target);
 // Device error word of the decode kernel (0 = none); reading clears it.
 int decode_poll_error(uint32_t *code);
+
+// ---- state carried from token to token -----------------------------------------------
+//
+// Models with recurrent layers keep, besides the paged cache, a fixed amount of state per sequence. A
+// state buffer holds two copies of every slot: a step reads the copy `read` of each of its sequences
+// and writes the copy `write`, so no thread can meet a value of this step where it expects the previous
+// one, and a step that is run again (a replay, a retry after an error) finds its inputs unchanged.
+struct StateBatch {
+  const uint32_t *first_row;  // [sequences + 1] batch rows of each sequence: [first_row[s], first_row[s + 1])
+  const uint32_t *read;       // [sequences] copy to read; kNoState: the sequence starts here, all zeros
+  const uint32_t *write;      // [sequences] copy to write
+  const uint32_t *seq_of_row; // [rows]
+  uint32_t rows, seqs;
+  bool single;                // every sequence has exactly one row
+};
+constexpr uint32_t kNoState = 0xFFFFFFFFu;
+
+// Causal per-channel convolution over time added to its input, for up to two sets of weights at once
+// (the two sublayers of a parallel layer): out_i = h + conv_i(h), conv_i(h)_t = sum_j w_i[c][j] h_(t - taps + 1 + j).
+// `state` is [copies][taps - 1][cols]: the last taps - 1 rows of h. w2 / out2 may be null.
+template <typename T>
+int launch_causal_conv(const T *h, const T *w1, const T *w2, uint32_t taps, T *state, StateBatch sb, T *out1, T *out2,
+                       uint32_t cols, cudaStream_t stream);
+// One row per sequence: residual add (as launch_residual_rmsnorm) or, with `tokens`, the embedding lookup,
+// then the norm and the convolutions, in one kernel.
+template <typename T>
+int launch_residual_norm_conv(const float *partial, uint32_t splits, size_t split_stride, const T *embed, const uint32_t *tokens,
+                              float *hidden, const float *norm_w, float eps, const T *w1, const T *w2, uint32_t taps, T *state,
+                              StateBatch sb, T *out1, T *out2, uint32_t cols, cudaStream_t stream);
+bool residual_norm_conv_supported(uint32_t cols, uint32_t taps);
+
+// Minimal gated recurrence, element by element: with the projections' partial sums [z | x | g] of `width`
+// columns each, z' = sigmoid(z + bias_z), u = x + bias_x, c = u >= 0 ? u + 1/2 : sigmoid(u),
+// S_t = (1 - z') S_(t-1) + z' c, out = S_t * silu(g). `state` is [copies][width] in f32.
+template <typename T>
+int launch_min_gru(const float *partial, uint32_t splits, size_t split_stride, const float *bias, float *state, StateBatch sb,
+                   T *out, uint32_t ldo, uint32_t width, cudaStream_t stream);
+
+// ---- latent attention ---------------------------------------------------------------------
+//
+// The cache of one layer holds, per token, the normalised latent (kv_rank values) followed by the rotated key
+// part that all heads share (rot_dim values): [block][slot][row_stride], row_stride a multiple of 8.
+struct LatentShape {
+  uint32_t heads, dim, rot_dim, value_dim, kv_rank, window, rope_dims, block_size, row_stride;
+  float scale, eps;
+  __host__ __device__ uint32_t q_dim() const { return dim + rot_dim; }
+  // Columns of the joint projection: queries, latent + shared key part, output gate.
+  __host__ __device__ uint32_t q_cols() const { return heads * (dim + rot_dim); }
+  __host__ __device__ uint32_t kv_cols() const { return kv_rank + rot_dim; }
+  __host__ __device__ uint32_t out_cols() const { return heads * value_dim; }
+  __host__ __device__ uint32_t cols() const { return q_cols() + kv_cols() + out_cols(); }
+  // First position that a query at `pos` sees.
+  __host__ __device__ uint32_t first_key(uint32_t pos) const { return window && pos + 1 > window ? pos + 1 - window : 0; }
+};
+// Folds the joint projection's partial sums: queries (rotated) to q [rows][heads][dim + rot_dim], the normalised
+// latent and the rotated shared key part to the cache row of the token.
+template <typename T>
+int launch_latent_prepare(const float *partial, uint32_t splits, size_t split_stride, const float *norm_w, const float *rope_cos,
+                          const float *rope_sin, const uint32_t *positions, const uint32_t *slot_block, const uint32_t *slot_slot,
+                          T *q, T *cache, LatentShape ls, uint32_t rows, cudaStream_t stream);
+// Any shape, any mix of rows: one CTA per (row, head). The query is taken into the latent space (w_uk), the
+// weighted latent back out of it (w_uv), and the result is gated: out[r * ldo + h * value_dim + v].
+template <typename T>
+int launch_latent_attention_generic(const T *q, const T *cache, const T *w_uk, const T *w_uv, const float *gate_partial,
+                                    uint32_t splits, size_t split_stride, LatentShape ls, AttnBatch batch, T *out, uint32_t ldo,
+                                    cudaStream_t stream);
 
 // ---- tensor-parallel hand-over ---------------------------------------------------
 

@@ -33,6 +33,12 @@ struct BatchView {
   uint64_t num_block_tables;
   uint64_t num_sequences;
   int has_prefill;
+  // Rows whose logits are wanted, in this order (null: the last row of every sequence).
+  const uint32_t *logit_rows;
+  uint64_t num_logit_rows;
+  // State slot of every sequence, for models that carry state from token to token (null for the others).
+  const uint32_t *state_slots;
+  uint64_t num_state_slots;
 };
 
 // Shard {start, len} (orion-distributed/src/lib.rs:116-130).
@@ -54,6 +60,10 @@ class ModelBase {
   virtual ~ModelBase() = default;
   virtual int load_tensor(const char *name, int dtype, const uint64_t *shape, int ndim,
                           const void *data) = 0;
+  // Whether the model has a place for a checkpoint tensor of this name; the others are skipped.
+  virtual bool uses_tensor(const char *name) const = 0;
+  // State slots the model was made with (0: nothing but the KV cache is carried from step to step).
+  virtual uint32_t num_state_slots() const { return 0; }
   virtual int init_random(uint64_t seed, float std) = 0;
   virtual int finalize() = 0;
   virtual int forward(const BatchView &b, float *logits_out, uint64_t logits_capacity,
@@ -69,6 +79,7 @@ class ModelBase {
 
 
 int create_model(OrionBackend *backend, const OrionModelDesc *desc, ModelBase **out);
+int create_layered_model(OrionBackend *backend, const OrionLayeredDesc *desc, ModelBase **out);
 // Loads every tensor the model uses from the `*.safetensors` files of a directory and finalizes
 // (CheckpointLoader, crates/orion-models/src/loader.rs:112-235).
 int load_checkpoint(ModelBase *model, const char *directory, uint64_t *tensors_loaded);

@@ -67,12 +67,16 @@ class SchedulerConfig:
     #: not in the reference: decode tokens at position total_len - 1 (their logical place) instead of
     #: total_len, so no cache slot is skipped and no step is refused
     logical_decode_positions: bool = False
+    #: not in the reference: a preempted sequence prefills its generated tokens again after its prompt.
+    #: An engine around a model with state slots turns this and logical_decode_positions on by itself.
+    recompute_on_preempt: bool = False
 
     def _c(self):
         return _ffi.OrionSchedulerConfig(self.max_num_seqs, self.max_num_batched_tokens, self.max_model_len or 0,
                                          int(self.enable_chunked_prefill), self.max_waiting_requests,
                                          self.request_timeout_secs or 0, int(self.prioritize_decode),
-                                         int(self.skip_cached_prefix), int(self.logical_decode_positions))
+                                         int(self.skip_cached_prefix), int(self.logical_decode_positions),
+                                         int(self.recompute_on_preempt))
 
 
 @dataclass(frozen=True)
@@ -146,14 +150,17 @@ def next_sequence_id() -> int:
 
 
 class KvCacheManager:
-    """``KvCacheManager`` (crates/orion-kv-cache/src/manager.rs:73-425)."""
+    """``KvCacheManager`` (crates/orion-kv-cache/src/manager.rs:73-425). With ``num_state_slots`` it also hands
+    out the state slots of models that carry recurrent state: one per sequence, from ``allocate`` to ``free``."""
 
-    def __init__(self, num_blocks: int, block_size: int, prefix_caching_enabled: bool, *, _borrowed=None, _keep=None):
+    def __init__(self, num_blocks: int, block_size: int, prefix_caching_enabled: bool, *, num_state_slots: int = 0,
+                 _borrowed=None, _keep=None):
         # A borrowed view keeps its owner alive (`_keep`); owners never point back at their views,
         # so there is no reference cycle and handles are destroyed in dependency order.
         self._keep = _keep
         self._owned = _borrowed is None
-        self._h = _borrowed or _ffi.lib().orion_kv_manager_create(num_blocks, block_size, int(prefix_caching_enabled))
+        self._h = _borrowed or _ffi.lib().orion_kv_manager_create_with_state(num_blocks, block_size,
+                                                                             int(prefix_caching_enabled), num_state_slots)
         if not self._h:
             raise EngineError(_ffi.last_error())
 
@@ -174,6 +181,14 @@ class KvCacheManager:
 
     def append_token(self, seq: int) -> None:
         check(_ffi.lib().orion_kv_manager_append_token(self._h, seq))
+
+    def extend(self, seq: int, count: int) -> None:
+        """``append_token`` for ``count`` tokens, all of them or none."""
+        check(_ffi.lib().orion_kv_manager_extend(self._h, seq, count))
+
+    def state_slot(self, seq: int) -> Optional[int]:
+        slot = C.c_uint32()
+        return int(slot.value) if _ffi.lib().orion_kv_manager_state_slot(self._h, seq, C.byref(slot)) else None
 
     def free(self, seq: int) -> None:
         _ffi.lib().orion_kv_manager_free(self._h, seq)

@@ -171,52 +171,16 @@ class HfConfig:
             has_qkv_bias=(arch == "qwen2"), tied_lm_head=self.ties_embeddings())
 
 
-class CudaTransformerModel:
-    """A GPU-executing decoder-only transformer with the reference's constructor convention."""
+class CudaModel:
+    """What every device model offers once it exists: weights in, batches forward. ``_h`` is the library's
+    handle, ``_meta`` the model's metadata (``vocab_size`` and ``name`` at least)."""
 
-    def __init__(self, meta: ModelMetadata, num_blocks: int, block_size: int, backend: CudaBackend, *,
-                 compute_dtype: DType = DType.BF16, max_batch_tokens: int = 8192,
-                 max_batch_sequences: int = 256, tp_rank: int = 0, tp_world: int = 1,
-                 nccl_unique_id: Optional[bytes] = None):
-        """``TransformerModel::new`` minus the weights, which arrive through ``load_tensor`` /
-        ``load_state`` (transformer.rs:148-177)."""
-        self._meta, self._backend, self._h = meta, backend, C.c_void_p()
-        d = _ffi.OrionModelDesc(
-            meta.hidden_size, meta.num_layers, meta.num_attention_heads, meta.num_kv_heads, meta.head_dim,
-            meta.vocab_size, meta.ffn_dim or 4 * meta.hidden_size, meta.max_position_embeddings,
-            meta.rope_theta, meta.rms_norm_eps, int(meta.has_qkv_bias), int(meta.tied_lm_head),
-            num_blocks, block_size, int(compute_dtype), max_batch_tokens, max_batch_sequences, tp_rank,
-            tp_world)
-        if nccl_unique_id is not None:
-            C.memmove(d.nccl_unique_id, nccl_unique_id, _ffi.NCCL_ID_BYTES)
-        self.compute_dtype, self.num_blocks, self.block_size = compute_dtype, num_blocks, block_size
-        self.tp_rank, self.tp_world = tp_rank, tp_world
-        check(_ffi.lib().orion_cuda_model_create(backend._h, C.byref(d), C.byref(self._h)))
+    _h = None
 
     def __del__(self):
         if getattr(self, "_h", None):
             _ffi.lib().orion_cuda_model_destroy(self._h)
             self._h = None
-
-    # ---- construction -------------------------------------------------------
-    @classmethod
-    def new(cls, meta: ModelMetadata, weights: Dict[str, np.ndarray], num_blocks: int, block_size: int,
-            backend: CudaBackend, **kw) -> "CudaTransformerModel":
-        m = cls(meta, num_blocks, block_size, backend, **kw)
-        m.load_state(weights)
-        return m
-
-    @classmethod
-    def from_directory(cls, directory: str, num_blocks: int, block_size: int, backend: CudaBackend,
-                       **kw) -> "CudaTransformerModel":
-        """transformer.rs:180-205: config.json + one or more safetensors shards."""
-        cfg = HfConfig.load(directory)
-        meta = cfg.to_metadata(os.path.basename(os.path.normpath(directory)) or "model")
-        if cfg.ties_embeddings():  # transformer.rs:108-112; an absent lm_head falls back to the embedding too
-            meta.tied_lm_head = True
-        m = cls(meta, num_blocks, block_size, backend, **kw)
-        m.load_checkpoint(directory)
-        return m
 
     def load_checkpoint(self, directory: str) -> int:
         """Every ``*.safetensors`` file of ``directory`` straight from its memory mapping to the
@@ -267,6 +231,8 @@ class CudaTransformerModel:
     def forward(self, batch: ForwardBatch, out: Optional[np.ndarray] = None) -> ForwardOutput:
         """``LanguageModel::forward`` (traits.rs:305). ``out`` may be a preallocated (for instance
         page-locked) float32 buffer of at least ``num_sequences * vocab_size`` elements."""
+        if batch.logit_rows is not None or batch.state_slots is not None:
+            return self._forward_rows(batch, out)
         args, keep = self._batch_args(batch)
         n = len(batch.sequence_ids) * self._meta.vocab_size
         if out is None:
@@ -276,14 +242,46 @@ class CudaTransformerModel:
         logits = out.reshape(-1)[:rows * self._meta.vocab_size].reshape(rows, self._meta.vocab_size)
         return ForwardOutput(logits, self._meta.vocab_size, list(batch.sequence_ids) if rows else [])
 
+    def _rows_args(self, batch: ForwardBatch):
+        """The trailing arguments of ``orion_cuda_model_forward_rows`` and the number of logit rows."""
+        P = lambda a: a.ctypes.data_as(C.POINTER(C.c_uint32))
+        slots = None if batch.state_slots is None else np.ascontiguousarray(batch.state_slots, np.uint32)
+        rows = None if batch.logit_rows is None else np.append(np.asarray(batch.logit_rows, np.uint32), np.uint32(0))
+        n = len(batch.sequence_ids) if rows is None else rows.size - 1
+        args = [None if slots is None else P(slots), 0 if slots is None else slots.size,
+                None if rows is None else P(rows), 0 if rows is None else n]
+        return args, (slots, rows), n
+
+    def _forward_rows(self, batch: ForwardBatch, out: Optional[np.ndarray]) -> ForwardOutput:
+        args, keep = self._batch_args(batch)
+        extra, keep2, n = self._rows_args(batch)
+        V = self._meta.vocab_size
+        if out is None:
+            out = np.empty(max(n * V, 1), np.float32)
+        check(_ffi.lib().orion_cuda_model_forward_rows(self._h, *args, *extra, None, out.ctypes.data_as(C.c_void_p), out.size))
+        rows = 0 if batch.is_empty() else n
+        if batch.logit_rows is None:
+            ids = list(batch.sequence_ids)
+        else:
+            seq_of_row = np.repeat(np.arange(len(batch.sequence_ids)), np.asarray(batch.slot_token_counts, np.int64))
+            ids = [batch.sequence_ids[seq_of_row[r]] for r in batch.logit_rows]
+        return ForwardOutput(out.reshape(-1)[:rows * V].reshape(rows, V), V, ids if rows else [])
+
+    def num_state_slots(self) -> int:
+        n = C.c_uint32()
+        check(_ffi.lib().orion_cuda_model_num_state_slots(self._h, C.byref(n)))
+        return int(n.value)
+
     def forward_greedy(self, batch: ForwardBatch, want_logits: bool = False):
         """forward + device-side greedy argmax; returns (token ids, logits or None)."""
         args, keep = self._batch_args(batch)
         S = len(batch.sequence_ids)
         ids = np.zeros(max(S, 1), np.uint32)
         logits = np.empty(max(S * self._meta.vocab_size, 1), np.float32) if want_logits else None
-        check(_ffi.lib().orion_cuda_model_forward_greedy(
-            self._h, *args, ids.ctypes.data_as(C.POINTER(C.c_uint32)),
+        extra, keep2, _ = self._rows_args(batch)
+        extra[2:] = [None, 0]  # one token per sequence
+        check(_ffi.lib().orion_cuda_model_forward_rows(
+            self._h, *args, *extra, ids.ctypes.data_as(C.POINTER(C.c_uint32)),
             logits.ctypes.data_as(C.c_void_p) if want_logits else None,
             logits.size if want_logits else 0))
         return ids[:S], (logits[:S * self._meta.vocab_size].reshape(S, -1) if want_logits else None)
@@ -321,6 +319,49 @@ class CudaTransformerModel:
         v = C.c_uint64()
         check(_ffi.lib().orion_cuda_model_last_launch_count(self._h, C.byref(v)))
         return v.value
+
+
+class CudaTransformerModel(CudaModel):
+    """A GPU-executing decoder-only transformer with the reference's constructor convention."""
+
+    def __init__(self, meta: ModelMetadata, num_blocks: int, block_size: int, backend: CudaBackend, *,
+                 compute_dtype: DType = DType.BF16, max_batch_tokens: int = 8192,
+                 max_batch_sequences: int = 256, tp_rank: int = 0, tp_world: int = 1,
+                 nccl_unique_id: Optional[bytes] = None):
+        """``TransformerModel::new`` minus the weights, which arrive through ``load_tensor`` /
+        ``load_state`` (transformer.rs:148-177)."""
+        self._meta, self._backend, self._h = meta, backend, C.c_void_p()
+        d = _ffi.OrionModelDesc(
+            meta.hidden_size, meta.num_layers, meta.num_attention_heads, meta.num_kv_heads, meta.head_dim,
+            meta.vocab_size, meta.ffn_dim or 4 * meta.hidden_size, meta.max_position_embeddings,
+            meta.rope_theta, meta.rms_norm_eps, int(meta.has_qkv_bias), int(meta.tied_lm_head),
+            num_blocks, block_size, int(compute_dtype), max_batch_tokens, max_batch_sequences, tp_rank,
+            tp_world)
+        if nccl_unique_id is not None:
+            C.memmove(d.nccl_unique_id, nccl_unique_id, _ffi.NCCL_ID_BYTES)
+        self.compute_dtype, self.num_blocks, self.block_size = compute_dtype, num_blocks, block_size
+        self.tp_rank, self.tp_world = tp_rank, tp_world
+        check(_ffi.lib().orion_cuda_model_create(backend._h, C.byref(d), C.byref(self._h)))
+
+    # ---- construction -------------------------------------------------------
+    @classmethod
+    def new(cls, meta: ModelMetadata, weights: Dict[str, np.ndarray], num_blocks: int, block_size: int,
+            backend: CudaBackend, **kw) -> "CudaTransformerModel":
+        m = cls(meta, num_blocks, block_size, backend, **kw)
+        m.load_state(weights)
+        return m
+
+    @classmethod
+    def from_directory(cls, directory: str, num_blocks: int, block_size: int, backend: CudaBackend,
+                       **kw) -> "CudaTransformerModel":
+        """transformer.rs:180-205: config.json + one or more safetensors shards."""
+        cfg = HfConfig.load(directory)
+        meta = cfg.to_metadata(os.path.basename(os.path.normpath(directory)) or "model")
+        if cfg.ties_embeddings():  # transformer.rs:108-112; an absent lm_head falls back to the embedding too
+            meta.tied_lm_head = True
+        m = cls(meta, num_blocks, block_size, backend, **kw)
+        m.load_checkpoint(directory)
+        return m
 
     def read_kv(self) -> np.ndarray:
         """This rank's arena as ``[layer][block][k|v][slot][local kv head][dim]`` f32."""

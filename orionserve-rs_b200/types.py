@@ -86,6 +86,10 @@ class ForwardBatch:
     context_lens: Sequence[int]
     block_tables: Sequence[Sequence[int]]
     has_prefill: bool = True
+    #: state slot of every sequence (models that carry recurrent state; the others take None)
+    state_slots: Optional[Sequence[int]] = None
+    #: batch rows whose logits are wanted, in this order; None: the last row of every sequence
+    logit_rows: Optional[Sequence[int]] = None
 
     def num_sequences(self) -> int:
         return len(self.sequence_ids)
@@ -135,7 +139,8 @@ class ForwardBatch:
 
 @dataclass
 class ForwardOutput:
-    """traits.rs:271-290: row-major ``[num_sequences, vocab_size]`` last-position logits."""
+    """traits.rs:271-290: row-major ``[num_sequences, vocab_size]`` last-position logits (or one row per
+    entry of the batch's ``logit_rows``; ``sequence_ids`` then names each row's sequence)."""
     logits: np.ndarray
     vocab_size: int
     sequence_ids: Sequence[int]
