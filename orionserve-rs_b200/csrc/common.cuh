@@ -116,6 +116,16 @@ __device__ __forceinline__ float from_f32<float>(float v) { return v; }
 template <>
 __device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __float2bfloat16_rn(v); }
 
+// GELU in its tanh form.
+__device__ __forceinline__ float gelu_tanh(float x) {
+  return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
+}
+// 1 / (1 + e^-x) without overflow on either side.
+__device__ __forceinline__ float sigmoid_f(float x) {
+  const float e = expf(-fabsf(x));
+  return (x >= 0.f ? 1.f : e) / (1.f + e);
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

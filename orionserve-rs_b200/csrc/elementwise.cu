@@ -636,11 +636,6 @@ int launch_swiglu(const float *partial, uint32_t splits, size_t split_stride, T 
 }
 
 template <typename T>
-__device__ __forceinline__ float gelu_f(float x) {  // the tanh form
-  return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
-}
-
-template <typename T>
 __global__ void __launch_bounds__(256)
 gelu_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, T *__restrict__ out, uint32_t ldo, uint32_t rows,
             uint32_t cols) {
@@ -650,7 +645,7 @@ gelu_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_str
   for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
     float v = partial[idx];
     for (uint32_t s = 1; s < splits; ++s) v += partial[s * split_stride + idx];
-    out[(idx / cols) * ldo + idx % cols] = from_f32<T>(gelu_f<T>(v));
+    out[(idx / cols) * ldo + idx % cols] = from_f32<T>(gelu_tanh(v));
   }
 }
 

@@ -208,7 +208,7 @@ template <int TOKN, int WST, int XST, int MT, bool PAIR = false>
 __global__ void __launch_bounds__(kThreads)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                float *__restrict__ partial, bf16 *__restrict__ act, uint32_t M, uint32_t N, uint32_t K,
-               uint32_t splits, uint32_t cluster_reduce, uint32_t ldc, ReadyWait ready) {
+               uint32_t splits, uint32_t cluster_reduce, uint32_t ldc, uint32_t epilogue, ReadyWait ready) {
   using Cfg = TcConfig<TOKN, WST, XST, MT, PAIR>;
   extern __shared__ uint8_t raw_smem[];
   uint8_t *smem = reinterpret_cast<uint8_t *>((reinterpret_cast<uintptr_t>(raw_smem) + 1023) &
@@ -408,6 +408,15 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
       if (cluster_reduce) {
 #pragma unroll
         for (int j = 0; j < 16; ++j) stage[(c + j) * kTileN + lq * 32 + lane] = __uint_as_float(r[j]);
+      } else if (epilogue == kGemmGelu || epilogue == kGemmStore) {  // activations in bf16, row stride ldc
+        if (n < N) {
+#pragma unroll
+          for (int j = 0; j < 16; ++j) {
+            const uint32_t tok = t0 + c + j;
+            const float v = __uint_as_float(r[j]);
+            if (tok < M) act[(size_t)tok * ldc + n] = __float2bfloat16_rn(epilogue == kGemmGelu ? gelu_tanh(v) : v);
+          }
+        }
       } else if (act != nullptr) {
         // Fused SwiGLU (tensor.rs:167-189): weight rows are interleaved, lane 2i holds gate_f and
         // lane 2i + 1 holds up_f of the same f for these 16 tokens. Each lane of a pair trades
@@ -541,11 +550,11 @@ int cached_map(const void *base, uint64_t rows, uint64_t k, uint64_t ld, uint32_
 
 template <int TOKN, int WST, int XST, int MT = 1, bool PAIR = false>
 int launch_tc(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, float *partial, bf16 *act,
-              uint32_t rows, uint32_t n, uint32_t k, uint32_t splits, bool cluster_reduce, uint32_t ldc,
+              uint32_t rows, uint32_t n, uint32_t k, uint32_t splits, bool cluster_reduce, uint32_t ldc, GemmEpilogue epi,
               cudaStream_t stream, ReadyWait ready = {}) {
   if (ldc == 0) ldc = n;
-  if (ldc != n && (splits != 1 || act != nullptr))
-    return set_error(ORION_ERR_INTERNAL, "a strided GEMM output needs one k split and f32 results");
+  if (ldc != n && (splits != 1 || epi == kGemmSwiglu))
+    return set_error(ORION_ERR_INTERNAL, "a strided GEMM output needs one k split and no SwiGLU");
   using Cfg = TcConfig<TOKN, WST, XST, MT, PAIR>;
   static_assert(Cfg::kSmemBytes <= 232448, "ring exceeds the shared memory of an SM");
   if (MT > 1 && cluster_reduce) return set_error(ORION_ERR_INTERNAL, "cluster split-K is built for one weight tile per CTA");
@@ -560,14 +569,14 @@ int launch_tc(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, float *p
       return set_error(ORION_ERR_INTERNAL, "the paired GEMM needs an even number of weight tile groups and no cluster split-K");
     ORION_CUDA_CHECK("gemm_tc", launch_pdl_cluster(gemm_tc_kernel<TOKN, WST, XST, MT, PAIR>, grid, dim3(kThreads), dim3(2, 1, 1),
                                                    Cfg::kSmemBytes, stream, *mw, *mx, partial, act, rows, n, k, splits,
-                                                   0u, ldc, ready));
+                                                   0u, ldc, (uint32_t)epi, ready));
   } else if (cluster_reduce)
     ORION_CUDA_CHECK("gemm_tc", launch_pdl_cluster(gemm_tc_kernel<TOKN, WST, XST, MT, PAIR>, grid, dim3(kThreads), dim3(1, 1, splits),
                                                    Cfg::kSmemBytes, stream, *mw, *mx, partial, act, rows, n, k, splits,
-                                                   1u, ldc, ready));
+                                                   1u, ldc, (uint32_t)epi, ready));
   else
     ORION_CUDA_CHECK("gemm_tc", launch_pdl(gemm_tc_kernel<TOKN, WST, XST, MT, PAIR>, grid, dim3(kThreads), Cfg::kSmemBytes, stream,
-                                           *mw, *mx, partial, act, rows, n, k, splits, 0u, ldc, ready));
+                                           *mw, *mx, partial, act, rows, n, k, splits, 0u, ldc, (uint32_t)epi, ready));
   count_launch();
   ORION_CUDA_CHECK("gemm_tc", cudaGetLastError());
   return ORION_OK;
@@ -626,12 +635,14 @@ bool gemm_tc_supported(uint32_t rows, uint32_t n, uint32_t k, uint32_t ldx, uint
 
 int launch_gemm_tc(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, float *partial,
                    uint32_t rows, uint32_t n, uint32_t k, uint32_t splits, cudaStream_t stream,
-                   bf16 *act, bool cluster_reduce, uint32_t ldc, ReadyWait ready) {
+                   bf16 *act, bool cluster_reduce, uint32_t ldc, ReadyWait ready, GemmEpilogue epi) {
   const uint32_t nkb = (k + kSlabK - 1) / kSlabK;
   if (cluster_reduce && (splits < 2 || splits > 8 || act != nullptr))
     return set_error(ORION_ERR_INTERNAL, "cluster split-K needs 2..8 splits and f32 output");
-  if (act != nullptr && (splits != 1 || n % 2 != 0))
+  if (epi == kGemmSwiglu && (splits != 1 || n % 2 != 0))
     return set_error(ORION_ERR_INTERNAL, "the fused SwiGLU epilogue needs one k split and an even row count");
+  if ((act != nullptr) != (epi != kGemmPartials) || (act != nullptr && splits != 1))
+    return set_error(ORION_ERR_INTERNAL, "a GEMM epilogue that stores activations needs one k split and a place for them");
   if (splits < 1 || splits > nkb)
     return set_error(ORION_ERR_INTERNAL, "gemm split count %u outside 1..%u", splits, nkb);
   const bool deep = g_small_stages >= 5;
@@ -640,28 +651,28 @@ int launch_gemm_tc(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, flo
   if (rows > 256 && g_prefill_fill == 1 && ((n + kTileN - 1) / kTileN) * ((rows + 255) / 256) < 148) tt = 128;
   switch (tt) {
     case 16:
-      return deep ? launch_tc<16, 6, 3>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, stream, ready)
-                  : launch_tc<16, 5, 3>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, stream, ready);
+      return deep ? launch_tc<16, 6, 3>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready)
+                  : launch_tc<16, 5, 3>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready);
     case 32:
-      return deep ? launch_tc<32, 6, 3>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, stream, ready)
-                  : launch_tc<32, 5, 3>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, stream, ready);
+      return deep ? launch_tc<32, 6, 3>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready)
+                  : launch_tc<32, 5, 3>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready);
     case 64:
-      return deep ? launch_tc<64, 5, 3>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, stream, ready)
-                  : launch_tc<64, 4, 4>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, stream, ready);
+      return deep ? launch_tc<64, 5, 3>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready)
+                  : launch_tc<64, 4, 4>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready);
     case 128:
       return g_mid_tile == 0
-                 ? launch_tc<128, 4, 2>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, stream, ready)
-                 : launch_tc<128, 6, 6>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, stream, ready);
+                 ? launch_tc<128, 4, 2>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready)
+                 : launch_tc<128, 6, 6>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready);
     default: {
       const uint32_t mt = (!cluster_reduce && prefill_weight_tiles(rows, n) == 2) ? 2 : 1;
       // CTA pairs: each CTA loads half of the activation tile, so the rings go a stage deeper
       const bool pair = (g_gemm_pair >= 2 || (g_gemm_pair == 1 && rows >= kPairMinRows)) && !cluster_reduce &&
                         (((n + mt * kTileN - 1) / (mt * kTileN)) & 1u) == 0;
       if (mt == 2)
-        return pair ? launch_tc<256, 4, 4, 2, true>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, stream, ready)
-                    : launch_tc<256, 3, 3, 2>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, stream, ready);
-      return pair ? launch_tc<256, 6, 6, 1, true>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, stream, ready)
-                  : launch_tc<256, 4, 4>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, stream, ready);
+        return pair ? launch_tc<256, 4, 4, 2, true>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready)
+                    : launch_tc<256, 3, 3, 2>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready);
+      return pair ? launch_tc<256, 6, 6, 1, true>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready)
+                  : launch_tc<256, 4, 4>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready);
     }
   }
 }
@@ -771,7 +782,15 @@ int launch_gemm_swiglu(const bf16 *x, uint32_t ldx, const bf16 *w_interleaved, u
                        uint32_t ffn, uint32_t k, cudaStream_t stream, ReadyWait ready) {
   if (!gemm_tc_supported(rows, 2 * ffn, k, ldx, ldw, x, w_interleaved))
     return set_error(ORION_ERR_INTERNAL, "tensor-core GEMM planned for an unaligned operand");
-  return launch_gemm_tc(x, ldx, w_interleaved, ldw, nullptr, rows, 2 * ffn, k, 1, stream, act, false, 0, ready);
+  return launch_gemm_tc(x, ldx, w_interleaved, ldw, nullptr, rows, 2 * ffn, k, 1, stream, act, false, 0, ready, kGemmSwiglu);
+}
+
+int launch_gemm_act(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, bf16 *act, uint32_t ld_act, uint32_t rows, uint32_t n,
+                    uint32_t k, GemmEpilogue epi, cudaStream_t stream) {
+  if (epi != kGemmGelu && epi != kGemmStore) return set_error(ORION_ERR_INTERNAL, "not an epilogue of this entry point");
+  if (!gemm_tc_supported(rows, n, k, ldx, ldw, x, w))
+    return set_error(ORION_ERR_INTERNAL, "tensor-core GEMM planned for an unaligned operand");
+  return launch_gemm_tc(x, ldx, w, ldw, nullptr, rows, n, k, 1, stream, act, false, ld_act, ReadyWait{}, epi);
 }
 
 template <>

@@ -283,6 +283,26 @@ int launch_latent_attention_generic(const T *q, const T *cache, const T *w_uk, c
                                     uint32_t splits, size_t split_stride, LatentShape ls, AttnBatch batch, T *out, uint32_t ldo,
                                     cudaStream_t stream);
 
+// Tuned path for rows that decode, one at a time or a few together (bf16; dim, kv_rank and rot_dim multiples of 16):
+// `row_list` names the batch rows, and item i of the buffers below belongs to row_list[i].
+bool latent_decode_supported(LatentShape ls);
+constexpr uint32_t kLatentMaxSplits = 16;
+// Pieces the window is cut into so that the batch fills the machine.
+uint32_t latent_decode_splits(LatentShape ls, uint32_t rows, uint32_t max_position);
+size_t latent_decode_scratch_floats(LatentShape ls, uint32_t rows, uint32_t splits);
+// Queries into the latent space: qa [rows][heads][kv_rank + rot_dim]. With `q` (from launch_latent_prepare) the
+// projection has been folded and the cache written; without it this launch does both from `partial`.
+int launch_latent_absorb(const float *partial, uint32_t splits, size_t split_stride, const bf16 *q, const bf16 *w_uk, const float *norm_w,
+                         const float *rope_cos, const float *rope_sin, const uint32_t *positions, const uint32_t *slot_block,
+                         const uint32_t *slot_slot, const uint32_t *row_list, uint32_t rows, bf16 *cache, bf16 *qa, LatentShape ls,
+                         cudaStream_t stream);
+// Attention over the cached latents (the rows of this step included), values and gate. `scratch` holds
+// latent_decode_scratch_floats floats; first_row as in StateBatch.
+int launch_latent_decode(const bf16 *qa, const bf16 *cache, const bf16 *w_uv, const float *gate_partial, uint32_t gate_splits,
+                         size_t split_stride, const uint32_t *row_list, const uint32_t *first_row, uint32_t rows, AttnBatch batch,
+                         uint32_t splits, float *scratch, LatentShape ls, bf16 *out, uint32_t ldo, cudaStream_t stream);
+int latent_poll_error(uint32_t *code);
+
 // ---- tensor-parallel hand-over ---------------------------------------------------
 
 constexpr int kMaxTpWorld = 8;
@@ -356,12 +376,17 @@ template <typename T>
 int launch_gemm_simt(const T *x, uint32_t ldx, const T *w, uint32_t ldw, float *out, uint32_t rows,
                      uint32_t n, uint32_t k, cudaStream_t stream);
 // tcgen05 / TMEM / TMA GEMM (bf16).
+enum GemmEpilogue : uint32_t { kGemmPartials = 0, kGemmSwiglu = 1, kGemmGelu = 2, kGemmStore = 3 };
 bool gemm_tc_supported(uint32_t rows, uint32_t n, uint32_t k, uint32_t ldx, uint32_t ldw,
                        const void *x, const void *w);
 int launch_gemm_tc(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, float *partial,
                    uint32_t rows, uint32_t n, uint32_t k, uint32_t splits, cudaStream_t stream,
                    bf16 *act = nullptr, bool cluster_reduce = false, uint32_t ldc = 0,
-                   ReadyWait ready = {});
+                   ReadyWait ready = {}, GemmEpilogue epi = kGemmPartials);
+// The same projection with its result stored as bf16 activations, act[r * ld_act + n] = f(x.w_n), f = GELU (tanh form)
+// or the identity. One k split only.
+int launch_gemm_act(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, bf16 *act, uint32_t ld_act, uint32_t rows, uint32_t n,
+                    uint32_t k, GemmEpilogue epi, cudaStream_t stream);
 // Gate/up projection with SwiGLU in the epilogue: `w_interleaved` is [2 * ffn][k] with gate row f
 // at 2f and up row f at 2f + 1; writes act[r][f] = silu(x.gate_f) * (x.up_f) and no partials.
 // One k split only (gemm_plan(...).splits == 1 and .tensor_core).

@@ -77,11 +77,33 @@ class LayeredModel final : public StepModel<T> {
     return g_step_graph && DTypeOf<T>::is_bf16 && meta_.decode && !meta_.zero_count && !prof_on_ && only_mask_ == 0 &&
            residual_norm_conv_supported(d_.hidden_size, d_.conv_taps);
   }
-  void graph_plan(uint32_t *splits, uint32_t *blocks_per_split) const override { *splits = 1, *blocks_per_split = 0; }
+  void graph_plan(uint32_t *splits, uint32_t *blocks_per_split) const override {
+    // the context splits of every attention layer, folded into one word
+    uint32_t h = 2166136261u;
+    for (const Layer &L : layers_)
+      if (tuned(L)) h = (h ^ context_splits(L, meta_.rows)) * 16777619u;
+    *splits = h, *blocks_per_split = 0;
+  }
   int check_batch(const BatchView &b) override;
-  size_t extra_words(uint64_t seqs) const override { return 3 * seqs + 1; }
+  // [first row of each sequence, S + 1][state copy to read, S][to write, S][rows that decode, kFewRows * S]
+  size_t extra_words(uint64_t seqs) const override { return (3 + kFewRows) * seqs + 1; }
   void fill_extra(const BatchView &b, uint32_t *w) override;
   void step_done(const BatchView &b) override;
+  int poll_errors() override {
+    ORION_TRY(Base::poll_errors());
+    uint32_t code = 0;
+    if (DTypeOf<T>::is_bf16) ORION_TRY(latent_poll_error(&code));
+    if (code) return set_error(ORION_ERR_BACKEND, "backend cuda failed at latent attention: a bounded pipeline wait ran out (code %u)", code);
+    return ORION_OK;
+  }
+  // Sequences with at most this many rows in a batch decode: each row reads the cache by itself.
+  static constexpr uint32_t kFewRows = 8;
+  bool tuned(const Layer &L) const { return DTypeOf<T>::is_bf16 && L.attention() && latent_decode_supported(L.ls); }
+  uint32_t context_splits(const Layer &L, uint32_t rows) const {
+    uint32_t s = latent_decode_splits(L.ls, rows, meta_.max_position);
+    while (s > 1 && latent_decode_scratch_floats(L.ls, rows, s) > scratch_floats_) --s;
+    return s;
+  }
   StateBatch state_batch() const {
     const uint32_t *x = d_meta_ + meta_.extra, S = meta_.seqs;
     return StateBatch{x, x + S + 1, x + 2 * S + 1, d_meta_ + meta_.seq_of_row, meta_.rows, S, meta_.decode};
@@ -97,6 +119,10 @@ class LayeredModel final : public StepModel<T> {
   T *conv_m_ = nullptr, *conv_f_ = nullptr;  // inputs of the mixer and the feed-forward
   T *cat_ = nullptr;                         // their activations, side by side
   T *qbuf_ = nullptr;
+  T *qa_ = nullptr;           // queries of decoding rows in the latent space
+  float *scratch_ = nullptr;  // their weighted latents per context split
+  size_t scratch_floats_ = 0;
+  uint32_t few_rows_ = 0;     // rows of this batch that decode
   struct Rope {
     double base;
     uint32_t dims;
@@ -203,6 +229,16 @@ int LayeredModel<T>::init() {
   ORION_TRY(alloc(&conv_f_, rows * H));
   ORION_TRY(zeroed(&cat_, rows * cat));  // columns that nobody writes meet zero weights and must be finite
   ORION_TRY(alloc(&qbuf_, rows * qcols));
+  size_t qa = 0;
+  const uint32_t few = (uint32_t)std::min<uint64_t>(rows, (uint64_t)kFewRows * d.max_batch_sequences);
+  for (const Layer &L : layers_) {
+    if (!tuned(L)) continue;
+    qa = std::max(qa, (size_t)few * L.ls.heads * L.ls.kv_cols());
+    for (uint32_t r = 1; r <= few; ++r)
+      scratch_floats_ = std::max(scratch_floats_, latent_decode_scratch_floats(L.ls, r, latent_decode_splits(L.ls, r, d.max_position_embeddings)));
+  }
+  ORION_TRY(alloc(&qa_, qa));
+  ORION_TRY(alloc(&scratch_, scratch_floats_));
   slots_.resize(d.num_state_slots);
   ORION_CUDA_CHECK("model init", cudaStreamSynchronize(stream_));
   return ORION_OK;
@@ -362,13 +398,16 @@ int LayeredModel<T>::check_batch(const BatchView &b) {
 template <typename T>
 void LayeredModel<T>::fill_extra(const BatchView &b, uint32_t *w) {
   const uint64_t S = b.num_sequences;
-  uint32_t *first = w, *read = w + S + 1, *write = read + S;
+  uint32_t *first = w, *read = w + S + 1, *write = read + S, *few = write + S;
   uint64_t row = 0;
+  few_rows_ = 0;
   for (uint64_t s = 0; s < S; ++s) {
     const uint32_t slot = b.state_slots[s], copy = slots_[slot].copy;
     first[s] = (uint32_t)row;
     read[s] = b.positions[row] == 0 ? kNoState : 2 * slot + copy;
     write[s] = 2 * slot + (copy ^ 1u);
+    if (b.slot_token_counts[s] <= kFewRows)
+      for (uint64_t i = 0; i < b.slot_token_counts[s]; ++i) few[few_rows_++] = (uint32_t)(row + i);
     row += b.slot_token_counts[s];
   }
   first[S] = (uint32_t)row;
@@ -395,6 +434,18 @@ int LayeredModel<T>::mixer(const Layer &L, const StateBatch &sb, const AttnBatch
   ORION_TRY(timed(kProfGemm, [&] { return launch_gemm<T>(conv_m_, H, L.w_mix, H, partial_, Tn, L.mix_in, H, p, stream_); }));
   if (!L.attention())
     return timed(kProfAttention, [&] { return launch_min_gru<T>(partial_, p.out_slabs, slab, L.mix_bias, L.rec_state, sb, cat_, L.cat, L.d.width, stream_); });
+  if constexpr (DTypeOf<T>::is_bf16) {
+    if (tuned(L) && few_rows_ == Tn) {
+      const uint32_t *first = d_meta_ + meta_.extra, *few = first + 3 * meta_.seqs + 1, sp = context_splits(L, Tn);
+      ORION_TRY(timed(kProfAttention, [&] {
+        return launch_latent_absorb(partial_, p.out_slabs, slab, nullptr, L.w_uk, L.latent_norm, L.rope_cos, L.rope_sin, ab.query_positions,
+                                    d_meta_ + meta_.slot_block, d_meta_ + meta_.slot_slot, few, Tn, L.cache, qa_, L.ls, stream_);
+      }));
+      return timed(kProfAttention, [&] {
+        return launch_latent_decode(qa_, L.cache, L.w_uv, partial_, p.out_slabs, slab, few, first, Tn, ab, sp, scratch_, L.ls, cat_, L.cat, stream_);
+      });
+    }
+  }
   ORION_TRY(timed(kProfAttention, [&] {
     return launch_latent_prepare<T>(partial_, p.out_slabs, slab, L.latent_norm, L.rope_cos, L.rope_sin, ab.query_positions,
                                     d_meta_ + meta_.slot_block, d_meta_ + meta_.slot_slot, qbuf_, L.cache, L.ls, Tn, stream_);
@@ -434,10 +485,19 @@ int LayeredModel<T>::run_step_body(bool want_argmax, int part) {
     if (L.d.ffn_dim) {
       const uint32_t F = L.d.ffn_dim;
       const GemmPlan p = plan_for(Tn, F, H, H);
-      ORION_TRY(timed(kProfGemm, [&] { return launch_gemm<T>(conv_f_, H, L.w_up, H, partial_, Tn, F, H, p, stream_); }));
-      ORION_TRY(timed(kProfElementwise, [&] {
-        return launch_gelu<T>(partial_, p.out_slabs, (size_t)Tn * F, cat_ + L.ff_at, L.cat, Tn, F, stream_);
-      }));
+      bool in_epilogue = false;
+      if constexpr (DTypeOf<T>::is_bf16) {
+        if (p.tensor_core && p.splits == 1) {  // GELU in the GEMM epilogue: no partials, no extra launch
+          in_epilogue = true;
+          ORION_TRY(timed(kProfGemm, [&] { return launch_gemm_act(conv_f_, H, L.w_up, H, cat_ + L.ff_at, L.cat, Tn, F, H, kGemmGelu, stream_); }));
+        }
+      }
+      if (!in_epilogue) {
+        ORION_TRY(timed(kProfGemm, [&] { return launch_gemm<T>(conv_f_, H, L.w_up, H, partial_, Tn, F, H, p, stream_); }));
+        ORION_TRY(timed(kProfElementwise, [&] {
+          return launch_gelu<T>(partial_, p.out_slabs, (size_t)Tn * F, cat_ + L.ff_at, L.cat, Tn, F, stream_);
+        }));
+      }
     }
     ORION_TRY(mixer(L, sb, ab));
     out = plan_for(Tn, H, L.cat, L.cat);

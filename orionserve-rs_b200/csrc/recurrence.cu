@@ -13,11 +13,6 @@
 namespace orion {
 namespace {
 
-__device__ __forceinline__ float sigmoid_f(float x) {
-  const float e = expf(-fabsf(x));
-  return (x >= 0.f ? 1.f : e) / (1.f + e);
-}
-
 // The map of one row and channel: S -> a S + b.
 __device__ __forceinline__ void min_gru_map(float z_pre, float x_pre, float &a, float &b) {
   const float z = sigmoid_f(z_pre), cand = x_pre >= 0.f ? x_pre + 0.5f : sigmoid_f(x_pre);

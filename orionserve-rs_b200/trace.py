@@ -28,15 +28,18 @@ STATE_SLOTS = 4
 class TraceRunner:
     """The live requests of a trace, their block tables and state slots, and the model they run on."""
 
-    def __init__(self, directory: str, dtype: DType, max_tokens: int):
-        blocks = (max_tokens + ROUND - 1) // ROUND * (ROUND // BLOCK)
-        self.model = load_model(directory, blocks, BLOCK, CudaBackend(0), compute_dtype=dtype,
-                                max_batch_tokens=blocks * BLOCK, max_batch_sequences=STATE_SLOTS,
-                                num_state_slots=STATE_SLOTS)
-        self.slots = self.model.num_state_slots()
-        self.cache = engine.KvCacheManager(blocks, BLOCK, False, num_state_slots=self.slots)
+    def __init__(self, model):
+        self.model = model
+        self.slots = model.num_state_slots()
+        self.cache = engine.KvCacheManager(model.num_blocks, model.block_size, False, num_state_slots=self.slots)
         self.live = {}  # request -> (sequence id, tokens so far)
         self.next_id = 1
+
+    @classmethod
+    def from_directory(cls, directory: str, dtype: DType, max_tokens: int) -> "TraceRunner":
+        blocks = (max_tokens + ROUND - 1) // ROUND * (ROUND // BLOCK)
+        return cls(load_model(directory, blocks, BLOCK, CudaBackend(0), compute_dtype=dtype, max_batch_tokens=blocks * BLOCK,
+                              max_batch_sequences=STATE_SLOTS, num_state_slots=STATE_SLOTS))
 
     def step(self, entries, end=()):
         """Runs one batch; returns the wanted logits [wanted, vocab] or None when nothing is wanted."""
@@ -79,7 +82,7 @@ def main(argv=None) -> int:
                     help=f"most tokens that live requests hold at any time, each rounded up to {ROUND}")
     args = ap.parse_args(argv)
     dtype = {"bfloat16": DType.BF16, "float32": DType.F32}[args.dtype]
-    runner = TraceRunner(args.model, dtype, args.max_tokens)
+    runner = TraceRunner.from_directory(args.model, dtype, args.max_tokens)
     for line in sys.stdin:
         if not line.strip():
             continue
