@@ -353,6 +353,132 @@ def run_serving(args):
 
 
 # ---------------------------------------------------------------------------------------------
+# Metapel (min-GRU and latent attention layers) beside the Llama layout at equal size
+# ---------------------------------------------------------------------------------------------
+
+# Layer sizes of real models, random weights; the layers alternate min-GRU and latent attention.
+METAPEL_SHAPES = {
+    "2048": dict(hidden=2048, ffn=8192, width=2048, heads=16, dim=128, rot=64, vdim=128, rank=512, window=1024),
+    "4096": dict(hidden=4096, ffn=16384, width=4096, heads=32, dim=128, rot=64, vdim=128, rank=512, window=1024),
+}
+METAPEL_VOCAB = 32768
+
+
+def metapel_meta(pkg, name, layers):
+    z = METAPEL_SHAPES[name]
+    gru = pkg.LayerSpec("mingru", z["ffn"], width=z["width"])
+    att = pkg.LayerSpec("latent_attention", z["ffn"], heads=z["heads"], dim=z["dim"], rot_dim=z["rot"], value_dim=z["vdim"],
+                        kv_rank=z["rank"], window=z["window"], rope_dims=z["rot"], rope_base=10000.0,
+                        scale=(z["dim"] + z["rot"]) ** -0.5)
+    return pkg.LayeredMetadata("Metapel", f"metapel-{name}", z["hidden"], METAPEL_VOCAB,
+                               [att if i % 2 else gru for i in range(layers)], 1e-6, 4)
+
+
+def metapel_work(meta, rows, contexts, prompts):
+    """(projection weight bytes, projection flops, cache bytes, attention flops) of one step. `contexts`: context
+    of every decoding row; `prompts`: lengths of whole prompts (positions 0 .. n - 1). The attention flops of a
+    prompt are those of the expanded form (scores over dim + rot, values over vdim, per head and visible key)."""
+    w = flops = cache = attn = 0
+    for s in meta.layers:
+        H = meta.hidden_size
+        if s.mixer == "mingru":
+            n = H * 3 * s.width + s.width * H
+        else:
+            n = H * (s.heads * (s.dim + s.rot_dim) + s.kv_rank + s.rot_dim + s.heads * s.value_dim) + s.heads * s.value_dim * H
+            absorb = s.heads * (s.dim + s.value_dim) * s.kv_rank
+            n += absorb
+            seen = [min(c, s.window) if s.window else c for c in contexts]
+            cache += sum(seen) * (s.kv_rank + s.rot_dim) * 2
+            attn += sum(seen) * s.heads * 2 * (2 * s.kv_rank + s.rot_dim)
+            for p in prompts:
+                keys = sum(min(i + 1, s.window or i + 1) for i in range(p))
+                attn += keys * s.heads * 2 * (s.dim + s.rot_dim + s.value_dim)
+        n += 2 * H * s.ffn_dim
+        w, flops = w + 2 * n, flops + 2 * n * rows
+    outs = len(contexts) + len(prompts)
+    return w + 2 * METAPEL_VOCAB * meta.hidden_size, flops + 2 * outs * METAPEL_VOCAB * meta.hidden_size, cache, attn
+
+
+def llama_work(m, rows, contexts, prompts):
+    w = weight_bytes_per_step(m)
+    flops = 2 * rows * m["num_layers"] * layer_param_count(m) + 2 * (len(contexts) + len(prompts)) * m["vocab_size"] * m["hidden_size"]
+    keys = sum(p * (p + 1) // 2 for p in prompts)
+    q = m["num_attention_heads"] * m["head_dim"]
+    return w, flops, kv_bytes_per_step(m, contexts) if contexts else 0, m["num_layers"] * (keys + sum(contexts)) * q * 4
+
+
+def run_metapel(args):
+    """Prefill and decode throughput of Metapel at a few layer sizes, and of the Llama layout (same hidden size, head
+    count and head size, four query heads per KV head, feed-forward of equal parameter count) on the same
+    batches. Times are CUDA events around whole replayed steps and around one kernel family run back to back."""
+    import __graft_entry__ as ge
+
+    pkg = ge.load_package()
+    backend = pkg.CudaBackend(0)
+    hbm, src = measured_peaks()
+    try:
+        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+            tflops = float(json.load(f)["bf16_tflops_sustained"])
+    except (OSError, ValueError, KeyError):
+        tflops = 1400.0
+    layers, out = args.layers if args.layers != 32 else 8, []
+    batches = [("decode", b, CONTEXT) for b in (1, 16, 64)] + [("prefill", 1, 2048), ("prefill", 4, 2048)]
+    with ClockSampler(0) as clocks:
+        for name in args.metapel_shapes.split(","):
+            z = METAPEL_SHAPES[name]
+            m = dict(hidden_size=z["hidden"], num_layers=layers, num_attention_heads=z["heads"], num_kv_heads=z["heads"] // 4,
+                     head_dim=128, vocab_size=METAPEL_VOCAB, ffn_dim=(z["ffn"] * 2 // 3 + 127) // 128 * 128,
+                     max_position_embeddings=8192, rope_theta=500000.0, rms_norm_eps=1e-5)
+            blocks = max(b * c // BLOCK for _, b, c in batches) + 64
+            for kind in ("metapel", "llama"):
+                kw = dict(compute_dtype=pkg.DType.BF16, max_batch_tokens=8192, max_batch_sequences=64)
+                if kind == "metapel":
+                    meta = metapel_meta(pkg, name, layers)
+                    model = pkg.CudaLayeredModel(meta, blocks, BLOCK, backend, **kw)
+                else:
+                    meta = pkg.ModelMetadata(architecture="llama", name="llama", dtype=pkg.DType.BF16, **m)
+                    model = pkg.CudaTransformerModel(meta, blocks, BLOCK, backend, **kw)
+                model.init_random(seed=1, std=0.02)
+                for mode, b, n in batches:
+                    if args.metapel_only and f"{mode}{b}" not in args.metapel_only.split(","):
+                        continue
+                    rng = np.random.default_rng(3)
+                    tables = [list(range(s * n // BLOCK, (s + 1) * n // BLOCK)) for s in range(b)]
+                    slots = list(range(b)) if kind == "metapel" else None
+                    ids = list(range(1, b + 1))
+                    prompt = rng.integers(0, METAPEL_VOCAB, n)
+                    count = n if mode == "prefill" else n - 1
+                    per = max(1, 8192 // n)
+                    for s0 in range(0, b, per):  # real prompts: the decode steps go on from their state and cache
+                        part = list(range(s0, min(b, s0 + per)))
+                        whole = pkg.ForwardBatch(np.tile(prompt[:count], len(part)), np.tile(np.arange(count), len(part)),
+                                                 [ids[s] for s in part], [count] * len(part), [count] * len(part),
+                                                 [tables[s] for s in part], state_slots=None if slots is None else part)
+                        model.forward(whole)
+                    if mode == "decode":
+                        model.forward(pkg.ForwardBatch(prompt[-1:].repeat(b), [n - 1] * b, ids, [1] * b, [n] * b, tables,
+                                                       has_prefill=False, state_slots=slots))
+                    rows, contexts, prompts = (b, [n] * b, []) if mode == "decode" else (b * n, [], [n] * b)
+                    steps = args.steps if mode == "decode" else max(3, args.steps // 5)
+                    model.replay(max(3, args.warmup))
+                    ms = model.replay(steps) / steps
+                    fam = {c: model.replay_categories(steps, c) / steps for c in ("gemm", "attention", "elementwise")}
+                    wb, fl, cb, af = (metapel_work(meta, rows, contexts, prompts) if kind == "metapel"
+                                      else llama_work(m, rows, contexts, prompts))
+                    gemm_s, attn_s = fam["gemm"] / 1e3, fam["attention"] / 1e3
+                    out.append({"model": kind, "shape": name, "layers": layers, "mode": mode, "sequences": b, "tokens_each": n,
+                                "ms_per_step": ms, "tokens_per_s": rows / ms * 1e3, "gemm_ms": fam["gemm"], "mixer_ms": fam["attention"],
+                                "elementwise_ms": fam["elementwise"], "launches": model.last_launch_count(),
+                                "gemm_frac": max(wb / gemm_s / hbm / 1e9, fl / gemm_s / tflops / 1e12),
+                                "step_frac": max((wb + cb) / (ms / 1e3) / hbm / 1e9, (fl + af) / (ms / 1e3) / tflops / 1e12)})
+                del model
+    print(json.dumps({"metric": "Metapel prefill and decode throughput beside the Llama layout", "unit": "tokens/s", "n_gpus": 1,
+                      "dtype": "bf16", "data": "synthetic", "peaks": {"hbm_gbs": hbm, "bf16_tflops_sustained": tflops, "source": src},
+                      "results": out, "clocks": clocks.summary()}))
+    return 0
+
+
+# ---------------------------------------------------------------------------------------------
 # Tensor-parallel parity, checked before anything is timed at N > 1
 # ---------------------------------------------------------------------------------------------
 
@@ -500,6 +626,8 @@ def tp_parity(pkg, backend, dist, rank, world, dtype_name="BF16", model=None, nu
 def run_ours(args):
     if args.workload in ("serving", "prefix"):
         return run_serving(args)
+    if args.workload == "metapel":
+        return run_metapel(args)
     import __graft_entry__ as ge
 
     pkg = ge.load_package()
@@ -714,9 +842,12 @@ def main():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", choices=("ours", "reference"), default="ours")
     ap.add_argument("--no-cpu-baseline", action="store_true")
-    ap.add_argument("--workload", choices=("decode", "serving", "prefix"), default="decode",
+    ap.add_argument("--workload", choices=("decode", "serving", "prefix", "metapel"), default="decode",
                     help="decode = the headline step (default); serving = continuous batching through the engine "
-                         "loop; prefix = shared-prefix requests on the Qwen2-7B shape through the engine loop")
+                         "loop; prefix = shared-prefix requests on the Qwen2-7B shape through the engine loop; metapel = prefill "
+                         "and decode of the Metapel design at a few sizes beside the Llama layout")
+    ap.add_argument("--metapel-shapes", default="2048,4096", help="metapel workload: layer sizes to run")
+    ap.add_argument("--metapel-only", default="", help="metapel workload: batches to run, for instance decode64,prefill1")
     ap.add_argument("--skip-cached-prefix", action="store_true",
                     help="engine workloads: start prefill after the tokens adopted from the prefix cache "
                          "(an extension; the reference shares the blocks but recomputes them)")

@@ -143,17 +143,25 @@ def test_mechanism_alone(pkg, backend, dtype, name):
     assert worst_error(f.run("q", t, [30, 2, 9, 1]), exp) < tol(dtype)
 
 
+def long_memory():
+    """Update gates that open for token 2 and stay almost shut for the others; 900 tokens, the first of them 2."""
+    width = 256
+    cfg = config(width, 80, [mingru(96)], taps=1)
+    w = silence(random_weights(cfg, seed=9), "canon")
+    w["l0.norm1"] = np.ones_like(w["l0.norm1"])
+    h = w["embed"][2].astype(np.float64)
+    z = np.tile(20.0 * h / np.sqrt((h ** 2).mean()) / width, (96, 1))
+    w["l0.mix.z"], w["l0.mix.z.b"] = (binding.round_to_bf16(x.astype(np.float32)) for x in (z, np.full(96, -10.0)))
+    w["l0.mix.x"], w["l0.mix.o"] = binding.round_to_bf16(w["l0.mix.x"] * 2), binding.round_to_bf16(w["l0.mix.o"] * 3)
+    return cfg, w, [2] + np.random.default_rng(2).integers(3, 80, 899).tolist()
+
+
 def test_long_recurrence_keeps_its_state(pkg, backend, dtype):
-    """Update gates near zero: the state of the first tokens is still most of the state after hundreds."""
-    cfg = config(64, 80, [mingru(96)], taps=1)
-    w = random_weights(cfg, seed=9)
-    w["l0.mix.z.b"] = binding.round_to_bf16(np.full(96, -7.0, np.float32))
-    w["l0.mix.z"] = np.zeros_like(w["l0.mix.z"])
-    w["l0.mix.x"] = binding.round_to_bf16(w["l0.mix.x"] * 200)
-    t = np.random.default_rng(2).integers(0, 80, 900).tolist()
+    """The state that the first token leaves is still there after hundreds of tokens."""
+    cfg, w, t = long_memory()
     exp = metapel.forward(t, cfg, w)
-    other = metapel.forward([(t[0] + 1) % 80] + t[1:], cfg, w)
-    assert worst_error(other[-1:], exp[-1:]) > 3 * tol(dtype), "the first token still shows at the end"
+    other = metapel.forward([3] + t[1:], cfg, w)
+    assert worst_error(other[-1:], exp[-1:]) > 0.2, "the first token still shows at the end"
     for sizes in ([900], [300, 1], [5, 70, 2]):
         f = Feeder(pkg, make_model(pkg, backend, cfg, w, dtype))
         assert worst_error(f.run("p", t, sizes), exp) < tol(dtype), sizes
@@ -167,6 +175,7 @@ def beacon_model(window, heads=2, dim=16, rank=32, vdim=16, width=128):
     cfg = config(width, 64, [latent(heads, dim, 16, vdim, rank, window)], taps=2)
     rng = np.random.default_rng(8)
     w = silence(random_weights(cfg, seed=8, gain=0.3), "canon")
+    w["l0.mix.dkv"] = w["l0.mix.dkv"] * 5  # the latents of other tokens point elsewhere
     hq, hk = (w["embed"][i].astype(np.float64) for i in (1, 2))
     hq, hk = hq / np.sqrt((hq ** 2).mean()), hk / np.sqrt((hk ** 2).mean())
     c = rng.standard_normal(rank)
@@ -174,14 +183,14 @@ def beacon_model(window, heads=2, dim=16, rank=32, vdim=16, width=128):
     w["l0.norm1"] = np.ones_like(w["l0.norm1"])
     w["l0.mix.dkv.norm"] = np.ones_like(w["l0.mix.dkv.norm"])
     dkv = w["l0.mix.dkv"].astype(np.float64)
-    dkv[:rank] += 4.0 * np.outer(c, hk) / width
+    dkv[:rank] += 6.0 * np.outer(c, hk) / width
     uk = w["l0.mix.uk"].astype(np.float64) + u.reshape(-1, 1) * c[None] / rank
     q = w["l0.mix.q"].astype(np.float64).reshape(heads, dim + 16, width)
     q[:, :dim] += 5.0 * u[:, :, None] * hq / width
     w["l0.mix.dkv"], w["l0.mix.uk"] = (binding.round_to_bf16(x.astype(np.float32)) for x in (dkv, uk))
     w["l0.mix.q"] = binding.round_to_bf16(q.reshape(-1, width).astype(np.float32))
-    w["l0.mix.uv"] = binding.round_to_bf16(w["l0.mix.uv"] * 6)
-    w["l0.mix.o"] = binding.round_to_bf16(w["l0.mix.o"] * 3)
+    w["l0.mix.uv"] = binding.round_to_bf16(w["l0.mix.uv"] * 8)
+    w["l0.mix.o"] = binding.round_to_bf16(w["l0.mix.o"] * 4)
     return cfg, w
 
 
