@@ -235,7 +235,8 @@ constexpr uint32_t kNoState = 0xFFFFFFFFu;
 
 // Causal per-channel convolution over time added to its input, for up to two sets of weights at once
 // (the two sublayers of a parallel layer): out_i = h + conv_i(h), conv_i(h)_t = sum_j w_i[c][j] h_(t - taps + 1 + j).
-// `state` is [copies][taps - 1][cols]: the last taps - 1 rows of h. w2 / out2 may be null.
+// The filters are stored by tap, w_i[j][c]. `state` is [copies][taps - 1][cols]: the last taps - 1 rows of h. w2 / out2
+// may be null.
 template <typename T>
 int launch_causal_conv(const T *h, const T *w1, const T *w2, uint32_t taps, T *state, StateBatch sb, T *out1, T *out2,
                        uint32_t cols, cudaStream_t stream);
@@ -245,6 +246,9 @@ template <typename T>
 int launch_residual_norm_conv(const float *partial, uint32_t splits, size_t split_stride, const T *embed, const uint32_t *tokens,
                               float *hidden, const float *norm_w, float eps, const T *w1, const T *w2, uint32_t taps, T *state,
                               StateBatch sb, T *out1, T *out2, uint32_t cols, cudaStream_t stream);
+// dst[c][r] = src[r][c]
+template <typename T>
+int launch_transpose(const T *src, T *dst, uint32_t rows, uint32_t cols, cudaStream_t stream);
 bool residual_norm_conv_supported(uint32_t cols, uint32_t taps);
 
 // Minimal gated recurrence, element by element: with the projections' partial sums [z | x | g] of `width`
@@ -257,7 +261,7 @@ int launch_min_gru(const float *partial, uint32_t splits, size_t split_stride, c
 // ---- latent attention ---------------------------------------------------------------------
 //
 // The cache of one layer holds, per token, the normalised latent (kv_rank values) followed by the rotated key
-// part that all heads share (rot_dim values): [block][slot][row_stride], row_stride a multiple of 8.
+// part that all heads share (rot_dim values): [block][slot][row_stride], row_stride an odd multiple of 8.
 struct LatentShape {
   uint32_t heads, dim, rot_dim, value_dim, kv_rank, window, rope_dims, block_size, row_stride;
   float scale, eps;
@@ -290,11 +294,8 @@ constexpr uint32_t kLatentMaxSplits = 16;
 // Pieces the window is cut into so that the batch fills the machine.
 uint32_t latent_decode_splits(LatentShape ls, uint32_t rows, uint32_t max_position);
 size_t latent_decode_scratch_floats(LatentShape ls, uint32_t rows, uint32_t splits);
-// Queries into the latent space: qa [rows][heads][kv_rank + rot_dim]. With `q` (from launch_latent_prepare) the
-// projection has been folded and the cache written; without it this launch does both from `partial`.
-int launch_latent_absorb(const float *partial, uint32_t splits, size_t split_stride, const bf16 *q, const bf16 *w_uk, const float *norm_w,
-                         const float *rope_cos, const float *rope_sin, const uint32_t *positions, const uint32_t *slot_block,
-                         const uint32_t *slot_slot, const uint32_t *row_list, uint32_t rows, bf16 *cache, bf16 *qa, LatentShape ls,
+// Queries (from launch_latent_prepare) into the latent space: qa [rows][heads][kv_rank + rot_dim].
+int launch_latent_absorb(const bf16 *q, const bf16 *w_uk, const uint32_t *row_list, uint32_t rows, bf16 *qa, LatentShape ls,
                          cudaStream_t stream);
 // Attention over the cached latents (the rows of this step included), values and gate. `scratch` holds
 // latent_decode_scratch_floats floats; first_row as in StateBatch.

@@ -5,8 +5,7 @@
 //   latent_prepare_kernel            folds the joint projection: queries rotated, latent normalised and cached
 //   latent_attention_generic_kernel  any shape and batch, f32 arithmetic: the f32 build and unusual shapes
 //   latent_absorb_kernel             rows that decode: their queries taken into the latent space, per head
-//                                    (W_uk^T q on mma.sync; on pure decode batches it folds the projection itself
-//                                    and writes the cache, so latent_prepare_kernel does not run)
+//                                    (W_uk^T q on mma.sync)
 //   latent_decode_kernel             rows that decode: scores and weighted latents over the window's cache rows
 //   latent_value_kernel              rows that decode: merges the context splits, W_uv per head, output gate
 #include "kernels.h"
@@ -69,6 +68,73 @@ latent_prepare_kernel(const float *__restrict__ partial, uint32_t splits, size_t
   for (uint32_t i = tid; i < ls.kv_rank; i += kPrepThreads)
     dst[i] = from_f32<T>(fold(lat + i, splits, split_stride) * scale * norm_w[i]);
   for (uint32_t i = tid; i < ls.rot_dim; i += kPrepThreads) dst[ls.kv_rank + i] = from_f32<T>(rotated(lat + ls.kv_rank, i));
+}
+
+// The same, four columns per thread and one round of loads: every part a multiple of four columns. blockIdx.y = 0
+// is the row's latent and shared key part, the others are 1024 query columns each.
+template <typename T>
+__device__ __forceinline__ void store4(T *p, float4 v);
+template <>
+__device__ __forceinline__ void store4<float>(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
+template <>
+__device__ __forceinline__ void store4<bf16>(bf16 *p, float4 v) {
+  uint2 x;
+  x.x = pack_bf16x2(v.x, v.y);
+  x.y = pack_bf16x2(v.z, v.w);
+  *reinterpret_cast<uint2 *>(p) = x;
+}
+__device__ __forceinline__ float4 rotate4(float4 v, float2 c, float2 s) {  // two neighbouring pairs
+  return make_float4(v.x * c.x - v.y * s.x, v.y * c.x + v.x * s.x, v.z * c.y - v.w * s.y, v.w * c.y + v.z * s.y);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kPrepThreads)
+latent_prepare_vec_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, const float *__restrict__ norm_w,
+                          const float *__restrict__ rope_cos, const float *__restrict__ rope_sin, const uint32_t *__restrict__ positions,
+                          const uint32_t *__restrict__ slot_block, const uint32_t *__restrict__ slot_slot, T *__restrict__ q,
+                          T *__restrict__ cache, LatentShape ls) {
+  __shared__ float red[kPrepThreads / 32];
+  pdl_trigger();
+  const uint32_t row = blockIdx.x, tid = threadIdx.x, half = ls.rope_dims / 2;
+  const float *cs = rope_cos + (size_t)positions[row] * half, *sn = rope_sin + (size_t)positions[row] * half;
+  const float *p = partial + (size_t)row * ls.cols();
+  if (blockIdx.y > 0) {
+    const uint32_t i = ((blockIdx.y - 1) * kPrepThreads + tid) * 4, d = i % ls.q_dim();
+    const bool live = i < ls.q_cols(), rot = live && d >= ls.dim && d - ls.dim < ls.rope_dims;
+    float2 c, sv;
+    if (rot) {  // rope_dims is a multiple of 4 here
+      c = *reinterpret_cast<const float2 *>(cs + (d - ls.dim) / 2);
+      sv = *reinterpret_cast<const float2 *>(sn + (d - ls.dim) / 2);
+    }
+    pdl_wait();
+    if (!live) return;
+    float4 v = sum_slabs4(p + i, splits, split_stride);
+    if (rot) v = rotate4(v, c, sv);
+    store4<T>(q + (size_t)row * ls.q_cols() + i, v);
+    return;
+  }
+  const float *lat = p + ls.q_cols();
+  T *dst = cache + ((size_t)slot_block[row] * ls.block_size + slot_slot[row]) * ls.row_stride;
+  const uint32_t i = tid * 4;
+  pdl_wait();
+  float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (i < ls.kv_cols()) v = sum_slabs4(lat + i, splits, split_stride);
+  float ss = i < ls.kv_rank ? v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w : 0.f;
+  ss = warp_sum(ss);
+  if ((tid & 31) == 0) red[tid >> 5] = ss;
+  __syncthreads();
+  float total = 0.f;
+#pragma unroll
+  for (uint32_t w = 0; w < kPrepThreads / 32; ++w) total += red[w];
+  if (i >= ls.kv_cols()) return;
+  if (i < ls.kv_rank) {
+    const float scale = 1.0f / sqrtf(total / (float)ls.kv_rank + ls.eps);
+    const float4 g = *reinterpret_cast<const float4 *>(norm_w + i);
+    v = make_float4(v.x * scale * g.x, v.y * scale * g.y, v.z * scale * g.z, v.w * scale * g.w);
+  } else if (i - ls.kv_rank < ls.rope_dims) {
+    v = rotate4(v, *reinterpret_cast<const float2 *>(cs + (i - ls.kv_rank) / 2), *reinterpret_cast<const float2 *>(sn + (i - ls.kv_rank) / 2));
+  }
+  store4<T>(dst + i, v);
 }
 
 constexpr uint32_t kGenThreads = 128, kGenKeys = 256;
@@ -161,55 +227,19 @@ __device__ __forceinline__ void cp_async16(void *smem, const void *gmem) {
 }
 __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 
-// CTA (x: head and 64-wide tile of the latent, or, past those, cache rows; y: tile of 32 listed rows).
+// CTA (x: head and 64-wide tile of the latent; y: tile of 32 listed rows).
 // A = W_uk of the head, [dim][64 latent columns] (transposed on the way into the fragments), B = the rows' queries.
 constexpr uint32_t kAbsorbTile = 64;
-template <bool kFold>
 __global__ void __launch_bounds__(128)
-latent_absorb_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, const bf16 *__restrict__ q,
-                     const bf16 *__restrict__ w_uk, const float *__restrict__ norm_w, const float *__restrict__ rope_cos,
-                     const float *__restrict__ rope_sin, const uint32_t *__restrict__ positions, const uint32_t *__restrict__ slot_block,
-                     const uint32_t *__restrict__ slot_slot, const uint32_t *__restrict__ row_list, uint32_t rows,
-                     bf16 *__restrict__ cache, bf16 *__restrict__ qa, LatentShape ls) {
+latent_absorb_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ w_uk, const uint32_t *__restrict__ row_list, uint32_t rows,
+                     bf16 *__restrict__ qa, LatentShape ls) {
   extern __shared__ __align__(16) uint8_t smem[];
   const uint32_t w_pitch = kAbsorbTile * 2 + 16, q_pitch = ls.dim * 2 + 16;
   uint8_t *w_s = smem, *q_s = smem + ls.dim * w_pitch;
   pdl_trigger();
   const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const uint32_t tiles = (ls.kv_rank + kAbsorbTile - 1) / kAbsorbTile, heads_part = ls.heads * tiles;
-  const uint32_t row0 = blockIdx.y * kRowTile, half = ls.rope_dims / 2;
-  const uint32_t qd = ls.q_dim(), width = ls.kv_cols();
-  // value i of a rotated part whose first column is `at`
-  auto rotated = [&](const float *at, uint32_t i, uint32_t pos) {
-    const float v = fold(at + i, splits, split_stride);
-    if (i >= 2 * half) return v;
-    const float other = fold(at + (i ^ 1), splits, split_stride), c = rope_cos[(size_t)pos * half + (i >> 1)],
-                s = rope_sin[(size_t)pos * half + (i >> 1)];
-    return (i & 1) ? v * c + other * s : v * c - other * s;
-  };
-  if (blockIdx.x >= heads_part) {  // cache rows, one warp each
-    const uint32_t r = row0 + (blockIdx.x - heads_part) * 4 + warp;
-    pdl_wait();
-    if (r >= rows) return;
-    const uint32_t row = row_list[r];
-    const float *lat = partial + (size_t)row * ls.cols() + ls.q_cols();
-    bf16 *dst = cache + ((size_t)slot_block[row] * ls.block_size + slot_slot[row]) * ls.row_stride;
-    float keep[16], ss = 0.f;  // kv_rank <= 512
-#pragma unroll
-    for (int k = 0; k < 16; ++k) {
-      const uint32_t i = k * 32 + lane;
-      keep[k] = i < ls.kv_rank ? fold(lat + i, splits, split_stride) : 0.f;
-      ss += keep[k] * keep[k];
-    }
-    const float scale = 1.0f / sqrtf(warp_sum(ss) / (float)ls.kv_rank + ls.eps);
-#pragma unroll
-    for (int k = 0; k < 16; ++k) {
-      const uint32_t i = k * 32 + lane;
-      if (i < ls.kv_rank) dst[i] = __float2bfloat16_rn(keep[k] * scale * norm_w[i]);
-    }
-    for (uint32_t i = lane; i < ls.rot_dim; i += 32) dst[ls.kv_rank + i] = __float2bfloat16_rn(rotated(lat + ls.kv_rank, i, positions[row]));
-    return;
-  }
+  const uint32_t tiles = (ls.kv_rank + kAbsorbTile - 1) / kAbsorbTile;
+  const uint32_t row0 = blockIdx.y * kRowTile, n = min(kRowTile, rows - row0), qd = ls.q_dim(), width = ls.kv_cols();
   const uint32_t head = blockIdx.x / tiles, r0 = (blockIdx.x % tiles) * kAbsorbTile;
   const uint32_t cols = min(kAbsorbTile, ls.kv_rank - r0);  // a multiple of 16
   for (uint32_t i = tid; i < ls.dim * (cols / 8); i += 128) {
@@ -217,33 +247,15 @@ latent_absorb_kernel(const float *__restrict__ partial, uint32_t splits, size_t 
     cp_async16(w_s + d * w_pitch + c * 16, w_uk + ((size_t)head * ls.dim + d) * ls.kv_rank + r0 + c * 8);
   }
   pdl_wait();
-  const uint32_t n = min(kRowTile, rows - row0);
-  for (uint32_t i = tid; i < kRowTile * (ls.dim / 2); i += 128) {
-    const uint32_t r = i / (ls.dim / 2), d = (i % (ls.dim / 2)) * 2;
-    uint32_t v = 0;
-    if (r < n) {
-      const uint32_t row = row_list[row0 + r];
-      if (kFold) {
-        const float *p = partial + (size_t)row * ls.cols() + head * qd + d;
-        float2 x = *reinterpret_cast<const float2 *>(p);
-        for (uint32_t s = 1; s < splits; ++s) {
-          const float2 y = *reinterpret_cast<const float2 *>(p + s * split_stride);
-          x.x += y.x, x.y += y.y;
-        }
-        v = pack_bf16x2(x.x, x.y);
-      } else {
-        v = *reinterpret_cast<const uint32_t *>(q + (size_t)row * ls.q_cols() + head * qd + d);
-      }
-    }
-    *reinterpret_cast<uint32_t *>(q_s + r * q_pitch + d * 2) = v;
+  const uint32_t groups = ls.dim / 8;
+  for (uint32_t i = tid; i < n * groups; i += 128)  // rows beyond n stay undefined and are not stored
+    cp_async16(q_s + (i / groups) * q_pitch + (i % groups) * 16, q + (size_t)row_list[row0 + i / groups] * ls.q_cols() + head * qd + (i % groups) * 8);
+  if (r0 == 0) {  // the rotated part goes along with the first tile
+    const uint32_t rg = ls.rot_dim / 8;
+    for (uint32_t i = tid; i < n * rg; i += 128)
+      *reinterpret_cast<uint4 *>(qa + ((size_t)(row0 + i / rg) * ls.heads + head) * width + ls.kv_rank + (i % rg) * 8) =
+          *reinterpret_cast<const uint4 *>(q + (size_t)row_list[row0 + i / rg] * ls.q_cols() + head * qd + ls.dim + (i % rg) * 8);
   }
-  if (r0 == 0)  // the rotated part goes along with the first tile
-    for (uint32_t i = tid; i < n * ls.rot_dim; i += 128) {
-      const uint32_t row = row_list[row0 + i / ls.rot_dim], d = i % ls.rot_dim;
-      bf16 *dst = qa + ((size_t)(row0 + i / ls.rot_dim) * ls.heads + head) * width + ls.kv_rank + d;
-      *dst = kFold ? __float2bfloat16_rn(rotated(partial + (size_t)row * ls.cols() + head * qd + ls.dim, d, positions[row]))
-                   : q[(size_t)row * ls.q_cols() + head * qd + ls.dim + d];
-    }
   cp_async_wait_all();
   __syncthreads();
   // warp = 16 latent columns (M), all 32 rows (four n-tiles)
@@ -278,14 +290,15 @@ latent_absorb_kernel(const float *__restrict__ partial, uint32_t splits, size_t 
 // of the 8 warps scores 32 of them over a quarter of the dimensions with its share of the queries held in
 // registers (keys on M, heads on N), the quarters are summed in shared memory, one group of eight lanes per
 // head keeps the running maximum and sum, and each warp then accumulates its own 16-wide slices of the weighted
-// latent. Cache rows come as one bulk copy per row, two tiles deep.
-constexpr uint32_t kTileKeys = 64, kDecThreads = 256, kDecStages = 2;
+// latent. The cache comes in whole blocks, one bulk copy each, two tiles deep; a row is an odd number of 16-byte
+// groups long (LatentShape::row_stride), so the fragments load without bank conflicts.
+constexpr uint32_t kTileKeys = 64, kCacheBlock = 16, kTileBlocks = kTileKeys / kCacheBlock, kDecThreads = 256, kDecStages = 2;
 constexpr uint32_t kScorePitch = kTileKeys + 8;  // floats
 constexpr uint32_t kProbPitch = kTileKeys + 8;   // bf16
 struct DecodeSmem {
   uint32_t pitch, ring, scores, probs, stats, bars, total;
-  __host__ __device__ DecodeSmem(uint32_t width, uint32_t heads) {
-    pitch = width * 2 + 16;  // an odd number of 16-byte groups: ldmatrix without bank conflicts
+  __host__ __device__ DecodeSmem(uint32_t row_stride, uint32_t heads) {
+    pitch = row_stride * 2;
     ring = 0;
     scores = ring + kDecStages * kTileKeys * pitch;
     probs = scores + 4 * heads * kScorePitch * 4;
@@ -303,7 +316,7 @@ latent_decode_kernel(const bf16 *__restrict__ qa, const bf16 *__restrict__ cache
   constexpr uint32_t kHeads = 8 * NT;
   extern __shared__ __align__(128) uint8_t smem[];
   const uint32_t width = ls.kv_cols();
-  const DecodeSmem lay(width, kHeads);
+  const DecodeSmem lay(ls.row_stride, kHeads);
   float *sS = reinterpret_cast<float *>(smem + lay.scores);
   uint8_t *sP = smem + lay.probs;
   float *sC = reinterpret_cast<float *>(smem + lay.stats);
@@ -313,23 +326,25 @@ latent_decode_kernel(const bf16 *__restrict__ qa, const bf16 *__restrict__ cache
   const uint32_t head0 = blockIdx.x * kHeads, item = blockIdx.y, split = blockIdx.z;
   const uint32_t row = row_list[item], pos = batch.query_positions[row], seq = batch.seq_of_row[row];
   const uint32_t *table = batch.tables_flat + batch.table_offsets[seq];
-  const uint32_t lo = ls.first_key(pos), all_tiles = (pos + 1 - lo + kTileKeys - 1) / kTileKeys;
+  // tiles start at block borders; keys before the window or past the row's own position are masked
+  const uint32_t lo = ls.first_key(pos), block0 = lo / kCacheBlock, last_block = pos / kCacheBlock;
+  const uint32_t all_tiles = (last_block - block0) / kTileBlocks + 1;
   const uint32_t per = (all_tiles + splits - 1) / splits;
   const uint32_t t_begin = min(split * per, all_tiles), ntiles = min(per, all_tiles - t_begin);
-  const uint32_t key0 = lo + t_begin * kTileKeys;
+  const uint32_t my_block0 = block0 + t_begin * kTileBlocks, key0 = my_block0 * kCacheBlock;
   if (tid < kDecStages) mbar_init(&full[tid], 1);
   mbar_fence_init();
   __syncthreads();
 
+  const uint32_t block_bytes = kCacheBlock * lay.pitch;
   auto issue = [&](uint32_t t) {  // warp 0
     uint64_t *bar = &full[t % kDecStages];
-    if (lane == 0) mbar_arrive_expect_tx(bar, kTileKeys * width * 2);
+    if (lane == 0) mbar_arrive_expect_tx(bar, kTileBlocks * block_bytes);
     __syncwarp();
-#pragma unroll
-    for (uint32_t i = lane; i < kTileKeys; i += 32) {
-      const uint32_t p = min(key0 + t * kTileKeys + i, pos);  // rows past the end repeat the last one and are masked
-      bulk_copy_g2s(smem + lay.ring + ((t % kDecStages) * kTileKeys + i) * lay.pitch,
-                    cache + ((size_t)table[p / ls.block_size] * ls.block_size + p % ls.block_size) * ls.row_stride, width * 2, bar);
+    if (lane < kTileBlocks) {  // blocks past the end repeat the last one and are masked
+      const uint32_t b = min(my_block0 + t * kTileBlocks + lane, last_block);
+      bulk_copy_g2s(smem + lay.ring + ((t % kDecStages) * kTileBlocks + lane) * block_bytes,
+                    cache + (size_t)table[b] * kCacheBlock * ls.row_stride, block_bytes, bar);
     }
   };
   // tiles that hold no row of this step are fetched before the kernel that writes those rows has finished
@@ -403,19 +418,19 @@ latent_decode_kernel(const bf16 *__restrict__ qa, const bf16 *__restrict__ cache
     }
     __syncthreads();
     if (scorer) {
-      const uint32_t left = pos + 1 - (key0 + t * kTileKeys);  // keys of this tile that exist
+      const uint32_t tile_key = key0 + t * kTileKeys;
       float v[kTileKeys / 8], tm = -INFINITY;
 #pragma unroll
       for (uint32_t i = 0; i < kTileKeys / 8; ++i) {
         const uint32_t key = i * 8 + sl;
         const float *p = sS + sh * kScorePitch + key;
         const float x = (p[0] + p[kHeads * kScorePitch]) + (p[2 * kHeads * kScorePitch] + p[3 * kHeads * kScorePitch]);
-        v[i] = key < left ? x * sl2 : -INFINITY;
+        v[i] = tile_key + key >= lo && tile_key + key <= pos ? x * sl2 : -INFINITY;
         tm = fmaxf(tm, v[i]);
       }
 #pragma unroll
       for (int off = 1; off < 8; off <<= 1) tm = fmaxf(tm, __shfl_xor_sync(0xffffffffu, tm, off));
-      const float nm = fmaxf(mx, tm), corr = fast_exp2(mx - nm);  // finite: the first key of a tile always exists
+      const float nm = fmaxf(mx, tm), corr = fast_exp2(mx - nm);  // finite: every tile holds a key that is seen
       float part = 0.f;
 #pragma unroll
       for (uint32_t i = 0; i < kTileKeys / 8; ++i) {
@@ -483,9 +498,9 @@ latent_decode_kernel(const bf16 *__restrict__ qa, const bf16 *__restrict__ cache
   }
 }
 
-// CTA (head and 64-wide tile of its values, tile of 32 listed rows): merged latents x W_uv, gated.
-constexpr uint32_t kValueTile = 64;
-__global__ void __launch_bounds__(128)
+// CTA (head and 64-wide tile of its values, tile of 16 listed rows): merged latents x W_uv, gated.
+constexpr uint32_t kValueTile = 64, kValueRows = 16, kValueThreads = 256;
+__global__ void __launch_bounds__(kValueThreads)
 latent_value_kernel(const float *__restrict__ part_o, const float *__restrict__ part_ml, uint32_t ctx_splits, const bf16 *__restrict__ w_uv,
                     const float *__restrict__ gate, uint32_t splits, size_t split_stride, const uint32_t *__restrict__ row_list,
                     uint32_t rows, bf16 *__restrict__ out, uint32_t ldo, LatentShape ls) {
@@ -495,64 +510,68 @@ latent_value_kernel(const float *__restrict__ part_o, const float *__restrict__ 
   pdl_trigger();
   const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const uint32_t tiles = (ls.value_dim + kValueTile - 1) / kValueTile;
-  const uint32_t head = blockIdx.x / tiles, v0 = (blockIdx.x % tiles) * kValueTile, row0 = blockIdx.y * kRowTile;
-  const uint32_t nv = min(kValueTile, ls.value_dim - v0), n = min(kRowTile, rows - row0), groups = ls.kv_rank / 8;
-  for (uint32_t i = tid; i < nv * groups; i += 128)
+  const uint32_t head = blockIdx.x / tiles, v0 = (blockIdx.x % tiles) * kValueTile, row0 = blockIdx.y * kValueRows;
+  const uint32_t nv = min(kValueTile, ls.value_dim - v0), n = min(kValueRows, rows - row0), groups = ls.kv_rank / 8;
+  for (uint32_t i = tid; i < nv * groups; i += kValueThreads)
     cp_async16(w_s + (i / groups) * pitch + (i % groups) * 16, w_uv + ((size_t)head * ls.value_dim + v0 + i / groups) * ls.kv_rank + (i % groups) * 8);
   pdl_wait();
-  for (uint32_t r = warp; r < kRowTile; r += 4) {  // one warp per row: merge its splits
-    const size_t base = ((size_t)(row0 + (r < n ? r : 0)) * ctx_splits) * ls.heads + head;
-    float mx = -INFINITY, total = 0.f;
-    for (uint32_t s = 0; s < ctx_splits; ++s) mx = fmaxf(mx, part_ml[(base + (size_t)s * ls.heads) * 2]);
-    for (uint32_t s = 0; s < ctx_splits; ++s) {
-      const float *ml = part_ml + (base + (size_t)s * ls.heads) * 2;
-      total += ml[0] == -INFINITY ? 0.f : fast_exp2(ml[0] - mx) * ml[1];
-    }
-    const float inv = r < n ? 1.0f / total : 0.f;
-    for (uint32_t d = lane * 4; d < ls.kv_rank; d += 128) {
+  for (uint32_t r = warp; r < n; r += kValueThreads / 32) {  // one warp per row: lane s weighs split s, then all sum
+    const size_t base = ((size_t)(row0 + r) * ctx_splits) * ls.heads + head;
+    float2 ml = make_float2(-INFINITY, 0.f);
+    if (lane < ctx_splits) ml = *reinterpret_cast<const float2 *>(part_ml + (base + (size_t)lane * ls.heads) * 2);
+    const float mx = warp_max(ml.x), e = ml.x == -INFINITY ? 0.f : fast_exp2(ml.x - mx);
+    const float wgt = e / warp_sum(e * ml.y);
+    for (uint32_t d0 = 0; d0 < ls.kv_rank; d0 += 128) {
+      const uint32_t d = d0 + lane * 4;
       float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-      for (uint32_t s = 0; s < ctx_splits; ++s) {
-        const size_t at = base + (size_t)s * ls.heads;
-        const float m = part_ml[at * 2], w = m == -INFINITY ? 0.f : fast_exp2(m - mx);
-        const float4 x = *reinterpret_cast<const float4 *>(part_o + at * ls.kv_rank + d);
-        a.x += w * x.x, a.y += w * x.y, a.z += w * x.z, a.w += w * x.w;
+      for (uint32_t s0 = 0; s0 < ctx_splits; s0 += 4) {
+        float4 x[4];
+#pragma unroll
+        for (uint32_t j = 0; j < 4; ++j)  // four independent loads in flight
+          x[j] = s0 + j < ctx_splits && d < ls.kv_rank
+                     ? *reinterpret_cast<const float4 *>(part_o + (base + (size_t)(s0 + j) * ls.heads) * ls.kv_rank + d)
+                     : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (uint32_t j = 0; j < 4; ++j) {
+          const float w = __shfl_sync(0xffffffffu, wgt, (s0 + j) & 31u);
+          if (s0 + j < ctx_splits) a.x += w * x[j].x, a.y += w * x[j].y, a.z += w * x[j].z, a.w += w * x[j].w;
+        }
       }
-      uint2 packed;
-      packed.x = pack_bf16x2(a.x * inv, a.y * inv);
-      packed.y = pack_bf16x2(a.z * inv, a.w * inv);
-      *reinterpret_cast<uint2 *>(o_s + r * pitch + d * 2) = packed;
+      if (d < ls.kv_rank) store4<bf16>(reinterpret_cast<bf16 *>(o_s + r * pitch) + d, a);
     }
   }
   cp_async_wait_all();
   __syncthreads();
-  if (warp * 16 >= nv) return;
-  float c[kRowTile / 8][4];
+  // warp = 16 values (M) x 8 rows (N); rows beyond n stay undefined and are not stored
+  const uint32_t vw = (warp & 3) * 16, rw = (warp >> 2) * 8;
+  if (vw >= nv || rw >= n) return;
+  // gate values of this thread's four results, in flight during the product
+  float g[4], c[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-  for (uint32_t t = 0; t < kRowTile / 8; ++t) c[t][0] = c[t][1] = c[t][2] = c[t][3] = 0.f;
+  for (uint32_t e = 0; e < 4; ++e) {
+    const uint32_t r = rw + (lane & 3) * 2 + (e & 1), v = v0 + vw + (lane >> 2) + (e >> 1) * 8;
+    g[e] = r < n && v < ls.value_dim
+               ? fold(gate + (size_t)row_list[row0 + r] * ls.cols() + ls.q_cols() + ls.kv_cols() + head * ls.value_dim + v, splits, split_stride)
+               : 0.f;
+  }
   const uint32_t mi = lane >> 3, rr = lane & 7;
-  const uint32_t wa = smem_u32(w_s) + (warp * 16 + rr + (mi & 1) * 8) * pitch + (mi >> 1) * 16;
-  const uint32_t ob = smem_u32(o_s) + (rr + (mi >> 1) * 8) * pitch + (mi & 1) * 16;
-  for (uint32_t k = 0; k < ls.kv_rank; k += 16) {
-    uint32_t a[4];
+  const uint32_t wa = smem_u32(w_s) + (vw + rr + (mi & 1) * 8) * pitch + (mi >> 1) * 16;
+  const uint32_t ob = smem_u32(o_s) + (rw + rr) * pitch + mi * 16;
+  for (uint32_t k = 0; k < ls.kv_rank; k += 32) {  // two steps of 16; the second may lie past the end
+    uint32_t a[4], b[4];
+    ldmatrix_x4(b, ob + k * 2);
     ldmatrix_x4(a, wa + k * 2);
-#pragma unroll
-    for (uint32_t t = 0; t < kRowTile / 16; ++t) {
-      uint32_t b[4];
-      ldmatrix_x4(b, ob + t * 16 * pitch + k * 2);
-      mma_bf16_16816(c[2 * t], a, b[0], b[1]);
-      mma_bf16_16816(c[2 * t + 1], a, b[2], b[3]);
+    mma_bf16_16816(c, a, b[0], b[1]);
+    if (k + 16 < ls.kv_rank) {
+      ldmatrix_x4(a, wa + k * 2 + 32);
+      mma_bf16_16816(c, a, b[2], b[3]);
     }
   }
 #pragma unroll
-  for (uint32_t t = 0; t < kRowTile / 8; ++t)
-#pragma unroll
-    for (uint32_t e = 0; e < 4; ++e) {
-      const uint32_t r = t * 8 + (lane & 3) * 2 + (e & 1), v = v0 + warp * 16 + (lane >> 2) + (e >> 1) * 8;
-      if (r >= n || v >= ls.value_dim) continue;
-      const uint32_t row = row_list[row0 + r], at = head * ls.value_dim + v;
-      const float g = fold(gate + (size_t)row * ls.cols() + ls.q_cols() + ls.kv_cols() + at, splits, split_stride);
-      out[(size_t)row * ldo + at] = __float2bfloat16_rn(c[t][e] * sigmoid_f(g));
-    }
+  for (uint32_t e = 0; e < 4; ++e) {
+    const uint32_t r = rw + (lane & 3) * 2 + (e & 1), v = v0 + vw + (lane >> 2) + (e >> 1) * 8;
+    if (r < n && v < ls.value_dim) out[(size_t)row_list[row0 + r] * ldo + head * ls.value_dim + v] = __float2bfloat16_rn(c[e] * sigmoid_f(g[e]));
+  }
 }
 
 inline int after_launch(const char *stage) {
@@ -568,6 +587,13 @@ int launch_latent_prepare(const float *partial, uint32_t splits, size_t split_st
                           const float *rope_sin, const uint32_t *positions, const uint32_t *slot_block, const uint32_t *slot_slot,
                           T *q, T *cache, LatentShape ls, uint32_t rows, cudaStream_t stream) {
   if (rows == 0) return ORION_OK;
+  if (ls.dim % 4 == 0 && ls.rot_dim % 4 == 0 && ls.rope_dims % 4 == 0 && ls.kv_rank % 4 == 0 && ls.out_cols() % 4 == 0 &&
+      ls.kv_cols() <= 4 * kPrepThreads) {
+    const dim3 grid(rows, 1 + (ls.q_cols() / 4 + kPrepThreads - 1) / kPrepThreads);
+    ORION_CUDA_CHECK("latent_prepare", launch_pdl(latent_prepare_vec_kernel<T>, grid, dim3(kPrepThreads), 0, stream, partial, splits,
+                                                  split_stride, norm_w, rope_cos, rope_sin, positions, slot_block, slot_slot, q, cache, ls));
+    return after_launch("latent_prepare");
+  }
   ORION_CUDA_CHECK("latent_prepare", launch_pdl(latent_prepare_kernel<T>, dim3(rows), dim3(kPrepThreads), 0, stream, partial, splits,
                                                 split_stride, norm_w, rope_cos, rope_sin, positions, slot_block, slot_slot, q, cache, ls));
   return after_launch("latent_prepare");
@@ -589,7 +615,7 @@ int launch_latent_attention_generic(const T *q, const T *cache, const T *w_uk, c
 
 bool latent_decode_supported(LatentShape ls) {
   return ls.kv_rank % 16 == 0 && ls.kv_rank <= 512 && ls.rot_dim % 16 == 0 && ls.dim % 16 == 0 && ls.dim > 0 && ls.dim <= 512 &&
-         ls.kv_cols() <= 640 && ls.cols() % 2 == 0 && ls.kv_cols() == ls.row_stride;
+         ls.kv_cols() <= 640 && ls.block_size == kCacheBlock && ls.row_stride % 16 == 8 && ls.row_stride >= ls.kv_cols();
 }
 
 namespace {
@@ -601,7 +627,7 @@ uint32_t latent_decode_splits(LatentShape ls, uint32_t rows, uint32_t max_positi
   const uint32_t keys = ls.window ? std::min(ls.window, max_position + 1) : max_position + 1;
   const uint32_t tiles = (keys + kTileKeys - 1) / kTileKeys;
   // one resident wave of CTAs, as far as there are tiles to hand out
-  const uint32_t resident = std::max(1u, std::min(8u, 227u * 1024u / (DecodeSmem(ls.kv_cols(), 8 * nt).total + 1024u)));
+  const uint32_t resident = std::max(1u, std::min(8u, 227u * 1024u / (DecodeSmem(ls.row_stride, 8 * nt).total + 1024u)));
   const uint32_t want = 148 * resident / std::max(1u, rows * groups);
   return std::max(1u, std::min({want, tiles, kLatentMaxSplits}));
 }
@@ -610,22 +636,16 @@ size_t latent_decode_scratch_floats(LatentShape ls, uint32_t rows, uint32_t spli
   return (size_t)rows * splits * ls.heads * (ls.kv_rank + 2);
 }
 
-int launch_latent_absorb(const float *partial, uint32_t splits, size_t split_stride, const bf16 *q, const bf16 *w_uk, const float *norm_w,
-                         const float *rope_cos, const float *rope_sin, const uint32_t *positions, const uint32_t *slot_block,
-                         const uint32_t *slot_slot, const uint32_t *row_list, uint32_t rows, bf16 *cache, bf16 *qa, LatentShape ls,
+int launch_latent_absorb(const bf16 *q, const bf16 *w_uk, const uint32_t *row_list, uint32_t rows, bf16 *qa, LatentShape ls,
                          cudaStream_t stream) {
   if (rows == 0) return ORION_OK;
   if (!latent_decode_supported(ls)) return set_error(ORION_ERR_INTERNAL, "latent decode attention does not cover this shape");
   const uint32_t tiles = (ls.kv_rank + kAbsorbTile - 1) / kAbsorbTile;
   const uint32_t smem = ls.dim * (kAbsorbTile * 2 + 16) + kRowTile * (ls.dim * 2 + 16);
-  const dim3 grid(ls.heads * tiles + (q ? 0 : kRowTile / 4), (rows + kRowTile - 1) / kRowTile);
-  static bool set_f[kMaxDeviceOrdinals] = {}, set_q[kMaxDeviceOrdinals] = {};
-  constexpr int kMost = 512 * (kAbsorbTile * 2 + 16) + kRowTile * (512 * 2 + 16);
-  ORION_CUDA_CHECK("latent_absorb attr", q ? ensure_dynamic_smem(latent_absorb_kernel<false>, kMost, set_q)
-                                           : ensure_dynamic_smem(latent_absorb_kernel<true>, kMost, set_f));
-  ORION_CUDA_CHECK("latent_absorb", launch_pdl(q ? latent_absorb_kernel<false> : latent_absorb_kernel<true>, grid, dim3(128), smem, stream,
-                                               partial, splits, split_stride, q, w_uk, norm_w, rope_cos, rope_sin, positions, slot_block,
-                                               slot_slot, row_list, rows, cache, qa, ls));
+  static bool attr_set[kMaxDeviceOrdinals] = {};
+  ORION_CUDA_CHECK("latent_absorb attr", ensure_dynamic_smem(latent_absorb_kernel, 512 * (kAbsorbTile * 2 + 16) + kRowTile * (512 * 2 + 16), attr_set));
+  ORION_CUDA_CHECK("latent_absorb", launch_pdl(latent_absorb_kernel, dim3(ls.heads * tiles, (rows + kRowTile - 1) / kRowTile), dim3(128), smem,
+                                               stream, q, w_uk, row_list, rows, qa, ls));
   return after_launch("latent_absorb");
 }
 
@@ -633,7 +653,7 @@ namespace {
 template <int NT, int KQ, int MT>
 int launch_decode(const bf16 *qa, const bf16 *cache, const uint32_t *row_list, const uint32_t *first_row, uint32_t rows, AttnBatch batch,
                   uint32_t splits, float *part_o, float *part_ml, LatentShape ls, cudaStream_t stream) {
-  const DecodeSmem lay(ls.kv_cols(), 8 * NT);
+  const DecodeSmem lay(ls.row_stride, 8 * NT);
   static bool attr_set[kMaxDeviceOrdinals] = {};
   ORION_CUDA_CHECK("latent_decode attr", ensure_dynamic_smem(latent_decode_kernel<NT, KQ, MT>, 227 * 1024, attr_set));
   ORION_CUDA_CHECK("latent_decode", launch_pdl(latent_decode_kernel<NT, KQ, MT>, dim3((ls.heads + 8 * NT - 1) / (8 * NT), rows, splits),
@@ -661,11 +681,11 @@ int launch_latent_decode(const bf16 *qa, const bf16 *cache, const bf16 *w_uv, co
     case 2: ORION_TRY(launch_decode_nt<2>(qa, cache, row_list, first_row, rows, batch, splits, part_o, part_ml, ls, stream)); break;
     default: ORION_TRY(launch_decode_nt<4>(qa, cache, row_list, first_row, rows, batch, splits, part_o, part_ml, ls, stream)); break;
   }
-  const uint32_t smem = (kValueTile + kRowTile) * (ls.kv_rank * 2 + 16);
+  const uint32_t smem = (kValueTile + kValueRows) * (ls.kv_rank * 2 + 16) + 32;
   static bool attr_set[kMaxDeviceOrdinals] = {};
-  ORION_CUDA_CHECK("latent_value attr", ensure_dynamic_smem(latent_value_kernel, (int)((kValueTile + kRowTile) * (512 * 2 + 16)), attr_set));
-  const dim3 grid(ls.heads * ((ls.value_dim + kValueTile - 1) / kValueTile), (rows + kRowTile - 1) / kRowTile);
-  ORION_CUDA_CHECK("latent_value", launch_pdl(latent_value_kernel, grid, dim3(128), smem, stream, part_o, part_ml, splits, w_uv, gate_partial,
+  ORION_CUDA_CHECK("latent_value attr", ensure_dynamic_smem(latent_value_kernel, (int)((kValueTile + kValueRows) * (512 * 2 + 16) + 32), attr_set));
+  const dim3 grid(ls.heads * ((ls.value_dim + kValueTile - 1) / kValueTile), (rows + kValueRows - 1) / kValueRows);
+  ORION_CUDA_CHECK("latent_value", launch_pdl(latent_value_kernel, grid, dim3(kValueThreads), smem, stream, part_o, part_ml, splits, w_uv, gate_partial,
                                               gate_splits, split_stride, row_list, rows, out, ldo, ls));
   return after_launch("latent_value");
 }

@@ -16,6 +16,9 @@ namespace orion {
 namespace {
 
 constexpr uint32_t pad8(uint32_t n) { return (n + 7) / 8 * 8; }
+// The same, to an odd number of groups of 8 (rows that follow one another in shared memory then start in
+// different banks).
+constexpr uint32_t odd_groups(uint32_t n) { return pad8(n) / 8 % 2 ? pad8(n) : pad8(n) + 8; }
 
 template <typename T>
 class LayeredModel final : public StepModel<T> {
@@ -67,7 +70,7 @@ class LayeredModel final : public StepModel<T> {
     float *vec = nullptr;
     uint64_t rows = 0, cols = 0, ld = 0;
     uint32_t index = 0;
-    bool matrix = true;
+    bool matrix = true, transposed = false;  // transposed: kept as [cols][rows]
   };
   bool place(const std::string &name, Place *p) const;
   std::vector<std::string> tensor_names() const;
@@ -174,7 +177,7 @@ int LayeredModel<T>::init() {
     ORION_TRY(zeroed(&L.conv_state, copies * keep * H));
     if (L.attention()) {
       L.ls = LatentShape{s.heads, s.dim, s.rot_dim, s.value_dim, s.kv_rank, s.window, s.rope_dims, d.block_size,
-                         pad8(s.kv_rank + s.rot_dim), (float)s.scale, (float)d.norm_eps};
+                         odd_groups(s.kv_rank + s.rot_dim), (float)s.scale, (float)d.norm_eps};
       L.mix_in = L.ls.cols(), L.mix_out = L.ls.out_cols();
       ORION_TRY(alloc(&L.latent_norm, s.kv_rank));
       ORION_TRY(alloc(&L.w_uk, (size_t)s.heads * s.dim * s.kv_rank));
@@ -251,6 +254,10 @@ bool LayeredModel<T>::place(const std::string &name, Place *p) const {
     p->dst = dst, p->rows = rows, p->cols = cols, p->ld = ld ? ld : cols, p->matrix = true;
     return rows > 0;
   };
+  auto filters = [&](T *dst) {
+    p->transposed = true;
+    return matrix(dst, H, d_.conv_taps);
+  };
   auto vector = [&](float *dst, uint64_t n) {
     p->vec = dst, p->rows = 1, p->cols = n, p->matrix = false;
     return n > 0;
@@ -265,9 +272,9 @@ bool LayeredModel<T>::place(const std::string &name, Place *p) const {
   const OrionLayerDesc &s = L.d;
   p->index = i;
   if (rest == "norm1") return vector(L.norm, H);
-  if (rest == "canon1") return matrix(L.conv1, H, d_.conv_taps);
+  if (rest == "canon1") return filters(L.conv1);
   if (s.ffn_dim) {
-    if (rest == "canon2") return matrix(L.conv2, H, d_.conv_taps);
+    if (rest == "canon2") return filters(L.conv2);
     if (rest == "mlp.up") return matrix(L.w_up, s.ffn_dim, H);
     if (rest == "mlp.down") return matrix(L.w_out + L.ff_at, H, s.ffn_dim, L.cat);
   }
@@ -316,13 +323,15 @@ int LayeredModel<T>::load_tensor(const char *name, int dtype, const uint64_t *sh
   finalized_ = false;
   if (!p.matrix) {
     ORION_TRY(upload_slice(nullptr, p.vec, data, dtype, C, 0, 1, 0, C));
-  } else if (p.ld == C) {
+  } else if (p.ld == C && !p.transposed) {
     ORION_TRY(upload_slice(p.dst, nullptr, data, dtype, C, 0, R, 0, C));
-  } else {  // a column block of a wider matrix
+  } else {  // a column block of a wider matrix, or filters
     T *tmp = nullptr;
     ORION_CUDA_CHECK("allocate staging", cudaMalloc(&tmp, R * C * sizeof(T)));
     int rc = upload_slice(tmp, nullptr, data, dtype, C, 0, R, 0, C);
-    if (rc == ORION_OK) rc = launch_copy_rows_strided<T>(tmp, p.dst, R, C, p.ld, stream_);
+    if (rc == ORION_OK)
+      rc = p.transposed ? launch_transpose<T>(tmp, p.dst, (uint32_t)R, (uint32_t)C, stream_)
+                        : launch_copy_rows_strided<T>(tmp, p.dst, R, C, p.ld, stream_);
     const cudaError_t e = cudaStreamSynchronize(stream_);
     cudaFree(tmp);
     ORION_TRY(rc);
@@ -434,22 +443,19 @@ int LayeredModel<T>::mixer(const Layer &L, const StateBatch &sb, const AttnBatch
   ORION_TRY(timed(kProfGemm, [&] { return launch_gemm<T>(conv_m_, H, L.w_mix, H, partial_, Tn, L.mix_in, H, p, stream_); }));
   if (!L.attention())
     return timed(kProfAttention, [&] { return launch_min_gru<T>(partial_, p.out_slabs, slab, L.mix_bias, L.rec_state, sb, cat_, L.cat, L.d.width, stream_); });
+  ORION_TRY(timed(kProfAttention, [&] {
+    return launch_latent_prepare<T>(partial_, p.out_slabs, slab, L.latent_norm, L.rope_cos, L.rope_sin, ab.query_positions,
+                                    d_meta_ + meta_.slot_block, d_meta_ + meta_.slot_slot, qbuf_, L.cache, L.ls, Tn, stream_);
+  }));
   if constexpr (DTypeOf<T>::is_bf16) {
     if (tuned(L) && few_rows_ == Tn) {
       const uint32_t *first = d_meta_ + meta_.extra, *few = first + 3 * meta_.seqs + 1, sp = context_splits(L, Tn);
-      ORION_TRY(timed(kProfAttention, [&] {
-        return launch_latent_absorb(partial_, p.out_slabs, slab, nullptr, L.w_uk, L.latent_norm, L.rope_cos, L.rope_sin, ab.query_positions,
-                                    d_meta_ + meta_.slot_block, d_meta_ + meta_.slot_slot, few, Tn, L.cache, qa_, L.ls, stream_);
-      }));
+      ORION_TRY(timed(kProfAttention, [&] { return launch_latent_absorb(qbuf_, L.w_uk, few, Tn, qa_, L.ls, stream_); }));
       return timed(kProfAttention, [&] {
         return launch_latent_decode(qa_, L.cache, L.w_uv, partial_, p.out_slabs, slab, few, first, Tn, ab, sp, scratch_, L.ls, cat_, L.cat, stream_);
       });
     }
   }
-  ORION_TRY(timed(kProfAttention, [&] {
-    return launch_latent_prepare<T>(partial_, p.out_slabs, slab, L.latent_norm, L.rope_cos, L.rope_sin, ab.query_positions,
-                                    d_meta_ + meta_.slot_block, d_meta_ + meta_.slot_slot, qbuf_, L.cache, L.ls, Tn, stream_);
-  }));
   return timed(kProfAttention, [&] {
     return launch_latent_attention_generic<T>(qbuf_, L.cache, L.w_uk, L.w_uv, partial_, p.out_slabs, slab, L.ls, ab, cat_, L.cat, stream_);
   });
