@@ -304,6 +304,27 @@ int launch_latent_decode(const bf16 *qa, const bf16 *cache, const bf16 *w_uv, co
                          uint32_t splits, float *scratch, LatentShape ls, bf16 *out, uint32_t ldo, cudaStream_t stream);
 int latent_poll_error(uint32_t *code);
 
+// Tuned path for prompt portions (bf16; dim, rot_dim and value_dim multiples of 16): keys and values are expanded once
+// per token. A portion's rows in the expanded buffers cover its own tokens and those before it that a window reaches.
+struct LatentPortion {
+  uint32_t seq, row, position, count;  // sequence; first expanded row, the position it stands for, number of rows
+};
+struct LatentTile {
+  uint32_t row_start, num_rows, position;  // batch rows of one sequence, position of the first
+  int32_t row_of_zero;                     // expanded row that position 0 of the sequence would have
+};
+constexpr uint32_t kLatentTileRows = 128;
+bool latent_prefill_supported(LatentShape ls);
+// Cached latents [rows][kv_rank] and rotated parts [rows][rot_dim] of the portions.
+int launch_latent_gather(const bf16 *cache, const uint32_t *tables_flat, const uint32_t *table_offsets, const LatentPortion *portions,
+                         uint32_t num_portions, uint32_t longest, bf16 *latents, bf16 *rotated, LatentShape ls, cudaStream_t stream);
+// `expanded`: [rows][heads * dim | heads * value_dim], the latents times W_uk and W_uv. The buffers hold
+// `rows_capacity` rows of finite values.
+int launch_latent_prefill(const bf16 *q, const bf16 *expanded, const bf16 *rotated, uint32_t rows_capacity, const float *gate_partial,
+                          uint32_t splits, size_t split_stride, const LatentTile *tiles, uint32_t num_tiles, LatentShape ls, bf16 *out,
+                          uint32_t ldo, cudaStream_t stream);
+int latent_prefill_poll_error(uint32_t *code);
+
 // ---- tensor-parallel hand-over ---------------------------------------------------
 
 constexpr int kMaxTpWorld = 8;

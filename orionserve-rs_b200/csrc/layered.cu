@@ -38,6 +38,13 @@ class LayeredModel final : public StepModel<T> {
     desc_.max_batch_tokens = d.max_batch_tokens, desc_.max_batch_sequences = d.max_batch_sequences, desc_.tp_world = 1;
   }
 
+  ~LayeredModel() override {
+    cudaSetDevice(ordinal_);
+    if (stream_) cudaStreamSynchronize(stream_);
+    for (T *p : {ext_latents_, ext_rot_, ext_kv_})
+      if (p) cudaFree(p);
+  }
+
   int init();
   int load_tensor(const char *name, int dtype, const uint64_t *shape, int ndim, const void *data) override;
   bool uses_tensor(const char *name) const override {
@@ -96,11 +103,15 @@ class LayeredModel final : public StepModel<T> {
     ORION_TRY(Base::poll_errors());
     uint32_t code = 0;
     if (DTypeOf<T>::is_bf16) ORION_TRY(latent_poll_error(&code));
+    if (DTypeOf<T>::is_bf16 && !code) ORION_TRY(latent_prefill_poll_error(&code));
     if (code) return set_error(ORION_ERR_BACKEND, "backend cuda failed at latent attention: a bounded pipeline wait ran out (code %u)", code);
     return ORION_OK;
   }
   // Sequences with at most this many rows in a batch decode: each row reads the cache by itself.
   static constexpr uint32_t kFewRows = 8;
+  size_t tile_words(uint64_t seqs, uint64_t rows) const override { return 4 * (2 * seqs + rows / kLatentTileRows + 1); }
+  int fill_tiles(const BatchView &b, uint32_t *t, typename Base::Meta &mt) override;
+  bool expands(const Layer &L) const { return DTypeOf<T>::is_bf16 && L.attention() && latent_prefill_supported(L.ls); }
   bool tuned(const Layer &L) const { return DTypeOf<T>::is_bf16 && L.attention() && latent_decode_supported(L.ls); }
   uint32_t context_splits(const Layer &L, uint32_t rows) const {
     uint32_t s = latent_decode_splits(L.ls, rows, meta_.max_position);
@@ -126,6 +137,9 @@ class LayeredModel final : public StepModel<T> {
   float *scratch_ = nullptr;  // their weighted latents per context split
   size_t scratch_floats_ = 0;
   uint32_t few_rows_ = 0;     // rows of this batch that decode
+  // Prompt portions of this batch (their descriptions follow the tiles in the batch metadata) and the expanded rows.
+  uint32_t portions_ = 0, longest_ = 0, ext_rows_ = 0, ext_cap_ = 0;
+  T *ext_latents_ = nullptr, *ext_rot_ = nullptr, *ext_kv_ = nullptr;
   struct Rope {
     double base;
     uint32_t dims;
@@ -180,8 +194,8 @@ int LayeredModel<T>::init() {
                          odd_groups(s.kv_rank + s.rot_dim), (float)s.scale, (float)d.norm_eps};
       L.mix_in = L.ls.cols(), L.mix_out = L.ls.out_cols();
       ORION_TRY(alloc(&L.latent_norm, s.kv_rank));
-      ORION_TRY(alloc(&L.w_uk, (size_t)s.heads * s.dim * s.kv_rank));
-      ORION_TRY(alloc(&L.w_uv, (size_t)s.heads * s.value_dim * s.kv_rank));
+      ORION_TRY(alloc(&L.w_uk, (size_t)s.heads * (s.dim + s.value_dim) * s.kv_rank));  // one matrix for the expansion of prompts
+      L.w_uv = L.w_uk + (size_t)s.heads * s.dim * s.kv_rank;
       ORION_TRY(zeroed(&L.cache, (size_t)d.num_blocks * d.block_size * L.ls.row_stride));
       qcols = std::max(qcols, (size_t)L.ls.q_cols());
       const Rope *r = nullptr;
@@ -409,7 +423,7 @@ void LayeredModel<T>::fill_extra(const BatchView &b, uint32_t *w) {
   const uint64_t S = b.num_sequences;
   uint32_t *first = w, *read = w + S + 1, *write = read + S, *few = write + S;
   uint64_t row = 0;
-  few_rows_ = 0;
+  few_rows_ = portions_ = 0;
   for (uint64_t s = 0; s < S; ++s) {
     const uint32_t slot = b.state_slots[s], copy = slots_[slot].copy;
     first[s] = (uint32_t)row;
@@ -420,6 +434,55 @@ void LayeredModel<T>::fill_extra(const BatchView &b, uint32_t *w) {
     row += b.slot_token_counts[s];
   }
   first[S] = (uint32_t)row;
+}
+
+// Portions and tiles of the sequences that bring more than a few rows, and room for their expanded rows.
+template <typename T>
+int LayeredModel<T>::fill_tiles(const BatchView &b, uint32_t *t, typename Base::Meta &mt) {
+  uint64_t reach = 0, wide = 0, rank = 0, rot = 0;  // tokens before a portion that some window reaches; buffer widths
+  bool any = false;
+  for (const Layer &L : layers_) {
+    if (!expands(L)) continue;
+    any = true;
+    reach = std::max(reach, L.d.window ? (uint64_t)L.d.window - 1 : UINT64_MAX);
+    wide = std::max(wide, (uint64_t)L.d.heads * (L.d.dim + L.d.value_dim));
+    rank = std::max(rank, (uint64_t)L.d.kv_rank);
+    rot = std::max(rot, (uint64_t)L.d.rot_dim);
+  }
+  if (!any) return ORION_OK;
+  auto *portions = reinterpret_cast<LatentPortion *>(t);
+  auto *tiles = reinterpret_cast<LatentTile *>(t + 4 * b.num_sequences);
+  uint64_t row = 0, ext = 0;
+  longest_ = 0;
+  for (uint64_t s = 0; s < b.num_sequences; ++s) {
+    const uint64_t n = b.slot_token_counts[s];
+    if (n > kFewRows) {
+      const uint64_t start = b.positions[row], before = std::min(start, reach);
+      if (ext + before + n > INT32_MAX) return set_error(ORION_ERR_INVALID_REQUEST, "prompt portions reach too many tokens");
+      portions[portions_++] = LatentPortion{(uint32_t)s, (uint32_t)ext, (uint32_t)(start - before), (uint32_t)(before + n)};
+      longest_ = std::max(longest_, (uint32_t)(before + n));
+      for (uint64_t i = 0; i < n; i += kLatentTileRows)
+        tiles[mt.num_tiles++] = LatentTile{(uint32_t)(row + i), (uint32_t)std::min<uint64_t>(kLatentTileRows, n - i), (uint32_t)(start + i),
+                                           (int32_t)((int64_t)(ext + before) - (int64_t)start)};
+      ext += before + n;
+    }
+    row += n;
+  }
+  ext_rows_ = (uint32_t)ext;
+  if (ext > ext_cap_) {
+    uint64_t cap = 1024;
+    while (cap < ext) cap *= 2;
+    ext_cap_ = 0;
+    for (auto [buf, width] : {std::make_pair(&ext_latents_, rank), std::make_pair(&ext_rot_, rot), std::make_pair(&ext_kv_, wide)}) {
+      if (*buf) cudaFree(*buf);  // the previous step has ended
+      *buf = nullptr;
+      const size_t bytes = std::max<size_t>(1, cap * width) * sizeof(T);
+      ORION_CUDA_CHECK("allocate expanded rows", cudaMalloc(buf, bytes));
+      ORION_CUDA_CHECK("allocate expanded rows", cudaMemsetAsync(*buf, 0, bytes, stream_));  // masked keys must be finite
+    }
+    ext_cap_ = (uint32_t)cap;
+  }
+  return ORION_OK;
 }
 
 template <typename T>
@@ -448,12 +511,32 @@ int LayeredModel<T>::mixer(const Layer &L, const StateBatch &sb, const AttnBatch
                                     d_meta_ + meta_.slot_block, d_meta_ + meta_.slot_slot, qbuf_, L.cache, L.ls, Tn, stream_);
   }));
   if constexpr (DTypeOf<T>::is_bf16) {
-    if (tuned(L) && few_rows_ == Tn) {
-      const uint32_t *first = d_meta_ + meta_.extra, *few = first + 3 * meta_.seqs + 1, sp = context_splits(L, Tn);
-      ORION_TRY(timed(kProfAttention, [&] { return launch_latent_absorb(qbuf_, L.w_uk, few, Tn, qa_, L.ls, stream_); }));
-      return timed(kProfAttention, [&] {
-        return launch_latent_decode(qa_, L.cache, L.w_uv, partial_, p.out_slabs, slab, few, first, Tn, ab, sp, scratch_, L.ls, cat_, L.cat, stream_);
-      });
+    if ((few_rows_ == 0 || tuned(L)) && (few_rows_ == Tn || expands(L))) {
+      const uint32_t *first = d_meta_ + meta_.extra, *few = first + 3 * meta_.seqs + 1;
+      if (few_rows_ > 0) {
+        const uint32_t sp = context_splits(L, few_rows_);
+        ORION_TRY(timed(kProfAttention, [&] { return launch_latent_absorb(qbuf_, L.w_uk, few, few_rows_, qa_, L.ls, stream_); }));
+        ORION_TRY(timed(kProfAttention, [&] {
+          return launch_latent_decode(qa_, L.cache, L.w_uv, partial_, p.out_slabs, slab, few, first, few_rows_, ab, sp, scratch_, L.ls, cat_,
+                                      L.cat, stream_);
+        }));
+      }
+      if (portions_ > 0) {
+        const auto *portions = reinterpret_cast<const LatentPortion *>(d_meta_ + meta_.tiles);
+        const auto *tiles = reinterpret_cast<const LatentTile *>(d_meta_ + meta_.tiles + 4 * meta_.seqs);
+        const uint32_t wide = L.d.heads * (L.d.dim + L.d.value_dim);
+        ORION_TRY(timed(kProfAttention, [&] {
+          return launch_latent_gather(L.cache, ab.tables_flat, ab.table_offsets, portions, portions_, longest_, ext_latents_, ext_rot_, L.ls, stream_);
+        }));
+        ORION_TRY(timed(kProfGemm, [&] {
+          return launch_gemm_act(ext_latents_, L.d.kv_rank, L.w_uk, L.d.kv_rank, ext_kv_, wide, ext_rows_, wide, L.d.kv_rank, kGemmStore, stream_);
+        }));
+        ORION_TRY(timed(kProfAttention, [&] {
+          return launch_latent_prefill(qbuf_, ext_kv_, ext_rot_, ext_cap_, partial_, p.out_slabs, slab, tiles, meta_.num_tiles, L.ls, cat_, L.cat,
+                                       stream_);
+        }));
+      }
+      return ORION_OK;
     }
   }
   return timed(kProfAttention, [&] {

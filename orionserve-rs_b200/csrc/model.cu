@@ -109,10 +109,14 @@ class Model final : public StepModel<T> {
   }
   bool leader() const override { return d_.tp_world <= 1 || d_.tp_rank == 0; }
   bool out_rows_fixed() const override { return d_.tp_world > 1; }
-  uint32_t prefill_tile_rows() const override {
+  uint32_t prefill_tile_rows() const {
     return DTypeOf<T>::is_bf16 && prefill_attention_supported(kv_, lq_) ? prefill_tile_positions(lq_, lkv_) : 0;
   }
-  bool decode_rows_apart() const override { return decode_attention_supported(kv_, lq_); }
+  size_t tile_words(uint64_t seqs, uint64_t rows) const override {
+    const uint32_t tile_rows = prefill_tile_rows();
+    return tile_rows ? 4 * (seqs + rows / tile_rows + 1) : 0;
+  }
+  int fill_tiles(const BatchView &b, uint32_t *t, typename Base::Meta &mt) override;
   int poll_errors() override {
     uint32_t code = 0;
     if (nccl_) {
@@ -391,6 +395,44 @@ int Model<T>::setup_head_peers() {
     head_flags_ = static_cast<uint32_t *>(p);
   }
   return nccl_->barrier(stream_);  // nobody starts a step before every mapping exists
+}
+
+template <typename T>
+int Model<T>::fill_tiles(const BatchView &b, uint32_t *t, typename Base::Meta &mt) {
+  const uint32_t tile_rows = prefill_tile_rows();
+  const uint64_t S = b.num_sequences, Tn = b.num_tokens;
+  if (tile_rows == 0) return ORION_OK;
+  if (decode_attention_supported(kv_, lq_)) {
+    uint64_t head = 0, tail = 0;
+    while (head < S && b.slot_token_counts[head] == 1) ++head;
+    while (tail < S && b.slot_token_counts[S - 1 - tail] == 1) ++tail;
+    if (std::max(head, tail) >= 8) {  // worth a launch of its own
+      mt.dec_rows = (uint32_t)std::max(head, tail);
+      mt.dec_row0 = head >= tail ? 0u : (uint32_t)(Tn - tail);
+    }
+  }
+  // Tiles of consecutive rows of one sequence for the prefill attention kernel.
+  uint64_t row = 0;
+  for (uint64_t s = 0; s < S; ++s) {
+    const uint64_t end = row + b.slot_token_counts[s];
+    if (row >= mt.dec_row0 && row < (uint64_t)mt.dec_row0 + mt.dec_rows) {  // a decode row: no tile
+      row = end;
+      continue;
+    }
+    while (row < end) {
+      const uint32_t n = (uint32_t)std::min<uint64_t>(tile_rows, end - row);
+      uint32_t max_pos = 0;
+      for (uint32_t i = 0; i < n; ++i) max_pos = std::max(max_pos, b.positions[row + i]);
+      t[0] = (uint32_t)row;
+      t[1] = n;
+      t[2] = (uint32_t)s;
+      t[3] = max_pos;
+      t += 4;
+      ++mt.num_tiles;
+      row += n;
+    }
+  }
+  return ORION_OK;
 }
 
 template <typename T>

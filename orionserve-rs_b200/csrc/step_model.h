@@ -78,9 +78,11 @@ class StepModel : public ModelBase {
   virtual void graph_plan(uint32_t *splits, uint32_t *blocks_per_split) const = 0;
   // Model-specific batch checks (before anything is launched), after the shared ones.
   virtual int check_batch(const BatchView &) { return ORION_OK; }
-  // Rows per prefill attention tile (0: the model uses no tiles) and whether runs of decode rows get no tile.
-  virtual uint32_t prefill_tile_rows() const { return 0; }
-  virtual bool decode_rows_apart() const { return false; }
+  // Description of the batch's prompt portions for the prefill attention kernel; called for batches that are not
+  // all single rows, before anything is launched. May use at most tile_words words at `t`.
+  struct Meta;
+  virtual size_t tile_words(uint64_t seqs, uint64_t rows) const { return 0; }
+  virtual int fill_tiles(const BatchView &, uint32_t *t, Meta &) { return ORION_OK; }
   // Words of model-specific batch description; their number may depend on the sequence count only.
   virtual size_t extra_words(uint64_t) const { return 0; }
   virtual void fill_extra(const BatchView &, uint32_t *) {}
@@ -473,9 +475,7 @@ int StepModel<T>::forward(const BatchView &b, float *logits_out, uint64_t logits
   mt.extra = mt.offsets + S + 1;
   mt.tables = mt.extra + extra_words(S);
   mt.tiles = mt.tables + table_entries;
-  const uint32_t tile_rows = prefill_tile_rows();
-  const size_t max_tiles = tile_rows ? S + Tn / tile_rows + 1 : 0;
-  mt.total = mt.tiles + 4 * max_tiles;
+  mt.total = mt.tiles + tile_words(S, Tn);
   if (table_entries > UINT32_MAX) return set_error(ORION_ERR_INVALID_REQUEST, "block tables too large");
   if (mt.total > meta_cap_) {
     const size_t cap = mt.total * 2 + 1024;
@@ -545,39 +545,7 @@ int StepModel<T>::forward(const BatchView &b, float *logits_out, uint64_t logits
   if (table_entries) std::memcpy(h + mt.tables, b.block_tables_flat, table_entries * sizeof(uint32_t));
   fill_extra(b, h + mt.extra);
   mt.decode = all_single;
-  if (tile_rows && !all_single) {
-    if (decode_rows_apart()) {
-      uint64_t head = 0, tail = 0;
-      while (head < S && b.slot_token_counts[head] == 1) ++head;
-      while (tail < S && b.slot_token_counts[S - 1 - tail] == 1) ++tail;
-      if (std::max(head, tail) >= 8) {  // worth a launch of its own
-        mt.dec_rows = (uint32_t)std::max(head, tail);
-        mt.dec_row0 = head >= tail ? 0u : (uint32_t)(Tn - tail);
-      }
-    }
-    // Tiles of consecutive rows of one sequence for the prefill attention kernel.
-    uint32_t *t = h + mt.tiles;
-    uint64_t row = 0;
-    for (uint64_t s = 0; s < S; ++s) {
-      const uint64_t end = row + b.slot_token_counts[s];
-      if (row >= mt.dec_row0 && row < (uint64_t)mt.dec_row0 + mt.dec_rows) {  // a decode row: no tile
-        row = end;
-        continue;
-      }
-      while (row < end) {
-        const uint32_t n = (uint32_t)std::min<uint64_t>(tile_rows, end - row);
-        uint32_t max_pos = 0;
-        for (uint32_t i = 0; i < n; ++i) max_pos = std::max(max_pos, b.positions[row + i]);
-        t[0] = (uint32_t)row;
-        t[1] = n;
-        t[2] = (uint32_t)s;
-        t[3] = max_pos;
-        t += 4;
-        ++mt.num_tiles;
-        row += n;
-      }
-    }
-  }
+  if (!all_single) ORION_TRY(fill_tiles(b, h + mt.tiles, mt));
   meta_ = mt;
 
   g_launch_count = 0;
