@@ -116,14 +116,22 @@ __device__ __forceinline__ float from_f32<float>(float v) { return v; }
 template <>
 __device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __float2bfloat16_rn(v); }
 
-// GELU in its tanh form.
-__device__ __forceinline__ float gelu_tanh(float x) {
-  return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
-}
-// 1 / (1 + e^-x) without overflow on either side.
+// 1 / (1 + e^-x), without overflow on either side; the fast form is a few units in the last place off.
 __device__ __forceinline__ float sigmoid_f(float x) {
   const float e = expf(-fabsf(x));
   return (x >= 0.f ? 1.f : e) / (1.f + e);
+}
+__device__ __forceinline__ float sigmoid_fast(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
+// The form for a build with storage type T: 16-bit results do not show the difference.
+template <typename T>
+__device__ __forceinline__ float sigmoid_for(float x) {
+  if constexpr (sizeof(T) == 2) return sigmoid_fast(x);
+  else return sigmoid_f(x);
+}
+// GELU in its tanh form: (1 + tanh(u)) / 2 = sigmoid(2u).
+template <typename T>
+__device__ __forceinline__ float gelu_tanh(float x) {
+  return x * sigmoid_for<T>(1.5957691216057308f * (x + 0.044715f * x * x * x));
 }
 
 __device__ __forceinline__ float warp_sum(float v) {

@@ -645,7 +645,21 @@ gelu_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_str
   for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
     float v = partial[idx];
     for (uint32_t s = 1; s < splits; ++s) v += partial[s * split_stride + idx];
-    out[(idx / cols) * ldo + idx % cols] = from_f32<T>(gelu_tanh(v));
+    out[(idx / cols) * ldo + idx % cols] = from_f32<T>(gelu_tanh<T>(v));
+  }
+}
+// Four columns per thread: cols, ldo and split_stride multiples of 4.
+template <typename T>
+__global__ void __launch_bounds__(256)
+gelu_vec_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, T *__restrict__ out, uint32_t ldo, uint32_t rows,
+                uint32_t cols) {
+  pdl_trigger();
+  pdl_wait();
+  const uint32_t cv = cols / 4;
+  const size_t total = (size_t)rows * cv;
+  for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
+    const float4 v = sum_slabs4(partial + 4 * idx, splits, split_stride);
+    st4<T>(out + (idx / cv) * ldo + idx % cv * 4, make_float4(gelu_tanh<T>(v.x), gelu_tanh<T>(v.y), gelu_tanh<T>(v.z), gelu_tanh<T>(v.w)));
   }
 }
 
@@ -653,6 +667,11 @@ template <typename T>
 int launch_gelu(const float *partial, uint32_t splits, size_t split_stride, T *out, uint32_t ldo, uint32_t rows, uint32_t cols,
                 cudaStream_t stream) {
   if (rows == 0 || cols == 0) return ORION_OK;
+  if (cols % 4 == 0 && ldo % 4 == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0) {
+    ORION_CUDA_CHECK("gelu", launch_pdl(gelu_vec_kernel<T>, dim3(grid_for((size_t)rows * cols / 4, 256)), dim3(256), 0, stream, partial, splits,
+                                        split_stride, out, ldo, rows, cols));
+    return after_launch("gelu");
+  }
   ORION_CUDA_CHECK("gelu", launch_pdl(gelu_kernel<T>, dim3(grid_for((size_t)rows * cols, 256)), dim3(256), 0, stream, partial, splits,
                                       split_stride, out, ldo, rows, cols));
   return after_launch("gelu");

@@ -414,7 +414,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
           for (int j = 0; j < 16; ++j) {
             const uint32_t tok = t0 + c + j;
             const float v = __uint_as_float(r[j]);
-            if (tok < M) act[(size_t)tok * ldc + n] = __float2bfloat16_rn(epilogue == kGemmGelu ? gelu_tanh(v) : v);
+            if (tok < M) act[(size_t)tok * ldc + n] = __float2bfloat16_rn(epilogue == kGemmGelu ? gelu_tanh<bf16>(v) : v);
           }
         }
       } else if (act != nullptr) {

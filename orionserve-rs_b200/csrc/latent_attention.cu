@@ -515,37 +515,8 @@ latent_value_kernel(const float *__restrict__ part_o, const float *__restrict__ 
   for (uint32_t i = tid; i < nv * groups; i += kValueThreads)
     cp_async16(w_s + (i / groups) * pitch + (i % groups) * 16, w_uv + ((size_t)head * ls.value_dim + v0 + i / groups) * ls.kv_rank + (i % groups) * 8);
   pdl_wait();
-  for (uint32_t r = warp; r < n; r += kValueThreads / 32) {  // one warp per row: lane s weighs split s, then all sum
-    const size_t base = ((size_t)(row0 + r) * ctx_splits) * ls.heads + head;
-    float2 ml = make_float2(-INFINITY, 0.f);
-    if (lane < ctx_splits) ml = *reinterpret_cast<const float2 *>(part_ml + (base + (size_t)lane * ls.heads) * 2);
-    const float mx = warp_max(ml.x), e = ml.x == -INFINITY ? 0.f : fast_exp2(ml.x - mx);
-    const float wgt = e / warp_sum(e * ml.y);
-    for (uint32_t d0 = 0; d0 < ls.kv_rank; d0 += 128) {
-      const uint32_t d = d0 + lane * 4;
-      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-      for (uint32_t s0 = 0; s0 < ctx_splits; s0 += 4) {
-        float4 x[4];
-#pragma unroll
-        for (uint32_t j = 0; j < 4; ++j)  // four independent loads in flight
-          x[j] = s0 + j < ctx_splits && d < ls.kv_rank
-                     ? *reinterpret_cast<const float4 *>(part_o + (base + (size_t)(s0 + j) * ls.heads) * ls.kv_rank + d)
-                     : make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-        for (uint32_t j = 0; j < 4; ++j) {
-          const float w = __shfl_sync(0xffffffffu, wgt, (s0 + j) & 31u);
-          if (s0 + j < ctx_splits) a.x += w * x[j].x, a.y += w * x[j].y, a.z += w * x[j].z, a.w += w * x[j].w;
-        }
-      }
-      if (d < ls.kv_rank) store4<bf16>(reinterpret_cast<bf16 *>(o_s + r * pitch) + d, a);
-    }
-  }
-  cp_async_wait_all();
-  __syncthreads();
-  // warp = 16 values (M) x 8 rows (N); rows beyond n stay undefined and are not stored
+  // warp = 16 values (M) x 8 rows (N) of the product; its gate values are fetched before everything else
   const uint32_t vw = (warp & 3) * 16, rw = (warp >> 2) * 8;
-  if (vw >= nv || rw >= n) return;
-  // gate values of this thread's four results, in flight during the product
   float g[4], c[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
   for (uint32_t e = 0; e < 4; ++e) {
@@ -554,6 +525,42 @@ latent_value_kernel(const float *__restrict__ part_o, const float *__restrict__ 
                ? fold(gate + (size_t)row_list[row0 + r] * ls.cols() + ls.q_cols() + ls.kv_cols() + head * ls.value_dim + v, splits, split_stride)
                : 0.f;
   }
+  for (uint32_t r = warp; r < n; r += kValueThreads / 32) {  // one warp per row: lane s weighs split s, then all sum
+    const size_t base = ((size_t)(row0 + r) * ctx_splits) * ls.heads + head;
+    float2 ml = make_float2(-INFINITY, 0.f);
+    if (lane < ctx_splits) ml = *reinterpret_cast<const float2 *>(part_ml + (base + (size_t)lane * ls.heads) * 2);
+    const float mx = warp_max(ml.x), e = ml.x == -INFINITY ? 0.f : fast_exp2(ml.x - mx);
+    const float wgt = e / warp_sum(e * ml.y);
+    float4 a[4];  // kv_rank <= 512: four groups of four per lane, two splits of all of them in flight
+#pragma unroll
+    for (uint32_t k = 0; k < 4; ++k) a[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (uint32_t s0 = 0; s0 < ctx_splits; s0 += 2) {
+      float4 x[2][4];
+#pragma unroll
+      for (uint32_t j = 0; j < 2; ++j)
+#pragma unroll
+        for (uint32_t k = 0; k < 4; ++k) {
+          const uint32_t d = k * 128 + lane * 4;
+          x[j][k] = s0 + j < ctx_splits && d < ls.kv_rank
+                        ? *reinterpret_cast<const float4 *>(part_o + (base + (size_t)(s0 + j) * ls.heads) * ls.kv_rank + d)
+                        : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+      for (uint32_t j = 0; j < 2; ++j) {
+        const float w = __shfl_sync(0xffffffffu, wgt, (s0 + j) & 31u);
+        if (s0 + j < ctx_splits) {
+#pragma unroll
+          for (uint32_t k = 0; k < 4; ++k) a[k].x += w * x[j][k].x, a[k].y += w * x[j][k].y, a[k].z += w * x[j][k].z, a[k].w += w * x[j][k].w;
+        }
+      }
+    }
+#pragma unroll
+    for (uint32_t k = 0; k < 4; ++k)
+      if (k * 128 + lane * 4 < ls.kv_rank) store4<bf16>(reinterpret_cast<bf16 *>(o_s + r * pitch) + k * 128 + lane * 4, a[k]);
+  }
+  cp_async_wait_all();
+  __syncthreads();
+  if (vw >= nv || rw >= n) return;  // rows beyond n stay undefined and are not stored
   const uint32_t mi = lane >> 3, rr = lane & 7;
   const uint32_t wa = smem_u32(w_s) + (vw + rr + (mi & 1) * 8) * pitch + (mi >> 1) * 16;
   const uint32_t ob = smem_u32(o_s) + (rw + rr) * pitch + mi * 16;

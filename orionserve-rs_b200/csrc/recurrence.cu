@@ -14,8 +14,9 @@ namespace orion {
 namespace {
 
 // The map of one row and channel: S -> a S + b.
+template <typename T>
 __device__ __forceinline__ void min_gru_map(float z_pre, float x_pre, float &a, float &b) {
-  const float z = sigmoid_f(z_pre), cand = x_pre >= 0.f ? x_pre + 0.5f : sigmoid_f(x_pre);
+  const float z = sigmoid_for<T>(z_pre), below = sigmoid_for<T>(x_pre), cand = x_pre >= 0.f ? x_pre + 0.5f : below;
   a = 1.f - z;
   b = z * cand;
 }
@@ -45,9 +46,9 @@ min_gru_step_kernel(const float *__restrict__ partial, uint32_t splits, size_t s
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     float a, b;
-    min_gru_map(zz[i], xx[i], a, b);
+    min_gru_map<T>(zz[i], xx[i], a, b);
     ss[i] = a * ss[i] + b;
-    o[i] = from_f32<T>(ss[i] * gg[i] * sigmoid_f(gg[i]));
+    o[i] = from_f32<T>(ss[i] * gg[i] * sigmoid_for<T>(gg[i]));
   }
   *reinterpret_cast<float4 *>(state + (size_t)sb.write[row] * width + c) = make_float4(ss[0], ss[1], ss[2], ss[3]);
 }
@@ -90,7 +91,7 @@ min_gru_scan_kernel(const float *__restrict__ partial, uint32_t splits, size_t s
 #pragma unroll
     for (uint32_t i = 0; i < kRows; ++i) {
       a[i] = 1.f, b[i] = 0.f;
-      if (row0 + i < end) min_gru_map(z[i] + bz, x[i] + bx, a[i], b[i]);
+      if (row0 + i < end) min_gru_map<T>(z[i] + bz, x[i] + bx, a[i], b[i]);
       gate[i] = g[i];
       A *= a[i];
       B = a[i] * B + b[i];
@@ -107,7 +108,7 @@ min_gru_scan_kernel(const float *__restrict__ partial, uint32_t splits, size_t s
 #pragma unroll
     for (uint32_t i = 0; i < kRows; ++i) {
       mine = a[i] * mine + b[i];
-      if (live && row0 + i < end) out[(size_t)(row0 + i) * ldo + c] = from_f32<T>(mine * gate[i] * sigmoid_f(gate[i]));
+      if (live && row0 + i < end) out[(size_t)(row0 + i) * ldo + c] = from_f32<T>(mine * gate[i] * sigmoid_for<T>(gate[i]));
     }
   }
   if (live && warp == 0) state[(size_t)sb.write[seq] * width + c] = s;

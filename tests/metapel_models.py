@@ -71,7 +71,8 @@ TUNED = config(128, 192, [mingru(160, 192), latent(5, 32, 16, 48, 64, 40, 128), 
                           mingru(64, 320)], taps=4)
 WIDE = config(256, 320, [latent(20, 64, 32, 64, 192, 150, 512, base=50000.0), mingru(384, 0),
                          latent(3, 48, 64, 80, 512, 77, 64, scale=0.05)], taps=5)
-CONFIGS = {"odd": ODD, "one_tap": ONE_TAP, "tuned": TUNED, "wide": WIDE}
+BROAD_VALUES = config(96, 128, [latent(2, 32, 0, 144, 128, 100, 64), latent(3, 80, 16, 256, 64, 30)], taps=2)
+CONFIGS = {"broad_values": BROAD_VALUES, "odd": ODD, "one_tap": ONE_TAP, "tuned": TUNED, "wide": WIDE}
 
 
 def make_model(pkg, backend, cfg, weights, dtype, blocks=64, tokens=1024, seqs=8):
