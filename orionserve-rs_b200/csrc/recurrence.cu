@@ -5,7 +5,10 @@
 //   min_gru_scan_kernel   any batch: CTA = (32 channels, sequence); lanes are channels, each warp takes
 //                         kRows consecutive rows of a tile, composes their maps S -> A S + B, the warps
 //                         exchange (A, B) through shared memory, and each warp then runs its own rows from
-//                         the state it starts at. The next tile's partial sums are in flight meanwhile.
+//                         the state it starts at. The next tile's partial sums are in flight meanwhile. When
+//                         there are too few (channels, sequences) to fill the machine, the CTAs of a cluster
+//                         take consecutive tiles of one sequence and exchange their tiles' maps through
+//                         distributed shared memory.
 #include "kernels.h"
 
 #include <algorithm>
@@ -53,13 +56,27 @@ min_gru_step_kernel(const float *__restrict__ partial, uint32_t splits, size_t s
   *reinterpret_cast<float4 *>(state + (size_t)sb.write[row] * width + c) = make_float4(ss[0], ss[1], ss[2], ss[3]);
 }
 
-constexpr uint32_t kRows = 8;  // rows per warp and tile
+constexpr uint32_t kRows = 4, kMaxWarps = 16, kMaxCluster = 8;  // rows per warp and tile, warps per CTA, CTAs per cluster
+
+__device__ __forceinline__ void store_cluster(float2 *local, uint32_t rank, float2 v) {  // into the same place of CTA `rank`
+  asm volatile(
+      "{\n\t.reg .b32 a;\n\t"
+      "mapa.shared::cluster.u32 a, %0, %1;\n\t"
+      "st.shared::cluster.v2.f32 [a], {%2, %3};\n\t}" ::"r"(smem_u32(local)),
+      "r"(rank), "f"(v.x), "f"(v.y)
+      : "memory");
+}
+__device__ __forceinline__ void cluster_sync() {
+  asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
 
 template <typename T>
-__global__ void __launch_bounds__(1024)
+__global__ void __launch_bounds__(32 * kMaxWarps, 2)
 min_gru_scan_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, const float *__restrict__ bias,
                     float *__restrict__ state, StateBatch sb, T *__restrict__ out, uint32_t ldo, uint32_t width) {
-  __shared__ float2 maps[2][32][32];  // [tile parity][warp][channel]
+  __shared__ float2 maps[2][kMaxWarps][32];      // [tile parity][warp][channel]
+  __shared__ float2 tiles[2][kMaxCluster][32];   // the same for the tiles of the cluster's CTAs
+  const uint32_t ctas = gridDim.z, rank = blockIdx.z;  // the cluster spans the grid's z
   pdl_trigger();
   pdl_wait();
   const uint32_t seq = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
@@ -83,10 +100,12 @@ min_gru_scan_kernel(const float *__restrict__ partial, uint32_t splits, size_t s
       }
     }
   };
-  fetch(first + warp * kRows);
+  const uint32_t step = ctas * warps * kRows, mine0 = (rank * warps + warp) * kRows;
+  fetch(first + mine0);
+  if (ctas > 1) cluster_sync();  // every CTA of the cluster has started before anyone stores into it
   uint32_t parity = 0;
-  for (uint32_t t0 = first; t0 < end; t0 += warps * kRows, parity ^= 1) {
-    const uint32_t row0 = t0 + warp * kRows;
+  for (uint32_t t0 = first; t0 < end; t0 += step, parity ^= 1) {
+    const uint32_t row0 = t0 + mine0;
     float a[kRows], b[kRows], gate[kRows], A = 1.f, B = 0.f;
 #pragma unroll
     for (uint32_t i = 0; i < kRows; ++i) {
@@ -96,14 +115,38 @@ min_gru_scan_kernel(const float *__restrict__ partial, uint32_t splits, size_t s
       A *= a[i];
       B = a[i] * B + b[i];
     }
-    fetch(row0 + warps * kRows);
+    fetch(row0 + step);
     maps[parity][warp][lane] = make_float2(A, B);
     __syncthreads();
-    float mine = s;  // the state this warp's rows start from; every warp ends up with the tile's last state in s
-    for (uint32_t k = 0; k < warps; ++k) {
-      const float2 m = maps[parity][k][lane];
-      if (k == warp) mine = s;
-      s = m.x * s + m.y;
+    float mine = s;  // the state this warp's rows start from; every warp ends up with the last state of all tiles in s
+    if (ctas > 1) {
+      if (warp < ctas) {  // warp k tells CTA k
+        float2 whole = make_float2(1.f, 0.f);
+        for (uint32_t k = 0; k < warps; ++k) {
+          const float2 m = maps[parity][k][lane];
+          whole = make_float2(m.x * whole.x, m.x * whole.y + m.y);
+        }
+        store_cluster(&tiles[parity][rank][lane], warp, whole);
+      }
+      cluster_sync();
+      float before = s;
+      for (uint32_t k = 0; k < ctas; ++k) {
+        const float2 m = tiles[parity][k][lane];
+        if (k == rank) before = s;
+        s = m.x * s + m.y;
+      }
+      mine = before;
+      for (uint32_t k = 0; k < warp; ++k) {
+        const float2 m = maps[parity][k][lane];
+        mine = m.x * mine + m.y;
+      }
+    } else {
+#pragma unroll 4
+      for (uint32_t k = 0; k < warps; ++k) {
+        const float2 m = maps[parity][k][lane];
+        if (k == warp) mine = s;
+        s = m.x * s + m.y;
+      }
     }
 #pragma unroll
     for (uint32_t i = 0; i < kRows; ++i) {
@@ -111,7 +154,7 @@ min_gru_scan_kernel(const float *__restrict__ partial, uint32_t splits, size_t s
       if (live && row0 + i < end) out[(size_t)(row0 + i) * ldo + c] = from_f32<T>(mine * gate[i] * sigmoid_for<T>(gate[i]));
     }
   }
-  if (live && warp == 0) state[(size_t)sb.write[seq] * width + c] = s;
+  if (live && warp == 0 && rank == 0) state[(size_t)sb.write[seq] * width + c] = s;
 }
 
 inline int after_launch(const char *stage) {
@@ -131,11 +174,18 @@ int launch_min_gru(const float *partial, uint32_t splits, size_t split_stride, c
                                            splits, split_stride, bias, state, sb, out, ldo, width));
     return after_launch("min_gru");
   }
-  // warps per CTA: enough for the mean sequence in one tile, at most 32
-  const uint32_t mean = (sb.rows + sb.seqs - 1) / sb.seqs;
-  const uint32_t warps = std::min(32u, std::max(1u, (mean + kRows - 1) / kRows));
-  ORION_CUDA_CHECK("min_gru", launch_pdl(min_gru_scan_kernel<T>, dim3((width + 31) / 32, sb.seqs), dim3(32 * warps), 0, stream, partial,
-                                         splits, split_stride, bias, state, sb, out, ldo, width));
+  // warps per CTA: enough for the mean sequence in one tile; CTAs per cluster: as long as they find tiles and places
+  const uint32_t mean = (sb.rows + sb.seqs - 1) / sb.seqs, groups = (width + 31) / 32 * sb.seqs;
+  uint32_t ctas = 1;
+  while (ctas < kMaxCluster && 2 * ctas * groups <= 2 * 148 && 2 * ctas * kMaxWarps * kRows <= mean) ctas *= 2;
+  const uint32_t warps = ctas > 1 ? kMaxWarps : std::min(kMaxWarps, std::max(1u, (mean + kRows - 1) / kRows));
+  const dim3 grid((width + 31) / 32, sb.seqs, ctas);
+  if (ctas > 1)
+    ORION_CUDA_CHECK("min_gru", launch_pdl_cluster(min_gru_scan_kernel<T>, grid, dim3(32 * warps), dim3(1, 1, ctas), 0, stream, partial,
+                                                   splits, split_stride, bias, state, sb, out, ldo, width));
+  else
+    ORION_CUDA_CHECK("min_gru", launch_pdl(min_gru_scan_kernel<T>, grid, dim3(32 * warps), 0, stream, partial, splits, split_stride, bias,
+                                           state, sb, out, ldo, width));
   return after_launch("min_gru");
 }
 template int launch_min_gru<float>(const float *, uint32_t, size_t, const float *, float *, StateBatch, float *, uint32_t, uint32_t,
