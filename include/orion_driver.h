@@ -43,8 +43,10 @@ typedef struct OrionCacheStats {
  * logical_decode_positions has none either: non-zero feeds a decode token at position
  * total_len - 1, its logical place, instead of the reference's total_len (scheduler.rs:283), so
  * that no cache slot is skipped and no step is refused. 0 = the reference's behaviour.
- * recompute_on_preempt: non-zero prefills a preempted sequence's generated tokens again after its prompt
- * (the reference leaves them out of the cache). An engine around a model with state slots sets this and
+ * recompute_on_preempt: for sequences that carry state from token to token. Non-zero prefills a preempted
+ * sequence's generated tokens again after its prompt (the reference leaves them out of the cache) and a
+ * failed step's prompt portions again, does not preempt to admit, schedules a sequence at most once per step
+ * and accepts a request only if prompt and output fit the cache together. An engine around a model with state slots sets this and
  * logical_decode_positions itself, and refuses skip_cached_prefix. */
 typedef struct OrionSchedulerConfig {
   uint64_t max_num_seqs, max_num_batched_tokens, max_model_len;

@@ -216,9 +216,11 @@ struct SchedulerConfig {  // crates/orion-core/src/config.rs:107-156
   // instead of total_len (scheduler.rs:283 counts the token that was just sampled), so no cache
   // slot is skipped and no step is refused for a block the table does not hold yet.
   bool logical_decode_positions = false;
-  // Not in the reference either: a preempted sequence that has generated tokens prefills them again after
-  // its prompt (the reference drops them from the cache and goes on behind them), so that what it carries
-  // is complete when it decodes on. Needed by models with recurrent state, which set it and
+  // Not in the reference either, for sequences whose tokens must be computed one after the other, each exactly once
+  // (recurrent state): a preempted sequence that has generated tokens prefills them again after its prompt (the
+  // reference drops them from the cache and goes on behind them); a step that failed is prefilled again; running
+  // sequences are not preempted to admit waiting ones; a sequence is in a step at most once; and a request is
+  // accepted only if prompt and output fit the cache together. Models with state slots set it and
   // logical_decode_positions themselves.
   bool recompute_on_preempt = false;
 };

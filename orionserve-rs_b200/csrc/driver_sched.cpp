@@ -102,7 +102,8 @@ int Scheduler::add_request(Sequence seq, SequenceId *id) {  // scheduler.rs:174-
                      seq.params().max_tokens, max_len);
   }
   // a prompt larger than the whole cache would block the queue head forever
-  const size_t blocks = cache_.blocks_needed_for(seq.prompt_len());
+  // (with recomputation the generated tokens are part of what has to fit again)
+  const size_t blocks = cache_.blocks_needed_for(config_.recompute_on_preempt ? needed : seq.prompt_len());
   if (blocks > cache_.total_blocks()) {
     stats_.total_rejected += 1;
     return set_error(ORION_ERR_CACHE_EXHAUSTED, "KV cache exhausted: needed %zu blocks, %zu free", blocks,
@@ -163,8 +164,13 @@ SchedulerOutput Scheduler::schedule() {  // scheduler.rs:239-263
 void Scheduler::schedule_decodes(SchedulerOutput &out, size_t budget, size_t &used) {  // scheduler.rs:267-313
   std::vector<std::pair<SequenceId, size_t>> candidates;  // collected first: the loop below mutates `running`
   const size_t shift = config_.logical_decode_positions ? 1 : 0;
+  // With prefills scheduled first, a prompt completed by this step is already in the Decoding state; its first
+  // output token is sampled by this step, so where every token has to follow the one before it, it waits for the next.
+  auto planned = [&](SequenceId id) {
+    return config_.recompute_on_preempt && std::any_of(out.scheduled.begin(), out.scheduled.end(), [&](const ScheduledSequence &s) { return s.id == id; });
+  };
   for (const Sequence &s : running_)
-    if (s.state() == SequenceState::Decoding) candidates.emplace_back(s.id(), s.total_len() - std::min(shift, s.total_len()));
+    if (s.state() == SequenceState::Decoding && !planned(s.id())) candidates.emplace_back(s.id(), s.total_len() - std::min(shift, s.total_len()));
   for (const auto &[id, total_len] : candidates) {
     if (used >= budget) break;
     // Room for the token about to be generated. Note the position: total_len counts the token
@@ -243,7 +249,9 @@ void Scheduler::schedule_prefills(SchedulerOutput &out, size_t budget, size_t &u
     const bool is_first_chunk = already == 0;  // only the first chunk allocates
     if (is_first_chunk && !cache_.has_free_state_slot()) break;  // a slot comes free when a sequence ends
     if (is_first_chunk && !cache_.can_allocate(prompt_len)) {
-      if (!preempt_one(out)) break;
+      // The reference makes room by preempting the newest running sequence, which goes back to the head of the
+      // queue; where that sequence would have to be computed again from its first token, it is left running.
+      if (config_.recompute_on_preempt || !preempt_one(out)) break;
       continue;
     }
     Sequence seq = std::move(waiting_.front());
