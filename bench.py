@@ -385,8 +385,8 @@ def metapel_work(meta, rows, contexts, prompts):
             n = H * 3 * s.width + s.width * H
         else:
             n = H * (s.heads * (s.dim + s.rot_dim) + s.kv_rank + s.rot_dim + s.heads * s.value_dim) + s.heads * s.value_dim * H
-            absorb = s.heads * (s.dim + s.value_dim) * s.kv_rank
-            n += absorb
+            if prompts:  # keys and values are expanded from the latents; decoding rows stay in the latent space
+                n += s.heads * (s.dim + s.value_dim) * s.kv_rank
             seen = [min(c, s.window) if s.window else c for c in contexts]
             cache += sum(seen) * (s.kv_rank + s.rot_dim) * 2
             attn += sum(seen) * s.heads * 2 * (2 * s.kv_rank + s.rot_dim)

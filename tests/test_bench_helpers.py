@@ -43,3 +43,19 @@ def test_decode_batches_are_valid_and_their_tables_disjoint(pkg):
         assert lens == [(c + 15) // 16 for c in contexts]
         used = flat[:int(offsets[-1])]
         assert len(set(used.tolist())) == len(used) and int(used.max()) < num_blocks
+
+
+def test_algorithmic_work_of_a_metapel_step(pkg):
+    z = dict(heads=4, dim=32, rot_dim=16, value_dim=24, kv_rank=64, window=10)
+    meta = pkg.LayeredMetadata("Metapel", "m", 48, 100, [pkg.LayerSpec("mingru", 20, width=30),
+                               pkg.LayerSpec("latent_attention", 0, **z)], 1e-5, 4)
+    gru = 48 * 3 * 30 + 30 * 48 + 2 * 48 * 20
+    att = 48 * (4 * 48 + 80 + 4 * 24) + 4 * 24 * 48
+    head = bench.METAPEL_VOCAB * 48
+    w, fl, cache, attn = bench.metapel_work(meta, 2, [7, 300], [])
+    assert w == 2 * (gru + att + head) and fl == 2 * 2 * (gru + att + head)
+    assert cache == (7 + 10) * 80 * 2 and attn == (7 + 10) * 4 * 2 * (2 * 64 + 16)
+    w, fl, cache, attn = bench.metapel_work(meta, 12, [], [12])
+    att += 4 * (32 + 24) * 64
+    assert w == 2 * (gru + att + head) and fl == 2 * (12 * (gru + att) + head)
+    assert cache == 0 and attn == (55 + 2 * 10) * 4 * 2 * (32 + 16 + 24)
