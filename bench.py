@@ -462,13 +462,14 @@ def run_metapel(args):
                     steps = args.steps if mode == "decode" else max(3, args.steps // 5)
                     model.replay(max(3, args.warmup))
                     ms = model.replay(steps) / steps
+                    launches = model.last_launch_count()
                     fam = {c: model.replay_categories(steps, c) / steps for c in ("gemm", "attention", "elementwise")}
                     wb, fl, cb, af = (metapel_work(meta, rows, contexts, prompts) if kind == "metapel"
                                       else llama_work(m, rows, contexts, prompts))
                     gemm_s, attn_s = fam["gemm"] / 1e3, fam["attention"] / 1e3
                     out.append({"model": kind, "shape": name, "layers": layers, "mode": mode, "sequences": b, "tokens_each": n,
                                 "ms_per_step": ms, "tokens_per_s": rows / ms * 1e3, "gemm_ms": fam["gemm"], "mixer_ms": fam["attention"],
-                                "elementwise_ms": fam["elementwise"], "launches": model.last_launch_count(),
+                                "elementwise_ms": fam["elementwise"], "launches": launches,
                                 "gemm_frac": max(wb / gemm_s / hbm / 1e9, fl / gemm_s / tflops / 1e12),
                                 "step_frac": max((wb + cb) / (ms / 1e3) / hbm / 1e9, (fl + af) / (ms / 1e3) / tflops / 1e12)})
                 del model

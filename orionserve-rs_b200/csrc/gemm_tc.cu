@@ -204,7 +204,9 @@ __device__ __forceinline__ constexpr uint32_t instr_desc() {
          ((uint32_t)(M >> 4) << 24);
 }
 
-template <int TOKN, int WST, int XST, int MT, bool PAIR = false>
+// ACT: the epilogue stores activations (kGemmGelu, kGemmStore); else f32 partials, or SwiGLU where `act` is given. A
+// template parameter, since the larger epilogue costs the weight-streaming shapes 0.8 us per launch.
+template <int TOKN, int WST, int XST, int MT, bool PAIR, bool ACT>
 __global__ void __launch_bounds__(kThreads)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                float *__restrict__ partial, bf16 *__restrict__ act, uint32_t M, uint32_t N, uint32_t K,
@@ -408,7 +410,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
       if (cluster_reduce) {
 #pragma unroll
         for (int j = 0; j < 16; ++j) stage[(c + j) * kTileN + lq * 32 + lane] = __uint_as_float(r[j]);
-      } else if (epilogue == kGemmGelu || epilogue == kGemmStore) {  // activations in bf16, row stride ldc
+      } else if constexpr (ACT) {  // activations in bf16, row stride ldc
         if (n < N) {
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
@@ -548,10 +550,10 @@ int cached_map(const void *base, uint64_t rows, uint64_t k, uint64_t ld, uint32_
   return ORION_OK;
 }
 
-template <int TOKN, int WST, int XST, int MT = 1, bool PAIR = false>
-int launch_tc(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, float *partial, bf16 *act,
+template <bool ACT, int TOKN, int WST, int XST, int MT, bool PAIR>
+int launch_tc_form(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, float *partial, bf16 *act,
               uint32_t rows, uint32_t n, uint32_t k, uint32_t splits, bool cluster_reduce, uint32_t ldc, GemmEpilogue epi,
-              cudaStream_t stream, ReadyWait ready = {}) {
+              cudaStream_t stream, ReadyWait ready) {
   if (ldc == 0) ldc = n;
   if (ldc != n && (splits != 1 || epi == kGemmSwiglu))
     return set_error(ORION_ERR_INTERNAL, "a strided GEMM output needs one k split and no SwiGLU");
@@ -559,7 +561,7 @@ int launch_tc(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, float *p
   static_assert(Cfg::kSmemBytes <= 232448, "ring exceeds the shared memory of an SM");
   if (MT > 1 && cluster_reduce) return set_error(ORION_ERR_INTERNAL, "cluster split-K is built for one weight tile per CTA");
   static bool attr_set[kMaxDeviceOrdinals] = {};
-  ORION_CUDA_CHECK("gemm_tc attr", ensure_dynamic_smem(gemm_tc_kernel<TOKN, WST, XST, MT, PAIR>, Cfg::kSmemBytes, attr_set));
+  ORION_CUDA_CHECK("gemm_tc attr", ensure_dynamic_smem(gemm_tc_kernel<TOKN, WST, XST, MT, PAIR, ACT>, Cfg::kSmemBytes, attr_set));
   const CUtensorMap *mw, *mx;
   ORION_TRY(cached_map(w, n, k, ldw, kTileN, &mw));
   ORION_TRY(cached_map(x, rows, k, ldx, Cfg::kXRows, &mx));
@@ -567,19 +569,27 @@ int launch_tc(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, float *p
   if (PAIR) {
     if (cluster_reduce || (grid.x & 1u))
       return set_error(ORION_ERR_INTERNAL, "the paired GEMM needs an even number of weight tile groups and no cluster split-K");
-    ORION_CUDA_CHECK("gemm_tc", launch_pdl_cluster(gemm_tc_kernel<TOKN, WST, XST, MT, PAIR>, grid, dim3(kThreads), dim3(2, 1, 1),
+    ORION_CUDA_CHECK("gemm_tc", launch_pdl_cluster(gemm_tc_kernel<TOKN, WST, XST, MT, PAIR, ACT>, grid, dim3(kThreads), dim3(2, 1, 1),
                                                    Cfg::kSmemBytes, stream, *mw, *mx, partial, act, rows, n, k, splits,
                                                    0u, ldc, (uint32_t)epi, ready));
   } else if (cluster_reduce)
-    ORION_CUDA_CHECK("gemm_tc", launch_pdl_cluster(gemm_tc_kernel<TOKN, WST, XST, MT, PAIR>, grid, dim3(kThreads), dim3(1, 1, splits),
+    ORION_CUDA_CHECK("gemm_tc", launch_pdl_cluster(gemm_tc_kernel<TOKN, WST, XST, MT, PAIR, ACT>, grid, dim3(kThreads), dim3(1, 1, splits),
                                                    Cfg::kSmemBytes, stream, *mw, *mx, partial, act, rows, n, k, splits,
                                                    1u, ldc, (uint32_t)epi, ready));
   else
-    ORION_CUDA_CHECK("gemm_tc", launch_pdl(gemm_tc_kernel<TOKN, WST, XST, MT, PAIR>, grid, dim3(kThreads), Cfg::kSmemBytes, stream,
+    ORION_CUDA_CHECK("gemm_tc", launch_pdl(gemm_tc_kernel<TOKN, WST, XST, MT, PAIR, ACT>, grid, dim3(kThreads), Cfg::kSmemBytes, stream,
                                            *mw, *mx, partial, act, rows, n, k, splits, 0u, ldc, (uint32_t)epi, ready));
   count_launch();
   ORION_CUDA_CHECK("gemm_tc", cudaGetLastError());
   return ORION_OK;
+}
+
+template <int TOKN, int WST, int XST, int MT = 1, bool PAIR = false>
+int launch_tc(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, float *partial, bf16 *act, uint32_t rows, uint32_t n,
+              uint32_t k, uint32_t splits, bool cluster_reduce, uint32_t ldc, GemmEpilogue epi, cudaStream_t stream, ReadyWait ready = {}) {
+  auto form = epi == kGemmGelu || epi == kGemmStore ? launch_tc_form<true, TOKN, WST, XST, MT, PAIR>
+                                                    : launch_tc_form<false, TOKN, WST, XST, MT, PAIR>;
+  return form(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready);
 }
 
 // 256-token tiles as CTA pairs (tcgen05 cta_group::2). Measured on the Llama-3-8B shape, projections of
