@@ -1,13 +1,13 @@
 """Replays a trace: steps of given tokens go through a model's forward, cache manager and state slots exactly
 as an engine's steps do, and the logits that are asked for are written out. Nothing is sampled.
 
-Standard input has one JSON object a line::
+Each input line is a JSON object for one step, here the eighth, which runs two requests and ends one::
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": []}
+    {"step": 7, "entries": [{"id": "x", "tokens": [11, 4], "want": [1]}, {"id": "y", "tokens": [9], "want": []}], "end": ["y"]}
 
-``entries`` are one batch: the next tokens of each request, and the places among them whose logits are
-wanted. ``end`` names the requests that are finished after the step. A step with wanted logits writes
-``<out>/<step>.f32`` (little-endian f32, one row per wanted place); every step prints ``done <step>``."""
+An entry continues a request with ``tokens``; ``want`` indexes those of them whose logits go to ``<out>/<step>.f32``
+(little-endian f32, a row per index, in the order given; no file when no entry wants any). ``end`` releases the
+blocks and state slots of requests. Once a step has run, ``done <step>`` is printed."""
 from __future__ import annotations
 
 import argparse
@@ -21,7 +21,7 @@ from .registry import load_model
 from .types import DType, ForwardBatch
 
 BLOCK = 16
-ROUND = 64  # live tokens are counted per request in units of this many
+ROUND = 64  # the capacity is given in units of this many tokens
 STATE_SLOTS = 4
 
 
@@ -79,7 +79,7 @@ def main(argv=None) -> int:
     ap.add_argument("--dtype", choices=("bfloat16", "float32"), default="bfloat16")
     ap.add_argument("--out", required=True, help="folder for the logits")
     ap.add_argument("--max-tokens", type=int, required=True,
-                    help=f"most tokens that live requests hold at any time, each rounded up to {ROUND}")
+                    help=f"capacity of the cache in tokens; a request takes a multiple of {ROUND} of them")
     args = ap.parse_args(argv)
     dtype = {"bfloat16": DType.BF16, "float32": DType.F32}[args.dtype]
     runner = TraceRunner.from_directory(args.model, dtype, args.max_tokens)

@@ -128,6 +128,8 @@ MECHANISMS = {
     "recurrence": (config(72, 90, [mingru(56)], taps=2), ("canon",)),
     "attention": (config(96, 90, [latent(4, 16, 16, 16, 48, 13)], taps=2), ("canon",)),
     "attention without a rotated part's influence": (config(96, 90, [latent(4, 16, 16, 16, 48, 300, base=30.0)], taps=2), ("canon", "mix.uk")),
+    "attention over everything before": (config(96, 90, [dict(e, mixer=dict(e["mixer"], mask=None)) for e in [latent(5, 32, 16, 32, 64, 0)]],
+                                                taps=2), ("canon",)),
     "final norm and head": (config(72, 90, [mingru(16)], taps=2), ("mix.o",)),
 }
 
