@@ -368,7 +368,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
       umma_commit(acc_ready);  // arrives when every MMA above has completed
       ORION_GTRACE(tslot, 4);
     }
-  } else if (warp >= 4) {
+  } else if (!ACT && warp >= 4) {
     // Epilogue warps: warp w may touch tensor-memory lanes 32*(w%4) .. +31.
     const uint32_t lq = warp & 3;
     // The partial buffer may still be read by the kernel before the producer of x: wait for the
@@ -410,15 +410,6 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
       if (cluster_reduce) {
 #pragma unroll
         for (int j = 0; j < 16; ++j) stage[(c + j) * kTileN + lq * 32 + lane] = __uint_as_float(r[j]);
-      } else if constexpr (ACT) {  // activations in bf16, row stride ldc
-        if (n < N) {
-#pragma unroll
-          for (int j = 0; j < 16; ++j) {
-            const uint32_t tok = t0 + c + j;
-            const float v = __uint_as_float(r[j]);
-            if (tok < M) act[(size_t)tok * ldc + n] = __float2bfloat16_rn(epilogue == kGemmGelu ? gelu_tanh<bf16>(v) : v);
-          }
-        }
       } else if (act != nullptr) {
         // Fused SwiGLU (tensor.rs:167-189): weight rows are interleaved, lane 2i holds gate_f and
         // lane 2i + 1 holds up_f of the same f for these 16 tokens. Each lane of a pair trades
@@ -443,6 +434,34 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
       }
       }
     }
+  }
+  if constexpr (ACT) {
+    // Activations in bf16, row stride ldc. All eight warps: the conversion is as long as a short k loop, and the
+    // producers and the issuing warp have nothing left to do. Warps 0-3 take the second half of the columns.
+    __syncwarp();
+    const uint32_t lq = warp & 3;
+    pdl_wait();  // `act` may still be read by the kernel before the producer of x
+    if (!mbar_wait(acc_ready, 0)) ok = false;
+    tc_fence_after();
+    constexpr int kCols = MT * TOKN, kHalf = kCols >= 32 ? kCols / 2 : kCols;
+    const int begin = warp >= 4 ? 0 : kHalf, end = warp >= 4 ? kHalf : kCols;
+#pragma unroll 1
+    for (int mc = begin; mc < end; mc += 16) {
+      uint32_t r[16];
+      tmem_ld16(tmem_base + ((lq * 32u) << 16) + (uint32_t)mc, r);
+      tmem_ld_wait();
+      const int mt = mc / TOKN, c = mc % TOKN;
+      const uint32_t n = n0 + mt * kTileN + lq * 32 + lane;
+      if (t0 + c >= M || n >= N) continue;
+      bf16 *dst = act + (size_t)(t0 + c) * ldc + n;
+      const uint32_t valid = M - (t0 + c);
+#pragma unroll
+      for (int j = 0; j < 16; ++j) {
+        const float v = __uint_as_float(r[j]);
+        if ((uint32_t)j < valid) dst[(size_t)j * ldc] = __float2bfloat16_rn(epilogue == kGemmGelu ? gelu_tanh<bf16>(v) : v);
+      }
+    }
+    __syncwarp();
   }
   if (cluster_reduce) {
     // The `splits` CTAs of one tile form a cluster (1, 1, splits). Every CTA sums a share of the
