@@ -5,8 +5,8 @@
 //    any mix of prefill and decode rows; one CTA per (row, query head). This is
 //    the correctness tier (f32 build) and the fallback for shapes the tuned
 //    kernel does not cover.
-//  * paged_decode_kernel: bf16, head_dim 128, 16-token blocks, one query row
-//    per sequence. One CTA per (kv head, sequence, context split); each warp owns
+//  * paged_decode_kernel: bf16, head_dim 128 (64 to 256 with the FORM parameter), 16-token
+//    blocks, query rows that decode. One CTA per (kv head, sequence, context split); each warp owns
 //    a private multi-stage ring of 8 KiB K/V chunks filled by bulk async copies
 //    (one copy per 16-token block of one head), computes Q.K^T and P.V with
 //    mma.sync m16n8k16 (tokens on M, the GQA group's query heads on N so the group
@@ -29,15 +29,15 @@ namespace {
 
 constexpr int kGenThreads = 128;
 constexpr int kGenChunk = 512;
-constexpr int kGenMaxDimsPerThread = 4;  // head_dim <= 512
+constexpr int kGenMaxDimsPerThread = 4;  // values of up to 512 dimensions
 
 template <typename T>
 __global__ void __launch_bounds__(kGenThreads)
 paged_attention_generic_kernel(const T *__restrict__ q, const T *__restrict__ arena, KvLayout kv,
                                uint32_t layer, AttnBatch batch, uint32_t q_heads,
-                               T *__restrict__ out) {
+                               T *__restrict__ out, AttnForm form) {
   extern __shared__ float smem[];
-  const uint32_t hd = kv.head_dim;
+  const uint32_t hd = kv.head_dim, vd = form.out_dim ? form.out_dim : kv.v_dim();
   float *q_s = smem;            // [hd]
   float *scores = smem + hd;    // [kGenChunk]
   __shared__ float red[kGenThreads / 32];
@@ -52,17 +52,17 @@ paged_attention_generic_kernel(const T *__restrict__ q, const T *__restrict__ ar
   const uint32_t seq = batch.seq_of_row[row];
   const uint32_t *table = batch.tables_flat + batch.table_offsets[seq];
   const uint32_t B = kv.block_size;
-  const float scale = 1.0f / sqrtf((float)hd);  // attention.rs:251
+  const float scale = form.scale != 0.f ? form.scale : 1.0f / sqrtf((float)hd);  // attention.rs:251
 
   for (uint32_t d = threadIdx.x; d < hd; d += blockDim.x)
     q_s[d] = to_f32<T>(q[((size_t)row * q_heads + head) * hd + d]);
   __syncthreads();
 
-  float m = -INFINITY, l = 0.0f;
+  float m = form.sinks ? form.sinks[head] : -INFINITY, l = form.sinks ? 1.0f : 0.0f;
   float acc[kGenMaxDimsPerThread] = {0.f, 0.f, 0.f, 0.f};
   const uint32_t attend = qpos + 1;  // attention.rs:253: positions 0..=query_position
 
-  for (uint32_t c0 = 0; c0 < attend; c0 += kGenChunk) {
+  for (uint32_t c0 = form.range.first(qpos); c0 < attend; c0 += kGenChunk) {
     const uint32_t n = min((uint32_t)kGenChunk, attend - c0);
     float cmax = -INFINITY;
     for (uint32_t p = threadIdx.x; p < n; p += blockDim.x) {
@@ -102,7 +102,7 @@ paged_attention_generic_kernel(const T *__restrict__ q, const T *__restrict__ ar
 #pragma unroll
     for (int j = 0; j < kGenMaxDimsPerThread; ++j) {
       const uint32_t d = threadIdx.x + j * kGenThreads;
-      if (d >= hd) break;
+      if (d >= vd) break;
       float a = acc[j] * corr;
       for (uint32_t p = 0; p < n; ++p) {
         const float w = scores[p];
@@ -119,8 +119,10 @@ paged_attention_generic_kernel(const T *__restrict__ q, const T *__restrict__ ar
 #pragma unroll
   for (int j = 0; j < kGenMaxDimsPerThread; ++j) {
     const uint32_t d = threadIdx.x + j * kGenThreads;
-    if (d >= hd) break;
-    out[((size_t)row * q_heads + head) * hd + d] = from_f32<T>(l > 0.0f ? acc[j] / l : acc[j]);
+    if (d >= vd) break;
+    float v = l > 0.0f ? acc[j] / l : acc[j];
+    if (form.gate) v *= form.gate[(size_t)row * q_heads + head];
+    out[(size_t)row * (form.ldo ? form.ldo : q_heads * vd) + (size_t)head * vd + d] = from_f32<T>(v);
   }
 }
 
@@ -131,14 +133,14 @@ paged_attention_generic_kernel(const T *__restrict__ q, const T *__restrict__ ar
 constexpr int kHd = 128;          // head_dim
 constexpr int kBlk = 16;          // tokens per KV block
 constexpr int kWarps = 4;         // warps per CTA, each with a private ring
-constexpr int kChunkBytes = 2 * kBlk * kHd * 2;  // K rows + V rows of one (block, head): 8 KiB
 constexpr int kMaxGroup = 8;      // query heads per kv head (N of the MMA)
 // Ring depth per warp is a template parameter: 2 stages = 65 KiB per CTA (3 CTAs per SM),
 // 3 = 97 KiB (2 per SM), 4 = 129 KiB (1 per SM). The merge buffers (16.3 KiB) reuse the ring.
 // After the ring: 512 bytes of barriers, then the bf16 q / k / v of the row when the kernel makes
 // them itself (kMaxGroup + 2 vectors of 256 bytes).
 constexpr int kStashOffset = 512;
-constexpr uint32_t decode_smem_bytes(int stages) { return kWarps * stages * kChunkBytes + 4096; }
+constexpr int chunk_bytes(int dk, int dv) { return kBlk * (dk + dv) * 2; }  // K rows + V rows of one (block, head): 8 KiB at 128
+constexpr uint32_t decode_smem_bytes(int stages, int dk = kHd, int dv = kHd) { return kWarps * stages * chunk_bytes(dk, dv) + 4096; }
 
 __device__ __forceinline__ float4 ld4(const float *p) { return *reinterpret_cast<const float4 *>(p); }
 __device__ __forceinline__ float4 add4(float4 a, float4 b) {
@@ -154,34 +156,54 @@ __device__ __forceinline__ void st4<bf16>(bf16 *dst, float4 v) {
   *reinterpret_cast<uint2 *>(dst) = packed;
 }
 
+// Value d of a head's output, gated, at its place in the output row; values beyond the head's own size are padding.
+__device__ __forceinline__ void store_head_value(const AttnForm &form, uint32_t q_heads, uint32_t padded, uint32_t row, uint32_t head,
+                                                 uint32_t d, float v, bf16 *out) {
+  const uint32_t n = form.out_dim ? form.out_dim : padded;
+  if (d >= n) return;
+  if (form.gate) v *= form.gate[(size_t)row * q_heads + head];
+  out[(size_t)row * (form.ldo ? form.ldo : q_heads * n) + (size_t)head * n + d] = __float2bfloat16_rn(v);
+}
+
 // Device error word: bit 0 = a ring wait ran out of polls.
 __device__ uint32_t g_decode_error = 0;
 
-template <int kStages>
+// DK, DV: sizes of the K and V rows. FORM: the mask, sinks, gate and row list of `form` and any number of query heads per
+// kv head (eight to a CTA); without it those branches and arguments are compiled out.
+template <int kStages, int DK, int DV, bool FORM>
 __global__ void __launch_bounds__(kWarps * 32)
 paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, KvLayout kv,
                     uint32_t layer, AttnBatch batch, uint32_t q_heads, uint32_t splits,
-                    DecodeScratch scratch, bf16 *__restrict__ out, FusedQkv fq) {
+                    DecodeScratch scratch, bf16 *__restrict__ out, FusedQkv fq, AttnForm form) {
+  constexpr int kChunkBytes = chunk_bytes(DK, DV);
   extern __shared__ __align__(1024) uint8_t dsmem[];
   uint8_t *ring = dsmem;  // [kWarps][kStages][kChunkBytes]
   uint64_t *bars = reinterpret_cast<uint64_t *>(dsmem + kWarps * kStages * kChunkBytes);
   bf16 *stash = reinterpret_cast<bf16 *>(dsmem + kWarps * kStages * kChunkBytes + kStashOffset);  // [group + 2][kHd]
 
-  const uint32_t kvh = blockIdx.x, row = blockIdx.y, split = blockIdx.z;
+  const uint32_t item = blockIdx.y, split = blockIdx.z, row = FORM && form.row_list ? form.row_list[item] : item;
   const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const uint32_t group = q_heads / kv.num_kv_heads;
+  const uint32_t all_group = q_heads / kv.num_kv_heads, group_tiles = FORM ? (all_group + kMaxGroup - 1) / kMaxGroup : 1;
+  const uint32_t kvh = FORM ? blockIdx.x / group_tiles : blockIdx.x;
+  const uint32_t g_first = FORM ? blockIdx.x % group_tiles * kMaxGroup : 0;  // query heads of this CTA inside the kv head's group
+  const uint32_t group = FORM ? min((uint32_t)kMaxGroup, all_group - g_first) : all_group;
+  const uint32_t head_first = kvh * all_group + g_first;
   const uint32_t ctx = batch.query_positions[row] + 1;  // attention.rs:253
-  const uint32_t *table = batch.tables_flat + batch.table_offsets[batch.seq_of_row[row]];
+  const uint32_t seq = batch.seq_of_row[row];
+  const uint32_t *table = batch.tables_flat + batch.table_offsets[seq];
+  const uint32_t first_key = FORM ? form.range.first(ctx - 1) : 0, block0 = first_key / kBlk;
   const uint32_t nblocks = (ctx + kBlk - 1) / kBlk;
+  // blocks from this one on hold rows of this step
+  const uint32_t fresh_block = FORM && form.first_row ? batch.query_positions[form.first_row[seq]] / kBlk : nblocks - 1;
   // Context split: a contiguous range of blocks; warps interleave inside it.
   // Splits of this row: with a length-proportional plan a row is cut into pieces of about
   // blocks_per_split blocks (a short context is not cut at all, a long one up to gridDim.z times), so
   // the CTAs of a ragged batch carry similar amounts; CTAs beyond the row's count have nothing to do.
-  const uint32_t bps = scratch.blocks_per_split;
+  const uint32_t bps = FORM ? 0 : scratch.blocks_per_split;
   const uint32_t my_splits = bps ? min(max((nblocks + bps / 2) / bps, 1u), splits) : splits;
   if (split >= my_splits) return;
-  const uint32_t per_split = (nblocks + my_splits - 1) / my_splits;
-  const uint32_t b_begin = min(split * per_split, nblocks);
+  const uint32_t per_split = (nblocks - block0 + my_splits - 1) / my_splits;
+  const uint32_t b_begin = min(block0 + split * per_split, nblocks);
   const uint32_t b_end = min(b_begin + per_split, nblocks);
 
   pdl_trigger();
@@ -215,22 +237,22 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
   // dependency wait; the sequence's newest block (the one the preceding
   // RoPE/KV-write kernel is filling) and the query only after it.
   const uint32_t pre = min(my_count, (uint32_t)kStages);
-  uint32_t deferred = UINT32_MAX;
+  uint32_t deferred = pre;  // the blocks of a warp ascend
   for (uint32_t i = 0; i < pre; ++i) {
     const uint32_t pb = entry(i);
-    if (b_begin + warp + i * kWarps == nblocks - 1) {
+    if (b_begin + warp + i * kWarps >= fresh_block) {
       deferred = i;
-      continue;
+      break;
     }
     if (lane == 0) issue(i, pb);
   }
   pdl_wait();
-  if (deferred != UINT32_MAX) {
-    const uint32_t pb = entry(deferred);
-    if (lane == 0) issue(deferred, pb);
+  for (uint32_t i = deferred; i < pre; ++i) {
+    const uint32_t pb = entry(i);
+    if (lane == 0) issue(i, pb);
   }
 
-  if (fq.partial != nullptr) {
+  if (!FORM && fq.partial != nullptr) {
     // q heads of the group, then k, then v of this kv head, from the projection's partial sums:
     // 16 threads per head, four dims of each RoPE half per thread (tensor.rs:283-298, products
     // rounded separately like the reference).
@@ -265,13 +287,13 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
   }
 
   // Q^T as the B operand (k = dim, n = head): per 16-dim chunk two packed regs.
-  uint32_t qb[kHd / 16][2];
+  uint32_t qb[DK / 16][2];
   {
     const uint32_t g = lane >> 2;
-    const bf16 *qrow = fq.partial != nullptr ? stash + (g < group ? g : 0) * kHd
-                                             : q + ((size_t)row * q_heads + (size_t)kvh * group + g) * kHd;
+    const bf16 *qrow = !FORM && fq.partial != nullptr ? stash + (g < group ? g : 0) * kHd
+                                                      : q + ((size_t)row * q_heads + (size_t)head_first + g) * DK;
 #pragma unroll
-    for (int c = 0; c < kHd / 16; ++c) {
+    for (int c = 0; c < DK / 16; ++c) {
       if (g < group) {
         qb[c][0] = *reinterpret_cast<const uint32_t *>(qrow + c * 16 + (lane & 3) * 2);
         qb[c][1] = *reinterpret_cast<const uint32_t *>(qrow + c * 16 + 8 + (lane & 3) * 2);
@@ -284,11 +306,16 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
 
   // Online softmax state for the two heads this lane sees in the C fragment
   // (columns 2*(lane%4) and +1), in the log2 domain.
-  const float sl2 = 1.4426950408889634f / sqrtf((float)kHd);
+  const float sl2 = FORM && form.scale != 0.f ? form.scale * 1.4426950408889634f : 1.4426950408889634f / sqrtf((float)DK);
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
-  float o[kHd / 16][4];
+  if (FORM && form.sinks && split == 0 && warp == 0) {  // one of the partial results starts with the sink
+    const uint32_t g0 = (lane & 3) * 2;
+    if (g0 < group) m0 = form.sinks[head_first + g0] * 1.4426950408889634f, l0 = lane < 4 ? 1.f : 0.f;
+    if (g0 + 1 < group) m1 = form.sinks[head_first + g0 + 1] * 1.4426950408889634f, l1 = lane < 4 ? 1.f : 0.f;
+  }
+  float o[DV / 16][4];
 #pragma unroll
-  for (int t = 0; t < kHd / 16; ++t) o[t][0] = o[t][1] = o[t][2] = o[t][3] = 0.f;
+  for (int t = 0; t < DV / 16; ++t) o[t][0] = o[t][1] = o[t][2] = o[t][3] = 0.f;
 
   const uint32_t t_lo = lane >> 2, t_hi = t_lo + 8;  // token rows of this lane in the C fragment
   bool ok = true;
@@ -306,10 +333,10 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
       break;
     }
     const uint32_t kbase = smem_u32(my_ring + stage * kChunkBytes);
-    const uint32_t vbase = kbase + kBlk * kHd * 2;
+    const uint32_t vbase = kbase + kBlk * DK * 2;
     const uint32_t lb = b_begin + warp + i * kWarps;
     const uint32_t valid = min((uint32_t)kBlk, ctx - lb * kBlk);  // tokens of this block in context
-    if (fq.partial != nullptr && lb == nblocks - 1) {
+    if (!FORM && fq.partial != nullptr && lb == nblocks - 1) {
       // The block that holds this step's token: its k and v rows come from the stash. Lanes 0-15
       // copy the sixteen 16-byte groups of k, lanes 16-31 those of v, into the landed chunk (for
       // this step) and into the arena (for the steps to come), both in the arena's swizzled order.
@@ -328,25 +355,27 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
       const uint32_t mi = lane >> 3, r = lane & 7;
       const uint32_t t = r + (mi & 1) * 8;
 #pragma unroll
-      for (int c = 0; c < kHd / 16; ++c) {
+      for (int c = 0; c < DK / 16; ++c) {
         uint32_t a[4];
         const uint32_t chunk = (uint32_t)c * 2 + (mi >> 1);
-        ldmatrix_x4(a, kbase + t * (kHd * 2) + ((chunk ^ (t & 7)) << 4));
+        ldmatrix_x4(a, kbase + t * (DK * 2) + ((chunk ^ (t & 7)) << 4));
         mma_bf16_16816(s, a, qb[c][0], qb[c][1]);
       }
     }
     // scale into the log2 domain and mask slots beyond the context
-    s[0] = (t_lo < valid) ? s[0] * sl2 : -INFINITY;
-    s[1] = (t_lo < valid) ? s[1] * sl2 : -INFINITY;
-    s[2] = (t_hi < valid) ? s[2] * sl2 : -INFINITY;
-    s[3] = (t_hi < valid) ? s[3] * sl2 : -INFINITY;
+    const uint32_t hidden = FORM && first_key > lb * kBlk ? first_key - lb * kBlk : 0;  // tokens of this block before the first key
+    const bool see_lo = t_lo < valid && (!FORM || t_lo >= hidden), see_hi = t_hi < valid && (!FORM || t_hi >= hidden);
+    s[0] = see_lo ? s[0] * sl2 : -INFINITY;
+    s[1] = see_lo ? s[1] * sl2 : -INFINITY;
+    s[2] = see_hi ? s[2] * sl2 : -INFINITY;
+    s[3] = see_hi ? s[3] * sl2 : -INFINITY;
     float bm0 = fmaxf(s[0], s[2]), bm1 = fmaxf(s[1], s[3]);
 #pragma unroll
     for (int off = 4; off <= 16; off <<= 1) {
       bm0 = fmaxf(bm0, __shfl_xor_sync(0xffffffffu, bm0, off));
       bm1 = fmaxf(bm1, __shfl_xor_sync(0xffffffffu, bm1, off));
     }
-    const float mn0 = fmaxf(m0, bm0), mn1 = fmaxf(m1, bm1);  // finite: token 0 is always valid
+    const float mn0 = fmaxf(m0, bm0), mn1 = fmaxf(m1, bm1);  // finite: some token of the block is always valid
     const float c0 = fast_exp2(m0 - mn0), c1 = fast_exp2(m1 - mn1);
     const float p0 = fast_exp2(s[0] - mn0), p1 = fast_exp2(s[1] - mn1);
     const float p2 = fast_exp2(s[2] - mn0), p3 = fast_exp2(s[3] - mn1);
@@ -362,10 +391,10 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
       const uint32_t mi = lane >> 3, r = lane & 7;
       const uint32_t t = r + (mi >> 1) * 8;
 #pragma unroll
-      for (int mt = 0; mt < kHd / 16; ++mt) {
+      for (int mt = 0; mt < DV / 16; ++mt) {
         uint32_t a[4];
         const uint32_t chunk = (uint32_t)mt * 2 + (mi & 1);
-        ldmatrix_x4_trans(a, vbase + t * (kHd * 2) + ((chunk ^ (t & 7)) << 4));
+        ldmatrix_x4_trans(a, vbase + t * (DV * 2) + ((chunk ^ (t & 7)) << 4));
         o[mt][0] *= c0;
         o[mt][1] *= c1;
         o[mt][2] *= c0;
@@ -389,18 +418,18 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
   }
   __syncthreads();  // every warp is done with its ring: reuse it for the merge
 
-  float *mo = reinterpret_cast<float *>(dsmem);            // [kWarps][kMaxGroup][kHd]
-  float *mml = mo + kWarps * kMaxGroup * kHd;              // [kWarps][kMaxGroup][2]
+  float *mo = reinterpret_cast<float *>(dsmem);            // [kWarps][kMaxGroup][DV]
+  float *mml = mo + kWarps * kMaxGroup * DV;               // [kWarps][kMaxGroup][2]
   {
     const uint32_t g0 = (lane & 3) * 2;
 #pragma unroll
-    for (int mt = 0; mt < kHd / 16; ++mt) {
+    for (int mt = 0; mt < DV / 16; ++mt) {
       const uint32_t d = mt * 16 + (lane >> 2);
-      float *base = mo + ((size_t)warp * kMaxGroup) * kHd;
-      base[(g0 + 0) * kHd + d] = o[mt][0];
-      base[(g0 + 1) * kHd + d] = o[mt][1];
-      base[(g0 + 0) * kHd + d + 8] = o[mt][2];
-      base[(g0 + 1) * kHd + d + 8] = o[mt][3];
+      float *base = mo + ((size_t)warp * kMaxGroup) * DV;
+      base[(g0 + 0) * DV + d] = o[mt][0];
+      base[(g0 + 1) * DV + d] = o[mt][1];
+      base[(g0 + 0) * DV + d + 8] = o[mt][2];
+      base[(g0 + 1) * DV + d + 8] = o[mt][3];
     }
     if (lane < 4) {
       float *ml = mml + ((size_t)warp * kMaxGroup + g0) * 2;
@@ -408,8 +437,7 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
     }
   }
   __syncthreads();
-  {
-    const uint32_t d = threadIdx.x;  // kWarps*32 == kHd threads: one output dim each
+  for (uint32_t d = threadIdx.x; d < (uint32_t)DV; d += kWarps * 32) {  // one output dim per thread and round
     for (uint32_t g = 0; g < group; ++g) {
       float mall = -INFINITY;
 #pragma unroll
@@ -419,15 +447,17 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
       for (int w = 0; w < kWarps; ++w) {
         const float mw = mml[(w * kMaxGroup + g) * 2];
         const float wgt = (mw == -INFINITY) ? 0.f : fast_exp2(mw - mall);
-        acc += wgt * mo[((size_t)w * kMaxGroup + g) * kHd + d];
+        acc += wgt * mo[((size_t)w * kMaxGroup + g) * DV + d];
         L += wgt * mml[(w * kMaxGroup + g) * 2 + 1];
       }
-      const uint32_t head = kvh * group + g;
+      const uint32_t head = head_first + g;
       if (my_splits == 1) {
-        out[((size_t)row * q_heads + head) * kHd + d] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
+        const float v = L > 0.f ? acc / L : 0.f;
+        if (FORM) store_head_value(form, q_heads, DV, row, head, d, v, out);
+        else out[((size_t)row * q_heads + head) * DV + d] = __float2bfloat16_rn(v);
       } else {
-        const size_t pi = ((size_t)row * q_heads + head) * scratch.max_splits + split;
-        scratch.partial_out[pi * kHd + d] = acc;
+        const size_t pi = ((size_t)item * q_heads + head) * scratch.max_splits + split;
+        scratch.partial_out[pi * DV + d] = acc;
         if (d == 0) {
           scratch.partial_ml[pi * 2] = mall;
           scratch.partial_ml[pi * 2 + 1] = L;
@@ -435,7 +465,7 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
       }
     }
   }
-  if (my_splits > 1 && scratch.counters != nullptr) {
+  if (!FORM && my_splits > 1 && scratch.counters != nullptr) {
     // The CTA that arrives last at its (row, kv head) merges the splits of the group's heads: its
     // partials and everybody else's are visible (fence before the arrival, fence after it), and it
     // puts the counter back to zero for the next launch.
@@ -487,28 +517,31 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
   }
 }
 
-__global__ void __launch_bounds__(kHd)
+template <int DV, bool FORM>
+__global__ void __launch_bounds__(DV)
 decode_combine_kernel(DecodeScratch scratch, uint32_t splits, uint32_t q_heads, const uint32_t *__restrict__ query_positions,
-                      bf16 *__restrict__ out) {
+                      bf16 *__restrict__ out, AttnForm form) {
   pdl_trigger();
   pdl_wait();
-  const uint32_t row = blockIdx.x, head = blockIdx.y, d = threadIdx.x;
-  if (scratch.blocks_per_split) {  // the row's own split count, as the decode kernel computed it
-    const uint32_t nblocks = query_positions[row] / kBlk + 1, bps = scratch.blocks_per_split;
+  const uint32_t item = blockIdx.x, head = blockIdx.y, d = threadIdx.x;
+  if (!FORM && scratch.blocks_per_split) {  // the row's own split count, as the decode kernel computed it
+    const uint32_t nblocks = query_positions[item] / kBlk + 1, bps = scratch.blocks_per_split;
     splits = min(max((nblocks + bps / 2) / bps, 1u), splits);
     if (splits == 1) return;  // written by the decode kernel itself
   }
-  const size_t base = ((size_t)row * q_heads + head) * scratch.max_splits;
+  const size_t base = ((size_t)item * q_heads + head) * scratch.max_splits;
   float mall = -INFINITY;
   for (uint32_t s = 0; s < splits; ++s) mall = fmaxf(mall, scratch.partial_ml[(base + s) * 2]);
   float acc = 0.f, L = 0.f;
   for (uint32_t s = 0; s < splits; ++s) {
     const float ms = scratch.partial_ml[(base + s) * 2];
     const float w = (ms == -INFINITY) ? 0.f : fast_exp2(ms - mall);
-    acc += w * scratch.partial_out[(base + s) * kHd + d];
+    acc += w * scratch.partial_out[(base + s) * DV + d];
     L += w * scratch.partial_ml[(base + s) * 2 + 1];
   }
-  out[((size_t)row * q_heads + head) * kHd + d] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
+  const float v = L > 0.f ? acc / L : 0.f;
+  if (FORM) store_head_value(form, q_heads, DV, form.row_list ? form.row_list[item] : item, head, d, v, out);
+  else out[((size_t)item * q_heads + head) * DV + d] = __float2bfloat16_rn(v);
 }
 
 inline int after_launch(const char *stage) {
@@ -522,21 +555,22 @@ inline int after_launch(const char *stage) {
 template <typename T>
 int launch_paged_attention_generic(const T *q, const T *arena, KvLayout kv, uint32_t layer,
                                    AttnBatch batch, uint32_t q_heads, T *out,
-                                   cudaStream_t stream) {
+                                   cudaStream_t stream, AttnForm form) {
   if (batch.rows == 0) return ORION_OK;
-  if (kv.head_dim > kGenThreads * kGenMaxDimsPerThread)
+  const uint32_t widest = kv.head_dim > kv.v_dim() ? kv.head_dim : kv.v_dim();
+  if (widest > kGenThreads * kGenMaxDimsPerThread)
     return set_error(ORION_ERR_INTERNAL, "head_dim %u exceeds the attention kernel limit of %d",
-                     kv.head_dim, kGenThreads * kGenMaxDimsPerThread);
+                     widest, kGenThreads * kGenMaxDimsPerThread);
   const size_t smem = (kv.head_dim + kGenChunk) * sizeof(float);
   ORION_CUDA_CHECK("paged_attention",
                    launch_pdl(paged_attention_generic_kernel<T>, dim3(batch.rows, q_heads), dim3(kGenThreads), smem,
-                              stream, q, arena, kv, layer, batch, q_heads, out));
+                              stream, q, arena, kv, layer, batch, q_heads, out, form));
   return after_launch("paged_attention");
 }
 template int launch_paged_attention_generic<float>(const float *, const float *, KvLayout, uint32_t,
-                                                   AttnBatch, uint32_t, float *, cudaStream_t);
+                                                   AttnBatch, uint32_t, float *, cudaStream_t, AttnForm);
 template int launch_paged_attention_generic<bf16>(const bf16 *, const bf16 *, KvLayout, uint32_t,
-                                                  AttnBatch, uint32_t, bf16 *, cudaStream_t);
+                                                  AttnBatch, uint32_t, bf16 *, cudaStream_t, AttnForm);
 
 namespace {
 int g_decode_stages = 3;                 // ring depth per warp (2, 3 or 4)
@@ -551,7 +585,7 @@ uint32_t g_decode_min_blocks = std::getenv("ORION_DECODE_MIN_BLOCKS") ? (uint32_
 }  // namespace
 
 bool decode_attention_supported(KvLayout kv, uint32_t q_heads) {
-  return kv.head_dim == kHd && kv.block_size == kBlk && kv.swizzle == 1 && kv.num_kv_heads > 0 &&
+  return kv.head_dim == kHd && kv.v_dim() == kHd && kv.block_size == kBlk && kv.swizzle == 1 && kv.num_kv_heads > 0 &&
          q_heads % kv.num_kv_heads == 0 && q_heads / kv.num_kv_heads <= kMaxGroup;
 }
 
@@ -629,11 +663,11 @@ int launch_decode_stages(const bf16 *q, const bf16 *arena, KvLayout kv, uint32_t
                          FusedQkv fq, cudaStream_t stream) {
   static bool attr_set[kMaxDeviceOrdinals] = {};
   ORION_CUDA_CHECK("paged_decode attr",
-                   ensure_dynamic_smem(paged_decode_kernel<STAGES>, (int)decode_smem_bytes(STAGES), attr_set));
+                   ensure_dynamic_smem(paged_decode_kernel<STAGES, kHd, kHd, false>, (int)decode_smem_bytes(STAGES), attr_set));
   ORION_CUDA_CHECK("paged_decode",
-                   launch_pdl(paged_decode_kernel<STAGES>, dim3(kv.num_kv_heads, batch.rows, splits),
+                   launch_pdl(paged_decode_kernel<STAGES, kHd, kHd, false>, dim3(kv.num_kv_heads, batch.rows, splits),
                               dim3(kWarps * 32), (size_t)decode_smem_bytes(STAGES), stream, q, arena, kv, layer,
-                              batch, q_heads, splits, scratch, out, fq));
+                              batch, q_heads, splits, scratch, out, fq, AttnForm{}));
   return ORION_OK;
 }
 }  // namespace
@@ -661,11 +695,62 @@ int launch_paged_attention_decode(const bf16 *q, const bf16 *arena, KvLayout kv,
   }
   ORION_TRY(after_launch("paged_decode"));
   if (splits > 1 && scratch.counters == nullptr) {
-    ORION_CUDA_CHECK("decode_combine", launch_pdl(decode_combine_kernel, dim3(batch.rows, q_heads), dim3(kHd), 0,
-                                                  stream, scratch, splits, q_heads, batch.query_positions, out));
+    ORION_CUDA_CHECK("decode_combine", launch_pdl(decode_combine_kernel<kHd, false>, dim3(batch.rows, q_heads), dim3(kHd), 0,
+                                                  stream, scratch, splits, q_heads, batch.query_positions, out, AttnForm{}));
     ORION_TRY(after_launch("decode_combine"));
   }
   return ORION_OK;
+}
+
+// ---- other forms of attention ----------------------------------------------------------------------
+
+bool attention_form_supported(KvLayout kv, uint32_t q_heads) {
+  auto size = [](uint32_t d) { return d == 64 || d == 128; };
+  const uint32_t dk = kv.head_dim, dv = kv.v_dim();
+  return kv.block_size == kBlk && kv.swizzle == 1 && kv.num_kv_heads > 0 && q_heads % kv.num_kv_heads == 0 &&
+         q_heads / kv.num_kv_heads <= 128 && ((size(dk) && size(dv)) || (dk == 256 && dv == 256)) &&
+         (uint64_t)kv.num_layers * kv.num_blocks * kv.num_kv_heads < (1ull << 31);
+}
+
+namespace {
+uint32_t group_tiles(KvLayout kv, uint32_t q_heads) { return (q_heads / kv.num_kv_heads + kMaxGroup - 1) / kMaxGroup; }
+
+template <int DK, int DV>
+int launch_decode_form(const bf16 *q, const bf16 *arena, KvLayout kv, uint32_t layer, AttnBatch batch, uint32_t rows, uint32_t q_heads,
+                       uint32_t splits, DecodeScratch scratch, AttnForm form, bf16 *out, cudaStream_t stream) {
+  constexpr int kFormStages = 3;
+  static bool attr_set[kMaxDeviceOrdinals] = {};
+  ORION_CUDA_CHECK("paged_decode attr", ensure_dynamic_smem(paged_decode_kernel<kFormStages, DK, DV, true>,
+                                                            (int)decode_smem_bytes(kFormStages, DK, DV), attr_set));
+  ORION_CUDA_CHECK("paged_decode", launch_pdl(paged_decode_kernel<kFormStages, DK, DV, true>,
+                                              dim3(kv.num_kv_heads * group_tiles(kv, q_heads), rows, splits), dim3(kWarps * 32),
+                                              (size_t)decode_smem_bytes(kFormStages, DK, DV), stream, q, arena, kv, layer, batch, q_heads,
+                                              splits, scratch, out, FusedQkv{}, form));
+  ORION_TRY(after_launch("paged_decode"));
+  if (splits == 1) return ORION_OK;
+  ORION_CUDA_CHECK("decode_combine", launch_pdl(decode_combine_kernel<DV, true>, dim3(rows, q_heads), dim3(DV), 0, stream, scratch, splits,
+                                                q_heads, batch.query_positions, out, form));
+  return after_launch("decode_combine");
+}
+}  // namespace
+
+uint32_t decode_form_splits(KvLayout kv, uint32_t q_heads, uint32_t rows, uint32_t most_keys) {
+  return decode_choose_splits(rows, kv.num_kv_heads * group_tiles(kv, q_heads), most_keys - 1, kv.block_size, 32);
+}
+
+int launch_paged_attention_decode_form(const bf16 *q, const bf16 *arena, KvLayout kv, uint32_t layer, AttnBatch batch, uint32_t rows,
+                                       uint32_t q_heads, uint32_t splits, DecodeScratch scratch, AttnForm form, bf16 *out,
+                                       cudaStream_t stream) {
+  if (rows == 0) return ORION_OK;
+  if (!attention_form_supported(kv, q_heads)) return set_error(ORION_ERR_INTERNAL, "decode attention kernel does not cover this shape");
+  if (splits < 1) splits = 1;
+  if (splits > 1 && (scratch.partial_out == nullptr || splits > scratch.max_splits))
+    return set_error(ORION_ERR_INTERNAL, "decode attention scratch too small for %u splits", splits);
+  const uint32_t dk = kv.head_dim, dv = kv.v_dim();
+  auto run = dk == 256 ? launch_decode_form<256, 256>
+             : dk == 64 ? (dv == 64 ? launch_decode_form<64, 64> : launch_decode_form<64, 128>)
+                        : (dv == 64 ? launch_decode_form<128, 64> : launch_decode_form<128, 128>);
+  return run(q, arena, kv, layer, batch, rows, q_heads, splits, scratch, form, out, stream);
 }
 
 int decode_poll_error(uint32_t *code) {

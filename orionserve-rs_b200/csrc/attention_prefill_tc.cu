@@ -1,12 +1,12 @@
-// Chunked-prefill paged attention on the 5th-generation tensor cores (bf16, head_dim 128, 16-token
-// blocks): the same arithmetic as attention_prefill.cu (transformer.rs:281-326, causal by absolute
+// Chunked-prefill paged attention on the 5th-generation tensor cores (bf16, head_dim 128, or 64 to 256
+// with the FORM parameter; 16-token blocks): the same arithmetic as attention_prefill.cu (transformer.rs:281-326, causal by absolute
 // position, attention.rs:252-253), with S = Q K^T and O += P V as tcgen05 MMAs whose accumulators
 // live in tensor memory.
 //
 // One CTA per (kv head, tile of query rows of one sequence), two CTAs per SM. The MMA's M dimension
 // is (query position, query head of the GQA group), 128 rows; a key tile is 64 keys = four KV blocks.
 //   warp 0     one lane fetches K and V of a key tile with tiled TMA copies straight out of the paged
-//              arena (one 3-D tensor map over [chunk][k|v x slot][dim]; a 16-slot x 64-dim box lands as
+//              arena (3-D tensor maps over [chunk][slot][dim], one for K and one for V; a 16-slot x 64-dim box lands as
 //              sixteen 128-byte rows, and because the arena keeps the 16-byte groups of a row XOR-permuted
 //              by slot & 7, those rows ARE the 128-byte-swizzled operand layout the MMA expects);
 //   warp 1     allocates tensor memory; one lane issues S = Q K^T (M 128, N 64, K 128) and, once the
@@ -35,27 +35,41 @@ constexpr int kM = 128;      // (position, head) rows per CTA
 constexpr int kKeys = 64;    // keys per tile
 constexpr int kStages = 2;
 constexpr int kThreads = 192;
-constexpr int kQBytes = 2 * kM * 128;        // two 64-dim halves of [128 rows][128 bytes]
-constexpr int kKBytes = 2 * kKeys * 128;     // two 64-dim halves of [64 keys][128 bytes]; P reuses it as [128 rows][128 bytes]
-constexpr int kStageBytes = 2 * kKBytes;     // K tile, then V tile
-constexpr int kBarOffset = kQBytes + kStages * kStageBytes;
-constexpr int kSmem = kBarOffset + 256 + 1024;
-constexpr uint32_t kTmemCols = 256;          // S: columns 0..63, O: columns 64..191
-constexpr uint32_t kTmemO = 64;
+constexpr uint32_t kTmemO = 64;              // S: columns 0..63 of tensor memory, O behind them
+// DK, DV: sizes of the K and V rows, multiples of 64.
+template <int DK, int DV>
+struct PrefillTcConfig {
+  static constexpr int kQBytes = DK / 64 * kM * 128;     // 64-dim slabs of [128 rows][128 bytes]
+  static constexpr int kKBytes = DK / 64 * kKeys * 128;  // 64-dim slabs of [64 keys][128 bytes]
+  static constexpr int kVBytes = DV / 64 * kKeys * 128;
+  static constexpr int kStageBytes = kKBytes + kVBytes;  // K tile, then V tile
+  // P, [128 rows][128 bytes], takes the place of the K tile where that is large enough
+  static constexpr bool kOwnP = kKBytes < kM * 128;
+  static constexpr int kPOffset = kQBytes + kStages * kStageBytes;
+  static constexpr int kBarOffset = kPOffset + (kOwnP ? kM * 128 : 0);
+  static constexpr int kSmem = kBarOffset + 256 + 1024;
+  static constexpr uint32_t kTmemCols = DV <= 64 ? 128 : (DV <= 128 ? 256 : 512);
+};
 constexpr float kRescaleThreshold = 8.0f;    // log2 units
 
 __device__ uint32_t g_prefill_tc_error = 0;
 
 __device__ __forceinline__ void softmax_bar() { asm volatile("bar.sync 1, 128;" ::: "memory"); }  // warps 2..5
 
-__global__ void __launch_bounds__(kThreads, 2)
-paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16 *__restrict__ q, KvLayout kv, uint32_t layer,
-                        AttnBatch batch, const PrefillTile *__restrict__ tiles, uint32_t q_heads, bf16 *__restrict__ out) {
+// FORM: the mask, sinks and gate of `form`; without it those branches and arguments are compiled out.
+template <int DK, int DV, bool FORM>
+__global__ void __launch_bounds__(kThreads, DV <= 128 ? 2 : 1)
+paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const bf16 *__restrict__ q,
+                        KvLayout kv, uint32_t layer, AttnBatch batch, const PrefillTile *__restrict__ tiles, uint32_t q_heads,
+                        bf16 *__restrict__ out, AttnForm form) {
+  using Cfg = PrefillTcConfig<DK, DV>;
+  constexpr int kQBytes = Cfg::kQBytes, kKBytes = Cfg::kKBytes, kStageBytes = Cfg::kStageBytes;
   extern __shared__ uint8_t raw_smem[];
   uint8_t *smem = reinterpret_cast<uint8_t *>((reinterpret_cast<uintptr_t>(raw_smem) + 1023) & ~uintptr_t(1023));
-  uint8_t *q_smem = smem;                 // [half 2][row 128][128 B]
-  uint8_t *ring = smem + kQBytes;         // [stage][K tile 16 KiB | V tile 16 KiB]
-  uint64_t *kv_full = reinterpret_cast<uint64_t *>(smem + kBarOffset);
+  uint8_t *q_smem = smem;                 // [slab][row 128][128 B]
+  uint8_t *ring = smem + kQBytes;         // [stage][K tile | V tile]
+  auto p_tile = [&](uint32_t stage) { return Cfg::kOwnP ? smem + Cfg::kPOffset : ring + stage * kStageBytes; };
+  uint64_t *kv_full = reinterpret_cast<uint64_t *>(smem + Cfg::kBarOffset);
   uint64_t *kv_empty = kv_full + kStages;
   uint64_t *q_ready = kv_empty + kStages;
   uint64_t *s_ready = q_ready + 1;
@@ -63,13 +77,15 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16 *
   uint64_t *o_ready = p_ready + 1;
   uint32_t *tmem_slot = reinterpret_cast<uint32_t *>(o_ready + 1);
 
-  pdl_trigger();
+  if (!FORM) pdl_trigger();
   const uint32_t kvh = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const PrefillTile tile = tiles[blockIdx.y];
   const uint32_t group = q_heads / kv.num_kv_heads;
   const uint32_t *table = batch.tables_flat + batch.table_offsets[tile.seq];
   const uint32_t nblocks = tile.max_position / kBlk + 1;
-  const uint32_t ntiles = (nblocks + (kKeys / kBlk) - 1) / (kKeys / kBlk);
+  // key tiles start at the block of the first key that the tile's first row sees
+  const uint32_t block0 = FORM ? form.range.first(batch.query_positions[tile.row_start]) / kBlk : 0;
+  const uint32_t ntiles = (nblocks - block0 + (kKeys / kBlk) - 1) / (kKeys / kBlk);
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < kStages; ++s) {
@@ -83,12 +99,14 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16 *
     mbar_fence_init();
   }
   if (warp == 1) {
-    tmem_alloc(tmem_slot, kTmemCols);
+    tmem_alloc(tmem_slot, Cfg::kTmemCols);
     tmem_relinquish();
   }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
+  // here only now: a dependent CTA that waits for this grid must not hold tensor memory that this CTA still needs
+  if (FORM) pdl_trigger();
   const uint32_t tmem_base = *tmem_slot;
   bool ok = true;
   // Once any wait of this CTA has run out, later waits give up at once: every thread still walks
@@ -115,22 +133,23 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16 *
         uint8_t *k_dst = ring + s * kStageBytes, *v_dst = k_dst + kKBytes;
 #pragma unroll
         for (uint32_t b = 0; b < kKeys / kBlk; ++b) {
-          // a block past the row's context repeats block 0: its keys are masked, its values must be finite
-          const uint32_t lb = j * (kKeys / kBlk) + b;
-          const uint32_t block = table[lb < nblocks ? lb : 0];
+          // a block past the row's context repeats the first one: its keys are masked, its values must be finite
+          const uint32_t lb = block0 + j * (kKeys / kBlk) + b;
+          const uint32_t block = table[lb < nblocks ? lb : block0];
           const int chunk = (int)((chunk0 + block) * kv.num_kv_heads + kvh);
 #pragma unroll
-          for (int h = 0; h < 2; ++h) {
-            tma_load_3d(k_dst + h * (kKeys * 128) + b * (kBlk * 128), &map_kv, h * 64, 0, chunk, &kv_full[s]);
-            tma_load_3d(v_dst + h * (kKeys * 128) + b * (kBlk * 128), &map_kv, h * 64, kBlk, chunk, &kv_full[s]);
-          }
+          for (int h = 0; h < DK / 64; ++h)
+            tma_load_3d(k_dst + h * (kKeys * 128) + b * (kBlk * 128), &map_k, h * 64, 0, chunk, &kv_full[s]);
+#pragma unroll
+          for (int h = 0; h < DV / 64; ++h)
+            tma_load_3d(v_dst + h * (kKeys * 128) + b * (kBlk * 128), &map_v, h * 64, 0, chunk, &kv_full[s]);
         }
       }
     }
   } else if (warp == 1) {
     // ---- MMA issue ----
     if (lane == 0) {
-      constexpr uint32_t idesc_s = idesc(kM, kKeys, false), idesc_o = idesc(kM, kHd, true);
+      constexpr uint32_t idesc_s = idesc(kM, kKeys, false), idesc_o = idesc(kM, DV, true);
       const uint32_t qa = smem_u32(q_smem);
       if (!wait(q_ready, 0)) ok = false;
       for (uint32_t j = 0; ok && j < ntiles; ++j) {
@@ -138,9 +157,9 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16 *
         if (!wait(&kv_full[s], (j / kStages) & 1)) { ok = false; break; }
         tc_fence_after();
         const uint32_t ka = smem_u32(ring + s * kStageBytes), va = ka + kKBytes;
-        // S = Q K^T: two 64-dim halves, four 16-dim steps each (+32 bytes inside the swizzle atom)
+        // S = Q K^T: 64-dim slabs, four 16-dim steps each (+32 bytes inside the swizzle atom)
 #pragma unroll
-        for (int ks = 0; ks < kHd / 16; ++ks) {
+        for (int ks = 0; ks < DK / 16; ++ks) {
           const uint32_t h = ks >> 2, kk = ks & 3;
           umma_bf16(tmem_base, desc_k_sw128(qa + h * (kM * 128) + kk * 32), desc_k_sw128(ka + h * (kKeys * 128) + kk * 32),
                     idesc_s, ks > 0 ? 1u : 0u);
@@ -148,10 +167,11 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16 *
         umma_commit(s_ready);
         if (!wait(p_ready, j & 1)) { ok = false; break; }
         tc_fence_after();
-        // O (+)= P V: P sits where the K tile was, [128 rows][64 keys]; V is [key][dim]: MN-major, 16 keys per step
+        // O (+)= P V: P is [128 rows][64 keys] (where the K tile was, if it fits there); V is [key][dim]: MN-major, 16 keys per step
+        const uint32_t pa = smem_u32(p_tile(s));
 #pragma unroll
         for (int ks = 0; ks < kKeys / 16; ++ks)
-          umma_bf16(tmem_base + kTmemO, desc_k_sw128(ka + ks * 32), desc_mn_sw128(va + ks * (16 * 128), kKeys * 128, 1024),
+          umma_bf16(tmem_base + kTmemO, desc_k_sw128(pa + ks * 32), desc_mn_sw128(va + ks * (16 * 128), kKeys * 128, 1024),
                     idesc_o, (j > 0 || ks > 0) ? 1u : 0u);
         umma_commit(o_ready);
         umma_commit(&kv_empty[s]);
@@ -167,10 +187,11 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16 *
     const uint32_t taddr = tmem_base + ((quad * 32u) << 16);
     pdl_wait();  // q comes from the preceding kernel
     const int pos = valid ? (int)batch.query_positions[row] : -1;
+    const int low = FORM && valid ? (int)form.range.first((uint32_t)pos) : 0;  // first key this row sees
     {
-      const uint4 *src = reinterpret_cast<const uint4 *>(q + ((size_t)row * q_heads + head) * kHd);
+      const uint4 *src = reinterpret_cast<const uint4 *>(q + ((size_t)row * q_heads + head) * DK);
 #pragma unroll
-      for (uint32_t c = 0; c < 16; ++c) {
+      for (uint32_t c = 0; c < DK / 8; ++c) {
         const uint4 v = valid ? src[c] : make_uint4(0u, 0u, 0u, 0u);
         *reinterpret_cast<uint4 *>(q_smem + (c >> 3) * (kM * 128) + m * 128 + (((c & 7) ^ (m & 7)) << 4)) = v;
       }
@@ -179,8 +200,9 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16 *
     softmax_bar();
     if (threadIdx.x == 64) mbar_arrive(q_ready);
 
-    const float sl2 = 1.4426950408889634f / sqrtf((float)kHd);
+    const float sl2 = FORM && form.scale != 0.f ? form.scale * 1.4426950408889634f : 1.4426950408889634f / sqrtf((float)DK);
     float ref = -INFINITY, l = 0.f;
+    if (FORM && form.sinks) ref = form.sinks[head] * 1.4426950408889634f, l = 1.f;
     for (uint32_t j = 0; j < ntiles; ++j) {
       const uint32_t s = j % kStages;
       if (!__all_sync(0xffffffffu, wait(s_ready, j & 1))) ok = false;  // no break: the barriers below stay matched
@@ -189,11 +211,11 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16 *
       tmem_ld32(taddr, sr[0]);
       tmem_ld32(taddr + 32, sr[1]);
       tmem_ld_wait();
-      const int key0 = (int)(j * kKeys);
+      const int key0 = (int)(block0 * kBlk + j * kKeys);
       float mx = -INFINITY;
 #pragma unroll
       for (int i = 0; i < kKeys; ++i) {
-        const float v = (key0 + i <= pos) ? __uint_as_float(sr[i >> 5][i & 31]) * sl2 : -INFINITY;
+        const float v = (key0 + i <= pos && (!FORM || key0 + i >= low)) ? __uint_as_float(sr[i >> 5][i & 31]) * sl2 : -INFINITY;
         sr[i >> 5][i & 31] = __float_as_uint(v);
         mx = fmaxf(mx, v);
       }
@@ -208,7 +230,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16 *
         // rescale this warp's rows of O in tensor memory (the MMAs of the previous tile have completed:
         // S of this tile was issued after them)
 #pragma unroll 1
-        for (uint32_t c = 0; c < kHd; c += 32) {
+        for (uint32_t c = 0; c < DV; c += 32) {
           uint32_t orow[32];
           tmem_ld32(taddr + kTmemO + c, orow);
           tmem_ld_wait();
@@ -220,7 +242,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16 *
       }
       l *= corr;
       const float base = ref == -INFINITY ? 0.f : ref;
-      uint8_t *p_row = ring + s * kStageBytes + m * 128;
+      uint8_t *p_row = p_tile(s) + m * 128;
 #pragma unroll
       for (int c = 0; c < kKeys / 8; ++c) {
         float p[8];
@@ -240,51 +262,63 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const bf16 *
     // ---- epilogue: O / l ----
     if (!__all_sync(0xffffffffu, ntiles == 0 || wait(o_ready, (ntiles - 1) & 1))) ok = false;
     tc_fence_after();
-    const float inv = l > 0.f ? 1.0f / l : 0.f;
-    bf16 *dst = out + ((size_t)row * q_heads + head) * kHd;
+    float inv = l > 0.f ? 1.0f / l : 0.f;
+    if (FORM && form.gate) inv *= form.gate[(size_t)row * q_heads + head];
+    const uint32_t od = FORM && form.out_dim ? form.out_dim : DV, ldo = FORM && form.ldo ? form.ldo : q_heads * od;
+    const bool whole_groups = !FORM || (od % 8 == 0 && ldo % 8 == 0);
+    bf16 *dst = out + (size_t)row * ldo + (size_t)head * od;
 #pragma unroll 1
-    for (uint32_t c = 0; c < kHd; c += 32) {
+    for (uint32_t c = 0; c < DV; c += 32) {
       uint32_t orow[32];
       tmem_ld32(taddr + kTmemO + c, orow);
       tmem_ld_wait();
       if (valid) {
 #pragma unroll
-        for (int i = 0; i < 32; i += 8)
-          *reinterpret_cast<uint4 *>(dst + c + i) =
-              make_uint4(pack2(__uint_as_float(orow[i]) * inv, __uint_as_float(orow[i + 1]) * inv),
-                         pack2(__uint_as_float(orow[i + 2]) * inv, __uint_as_float(orow[i + 3]) * inv),
-                         pack2(__uint_as_float(orow[i + 4]) * inv, __uint_as_float(orow[i + 5]) * inv),
-                         pack2(__uint_as_float(orow[i + 6]) * inv, __uint_as_float(orow[i + 7]) * inv));
+        for (int i = 0; i < 32; i += 8) {
+          if (!whole_groups) {
+#pragma unroll
+            for (int k = 0; k < 8; ++k)
+              if (c + i + k < od) dst[c + i + k] = __float2bfloat16_rn(__uint_as_float(orow[i + k]) * inv);
+          } else if (!FORM || c + i < od) {
+            *reinterpret_cast<uint4 *>(dst + c + i) =
+                make_uint4(pack2(__uint_as_float(orow[i]) * inv, __uint_as_float(orow[i + 1]) * inv),
+                           pack2(__uint_as_float(orow[i + 2]) * inv, __uint_as_float(orow[i + 3]) * inv),
+                           pack2(__uint_as_float(orow[i + 4]) * inv, __uint_as_float(orow[i + 5]) * inv),
+                           pack2(__uint_as_float(orow[i + 6]) * inv, __uint_as_float(orow[i + 7]) * inv));
+          }
+        }
       }
     }
   }
   if (!ok && lane == 0) atomicOr(&g_prefill_tc_error, 1u);
   tc_fence_before();
   __syncthreads();
-  if (warp == 1) tmem_dealloc(tmem_base, kTmemCols);
+  if (warp == 1) tmem_dealloc(tmem_base, Cfg::kTmemCols);
 }
 
 // ---- host side -----------------------------------------------------------------
 
-// The arena as [chunk = (layer, block, kv head)][32 rows: 16 K slots then 16 V slots][128 dims]; a box is 16 rows x
-// 64 dims with no swizzle of its own (the rows are stored pre-permuted).
-int arena_map(const bf16 *arena, KvLayout kv, const CUtensorMap **out) {
+// The K or the V rows of the arena as [chunk = (layer, block, kv head)][16 slots][dims]; a box is 16 rows x 64 dims with
+// no swizzle of its own (the rows are stored pre-permuted).
+int arena_map(const bf16 *arena, KvLayout kv, bool values, const CUtensorMap **out) {
   static std::mutex mu;
-  static std::map<std::tuple<const void *, uint64_t>, CUtensorMap> cache;
+  static std::map<std::tuple<const void *, uint64_t, uint32_t, uint32_t, bool>, CUtensorMap> cache;
   EncodeFn fn = encode_fn();
   if (!fn) return set_error(ORION_ERR_BACKEND, "backend cuda failed at tensor map: driver entry point missing");
   const uint64_t chunks = (uint64_t)kv.num_layers * kv.num_blocks * kv.num_kv_heads;
   std::lock_guard<std::mutex> lock(mu);
-  auto key = std::make_tuple((const void *)arena, chunks);
+  auto key = std::make_tuple((const void *)arena, chunks, kv.head_dim, kv.v_dim(), values);
   auto it = cache.find(key);
   if (it == cache.end()) {
     if (cache.size() > 4096) cache.clear();
     CUtensorMap m;
-    const cuuint64_t dims[3] = {(cuuint64_t)kHd, (cuuint64_t)2 * kBlk, chunks};
-    const cuuint64_t strides[2] = {(cuuint64_t)kHd * 2, (cuuint64_t)2 * kBlk * kHd * 2};
+    const cuuint64_t cols = values ? kv.v_dim() : kv.head_dim;
+    const cuuint64_t dims[3] = {cols, (cuuint64_t)kBlk, chunks};
+    const cuuint64_t strides[2] = {cols * 2, (cuuint64_t)kv.chunk_elems() * 2};
+    bf16 *base = const_cast<bf16 *>(arena) + (values ? (size_t)kBlk * kv.head_dim : 0);
     const cuuint32_t box[3] = {64, (cuuint32_t)kBlk, 1};
     const cuuint32_t estr[3] = {1, 1, 1};
-    const CUresult r = fn(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<bf16 *>(arena), dims, strides, box, estr,
+    const CUresult r = fn(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, base, dims, strides, box, estr,
                           CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_NONE, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
                           CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     if (r != CUDA_SUCCESS)
@@ -293,6 +327,22 @@ int arena_map(const bf16 *arena, KvLayout kv, const CUtensorMap **out) {
     it = cache.emplace(key, m).first;
   }
   *out = &it->second;
+  return ORION_OK;
+}
+
+template <int DK, int DV, bool FORM>
+int launch_prefill_tc(const bf16 *q, const bf16 *arena, KvLayout kv, uint32_t layer, AttnBatch batch, const PrefillTile *tiles,
+                      uint32_t num_tiles, uint32_t q_heads, AttnForm form, bf16 *out, cudaStream_t stream) {
+  using Cfg = PrefillTcConfig<DK, DV>;
+  const CUtensorMap *mk = nullptr, *mv = nullptr;
+  ORION_TRY(arena_map(arena, kv, false, &mk));
+  ORION_TRY(arena_map(arena, kv, true, &mv));
+  static bool attr_set[kMaxDeviceOrdinals] = {};
+  ORION_CUDA_CHECK("paged_prefill_tc attr", ensure_dynamic_smem(paged_prefill_tc_kernel<DK, DV, FORM>, Cfg::kSmem, attr_set));
+  ORION_CUDA_CHECK("paged_prefill_tc", launch_pdl(paged_prefill_tc_kernel<DK, DV, FORM>, dim3(kv.num_kv_heads, num_tiles), dim3(kThreads),
+                                                  (size_t)Cfg::kSmem, stream, *mk, *mv, q, kv, layer, batch, tiles, q_heads, out, form));
+  count_launch();
+  ORION_CUDA_CHECK("paged_prefill_tc", cudaGetLastError());
   return ORION_OK;
 }
 
@@ -312,15 +362,20 @@ int launch_paged_attention_prefill_tc(const bf16 *q, const bf16 *arena, KvLayout
   if (num_tiles == 0) return ORION_OK;
   if (!prefill_attention_tc_supported(kv, q_heads, arena))
     return set_error(ORION_ERR_INTERNAL, "tensor-core prefill attention does not cover this shape");
-  const CUtensorMap *map = nullptr;
-  ORION_TRY(arena_map(arena, kv, &map));
-  static bool attr_set[kMaxDeviceOrdinals] = {};
-  ORION_CUDA_CHECK("paged_prefill_tc attr", ensure_dynamic_smem(paged_prefill_tc_kernel, (int)kSmem, attr_set));
-  ORION_CUDA_CHECK("paged_prefill_tc", launch_pdl(paged_prefill_tc_kernel, dim3(kv.num_kv_heads, num_tiles), dim3(kThreads),
-                                                  (size_t)kSmem, stream, *map, q, kv, layer, batch, tiles, q_heads, out));
-  count_launch();
-  ORION_CUDA_CHECK("paged_prefill_tc", cudaGetLastError());
-  return ORION_OK;
+  return launch_prefill_tc<kHd, kHd, false>(q, arena, kv, layer, batch, tiles, num_tiles, q_heads, AttnForm{}, out, stream);
+}
+
+int launch_paged_attention_prefill_form(const bf16 *q, const bf16 *arena, KvLayout kv, uint32_t layer, AttnBatch batch,
+                                        const PrefillTile *tiles, uint32_t num_tiles, uint32_t q_heads, AttnForm form, bf16 *out,
+                                        cudaStream_t stream) {
+  if (num_tiles == 0) return ORION_OK;
+  if (!attention_form_supported(kv, q_heads) || encode_fn() == nullptr)
+    return set_error(ORION_ERR_INTERNAL, "tensor-core prefill attention does not cover this shape");
+  const uint32_t dk = kv.head_dim, dv = kv.v_dim();
+  auto run = dk == 256 ? launch_prefill_tc<256, 256, true>
+             : dk == 64 ? (dv == 64 ? launch_prefill_tc<64, 64, true> : launch_prefill_tc<64, 128, true>)
+                        : (dv == 64 ? launch_prefill_tc<128, 64, true> : launch_prefill_tc<128, 128, true>);
+  return run(q, arena, kv, layer, batch, tiles, num_tiles, q_heads, form, out, stream);
 }
 
 int prefill_tc_poll_error(uint32_t *code) {

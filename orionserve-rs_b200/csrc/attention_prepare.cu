@@ -1,0 +1,205 @@
+// What attention with per-projection query / key norms, rotation in neighbouring pairs and per-head output gates needs
+// between its joint projection and the attention kernels: one pass over the projection's partial sums that normalises,
+// rotates, and leaves queries, cached keys and values, and gates. One CTA per row.
+#include "kernels.h"
+#include "mma.cuh"
+
+namespace orion {
+namespace {
+
+__device__ __forceinline__ float fold(const float *p, uint32_t splits, size_t stride) {
+  float v = p[0];
+  for (uint32_t s = 1; s < splits; ++s) v += p[s * stride];
+  return v;
+}
+
+// Sums of two values over the CTA (at most 32 warps), the same in every thread.
+__device__ __forceinline__ float2 block_sum2(float a, float b, float2 *red) {
+  a = warp_sum(a), b = warp_sum(b);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = make_float2(a, b);
+  __syncthreads();
+  float2 t = make_float2(0.f, 0.f);
+  for (uint32_t w = 0; w < blockDim.x / 32; ++w) t.x += red[w].x, t.y += red[w].y;
+  return t;
+}
+
+// Any sizes, one column at a time; the partial sums are folded once for the norms and once for the values.
+template <typename T>
+__global__ void __launch_bounds__(256)
+attention_prepare_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, AttnInputs in,
+                         const uint32_t *__restrict__ positions, const uint32_t *__restrict__ slot_block,
+                         const uint32_t *__restrict__ slot_slot, T *__restrict__ q_out, T *__restrict__ arena, KvLayout kv, uint32_t layer,
+                         float *__restrict__ gate) {
+  __shared__ float2 red[32];
+  pdl_trigger();
+  pdl_wait();
+  const uint32_t row = blockIdx.x, tid = threadIdx.x, half = in.rope_dims / 2;
+  const float *p = partial + (size_t)row * in.ld;
+  const uint32_t nq = in.q_heads * in.dim, nk = in.kv_heads * in.dim, nv = in.kv_heads * in.value_dim;
+  float sq = 0.f, sk = 0.f;
+  for (uint32_t i = tid; i < nq + nk; i += blockDim.x) {
+    const float v = fold(p + i, splits, split_stride);
+    if (i < nq) sq += v * v;
+    else sk += v * v;
+  }
+  const float2 ss = block_sum2(sq, sk, red);
+  const float scale_q = 1.0f / sqrtf(ss.x / (float)nq + in.eps), scale_k = 1.0f / sqrtf(ss.y / (float)nk + in.eps);
+  const float *cs = in.rope_cos + (size_t)positions[row] * half, *sn = in.rope_sin + (size_t)positions[row] * half;
+  const uint32_t block = slot_block[row], slot = slot_slot[row];
+  for (uint32_t i = tid; i < nq + nk; i += blockDim.x) {
+    const bool is_q = i < nq;
+    const uint32_t c = is_q ? i : i - nq, head = c / in.dim, d = c % in.dim;
+    const float *w = is_q ? in.q_norm : in.k_norm;
+    const float scale = is_q ? scale_q : scale_k;
+    auto value = [&](uint32_t at) { return w ? fold(p + at, splits, split_stride) * scale * w[is_q ? at : at - nq] : fold(p + at, splits, split_stride); };
+    float v = value(i);
+    if (d < 2 * half) {
+      const float other = value((d & 1) ? i - 1 : i + 1), co = cs[d >> 1], si = sn[d >> 1];
+      v = (d & 1) ? v * co + other * si : v * co - other * si;
+    }
+    if (is_q) q_out[((size_t)row * in.q_heads + head) * kv.head_dim + d] = from_f32<T>(v);
+    else arena[kv.row(layer, block, head, 0, slot) + kv.col(slot, d)] = from_f32<T>(v);
+  }
+  for (uint32_t i = tid; i < nv; i += blockDim.x)
+    arena[kv.row(layer, block, i / in.value_dim, 1, slot) + kv.col(slot, i % in.value_dim)] = from_f32<T>(fold(p + nq + nk + i, splits, split_stride));
+  if (gate)
+    for (uint32_t h = tid; h < in.q_heads; h += blockDim.x)
+      gate[(size_t)row * in.q_heads + h] = sigmoid_f(fold(p + nq + nk + nv + h, splits, split_stride));
+}
+
+template <typename T>
+__device__ __forceinline__ void store4(T *p, float4 v);
+template <>
+__device__ __forceinline__ void store4<float>(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
+template <>
+__device__ __forceinline__ void store4<bf16>(bf16 *p, float4 v) {
+  *reinterpret_cast<uint2 *>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+}
+
+// The same, four columns per thread and GROUPS rounds kept in registers, so each partial sum is read once: every size and
+// stride a multiple of four.
+template <typename T, int GROUPS>
+__global__ void __launch_bounds__(512)
+attention_prepare_vec_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, AttnInputs in,
+                             const uint32_t *__restrict__ positions, const uint32_t *__restrict__ slot_block,
+                             const uint32_t *__restrict__ slot_slot, T *__restrict__ q_out, T *__restrict__ arena, KvLayout kv,
+                             uint32_t layer, float *__restrict__ gate) {
+  __shared__ float2 red[32];
+  pdl_trigger();
+  const uint32_t row = blockIdx.x, tid = threadIdx.x, half = in.rope_dims / 2;
+  const float *p = partial + (size_t)row * in.ld;
+  const uint32_t nq = in.q_heads * in.dim, nk = in.kv_heads * in.dim, nv = in.kv_heads * in.value_dim, all = nq + nk + nv;
+  const uint32_t pos = positions[row], block = slot_block[row], slot = slot_slot[row];
+  float4 gain[GROUPS];
+  float2 co[GROUPS], si[GROUPS];
+#pragma unroll
+  for (int g = 0; g < GROUPS; ++g) {  // gains and angles do not depend on the projection
+    const uint32_t i = (tid + g * blockDim.x) * 4;
+    gain[g] = make_float4(1.f, 1.f, 1.f, 1.f), co[g] = make_float2(1.f, 1.f), si[g] = make_float2(0.f, 0.f);
+    if (i < nq + nk) {
+      if (in.q_norm) gain[g] = *reinterpret_cast<const float4 *>(i < nq ? in.q_norm + i : in.k_norm + (i - nq));
+      const uint32_t d = (i < nq ? i : i - nq) % in.dim;
+      if (d < in.rope_dims) {
+        co[g] = *reinterpret_cast<const float2 *>(in.rope_cos + (size_t)pos * half + d / 2);
+        si[g] = *reinterpret_cast<const float2 *>(in.rope_sin + (size_t)pos * half + d / 2);
+      }
+    }
+  }
+  pdl_wait();
+  float4 v[GROUPS];
+  float sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int g = 0; g < GROUPS; ++g) {
+    const uint32_t i = (tid + g * blockDim.x) * 4;
+    v[g] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i >= all) continue;
+    v[g] = sum_slabs4(p + i, splits, split_stride);
+    const float s = v[g].x * v[g].x + v[g].y * v[g].y + v[g].z * v[g].z + v[g].w * v[g].w;
+    if (i < nq) sq += s;
+    else if (i < nq + nk) sk += s;
+  }
+  if (gate && tid < in.q_heads) gate[(size_t)row * in.q_heads + tid] = sigmoid_f(fold(p + all + tid, splits, split_stride));
+  const float2 ss = block_sum2(sq, sk, red);
+  const float scale_q = in.q_norm ? 1.0f / sqrtf(ss.x / (float)nq + in.eps) : 1.f;
+  const float scale_k = in.q_norm ? 1.0f / sqrtf(ss.y / (float)nk + in.eps) : 1.f;
+#pragma unroll
+  for (int g = 0; g < GROUPS; ++g) {
+    const uint32_t i = (tid + g * blockDim.x) * 4;
+    if (i >= all) continue;
+    float4 x = v[g];
+    if (i < nq + nk) {
+      const float s = i < nq ? scale_q : scale_k;
+      x = make_float4(x.x * s * gain[g].x, x.y * s * gain[g].y, x.z * s * gain[g].z, x.w * s * gain[g].w);
+      x = make_float4(x.x * co[g].x - x.y * si[g].x, x.y * co[g].x + x.x * si[g].x, x.z * co[g].y - x.w * si[g].y, x.w * co[g].y + x.z * si[g].y);
+    }
+    if (i < nq) {
+      store4<T>(q_out + ((size_t)row * in.q_heads + i / in.dim) * kv.head_dim + i % in.dim, x);
+    } else {
+      const uint32_t is_v = i >= nq + nk, c = is_v ? i - nq - nk : i - nq, n = is_v ? in.value_dim : in.dim;
+      store4<T>(arena + kv.row(layer, block, c / n, is_v, slot) + kv.col(slot, c % n), x);
+    }
+  }
+}
+
+template <typename T>
+__global__ void arena_rows_kernel(const T *__restrict__ arena, KvLayout kv, uint32_t dim, uint32_t value_dim, float *__restrict__ out) {
+  const size_t tokens = (size_t)kv.num_blocks * kv.num_kv_heads * kv.block_size, keys = tokens * dim, all = keys + tokens * value_dim;
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < all; i += (size_t)gridDim.x * blockDim.x) {
+    const uint32_t is_v = i >= keys, n = is_v ? value_dim : dim;
+    const size_t j = is_v ? i - keys : i, t = j / n;
+    const uint32_t slot = t % kv.block_size, head = t / kv.block_size % kv.num_kv_heads;
+    const uint32_t block = (uint32_t)(t / kv.block_size / kv.num_kv_heads);
+    out[i] = to_f32<T>(arena[kv.row(0, block, head, is_v, slot) + kv.col(slot, j % n)]);
+  }
+}
+
+inline int after_launch(const char *stage) {
+  count_launch();
+  ORION_CUDA_CHECK(stage, cudaGetLastError());
+  return ORION_OK;
+}
+
+template <typename T, int GROUPS>
+int launch_vec(const float *partial, uint32_t splits, size_t split_stride, AttnInputs in, const uint32_t *positions, const uint32_t *slot_block,
+               const uint32_t *slot_slot, T *q_out, T *arena, KvLayout kv, uint32_t layer, float *gate, uint32_t rows, uint32_t threads,
+               cudaStream_t stream) {
+  ORION_CUDA_CHECK("attention_prepare", launch_pdl(attention_prepare_vec_kernel<T, GROUPS>, dim3(rows), dim3(threads), 0, stream, partial, splits,
+                                                   split_stride, in, positions, slot_block, slot_slot, q_out, arena, kv, layer, gate));
+  return after_launch("attention_prepare");
+}
+
+}  // namespace
+
+template <typename T>
+int launch_attention_prepare(const float *partial, uint32_t splits, size_t split_stride, AttnInputs in, const uint32_t *positions,
+                             const uint32_t *slot_block, const uint32_t *slot_slot, T *q_out, T *arena, KvLayout kv, uint32_t layer,
+                             float *gate, uint32_t rows, cudaStream_t stream) {
+  if (rows == 0) return ORION_OK;
+  if ((in.q_norm == nullptr) != (in.k_norm == nullptr)) return set_error(ORION_ERR_INTERNAL, "query and key norms come together");
+  const uint32_t groups = (in.q_heads * in.dim + in.kv_heads * (in.dim + in.value_dim)) / 4;
+  const uint32_t rounds = groups <= 256 ? 1 : (groups <= 1024 ? 2 : (groups <= 2048 ? 4 : 8));
+  const uint32_t threads = ((groups + rounds - 1) / rounds + 31) / 32 * 32;
+  if (in.dim % 4 == 0 && in.value_dim % 4 == 0 && in.rope_dims % 4 == 0 && in.ld % 4 == 0 && split_stride % 4 == 0 && kv.head_dim % 4 == 0 &&
+      kv.v_dim() % 4 == 0 && threads <= 512 && in.q_heads <= threads) {
+    auto run = rounds == 1 ? launch_vec<T, 1> : (rounds == 2 ? launch_vec<T, 2> : (rounds == 4 ? launch_vec<T, 4> : launch_vec<T, 8>));
+    return run(partial, splits, split_stride, in, positions, slot_block, slot_slot, q_out, arena, kv, layer, gate, rows, threads, stream);
+  }
+  ORION_CUDA_CHECK("attention_prepare", launch_pdl(attention_prepare_kernel<T>, dim3(rows), dim3(256), 0, stream, partial, splits, split_stride, in,
+                                                   positions, slot_block, slot_slot, q_out, arena, kv, layer, gate));
+  return after_launch("attention_prepare");
+}
+
+template <typename T>
+int launch_arena_rows(const T *arena, KvLayout kv, uint32_t dim, uint32_t value_dim, float *out, cudaStream_t stream) {
+  arena_rows_kernel<T><<<148 * 8, 256, 0, stream>>>(arena, kv, dim, value_dim, out);
+  return after_launch("arena_rows");
+}
+
+#define ORION_INSTANTIATE(T)                                                                                                            \
+  template int launch_attention_prepare<T>(const float *, uint32_t, size_t, AttnInputs, const uint32_t *, const uint32_t *, const uint32_t *, \
+                                           T *, T *, KvLayout, uint32_t, float *, uint32_t, cudaStream_t);                              \
+  template int launch_arena_rows<T>(const T *, KvLayout, uint32_t, uint32_t, float *, cudaStream_t);
+ORION_INSTANTIATE(float)
+ORION_INSTANTIATE(bf16)
+
+}  // namespace orion

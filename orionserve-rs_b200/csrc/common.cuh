@@ -134,6 +134,13 @@ __device__ __forceinline__ float gelu_tanh(float x) {
   return x * sigmoid_for<T>(1.5957691216057308f * (x + 0.044715f * x * x * x));
 }
 
+__device__ __forceinline__ float relu2(float x) {
+  const float r = fmaxf(x, 0.f);
+  return r * r;
+}
+template <typename T>
+__device__ __forceinline__ float silu_for(float x) { return x * sigmoid_for<T>(x); }
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

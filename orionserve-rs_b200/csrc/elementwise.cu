@@ -635,46 +635,184 @@ int launch_swiglu(const float *partial, uint32_t splits, size_t split_stride, T 
   return after_launch("swiglu");
 }
 
+// Activation of a dense feed-forward.
+template <typename T>
+__device__ __forceinline__ float ffn_activation(FfnAct f, float v) {
+  return f == kActRelu2 ? relu2(v) : gelu_tanh<T>(v);
+}
 template <typename T>
 __global__ void __launch_bounds__(256)
-gelu_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, T *__restrict__ out, uint32_t ldo, uint32_t rows,
-            uint32_t cols) {
+ffn_act_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, const float *__restrict__ bias, FfnAct f,
+               T *__restrict__ out, uint32_t ldo, uint32_t rows, uint32_t cols) {
   pdl_trigger();
   pdl_wait();
   const size_t total = (size_t)rows * cols;
   for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
     float v = partial[idx];
     for (uint32_t s = 1; s < splits; ++s) v += partial[s * split_stride + idx];
-    out[(idx / cols) * ldo + idx % cols] = from_f32<T>(gelu_tanh<T>(v));
+    if (bias) v += bias[idx % cols];
+    out[(idx / cols) * ldo + idx % cols] = from_f32<T>(ffn_activation<T>(f, v));
   }
 }
 // Four columns per thread: cols, ldo and split_stride multiples of 4.
 template <typename T>
 __global__ void __launch_bounds__(256)
-gelu_vec_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, T *__restrict__ out, uint32_t ldo, uint32_t rows,
-                uint32_t cols) {
+ffn_act_vec_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, const float *__restrict__ bias, FfnAct f,
+                   T *__restrict__ out, uint32_t ldo, uint32_t rows, uint32_t cols) {
   pdl_trigger();
   pdl_wait();
   const uint32_t cv = cols / 4;
   const size_t total = (size_t)rows * cv;
   for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
-    const float4 v = sum_slabs4(partial + 4 * idx, splits, split_stride);
-    st4<T>(out + (idx / cv) * ldo + idx % cv * 4, make_float4(gelu_tanh<T>(v.x), gelu_tanh<T>(v.y), gelu_tanh<T>(v.z), gelu_tanh<T>(v.w)));
+    float4 v = sum_slabs4(partial + 4 * idx, splits, split_stride);
+    const uint32_t c = idx % cv * 4;
+    if (bias) v = add4(v, ld4(bias + c));
+    st4<T>(out + (idx / cv) * ldo + c, make_float4(ffn_activation<T>(f, v.x), ffn_activation<T>(f, v.y), ffn_activation<T>(f, v.z), ffn_activation<T>(f, v.w)));
   }
 }
 
 template <typename T>
-int launch_gelu(const float *partial, uint32_t splits, size_t split_stride, T *out, uint32_t ldo, uint32_t rows, uint32_t cols,
-                cudaStream_t stream) {
+int launch_ffn_act(const float *partial, uint32_t splits, size_t split_stride, const float *bias, FfnAct f, T *out, uint32_t ldo, uint32_t rows,
+                   uint32_t cols, cudaStream_t stream) {
   if (rows == 0 || cols == 0) return ORION_OK;
   if (cols % 4 == 0 && ldo % 4 == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0) {
-    ORION_CUDA_CHECK("gelu", launch_pdl(gelu_vec_kernel<T>, dim3(grid_for((size_t)rows * cols / 4, 256)), dim3(256), 0, stream, partial, splits,
-                                        split_stride, out, ldo, rows, cols));
-    return after_launch("gelu");
+    ORION_CUDA_CHECK("ffn_act", launch_pdl(ffn_act_vec_kernel<T>, dim3(grid_for((size_t)rows * cols / 4, 256)), dim3(256), 0, stream, partial, splits,
+                                           split_stride, bias, f, out, ldo, rows, cols));
+    return after_launch("ffn_act");
   }
-  ORION_CUDA_CHECK("gelu", launch_pdl(gelu_kernel<T>, dim3(grid_for((size_t)rows * cols, 256)), dim3(256), 0, stream, partial, splits,
-                                      split_stride, out, ldo, rows, cols));
-  return after_launch("gelu");
+  ORION_CUDA_CHECK("ffn_act", launch_pdl(ffn_act_kernel<T>, dim3(grid_for((size_t)rows * cols, 256)), dim3(256), 0, stream, partial, splits,
+                                         split_stride, bias, f, out, ldo, rows, cols));
+  return after_launch("ffn_act");
+}
+
+// ---- a sublayer whose output is normalised before it joins the residual stream -----------------------------
+
+// Value c of a sublayer's output for one row.
+__device__ __forceinline__ float sublayer_value(const SublayerOutput &y, uint32_t row, uint32_t H, uint32_t c) {
+  float v = 0.f;
+  if (y.partial)
+    for (uint32_t s = 0; s < y.splits; ++s) v += y.partial[s * y.split_stride + (size_t)row * H + c];
+  if (y.bias) v += y.bias[c];
+  for (uint32_t k = 0; k < y.top; ++k) {
+    const float *p = y.rows + (size_t)y.place[(size_t)row * y.top + k] * H + c;
+    for (uint32_t s = 0; s < y.rows_splits; ++s) v += p[s * y.rows_stride];
+  }
+  return v;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kNormThreads)
+post_norm_residual_kernel(SublayerOutput y, float *__restrict__ hidden, const float *__restrict__ post_w, float mult,
+                          const float *__restrict__ pre_w, float eps, T *__restrict__ out, const uint32_t *__restrict__ row_map, uint32_t H) {
+  using Acc = typename NormAcc<T>::type;
+  __shared__ Acc red[32];
+  extern __shared__ float row_cache[];  // H floats
+  pdl_trigger();
+  pdl_wait();
+  const uint32_t row = row_map ? row_map[blockIdx.x] : blockIdx.x;
+  float *h = hidden + (size_t)row * H;
+  Acc ss = Acc(0);
+  for (uint32_t c = threadIdx.x; c < H; c += blockDim.x) {
+    const float v = sublayer_value(y, row, H, c);
+    row_cache[c] = v;
+    ss += (Acc)v * (Acc)v;
+  }
+  const float s1 = norm_scale<Acc>(block_sum<Acc>(ss, red), H, eps);
+  ss = Acc(0);
+  for (uint32_t c = threadIdx.x; c < H; c += blockDim.x) {
+    const float v = h[c] + mult * (row_cache[c] * s1 * post_w[c]);
+    if (!row_map) h[c] = v;
+    row_cache[c] = v;
+    ss += (Acc)v * (Acc)v;
+  }
+  const float s2 = norm_scale<Acc>(block_sum<Acc>(ss, red), H, eps);
+  T *o = out + (size_t)blockIdx.x * H;
+  for (uint32_t c = threadIdx.x; c < H; c += blockDim.x) o[c] = from_f32<T>(row_cache[c] * s2 * pre_w[c]);
+}
+
+// Row widths that are multiples of 4: a row's values stay in registers between the two norms.
+template <typename T, int CHUNKS>
+__global__ void __launch_bounds__(512)
+post_norm_residual_vec_kernel(SublayerOutput y, float *__restrict__ hidden, const float *__restrict__ post_w, float mult,
+                              const float *__restrict__ pre_w, float eps, T *__restrict__ out, const uint32_t *__restrict__ row_map, uint32_t H) {
+  using Acc = typename NormAcc<T>::type;
+  __shared__ Acc red[32];
+  pdl_trigger();
+  const uint32_t nvec = H / 4;
+  float4 pw[CHUNKS], nw[CHUNKS], bv[CHUNKS];
+#pragma unroll
+  for (int c = 0; c < CHUNKS; ++c) {  // immutable: fetched before the dependency wait
+    const uint32_t idx = threadIdx.x + c * blockDim.x;
+    pw[c] = nw[c] = bv[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (idx < nvec) {
+      pw[c] = ld4(post_w + 4 * (size_t)idx), nw[c] = ld4(pre_w + 4 * (size_t)idx);
+      if (y.bias) bv[c] = ld4(y.bias + 4 * (size_t)idx);
+    }
+  }
+  pdl_wait();
+  const uint32_t row = row_map ? row_map[blockIdx.x] : blockIdx.x;
+  float *h = hidden + (size_t)row * H;
+  float4 v[CHUNKS], x[CHUNKS];
+  Acc ss = Acc(0);
+#pragma unroll
+  for (int c = 0; c < CHUNKS; ++c) {
+    const uint32_t idx = threadIdx.x + c * blockDim.x;
+    v[c] = x[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (idx >= nvec) continue;
+    x[c] = ld4(h + 4 * (size_t)idx);
+    if (y.partial) v[c] = sum_slabs4(y.partial + (size_t)row * H + 4 * (size_t)idx, y.splits, y.split_stride);
+    v[c] = add4(v[c], bv[c]);
+    for (uint32_t k = 0; k < y.top; ++k)
+      v[c] = add4(v[c], sum_slabs4(y.rows + (size_t)y.place[(size_t)row * y.top + k] * H + 4 * (size_t)idx, y.rows_splits, y.rows_stride));
+    ss += (Acc)v[c].x * (Acc)v[c].x + (Acc)v[c].y * (Acc)v[c].y + (Acc)v[c].z * (Acc)v[c].z + (Acc)v[c].w * (Acc)v[c].w;
+  }
+  const float s1 = norm_scale<Acc>(block_sum<Acc>(ss, red), H, eps);
+  ss = Acc(0);
+#pragma unroll
+  for (int c = 0; c < CHUNKS; ++c) {
+    const uint32_t idx = threadIdx.x + c * blockDim.x;
+    if (idx >= nvec) continue;
+    x[c] = make_float4(x[c].x + mult * (v[c].x * s1 * pw[c].x), x[c].y + mult * (v[c].y * s1 * pw[c].y), x[c].z + mult * (v[c].z * s1 * pw[c].z),
+                       x[c].w + mult * (v[c].w * s1 * pw[c].w));
+    if (!row_map) *reinterpret_cast<float4 *>(h + 4 * (size_t)idx) = x[c];
+    ss += (Acc)x[c].x * (Acc)x[c].x + (Acc)x[c].y * (Acc)x[c].y + (Acc)x[c].z * (Acc)x[c].z + (Acc)x[c].w * (Acc)x[c].w;
+  }
+  const float s2 = norm_scale<Acc>(block_sum<Acc>(ss, red), H, eps);
+  T *o = out + (size_t)blockIdx.x * H;
+#pragma unroll
+  for (int c = 0; c < CHUNKS; ++c) {
+    const uint32_t idx = threadIdx.x + c * blockDim.x;
+    if (idx < nvec)
+      st4<T>(o + 4 * (size_t)idx, make_float4(x[c].x * s2 * nw[c].x, x[c].y * s2 * nw[c].y, x[c].z * s2 * nw[c].z, x[c].w * s2 * nw[c].w));
+  }
+}
+
+namespace {
+template <typename T, int CHUNKS>
+int launch_post_norm_vec(SublayerOutput y, float *hidden, const float *post_w, float mult, const float *pre_w, float eps, T *out,
+                         const uint32_t *row_map, uint32_t out_rows, uint32_t H, uint32_t threads, cudaStream_t stream) {
+  ORION_CUDA_CHECK("post_norm_residual", launch_pdl(post_norm_residual_vec_kernel<T, CHUNKS>, dim3(out_rows), dim3(threads), 0, stream, y, hidden,
+                                                    post_w, mult, pre_w, eps, out, row_map, H));
+  return after_launch("post_norm_residual");
+}
+}  // namespace
+
+template <typename T>
+int launch_post_norm_residual(SublayerOutput y, float *hidden, const float *post_w, float mult, const float *pre_w, float eps, T *out,
+                              const uint32_t *row_map, uint32_t out_rows, uint32_t H, cudaStream_t stream) {
+  if (out_rows == 0) return ORION_OK;
+  if (H % 4 == 0 && H / 4 <= 2048 && y.split_stride % 4 == 0 && y.rows_stride % 4 == 0) {
+    const uint32_t nvec = H / 4, threads = nvec >= 512 ? 512 : (nvec + 31) / 32 * 32, chunks = (nvec + threads - 1) / threads;
+    auto run = chunks == 1 ? launch_post_norm_vec<T, 1> : (chunks == 2 ? launch_post_norm_vec<T, 2> : launch_post_norm_vec<T, 4>);
+    return run(y, hidden, post_w, mult, pre_w, eps, out, row_map, out_rows, H, threads, stream);
+  }
+  const size_t smem = (size_t)H * sizeof(float);
+  if (smem > 200 * 1024) return set_error(ORION_ERR_INTERNAL, "hidden size %u too large for the fused norm kernel", H);
+  static bool attr_set[kMaxDeviceOrdinals] = {};
+  ORION_CUDA_CHECK("post_norm_residual attr", ensure_dynamic_smem(post_norm_residual_kernel<T>, 200 * 1024, attr_set));
+  ORION_CUDA_CHECK("post_norm_residual", launch_pdl(post_norm_residual_kernel<T>, dim3(out_rows), dim3(kNormThreads), smem, stream, y, hidden, post_w,
+                                                    mult, pre_w, eps, out, row_map, H));
+  return after_launch("post_norm_residual");
 }
 
 // dst[r * dst_stride + c] = src[r * cols + c]: spreads the rows of a contiguous matrix over a
@@ -800,7 +938,9 @@ int launch_fill_normal(T *dst, size_t n, uint64_t seed, cudaStream_t stream) {
   template int launch_copy_rows_strided<T>(const T *, T *, size_t, size_t, size_t, cudaStream_t);   \
   template int launch_swiglu<T>(const float *, uint32_t, size_t, T *, uint32_t, uint32_t,         \
                                 cudaStream_t, bool);                                              \
-  template int launch_gelu<T>(const float *, uint32_t, size_t, T *, uint32_t, uint32_t, uint32_t, cudaStream_t); \
+  template int launch_ffn_act<T>(const float *, uint32_t, size_t, const float *, FfnAct, T *, uint32_t, uint32_t, uint32_t, cudaStream_t); \
+  template int launch_post_norm_residual<T>(SublayerOutput, float *, const float *, float, const float *, float, T *, const uint32_t *, \
+                                            uint32_t, uint32_t, cudaStream_t);                    \
   template int launch_convert_from_f32<T>(const float *, T *, size_t, cudaStream_t);              \
   template int launch_convert_to_f32<T>(const T *, float *, size_t, cudaStream_t);                \
   template int launch_arena_to_reference_order<T>(const T *, KvLayout, float *, cudaStream_t);    \

@@ -204,13 +204,13 @@ __device__ __forceinline__ constexpr uint32_t instr_desc() {
          ((uint32_t)(M >> 4) << 24);
 }
 
-// ACT: the epilogue stores activations (kGemmGelu, kGemmStore); else f32 partials, or SwiGLU where `act` is given. A
+// ACT: the epilogue stores activations (kGemmGelu, kGemmRelu2, kGemmStore); else f32 partials, or SwiGLU where `act` is given. A
 // template parameter, since the larger epilogue costs the weight-streaming shapes 0.8 us per launch.
 template <int TOKN, int WST, int XST, int MT, bool PAIR, bool ACT>
 __global__ void __launch_bounds__(kThreads)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                float *__restrict__ partial, bf16 *__restrict__ act, uint32_t M, uint32_t N, uint32_t K,
-               uint32_t splits, uint32_t cluster_reduce, uint32_t ldc, uint32_t epilogue, ReadyWait ready) {
+               uint32_t splits, uint32_t cluster_reduce, uint32_t ldc, uint32_t epilogue, ReadyWait ready, const float *__restrict__ bias) {
   using Cfg = TcConfig<TOKN, WST, XST, MT, PAIR>;
   extern __shared__ uint8_t raw_smem[];
   uint8_t *smem = reinterpret_cast<uint8_t *>((reinterpret_cast<uintptr_t>(raw_smem) + 1023) &
@@ -455,10 +455,11 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
       if (t0 + c >= M || n >= N) continue;
       bf16 *dst = act + (size_t)(t0 + c) * ldc + n;
       const uint32_t valid = M - (t0 + c);
+      const float b = bias ? bias[n] : 0.f;
 #pragma unroll
       for (int j = 0; j < 16; ++j) {
-        const float v = __uint_as_float(r[j]);
-        if ((uint32_t)j < valid) dst[(size_t)j * ldc] = __float2bfloat16_rn(epilogue == kGemmGelu ? gelu_tanh<bf16>(v) : v);
+        const float v = __uint_as_float(r[j]) + b;
+        if ((uint32_t)j < valid) dst[(size_t)j * ldc] = __float2bfloat16_rn(epilogue == kGemmGelu ? gelu_tanh<bf16>(v) : (epilogue == kGemmRelu2 ? relu2(v) : v));
       }
     }
     __syncwarp();
@@ -572,7 +573,7 @@ int cached_map(const void *base, uint64_t rows, uint64_t k, uint64_t ld, uint32_
 template <bool ACT, int TOKN, int WST, int XST, int MT, bool PAIR>
 int launch_tc_form(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, float *partial, bf16 *act,
               uint32_t rows, uint32_t n, uint32_t k, uint32_t splits, bool cluster_reduce, uint32_t ldc, GemmEpilogue epi,
-              cudaStream_t stream, ReadyWait ready) {
+              cudaStream_t stream, ReadyWait ready, const float *bias) {
   if (ldc == 0) ldc = n;
   if (ldc != n && (splits != 1 || epi == kGemmSwiglu))
     return set_error(ORION_ERR_INTERNAL, "a strided GEMM output needs one k split and no SwiGLU");
@@ -590,14 +591,14 @@ int launch_tc_form(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, flo
       return set_error(ORION_ERR_INTERNAL, "the paired GEMM needs an even number of weight tile groups and no cluster split-K");
     ORION_CUDA_CHECK("gemm_tc", launch_pdl_cluster(gemm_tc_kernel<TOKN, WST, XST, MT, PAIR, ACT>, grid, dim3(kThreads), dim3(2, 1, 1),
                                                    Cfg::kSmemBytes, stream, *mw, *mx, partial, act, rows, n, k, splits,
-                                                   0u, ldc, (uint32_t)epi, ready));
+                                                   0u, ldc, (uint32_t)epi, ready, bias));
   } else if (cluster_reduce)
     ORION_CUDA_CHECK("gemm_tc", launch_pdl_cluster(gemm_tc_kernel<TOKN, WST, XST, MT, PAIR, ACT>, grid, dim3(kThreads), dim3(1, 1, splits),
                                                    Cfg::kSmemBytes, stream, *mw, *mx, partial, act, rows, n, k, splits,
-                                                   1u, ldc, (uint32_t)epi, ready));
+                                                   1u, ldc, (uint32_t)epi, ready, bias));
   else
     ORION_CUDA_CHECK("gemm_tc", launch_pdl(gemm_tc_kernel<TOKN, WST, XST, MT, PAIR, ACT>, grid, dim3(kThreads), Cfg::kSmemBytes, stream,
-                                           *mw, *mx, partial, act, rows, n, k, splits, 0u, ldc, (uint32_t)epi, ready));
+                                           *mw, *mx, partial, act, rows, n, k, splits, 0u, ldc, (uint32_t)epi, ready, bias));
   count_launch();
   ORION_CUDA_CHECK("gemm_tc", cudaGetLastError());
   return ORION_OK;
@@ -605,10 +606,11 @@ int launch_tc_form(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, flo
 
 template <int TOKN, int WST, int XST, int MT = 1, bool PAIR = false>
 int launch_tc(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, float *partial, bf16 *act, uint32_t rows, uint32_t n,
-              uint32_t k, uint32_t splits, bool cluster_reduce, uint32_t ldc, GemmEpilogue epi, cudaStream_t stream, ReadyWait ready = {}) {
-  auto form = epi == kGemmGelu || epi == kGemmStore ? launch_tc_form<true, TOKN, WST, XST, MT, PAIR>
+              uint32_t k, uint32_t splits, bool cluster_reduce, uint32_t ldc, GemmEpilogue epi, cudaStream_t stream, ReadyWait ready,
+              const float *bias) {
+  auto form = epi == kGemmGelu || epi == kGemmStore || epi == kGemmRelu2 ? launch_tc_form<true, TOKN, WST, XST, MT, PAIR>
                                                     : launch_tc_form<false, TOKN, WST, XST, MT, PAIR>;
-  return form(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready);
+  return form(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready, bias);
 }
 
 // 256-token tiles as CTA pairs (tcgen05 cta_group::2). Measured on the Llama-3-8B shape, projections of
@@ -664,7 +666,7 @@ bool gemm_tc_supported(uint32_t rows, uint32_t n, uint32_t k, uint32_t ldx, uint
 
 int launch_gemm_tc(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, float *partial,
                    uint32_t rows, uint32_t n, uint32_t k, uint32_t splits, cudaStream_t stream,
-                   bf16 *act, bool cluster_reduce, uint32_t ldc, ReadyWait ready, GemmEpilogue epi) {
+                   bf16 *act, bool cluster_reduce, uint32_t ldc, ReadyWait ready, GemmEpilogue epi, const float *bias) {
   const uint32_t nkb = (k + kSlabK - 1) / kSlabK;
   if (cluster_reduce && (splits < 2 || splits > 8 || act != nullptr))
     return set_error(ORION_ERR_INTERNAL, "cluster split-K needs 2..8 splits and f32 output");
@@ -680,28 +682,28 @@ int launch_gemm_tc(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, flo
   if (rows > 256 && g_prefill_fill == 1 && ((n + kTileN - 1) / kTileN) * ((rows + 255) / 256) < 148) tt = 128;
   switch (tt) {
     case 16:
-      return deep ? launch_tc<16, 6, 3>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready)
-                  : launch_tc<16, 5, 3>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready);
+      return deep ? launch_tc<16, 6, 3>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready, bias)
+                  : launch_tc<16, 5, 3>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready, bias);
     case 32:
-      return deep ? launch_tc<32, 6, 3>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready)
-                  : launch_tc<32, 5, 3>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready);
+      return deep ? launch_tc<32, 6, 3>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready, bias)
+                  : launch_tc<32, 5, 3>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready, bias);
     case 64:
-      return deep ? launch_tc<64, 5, 3>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready)
-                  : launch_tc<64, 4, 4>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready);
+      return deep ? launch_tc<64, 5, 3>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready, bias)
+                  : launch_tc<64, 4, 4>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready, bias);
     case 128:
       return g_mid_tile == 0
-                 ? launch_tc<128, 4, 2>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready)
-                 : launch_tc<128, 6, 6>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready);
+                 ? launch_tc<128, 4, 2>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready, bias)
+                 : launch_tc<128, 6, 6>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready, bias);
     default: {
       const uint32_t mt = (!cluster_reduce && prefill_weight_tiles(rows, n) == 2) ? 2 : 1;
       // CTA pairs: each CTA loads half of the activation tile, so the rings go a stage deeper
       const bool pair = (g_gemm_pair >= 2 || (g_gemm_pair == 1 && rows >= kPairMinRows)) && !cluster_reduce &&
                         (((n + mt * kTileN - 1) / (mt * kTileN)) & 1u) == 0;
       if (mt == 2)
-        return pair ? launch_tc<256, 4, 4, 2, true>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready)
-                    : launch_tc<256, 3, 3, 2>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready);
-      return pair ? launch_tc<256, 6, 6, 1, true>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready)
-                  : launch_tc<256, 4, 4>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready);
+        return pair ? launch_tc<256, 4, 4, 2, true>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready, bias)
+                    : launch_tc<256, 3, 3, 2>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready, bias);
+      return pair ? launch_tc<256, 6, 6, 1, true>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready, bias)
+                  : launch_tc<256, 4, 4>(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready, bias);
     }
   }
 }
@@ -815,11 +817,11 @@ int launch_gemm_swiglu(const bf16 *x, uint32_t ldx, const bf16 *w_interleaved, u
 }
 
 int launch_gemm_act(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, bf16 *act, uint32_t ld_act, uint32_t rows, uint32_t n,
-                    uint32_t k, GemmEpilogue epi, cudaStream_t stream) {
-  if (epi != kGemmGelu && epi != kGemmStore) return set_error(ORION_ERR_INTERNAL, "not an epilogue of this entry point");
+                    uint32_t k, GemmEpilogue epi, cudaStream_t stream, const float *bias) {
+  if (epi != kGemmGelu && epi != kGemmStore && epi != kGemmRelu2) return set_error(ORION_ERR_INTERNAL, "not an epilogue of this entry point");
   if (!gemm_tc_supported(rows, n, k, ldx, ldw, x, w))
     return set_error(ORION_ERR_INTERNAL, "tensor-core GEMM planned for an unaligned operand");
-  return launch_gemm_tc(x, ldx, w, ldw, nullptr, rows, n, k, 1, stream, act, false, ld_act, ReadyWait{}, epi);
+  return launch_gemm_tc(x, ldx, w, ldw, nullptr, rows, n, k, 1, stream, act, false, ld_act, ReadyWait{}, epi, bias);
 }
 
 template <>

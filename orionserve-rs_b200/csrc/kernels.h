@@ -11,7 +11,7 @@
 namespace orion {
 
 // Shape of the paged KV arena of one rank:
-// [layer][block][local kv head][k|v][slot][dim]. Each (block, head) owns one
+// [layer][block][local kv head][k|v][slot][dim] (K and V rows may differ in size). Each (block, head) owns one
 // contiguous chunk holding its K rows followed by its V rows, so a decode CTA
 // fetches a 16-token block of one head with a single bulk copy.
 // With `swizzle` set (16-bit storage, head_dim a multiple of 64) the 16-byte
@@ -19,7 +19,9 @@ namespace orion {
 // lands in shared memory in a layout ldmatrix reads without bank conflicts.
 struct KvLayout {
   uint32_t num_layers, num_blocks, num_kv_heads, block_size, head_dim, swizzle;
-  __host__ __device__ size_t chunk_elems() const { return size_t(2) * block_size * head_dim; }
+  uint32_t value_dim = 0;  // size of a V row; 0 = head_dim
+  __host__ __device__ uint32_t v_dim() const { return value_dim ? value_dim : head_dim; }
+  __host__ __device__ size_t chunk_elems() const { return size_t(block_size) * (head_dim + v_dim()); }
   __host__ __device__ size_t layer_elems() const {
     return size_t(num_blocks) * num_kv_heads * chunk_elems();
   }
@@ -27,7 +29,7 @@ struct KvLayout {
   __host__ __device__ size_t row(uint32_t layer, uint32_t block, uint32_t head, uint32_t is_v,
                                  uint32_t slot) const {
     return layer * layer_elems() + (size_t(block) * num_kv_heads + head) * chunk_elems() +
-           (size_t(is_v) * block_size + slot) * head_dim;
+           (is_v ? size_t(block_size) * head_dim + size_t(slot) * v_dim() : size_t(slot) * head_dim);
   }
   // Position of logical dim `d` inside the row of `slot`.
   __host__ __device__ uint32_t col(uint32_t slot, uint32_t d) const {
@@ -81,10 +83,29 @@ int launch_swiglu(const float *partial, uint32_t splits, size_t split_stride, T 
 template <typename T>
 int launch_copy_rows_strided(const T *src, T *dst, size_t rows, size_t cols, size_t dst_stride, cudaStream_t stream);
 
-// out[r * ldo + c] = gelu(sum_s partial[s][r][c]), the tanh form.
+// out[r * ldo + c] = f(sum_s partial[s][r][c] + bias[c]), f = GELU (tanh form) or the square of relu; bias may be null.
+enum FfnAct : uint32_t { kActGelu = 0, kActRelu2 = 1 };
 template <typename T>
-int launch_gelu(const float *partial, uint32_t splits, size_t split_stride, T *out, uint32_t ldo, uint32_t rows, uint32_t cols,
-                cudaStream_t stream);
+int launch_ffn_act(const float *partial, uint32_t splits, size_t split_stride, const float *bias, FfnAct f, T *out, uint32_t ldo, uint32_t rows,
+                   uint32_t cols, cudaStream_t stream);
+
+// A sublayer's output y that is normalised before it is added: hidden += mult * rms_norm(y) * post_w, then
+// out[i] = rms_norm(hidden[src(i)]) * pre_w with src and row_map as in launch_residual_rmsnorm. y is the sum of a projection's
+// slabs (partial may be null), a bias (may be null) and, where a row went through `top` experts, the rows place[r * top + k]
+// of the experts' output (each the sum of rows_splits slabs).
+struct SublayerOutput {
+  const float *partial = nullptr;
+  uint32_t splits = 0;
+  size_t split_stride = 0;
+  const float *bias = nullptr;
+  const float *rows = nullptr;
+  const uint32_t *place = nullptr;
+  uint32_t top = 0, rows_splits = 0;
+  size_t rows_stride = 0;
+};
+template <typename T>
+int launch_post_norm_residual(SublayerOutput y, float *hidden, const float *post_w, float mult, const float *pre_w, float eps, T *out,
+                              const uint32_t *row_map, uint32_t out_rows, uint32_t hidden_size, cudaStream_t stream);
 
 // out[r][n] = sum_s partial[s][r][n] + bias[n]  (finishes tensor::linear, tensor.rs:126).
 int launch_finish_linear(const float *partial, uint32_t splits, size_t split_stride,
@@ -132,11 +153,56 @@ struct AttnBatch {
   uint32_t max_position;            // largest query position in the batch
 };
 
+// Which of the positions up to its own a query sees: the last `window` of them (0 = no window), of those the ones in
+// its own chunk of `chunk` positions, counted from the sequence's start (0 = no chunks).
+struct KeyRange {
+  uint32_t window = 0, chunk = 0;
+  __host__ __device__ uint32_t first(uint32_t pos) const {
+    const uint32_t w = window && pos + 1 > window ? pos + 1 - window : 0, c = chunk ? pos / chunk * chunk : 0;
+    return w > c ? w : c;
+  }
+  // The most positions a query up to `max_position` sees.
+  __host__ __device__ uint32_t most(uint32_t max_position) const {
+    uint32_t n = max_position + 1;
+    if (window && window < n) n = window;
+    return chunk && chunk < n ? chunk : n;
+  }
+};
+// What a design adds to causal attention over everything before; the defaults add nothing.
+struct AttnForm {
+  float scale = 0.f;              // of the scores; 0 = 1 / sqrt(head_dim)
+  KeyRange range;
+  const float *sinks = nullptr;   // [q_heads] logits that enter the denominator once and carry no value
+  const float *gate = nullptr;    // [rows][q_heads] factors of the heads' outputs
+  uint32_t out_dim = 0, ldo = 0;  // values stored per head and row stride of the output; 0 = v_dim() and q_heads * out_dim
+  // Decode only: the batch rows that decode (item i of the scratch belongs to row_list[i]), and the first row of every
+  // sequence, since several rows of one sequence may decode together. Null: every row, one per sequence.
+  const uint32_t *row_list = nullptr, *first_row = nullptr;
+};
+
 // Any shape, any mix of prefill and decode rows: one CTA per (row, query head),
 // causal by absolute position (attention.rs:219-295).
 template <typename T>
 int launch_paged_attention_generic(const T *q, const T *arena, KvLayout kv, uint32_t layer,
-                                   AttnBatch batch, uint32_t q_heads, T *out, cudaStream_t stream);
+                                   AttnBatch batch, uint32_t q_heads, T *out, cudaStream_t stream, AttnForm form = {});
+
+// Folds the partial sums of a joint projection [q | k | v | g] (row stride `ld`): RMS norms over all heads of q and of k
+// together (gains may be null: no norm), rotation of the first rope_dims dimensions of every head in neighbouring pairs
+// (2i, 2i + 1) by the table's angles, q to `q_out` [rows][q_heads][kv.head_dim], k and v to the arena, and sigmoid(g), one
+// value per query head, to `gate` [rows][q_heads] (may be null: no such columns). dim and value_dim are what the projection
+// holds per head; the arena's rows may be longer, and what is beyond stays as it is.
+struct AttnInputs {
+  uint32_t q_heads, kv_heads, dim, value_dim, rope_dims, ld;
+  float eps;
+  const float *q_norm, *k_norm, *rope_cos, *rope_sin;
+};
+template <typename T>
+int launch_attention_prepare(const float *partial, uint32_t splits, size_t split_stride, AttnInputs in, const uint32_t *positions,
+                             const uint32_t *slot_block, const uint32_t *slot_slot, T *q_out, T *arena, KvLayout kv, uint32_t layer,
+                             float *gate, uint32_t rows, cudaStream_t stream);
+// K and V rows of one layer's arena as f32, [k|v][block][kv head][slot][dim] with dim values of a K row, value_dim of a V row.
+template <typename T>
+int launch_arena_rows(const T *arena, KvLayout kv, uint32_t dim, uint32_t value_dim, float *out, cudaStream_t stream);
 
 // Tuned prefill / mixed-batch path (bf16, head_dim 128, block 16): the batch is cut into
 // tiles of consecutive rows of one sequence (prefill_tile_positions rows at most); one CTA per
@@ -160,6 +226,17 @@ int launch_paged_attention_prefill_tc(const bf16 *q, const bf16 *arena, KvLayout
                                       AttnBatch batch, const PrefillTile *tiles, uint32_t num_tiles,
                                       uint32_t q_heads, bf16 *out, cudaStream_t stream);
 int prefill_tc_poll_error(uint32_t *code);
+// Other forms of attention on the same kernels: head and value sizes of 64, 128 or 256 (an arena pads to them; above 128
+// both 256), 16-token blocks. Their prefill tiles are 128 / (query heads per kv head) positions.
+bool attention_form_supported(KvLayout kv, uint32_t q_heads);
+// The size a head dimension is padded to in such an arena; 0 = no padding makes the kernels cover it.
+inline uint32_t attention_padded_dim(uint32_t dim, uint32_t other) {
+  if (dim == 0 || other == 0 || dim > 256 || other > 256) return 0;
+  return dim > 128 || other > 128 ? 256 : (dim > 64 ? 128 : 64);
+}
+int launch_paged_attention_prefill_form(const bf16 *q, const bf16 *arena, KvLayout kv, uint32_t layer, AttnBatch batch,
+                                        const PrefillTile *tiles, uint32_t num_tiles, uint32_t q_heads, AttnForm form, bf16 *out,
+                                        cudaStream_t stream);
 
 // Tuned decode path (bf16, head_dim 128, block 16, one query row per sequence):
 // one CTA per (sequence, kv head, context split); the query heads of a GQA group
@@ -212,6 +289,12 @@ int launch_paged_attention_decode(const bf16 *q, const bf16 *arena, KvLayout kv,
                                   AttnBatch batch, uint32_t q_heads, uint32_t splits,
                                   DecodeScratch scratch, bf16 *out, cudaStream_t stream,
                                   FusedQkv fused = {});
+// The same for other forms of attention and any number of query heads per kv head (eight share a CTA); `rows` of the
+// batch are those of form.row_list.
+uint32_t decode_form_splits(KvLayout kv, uint32_t q_heads, uint32_t rows, uint32_t most_keys);
+int launch_paged_attention_decode_form(const bf16 *q, const bf16 *arena, KvLayout kv, uint32_t layer, AttnBatch batch, uint32_t rows,
+                                       uint32_t q_heads, uint32_t splits, DecodeScratch scratch, AttnForm form, bf16 *out,
+                                       cudaStream_t stream);
 // Tuning: ring depth per warp (2..4) and the CTA count the context split aims for (0 keeps it).
 void decode_set_tuning(int stages, uint32_t cta_target);
 // Device error word of the decode kernel (0 = none); reading clears it.
@@ -272,7 +355,7 @@ struct LatentShape {
   __host__ __device__ uint32_t out_cols() const { return heads * value_dim; }
   __host__ __device__ uint32_t cols() const { return q_cols() + kv_cols() + out_cols(); }
   // First position that a query at `pos` sees.
-  __host__ __device__ uint32_t first_key(uint32_t pos) const { return window && pos + 1 > window ? pos + 1 - window : 0; }
+  __host__ __device__ uint32_t first_key(uint32_t pos) const { return KeyRange{window, 0}.first(pos); }
 };
 // Folds the joint projection's partial sums: queries (rotated) to q [rows][heads][dim + rot_dim], the normalised
 // latent and the rotated shared key part to the cache row of the token.
@@ -398,17 +481,17 @@ template <typename T>
 int launch_gemm_simt(const T *x, uint32_t ldx, const T *w, uint32_t ldw, float *out, uint32_t rows,
                      uint32_t n, uint32_t k, cudaStream_t stream);
 // tcgen05 / TMEM / TMA GEMM (bf16).
-enum GemmEpilogue : uint32_t { kGemmPartials = 0, kGemmSwiglu = 1, kGemmGelu = 2, kGemmStore = 3 };
+enum GemmEpilogue : uint32_t { kGemmPartials = 0, kGemmSwiglu = 1, kGemmGelu = 2, kGemmStore = 3, kGemmRelu2 = 4 };
 bool gemm_tc_supported(uint32_t rows, uint32_t n, uint32_t k, uint32_t ldx, uint32_t ldw,
                        const void *x, const void *w);
 int launch_gemm_tc(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, float *partial,
                    uint32_t rows, uint32_t n, uint32_t k, uint32_t splits, cudaStream_t stream,
                    bf16 *act = nullptr, bool cluster_reduce = false, uint32_t ldc = 0,
-                   ReadyWait ready = {}, GemmEpilogue epi = kGemmPartials);
-// The same projection with its result stored as bf16 activations, act[r * ld_act + n] = f(x.w_n), f = GELU (tanh form)
-// or the identity. One k split only.
+                   ReadyWait ready = {}, GemmEpilogue epi = kGemmPartials, const float *bias = nullptr);
+// The same projection with its result stored as bf16 activations, act[r * ld_act + n] = f(x.w_n + bias[n]), f = GELU (tanh
+// form), the square of relu or the identity; bias may be null. One k split only.
 int launch_gemm_act(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, bf16 *act, uint32_t ld_act, uint32_t rows, uint32_t n,
-                    uint32_t k, GemmEpilogue epi, cudaStream_t stream);
+                    uint32_t k, GemmEpilogue epi, cudaStream_t stream, const float *bias = nullptr);
 // Gate/up projection with SwiGLU in the epilogue: `w_interleaved` is [2 * ffn][k] with gate row f
 // at 2f and up row f at 2f + 1; writes act[r][f] = silu(x.gate_f) * (x.up_f) and no partials.
 // One k split only (gemm_plan(...).splits == 1 and .tensor_core).

@@ -584,7 +584,7 @@ int LayeredModel<T>::run_step_body(bool want_argmax, int part) {
       if (!in_epilogue) {
         ORION_TRY(timed(kProfGemm, [&] { return launch_gemm<T>(conv_f_, H, L.w_up, H, partial_, Tn, F, H, p, stream_); }));
         ORION_TRY(timed(kProfElementwise, [&] {
-          return launch_gelu<T>(partial_, p.out_slabs, (size_t)Tn * F, cat_ + L.ff_at, L.cat, Tn, F, stream_);
+          return launch_ffn_act<T>(partial_, p.out_slabs, (size_t)Tn * F, nullptr, kActGelu, cat_ + L.ff_at, L.cat, Tn, F, stream_);
         }));
       }
     }
