@@ -408,6 +408,67 @@ int launch_latent_prefill(const bf16 *q, const bf16 *expanded, const bf16 *rotat
                           uint32_t ldo, cudaStream_t stream);
 int latent_prefill_poll_error(uint32_t *code);
 
+// ---- mixture of experts ------------------------------------------------------------------------
+//
+// Every row goes through `top` of the experts, chosen by the largest sigmoid of the router's logits; the score multiplies
+// the expert's input. A shared expert (shared_ffn = 0: none) takes every row as it is. An expert is W_down (silu(W_gate x) *
+// (W_up x)). Rows are copied into the order of their experts, and the two products run over tiles of rows of one expert.
+// Expert weights are stacked: up [experts][2 * ffn][hidden] with gate row f at 2f and up row f at 2f + 1, down
+// [experts][hidden][ffn]; the shared expert's the same with one expert.
+struct MoeShape {
+  uint32_t hidden, experts, top, ffn, shared_ffn;
+};
+struct MoeTile {
+  uint32_t expert, row, count;  // sorted rows [row, row + count) go through `expert`; count 0: nothing to do
+};
+struct MoePlan {
+  uint32_t tile_rows;             // rows per tile
+  uint32_t tiles;                 // entries of the tile list
+  uint32_t up_splits, down_splits;  // k splits of the two products
+  bool tensor_core;
+};
+MoePlan moe_plan(bool is_bf16, MoeShape s, uint32_t rows);
+constexpr uint32_t kMoeMaxExperts = 1024;
+// Device buffers of a step of up to the largest batch.
+template <typename T>
+struct MoeBuffers {
+  uint32_t *chosen = nullptr;  // [rows][top]
+  float *score = nullptr;      // [rows][top]
+  uint32_t *histogram = nullptr;  // [moe_histogram_words]
+  uint32_t *place = nullptr;   // [rows][top]: sorted row of each choice
+  float *row_score = nullptr;  // [rows * top] by sorted row
+  MoeTile *tiles = nullptr;    // [plan.tiles]
+  T *x = nullptr;              // [rows * top][hidden] sorted rows
+  T *act = nullptr;            // [rows * top][ffn], then [rows][shared_ffn]
+  float *up = nullptr;         // k-split products of `up`, moe_up_floats
+  float *down = nullptr;       // [splits][rows * top][hidden]
+};
+size_t moe_histogram_words(MoeShape s, uint32_t rows);
+size_t moe_up_floats(bool is_bf16, MoeShape s, uint32_t rows);
+// Experts and scores of every row from the router's partial sums [splits][rows][experts], and the sorted order.
+template <typename T>
+int launch_moe_route(const float *logits, uint32_t splits, size_t split_stride, const T *x, MoeShape s, MoePlan plan, MoeBuffers<T> b,
+                     uint32_t rows, cudaStream_t stream);
+// Both products: `down` of the sorted rows into b.down, of the shared expert into shared_out [down_splits][rows][hidden].
+template <typename T>
+int launch_moe_experts(const T *x, const T *w_up, const T *w_down, const T *shared_up, const T *shared_down, MoeShape s, MoePlan plan,
+                       MoeBuffers<T> b, float *shared_out, uint32_t rows, cudaStream_t stream);
+// One product of the grouped kind on tcgen05: rows of `x` by tile through rows [expert * n, (expert + 1) * n) of `w`, and rows of
+// `shared_x` through `shared_w` (shared_n = 0: none). swiglu: activations to act / shared_act (row stride n / 2, shared_n / 2),
+// the products multiplied by row_score; else f32 to out / shared_out, [splits][rows][n].
+struct MoeProduct {
+  const bf16 *x, *w, *shared_x, *shared_w;
+  uint32_t n, k, shared_n, shared_k;
+  uint32_t sorted_rows, rows, experts;
+  const MoeTile *tiles;
+  const float *row_score;
+  bf16 *act, *shared_act;
+  float *out, *shared_out;
+};
+bool moe_tc_supported(MoeShape s);
+int launch_moe_product_tc(const MoeProduct &p, bool swiglu, uint32_t splits, MoePlan plan, cudaStream_t stream);
+int moe_poll_error(uint32_t *code);
+
 // ---- tensor-parallel hand-over ---------------------------------------------------
 
 constexpr int kMaxTpWorld = 8;

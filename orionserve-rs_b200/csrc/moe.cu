@@ -1,0 +1,328 @@
+// Mixture of experts: the choice of experts, the order of rows by expert, and the grouped products of the f32 build and of
+// sizes the tensor cores do not take (moe_gemm_tc.cu has the others).
+//   moe_choose_kernel  one warp per row: sigmoid scores of the router's logits, the `top` largest (the lower index of equal
+//                      ones), and a histogram per 64 rows
+//   moe_place_kernel   one warp per row: its places in the order by expert (rows of an expert keep their order, so the order
+//                      does not depend on timing), and the row copied there; the first CTA lists the tiles
+//   moe_simt_kernel    64 rows x 64 columns of one tile, k ascending, optionally with SwiGLU on the scored products
+//   moe_swiglu_kernel  the same activation on k-split products
+#include "kernels.h"
+#include "mma.cuh"
+
+#include <algorithm>
+
+namespace orion {
+namespace {
+
+constexpr uint32_t kRowBlock = 64;   // rows of one histogram
+constexpr uint32_t kChooseWarps = 8, kPlaceRows = 8;
+
+__global__ void __launch_bounds__(kChooseWarps * 32)
+moe_choose_kernel(const float *__restrict__ logits, uint32_t splits, size_t split_stride, uint32_t experts, uint32_t top, uint32_t rows,
+                  uint32_t *__restrict__ chosen, float *__restrict__ score, uint32_t *__restrict__ histogram) {
+  extern __shared__ float smem[];  // [warps][experts] scores, [experts] counts
+  uint32_t *count = reinterpret_cast<uint32_t *>(smem + kChooseWarps * experts);
+  pdl_trigger();
+  pdl_wait();
+  const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  float *mine = smem + warp * experts;
+  for (uint32_t e = tid; e < experts; e += blockDim.x) count[e] = 0;
+  __syncthreads();
+  const uint32_t end = min(rows, (blockIdx.x + 1) * kRowBlock);
+  for (uint32_t row = blockIdx.x * kRowBlock + warp; row < end; row += kChooseWarps) {
+    for (uint32_t e = lane; e < experts; e += 32) {
+      const float *p = logits + (size_t)row * experts + e;
+      float z = p[0];
+      for (uint32_t s = 1; s < splits; ++s) z += p[s * split_stride];
+      mine[e] = sigmoid_f(z);
+    }
+    __syncwarp();
+    for (uint32_t k = 0; k < top; ++k) {
+      float best = -1.f;
+      uint32_t at = 0xFFFFFFFFu;
+      for (uint32_t e = lane; e < experts; e += 32)
+        if (mine[e] > best) best = mine[e], at = e;
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+        const uint32_t oi = __shfl_xor_sync(0xffffffffu, at, o);
+        if (ov > best || (ov == best && oi < at)) best = ov, at = oi;
+      }
+      if (at >= experts) at = k;  // only if scores are not numbers: stay inside the expert list (top <= experts)
+      __syncwarp();
+      if (lane == 0) {
+        mine[at] = -2.f;
+        chosen[(size_t)row * top + k] = at;
+        score[(size_t)row * top + k] = best;
+        atomicAdd(&count[at], 1u);
+      }
+      __syncwarp();
+    }
+  }
+  __syncthreads();
+  for (uint32_t e = tid; e < experts; e += blockDim.x) histogram[(size_t)blockIdx.x * experts + e] = count[e];
+}
+
+// Exclusive prefix sums of f(value[i]) over `n` values in shared memory, by one warp.
+template <typename F>
+__device__ __forceinline__ void warp_prefix(const uint32_t *value, uint32_t n, uint32_t *prefix, F f) {
+  const uint32_t lane = threadIdx.x & 31;
+  uint32_t carry = 0;
+  for (uint32_t i0 = 0; i0 < n; i0 += 32) {
+    const uint32_t own = i0 + lane < n ? f(value[i0 + lane]) : 0;
+    uint32_t v = own;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const uint32_t up = __shfl_up_sync(0xffffffffu, v, o);
+      if (lane >= (uint32_t)o) v += up;
+    }
+    if (i0 + lane < n) prefix[i0 + lane] = carry + v - own;
+    carry += __shfl_sync(0xffffffffu, v, 31);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kPlaceRows * 32)
+moe_place_kernel(const uint32_t *__restrict__ chosen, const float *__restrict__ score, const uint32_t *__restrict__ histogram,
+                 const T *__restrict__ x, MoeShape s, uint32_t rows, uint32_t tile_rows, uint32_t max_tiles, uint32_t *__restrict__ place,
+                 float *__restrict__ row_score, MoeTile *__restrict__ tiles, T *__restrict__ sorted) {
+  extern __shared__ uint32_t words[];
+  uint32_t *total = words, *before = total + s.experts, *first = before + s.experts, *tile_at = first + s.experts;
+  pdl_trigger();
+  pdl_wait();
+  const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, E = s.experts, top = s.top;
+  for (uint32_t e = tid; e < 2 * E; e += blockDim.x) total[e] = 0;  // and `before`
+  __syncthreads();
+  const uint32_t row0 = blockIdx.x * kPlaceRows, block = row0 / kRowBlock, blocks = (rows + kRowBlock - 1) / kRowBlock;
+  for (uint32_t i = tid; i < blocks * E; i += blockDim.x) {
+    const uint32_t v = histogram[i], e = i % E;
+    if (v == 0) continue;
+    atomicAdd(&total[e], v);
+    if (i / E < block) atomicAdd(&before[e], v);
+  }
+  __syncthreads();
+  if (warp == 0) warp_prefix(total, E, first, [](uint32_t v) { return v; });
+  if (warp == 1 && blockIdx.x == 0) warp_prefix(total, E, tile_at, [&](uint32_t v) { return (v + tile_rows - 1) / tile_rows; });
+  __syncthreads();
+  if (blockIdx.x == 0) {
+    for (uint32_t e = tid; e < E; e += blockDim.x)
+      for (uint32_t t = 0; t * tile_rows < total[e]; ++t)
+        if (tile_at[e] + t < max_tiles) tiles[tile_at[e] + t] = MoeTile{e, first[e] + t * tile_rows, min(tile_rows, total[e] - t * tile_rows)};
+    const uint32_t used = tile_at[E - 1] + (total[E - 1] + tile_rows - 1) / tile_rows;
+    for (uint32_t t = used + tid; t < max_tiles; t += blockDim.x) tiles[t] = MoeTile{0, 0, 0};
+  }
+  const uint32_t row = row0 + warp;
+  if (row >= rows) return;
+  for (uint32_t k = 0; k < top; ++k) {
+    const uint32_t at = row * top + k, e = chosen[at];
+    uint32_t rank = 0;  // choices of the same expert before this one in the block of rows
+    for (uint32_t j = block * kRowBlock * top; j < at; j += 32) {
+      const uint32_t other = j + lane < at ? chosen[j + lane] : 0xFFFFFFFFu;
+      rank += __popc(__ballot_sync(0xffffffffu, other == e));
+    }
+    const uint32_t to = first[e] + before[e] + rank;
+    if (lane == 0) {
+      place[at] = to;
+      row_score[to] = score[at];
+    }
+    const T *src = x + (size_t)row * s.hidden;
+    T *dst = sorted + (size_t)to * s.hidden;
+    constexpr uint32_t kVec = 16 / sizeof(T);
+    if (s.hidden % kVec == 0) {
+      for (uint32_t c = lane; c < s.hidden / kVec; c += 32) reinterpret_cast<uint4 *>(dst)[c] = reinterpret_cast<const uint4 *>(src)[c];
+    } else {
+      for (uint32_t c = lane; c < s.hidden; c += 32) dst[c] = src[c];
+    }
+  }
+}
+
+// silu(w g) * (w u): the score of a routed row multiplies what the expert reads.
+template <typename T>
+__device__ __forceinline__ float scored_swiglu(float g, float u, float w) {
+  return silu_for<T>(w * g) * (w * u);
+}
+
+constexpr uint32_t BM = 64, BN = 64, BK = 16;
+template <typename T>
+struct SimtFamily {
+  const T *x, *w;
+  uint32_t n, k;
+  T *act;
+  float *out;
+};
+template <typename T, bool SWIGLU>
+__global__ void __launch_bounds__(256)
+moe_simt_kernel(SimtFamily<T> routed, SimtFamily<T> shared, uint32_t shared_tiles, uint32_t rows, const MoeTile *__restrict__ tiles,
+                const float *__restrict__ row_score) {
+  __shared__ float xs[BK][BM + 1], ws[BK][BN + 1];
+  pdl_trigger();
+  pdl_wait();
+  const bool is_shared = blockIdx.y < shared_tiles;
+  const SimtFamily<T> f = is_shared ? shared : routed;
+  MoeTile t;
+  if (is_shared) t = MoeTile{0, blockIdx.y * BM, min(BM, rows - blockIdx.y * BM)};
+  else t = tiles[blockIdx.y - shared_tiles];
+  const uint32_t n0 = blockIdx.x * BN;
+  if (t.count == 0 || n0 >= f.n) return;
+  const T *w = f.w + (size_t)t.expert * f.n * f.k;
+  const uint32_t tx = threadIdx.x % 16, ty = threadIdx.x / 16;
+  float acc[4][4] = {};
+  for (uint32_t k0 = 0; k0 < f.k; k0 += BK) {
+    for (uint32_t idx = threadIdx.x; idx < BM * BK; idx += 256) {
+      const uint32_t r = idx / BK, k = k0 + idx % BK;
+      xs[idx % BK][r] = r < t.count && k < f.k ? to_f32<T>(f.x[(size_t)(t.row + r) * f.k + k]) : 0.f;
+      ws[idx % BK][r] = n0 + r < f.n && k < f.k ? to_f32<T>(w[(size_t)(n0 + r) * f.k + k]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (uint32_t k = 0; k < BK; ++k) {
+      float a[4], b[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) a[i] = xs[k][ty * 4 + i], b[i] = ws[k][tx * 4 + i];
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const uint32_t r = ty * 4 + i;
+    if (r >= t.count) continue;
+    const size_t row = t.row + r;
+    const float score = is_shared || !SWIGLU ? 1.f : row_score[row];
+#pragma unroll
+    for (int j = 0; j < 4; j += SWIGLU ? 2 : 1) {
+      const uint32_t n = n0 + tx * 4 + j;
+      if (n >= f.n) continue;
+      if (SWIGLU) f.act[row * (f.n / 2) + n / 2] = from_f32<T>(scored_swiglu<T>(acc[i][j], acc[i][j + (SWIGLU ? 1 : 0)], score));
+      else f.out[row * f.n + n] = acc[i][j];
+    }
+  }
+}
+
+// Products [splits][rows][2 * ffn] with gate and up in neighbouring columns -> act [rows][ffn]; routed rows first.
+template <typename T>
+__global__ void __launch_bounds__(256)
+moe_swiglu_kernel(const float *__restrict__ up, uint32_t splits, MoeShape s, uint32_t rows, const float *__restrict__ row_score, T *__restrict__ act) {
+  pdl_trigger();
+  pdl_wait();
+  const size_t sorted = (size_t)rows * s.top, routed = sorted * s.ffn, all = routed + (size_t)rows * s.shared_ffn;
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < all; i += (size_t)gridDim.x * blockDim.x) {
+    const bool is_shared = i >= routed;
+    const size_t stride = is_shared ? (size_t)rows * 2 * s.shared_ffn : sorted * 2 * s.ffn;
+    const float2 *p = reinterpret_cast<const float2 *>(up + (is_shared ? splits * sorted * 2 * s.ffn + 2 * (i - routed) : 2 * i));
+    float2 v = make_float2(0.f, 0.f);
+    for (uint32_t k = 0; k < splits; ++k) {
+      const float2 q = p[k * stride / 2];
+      v.x += q.x, v.y += q.y;
+    }
+    act[i] = from_f32<T>(scored_swiglu<T>(v.x, v.y, is_shared ? 1.f : row_score[i / s.ffn]));
+  }
+}
+
+inline int after_launch(const char *stage) {
+  count_launch();
+  ORION_CUDA_CHECK(stage, cudaGetLastError());
+  return ORION_OK;
+}
+
+}  // namespace
+
+size_t moe_histogram_words(MoeShape s, uint32_t rows) { return (size_t)((rows + kRowBlock - 1) / kRowBlock) * s.experts; }
+
+MoePlan moe_plan(bool is_bf16, MoeShape s, uint32_t rows) {
+  MoePlan p{BM, 0, 1, 1, is_bf16 && moe_tc_supported(s)};
+  const uint64_t choices = (uint64_t)rows * s.top;
+  if (p.tensor_core) {
+    // Few rows: one tile holds every row of an expert and all rows of the shared one. More: by the mean rows of an expert.
+    const uint64_t mean = (choices + s.experts - 1) / s.experts;
+    p.tile_rows = rows <= 16 ? 16 : (rows <= 32 ? 32 : (rows <= 64 || mean <= 48 ? 64 : (mean <= 160 ? 128 : 256)));
+  }
+  const uint64_t busy = std::min<uint64_t>(s.experts, choices);  // experts that have rows, at most
+  p.tiles = (uint32_t)(busy + choices / p.tile_rows);
+  if (p.tensor_core && rows <= 64) {
+    // k splits until a wave of two CTAs per SM is full, at least four k slabs each
+    auto splits = [&](uint32_t n, uint32_t shared_n, uint32_t k) {
+      const uint64_t ctas = busy * ((n + 127) / 128) + (shared_n + 127) / 128;
+      const uint32_t most = std::max(1u, (k + 63) / 64 / 4);
+      return (uint32_t)std::max<uint64_t>(1, std::min<uint64_t>({296 / std::max<uint64_t>(1, ctas), most, 8}));
+    };
+    p.up_splits = splits(2 * s.ffn, 2 * s.shared_ffn, s.hidden);
+    p.down_splits = splits(s.hidden, s.shared_ffn ? s.hidden : 0, s.ffn);
+  }
+  return p;
+}
+
+size_t moe_up_floats(bool is_bf16, MoeShape s, uint32_t rows) {
+  const MoePlan p = moe_plan(is_bf16, s, rows);
+  return p.up_splits == 1 ? 0 : (size_t)p.up_splits * rows * 2 * ((size_t)s.top * s.ffn + s.shared_ffn);
+}
+
+template <typename T>
+int launch_moe_route(const float *logits, uint32_t splits, size_t split_stride, const T *x, MoeShape s, MoePlan plan, MoeBuffers<T> b,
+                     uint32_t rows, cudaStream_t stream) {
+  if (rows == 0) return ORION_OK;
+  if (s.experts == 0 || s.experts > kMoeMaxExperts || s.top == 0 || s.top > s.experts)
+    return set_error(ORION_ERR_INTERNAL, "routing of %u among %u experts is not supported (at most %u)", s.top, s.experts, kMoeMaxExperts);
+  ORION_CUDA_CHECK("moe_choose", launch_pdl(moe_choose_kernel, dim3((rows + kRowBlock - 1) / kRowBlock), dim3(kChooseWarps * 32),
+                                            (kChooseWarps + 1) * s.experts * sizeof(float), stream, logits, splits, split_stride, s.experts, s.top,
+                                            rows, b.chosen, b.score, b.histogram));
+  ORION_TRY(after_launch("moe_choose"));
+  ORION_CUDA_CHECK("moe_place", launch_pdl(moe_place_kernel<T>, dim3((rows + kPlaceRows - 1) / kPlaceRows), dim3(kPlaceRows * 32),
+                                           4 * s.experts * sizeof(uint32_t), stream, b.chosen, b.score, b.histogram, x, s, rows, plan.tile_rows,
+                                           plan.tiles, b.place, b.row_score, b.tiles, b.x));
+  return after_launch("moe_place");
+}
+
+namespace {
+template <typename T>
+int launch_simt(bool swiglu, SimtFamily<T> routed, SimtFamily<T> shared, MoePlan plan, const MoeBuffers<T> &b, uint32_t rows, cudaStream_t stream) {
+  const uint32_t shared_tiles = shared.n ? (rows + BM - 1) / BM : 0;
+  const dim3 grid((std::max(routed.n, shared.n) + BN - 1) / BN, shared_tiles + plan.tiles);
+  auto kernel = swiglu ? moe_simt_kernel<T, true> : moe_simt_kernel<T, false>;
+  ORION_CUDA_CHECK("moe_simt", launch_pdl(kernel, grid, dim3(256), 0, stream, routed, shared, shared_tiles, rows, (const MoeTile *)b.tiles,
+                                          (const float *)b.row_score));
+  return after_launch("moe_simt");
+}
+}  // namespace
+
+template <typename T>
+int launch_moe_experts(const T *x, const T *w_up, const T *w_down, const T *shared_up, const T *shared_down, MoeShape s, MoePlan plan,
+                       MoeBuffers<T> b, float *shared_out, uint32_t rows, cudaStream_t stream) {
+  if (rows == 0) return ORION_OK;
+  const size_t sorted = (size_t)rows * s.top;
+  T *shared_act = b.act + sorted * s.ffn;
+  if constexpr (sizeof(T) == 2) {
+    if (plan.tensor_core) {
+      const bool fused = plan.up_splits == 1;
+      float *shared_up_out = fused ? nullptr : b.up + plan.up_splits * sorted * 2 * s.ffn;
+      MoeProduct p{b.x, w_up, x, shared_up, 2 * s.ffn, s.hidden, 2 * s.shared_ffn, s.hidden, (uint32_t)sorted, rows, s.experts, b.tiles, b.row_score,
+                   b.act, shared_act, fused ? nullptr : b.up, shared_up_out};
+      ORION_TRY(launch_moe_product_tc(p, fused, plan.up_splits, plan, stream));
+      if (!fused) {
+        const size_t n = sorted * s.ffn + (size_t)rows * s.shared_ffn;
+        ORION_CUDA_CHECK("moe_swiglu", launch_pdl(moe_swiglu_kernel<T>, dim3((uint32_t)std::min<size_t>((n + 255) / 256, 148 * 8)), dim3(256), 0, stream,
+                                                  (const float *)b.up, plan.up_splits, s, rows, (const float *)b.row_score, b.act));
+        ORION_TRY(after_launch("moe_swiglu"));
+      }
+      MoeProduct d{b.act, w_down, shared_act, shared_down, s.hidden, s.ffn, s.shared_ffn ? s.hidden : 0, s.shared_ffn, (uint32_t)sorted, rows, s.experts,
+                   b.tiles, nullptr, nullptr, nullptr, b.down, shared_out};
+      return launch_moe_product_tc(d, false, plan.down_splits, plan, stream);
+    }
+  }
+  ORION_TRY(launch_simt<T>(true, {b.x, w_up, 2 * s.ffn, s.hidden, b.act, nullptr}, {x, shared_up, 2 * s.shared_ffn, s.hidden, shared_act, nullptr}, plan,
+                           b, rows, stream));
+  return launch_simt<T>(false, {b.act, w_down, s.hidden, s.ffn, nullptr, b.down},
+                        {shared_act, shared_down, s.shared_ffn ? s.hidden : 0, s.shared_ffn, nullptr, shared_out}, plan, b, rows, stream);
+}
+
+#define ORION_INSTANTIATE(T)                                                                                                            \
+  template int launch_moe_route<T>(const float *, uint32_t, size_t, const T *, MoeShape, MoePlan, MoeBuffers<T>, uint32_t, cudaStream_t); \
+  template int launch_moe_experts<T>(const T *, const T *, const T *, const T *, const T *, MoeShape, MoePlan, MoeBuffers<T>, float *,    \
+                                     uint32_t, cudaStream_t);
+ORION_INSTANTIATE(float)
+ORION_INSTANTIATE(bf16)
+
+}  // namespace orion
