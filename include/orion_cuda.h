@@ -124,31 +124,51 @@ void orion_cuda_model_destroy(OrionModel *model);
 
 /* ---- layer-list models (no reference counterpart) ----
  * Decoders whose layers are listed one by one, each with a token mixer of its own sizes and an
- * optional feed-forward. A layer is parallel: h = RMSNorm(x); the mixer and the feed-forward each read
- * h plus a causal per-channel convolution of h over `conv_taps` tokens, and both results are added to
- * x. The logits are the final norm's output times the embedding table. Metapel is the one design
- * of this kind. */
-enum { ORION_MIXER_MIN_GRU = 0, ORION_MIXER_LATENT_ATTENTION = 1 };
+ * optional feed-forward. A layer is one of two blocks, the same throughout a model.
+ * Parallel: h = RMSNorm(x); the mixer and the feed-forward each read h plus a causal per-channel
+ * convolution of h over `conv_taps` tokens, and both results are added to x.
+ * Sandwich: x += m RMSNorm(mixer(RMSNorm(x))), then x += m RMSNorm(ffn(RMSNorm(x))), m = residual_mult.
+ * The logits are the final norm's output times the embedding table or an output matrix of their own.
+ * Metapel is a design with parallel blocks, Zulozen one with sandwich blocks. */
+enum { ORION_MIXER_MIN_GRU = 0, ORION_MIXER_LATENT_ATTENTION = 1, ORION_MIXER_ATTENTION = 2 };
+enum { ORION_BLOCK_PARALLEL = 0, ORION_BLOCK_SANDWICH = 1 };
+enum { ORION_ACT_GELU_TANH = 0, ORION_ACT_RELU2 = 1 };
 typedef struct OrionLayerDesc {
   uint32_t mixer;    /* ORION_MIXER_* */
-  uint32_t ffn_dim;  /* width of the dense GELU feed-forward; 0 = the layer has none */
+  uint32_t ffn_dim;  /* width of the feed-forward, or of each of its experts; 0 = the layer has none */
   uint32_t width;    /* min_gru: channels of the recurrence */
   /* latent_attention: query heads, unrotated and rotated query/key dimensions and value size per head,
    * latent size, sliding window in tokens (0 = every earlier token is seen), rotated pairs' dimensions
-   * and base, score scale */
+   * and base, score scale. attention: the same without rot_dim and kv_rank; dim is the whole size of a
+   * query or key, of which the first rope_dims rotate */
   uint32_t heads, dim, rot_dim, value_dim, kv_rank, window, rope_dims;
   double rope_base, scale;
+  /* attention: key/value heads (each shared by heads / kv_heads query heads); chunk size (a position sees
+   * those before it in its own chunk, chunks counted from position 0; 0 = no chunks); whether queries and
+   * keys are normalised (RMS over all heads at once, before the rotation), whether every head has a
+   * learned logit in its softmax denominator, and whether a sigmoid per head gates its output */
+  uint32_t kv_heads, chunk, qk_norm, sinks, head_gate;
+  /* dense feed-forward (experts = 0): ORION_ACT_*, and whether both projections have biases (sandwich
+   * blocks only) */
+  uint32_t activation, ffn_bias;
+  /* mixture of experts (sandwich blocks only): SwiGLU experts, of which every token uses experts_per_token,
+   * chosen and weighted (at their input) by the sigmoid of the router's logits; width of an expert that
+   * every token uses (0 = none) */
+  uint32_t experts, experts_per_token, shared_dim;
 } OrionLayerDesc;
 typedef struct OrionLayeredDesc {
   uint32_t hidden_size, vocab_size, num_layers;
   const OrionLayerDesc *layers; /* [num_layers], read during the call only */
   double norm_eps;
-  uint32_t conv_taps;           /* 1 or more; conv_taps - 1 rows of h per layer are a sequence's state */
+  uint32_t conv_taps;           /* parallel blocks: 1 or more; conv_taps - 1 rows of h per layer are a sequence's state */
   uint32_t max_position_embeddings; /* positions the rotation tables cover */
-  uint32_t num_blocks, block_size;  /* paged latent cache */
-  uint32_t num_state_slots;         /* sequences whose state is held at any time */
+  uint32_t num_blocks, block_size;  /* paged cache of latents, or of keys and values */
+  uint32_t num_state_slots;         /* sequences whose state is held at any time (models with state) */
   uint32_t compute_dtype;           /* ORION_DTYPE_F32 or ORION_DTYPE_BF16 */
   uint32_t max_batch_tokens, max_batch_sequences;
+  uint32_t block;                   /* ORION_BLOCK_* */
+  uint32_t untied_lm_head;          /* the logits have a matrix of their own */
+  double residual_mult;             /* sandwich blocks */
 } OrionLayeredDesc;
 int orion_cuda_model_create_layered(OrionBackend *backend, const OrionLayeredDesc *desc, OrionModel **out);
 /* State slots of the model: 0 for models that carry nothing but the KV cache from step to step. */
@@ -172,8 +192,8 @@ int orion_cuda_selftest_peer_wait(OrionBackend *backend, uint64_t limit_us, uint
 
 /* Reads and clears the time-out words of the backend's device (no reference counterpart): bit 0 the
  * projection GEMM, bit 1 decode attention, bit 2 prefill attention, bit 3 the tensor-parallel
- * hand-over. A set bit means a bounded device-side wait of that kernel family gave up since the last
- * read. orion_cuda_model_forward reads the words itself after every step; a caller that launches
+ * hand-over, bit 4 the grouped products of a mixture of experts. A set bit means a bounded
+ * device-side wait of that kernel family gave up since the last read. orion_cuda_model_forward reads the words itself after every step; a caller that launches
  * kernels through the stand-alone entry points (orion_cuda_paged_decode_attention_noalloc) and wants
  * to know whether one of its launches timed out synchronises its stream and calls this. */
 int orion_cuda_poll_wait_timeouts(OrionBackend *backend, uint32_t *mask);

@@ -46,8 +46,8 @@ typedef struct OrionCacheStats {
  * recompute_on_preempt: for sequences that carry state from token to token. Non-zero prefills a preempted
  * sequence's generated tokens again after its prompt (the reference leaves them out of the cache) and a
  * failed step's prompt portions again, does not preempt to admit, schedules a sequence at most once per step
- * and accepts a request only if prompt and output fit the cache together. An engine around a model with state slots sets this and
- * logical_decode_positions itself, and refuses skip_cached_prefix. */
+ * and accepts a request only if prompt and output fit the cache together. An engine around a layer-list model sets this and
+ * logical_decode_positions itself, and refuses skip_cached_prefix if the model has state slots. */
 typedef struct OrionSchedulerConfig {
   uint64_t max_num_seqs, max_num_batched_tokens, max_model_len;
   uint32_t enable_chunked_prefill;

@@ -40,7 +40,9 @@ class OrionModelDesc(C.Structure):
 
 class OrionLayerDesc(C.Structure):
     _fields_ = [(n, C.c_uint32) for n in ("mixer", "ffn_dim", "width", "heads", "dim", "rot_dim", "value_dim", "kv_rank",
-                                          "window", "rope_dims")] + [("rope_base", C.c_double), ("scale", C.c_double)]
+                                          "window", "rope_dims")] + [("rope_base", C.c_double), ("scale", C.c_double)] + \
+               [(n, C.c_uint32) for n in ("kv_heads", "chunk", "qk_norm", "sinks", "head_gate", "activation", "ffn_bias", "experts",
+                                          "experts_per_token", "shared_dim")]
 
 
 class OrionLayeredDesc(C.Structure):
@@ -48,10 +50,13 @@ class OrionLayeredDesc(C.Structure):
                 ("layers", C.POINTER(OrionLayerDesc)), ("norm_eps", C.c_double), ("conv_taps", C.c_uint32),
                 ("max_position_embeddings", C.c_uint32), ("num_blocks", C.c_uint32), ("block_size", C.c_uint32),
                 ("num_state_slots", C.c_uint32), ("compute_dtype", C.c_uint32), ("max_batch_tokens", C.c_uint32),
-                ("max_batch_sequences", C.c_uint32)]
+                ("max_batch_sequences", C.c_uint32), ("block", C.c_uint32), ("untied_lm_head", C.c_uint32),
+                ("residual_mult", C.c_double)]
 
 
-MIXER_MIN_GRU, MIXER_LATENT_ATTENTION = 0, 1
+MIXER_MIN_GRU, MIXER_LATENT_ATTENTION, MIXER_ATTENTION = 0, 1, 2
+BLOCK_PARALLEL, BLOCK_SANDWICH = 0, 1
+ACT_GELU_TANH, ACT_RELU2 = 0, 1
 
 _lib = None
 

@@ -220,7 +220,7 @@ struct SchedulerConfig {  // crates/orion-core/src/config.rs:107-156
   // (recurrent state): a preempted sequence that has generated tokens prefills them again after its prompt (the
   // reference drops them from the cache and goes on behind them); a step that failed is prefilled again; running
   // sequences are not preempted to admit waiting ones; a sequence is in a step at most once; and a request is
-  // accepted only if prompt and output fit the cache together. Models with state slots set it and
+  // accepted only if prompt and output fit the cache together. Layer-list models set it and
   // logical_decode_positions themselves.
   bool recompute_on_preempt = false;
 };

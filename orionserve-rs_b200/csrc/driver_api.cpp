@@ -261,16 +261,12 @@ OrionEngine *orion_engine_create(OrionModel *model, OrionForwardFn forward, void
   }
   ForwardFn fn;
   SchedulerConfig cfg = to_config(config);
-  size_t state_slots = 0;
-  if (model && (state_slots = model->impl->num_state_slots()) > 0) {
-    // State is carried from token to token: positions follow one another without a gap, and nothing of a
-    // sequence can be skipped because another one has cached it.
-    if (cfg.skip_cached_prefix) {
-      set_error(ORION_ERR_INVALID_REQUEST, "skip_cached_prefix: a model with recurrent state computes every token of a sequence");
-      return nullptr;
-    }
-    cfg.logical_decode_positions = cfg.recompute_on_preempt = true;
+  const size_t state_slots = model ? model->impl->num_state_slots() : 0;
+  if (state_slots > 0 && cfg.skip_cached_prefix) {  // nothing of a sequence can be skipped because another one has cached it
+    set_error(ORION_ERR_INVALID_REQUEST, "skip_cached_prefix: a model with recurrent state computes every token of a sequence");
+    return nullptr;
   }
+  if (model && model->impl->logical_positions()) cfg.logical_decode_positions = cfg.recompute_on_preempt = true;
   if (model) {
     ModelBase *impl = model->impl.get();
     fn = [impl](const HostBatch &b, uint32_t *token_ids) -> int {

@@ -64,6 +64,9 @@ class ModelBase {
   virtual bool uses_tensor(const char *name) const = 0;
   // State slots the model was made with (0: nothing but the KV cache is carried from step to step).
   virtual uint32_t num_state_slots() const { return 0; }
+  // Whether an engine has to feed every token at its own place in the sequence, and a preempted sequence's generated tokens
+  // again (the reference's engine does neither).
+  virtual bool logical_positions() const { return false; }
   virtual int init_random(uint64_t seed, float std) = 0;
   virtual int finalize() = 0;
   virtual int forward(const BatchView &b, float *logits_out, uint64_t logits_capacity,

@@ -68,7 +68,7 @@ class SchedulerConfig:
     #: total_len, so no cache slot is skipped and no step is refused
     logical_decode_positions: bool = False
     #: not in the reference: a preempted sequence prefills its generated tokens again after its prompt.
-    #: An engine around a model with state slots turns this and logical_decode_positions on by itself.
+    #: An engine around a layer-list model turns this and logical_decode_positions on by itself.
     recompute_on_preempt: bool = False
 
     def _c(self):

@@ -7,11 +7,11 @@ import os
 
 from .backend import CudaBackend
 from .errors import ModelError
-from .layered import CudaLayeredModel
+from .layered import READERS, CudaLayeredModel
 from .model import CudaModel, CudaTransformerModel
 
 #: config.json "architecture" -> model class; configs without that key are Hugging Face ones
-ARCHITECTURES = {"Metapel": CudaLayeredModel}
+ARCHITECTURES = {name: CudaLayeredModel for name in READERS}
 
 
 def model_class(directory: str):
