@@ -353,7 +353,8 @@ def run_serving(args):
 
 
 # ---------------------------------------------------------------------------------------------
-# Metapel (min-GRU and latent attention layers) beside the Llama layout at equal size
+# Layer-list designs beside the Llama layout at equal size: Metapel (min-GRU and latent attention layers) and Zulozen
+# (chunked attention with sinks, dense and mixture-of-experts feed-forwards)
 # ---------------------------------------------------------------------------------------------
 
 # Layer sizes of real models, random weights; the layers alternate min-GRU and latent attention.
@@ -361,7 +362,15 @@ METAPEL_SHAPES = {
     "2048": dict(hidden=2048, ffn=8192, width=2048, heads=16, dim=128, rot=64, vdim=128, rank=512, window=1024),
     "4096": dict(hidden=4096, ffn=16384, width=4096, heads=32, dim=128, rot=64, vdim=128, rank=512, window=1024),
 }
-METAPEL_VOCAB = 32768
+LAYERED_VOCAB = 32768
+
+
+# The layers alternate a dense feed-forward and a mixture; a token's experts and the shared one together are as large as the dense
+# one. Contexts and prompts of the batches below stay inside one chunk, so attention does the work of the Llama layout's.
+ZULOZEN_SHAPES = {
+    "2048": dict(hidden=2048, ffn=8192, heads=16, dim=128, rot=64, chunk=2048, experts=16, top=2, expert_ffn=1408, shared=2816),
+    "4096": dict(hidden=4096, ffn=16384, heads=32, dim=128, rot=64, chunk=2048, experts=16, top=2, expert_ffn=2816, shared=5632),
+}
 
 
 def metapel_meta(pkg, name, layers):
@@ -370,7 +379,7 @@ def metapel_meta(pkg, name, layers):
     att = pkg.LayerSpec("latent_attention", z["ffn"], heads=z["heads"], dim=z["dim"], rot_dim=z["rot"], value_dim=z["vdim"],
                         kv_rank=z["rank"], window=z["window"], rope_dims=z["rot"], rope_base=10000.0,
                         scale=(z["dim"] + z["rot"]) ** -0.5)
-    return pkg.LayeredMetadata("Metapel", f"metapel-{name}", z["hidden"], METAPEL_VOCAB,
+    return pkg.LayeredMetadata("Metapel", f"metapel-{name}", z["hidden"], LAYERED_VOCAB,
                                [att if i % 2 else gru for i in range(layers)], 1e-6, 4)
 
 
@@ -396,7 +405,39 @@ def metapel_work(meta, rows, contexts, prompts):
         n += 2 * H * s.ffn_dim
         w, flops = w + 2 * n, flops + 2 * n * rows
     outs = len(contexts) + len(prompts)
-    return w + 2 * METAPEL_VOCAB * meta.hidden_size, flops + 2 * outs * METAPEL_VOCAB * meta.hidden_size, cache, attn
+    return w + 2 * LAYERED_VOCAB * meta.hidden_size, flops + 2 * outs * LAYERED_VOCAB * meta.hidden_size, cache, attn
+
+
+def zulozen_meta(pkg, name, layers):
+    z = ZULOZEN_SHAPES[name]
+    att = dict(heads=z["heads"], kv_heads=z["heads"] // 4, dim=z["dim"], value_dim=z["dim"], chunk=z["chunk"], rope_dims=z["rot"],
+               rope_base=10000.0, scale=z["dim"] ** -0.5, qk_norm=True, sinks=True, head_gate=True)
+    dense = pkg.LayerSpec("attention", z["ffn"], activation="relu2", ffn_bias=True, **att)
+    mix = pkg.LayerSpec("attention", z["expert_ffn"], experts=z["experts"], experts_per_token=z["top"], shared_dim=z["shared"], **att)
+    return pkg.LayeredMetadata("Zulozen", f"zulozen-{name}", z["hidden"], LAYERED_VOCAB, [mix if i % 2 else dense for i in range(layers)],
+                               1e-6, block="sandwich", untied_lm_head=True, residual_mult=0.5)
+
+
+def zulozen_work(meta, rows, contexts, prompts):
+    """As ``metapel_work``. The weights of a mixture are those of the experts that `rows` independent choices reach on average."""
+    w = flops = cache = attn = 0
+    H = meta.hidden_size
+    for s in meta.layers:
+        n = H * (s.heads * s.dim + s.kv_heads * (s.dim + s.value_dim) + s.heads) + s.heads * s.value_dim * H
+        if s.experts:
+            fixed, one = H * s.experts + 3 * H * s.shared_dim, 3 * H * s.ffn_dim
+            reached = s.experts * (1.0 - (1.0 - s.experts_per_token / s.experts) ** rows)
+            w, n = w + 2 * int(reached * one), n + fixed
+            flops += 2 * s.experts_per_token * one * rows
+        else:
+            n += 2 * H * s.ffn_dim
+        seen = [(c - 1) % s.chunk + 1 if s.chunk else c for c in contexts]
+        cache += sum(seen) * s.kv_heads * (s.dim + s.value_dim) * 2
+        keys = sum(seen) + sum((i % s.chunk if s.chunk else i) + 1 for p in prompts for i in range(p))
+        attn += keys * s.heads * 2 * (s.dim + s.value_dim)
+        w, flops = w + 2 * n, flops + 2 * n * rows
+    outs = len(contexts) + len(prompts)
+    return w + 2 * LAYERED_VOCAB * H, flops + 2 * outs * LAYERED_VOCAB * H, cache, attn
 
 
 def llama_work(m, rows, contexts, prompts):
@@ -407,8 +448,8 @@ def llama_work(m, rows, contexts, prompts):
     return w, flops, kv_bytes_per_step(m, contexts) if contexts else 0, m["num_layers"] * (keys + sum(contexts)) * q * 4
 
 
-def run_metapel(args):
-    """Prefill and decode throughput of Metapel at a few layer sizes, and of the Llama layout (same hidden size, head
+def run_layered(args):
+    """Prefill and decode throughput of a layer-list design at a few layer sizes, and of the Llama layout (same hidden size, head
     count and head size, four query heads per KV head, feed-forward of equal parameter count) on the same
     batches. Times are CUDA events around whole replayed steps and around one kernel family run back to back."""
     import __graft_entry__ as ge
@@ -421,32 +462,35 @@ def run_metapel(args):
             tflops = float(json.load(f)["bf16_tflops_sustained"])
     except (OSError, ValueError, KeyError):
         tflops = 1400.0
+    design = args.workload
+    shapes, make_meta, work = {"metapel": (METAPEL_SHAPES, metapel_meta, metapel_work),
+                               "zulozen": (ZULOZEN_SHAPES, zulozen_meta, zulozen_work)}[design]
     layers, out = args.layers if args.layers != 32 else 8, []
     batches = [("decode", b, CONTEXT) for b in (1, 16, 64)] + [("prefill", 1, 2048), ("prefill", 4, 2048)]
     with ClockSampler(0) as clocks:
-        for name in args.metapel_shapes.split(","):
-            z = METAPEL_SHAPES[name]
+        for name in args.layered_shapes.split(","):
+            z = shapes[name]
             m = dict(hidden_size=z["hidden"], num_layers=layers, num_attention_heads=z["heads"], num_kv_heads=z["heads"] // 4,
-                     head_dim=128, vocab_size=METAPEL_VOCAB, ffn_dim=(z["ffn"] * 2 // 3 + 127) // 128 * 128,
+                     head_dim=128, vocab_size=LAYERED_VOCAB, ffn_dim=(z["ffn"] * 2 // 3 + 127) // 128 * 128,
                      max_position_embeddings=8192, rope_theta=500000.0, rms_norm_eps=1e-5)
             blocks = max(b * c // BLOCK for _, b, c in batches) + 64
-            for kind in ("metapel", "llama"):
+            for kind in (design, "llama"):
                 kw = dict(compute_dtype=pkg.DType.BF16, max_batch_tokens=8192, max_batch_sequences=64)
-                if kind == "metapel":
-                    meta = metapel_meta(pkg, name, layers)
+                if kind == design:
+                    meta = make_meta(pkg, name, layers)
                     model = pkg.CudaLayeredModel(meta, blocks, BLOCK, backend, **kw)
                 else:
                     meta = pkg.ModelMetadata(architecture="llama", name="llama", dtype=pkg.DType.BF16, **m)
                     model = pkg.CudaTransformerModel(meta, blocks, BLOCK, backend, **kw)
                 model.init_random(seed=1, std=0.02)
                 for mode, b, n in batches:
-                    if args.metapel_only and f"{mode}{b}" not in args.metapel_only.split(","):
+                    if args.layered_only and f"{mode}{b}" not in args.layered_only.split(","):
                         continue
                     rng = np.random.default_rng(3)
                     tables = [list(range(s * n // BLOCK, (s + 1) * n // BLOCK)) for s in range(b)]
-                    slots = list(range(b)) if kind == "metapel" else None
+                    slots = list(range(b)) if model.num_state_slots() else None
                     ids = list(range(1, b + 1))
-                    prompt = rng.integers(0, METAPEL_VOCAB, n)
+                    prompt = rng.integers(0, LAYERED_VOCAB, n)
                     count = n if mode == "prefill" else n - 1
                     per = max(1, 8192 // n)
                     for s0 in range(0, b, per):  # real prompts: the decode steps go on from their state and cache
@@ -464,7 +508,7 @@ def run_metapel(args):
                     ms = model.replay(steps) / steps
                     launches = model.last_launch_count()
                     fam = {c: model.replay_categories(steps, c) / steps for c in ("gemm", "attention", "elementwise")}
-                    wb, fl, cb, af = (metapel_work(meta, rows, contexts, prompts) if kind == "metapel"
+                    wb, fl, cb, af = (work(meta, rows, contexts, prompts) if kind == design
                                       else llama_work(m, rows, contexts, prompts))
                     gemm_s, attn_s = fam["gemm"] / 1e3, fam["attention"] / 1e3
                     out.append({"model": kind, "shape": name, "layers": layers, "mode": mode, "sequences": b, "tokens_each": n,
@@ -473,7 +517,7 @@ def run_metapel(args):
                                 "gemm_frac": max(wb / gemm_s / hbm / 1e9, fl / gemm_s / tflops / 1e12),
                                 "step_frac": max((wb + cb) / (ms / 1e3) / hbm / 1e9, (fl + af) / (ms / 1e3) / tflops / 1e12)})
                 del model
-    print(json.dumps({"metric": "Metapel prefill and decode throughput beside the Llama layout", "unit": "tokens/s", "n_gpus": 1,
+    print(json.dumps({"metric": f"{design.capitalize()} prefill and decode throughput beside the Llama layout", "unit": "tokens/s", "n_gpus": 1,
                       "dtype": "bf16", "data": "synthetic", "peaks": {"hbm_gbs": hbm, "bf16_tflops_sustained": tflops, "source": src},
                       "results": out, "clocks": clocks.summary()}))
     return 0
@@ -627,8 +671,8 @@ def tp_parity(pkg, backend, dist, rank, world, dtype_name="BF16", model=None, nu
 def run_ours(args):
     if args.workload in ("serving", "prefix"):
         return run_serving(args)
-    if args.workload == "metapel":
-        return run_metapel(args)
+    if args.workload in ("metapel", "zulozen"):
+        return run_layered(args)
     import __graft_entry__ as ge
 
     pkg = ge.load_package()
@@ -843,12 +887,13 @@ def main():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", choices=("ours", "reference"), default="ours")
     ap.add_argument("--no-cpu-baseline", action="store_true")
-    ap.add_argument("--workload", choices=("decode", "serving", "prefix", "metapel"), default="decode",
+    ap.add_argument("--workload", choices=("decode", "serving", "prefix", "metapel", "zulozen"), default="decode",
                     help="decode = the headline step (default); serving = continuous batching through the engine "
-                         "loop; prefix = shared-prefix requests on the Qwen2-7B shape through the engine loop; metapel = prefill "
-                         "and decode of the Metapel design at a few sizes beside the Llama layout")
-    ap.add_argument("--metapel-shapes", default="2048,4096", help="metapel workload: layer sizes to run")
-    ap.add_argument("--metapel-only", default="", help="metapel workload: batches to run, for instance decode64,prefill1")
+                         "loop; prefix = shared-prefix requests on the Qwen2-7B shape through the engine loop; metapel, zulozen = "
+                         "prefill and decode of that design at a few sizes beside the Llama layout")
+    ap.add_argument("--layered-shapes", "--metapel-shapes", default="2048,4096", help="metapel and zulozen workloads: layer sizes to run")
+    ap.add_argument("--layered-only", "--metapel-only", default="",
+                    help="metapel and zulozen workloads: batches to run, for instance decode64,prefill1")
     ap.add_argument("--skip-cached-prefix", action="store_true",
                     help="engine workloads: start prefill after the tokens adopted from the prefix cache "
                          "(an extension; the reference shares the blocks but recomputes them)")

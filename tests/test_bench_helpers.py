@@ -51,7 +51,7 @@ def test_algorithmic_work_of_a_metapel_step(pkg):
                                pkg.LayerSpec("latent_attention", 0, **z)], 1e-5, 4)
     gru = 48 * 3 * 30 + 30 * 48 + 2 * 48 * 20
     att = 48 * (4 * 48 + 80 + 4 * 24) + 4 * 24 * 48
-    head = bench.METAPEL_VOCAB * 48
+    head = bench.LAYERED_VOCAB * 48
     w, fl, cache, attn = bench.metapel_work(meta, 2, [7, 300], [])
     assert w == 2 * (gru + att + head) and fl == 2 * 2 * (gru + att + head)
     assert cache == (7 + 10) * 80 * 2 and attn == (7 + 10) * 4 * 2 * (2 * 64 + 16)
@@ -59,3 +59,19 @@ def test_algorithmic_work_of_a_metapel_step(pkg):
     att += 4 * (32 + 24) * 64
     assert w == 2 * (gru + att + head) and fl == 2 * (12 * (gru + att) + head)
     assert cache == 0 and attn == (55 + 2 * 10) * 4 * 2 * (32 + 16 + 24)
+
+
+def test_algorithmic_work_of_a_zulozen_step(pkg):
+    att = dict(heads=4, kv_heads=2, dim=32, value_dim=24, chunk=10)
+    meta = pkg.LayeredMetadata("Zulozen", "m", 48, 100, [pkg.LayerSpec("attention", 20, **att),
+                               pkg.LayerSpec("attention", 12, experts=4, experts_per_token=1, shared_dim=8, **att)], 1e-5, block="sandwich")
+    mix = 48 * (4 * 32 + 2 * 56 + 4) + 4 * 24 * 48
+    dense, fixed, expert = 2 * 48 * 20, 4 * 48 + 3 * 48 * 8, 3 * 48 * 12
+    head = bench.LAYERED_VOCAB * 48
+    w, fl, cache, attn = bench.zulozen_work(meta, 1, [27], [])  # one row reaches one expert; 7 keys of its chunk
+    assert w == 2 * (2 * mix + dense + fixed + expert + head) == fl
+    assert cache == 2 * 7 * 2 * 56 * 2 and attn == 2 * 7 * 4 * 2 * 56
+    w, fl, cache, attn = bench.zulozen_work(meta, 12, [], [12])
+    assert w == 2 * (2 * mix + dense + fixed + head) + 2 * int(4 * (1 - 0.75 ** 12) * expert)
+    assert fl == 2 * (12 * (2 * mix + dense + fixed + expert) + head)
+    assert cache == 0 and attn == 2 * (55 + 3) * 4 * 2 * 56
