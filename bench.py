@@ -490,17 +490,17 @@ def run_layered(args):
                     tables = [list(range(s * n // BLOCK, (s + 1) * n // BLOCK)) for s in range(b)]
                     slots = list(range(b)) if model.num_state_slots() else None
                     ids = list(range(1, b + 1))
-                    prompt = rng.integers(0, LAYERED_VOCAB, n)
+                    text = rng.integers(0, LAYERED_VOCAB, (b, n))  # rows of their own: equal ones would share their experts
                     count = n if mode == "prefill" else n - 1
                     per = max(1, 8192 // n)
                     for s0 in range(0, b, per):  # real prompts: the decode steps go on from their state and cache
                         part = list(range(s0, min(b, s0 + per)))
-                        whole = pkg.ForwardBatch(np.tile(prompt[:count], len(part)), np.tile(np.arange(count), len(part)),
+                        whole = pkg.ForwardBatch(text[part, :count].ravel(), np.tile(np.arange(count), len(part)),
                                                  [ids[s] for s in part], [count] * len(part), [count] * len(part),
                                                  [tables[s] for s in part], state_slots=None if slots is None else part)
                         model.forward(whole)
                     if mode == "decode":
-                        model.forward(pkg.ForwardBatch(prompt[-1:].repeat(b), [n - 1] * b, ids, [1] * b, [n] * b, tables,
+                        model.forward(pkg.ForwardBatch(text[:, -1], [n - 1] * b, ids, [1] * b, [n] * b, tables,
                                                        has_prefill=False, state_slots=slots))
                     rows, contexts, prompts = (b, [n] * b, []) if mode == "decode" else (b * n, [], [n] * b)
                     steps = args.steps if mode == "decode" else max(3, args.steps // 5)

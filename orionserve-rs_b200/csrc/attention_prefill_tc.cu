@@ -213,11 +213,21 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
       tmem_ld_wait();
       const int key0 = (int)(block0 * kBlk + j * kKeys);
       float mx = -INFINITY;
+      // most key tiles are seen whole by every row of a warp (rows past the tile are not stored)
+      if (__all_sync(0xffffffffu, !valid || (key0 + kKeys - 1 <= pos && (!FORM || key0 >= low)))) {
+#pragma unroll
+        for (int i = 0; i < kKeys; ++i) {
+          const float v = __uint_as_float(sr[i >> 5][i & 31]) * sl2;
+          sr[i >> 5][i & 31] = __float_as_uint(v);
+          mx = fmaxf(mx, v);
+        }
+      } else {
 #pragma unroll
       for (int i = 0; i < kKeys; ++i) {
         const float v = (key0 + i <= pos && (!FORM || key0 + i >= low)) ? __uint_as_float(sr[i >> 5][i & 31]) * sl2 : -INFINITY;
         sr[i >> 5][i & 31] = __float_as_uint(v);
         mx = fmaxf(mx, v);
+      }
       }
       // The reference of the exponentials moves only when the maximum runs away from it.
       float corr = 1.0f;

@@ -77,9 +77,10 @@ __device__ __forceinline__ void store4<bf16>(bf16 *p, float4 v) {
 }
 
 // The same, four columns per thread and GROUPS rounds kept in registers, so each partial sum is read once: every size and
-// stride a multiple of four.
-template <typename T, int GROUPS>
-__global__ void __launch_bounds__(512)
+// stride a multiple of four. SLABS: the projection has at most that many (prompts; 0 = any number); gains and angles are then
+// read when they are needed, not while the projection is still running, which leaves registers for more rows per SM.
+template <typename T, int GROUPS, int SLABS>
+__global__ void __launch_bounds__(512, SLABS == 0 ? 1 : (SLABS == 1 && GROUPS <= 2 ? 3 : 2))
 attention_prepare_vec_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, AttnInputs in,
                              const uint32_t *__restrict__ positions, const uint32_t *__restrict__ slot_block,
                              const uint32_t *__restrict__ slot_slot, T *__restrict__ q_out, T *__restrict__ arena, KvLayout kv,
@@ -90,20 +91,24 @@ attention_prepare_vec_kernel(const float *__restrict__ partial, uint32_t splits,
   const float *p = partial + (size_t)row * in.ld;
   const uint32_t nq = in.q_heads * in.dim, nk = in.kv_heads * in.dim, nv = in.kv_heads * in.value_dim, all = nq + nk + nv;
   const uint32_t pos = positions[row], block = slot_block[row], slot = slot_slot[row];
-  float4 gain[GROUPS];
-  float2 co[GROUPS], si[GROUPS];
-#pragma unroll
-  for (int g = 0; g < GROUPS; ++g) {  // gains and angles do not depend on the projection
-    const uint32_t i = (tid + g * blockDim.x) * 4;
-    gain[g] = make_float4(1.f, 1.f, 1.f, 1.f), co[g] = make_float2(1.f, 1.f), si[g] = make_float2(0.f, 0.f);
-    if (i < nq + nk) {
-      if (in.q_norm) gain[g] = *reinterpret_cast<const float4 *>(i < nq ? in.q_norm + i : in.k_norm + (i - nq));
-      const uint32_t d = (i < nq ? i : i - nq) % in.dim;
-      if (d < in.rope_dims) {
-        co[g] = *reinterpret_cast<const float2 *>(in.rope_cos + (size_t)pos * half + d / 2);
-        si[g] = *reinterpret_cast<const float2 *>(in.rope_sin + (size_t)pos * half + d / 2);
-      }
+  // gain and angles of the four columns from i on
+  auto constants = [&](uint32_t i, float4 &gain, float2 &co, float2 &si) {
+    gain = make_float4(1.f, 1.f, 1.f, 1.f), co = make_float2(1.f, 1.f), si = make_float2(0.f, 0.f);
+    if (i >= nq + nk) return;
+    if (in.q_norm) gain = *reinterpret_cast<const float4 *>(i < nq ? in.q_norm + i : in.k_norm + (i - nq));
+    const uint32_t d = (i < nq ? i : i - nq) % in.dim;
+    if (d < in.rope_dims) {
+      co = *reinterpret_cast<const float2 *>(in.rope_cos + (size_t)pos * half + d / 2);
+      si = *reinterpret_cast<const float2 *>(in.rope_sin + (size_t)pos * half + d / 2);
     }
+  };
+  constexpr bool kLate = SLABS != 0;
+  constexpr int kEarly = kLate ? 1 : GROUPS;
+  float4 gain[kEarly];
+  float2 co[kEarly], si[kEarly];
+  if (!kLate) {
+#pragma unroll
+    for (int g = 0; g < kEarly; ++g) constants((tid + g * blockDim.x) * 4, gain[g], co[g], si[g]);
   }
   pdl_wait();
   float4 v[GROUPS];
@@ -113,7 +118,7 @@ attention_prepare_vec_kernel(const float *__restrict__ partial, uint32_t splits,
     const uint32_t i = (tid + g * blockDim.x) * 4;
     v[g] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (i >= all) continue;
-    v[g] = sum_slabs4(p + i, splits, split_stride);
+    v[g] = sum_slabs4_most<SLABS>(p + i, splits, split_stride);
     const float s = v[g].x * v[g].x + v[g].y * v[g].y + v[g].z * v[g].z + v[g].w * v[g].w;
     if (i < nq) sq += s;
     else if (i < nq + nk) sk += s;
@@ -128,9 +133,11 @@ attention_prepare_vec_kernel(const float *__restrict__ partial, uint32_t splits,
     if (i >= all) continue;
     float4 x = v[g];
     if (i < nq + nk) {
+      const int e = kLate ? 0 : g;
+      if (kLate) constants(i, gain[e], co[e], si[e]);
       const float s = i < nq ? scale_q : scale_k;
-      x = make_float4(x.x * s * gain[g].x, x.y * s * gain[g].y, x.z * s * gain[g].z, x.w * s * gain[g].w);
-      x = make_float4(x.x * co[g].x - x.y * si[g].x, x.y * co[g].x + x.x * si[g].x, x.z * co[g].y - x.w * si[g].y, x.w * co[g].y + x.z * si[g].y);
+      x = make_float4(x.x * s * gain[e].x, x.y * s * gain[e].y, x.z * s * gain[e].z, x.w * s * gain[e].w);
+      x = make_float4(x.x * co[e].x - x.y * si[e].x, x.y * co[e].x + x.x * si[e].x, x.z * co[e].y - x.w * si[e].y, x.w * co[e].y + x.z * si[e].y);
     }
     if (i < nq) {
       store4<T>(q_out + ((size_t)row * in.q_heads + i / in.dim) * kv.head_dim + i % in.dim, x);
@@ -159,11 +166,11 @@ inline int after_launch(const char *stage) {
   return ORION_OK;
 }
 
-template <typename T, int GROUPS>
+template <typename T, int GROUPS, int SLABS>
 int launch_vec(const float *partial, uint32_t splits, size_t split_stride, AttnInputs in, const uint32_t *positions, const uint32_t *slot_block,
                const uint32_t *slot_slot, T *q_out, T *arena, KvLayout kv, uint32_t layer, float *gate, uint32_t rows, uint32_t threads,
                cudaStream_t stream) {
-  ORION_CUDA_CHECK("attention_prepare", launch_pdl(attention_prepare_vec_kernel<T, GROUPS>, dim3(rows), dim3(threads), 0, stream, partial, splits,
+  ORION_CUDA_CHECK("attention_prepare", launch_pdl(attention_prepare_vec_kernel<T, GROUPS, SLABS>, dim3(rows), dim3(threads), 0, stream, partial, splits,
                                                    split_stride, in, positions, slot_block, slot_slot, q_out, arena, kv, layer, gate));
   return after_launch("attention_prepare");
 }
@@ -181,7 +188,12 @@ int launch_attention_prepare(const float *partial, uint32_t splits, size_t split
   const uint32_t threads = ((groups + rounds - 1) / rounds + 31) / 32 * 32;
   if (in.dim % 4 == 0 && in.value_dim % 4 == 0 && in.rope_dims % 4 == 0 && in.ld % 4 == 0 && split_stride % 4 == 0 && kv.head_dim % 4 == 0 &&
       kv.v_dim() % 4 == 0 && threads <= 512 && in.q_heads <= threads) {
-    auto run = rounds == 1 ? launch_vec<T, 1> : (rounds == 2 ? launch_vec<T, 2> : (rounds == 4 ? launch_vec<T, 4> : launch_vec<T, 8>));
+    const int slabs = slab_variant(rows, splits);
+    auto pick = [&](auto none, auto one, auto four) { return slabs == 1 ? one : (slabs == 4 ? four : none); };
+    auto run = rounds == 1   ? pick(launch_vec<T, 1, 0>, launch_vec<T, 1, 1>, launch_vec<T, 1, 4>)
+               : rounds == 2 ? pick(launch_vec<T, 2, 0>, launch_vec<T, 2, 1>, launch_vec<T, 2, 4>)
+               : rounds == 4 ? pick(launch_vec<T, 4, 0>, launch_vec<T, 4, 1>, launch_vec<T, 4, 4>)
+                             : launch_vec<T, 8, 0>;
     return run(partial, splits, split_stride, in, positions, slot_block, slot_slot, q_out, arena, kv, layer, gate, rows, threads, stream);
   }
   ORION_CUDA_CHECK("attention_prepare", launch_pdl(attention_prepare_kernel<T>, dim3(rows), dim3(256), 0, stream, partial, splits, split_stride, in,

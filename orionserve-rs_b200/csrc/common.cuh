@@ -178,6 +178,24 @@ __device__ __forceinline__ float4 sum_slabs4(const float *p, uint32_t n, size_t 
   return acc;
 }
 
+// The same for a number of slabs that is known to be at most MOST, in one batch; MOST = 0: any number.
+template <int MOST>
+__device__ __forceinline__ float4 sum_slabs4_most(const float *p, uint32_t n, size_t stride) {
+  if (MOST == 0) return sum_slabs4(p, n, stride);
+  float4 acc = *reinterpret_cast<const float4 *>(p);
+  if (MOST > 1) {
+    float4 x[MOST > 1 ? MOST - 1 : 1];
+#pragma unroll
+    for (int j = 1; j < MOST; ++j)
+      x[j - 1] = (uint32_t)j < n ? *reinterpret_cast<const float4 *>(p + (size_t)j * stride) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int j = 1; j < MOST; ++j) acc.x += x[j - 1].x, acc.y += x[j - 1].y, acc.z += x[j - 1].z, acc.w += x[j - 1].w;
+  }
+  return acc;
+}
+// Slab bound of a row-wise kernel's variant: prompts have few slabs and many rows, decode batches the reverse.
+inline int slab_variant(uint32_t rows, uint32_t slabs) { return slabs <= 1 ? 1 : (slabs <= 4 && rows > 256 ? 4 : 0); }
+
 // ---- PTX wrappers ------------------------------------------------------------
 
 __device__ __forceinline__ uint32_t smem_u32(const void *p) {

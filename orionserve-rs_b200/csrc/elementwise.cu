@@ -730,25 +730,29 @@ post_norm_residual_kernel(SublayerOutput y, float *__restrict__ hidden, const fl
   for (uint32_t c = threadIdx.x; c < H; c += blockDim.x) o[c] = from_f32<T>(row_cache[c] * s2 * pre_w[c]);
 }
 
-// Row widths that are multiples of 4: a row's values stay in registers between the two norms.
-template <typename T, int CHUNKS>
-__global__ void __launch_bounds__(512)
+// Row widths that are multiples of 4: a row's values stay in registers between the two norms. SLABS: every sum has
+// at most that many (prompts; 0 = any number); gains are then read when they are needed, which leaves registers for more rows
+// per SM.
+template <typename T, int CHUNKS, int SLABS>
+__global__ void __launch_bounds__(512, SLABS == 0 ? 1 : (SLABS == 1 && CHUNKS <= 2 ? 3 : 2))
 post_norm_residual_vec_kernel(SublayerOutput y, float *__restrict__ hidden, const float *__restrict__ post_w, float mult,
                               const float *__restrict__ pre_w, float eps, T *__restrict__ out, const uint32_t *__restrict__ row_map, uint32_t H) {
   using Acc = typename NormAcc<T>::type;
   __shared__ Acc red[32];
   pdl_trigger();
   const uint32_t nvec = H / 4;
-  float4 pw[CHUNKS], nw[CHUNKS], bv[CHUNKS];
+  constexpr bool kLate = SLABS != 0;
+  constexpr int kEarly = kLate ? 1 : CHUNKS;
+  float4 pw[kEarly], nw[kEarly];
+  if (!kLate) {
 #pragma unroll
-  for (int c = 0; c < CHUNKS; ++c) {  // immutable: fetched before the dependency wait
-    const uint32_t idx = threadIdx.x + c * blockDim.x;
-    pw[c] = nw[c] = bv[c] = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (idx < nvec) {
-      pw[c] = ld4(post_w + 4 * (size_t)idx), nw[c] = ld4(pre_w + 4 * (size_t)idx);
-      if (y.bias) bv[c] = ld4(y.bias + 4 * (size_t)idx);
+    for (int c = 0; c < kEarly; ++c) {  // immutable: fetched before the dependency wait
+      const uint32_t idx = threadIdx.x + c * blockDim.x;
+      pw[c] = nw[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (idx < nvec) pw[c] = ld4(post_w + 4 * (size_t)idx), nw[c] = ld4(pre_w + 4 * (size_t)idx);
     }
   }
+  auto slabs = [](const float *p, uint32_t n, size_t stride) { return sum_slabs4_most<SLABS>(p, n, stride); };
   pdl_wait();
   const uint32_t row = row_map ? row_map[blockIdx.x] : blockIdx.x;
   float *h = hidden + (size_t)row * H;
@@ -760,10 +764,10 @@ post_norm_residual_vec_kernel(SublayerOutput y, float *__restrict__ hidden, cons
     v[c] = x[c] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (idx >= nvec) continue;
     x[c] = ld4(h + 4 * (size_t)idx);
-    if (y.partial) v[c] = sum_slabs4(y.partial + (size_t)row * H + 4 * (size_t)idx, y.splits, y.split_stride);
-    v[c] = add4(v[c], bv[c]);
+    if (y.partial) v[c] = slabs(y.partial + (size_t)row * H + 4 * (size_t)idx, y.splits, y.split_stride);
+    if (y.bias) v[c] = add4(v[c], ld4(y.bias + 4 * (size_t)idx));
     for (uint32_t k = 0; k < y.top; ++k)
-      v[c] = add4(v[c], sum_slabs4(y.rows + (size_t)y.place[(size_t)row * y.top + k] * H + 4 * (size_t)idx, y.rows_splits, y.rows_stride));
+      v[c] = add4(v[c], slabs(y.rows + (size_t)y.place[(size_t)row * y.top + k] * H + 4 * (size_t)idx, y.rows_splits, y.rows_stride));
     ss += (Acc)v[c].x * (Acc)v[c].x + (Acc)v[c].y * (Acc)v[c].y + (Acc)v[c].z * (Acc)v[c].z + (Acc)v[c].w * (Acc)v[c].w;
   }
   const float s1 = norm_scale<Acc>(block_sum<Acc>(ss, red), H, eps);
@@ -772,8 +776,9 @@ post_norm_residual_vec_kernel(SublayerOutput y, float *__restrict__ hidden, cons
   for (int c = 0; c < CHUNKS; ++c) {
     const uint32_t idx = threadIdx.x + c * blockDim.x;
     if (idx >= nvec) continue;
-    x[c] = make_float4(x[c].x + mult * (v[c].x * s1 * pw[c].x), x[c].y + mult * (v[c].y * s1 * pw[c].y), x[c].z + mult * (v[c].z * s1 * pw[c].z),
-                       x[c].w + mult * (v[c].w * s1 * pw[c].w));
+    const float4 w = kLate ? ld4(post_w + 4 * (size_t)idx) : pw[kLate ? 0 : c];
+    x[c] = make_float4(x[c].x + mult * (v[c].x * s1 * w.x), x[c].y + mult * (v[c].y * s1 * w.y), x[c].z + mult * (v[c].z * s1 * w.z),
+                       x[c].w + mult * (v[c].w * s1 * w.w));
     if (!row_map) *reinterpret_cast<float4 *>(h + 4 * (size_t)idx) = x[c];
     ss += (Acc)x[c].x * (Acc)x[c].x + (Acc)x[c].y * (Acc)x[c].y + (Acc)x[c].z * (Acc)x[c].z + (Acc)x[c].w * (Acc)x[c].w;
   }
@@ -782,16 +787,17 @@ post_norm_residual_vec_kernel(SublayerOutput y, float *__restrict__ hidden, cons
 #pragma unroll
   for (int c = 0; c < CHUNKS; ++c) {
     const uint32_t idx = threadIdx.x + c * blockDim.x;
-    if (idx < nvec)
-      st4<T>(o + 4 * (size_t)idx, make_float4(x[c].x * s2 * nw[c].x, x[c].y * s2 * nw[c].y, x[c].z * s2 * nw[c].z, x[c].w * s2 * nw[c].w));
+    if (idx >= nvec) continue;
+    const float4 w = kLate ? ld4(pre_w + 4 * (size_t)idx) : nw[kLate ? 0 : c];
+    st4<T>(o + 4 * (size_t)idx, make_float4(x[c].x * s2 * w.x, x[c].y * s2 * w.y, x[c].z * s2 * w.z, x[c].w * s2 * w.w));
   }
 }
 
 namespace {
-template <typename T, int CHUNKS>
+template <typename T, int CHUNKS, int SLABS>
 int launch_post_norm_vec(SublayerOutput y, float *hidden, const float *post_w, float mult, const float *pre_w, float eps, T *out,
                          const uint32_t *row_map, uint32_t out_rows, uint32_t H, uint32_t threads, cudaStream_t stream) {
-  ORION_CUDA_CHECK("post_norm_residual", launch_pdl(post_norm_residual_vec_kernel<T, CHUNKS>, dim3(out_rows), dim3(threads), 0, stream, y, hidden,
+  ORION_CUDA_CHECK("post_norm_residual", launch_pdl(post_norm_residual_vec_kernel<T, CHUNKS, SLABS>, dim3(out_rows), dim3(threads), 0, stream, y, hidden,
                                                     post_w, mult, pre_w, eps, out, row_map, H));
   return after_launch("post_norm_residual");
 }
@@ -803,7 +809,12 @@ int launch_post_norm_residual(SublayerOutput y, float *hidden, const float *post
   if (out_rows == 0) return ORION_OK;
   if (H % 4 == 0 && H / 4 <= 2048 && y.split_stride % 4 == 0 && y.rows_stride % 4 == 0) {
     const uint32_t nvec = H / 4, threads = nvec >= 512 ? 512 : (nvec + 31) / 32 * 32, chunks = (nvec + threads - 1) / threads;
-    auto run = chunks == 1 ? launch_post_norm_vec<T, 1> : (chunks == 2 ? launch_post_norm_vec<T, 2> : launch_post_norm_vec<T, 4>);
+    const uint32_t a = y.partial ? y.splits : 1, b = y.top ? y.rows_splits : 1;
+    const int slabs = slab_variant(out_rows, a > b ? a : b);
+    auto pick = [&](auto none, auto one, auto four) { return slabs == 1 ? one : (slabs == 4 ? four : none); };
+    auto run = chunks == 1   ? pick(launch_post_norm_vec<T, 1, 0>, launch_post_norm_vec<T, 1, 1>, launch_post_norm_vec<T, 1, 4>)
+               : chunks == 2 ? pick(launch_post_norm_vec<T, 2, 0>, launch_post_norm_vec<T, 2, 1>, launch_post_norm_vec<T, 2, 4>)
+                             : pick(launch_post_norm_vec<T, 4, 0>, launch_post_norm_vec<T, 4, 1>, launch_post_norm_vec<T, 4, 4>);
     return run(y, hidden, post_w, mult, pre_w, eps, out, row_map, out_rows, H, threads, stream);
   }
   const size_t smem = (size_t)H * sizeof(float);

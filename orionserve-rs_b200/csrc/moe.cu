@@ -1,9 +1,10 @@
 // Mixture of experts: the choice of experts, the order of rows by expert, and the grouped products of the f32 build and of
 // sizes the tensor cores do not take (moe_gemm_tc.cu has the others).
 //   moe_choose_kernel  one warp per row: sigmoid scores of the router's logits, the `top` largest (the lower index of equal
-//                      ones), and a histogram per 64 rows
+//                      ones), and a histogram per block of rows
 //   moe_place_kernel   one warp per row: its places in the order by expert (rows of an expert keep their order, so the order
 //                      does not depend on timing), and the row copied there; the first CTA lists the tiles
+//   moe_route_kernel   both for up to 64 rows, in one cluster
 //   moe_simt_kernel    64 rows x 64 columns of one tile, k ascending, optionally with SwiGLU on the scored products
 //   moe_swiglu_kernel  the same activation on k-split products
 #include "kernels.h"
@@ -14,51 +15,64 @@
 namespace orion {
 namespace {
 
-constexpr uint32_t kRowBlock = 64;   // rows of one histogram
-constexpr uint32_t kChooseWarps = 8, kPlaceRows = 8;
+// Rows of one histogram: 8 (a warp each), or 64 in batches whose blocks would otherwise be many.
+__host__ __device__ inline uint32_t row_block(uint32_t rows) { return rows <= 512 ? 8 : 64; }
+constexpr uint32_t kPlaceRows = 8;
+constexpr uint32_t kClusterRows = 64;  // batches of up to this many rows: one kernel, a cluster of a CTA per 8 rows
 
-__global__ void __launch_bounds__(kChooseWarps * 32)
+// One warp: scores of one row in `mine`, its choices to chosen / score, counted in `count` (shared memory).
+__device__ __forceinline__ void choose_row(const float *__restrict__ logits, uint32_t splits, size_t split_stride, uint32_t experts, uint32_t top,
+                                           float *mine, uint32_t *chosen, float *score, uint32_t *count) {
+  const uint32_t lane = threadIdx.x & 31;
+  for (uint32_t e = lane; e < experts; e += 32) {
+    float z = 0.f;
+    for (uint32_t s0 = 0; s0 < splits; s0 += 8) {  // eight independent loads in flight
+      float x[8];
+#pragma unroll
+      for (uint32_t s = 0; s < 8; ++s) x[s] = s0 + s < splits ? logits[(s0 + s) * split_stride + e] : 0.f;
+#pragma unroll
+      for (uint32_t s = 0; s < 8; ++s) z += x[s];
+    }
+    mine[e] = sigmoid_f(z);
+  }
+  __syncwarp();
+  for (uint32_t k = 0; k < top; ++k) {
+    float best = -1.f;
+    uint32_t at = 0xFFFFFFFFu;
+    for (uint32_t e = lane; e < experts; e += 32)
+      if (mine[e] > best) best = mine[e], at = e;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+      const uint32_t oi = __shfl_xor_sync(0xffffffffu, at, o);
+      if (ov > best || (ov == best && oi < at)) best = ov, at = oi;
+    }
+    if (at >= experts) at = k;  // only if scores are not numbers: stay inside the expert list (top <= experts)
+    __syncwarp();
+    if (lane == 0) {
+      mine[at] = -2.f;
+      chosen[k] = at;
+      score[k] = best;
+      atomicAdd(&count[at], 1u);
+    }
+    __syncwarp();
+  }
+}
+
+__global__ void __launch_bounds__(1024)
 moe_choose_kernel(const float *__restrict__ logits, uint32_t splits, size_t split_stride, uint32_t experts, uint32_t top, uint32_t rows,
                   uint32_t *__restrict__ chosen, float *__restrict__ score, uint32_t *__restrict__ histogram) {
   extern __shared__ float smem[];  // [warps][experts] scores, [experts] counts
-  uint32_t *count = reinterpret_cast<uint32_t *>(smem + kChooseWarps * experts);
+  const uint32_t tid = threadIdx.x, warp = tid >> 5, warps = blockDim.x >> 5, block = row_block(rows);
+  uint32_t *count = reinterpret_cast<uint32_t *>(smem + warps * experts);
   pdl_trigger();
   pdl_wait();
-  const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  float *mine = smem + warp * experts;
   for (uint32_t e = tid; e < experts; e += blockDim.x) count[e] = 0;
   __syncthreads();
-  const uint32_t end = min(rows, (blockIdx.x + 1) * kRowBlock);
-  for (uint32_t row = blockIdx.x * kRowBlock + warp; row < end; row += kChooseWarps) {
-    for (uint32_t e = lane; e < experts; e += 32) {
-      const float *p = logits + (size_t)row * experts + e;
-      float z = p[0];
-      for (uint32_t s = 1; s < splits; ++s) z += p[s * split_stride];
-      mine[e] = sigmoid_f(z);
-    }
-    __syncwarp();
-    for (uint32_t k = 0; k < top; ++k) {
-      float best = -1.f;
-      uint32_t at = 0xFFFFFFFFu;
-      for (uint32_t e = lane; e < experts; e += 32)
-        if (mine[e] > best) best = mine[e], at = e;
-#pragma unroll
-      for (int o = 16; o > 0; o >>= 1) {
-        const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-        const uint32_t oi = __shfl_xor_sync(0xffffffffu, at, o);
-        if (ov > best || (ov == best && oi < at)) best = ov, at = oi;
-      }
-      if (at >= experts) at = k;  // only if scores are not numbers: stay inside the expert list (top <= experts)
-      __syncwarp();
-      if (lane == 0) {
-        mine[at] = -2.f;
-        chosen[(size_t)row * top + k] = at;
-        score[(size_t)row * top + k] = best;
-        atomicAdd(&count[at], 1u);
-      }
-      __syncwarp();
-    }
-  }
+  const uint32_t end = min(rows, (blockIdx.x + 1) * block);
+  for (uint32_t row = blockIdx.x * block + warp; row < end; row += warps)
+    choose_row(logits + (size_t)row * experts, splits, split_stride, experts, top, smem + warp * experts, chosen + (size_t)row * top,
+               score + (size_t)row * top, count);
   __syncthreads();
   for (uint32_t e = tid; e < experts; e += blockDim.x) histogram[(size_t)blockIdx.x * experts + e] = count[e];
 }
@@ -81,6 +95,29 @@ __device__ __forceinline__ void warp_prefix(const uint32_t *value, uint32_t n, u
   }
 }
 
+// The tile list from the rows of every expert (total), their first rows and their first tiles; by a whole CTA.
+__device__ __forceinline__ void list_tiles(const uint32_t *total, const uint32_t *first, const uint32_t *tile_at, uint32_t E, uint32_t tile_rows,
+                                           uint32_t max_tiles, MoeTile *tiles) {
+  for (uint32_t e = threadIdx.x; e < E; e += blockDim.x)
+    for (uint32_t t = 0; t * tile_rows < total[e]; ++t)
+      if (tile_at[e] + t < max_tiles) tiles[tile_at[e] + t] = MoeTile{e, first[e] + t * tile_rows, min(tile_rows, total[e] - t * tile_rows)};
+  const uint32_t used = tile_at[E - 1] + (total[E - 1] + tile_rows - 1) / tile_rows;
+  for (uint32_t t = used + threadIdx.x; t < max_tiles; t += blockDim.x) tiles[t] = MoeTile{0, 0, 0};
+}
+
+// Copies a row, by one warp.
+template <typename T>
+__device__ __forceinline__ void copy_row(const T *src, T *dst, uint32_t n) {
+  const uint32_t lane = threadIdx.x & 31;
+  constexpr uint32_t kVec = 16 / sizeof(T);
+  if (n % kVec == 0) {
+#pragma unroll 4
+    for (uint32_t c = lane; c < n / kVec; c += 32) reinterpret_cast<uint4 *>(dst)[c] = reinterpret_cast<const uint4 *>(src)[c];
+  } else {
+    for (uint32_t c = lane; c < n; c += 32) dst[c] = src[c];
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(kPlaceRows * 32)
 moe_place_kernel(const uint32_t *__restrict__ chosen, const float *__restrict__ score, const uint32_t *__restrict__ histogram,
@@ -90,10 +127,10 @@ moe_place_kernel(const uint32_t *__restrict__ chosen, const float *__restrict__ 
   uint32_t *total = words, *before = total + s.experts, *first = before + s.experts, *tile_at = first + s.experts;
   pdl_trigger();
   pdl_wait();
-  const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, E = s.experts, top = s.top;
+  const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, E = s.experts, top = s.top, per = row_block(rows);
   for (uint32_t e = tid; e < 2 * E; e += blockDim.x) total[e] = 0;  // and `before`
   __syncthreads();
-  const uint32_t row0 = blockIdx.x * kPlaceRows, block = row0 / kRowBlock, blocks = (rows + kRowBlock - 1) / kRowBlock;
+  const uint32_t row0 = blockIdx.x * kPlaceRows, block = row0 / per, blocks = (rows + per - 1) / per;
   for (uint32_t i = tid; i < blocks * E; i += blockDim.x) {
     const uint32_t v = histogram[i], e = i % E;
     if (v == 0) continue;
@@ -104,19 +141,13 @@ moe_place_kernel(const uint32_t *__restrict__ chosen, const float *__restrict__ 
   if (warp == 0) warp_prefix(total, E, first, [](uint32_t v) { return v; });
   if (warp == 1 && blockIdx.x == 0) warp_prefix(total, E, tile_at, [&](uint32_t v) { return (v + tile_rows - 1) / tile_rows; });
   __syncthreads();
-  if (blockIdx.x == 0) {
-    for (uint32_t e = tid; e < E; e += blockDim.x)
-      for (uint32_t t = 0; t * tile_rows < total[e]; ++t)
-        if (tile_at[e] + t < max_tiles) tiles[tile_at[e] + t] = MoeTile{e, first[e] + t * tile_rows, min(tile_rows, total[e] - t * tile_rows)};
-    const uint32_t used = tile_at[E - 1] + (total[E - 1] + tile_rows - 1) / tile_rows;
-    for (uint32_t t = used + tid; t < max_tiles; t += blockDim.x) tiles[t] = MoeTile{0, 0, 0};
-  }
+  if (blockIdx.x == 0) list_tiles(total, first, tile_at, E, tile_rows, max_tiles, tiles);
   const uint32_t row = row0 + warp;
   if (row >= rows) return;
   for (uint32_t k = 0; k < top; ++k) {
     const uint32_t at = row * top + k, e = chosen[at];
     uint32_t rank = 0;  // choices of the same expert before this one in the block of rows
-    for (uint32_t j = block * kRowBlock * top; j < at; j += 32) {
+    for (uint32_t j = block * per * top; j < at; j += 32) {
       const uint32_t other = j + lane < at ? chosen[j + lane] : 0xFFFFFFFFu;
       rank += __popc(__ballot_sync(0xffffffffu, other == e));
     }
@@ -125,15 +156,73 @@ moe_place_kernel(const uint32_t *__restrict__ chosen, const float *__restrict__ 
       place[at] = to;
       row_score[to] = score[at];
     }
-    const T *src = x + (size_t)row * s.hidden;
-    T *dst = sorted + (size_t)to * s.hidden;
-    constexpr uint32_t kVec = 16 / sizeof(T);
-    if (s.hidden % kVec == 0) {
-      for (uint32_t c = lane; c < s.hidden / kVec; c += 32) reinterpret_cast<uint4 *>(dst)[c] = reinterpret_cast<const uint4 *>(src)[c];
-    } else {
-      for (uint32_t c = lane; c < s.hidden; c += 32) dst[c] = src[c];
+    copy_row(x + (size_t)row * s.hidden, sorted + (size_t)to * s.hidden, s.hidden);
+  }
+}
+
+__device__ __forceinline__ uint32_t ld_dsmem_u32(const uint32_t *local, uint32_t rank) {
+  uint32_t addr, v;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(addr) : "r"(smem_u32(local)), "r"(rank));
+  asm volatile("ld.shared::cluster.u32 %0, [%1];" : "=r"(v) : "r"(addr) : "memory");
+  return v;
+}
+
+// Few rows: both steps in one kernel. The CTAs of the one cluster take eight rows each and read each other's counts through
+// distributed shared memory.
+template <typename T>
+__global__ void __launch_bounds__(kPlaceRows * 32)
+moe_route_kernel(const float *__restrict__ logits, uint32_t splits, size_t split_stride, const T *__restrict__ x, MoeShape s, uint32_t rows,
+                 uint32_t tile_rows, uint32_t max_tiles, uint32_t *__restrict__ place, float *__restrict__ row_score, MoeTile *__restrict__ tiles,
+                 T *__restrict__ sorted) {
+  extern __shared__ float smem[];  // [8][experts] scores, then words
+  const uint32_t E = s.experts, top = s.top, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  uint32_t *count = reinterpret_cast<uint32_t *>(smem + kPlaceRows * E), *total = count + E, *before = total + E, *first = before + E,
+           *tile_at = first + E, *chosen = tile_at + E;
+  float *score = reinterpret_cast<float *>(chosen + kPlaceRows * top);
+  pdl_trigger();
+  for (uint32_t e = tid; e < E; e += blockDim.x) count[e] = 0;
+  __syncthreads();
+  pdl_wait();
+  const uint32_t row = blockIdx.x * kPlaceRows + warp;
+  if (row < rows)
+    choose_row(logits + (size_t)row * E, splits, split_stride, E, top, smem + warp * E, chosen + warp * top, score + warp * top, count);
+  __syncthreads();
+  asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+  asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+  for (uint32_t e = tid; e < E; e += blockDim.x) {
+    uint32_t all = 0, lower = 0;
+    for (uint32_t r = 0; r < gridDim.x; ++r) {
+      const uint32_t v = ld_dsmem_u32(count + e, r);
+      all += v;
+      if (r < blockIdx.x) lower += v;
+    }
+    total[e] = all, before[e] = lower;
+  }
+  __syncwarp();
+  asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");  // nobody leaves while its counts may still be read
+  __syncthreads();
+  if (warp == 0) warp_prefix(total, E, first, [](uint32_t v) { return v; });
+  if (warp == 1) warp_prefix(total, E, tile_at, [&](uint32_t v) { return (v + tile_rows - 1) / tile_rows; });
+  __syncthreads();
+  if (blockIdx.x == 0) list_tiles(total, first, tile_at, E, tile_rows, max_tiles, tiles);
+  if (row < rows) {
+    for (uint32_t k = 0; k < top; ++k) {
+      const uint32_t at = warp * top + k, e = chosen[at];
+      uint32_t rank = 0;
+      for (uint32_t j = 0; j < at; j += 32) {
+        const uint32_t other = j + lane < at ? chosen[j + lane] : 0xFFFFFFFFu;
+        rank += __popc(__ballot_sync(0xffffffffu, other == e));
+      }
+      const uint32_t to = first[e] + before[e] + rank;
+      if (lane == 0) {
+        place[row * top + k] = to;
+        row_score[to] = score[at];
+      }
+      copy_row(x + (size_t)row * s.hidden, sorted + (size_t)to * s.hidden, s.hidden);
     }
   }
+  __syncwarp();
+  asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
 }
 
 // silu(w g) * (w u): the score of a routed row multiplies what the expert reads.
@@ -230,7 +319,10 @@ inline int after_launch(const char *stage) {
 
 }  // namespace
 
-size_t moe_histogram_words(MoeShape s, uint32_t rows) { return (size_t)((rows + kRowBlock - 1) / kRowBlock) * s.experts; }
+size_t moe_histogram_words(MoeShape s, uint32_t rows) {
+  const uint32_t most = std::max((rows + 63) / 64, (std::min(rows, 512u) + 7) / 8);
+  return (size_t)most * s.experts;
+}
 
 MoePlan moe_plan(bool is_bf16, MoeShape s, uint32_t rows) {
   MoePlan p{BM, 0, 1, 1, is_bf16 && moe_tc_supported(s)};
@@ -266,8 +358,20 @@ int launch_moe_route(const float *logits, uint32_t splits, size_t split_stride, 
   if (rows == 0) return ORION_OK;
   if (s.experts == 0 || s.experts > kMoeMaxExperts || s.top == 0 || s.top > s.experts)
     return set_error(ORION_ERR_INTERNAL, "routing of %u among %u experts is not supported (at most %u)", s.top, s.experts, kMoeMaxExperts);
-  ORION_CUDA_CHECK("moe_choose", launch_pdl(moe_choose_kernel, dim3((rows + kRowBlock - 1) / kRowBlock), dim3(kChooseWarps * 32),
-                                            (kChooseWarps + 1) * s.experts * sizeof(float), stream, logits, splits, split_stride, s.experts, s.top,
+  if (rows <= kClusterRows) {
+    const uint32_t ctas = (rows + kPlaceRows - 1) / kPlaceRows;
+    const size_t smem = ((kPlaceRows + 5) * (size_t)s.experts + 2 * kPlaceRows * s.top) * 4;
+    static bool attr_set[kMaxDeviceOrdinals] = {};
+    ORION_CUDA_CHECK("moe_route attr", ensure_dynamic_smem(moe_route_kernel<T>, ((kPlaceRows + 5) + 2 * kPlaceRows) * kMoeMaxExperts * 4, attr_set));
+    ORION_CUDA_CHECK("moe_route", launch_pdl_cluster(moe_route_kernel<T>, dim3(ctas), dim3(kPlaceRows * 32), dim3(ctas), smem, stream, logits, splits,
+                                                     split_stride, x, s, rows, plan.tile_rows, plan.tiles, b.place, b.row_score, b.tiles, b.x));
+    return after_launch("moe_route");
+  }
+  const uint32_t block = row_block(rows), threads = block == 8 ? 256 : 1024;
+  static bool attr_set[kMaxDeviceOrdinals] = {};
+  ORION_CUDA_CHECK("moe_choose attr", ensure_dynamic_smem(moe_choose_kernel, 33 * kMoeMaxExperts * (int)sizeof(float), attr_set));
+  ORION_CUDA_CHECK("moe_choose", launch_pdl(moe_choose_kernel, dim3((rows + block - 1) / block), dim3(threads),
+                                            (threads / 32 + 1) * s.experts * sizeof(float), stream, logits, splits, split_stride, s.experts, s.top,
                                             rows, b.chosen, b.score, b.histogram));
   ORION_TRY(after_launch("moe_choose"));
   ORION_CUDA_CHECK("moe_place", launch_pdl(moe_place_kernel<T>, dim3((rows + kPlaceRows - 1) / kPlaceRows), dim3(kPlaceRows * 32),

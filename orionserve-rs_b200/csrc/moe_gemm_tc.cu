@@ -54,6 +54,9 @@ moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
            *acc_ready = empty_x + XST;
   uint32_t *tmem_slot = reinterpret_cast<uint32_t *>(acc_ready + 1);
   const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const bool shared = blockIdx.y < a.shared_tiles;
+  const uint32_t n = shared ? a.shared_n : a.n, k = shared ? a.shared_k : a.k, n0 = blockIdx.x * (MT * kTileN), split = blockIdx.z;
+  if (n0 >= n) return;  // the grid is as wide as the wider of the two products
   if (threadIdx.x == 0) {
     for (int s = 0; s < WST; ++s) mbar_init(&full_w[s], 1), mbar_init(&empty_w[s], 1);
     for (int s = 0; s < XST; ++s) mbar_init(&full_x[s], 1), mbar_init(&empty_x[s], 1);
@@ -71,7 +74,6 @@ moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
   pdl_trigger();
   const uint32_t tmem_base = *tmem_slot;
 
-  const bool shared = blockIdx.y < a.shared_tiles;
   MoeTile tile;
   if (shared) {
     tile = MoeTile{0, blockIdx.y * TOKN, min((uint32_t)TOKN, a.rows - blockIdx.y * TOKN)};
@@ -79,8 +81,7 @@ moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
     pdl_wait();
     tile = a.tiles[blockIdx.y - a.shared_tiles];
   }
-  const uint32_t n = shared ? a.shared_n : a.n, k = shared ? a.shared_k : a.k, n0 = blockIdx.x * (MT * kTileN), split = blockIdx.z;
-  const bool live = tile.count > 0 && n0 < n;
+  const bool live = tile.count > 0;
   const uint32_t nkb = (k + kSlabK - 1) / kSlabK;
   const uint32_t kb_begin = split * nkb / a.splits, my_kb = live ? (split + 1) * nkb / a.splits - kb_begin : 0;
   const CUtensorMap *mw = shared ? &map_sw : &map_w, *mx = shared ? &map_sx : &map_x;
