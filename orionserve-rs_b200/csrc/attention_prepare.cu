@@ -80,7 +80,7 @@ __device__ __forceinline__ void store4<bf16>(bf16 *p, float4 v) {
 // stride a multiple of four. SLABS: the projection has at most that many (prompts; 0 = any number); gains and angles are then
 // read when they are needed, not while the projection is still running, which leaves registers for more rows per SM.
 template <typename T, int GROUPS, int SLABS>
-__global__ void __launch_bounds__(512, SLABS == 0 ? 1 : (SLABS == 1 && GROUPS <= 2 ? 3 : 2))
+__global__ void __launch_bounds__(512, SLABS == 0 ? 1 : (SLABS == 1 ? 3 : 2))
 attention_prepare_vec_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, AttnInputs in,
                              const uint32_t *__restrict__ positions, const uint32_t *__restrict__ slot_block,
                              const uint32_t *__restrict__ slot_slot, T *__restrict__ q_out, T *__restrict__ arena, KvLayout kv,
