@@ -223,11 +223,11 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         }
       } else {
 #pragma unroll
-      for (int i = 0; i < kKeys; ++i) {
-        const float v = (key0 + i <= pos && (!FORM || key0 + i >= low)) ? __uint_as_float(sr[i >> 5][i & 31]) * sl2 : -INFINITY;
-        sr[i >> 5][i & 31] = __float_as_uint(v);
-        mx = fmaxf(mx, v);
-      }
+        for (int i = 0; i < kKeys; ++i) {
+          const float v = (key0 + i <= pos && (!FORM || key0 + i >= low)) ? __uint_as_float(sr[i >> 5][i & 31]) * sl2 : -INFINITY;
+          sr[i >> 5][i & 31] = __float_as_uint(v);
+          mx = fmaxf(mx, v);
+        }
       }
       // The reference of the exponentials moves only when the maximum runs away from it.
       float corr = 1.0f;
