@@ -130,9 +130,12 @@ void orion_cuda_model_destroy(OrionModel *model);
  * Sandwich: x += m RMSNorm(mixer(RMSNorm(x))), then x += m RMSNorm(ffn(RMSNorm(x))), m = residual_mult.
  * The logits are the final norm's output times the embedding table or an output matrix of their own.
  * Metapel is a design with parallel blocks, Zulozen one with sandwich blocks. */
-enum { ORION_MIXER_MIN_GRU = 0, ORION_MIXER_LATENT_ATTENTION = 1, ORION_MIXER_ATTENTION = 2 };
-enum { ORION_BLOCK_PARALLEL = 0, ORION_BLOCK_SANDWICH = 1 };
-enum { ORION_ACT_GELU_TANH = 0, ORION_ACT_RELU2 = 1 };
+enum { ORION_MIXER_MIN_GRU = 0, ORION_MIXER_LATENT_ATTENTION = 1, ORION_MIXER_ATTENTION = 2, ORION_MIXER_GLA = 3 };
+enum { ORION_BLOCK_PARALLEL = 0, ORION_BLOCK_SANDWICH = 1, ORION_BLOCK_PRENORM = 2 };
+enum { ORION_ACT_GELU_TANH = 0, ORION_ACT_RELU2 = 1, ORION_ACT_GEGLU_TANH = 2 };
+enum { ORION_QK_NORM_NONE = 0, ORION_QK_NORM_ALL_HEADS = 1, ORION_QK_NORM_PER_HEAD = 2 };
+enum { ORION_ROUTER_SIGMOID_INPUT = 0, ORION_ROUTER_SOFTMAX = 1 };
+enum { ORION_EXPERT_SWIGLU = 0, ORION_EXPERT_CLAMPED = 1 };
 typedef struct OrionLayerDesc {
   uint32_t mixer;    /* ORION_MIXER_* */
   uint32_t ffn_dim;  /* width of the feed-forward, or of each of its experts; 0 = the layer has none */
@@ -144,17 +147,35 @@ typedef struct OrionLayerDesc {
   uint32_t heads, dim, rot_dim, value_dim, kv_rank, window, rope_dims;
   double rope_base, scale;
   /* attention: key/value heads (each shared by heads / kv_heads query heads); chunk size (a position sees
-   * those before it in its own chunk, chunks counted from position 0; 0 = no chunks); whether queries and
-   * keys are normalised (RMS over all heads at once, before the rotation), whether every head has a
-   * learned logit in its softmax denominator, and whether a sigmoid per head gates its output */
+   * those before it in its own chunk, chunks counted from position 0; 0 = no chunks); how queries and
+   * keys are normalised before the rotation (ORION_QK_NORM_*: RMS over all heads at once, or per head with
+   * gains that the heads share), whether every head has a learned logit in its softmax denominator, and
+   * whether a sigmoid per head gates its output */
   uint32_t kv_heads, chunk, qk_norm, sinks, head_gate;
-  /* dense feed-forward (experts = 0): ORION_ACT_*, and whether both projections have biases (sandwich
-   * blocks only) */
+  /* dense feed-forward (experts = 0): ORION_ACT_* (the gated one in prenorm blocks only), and whether both
+   * projections have biases (sandwich blocks only) */
   uint32_t activation, ffn_bias;
-  /* mixture of experts (sandwich blocks only): SwiGLU experts, of which every token uses experts_per_token,
-   * chosen and weighted (at their input) by the sigmoid of the router's logits; width of an expert that
-   * every token uses (0 = none) */
+  /* mixture of experts (not in parallel blocks): gated experts, of which every token uses experts_per_token,
+   * chosen and weighted as ORION_ROUTER_* says; width of an expert that every token uses (0 = none) */
   uint32_t experts, experts_per_token, shared_dim;
+  /* attention: the first keep_first positions are seen besides the window; dimension i rotates with
+   * i + rope_dims / 2 (else with its neighbour); q, k and v have biases; every value of the output has a
+   * sigmoid gate of its own. With ORION_QK_NORM_PER_HEAD only: rope_halves, qkv_bias, value_gate.
+   * Scores become softcap * tanh(score / softcap) (0 = they stay). yarn_factor > 0: frequencies are
+   * stretched by that factor, those of fewer than yarn_slow turns within yarn_original positions wholly,
+   * those of more than yarn_fast not at all */
+  uint32_t keep_first, rope_halves, qkv_bias, value_gate;
+  double softcap, yarn_factor, yarn_original, yarn_fast, yarn_slow;
+  /* gla: heads, dim and value_dim as above; decays are formed through decay_rank values and raised to
+   * 1 / decay_tau */
+  double decay_tau;
+  uint32_t decay_rank;
+  /* router: ORION_ROUTER_SIGMOID_INPUT (sigmoid of the logits, the score multiplies the expert's input) or
+   * ORION_ROUTER_SOFTMAX (over all outputs; the score multiplies the expert's output; a correction per output
+   * takes part in the choice only); outputs past the experts whose expert returns its input. Experts:
+   * ORION_EXPERT_*, with the limits of the clamped form */
+  uint32_t router, router_identity, expert_form;
+  double expert_limit, shared_limit;
 } OrionLayerDesc;
 typedef struct OrionLayeredDesc {
   uint32_t hidden_size, vocab_size, num_layers;
@@ -168,7 +189,13 @@ typedef struct OrionLayeredDesc {
   uint32_t max_batch_tokens, max_batch_sequences;
   uint32_t block;                   /* ORION_BLOCK_* */
   uint32_t untied_lm_head;          /* the logits have a matrix of their own */
-  double residual_mult;             /* sandwich blocks */
+  double residual_mult;             /* sandwich and prenorm blocks */
+  double embed_scale;               /* of the embedding's rows as they enter the first layer */
+  double logit_softcap;             /* logits become cap * tanh(logit / cap); 0 = they stay */
+  /* layers loop_start .. loop_stop - 1 run loop_times times in a row (0 = no loop), each pass with a cache and
+   * state of its own; ahead of a pass the rows of `loop.step` join the stream, and from the second pass on
+   * what entered the first layer of the model. Prenorm blocks only */
+  uint32_t loop_start, loop_stop, loop_times;
 } OrionLayeredDesc;
 int orion_cuda_model_create_layered(OrionBackend *backend, const OrionLayeredDesc *desc, OrionModel **out);
 /* State slots of the model: 0 for models that carry nothing but the KV cache from step to step. */
@@ -192,7 +219,7 @@ int orion_cuda_selftest_peer_wait(OrionBackend *backend, uint64_t limit_us, uint
 
 /* Reads and clears the time-out words of the backend's device (no reference counterpart): bit 0 the
  * projection GEMM, bit 1 decode attention, bit 2 prefill attention, bit 3 the tensor-parallel
- * hand-over, bit 4 the grouped products of a mixture of experts. A set bit means a bounded
+ * hand-over, bit 4 the grouped products of a mixture of experts, bit 5 gated linear attention. A set bit means a bounded
  * device-side wait of that kernel family gave up since the last read. orion_cuda_model_forward reads the words itself after every step; a caller that launches
  * kernels through the stand-alone entry points (orion_cuda_paged_decode_attention_noalloc) and wants
  * to know whether one of its launches timed out synchronises its stream and calls this. */

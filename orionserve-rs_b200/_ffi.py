@@ -42,7 +42,10 @@ class OrionLayerDesc(C.Structure):
     _fields_ = [(n, C.c_uint32) for n in ("mixer", "ffn_dim", "width", "heads", "dim", "rot_dim", "value_dim", "kv_rank",
                                           "window", "rope_dims")] + [("rope_base", C.c_double), ("scale", C.c_double)] + \
                [(n, C.c_uint32) for n in ("kv_heads", "chunk", "qk_norm", "sinks", "head_gate", "activation", "ffn_bias", "experts",
-                                          "experts_per_token", "shared_dim")]
+                                          "experts_per_token", "shared_dim", "keep_first", "rope_halves", "qkv_bias", "value_gate")] + \
+               [(n, C.c_double) for n in ("softcap", "yarn_factor", "yarn_original", "yarn_fast", "yarn_slow", "decay_tau")] + \
+               [(n, C.c_uint32) for n in ("decay_rank", "router", "router_identity", "expert_form")] + \
+               [(n, C.c_double) for n in ("expert_limit", "shared_limit")]
 
 
 class OrionLayeredDesc(C.Structure):
@@ -51,12 +54,16 @@ class OrionLayeredDesc(C.Structure):
                 ("max_position_embeddings", C.c_uint32), ("num_blocks", C.c_uint32), ("block_size", C.c_uint32),
                 ("num_state_slots", C.c_uint32), ("compute_dtype", C.c_uint32), ("max_batch_tokens", C.c_uint32),
                 ("max_batch_sequences", C.c_uint32), ("block", C.c_uint32), ("untied_lm_head", C.c_uint32),
-                ("residual_mult", C.c_double)]
+                ("residual_mult", C.c_double), ("embed_scale", C.c_double), ("logit_softcap", C.c_double),
+                ("loop_start", C.c_uint32), ("loop_stop", C.c_uint32), ("loop_times", C.c_uint32)]
 
 
-MIXER_MIN_GRU, MIXER_LATENT_ATTENTION, MIXER_ATTENTION = 0, 1, 2
-BLOCK_PARALLEL, BLOCK_SANDWICH = 0, 1
-ACT_GELU_TANH, ACT_RELU2 = 0, 1
+MIXER_MIN_GRU, MIXER_LATENT_ATTENTION, MIXER_ATTENTION, MIXER_GLA = 0, 1, 2, 3
+BLOCK_PARALLEL, BLOCK_SANDWICH, BLOCK_PRENORM = 0, 1, 2
+ACT_GELU_TANH, ACT_RELU2, ACT_GEGLU_TANH = 0, 1, 2
+QK_NORM_NONE, QK_NORM_ALL_HEADS, QK_NORM_PER_HEAD = 0, 1, 2
+ROUTER_SIGMOID_INPUT, ROUTER_SOFTMAX = 0, 1
+EXPERT_SWIGLU, EXPERT_CLAMPED = 0, 1
 
 _lib = None
 

@@ -60,18 +60,21 @@ paged_attention_generic_kernel(const T *__restrict__ q, const T *__restrict__ ar
 
   float m = form.sinks ? form.sinks[head] : -INFINITY, l = form.sinks ? 1.0f : 0.0f;
   float acc[kGenMaxDimsPerThread] = {0.f, 0.f, 0.f, 0.f};
-  const uint32_t attend = qpos + 1;  // attention.rs:253: positions 0..=query_position
+  // positions 0..=query_position (attention.rs:253), or the first `kept` ones and those from `first` on
+  const uint32_t first = form.range.first(qpos), kept = form.range.kept(qpos), visible = kept + qpos + 1 - first;
+  auto position = [&](uint32_t i) { return i < kept ? i : first - kept + i; };
 
-  for (uint32_t c0 = form.range.first(qpos); c0 < attend; c0 += kGenChunk) {
-    const uint32_t n = min((uint32_t)kGenChunk, attend - c0);
+  for (uint32_t c0 = 0; c0 < visible; c0 += kGenChunk) {
+    const uint32_t n = min((uint32_t)kGenChunk, visible - c0);
     float cmax = -INFINITY;
     for (uint32_t p = threadIdx.x; p < n; p += blockDim.x) {
-      const uint32_t pos = c0 + p, slot = pos % B;
+      const uint32_t pos = position(c0 + p), slot = pos % B;
       const T *k = arena + kv.row(layer, table[pos / B], kvh, 0, slot);
       float dot = 0.0f;  // attention.rs:270-273: sequential, unfused
       for (uint32_t d = 0; d < hd; ++d)
         dot = __fadd_rn(dot, __fmul_rn(q_s[d], to_f32<T>(k[kv.col(slot, d)])));
-      const float s = __fmul_rn(dot, scale);
+      float s = __fmul_rn(dot, scale);
+      if (form.softcap != 0.f) s = softcap_f(s, form.softcap);
       scores[p] = s;
       cmax = fmaxf(cmax, s);
     }
@@ -107,7 +110,7 @@ paged_attention_generic_kernel(const T *__restrict__ q, const T *__restrict__ ar
       for (uint32_t p = 0; p < n; ++p) {
         const float w = scores[p];
         if (w == 0.0f) continue;  // attention.rs:283-285
-        const uint32_t pos = c0 + p, slot = pos % B;
+        const uint32_t pos = position(c0 + p), slot = pos % B;
         const T *v = arena + kv.row(layer, table[pos / B], kvh, 1, slot);
         a = __fadd_rn(a, __fmul_rn(w, to_f32<T>(v[kv.col(slot, d)])));
       }
@@ -122,6 +125,7 @@ paged_attention_generic_kernel(const T *__restrict__ q, const T *__restrict__ ar
     if (d >= vd) break;
     float v = l > 0.0f ? acc[j] / l : acc[j];
     if (form.gate) v *= form.gate[(size_t)row * q_heads + head];
+    if (form.value_gate) v *= to_f32<T>(static_cast<const T *>(form.value_gate)[((size_t)row * q_heads + head) * vd + d]);
     out[(size_t)row * (form.ldo ? form.ldo : q_heads * vd) + (size_t)head * vd + d] = from_f32<T>(v);
   }
 }
@@ -162,6 +166,7 @@ __device__ __forceinline__ void store_head_value(const AttnForm &form, uint32_t 
   const uint32_t n = form.out_dim ? form.out_dim : padded;
   if (d >= n) return;
   if (form.gate) v *= form.gate[(size_t)row * q_heads + head];
+  if (form.value_gate) v *= __bfloat162float(static_cast<const bf16 *>(form.value_gate)[((size_t)row * q_heads + head) * n + d]);
   out[(size_t)row * (form.ldo ? form.ldo : q_heads * n) + (size_t)head * n + d] = __float2bfloat16_rn(v);
 }
 
@@ -193,6 +198,9 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
   const uint32_t *table = batch.tables_flat + batch.table_offsets[seq];
   const uint32_t first_key = FORM ? form.range.first(ctx - 1) : 0, block0 = first_key / kBlk;
   const uint32_t nblocks = (ctx + kBlk - 1) / kBlk;
+  // The row reads `kept_blk` blocks from the sequence's start, then those from block0 on: index i -> logical block.
+  const uint32_t kept_blk = FORM ? form.range.kept_blocks(block0, kBlk) : 0, count = kept_blk + nblocks - block0;
+  auto logical = [&](uint32_t i) { return !FORM || i < kept_blk ? i : block0 - kept_blk + i; };
   // blocks from this one on hold rows of this step
   const uint32_t fresh_block = FORM && form.first_row ? batch.query_positions[form.first_row[seq]] / kBlk : nblocks - 1;
   // Context split: a contiguous range of blocks; warps interleave inside it.
@@ -202,9 +210,9 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
   const uint32_t bps = FORM ? 0 : scratch.blocks_per_split;
   const uint32_t my_splits = bps ? min(max((nblocks + bps / 2) / bps, 1u), splits) : splits;
   if (split >= my_splits) return;
-  const uint32_t per_split = (nblocks - block0 + my_splits - 1) / my_splits;
-  const uint32_t b_begin = min(block0 + split * per_split, nblocks);
-  const uint32_t b_end = min(b_begin + per_split, nblocks);
+  const uint32_t per_split = (count + my_splits - 1) / my_splits;
+  const uint32_t b_begin = min(split * per_split, count);
+  const uint32_t b_end = min(b_begin + per_split, count);
 
   pdl_trigger();
   if (threadIdx.x < kWarps * kStages) mbar_init(&bars[threadIdx.x], 1);
@@ -214,14 +222,14 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
   uint8_t *my_ring = ring + warp * kStages * kChunkBytes;
   uint64_t *my_bars = bars + warp * kStages;
   const size_t layer_base = (size_t)layer * kv.layer_elems();
-  // Block i of this warp (i = 0, 1, ...) is logical block b_begin + warp + i*kWarps.
+  // Block i of this warp (i = 0, 1, ...) is logical(b_begin + warp + i*kWarps).
   const uint32_t my_count = (b_end > b_begin + warp) ? (b_end - b_begin - warp + kWarps - 1) / kWarps : 0;
 
   // Block-table entries are prefetched 32 at a time into one register per lane
   // (two groups in flight) so that issuing a copy never waits on a global load.
   auto load_group = [&](uint32_t g) -> uint32_t {
     const uint32_t idx = g * 32 + lane;
-    return idx < my_count ? table[b_begin + warp + idx * kWarps] : 0u;
+    return idx < my_count ? table[logical(b_begin + warp + idx * kWarps)] : 0u;
   };
   uint32_t tgroup = 0, tbl_a = load_group(0), tbl_b = load_group(1);
   auto entry = [&](uint32_t i) -> uint32_t {  // warp-uniform i, called by all lanes
@@ -240,7 +248,7 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
   uint32_t deferred = pre;  // the blocks of a warp ascend
   for (uint32_t i = 0; i < pre; ++i) {
     const uint32_t pb = entry(i);
-    if (b_begin + warp + i * kWarps >= fresh_block) {
+    if (logical(b_begin + warp + i * kWarps) >= fresh_block) {
       deferred = i;
       break;
     }
@@ -306,7 +314,12 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
 
   // Online softmax state for the two heads this lane sees in the C fragment
   // (columns 2*(lane%4) and +1), in the log2 domain.
-  const float sl2 = FORM && form.scale != 0.f ? form.scale * 1.4426950408889634f : 1.4426950408889634f / sqrtf((float)DK);
+  float sl2 = FORM && form.scale != 0.f ? form.scale * 1.4426950408889634f : 1.4426950408889634f / sqrtf((float)DK);
+  float cap_in = 0.f, cap_out = 0.f;
+  if (FORM && form.softcap != 0.f) {  // the cap leaves scores in the log2 domain
+    cap_out = form.softcap * 1.4426950408889634f, cap_in = 2.f * sl2 / form.softcap;
+    sl2 = 1.f;
+  }
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
   if (FORM && form.sinks && split == 0 && warp == 0) {  // one of the partial results starts with the sink
     const uint32_t g0 = (lane & 3) * 2;
@@ -334,7 +347,7 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
     }
     const uint32_t kbase = smem_u32(my_ring + stage * kChunkBytes);
     const uint32_t vbase = kbase + kBlk * DK * 2;
-    const uint32_t lb = b_begin + warp + i * kWarps;
+    const uint32_t lb = logical(b_begin + warp + i * kWarps);
     const uint32_t valid = min((uint32_t)kBlk, ctx - lb * kBlk);  // tokens of this block in context
     if (!FORM && fq.partial != nullptr && lb == nblocks - 1) {
       // The block that holds this step's token: its k and v rows come from the stash. Lanes 0-15
@@ -364,7 +377,12 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
     }
     // scale into the log2 domain and mask slots beyond the context
     const uint32_t hidden = FORM && first_key > lb * kBlk ? first_key - lb * kBlk : 0;  // tokens of this block before the first key
-    const bool see_lo = t_lo < valid && (!FORM || t_lo >= hidden), see_hi = t_hi < valid && (!FORM || t_hi >= hidden);
+    const uint32_t kept = FORM && form.range.keep > lb * kBlk ? form.range.keep - lb * kBlk : 0;  // but those of it are seen
+    const bool see_lo = t_lo < valid && (!FORM || t_lo >= hidden || t_lo < kept), see_hi = t_hi < valid && (!FORM || t_hi >= hidden || t_hi < kept);
+    if (FORM && form.softcap != 0.f) {
+#pragma unroll
+      for (int k = 0; k < 4; ++k) s[k] = softcap_log2(s[k], cap_in, cap_out);
+    }
     s[0] = see_lo ? s[0] * sl2 : -INFINITY;
     s[1] = see_lo ? s[1] * sl2 : -INFINITY;
     s[2] = see_hi ? s[2] * sl2 : -INFINITY;

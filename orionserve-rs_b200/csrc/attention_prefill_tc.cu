@@ -85,7 +85,10 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
   const uint32_t nblocks = tile.max_position / kBlk + 1;
   // key tiles start at the block of the first key that the tile's first row sees
   const uint32_t block0 = FORM ? form.range.first(batch.query_positions[tile.row_start]) / kBlk : 0;
-  const uint32_t ntiles = (nblocks - block0 + (kKeys / kBlk) - 1) / (kKeys / kBlk);
+  // before them come the blocks of the positions that every row keeps: index i -> logical block
+  const uint32_t kept_blk = FORM ? form.range.kept_blocks(block0, kBlk) : 0;
+  auto logical = [&](uint32_t i) { return !FORM || i < kept_blk ? i : block0 - kept_blk + i; };
+  const uint32_t ntiles = (kept_blk + nblocks - block0 + (kKeys / kBlk) - 1) / (kKeys / kBlk);
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < kStages; ++s) {
@@ -134,7 +137,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
 #pragma unroll
         for (uint32_t b = 0; b < kKeys / kBlk; ++b) {
           // a block past the row's context repeats the first one: its keys are masked, its values must be finite
-          const uint32_t lb = block0 + j * (kKeys / kBlk) + b;
+          const uint32_t lb = FORM ? logical(j * (kKeys / kBlk) + b) : j * (kKeys / kBlk) + b;
           const uint32_t block = table[lb < nblocks ? lb : block0];
           const int chunk = (int)((chunk0 + block) * kv.num_kv_heads + kvh);
 #pragma unroll
@@ -200,7 +203,13 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     softmax_bar();
     if (threadIdx.x == 64) mbar_arrive(q_ready);
 
-    const float sl2 = FORM && form.scale != 0.f ? form.scale * 1.4426950408889634f : 1.4426950408889634f / sqrtf((float)DK);
+    float sl2 = FORM && form.scale != 0.f ? form.scale * 1.4426950408889634f : 1.4426950408889634f / sqrtf((float)DK);
+    const int keep = FORM ? (int)form.range.keep : 0;
+    float cap_in = 0.f, cap_out = 0.f;
+    if (FORM && form.softcap != 0.f) {  // the cap leaves scores in the log2 domain
+      cap_out = form.softcap * 1.4426950408889634f, cap_in = 2.f * sl2 / form.softcap;
+      sl2 = 1.f;
+    }
     float ref = -INFINITY, l = 0.f;
     if (FORM && form.sinks) ref = form.sinks[head] * 1.4426950408889634f, l = 1.f;
     for (uint32_t j = 0; j < ntiles; ++j) {
@@ -211,10 +220,15 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
       tmem_ld32(taddr, sr[0]);
       tmem_ld32(taddr + 32, sr[1]);
       tmem_ld_wait();
-      const int key0 = (int)(block0 * kBlk + j * kKeys);
+      const bool straight = !FORM || j * (kKeys / kBlk) >= kept_blk || kept_blk == block0;  // the tile's keys follow one another
+      const int key0 = (int)((FORM ? logical(j * (kKeys / kBlk)) : j * (kKeys / kBlk)) * kBlk);
       float mx = -INFINITY;
+      if (FORM && form.softcap != 0.f) {
+#pragma unroll
+        for (int i = 0; i < kKeys; ++i) sr[i >> 5][i & 31] = __float_as_uint(softcap_log2(__uint_as_float(sr[i >> 5][i & 31]), cap_in, cap_out));
+      }
       // most key tiles are seen whole by every row of a warp (rows past the tile are not stored)
-      if (__all_sync(0xffffffffu, !valid || (key0 + kKeys - 1 <= pos && (!FORM || key0 >= low)))) {
+      if (straight && __all_sync(0xffffffffu, !valid || (key0 + kKeys - 1 <= pos && (!FORM || key0 >= low)))) {
 #pragma unroll
         for (int i = 0; i < kKeys; ++i) {
           const float v = __uint_as_float(sr[i >> 5][i & 31]) * sl2;
@@ -222,9 +236,13 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
           mx = fmaxf(mx, v);
         }
       } else {
+        int from[kKeys / kBlk];  // first key of every block
+#pragma unroll
+        for (int b = 0; b < kKeys / kBlk; ++b) from[b] = straight ? key0 + b * kBlk : (int)(logical(j * (kKeys / kBlk) + b) * kBlk);
 #pragma unroll
         for (int i = 0; i < kKeys; ++i) {
-          const float v = (key0 + i <= pos && (!FORM || key0 + i >= low)) ? __uint_as_float(sr[i >> 5][i & 31]) * sl2 : -INFINITY;
+          const int key = from[i / kBlk] + i % kBlk;
+          const float v = (key <= pos && (!FORM || key >= low || key < keep)) ? __uint_as_float(sr[i >> 5][i & 31]) * sl2 : -INFINITY;
           sr[i >> 5][i & 31] = __float_as_uint(v);
           mx = fmaxf(mx, v);
         }
@@ -277,11 +295,29 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     const uint32_t od = FORM && form.out_dim ? form.out_dim : DV, ldo = FORM && form.ldo ? form.ldo : q_heads * od;
     const bool whole_groups = !FORM || (od % 8 == 0 && ldo % 8 == 0);
     bf16 *dst = out + (size_t)row * ldo + (size_t)head * od;
+    const bf16 *vgate = FORM && form.value_gate ? static_cast<const bf16 *>(form.value_gate) + ((size_t)row * q_heads + head) * od : nullptr;
 #pragma unroll 1
     for (uint32_t c = 0; c < DV; c += 32) {
       uint32_t orow[32];
       tmem_ld32(taddr + kTmemO + c, orow);
       tmem_ld_wait();
+      if (FORM && vgate && valid) {
+#pragma unroll
+        for (int i = 0; i < 32; i += 8) {
+          if (c + i >= od) continue;
+          if (whole_groups) {
+            const uint4 g = *reinterpret_cast<const uint4 *>(vgate + c + i);
+            const uint32_t w[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+            for (int k = 0; k < 8; ++k)  // the bits of a bf16 are the upper half of the f32
+              orow[i + k] = __float_as_uint(__uint_as_float(orow[i + k]) * __uint_as_float(k & 1 ? w[k / 2] & 0xFFFF0000u : w[k / 2] << 16));
+          } else {
+#pragma unroll
+            for (int k = 0; k < 8; ++k)
+              if (c + i + k < od) orow[i + k] = __float_as_uint(__uint_as_float(orow[i + k]) * __bfloat162float(vgate[c + i + k]));
+          }
+        }
+      }
       if (valid) {
 #pragma unroll
         for (int i = 0; i < 32; i += 8) {

@@ -1,6 +1,6 @@
-// What attention with per-projection query / key norms, rotation in neighbouring pairs and per-head output gates needs
-// between its joint projection and the attention kernels: one pass over the projection's partial sums that normalises,
-// rotates, and leaves queries, cached keys and values, and gates. One CTA per row.
+// What attention with query / key norms, rotation of part of each head and output gates needs between its joint projection
+// and the attention kernels: one pass over the projection's partial sums that normalises, rotates, and leaves queries, cached
+// keys and values, and gates. One CTA per row where a norm spans all heads, one warp per row and head where it does not.
 #include "kernels.h"
 #include "mma.cuh"
 
@@ -148,6 +148,91 @@ attention_prepare_vec_kernel(const float *__restrict__ partial, uint32_t splits,
   }
 }
 
+constexpr uint32_t kHeadWarps = 8;
+
+template <int VEC>
+__device__ __forceinline__ void load_folded(const float *p, uint32_t splits, size_t stride, float (&v)[VEC]) {
+  if (VEC == 4) {
+    const float4 x = sum_slabs4(p, splits, stride);
+    v[0] = x.x, v[1 % VEC] = x.y, v[2 % VEC] = x.z, v[3 % VEC] = x.w;
+  } else {
+    v[0] = fold(p, splits, stride);
+  }
+}
+template <typename T, int VEC>
+__device__ __forceinline__ void store_values(T *p, const float (&v)[VEC]) {
+  if (VEC == 4) store4<T>(p, make_float4(v[0], v[1 % VEC], v[2 % VEC], v[3 % VEC]));
+  else p[0] = from_f32<T>(v[0]);
+}
+
+// A warp per (row, head of q, k, v or the gate). VEC columns per lane and round: 4 where sizes, strides and rotated halves are multiples
+// of 4. A head that rotates passes through shared memory, since its pairs may be any distance apart.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(kHeadWarps * 32)
+attention_prepare_heads_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, AttnInputs in,
+                               const uint32_t *__restrict__ positions, const uint32_t *__restrict__ slot_block,
+                               const uint32_t *__restrict__ slot_slot, T *__restrict__ q_out, T *__restrict__ arena, KvLayout kv, uint32_t layer,
+                               T *__restrict__ value_gate) {
+  extern __shared__ __align__(16) float head_values[];  // [kHeadWarps][dim]
+  pdl_trigger();
+  const uint32_t row = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, half = in.rope_dims / 2;
+  const uint32_t nq = in.q_heads * in.dim, nk = in.kv_heads * in.dim, nv = in.kv_heads * in.value_dim;
+  const uint32_t pos = positions[row], block = slot_block[row], slot = slot_slot[row];
+  const float *cs = in.rope_cos + (size_t)pos * half, *sn = in.rope_sin + (size_t)pos * half;
+  const uint32_t first_v = in.q_heads + in.kv_heads, first_gate = first_v + in.kv_heads, heads = first_gate + (value_gate ? in.q_heads : 0);
+  float *buf = head_values + warp * in.dim;
+  pdl_wait();
+  for (uint32_t t = blockIdx.y * kHeadWarps + warp; t < heads; t += gridDim.y * kHeadWarps) {
+    if (t >= first_v) {  // values and gates pass straight through
+      const bool is_gate = t >= first_gate;
+      const uint32_t head = is_gate ? t - first_gate : t - first_v, at = nq + nk + (is_gate ? nv : 0) + head * in.value_dim;
+      T *dst = is_gate ? value_gate + ((size_t)row * in.q_heads + head) * in.value_dim : arena + kv.row(layer, block, head, 1, slot);
+      for (uint32_t d = lane * VEC; d < in.value_dim; d += 32 * VEC) {
+        float v[VEC];
+        load_folded<VEC>(partial + (size_t)row * in.ld + at + d, splits, split_stride, v);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[i] = is_gate ? sigmoid_for<T>(v[i]) : v[i] + (in.bias ? in.bias[at + d + i] : 0.f);
+        store_values<T, VEC>(dst + (is_gate ? d : kv.col(slot, d)), v);
+      }
+      continue;
+    }
+    const bool is_q = t < in.q_heads;
+    const uint32_t head = is_q ? t : t - in.q_heads, at = is_q ? head * in.dim : nq + head * in.dim;
+    const float *gain = is_q ? in.q_norm : in.k_norm;
+    float ss = 0.f;
+    for (uint32_t d = lane * VEC; d < in.dim; d += 32 * VEC) {
+      float v[VEC];
+      load_folded<VEC>(partial + (size_t)row * in.ld + at + d, splits, split_stride, v);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) {
+        if (in.bias) v[i] += in.bias[at + d + i];
+        ss += v[i] * v[i];
+        if (gain) v[i] *= gain[d + i];
+      }
+      store_values<float, VEC>(buf + d, v);
+    }
+    const float scale = gain ? 1.0f / sqrtf(warp_sum(ss) / (float)in.dim + in.eps) : 1.f;
+    __syncwarp();
+    T *dst = is_q ? q_out + ((size_t)row * in.q_heads + head) * kv.head_dim : arena + kv.row(layer, block, head, 0, slot);
+    for (uint32_t d = lane * VEC; d < in.dim; d += 32 * VEC) {
+      float v[VEC];
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) {
+        const uint32_t c = d + i;
+        v[i] = buf[c];
+        if (c < 2 * half) {
+          const uint32_t pair = in.halves ? (c < half ? c : c - half) : c >> 1, other = in.halves ? (c < half ? c + half : c - half) : c ^ 1u;
+          const bool second = in.halves ? c >= half : c & 1u;
+          v[i] = second ? v[i] * cs[pair] + buf[other] * sn[pair] : v[i] * cs[pair] - buf[other] * sn[pair];
+        }
+        v[i] *= scale;
+      }
+      store_values<T, VEC>(dst + (is_q ? d : kv.col(slot, d)), v);
+    }
+    __syncwarp();
+  }
+}
+
 template <typename T>
 __global__ void arena_rows_kernel(const T *__restrict__ arena, KvLayout kv, uint32_t dim, uint32_t value_dim, float *__restrict__ out) {
   const size_t tokens = (size_t)kv.num_blocks * kv.num_kv_heads * kv.block_size, keys = tokens * dim, all = keys + tokens * value_dim;
@@ -180,8 +265,23 @@ int launch_vec(const float *partial, uint32_t splits, size_t split_stride, AttnI
 template <typename T>
 int launch_attention_prepare(const float *partial, uint32_t splits, size_t split_stride, AttnInputs in, const uint32_t *positions,
                              const uint32_t *slot_block, const uint32_t *slot_slot, T *q_out, T *arena, KvLayout kv, uint32_t layer,
-                             float *gate, uint32_t rows, cudaStream_t stream) {
+                             float *gate, uint32_t rows, cudaStream_t stream, T *value_gate) {
   if (rows == 0) return ORION_OK;
+  if (in.per_head) {
+    if (gate) return set_error(ORION_ERR_INTERNAL, "a gate per head is not built for this layout");
+    const bool vec = in.dim % 4 == 0 && in.value_dim % 4 == 0 && in.rope_dims % 4 == 0 && in.ld % 4 == 0 && split_stride % 4 == 0 &&
+                     kv.head_dim % 4 == 0 && kv.v_dim() % 4 == 0;
+    const uint32_t heads = 2 * in.kv_heads + in.q_heads * (value_gate ? 2 : 1), most = (heads + kHeadWarps - 1) / kHeadWarps;
+    // decode batches: a warp per head; prompts: a CTA per row
+    const uint32_t split = rows >= 1024 ? 1 : (most < 1024 / rows + 1 ? most : 1024 / rows + 1);
+    const size_t smem = (size_t)kHeadWarps * in.dim * sizeof(float);
+    if (smem > 48 * 1024) return set_error(ORION_ERR_INTERNAL, "query and key heads of %u values are not supported", in.dim);
+    ORION_CUDA_CHECK("attention_prepare", launch_pdl(vec ? attention_prepare_heads_kernel<T, 4> : attention_prepare_heads_kernel<T, 1>, dim3(rows, split),
+                                                     dim3(kHeadWarps * 32), smem, stream, partial, splits, split_stride, in, positions, slot_block,
+                                                     slot_slot, q_out, arena, kv, layer, value_gate));
+    return after_launch("attention_prepare");
+  }
+  if (in.halves || in.bias || value_gate) return set_error(ORION_ERR_INTERNAL, "rotated halves, biases and gates per value come with norms per head");
   if ((in.q_norm == nullptr) != (in.k_norm == nullptr)) return set_error(ORION_ERR_INTERNAL, "query and key norms come together");
   const uint32_t groups = (in.q_heads * in.dim + in.kv_heads * (in.dim + in.value_dim)) / 4;
   const uint32_t rounds = groups <= 256 ? 1 : (groups <= 1024 ? 2 : (groups <= 2048 ? 4 : 8));
@@ -209,7 +309,7 @@ int launch_arena_rows(const T *arena, KvLayout kv, uint32_t dim, uint32_t value_
 
 #define ORION_INSTANTIATE(T)                                                                                                            \
   template int launch_attention_prepare<T>(const float *, uint32_t, size_t, AttnInputs, const uint32_t *, const uint32_t *, const uint32_t *, \
-                                           T *, T *, KvLayout, uint32_t, float *, uint32_t, cudaStream_t);                              \
+                                           T *, T *, KvLayout, uint32_t, float *, uint32_t, cudaStream_t, T *);                         \
   template int launch_arena_rows<T>(const T *, KvLayout, uint32_t, uint32_t, float *, cudaStream_t);
 ORION_INSTANTIATE(float)
 ORION_INSTANTIATE(bf16)

@@ -550,13 +550,14 @@ int orion_cuda_poll_wait_timeouts(OrionBackend *backend, uint32_t *mask) {
   orion::clear_error();
   ORION_TRY(orion::check_backend(backend));
   if (!mask) return orion::set_error(ORION_ERR_INVALID_REQUEST, "null output pointer");
-  uint32_t gemm = 0, decode = 0, prefill = 0, tp = 0, experts = 0;
+  uint32_t gemm = 0, decode = 0, prefill = 0, tp = 0, experts = 0, linear = 0;
   ORION_TRY(orion::gemm_tc_poll_error(&gemm));
   ORION_TRY(orion::decode_poll_error(&decode));
   ORION_TRY(orion::prefill_poll_error(&prefill));
   ORION_TRY(orion::tp_poll_error(&tp));
   ORION_TRY(orion::moe_poll_error(&experts));
-  *mask = (gemm ? 1u : 0u) | (decode ? 2u : 0u) | (prefill ? 4u : 0u) | (tp ? 8u : 0u) | (experts ? 16u : 0u);
+  ORION_TRY(orion::gla_poll_error(&linear));
+  *mask = (gemm ? 1u : 0u) | (decode ? 2u : 0u) | (prefill ? 4u : 0u) | (tp ? 8u : 0u) | (experts ? 16u : 0u) | (linear ? 32u : 0u);
   return ORION_OK;
 }
 

@@ -141,6 +141,30 @@ __device__ __forceinline__ float relu2(float x) {
 template <typename T>
 __device__ __forceinline__ float silu_for(float x) { return x * sigmoid_for<T>(x); }
 
+// Gated feed-forwards, f(gate) * up: SwiGLU, GELU (tanh form), or a clamped form with both inputs limited,
+// g sigmoid(1.702 g) (u + 1) with g at most and |u| at most `limit`.
+enum GatedKind : uint32_t { kGatedSilu = 0, kGatedGelu = 1, kGatedClamped = 2 };
+struct GatedAct {
+  GatedKind kind = kGatedSilu;
+  float limit = 0.f;
+};
+template <typename T>
+__device__ __forceinline__ float gated(GatedAct f, float g, float u) {
+  if (f.kind == kGatedSilu) return silu_for<T>(g) * u;
+  if (f.kind == kGatedGelu) return gelu_tanh<T>(g) * u;
+  g = fminf(g, f.limit);
+  return g * sigmoid_for<T>(1.702f * g) * (fminf(fmaxf(u, -f.limit), f.limit) + 1.f);
+}
+
+__device__ __forceinline__ float softcap_f(float x, float cap) { return cap * tanhf(x / cap); }
+// out * tanh(y), 2 y log2(e) = x * in, as out - 2 out / (1 + 2^(x in)): one exponential and one reciprocal. The error is a few roundings
+// of `out`, whatever the size of the result.
+__device__ __forceinline__ float softcap_log2(float x, float in, float out) {
+  float e;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(fminf(x * in, 100.f)));
+  return out - __fdividef(2.f * out, 1.f + e);
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

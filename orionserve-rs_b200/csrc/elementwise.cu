@@ -54,7 +54,7 @@ template <typename T>
 __global__ void __launch_bounds__(kNormThreads)
 embed_rmsnorm_kernel(const T *__restrict__ embed, const uint32_t *__restrict__ tokens,
                      const float *__restrict__ w, float eps, float *__restrict__ hidden,
-                     T *__restrict__ normed, uint32_t H) {
+                     T *__restrict__ normed, uint32_t H, float factor, const float *__restrict__ shift) {
   using Acc = typename NormAcc<T>::type;
   __shared__ Acc red[32];
   pdl_trigger();
@@ -64,7 +64,8 @@ embed_rmsnorm_kernel(const T *__restrict__ embed, const uint32_t *__restrict__ t
   float *h = hidden + (size_t)row * H;
   Acc ss = Acc(0);
   for (uint32_t c = threadIdx.x; c < H; c += blockDim.x) {
-    const float v = to_f32<T>(src[c]);
+    float v = to_f32<T>(src[c]) * factor;
+    if (shift) v += shift[c];
     h[c] = v;
     ss += (Acc)v * (Acc)v;
   }
@@ -524,11 +525,11 @@ inline int after_launch(const char *stage) {
 template <typename T>
 int launch_embed_rmsnorm(const T *embed, const uint32_t *tokens, const float *norm_w, float eps,
                          float *hidden, T *normed, uint32_t rows, uint32_t hidden_size,
-                         cudaStream_t stream) {
+                         cudaStream_t stream, float scale, const float *shift) {
   if (rows == 0) return ORION_OK;
   ORION_CUDA_CHECK("embed_rmsnorm", launch_pdl(embed_rmsnorm_kernel<T>, dim3(rows), dim3(kNormThreads), 0,
                                                stream, embed, tokens, norm_w, eps, hidden, normed,
-                                               hidden_size));
+                                               hidden_size, scale, shift));
   return after_launch("embed_rmsnorm");
 }
 
@@ -635,6 +636,47 @@ int launch_swiglu(const float *partial, uint32_t splits, size_t split_stride, T 
   return after_launch("swiglu");
 }
 
+// Gated activations over [rows][2 * ffn] partials with gate f and up f in columns 2f and 2f + 1.
+template <typename T>
+__global__ void __launch_bounds__(256)
+gated_act_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, GatedAct f, T *__restrict__ act, uint32_t ldo,
+                 uint32_t rows, uint32_t ffn) {
+  pdl_trigger();
+  pdl_wait();
+  const size_t total = (size_t)rows * ffn;
+  for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
+    const float *p = partial + 2 * idx;
+    float g = p[0], u = p[1];
+    for (uint32_t s = 1; s < splits; ++s) g += p[s * split_stride], u += p[s * split_stride + 1];
+    act[idx / ffn * ldo + idx % ffn] = from_f32<T>(gated<T>(f, g, u));
+  }
+}
+// Four outputs per thread: ffn, ldo and split_stride multiples of 4.
+template <typename T>
+__global__ void __launch_bounds__(256)
+gated_act_vec_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, GatedAct f, T *__restrict__ act, uint32_t ldo,
+                     uint32_t rows, uint32_t ffn) {
+  pdl_trigger();
+  pdl_wait();
+  const uint32_t fv = ffn / 4;
+  const size_t total = (size_t)rows * fv;
+  for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
+    const float *p = partial + 8 * idx;
+    const float4 a = sum_slabs4(p, splits, split_stride), b = sum_slabs4(p + 4, splits, split_stride);
+    st4<T>(act + idx / fv * ldo + idx % fv * 4, make_float4(gated<T>(f, a.x, a.y), gated<T>(f, a.z, a.w), gated<T>(f, b.x, b.y), gated<T>(f, b.z, b.w)));
+  }
+}
+template <typename T>
+int launch_gated_act(const float *partial, uint32_t splits, size_t split_stride, GatedAct f, T *act, uint32_t ldo, uint32_t rows, uint32_t ffn,
+                     cudaStream_t stream) {
+  if (rows == 0 || ffn == 0) return ORION_OK;
+  const bool vec = ffn % 4 == 0 && ldo % 4 == 0 && split_stride % 4 == 0;
+  const size_t n = (size_t)rows * ffn / (vec ? 4 : 1);
+  ORION_CUDA_CHECK("gated_act", launch_pdl(vec ? gated_act_vec_kernel<T> : gated_act_kernel<T>, dim3(grid_for(n, 256)), dim3(256), 0, stream, partial,
+                                           splits, split_stride, f, act, ldo, rows, ffn));
+  return after_launch("gated_act");
+}
+
 // Activation of a dense feed-forward.
 template <typename T>
 __device__ __forceinline__ float ffn_activation(FfnAct f, float v) {
@@ -685,25 +727,40 @@ int launch_ffn_act(const float *partial, uint32_t splits, size_t split_stride, c
   return after_launch("ffn_act");
 }
 
-// ---- a sublayer whose output is normalised before it joins the residual stream -----------------------------
+// ---- a sublayer's output joins the residual stream, normalised before that or as it is -------------------
 
 // Value c of a sublayer's output for one row.
+template <typename T>
 __device__ __forceinline__ float sublayer_value(const SublayerOutput &y, uint32_t row, uint32_t H, uint32_t c) {
   float v = 0.f;
   if (y.partial)
     for (uint32_t s = 0; s < y.splits; ++s) v += y.partial[s * y.split_stride + (size_t)row * H + c];
   if (y.bias) v += y.bias[c];
   for (uint32_t k = 0; k < y.top; ++k) {
-    const float *p = y.rows + (size_t)y.place[(size_t)row * y.top + k] * H + c;
-    for (uint32_t s = 0; s < y.rows_splits; ++s) v += p[s * y.rows_stride];
+    const uint32_t at = y.place[(size_t)row * y.top + k];
+    float x = 0.f;
+    if (at == kNoPlace) {
+      x = to_f32<T>(static_cast<const T *>(y.identity)[(size_t)row * H + c]);
+    } else {
+      const float *p = y.rows + (size_t)at * H + c;
+      for (uint32_t s = 0; s < y.rows_splits; ++s) x += p[s * y.rows_stride];
+    }
+    v += y.weight ? y.weight[(size_t)row * y.top + k] * x : x;
   }
   return v;
 }
 
+// What joins the stream after the sublayer, value c of one row.
+template <typename T>
+__device__ __forceinline__ float added_value(const StreamAddition<T> &a, uint32_t row, uint32_t H, uint32_t c) {
+  float v = a.embed ? a.scale * to_f32<T>(a.embed[(size_t)a.tokens[row] * H + c]) : 0.f;
+  return a.shift ? v + a.shift[c] : v;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(kNormThreads)
-post_norm_residual_kernel(SublayerOutput y, float *__restrict__ hidden, const float *__restrict__ post_w, float mult,
-                          const float *__restrict__ pre_w, float eps, T *__restrict__ out, const uint32_t *__restrict__ row_map, uint32_t H) {
+post_norm_residual_kernel(SublayerOutput y, float *__restrict__ hidden, const float *__restrict__ post_w, float mult, StreamAddition<T> add,
+                          const float *__restrict__ pre_w, float eps, T *out, const uint32_t *__restrict__ row_map, uint32_t H) {
   using Acc = typename NormAcc<T>::type;
   __shared__ Acc red[32];
   extern __shared__ float row_cache[];  // H floats
@@ -713,14 +770,14 @@ post_norm_residual_kernel(SublayerOutput y, float *__restrict__ hidden, const fl
   float *h = hidden + (size_t)row * H;
   Acc ss = Acc(0);
   for (uint32_t c = threadIdx.x; c < H; c += blockDim.x) {
-    const float v = sublayer_value(y, row, H, c);
+    const float v = sublayer_value<T>(y, row, H, c);
     row_cache[c] = v;
     ss += (Acc)v * (Acc)v;
   }
-  const float s1 = norm_scale<Acc>(block_sum<Acc>(ss, red), H, eps);
+  const float s1 = post_w ? norm_scale<Acc>(block_sum<Acc>(ss, red), H, eps) : 1.f;
   ss = Acc(0);
   for (uint32_t c = threadIdx.x; c < H; c += blockDim.x) {
-    const float v = h[c] + mult * (row_cache[c] * s1 * post_w[c]);
+    const float v = h[c] + mult * (post_w ? row_cache[c] * s1 * post_w[c] : row_cache[c]) + added_value<T>(add, row, H, c);
     if (!row_map) h[c] = v;
     row_cache[c] = v;
     ss += (Acc)v * (Acc)v;
@@ -733,10 +790,23 @@ post_norm_residual_kernel(SublayerOutput y, float *__restrict__ hidden, const fl
 // Row widths that are multiples of 4: a row's values stay in registers between the two norms. SLABS: every sum has
 // at most that many (prompts; 0 = any number); gains are then read when they are needed, which leaves registers for more rows
 // per SM.
-template <typename T, int CHUNKS, int SLABS>
+// POST: the output is normalised; otherwise it joins as it is, with the experts' weights, the identity experts and what `add` names.
+template <typename T>
+__device__ __forceinline__ float4 load4(const T *p);
+template <>
+__device__ __forceinline__ float4 load4<float>(const float *p) { return ld4(p); }
+template <>
+__device__ __forceinline__ float4 load4<bf16>(const bf16 *p) {
+  const uint2 v = *reinterpret_cast<const uint2 *>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&v.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&v.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ float4 axpy4(float a, float4 x, float4 y) { return make_float4(a * x.x + y.x, a * x.y + y.y, a * x.z + y.z, a * x.w + y.w); }
+
+template <typename T, int CHUNKS, int SLABS, bool POST>
 __global__ void __launch_bounds__(512, SLABS == 0 ? 1 : (SLABS == 1 && CHUNKS <= 2 ? 3 : 2))
-post_norm_residual_vec_kernel(SublayerOutput y, float *__restrict__ hidden, const float *__restrict__ post_w, float mult,
-                              const float *__restrict__ pre_w, float eps, T *__restrict__ out, const uint32_t *__restrict__ row_map, uint32_t H) {
+post_norm_residual_vec_kernel(SublayerOutput y, float *__restrict__ hidden, const float *__restrict__ post_w, float mult, StreamAddition<T> add,
+                              const float *__restrict__ pre_w, float eps, T *out, const uint32_t *__restrict__ row_map, uint32_t H) {
   using Acc = typename NormAcc<T>::type;
   __shared__ Acc red[32];
   pdl_trigger();
@@ -749,7 +819,10 @@ post_norm_residual_vec_kernel(SublayerOutput y, float *__restrict__ hidden, cons
     for (int c = 0; c < kEarly; ++c) {  // immutable: fetched before the dependency wait
       const uint32_t idx = threadIdx.x + c * blockDim.x;
       pw[c] = nw[c] = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (idx < nvec) pw[c] = ld4(post_w + 4 * (size_t)idx), nw[c] = ld4(pre_w + 4 * (size_t)idx);
+      if (idx < nvec) {
+        if (POST) pw[c] = ld4(post_w + 4 * (size_t)idx);
+        nw[c] = ld4(pre_w + 4 * (size_t)idx);
+      }
     }
   }
   auto slabs = [](const float *p, uint32_t n, size_t stride) { return sum_slabs4_most<SLABS>(p, n, stride); };
@@ -766,19 +839,33 @@ post_norm_residual_vec_kernel(SublayerOutput y, float *__restrict__ hidden, cons
     x[c] = ld4(h + 4 * (size_t)idx);
     if (y.partial) v[c] = slabs(y.partial + (size_t)row * H + 4 * (size_t)idx, y.splits, y.split_stride);
     if (y.bias) v[c] = add4(v[c], ld4(y.bias + 4 * (size_t)idx));
-    for (uint32_t k = 0; k < y.top; ++k)
-      v[c] = add4(v[c], slabs(y.rows + (size_t)y.place[(size_t)row * y.top + k] * H + 4 * (size_t)idx, y.rows_splits, y.rows_stride));
-    ss += (Acc)v[c].x * (Acc)v[c].x + (Acc)v[c].y * (Acc)v[c].y + (Acc)v[c].z * (Acc)v[c].z + (Acc)v[c].w * (Acc)v[c].w;
+    for (uint32_t k = 0; k < y.top; ++k) {
+      const uint32_t at = y.place[(size_t)row * y.top + k];
+      if (POST) {
+        v[c] = add4(v[c], slabs(y.rows + (size_t)at * H + 4 * (size_t)idx, y.rows_splits, y.rows_stride));
+      } else {
+        const float4 e = at == kNoPlace ? load4<T>(static_cast<const T *>(y.identity) + (size_t)row * H + 4 * (size_t)idx)
+                                        : slabs(y.rows + (size_t)at * H + 4 * (size_t)idx, y.rows_splits, y.rows_stride);
+        v[c] = axpy4(y.weight ? y.weight[(size_t)row * y.top + k] : 1.f, e, v[c]);
+      }
+    }
+    if (POST) ss += (Acc)v[c].x * (Acc)v[c].x + (Acc)v[c].y * (Acc)v[c].y + (Acc)v[c].z * (Acc)v[c].z + (Acc)v[c].w * (Acc)v[c].w;
   }
-  const float s1 = norm_scale<Acc>(block_sum<Acc>(ss, red), H, eps);
+  const float s1 = POST ? norm_scale<Acc>(block_sum<Acc>(ss, red), H, eps) : 1.f;
   ss = Acc(0);
 #pragma unroll
   for (int c = 0; c < CHUNKS; ++c) {
     const uint32_t idx = threadIdx.x + c * blockDim.x;
     if (idx >= nvec) continue;
-    const float4 w = kLate ? ld4(post_w + 4 * (size_t)idx) : pw[kLate ? 0 : c];
-    x[c] = make_float4(x[c].x + mult * (v[c].x * s1 * w.x), x[c].y + mult * (v[c].y * s1 * w.y), x[c].z + mult * (v[c].z * s1 * w.z),
-                       x[c].w + mult * (v[c].w * s1 * w.w));
+    if (POST) {
+      const float4 w = kLate ? ld4(post_w + 4 * (size_t)idx) : pw[kLate ? 0 : c];
+      x[c] = make_float4(x[c].x + mult * (v[c].x * s1 * w.x), x[c].y + mult * (v[c].y * s1 * w.y), x[c].z + mult * (v[c].z * s1 * w.z),
+                         x[c].w + mult * (v[c].w * s1 * w.w));
+    } else {
+      x[c] = axpy4(mult, v[c], x[c]);
+      if (add.embed) x[c] = axpy4(add.scale, load4<T>(add.embed + (size_t)add.tokens[row] * H + 4 * (size_t)idx), x[c]);
+      if (add.shift) x[c] = add4(x[c], ld4(add.shift + 4 * (size_t)idx));
+    }
     if (!row_map) *reinterpret_cast<float4 *>(h + 4 * (size_t)idx) = x[c];
     ss += (Acc)x[c].x * (Acc)x[c].x + (Acc)x[c].y * (Acc)x[c].y + (Acc)x[c].z * (Acc)x[c].z + (Acc)x[c].w * (Acc)x[c].w;
   }
@@ -794,36 +881,66 @@ post_norm_residual_vec_kernel(SublayerOutput y, float *__restrict__ hidden, cons
 }
 
 namespace {
-template <typename T, int CHUNKS, int SLABS>
-int launch_post_norm_vec(SublayerOutput y, float *hidden, const float *post_w, float mult, const float *pre_w, float eps, T *out,
-                         const uint32_t *row_map, uint32_t out_rows, uint32_t H, uint32_t threads, cudaStream_t stream) {
-  ORION_CUDA_CHECK("post_norm_residual", launch_pdl(post_norm_residual_vec_kernel<T, CHUNKS, SLABS>, dim3(out_rows), dim3(threads), 0, stream, y, hidden,
-                                                    post_w, mult, pre_w, eps, out, row_map, H));
-  return after_launch("post_norm_residual");
+template <typename T, int CHUNKS, int SLABS, bool POST>
+int launch_post_norm_vec(SublayerOutput y, float *hidden, const float *post_w, float mult, StreamAddition<T> add, const float *pre_w, float eps,
+                         T *out, const uint32_t *row_map, uint32_t out_rows, uint32_t H, uint32_t threads, cudaStream_t stream) {
+  ORION_CUDA_CHECK("sublayer_residual", launch_pdl(post_norm_residual_vec_kernel<T, CHUNKS, SLABS, POST>, dim3(out_rows), dim3(threads), 0, stream, y,
+                                                   hidden, post_w, mult, add, pre_w, eps, out, row_map, H));
+  return after_launch("sublayer_residual");
 }
-}  // namespace
 
-template <typename T>
-int launch_post_norm_residual(SublayerOutput y, float *hidden, const float *post_w, float mult, const float *pre_w, float eps, T *out,
-                              const uint32_t *row_map, uint32_t out_rows, uint32_t H, cudaStream_t stream) {
+template <typename T, bool POST>
+int launch_join(SublayerOutput y, float *hidden, const float *post_w, float mult, StreamAddition<T> add, const float *pre_w, float eps, T *out,
+                const uint32_t *row_map, uint32_t out_rows, uint32_t H, cudaStream_t stream) {
   if (out_rows == 0) return ORION_OK;
   if (H % 4 == 0 && H / 4 <= 2048 && y.split_stride % 4 == 0 && y.rows_stride % 4 == 0) {
     const uint32_t nvec = H / 4, threads = nvec >= 512 ? 512 : (nvec + 31) / 32 * 32, chunks = (nvec + threads - 1) / threads;
     const uint32_t a = y.partial ? y.splits : 1, b = y.top ? y.rows_splits : 1;
     const int slabs = slab_variant(out_rows, a > b ? a : b);
     auto pick = [&](auto none, auto one, auto four) { return slabs == 1 ? one : (slabs == 4 ? four : none); };
-    auto run = chunks == 1   ? pick(launch_post_norm_vec<T, 1, 0>, launch_post_norm_vec<T, 1, 1>, launch_post_norm_vec<T, 1, 4>)
-               : chunks == 2 ? pick(launch_post_norm_vec<T, 2, 0>, launch_post_norm_vec<T, 2, 1>, launch_post_norm_vec<T, 2, 4>)
-                             : pick(launch_post_norm_vec<T, 4, 0>, launch_post_norm_vec<T, 4, 1>, launch_post_norm_vec<T, 4, 4>);
-    return run(y, hidden, post_w, mult, pre_w, eps, out, row_map, out_rows, H, threads, stream);
+    auto run = chunks == 1   ? pick(launch_post_norm_vec<T, 1, 0, POST>, launch_post_norm_vec<T, 1, 1, POST>, launch_post_norm_vec<T, 1, 4, POST>)
+               : chunks == 2 ? pick(launch_post_norm_vec<T, 2, 0, POST>, launch_post_norm_vec<T, 2, 1, POST>, launch_post_norm_vec<T, 2, 4, POST>)
+                             : pick(launch_post_norm_vec<T, 4, 0, POST>, launch_post_norm_vec<T, 4, 1, POST>, launch_post_norm_vec<T, 4, 4, POST>);
+    return run(y, hidden, post_w, mult, add, pre_w, eps, out, row_map, out_rows, H, threads, stream);
   }
   const size_t smem = (size_t)H * sizeof(float);
   if (smem > 200 * 1024) return set_error(ORION_ERR_INTERNAL, "hidden size %u too large for the fused norm kernel", H);
   static bool attr_set[kMaxDeviceOrdinals] = {};
-  ORION_CUDA_CHECK("post_norm_residual attr", ensure_dynamic_smem(post_norm_residual_kernel<T>, 200 * 1024, attr_set));
-  ORION_CUDA_CHECK("post_norm_residual", launch_pdl(post_norm_residual_kernel<T>, dim3(out_rows), dim3(kNormThreads), smem, stream, y, hidden, post_w,
-                                                    mult, pre_w, eps, out, row_map, H));
-  return after_launch("post_norm_residual");
+  ORION_CUDA_CHECK("sublayer_residual attr", ensure_dynamic_smem(post_norm_residual_kernel<T>, 200 * 1024, attr_set));
+  ORION_CUDA_CHECK("sublayer_residual", launch_pdl(post_norm_residual_kernel<T>, dim3(out_rows), dim3(kNormThreads), smem, stream, y, hidden, post_w,
+                                                   mult, add, pre_w, eps, out, row_map, H));
+  return after_launch("sublayer_residual");
+}
+}  // namespace
+
+template <typename T>
+int launch_post_norm_residual(SublayerOutput y, float *hidden, const float *post_w, float mult, const float *pre_w, float eps, T *out,
+                              const uint32_t *row_map, uint32_t out_rows, uint32_t H, cudaStream_t stream) {
+  return launch_join<T, true>(y, hidden, post_w, mult, StreamAddition<T>{}, pre_w, eps, out, row_map, out_rows, H, stream);
+}
+template <typename T>
+int launch_sublayer_residual(SublayerOutput y, float *hidden, float mult, StreamAddition<T> add, const float *pre_w, float eps, T *out,
+                             const uint32_t *row_map, uint32_t out_rows, uint32_t H, cudaStream_t stream) {
+  return launch_join<T, false>(y, hidden, nullptr, mult, add, pre_w, eps, out, row_map, out_rows, H, stream);
+}
+
+namespace {
+__global__ void __launch_bounds__(256) softcap_kernel(float *__restrict__ x, uint32_t cols, uint32_t ld, float cap) {
+  pdl_trigger();
+  pdl_wait();
+  float *row = x + (size_t)blockIdx.y * ld;
+  for (uint32_t c = blockIdx.x * blockDim.x + threadIdx.x; c < cols; c += gridDim.x * blockDim.x) row[c] = softcap_f(row[c], cap);
+}
+}  // namespace
+int launch_softcap(float *x, uint32_t rows, uint32_t cols, uint32_t ld, float cap, cudaStream_t stream) {
+  if (rows == 0 || cols == 0) return ORION_OK;
+  const uint32_t per_row = (cols + 1023) / 1024;
+  for (uint32_t r = 0; r < rows; r += 65535) {
+    const uint32_t n = rows - r < 65535 ? rows - r : 65535;
+    ORION_CUDA_CHECK("softcap", launch_pdl(softcap_kernel, dim3(per_row, n), dim3(256), 0, stream, x + (size_t)r * ld, cols, ld, cap));
+    ORION_TRY(after_launch("softcap"));
+  }
+  return ORION_OK;
 }
 
 // dst[r * dst_stride + c] = src[r * cols + c]: spreads the rows of a contiguous matrix over a
@@ -934,7 +1051,7 @@ int launch_fill_normal(T *dst, size_t n, uint64_t seed, cudaStream_t stream) {
 
 #define ORION_INSTANTIATE(T)                                                                      \
   template int launch_embed_rmsnorm<T>(const T *, const uint32_t *, const float *, float, float *, \
-                                       T *, uint32_t, uint32_t, cudaStream_t);                    \
+                                       T *, uint32_t, uint32_t, cudaStream_t, float, const float *); \
   template int launch_residual_rmsnorm<T>(const float *, uint32_t, size_t, float *, const float *, \
                                           float, T *, const uint32_t *, uint32_t, uint32_t,       \
                                           cudaStream_t, uint32_t *);                              \
@@ -952,6 +1069,9 @@ int launch_fill_normal(T *dst, size_t n, uint64_t seed, cudaStream_t stream) {
   template int launch_ffn_act<T>(const float *, uint32_t, size_t, const float *, FfnAct, T *, uint32_t, uint32_t, uint32_t, cudaStream_t); \
   template int launch_post_norm_residual<T>(SublayerOutput, float *, const float *, float, const float *, float, T *, const uint32_t *, \
                                             uint32_t, uint32_t, cudaStream_t);                    \
+  template int launch_sublayer_residual<T>(SublayerOutput, float *, float, StreamAddition<T>, const float *, float, T *, const uint32_t *, uint32_t, \
+                                           uint32_t, cudaStream_t);                               \
+  template int launch_gated_act<T>(const float *, uint32_t, size_t, GatedAct, T *, uint32_t, uint32_t, uint32_t, cudaStream_t); \
   template int launch_convert_from_f32<T>(const float *, T *, size_t, cudaStream_t);              \
   template int launch_convert_to_f32<T>(const T *, float *, size_t, cudaStream_t);                \
   template int launch_arena_to_reference_order<T>(const T *, KvLayout, float *, cudaStream_t);    \

@@ -204,7 +204,7 @@ __device__ __forceinline__ constexpr uint32_t instr_desc() {
          ((uint32_t)(M >> 4) << 24);
 }
 
-// ACT: the epilogue stores activations (kGemmGelu, kGemmRelu2, kGemmStore); else f32 partials, or SwiGLU where `act` is given. A
+// ACT: the epilogue stores activations (kGemmGelu, kGemmRelu2, kGemmGeglu, kGemmStore); else f32 partials, or SwiGLU where `act` is given. A
 // template parameter, since the larger epilogue costs the weight-streaming shapes 0.8 us per launch.
 template <int TOKN, int WST, int XST, int MT, bool PAIR, bool ACT>
 __global__ void __launch_bounds__(kThreads)
@@ -452,6 +452,19 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
       tmem_ld_wait();
       const int mt = mc / TOKN, c = mc % TOKN;
       const uint32_t n = n0 + mt * kTileN + lq * 32 + lane;
+      if (epilogue == kGemmGeglu) {
+        // lane 2i holds gate f, lane 2i + 1 up f; a pair trades halves and each finishes one token of every two
+        const uint32_t odd = lane & 1u;
+        bf16 *dst = act + (size_t)(t0 + c) * ldc + (n >> 1);
+#pragma unroll
+        for (int jj = 0; jj < 8; ++jj) {
+          const uint32_t recv = __shfl_xor_sync(0xffffffffu, odd ? r[2 * jj] : r[2 * jj + 1], 1);
+          const float g = __uint_as_float(odd ? recv : r[2 * jj]), u = __uint_as_float(odd ? r[2 * jj + 1] : recv);
+          const uint32_t j = 2 * jj + odd;
+          if (t0 + c + j < M && n < N) dst[(size_t)j * ldc] = __float2bfloat16_rn(gelu_tanh<bf16>(g) * u);
+        }
+        continue;
+      }
       if (t0 + c >= M || n >= N) continue;
       bf16 *dst = act + (size_t)(t0 + c) * ldc + n;
       const uint32_t valid = M - (t0 + c);
@@ -608,7 +621,7 @@ template <int TOKN, int WST, int XST, int MT = 1, bool PAIR = false>
 int launch_tc(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, float *partial, bf16 *act, uint32_t rows, uint32_t n,
               uint32_t k, uint32_t splits, bool cluster_reduce, uint32_t ldc, GemmEpilogue epi, cudaStream_t stream, ReadyWait ready,
               const float *bias) {
-  auto form = epi == kGemmGelu || epi == kGemmStore || epi == kGemmRelu2 ? launch_tc_form<true, TOKN, WST, XST, MT, PAIR>
+  auto form = epi == kGemmGelu || epi == kGemmStore || epi == kGemmRelu2 || epi == kGemmGeglu ? launch_tc_form<true, TOKN, WST, XST, MT, PAIR>
                                                     : launch_tc_form<false, TOKN, WST, XST, MT, PAIR>;
   return form(x, ldx, w, ldw, partial, act, rows, n, k, splits, cluster_reduce, ldc, epi, stream, ready, bias);
 }
@@ -670,8 +683,8 @@ int launch_gemm_tc(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, flo
   const uint32_t nkb = (k + kSlabK - 1) / kSlabK;
   if (cluster_reduce && (splits < 2 || splits > 8 || act != nullptr))
     return set_error(ORION_ERR_INTERNAL, "cluster split-K needs 2..8 splits and f32 output");
-  if (epi == kGemmSwiglu && (splits != 1 || n % 2 != 0))
-    return set_error(ORION_ERR_INTERNAL, "the fused SwiGLU epilogue needs one k split and an even row count");
+  if ((epi == kGemmSwiglu || epi == kGemmGeglu) && (splits != 1 || n % 2 != 0))
+    return set_error(ORION_ERR_INTERNAL, "a gated epilogue needs one k split and an even row count");
   if ((act != nullptr) != (epi != kGemmPartials) || (act != nullptr && splits != 1))
     return set_error(ORION_ERR_INTERNAL, "a GEMM epilogue that stores activations needs one k split and a place for them");
   if (splits < 1 || splits > nkb)
@@ -818,7 +831,7 @@ int launch_gemm_swiglu(const bf16 *x, uint32_t ldx, const bf16 *w_interleaved, u
 
 int launch_gemm_act(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, bf16 *act, uint32_t ld_act, uint32_t rows, uint32_t n,
                     uint32_t k, GemmEpilogue epi, cudaStream_t stream, const float *bias) {
-  if (epi != kGemmGelu && epi != kGemmStore && epi != kGemmRelu2) return set_error(ORION_ERR_INTERNAL, "not an epilogue of this entry point");
+  if (epi != kGemmGelu && epi != kGemmStore && epi != kGemmRelu2 && epi != kGemmGeglu) return set_error(ORION_ERR_INTERNAL, "not an epilogue of this entry point");
   if (!gemm_tc_supported(rows, n, k, ldx, ldw, x, w))
     return set_error(ORION_ERR_INTERNAL, "tensor-core GEMM planned for an unaligned operand");
   return launch_gemm_tc(x, ldx, w, ldw, nullptr, rows, n, k, 1, stream, act, false, ld_act, ReadyWait{}, epi, bias);

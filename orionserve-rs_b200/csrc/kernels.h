@@ -42,7 +42,7 @@ struct KvLayout {
 template <typename T>
 int launch_embed_rmsnorm(const T *embed, const uint32_t *tokens, const float *norm_w, float eps,
                          float *hidden, T *normed, uint32_t rows, uint32_t hidden_size,
-                         cudaStream_t stream);
+                         cudaStream_t stream, float scale = 1.f, const float *shift = nullptr);  // hidden = scale * embed (+ shift, one vector)
 
 // hidden[r] += sum_s partial[s][r] (+ nothing else); out[i] = rms_norm(hidden[src(i)]) * w,
 // src(i) = row_map ? row_map[i] : i. With row_map the residual is not written
@@ -79,6 +79,10 @@ int launch_rope_rows(T *x, const uint32_t *positions, const float *rope_cos, con
 template <typename T>
 int launch_swiglu(const float *partial, uint32_t splits, size_t split_stride, T *act, uint32_t rows,
                   uint32_t ffn, cudaStream_t stream, bool interleaved = false);
+// The interleaved form with any gated activation and row stride `ldo`.
+template <typename T>
+int launch_gated_act(const float *partial, uint32_t splits, size_t split_stride, GatedAct f, T *act, uint32_t ldo, uint32_t rows, uint32_t ffn,
+                     cudaStream_t stream);
 // dst[r * dst_stride + c] = src[r * cols + c]
 template <typename T>
 int launch_copy_rows_strided(const T *src, T *dst, size_t rows, size_t cols, size_t dst_stride, cudaStream_t stream);
@@ -102,10 +106,27 @@ struct SublayerOutput {
   const uint32_t *place = nullptr;
   uint32_t top = 0, rows_splits = 0;
   size_t rows_stride = 0;
+  const float *weight = nullptr;   // [rows][top] factors of the experts' rows; null = 1
+  const void *identity = nullptr;  // [row][hidden] of T: what a choice with the place kNoPlace contributes
 };
+constexpr uint32_t kNoPlace = 0xFFFFFFFFu;
 template <typename T>
 int launch_post_norm_residual(SublayerOutput y, float *hidden, const float *post_w, float mult, const float *pre_w, float eps, T *out,
                               const uint32_t *row_map, uint32_t out_rows, uint32_t hidden_size, cudaStream_t stream);
+// Pre-norm layers: the output joins as it is, hidden += mult * y, and what comes ahead of the next layer follows it:
+// hidden += scale * embed[tokens[r]] (embed may be null), hidden += shift (a vector, may be null). `y.identity` may be `out`.
+template <typename T>
+struct StreamAddition {
+  const T *embed = nullptr;
+  const uint32_t *tokens = nullptr;
+  float scale = 1.f;
+  const float *shift = nullptr;
+};
+template <typename T>
+int launch_sublayer_residual(SublayerOutput y, float *hidden, float mult, StreamAddition<T> add, const float *pre_w, float eps, T *out,
+                             const uint32_t *row_map, uint32_t out_rows, uint32_t hidden_size, cudaStream_t stream);
+// x[r * ld + c] = cap * tanh(x[r * ld + c] / cap)
+int launch_softcap(float *x, uint32_t rows, uint32_t cols, uint32_t ld, float cap, cudaStream_t stream);
 
 // out[r][n] = sum_s partial[s][r][n] + bias[n]  (finishes tensor::linear, tensor.rs:126).
 int launch_finish_linear(const float *partial, uint32_t splits, size_t split_stride,
@@ -154,18 +175,30 @@ struct AttnBatch {
 };
 
 // Which of the positions up to its own a query sees: the last `window` of them (0 = no window), of those the ones in
-// its own chunk of `chunk` positions, counted from the sequence's start (0 = no chunks).
+// its own chunk of `chunk` positions, counted from the sequence's start (0 = no chunks), and besides them the first `keep`
+// positions of the sequence.
 struct KeyRange {
-  uint32_t window = 0, chunk = 0;
+  uint32_t window = 0, chunk = 0, keep = 0;
+  // The first position of the run that ends with the query itself.
   __host__ __device__ uint32_t first(uint32_t pos) const {
     const uint32_t w = window && pos + 1 > window ? pos + 1 - window : 0, c = chunk ? pos / chunk * chunk : 0;
     return w > c ? w : c;
   }
+  // Positions before that run which the query sees as well: 0 .. kept(pos) - 1.
+  __host__ __device__ uint32_t kept(uint32_t pos) const {
+    const uint32_t f = first(pos);
+    return keep < f ? keep : f;
+  }
+  // Blocks of `size` positions before the one that the run begins in (`block0`) which hold kept positions.
+  __host__ __device__ uint32_t kept_blocks(uint32_t block0, uint32_t size) const {
+    const uint32_t n = (keep + size - 1) / size;
+    return n < block0 ? n : block0;
+  }
   // The most positions a query up to `max_position` sees.
   __host__ __device__ uint32_t most(uint32_t max_position) const {
     uint32_t n = max_position + 1;
-    if (window && window < n) n = window;
-    return chunk && chunk < n ? chunk : n;
+    if (window && window < n && keep < n - window) n = window + keep;
+    return chunk && chunk < n && keep < n - chunk ? chunk + keep : n;
   }
 };
 // What a design adds to causal attention over everything before; the defaults add nothing.
@@ -174,6 +207,8 @@ struct AttnForm {
   KeyRange range;
   const float *sinks = nullptr;   // [q_heads] logits that enter the denominator once and carry no value
   const float *gate = nullptr;    // [rows][q_heads] factors of the heads' outputs
+  const void *value_gate = nullptr;  // [rows][q_heads * out_dim] of T: factors of the values
+  float softcap = 0.f;            // scores become softcap * tanh(score / softcap); 0 = they stay
   uint32_t out_dim = 0, ldo = 0;  // values stored per head and row stride of the output; 0 = v_dim() and q_heads * out_dim
   // Decode only: the batch rows that decode (item i of the scratch belongs to row_list[i]), and the first row of every
   // sequence, since several rows of one sequence may decode together. Null: every row, one per sequence.
@@ -191,15 +226,21 @@ int launch_paged_attention_generic(const T *q, const T *arena, KvLayout kv, uint
 // (2i, 2i + 1) by the table's angles, q to `q_out` [rows][q_heads][kv.head_dim], k and v to the arena, and sigmoid(g), one
 // value per query head, to `gate` [rows][q_heads] (may be null: no such columns). dim and value_dim are what the projection
 // holds per head; the arena's rows may be longer, and what is beyond stays as it is.
+//
+// per_head: the other family of layouts. Every head is normalised by itself (gains of dim values, shared by the heads), dimension
+// i rotates with i + rope_dims / 2 if `halves` is set, q, k and v have biases ([q | k | v], may be null), and g has a column per
+// value: sigmoid(g) goes to `value_gate` [rows][q_heads * value_dim] (null: no such columns) instead of `gate`.
 struct AttnInputs {
   uint32_t q_heads, kv_heads, dim, value_dim, rope_dims, ld;
   float eps;
   const float *q_norm, *k_norm, *rope_cos, *rope_sin;
+  bool per_head = false, halves = false;
+  const float *bias = nullptr;
 };
 template <typename T>
 int launch_attention_prepare(const float *partial, uint32_t splits, size_t split_stride, AttnInputs in, const uint32_t *positions,
                              const uint32_t *slot_block, const uint32_t *slot_slot, T *q_out, T *arena, KvLayout kv, uint32_t layer,
-                             float *gate, uint32_t rows, cudaStream_t stream);
+                             float *gate, uint32_t rows, cudaStream_t stream, T *value_gate = nullptr);
 // K and V rows of one layer's arena as f32, [k|v][block][kv head][slot][dim] with dim values of a K row, value_dim of a V row.
 template <typename T>
 int launch_arena_rows(const T *arena, KvLayout kv, uint32_t dim, uint32_t value_dim, float *out, cudaStream_t stream);
@@ -341,6 +382,47 @@ template <typename T>
 int launch_min_gru(const float *partial, uint32_t splits, size_t split_stride, const float *bias, float *state, StateBatch sb,
                    T *out, uint32_t ldo, uint32_t width, cudaStream_t stream);
 
+// Gated linear attention: per head a state S of dim x value_dim, S_t = diag(alpha_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t,
+// out = rms_norm(o_t) * norm * silu(g). The joint projection holds [q | k | v | g | a] per row (row stride ld), a of `rank` values for
+// all heads; q is scaled by dim^(-1/2), alpha = sigmoid(W a + bias)^(1 / tau), one value per key channel, W [heads * dim][rank].
+// `state` is [copies][heads][dim][value_dim] in f32.
+struct GlaShape {
+  uint32_t heads, dim, value_dim, rank, ld;
+  float tau, eps;
+  __host__ __device__ uint32_t q_cols() const { return heads * dim; }
+  __host__ __device__ uint32_t v_cols() const { return heads * value_dim; }
+  __host__ __device__ uint32_t cols() const { return 2 * q_cols() + 2 * v_cols() + rank; }
+  __host__ __device__ size_t state_floats() const { return (size_t)heads * dim * value_dim; }
+};
+template <typename T>
+struct GlaWeights {
+  const T *decay;           // [heads * dim][rank]
+  const float *bias, *norm;  // [heads * dim], [value_dim]
+};
+// Token by token: the sequences of the batch that have at most `most_rows` rows.
+template <typename T>
+int launch_gla_steps(const float *partial, uint32_t splits, size_t split_stride, GlaShape s, GlaWeights<T> w, float *state, StateBatch sb,
+                     uint32_t most_rows, T *out, uint32_t ldo, cudaStream_t stream);
+// Prompt portions, kGlaChunk rows at a time: within a chunk the scores of all pairs of rows, between chunks the state.
+constexpr uint32_t kGlaChunk = 64;
+struct GlaChunk {
+  uint32_t row, count, pad0, pad1;  // batch rows [row, row + count) of one sequence
+};
+struct GlaPortion {
+  uint32_t seq, chunk, chunks, pad;  // its chunks follow one another in the list
+};
+struct GlaPortions {
+  const GlaChunk *chunks;
+  const GlaPortion *portions;
+  uint32_t num_chunks, num_portions;
+};
+bool gla_chunks_supported(GlaShape s);
+// Bytes of scratch that a batch needs (chunk operands, then the heads' outputs in f32).
+size_t gla_scratch_bytes(GlaShape s, uint32_t chunks, uint32_t rows);
+int launch_gla_chunks(const float *partial, uint32_t splits, size_t split_stride, GlaShape s, GlaWeights<bf16> w, float *state, StateBatch sb,
+                      GlaPortions p, void *scratch, bf16 *out, uint32_t ldo, cudaStream_t stream);
+int gla_poll_error(uint32_t *code);
+
 // ---- latent attention ---------------------------------------------------------------------
 //
 // The cache of one layer holds, per token, the normalised latent (kv_rank values) followed by the rotated key
@@ -415,8 +497,15 @@ int latent_prefill_poll_error(uint32_t *code);
 // (W_up x)). Rows are copied into the order of their experts, and the two products run over tiles of rows of one expert.
 // Expert weights are stacked: up [experts][2 * ffn][hidden] with gate row f at 2f and up row f at 2f + 1, down
 // [experts][hidden][ffn]; the shared expert's the same with one expert.
+// Variants: softmax of the logits for the sigmoid; a correction per output of the router that takes part in the choice only;
+// `identity` further outputs of the router whose experts return their input (they take no part in the products); scores that
+// multiply the experts' outputs (where they are summed: SublayerOutput::weight); other gated activations.
 struct MoeShape {
   uint32_t hidden, experts, top, ffn, shared_ffn;
+  uint32_t identity = 0;
+  bool softmax = false, weigh_output = false;
+  GatedAct act{}, shared_act{};
+  __host__ __device__ uint32_t outputs() const { return experts + identity; }
 };
 struct MoeTile {
   uint32_t expert, row, count;  // sorted rows [row, row + count) go through `expert`; count 0: nothing to do
@@ -433,9 +522,9 @@ constexpr uint32_t kMoeMaxExperts = 1024;
 template <typename T>
 struct MoeBuffers {
   uint32_t *chosen = nullptr;  // [rows][top]
-  float *score = nullptr;      // [rows][top]
+  float *score = nullptr;      // [rows][top] (batches of few rows: only with weigh_output)
   uint32_t *histogram = nullptr;  // [moe_histogram_words]
-  uint32_t *place = nullptr;   // [rows][top]: sorted row of each choice
+  uint32_t *place = nullptr;   // [rows][top]: sorted row of each choice, kNoPlace for an identity expert
   float *row_score = nullptr;  // [rows * top] by sorted row
   MoeTile *tiles = nullptr;    // [plan.tiles]
   T *x = nullptr;              // [rows * top][hidden] sorted rows
@@ -445,17 +534,18 @@ struct MoeBuffers {
 };
 size_t moe_histogram_words(MoeShape s, uint32_t rows);
 size_t moe_up_floats(bool is_bf16, MoeShape s, uint32_t rows);
-// Experts and scores of every row from the router's partial sums [splits][rows][experts], and the sorted order.
+// Experts and scores of every row from the router's partial sums [splits][rows][outputs], and the sorted order. correction:
+// [outputs], may be null.
 template <typename T>
-int launch_moe_route(const float *logits, uint32_t splits, size_t split_stride, const T *x, MoeShape s, MoePlan plan, MoeBuffers<T> b,
-                     uint32_t rows, cudaStream_t stream);
+int launch_moe_route(const float *logits, uint32_t splits, size_t split_stride, const float *correction, const T *x, MoeShape s, MoePlan plan,
+                     MoeBuffers<T> b, uint32_t rows, cudaStream_t stream);
 // Both products: `down` of the sorted rows into b.down, of the shared expert into shared_out [down_splits][rows][hidden].
 template <typename T>
 int launch_moe_experts(const T *x, const T *w_up, const T *w_down, const T *shared_up, const T *shared_down, MoeShape s, MoePlan plan,
                        MoeBuffers<T> b, float *shared_out, uint32_t rows, cudaStream_t stream);
 // One product of the grouped kind on tcgen05: rows of `x` by tile through rows [expert * n, (expert + 1) * n) of `w`, and rows of
 // `shared_x` through `shared_w` (shared_n = 0: none). swiglu: activations to act / shared_act (row stride n / 2, shared_n / 2),
-// the products multiplied by row_score; else f32 to out / shared_out, [splits][rows][n].
+// the products multiplied by row_score (null = 1); else f32 to out / shared_out, [splits][rows][n].
 struct MoeProduct {
   const bf16 *x, *w, *shared_x, *shared_w;
   uint32_t n, k, shared_n, shared_k;
@@ -464,6 +554,7 @@ struct MoeProduct {
   const float *row_score;
   bf16 *act, *shared_act;
   float *out, *shared_out;
+  GatedAct f{}, shared_f{};
 };
 bool moe_tc_supported(MoeShape s);
 int launch_moe_product_tc(const MoeProduct &p, bool swiglu, uint32_t splits, MoePlan plan, cudaStream_t stream);
@@ -542,7 +633,7 @@ template <typename T>
 int launch_gemm_simt(const T *x, uint32_t ldx, const T *w, uint32_t ldw, float *out, uint32_t rows,
                      uint32_t n, uint32_t k, cudaStream_t stream);
 // tcgen05 / TMEM / TMA GEMM (bf16).
-enum GemmEpilogue : uint32_t { kGemmPartials = 0, kGemmSwiglu = 1, kGemmGelu = 2, kGemmStore = 3, kGemmRelu2 = 4 };
+enum GemmEpilogue : uint32_t { kGemmPartials = 0, kGemmSwiglu = 1, kGemmGelu = 2, kGemmStore = 3, kGemmRelu2 = 4, kGemmGeglu = 5 };
 bool gemm_tc_supported(uint32_t rows, uint32_t n, uint32_t k, uint32_t ldx, uint32_t ldw,
                        const void *x, const void *w);
 int launch_gemm_tc(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, float *partial,
@@ -550,7 +641,8 @@ int launch_gemm_tc(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, flo
                    bf16 *act = nullptr, bool cluster_reduce = false, uint32_t ldc = 0,
                    ReadyWait ready = {}, GemmEpilogue epi = kGemmPartials, const float *bias = nullptr);
 // The same projection with its result stored as bf16 activations, act[r * ld_act + n] = f(x.w_n + bias[n]), f = GELU (tanh
-// form), the square of relu or the identity; bias may be null. One k split only.
+// form), the square of relu or the identity; bias may be null. kGemmGeglu: rows 2f and 2f + 1 of w are gate and up of the same f, and
+// act[r * ld_act + f] = GELU(gate) * up. One k split only.
 int launch_gemm_act(const bf16 *x, uint32_t ldx, const bf16 *w, uint32_t ldw, bf16 *act, uint32_t ld_act, uint32_t rows, uint32_t n,
                     uint32_t k, GemmEpilogue epi, cudaStream_t stream, const float *bias = nullptr);
 // Gate/up projection with SwiGLU in the epilogue: `w_interleaved` is [2 * ffn][k] with gate row f

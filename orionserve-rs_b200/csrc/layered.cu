@@ -20,26 +20,35 @@ int LayeredModel<T>::check_layer(uint32_t i) const {
   switch (s.mixer) {
     case ORION_MIXER_MIN_GRU: sizes = s.width > 0; break;
     case ORION_MIXER_LATENT_ATTENTION: sizes = s.heads > 0 && s.dim + s.rot_dim > 0 && s.value_dim > 0 && s.kv_rank > 0; break;
+    case ORION_MIXER_GLA: sizes = s.heads > 0 && s.dim > 0 && s.value_dim > 0 && s.decay_rank > 0 && s.decay_tau > 0; break;
     case ORION_MIXER_ATTENTION: sizes = s.heads > 0 && s.kv_heads > 0 && s.heads % s.kv_heads == 0 && s.dim > 0 && s.value_dim > 0; break;
   }
   if (!sizes)
     return set_error(ORION_ERR_MODEL, "config.json is malformed: layer %u has an unknown mixer, a size of zero or uneven groups of heads", i);
   const uint32_t rotates = s.mixer == ORION_MIXER_ATTENTION ? s.dim : s.rot_dim;
-  if (s.mixer != ORION_MIXER_MIN_GRU && (s.rope_dims % 2 != 0 || s.rope_dims > rotates))
+  if ((s.mixer == ORION_MIXER_ATTENTION || s.mixer == ORION_MIXER_LATENT_ATTENTION) && (s.rope_dims % 2 != 0 || s.rope_dims > rotates))
     return set_error(ORION_ERR_MODEL, "config.json is malformed: layer %u rotates %u of %u dimensions", i, s.rope_dims, rotates);
-  if (s.experts > 0 && (s.ffn_dim == 0 || s.experts_per_token == 0 || s.experts_per_token > s.experts || s.experts > kMoeMaxExperts))
-    return set_error(ORION_ERR_MODEL, "config.json is malformed: layer %u uses %u of %u experts of width %u (at most %u experts)", i,
-                     s.experts_per_token, s.experts, s.ffn_dim, kMoeMaxExperts);
-  if (s.activation > ORION_ACT_RELU2) return set_error(ORION_ERR_MODEL, "config.json is malformed: layer %u has an unknown activation", i);
-  if (!sandwich() && (s.experts > 0 || s.ffn_bias))
+  const uint64_t outputs = (uint64_t)s.experts + s.router_identity;
+  if (s.experts > 0 && (s.ffn_dim == 0 || s.experts_per_token == 0 || s.experts_per_token > outputs || outputs > kMoeMaxExperts))
+    return set_error(ORION_ERR_MODEL, "config.json is malformed: layer %u uses %u of %llu experts of width %u (at most %u experts)", i,
+                     s.experts_per_token, (unsigned long long)outputs, s.ffn_dim, kMoeMaxExperts);
+  if (s.activation > ORION_ACT_GEGLU_TANH || s.router > ORION_ROUTER_SOFTMAX || s.expert_form > ORION_EXPERT_CLAMPED || s.qk_norm > ORION_QK_NORM_PER_HEAD)
+    return set_error(ORION_ERR_MODEL, "config.json is malformed: layer %u has an unknown activation, router or norm", i);
+  if (s.mixer == ORION_MIXER_ATTENTION && s.qk_norm != ORION_QK_NORM_PER_HEAD && (s.rope_halves || s.qkv_bias || s.value_gate))
+    return set_error(ORION_ERR_MODEL, "layer %u: rotated halves, biases and gates per value come with norms per head", i);
+  if (s.mixer == ORION_MIXER_ATTENTION && s.qk_norm == ORION_QK_NORM_PER_HEAD && s.head_gate)
+    return set_error(ORION_ERR_MODEL, "layer %u: a gate per head comes with norms over all heads", i);
+  if (d_.block == ORION_BLOCK_PARALLEL && (s.experts > 0 || s.ffn_bias))
     return set_error(ORION_ERR_MODEL, "layer %u: a parallel block has a dense feed-forward without biases", i);
+  if (d_.block != ORION_BLOCK_PRENORM && (s.activation == ORION_ACT_GEGLU_TANH || s.router != ORION_ROUTER_SIGMOID_INPUT || s.router_identity))
+    return set_error(ORION_ERR_MODEL, "layer %u: gated dense feed-forwards and softmax routers come with prenorm blocks", i);
   return ORION_OK;
 }
 
 template <typename T>
 int LayeredModel<T>::init() {
   const OrionLayeredDesc &d = d_;
-  if (d.hidden_size == 0 || d.vocab_size == 0 || d.num_layers == 0 || d.block > ORION_BLOCK_SANDWICH || (!sandwich() && d.conv_taps == 0))
+  if (d.hidden_size == 0 || d.vocab_size == 0 || d.num_layers == 0 || d.block > ORION_BLOCK_PRENORM || (parallel() && d.conv_taps == 0))
     return set_error(ORION_ERR_MODEL, "config.json is malformed: a model dimension is zero");
   if (d.block_size == 0 || d.max_batch_tokens == 0 || d.max_batch_sequences == 0 || d.num_state_slots == 0)
     return set_error(ORION_ERR_INVALID_REQUEST,
@@ -47,12 +56,35 @@ int LayeredModel<T>::init() {
   for (uint32_t i = 0; i < d.num_layers; ++i) ORION_TRY(check_layer(i));
   ORION_TRY(Base::init_step({d.hidden_size, d.vocab_size, d.max_position_embeddings, d.num_blocks, d.block_size, d.max_batch_tokens,
                              d.max_batch_sequences}));
-  layers_.resize(d.num_layers);
-  for (uint32_t i = 0; i < d.num_layers; ++i) {
-    layers_[i].d = specs_[i];
-    ORION_TRY(init_layer(layers_[i]));
-  }
   const size_t H = d.hidden_size;
+  const bool loop = d.loop_times > 0;
+  if (loop && (d.block != ORION_BLOCK_PRENORM || d.loop_start >= d.loop_stop || d.loop_stop > d.num_layers))
+    return set_error(ORION_ERR_MODEL, "config.json is malformed: layers %u to %u of %u cannot be looped", d.loop_start, d.loop_stop, d.num_layers);
+  if (loop) ORION_TRY(alloc(&loop_step_, d.loop_times * H));
+  first_run_.resize(d.num_layers);
+  auto run = [&](uint32_t i, uint32_t pass) -> int {
+    if (pass == 0) {
+      first_run_[i] = (uint32_t)layers_.size();
+      layers_.emplace_back();
+      layers_.back().d = specs_[i];
+      ORION_TRY(init_layer(layers_.back()));
+    } else {
+      const Layer again = layers_[first_run_[i]];
+      layers_.push_back(again);
+    }
+    Layer &L = layers_.back();
+    const bool begins = loop && i == d.loop_start;
+    L.shift = begins ? loop_step_ + pass * H : nullptr;
+    L.restart = begins && pass > 0;
+    return init_memory(L);
+  };
+  for (uint32_t i = 0; i < d.num_layers;) {
+    const bool first = loop && i == d.loop_start;
+    const uint32_t stop = first ? d.loop_stop : i + 1;
+    for (uint32_t pass = 0; pass < (first ? d.loop_times : 1); ++pass)
+      for (uint32_t k = i; k < stop; ++k) ORION_TRY(run(k, pass));
+    i = stop;
+  }
   ORION_TRY(alloc(&embed_, (size_t)d.vocab_size * H));
   if (d.untied_lm_head) ORION_TRY(alloc(&head_, (size_t)d.vocab_size * H));
   ORION_TRY(alloc(&final_norm_, H));
@@ -68,17 +100,34 @@ int LayeredModel<T>::init_rope(Layer &L) {
   const OrionLayerDesc &s = L.d;
   const Rope *r = nullptr;
   for (const Rope &x : ropes_)
-    if (x.base == s.rope_base && x.dims == s.rope_dims) r = &x;
+    if (x.base == s.rope_base && x.dims == s.rope_dims && x.factor == s.yarn_factor && x.original == s.yarn_original && x.fast == s.yarn_fast &&
+        x.slow == s.yarn_slow)
+      r = &x;
   if (!r) {
     const size_t half = s.rope_dims / 2, positions = d_.max_position_embeddings, n = positions * half;
     std::vector<float> c(n ? n : 1), sn(n ? n : 1);
+    std::vector<double> freq(half);
+    const double dims = s.rope_dims;
+    for (size_t k = 0; k < half; ++k) freq[k] = std::pow(s.rope_base, -2.0 * (double)k / dims);
+    double mult = 1.0;
+    if (s.yarn_factor > 0) {
+      // A pair that turns `fast` times or more within the original length keeps its frequency, one that turns `slow` times or less
+      // is stretched by the factor, and those between are blended by their place.
+      auto place = [&](double turns) { return dims * std::log(s.yarn_original / (2.0 * M_PI * turns)) / (2.0 * std::log(s.rope_base)); };
+      const double lo = std::max(std::floor(place(s.yarn_fast)), 0.0), hi = std::min(std::ceil(place(s.yarn_slow)), dims - 1.0);
+      for (size_t k = 0; k < half; ++k) {
+        const double ramp = std::min(1.0, std::max(0.0, ((double)k - lo) / std::max(hi - lo, 0.001)));
+        freq[k] = freq[k] / s.yarn_factor * ramp + freq[k] * (1.0 - ramp);
+      }
+      mult = 0.1 * std::log(s.yarn_factor) + 1.0;
+    }
     for (size_t p = 0; p < positions; ++p)
       for (size_t k = 0; k < half; ++k) {
-        const double angle = (double)p * std::pow(s.rope_base, -2.0 * (double)k / (double)s.rope_dims);
-        c[p * half + k] = (float)std::cos(angle);
-        sn[p * half + k] = (float)std::sin(angle);
+        const double angle = (double)p * freq[k];
+        c[p * half + k] = (float)(mult * std::cos(angle));
+        sn[p * half + k] = (float)(mult * std::sin(angle));
       }
-    Rope fresh{s.rope_base, s.rope_dims, nullptr, nullptr};
+    Rope fresh{s.rope_base, s.yarn_factor, s.yarn_original, s.yarn_fast, s.yarn_slow, s.rope_dims, nullptr, nullptr};
     ORION_TRY(alloc(&fresh.cos, n));
     ORION_TRY(alloc(&fresh.sin, n));
     ORION_CUDA_CHECK("upload rope", cudaMemcpy(fresh.cos, c.data(), n * sizeof(float), cudaMemcpyHostToDevice));
@@ -94,14 +143,10 @@ template <typename T>
 int LayeredModel<T>::init_layer(Layer &L) {
   const OrionLayeredDesc &d = d_;
   const OrionLayerDesc &s = L.d;
-  const size_t H = d.hidden_size, copies = 2 * (size_t)d.num_state_slots, keep = d.conv_taps ? d.conv_taps - 1 : 0;
+  const size_t H = d.hidden_size;
   ORION_TRY(alloc(&L.norm, H));
-  if (sandwich()) {
-    ORION_TRY(alloc(&L.norm_post, H));
-  } else {
-    ORION_TRY(alloc(&L.conv1, H * d.conv_taps));
-    ORION_TRY(zeroed(&L.conv_state, copies * keep * H));
-  }
+  if (sandwich()) ORION_TRY(alloc(&L.norm_post, H));
+  if (parallel()) ORION_TRY(alloc(&L.conv1, H * d.conv_taps));
   if (L.latent()) {
     L.ls = LatentShape{s.heads, s.dim, s.rot_dim, s.value_dim, s.kv_rank, s.window, s.rope_dims, d.block_size,
                        odd_groups(s.kv_rank + s.rot_dim), (float)s.scale, (float)d.norm_eps};
@@ -112,22 +157,27 @@ int LayeredModel<T>::init_layer(Layer &L) {
     ORION_TRY(init_rope(L));
   } else if (L.attention()) {
     // [q | k | v | gate], the rows of the matrix padded so that the partial sums of a row start on 32 bytes
-    L.mix_in = pad8(s.heads * s.dim + s.kv_heads * (s.dim + s.value_dim) + (s.head_gate ? s.heads : 0));
+    const uint32_t qkv = s.heads * s.dim + s.kv_heads * (s.dim + s.value_dim);
+    L.mix_in = pad8(qkv + (s.head_gate ? s.heads : 0) + (s.value_gate ? s.heads * s.value_dim : 0));
     L.mix_out = s.heads * s.value_dim;
     ORION_TRY(init_rope(L));
     if (s.qk_norm) {
-      ORION_TRY(alloc(&L.q_norm, (size_t)s.heads * s.dim));
-      ORION_TRY(alloc(&L.k_norm, (size_t)s.kv_heads * s.dim));
+      const bool own = s.qk_norm == ORION_QK_NORM_PER_HEAD;
+      ORION_TRY(alloc(&L.q_norm, (size_t)(own ? 1 : s.heads) * s.dim));
+      ORION_TRY(alloc(&L.k_norm, (size_t)(own ? 1 : s.kv_heads) * s.dim));
     }
+    if (s.qkv_bias) ORION_TRY(alloc(&L.mix_bias, qkv));
     if (s.sinks) ORION_TRY(alloc(&L.sinks, s.heads));
     // 16-bit caches pad the heads to sizes of the tensor-core kernels where those cover them
     const uint32_t dk = DTypeOf<T>::is_bf16 ? attention_padded_dim(s.dim, s.value_dim) : 0;
     const uint32_t dv = DTypeOf<T>::is_bf16 ? attention_padded_dim(s.value_dim, s.dim) : 0;
     L.kv = KvLayout{1, d.num_blocks, s.kv_heads, d.block_size, dk ? dk : s.dim, dk ? 1u : 0u, dk ? dv : s.value_dim};
     L.tuned = DTypeOf<T>::is_bf16 && attention_form_supported(L.kv, s.heads);
-    L.in = AttnInputs{s.heads, s.kv_heads, s.dim, s.value_dim, s.rope_dims, L.mix_in, (float)d.norm_eps, L.q_norm, L.k_norm, L.rope_cos, L.rope_sin};
+    L.in = AttnInputs{s.heads, s.kv_heads, s.dim, s.value_dim, s.rope_dims, L.mix_in, (float)d.norm_eps, L.q_norm, L.k_norm, L.rope_cos, L.rope_sin,
+                      s.qk_norm == ORION_QK_NORM_PER_HEAD, s.rope_halves != 0, L.mix_bias};
     L.form.scale = (float)s.scale;
-    L.form.range = KeyRange{s.window, s.chunk};
+    L.form.softcap = (float)s.softcap;
+    L.form.range = KeyRange{s.window, s.chunk, s.keep_first};
     L.form.sinks = L.sinks;
     L.form.out_dim = s.value_dim;
     if (L.tuned) {
@@ -136,29 +186,35 @@ int LayeredModel<T>::init_layer(Layer &L) {
       for (const TileSet &t : tile_sets_) known |= t.positions == positions;
       if (!known) tile_sets_.push_back(TileSet{positions, 0, 0});
     }
+  } else if (L.linear()) {
+    L.gla = GlaShape{s.heads, s.dim, s.value_dim, s.decay_rank, 0, (float)s.decay_tau, (float)d.norm_eps};
+    L.mix_in = L.gla.ld = pad8(L.gla.cols());
+    L.mix_out = L.gla.v_cols();
+    ORION_TRY(alloc(&L.w_decay, (size_t)L.gla.q_cols() * s.decay_rank));
+    ORION_TRY(alloc(&L.mix_bias, L.gla.q_cols()));
+    ORION_TRY(alloc(&L.out_norm, s.value_dim));
   } else {
     L.mix_in = 3 * s.width, L.mix_out = s.width;
     ORION_TRY(alloc(&L.mix_bias, 2 * (size_t)s.width));
-    ORION_TRY(zeroed(&L.rec_state, copies * s.width));
   }
-  if (L.cache_elems()) ORION_TRY(zeroed(&L.cache, d.num_blocks * L.cache_elems()));
   ORION_TRY(zeroed(&L.w_mix, (size_t)L.mix_in * H));
   // Activations start at multiples of 8 columns; the weights of the columns between them are zero.
-  L.ff_at = sandwich() ? 0 : pad8(L.mix_out);
-  L.cat = sandwich() ? pad8(L.mix_out) : L.ff_at + pad8(s.ffn_dim);
-  L.ff_ld = sandwich() ? pad8(s.ffn_dim) : L.cat;
+  L.ff_at = parallel() ? pad8(L.mix_out) : 0;
+  L.cat = parallel() ? L.ff_at + pad8(s.ffn_dim) : pad8(L.mix_out);
+  L.ff_ld = parallel() ? L.cat : pad8(s.ffn_dim);
   if (L.attention()) L.form.ldo = L.cat;
   ORION_TRY(zeroed(&L.w_out, H * L.cat));
   if (!L.has_ffn()) return ORION_OK;
-  if (sandwich()) {
-    ORION_TRY(alloc(&L.norm2, H));
-    ORION_TRY(alloc(&L.norm2_post, H));
-  } else {
-    ORION_TRY(alloc(&L.conv2, H * d.conv_taps));
-  }
+  if (parallel()) ORION_TRY(alloc(&L.conv2, H * d.conv_taps));
+  else ORION_TRY(alloc(&L.norm2, H));
+  if (sandwich()) ORION_TRY(alloc(&L.norm2_post, H));
   if (s.experts > 0) {
-    L.moe = MoeShape{d.hidden_size, s.experts, s.experts_per_token, s.ffn_dim, s.shared_dim};
-    ORION_TRY(alloc(&L.w_router, (size_t)s.experts * H));
+    L.moe = MoeShape{d.hidden_size, s.experts, s.experts_per_token, s.ffn_dim, s.shared_dim, s.router_identity};
+    L.moe.softmax = L.moe.weigh_output = s.router == ORION_ROUTER_SOFTMAX;
+    const GatedKind kind = s.expert_form == ORION_EXPERT_CLAMPED ? kGatedClamped : kGatedSilu;
+    L.moe.act = GatedAct{kind, (float)s.expert_limit}, L.moe.shared_act = GatedAct{kind, (float)s.shared_limit};
+    ORION_TRY(alloc(&L.w_router, (size_t)L.moe.outputs() * H));
+    if (L.moe.softmax) ORION_TRY(alloc(&L.correction, L.moe.outputs()));
     ORION_TRY(alloc(&L.e_up, (size_t)s.experts * 2 * s.ffn_dim * H));
     ORION_TRY(alloc(&L.e_down, (size_t)s.experts * H * s.ffn_dim));
     if (s.shared_dim) {
@@ -167,12 +223,22 @@ int LayeredModel<T>::init_layer(Layer &L) {
     }
     return ORION_OK;
   }
-  ORION_TRY(alloc(&L.w_up, (size_t)s.ffn_dim * H));
-  if (sandwich()) ORION_TRY(zeroed(&L.w_down, H * L.ff_ld));
+  ORION_TRY(alloc(&L.w_up, (size_t)(L.gated_ffn() ? 2 : 1) * s.ffn_dim * H));
+  if (!parallel()) ORION_TRY(zeroed(&L.w_down, H * L.ff_ld));
   if (s.ffn_bias) {
     ORION_TRY(alloc(&L.up_bias, s.ffn_dim));
     ORION_TRY(alloc(&L.down_bias, H));
   }
+  return ORION_OK;
+}
+
+template <typename T>
+int LayeredModel<T>::init_memory(Layer &L) {
+  const size_t copies = 2 * (size_t)d_.num_state_slots, keep = d_.conv_taps ? d_.conv_taps - 1 : 0;
+  if (parallel()) ORION_TRY(zeroed(&L.conv_state, copies * keep * d_.hidden_size));
+  if (L.linear()) ORION_TRY(zeroed(&L.rec_state, copies * L.gla.state_floats()));
+  if (L.d.mixer == ORION_MIXER_MIN_GRU) ORION_TRY(zeroed(&L.rec_state, copies * L.d.width));
+  if (L.cache_elems()) ORION_TRY(zeroed(&L.cache, d_.num_blocks * L.cache_elems()));
   return ORION_OK;
 }
 
@@ -183,14 +249,14 @@ int LayeredModel<T>::init_buffers() {
   const OrionLayeredDesc &d = d_;
   const size_t H = d.hidden_size, rows = d.max_batch_tokens;
   const uint32_t few = (uint32_t)std::min<uint64_t>(rows, (uint64_t)kFewRows * d.max_batch_sequences);
-  size_t cat = 0, qcols = 0, gates = 0, qa = 0;
+  size_t cat = 0, qcols = 0, gates = 0, value_gates = 0, qa = 0;
   struct { size_t choices = 0, histogram = 0, tiles = 0, x = 0, act = 0, up = 0, down = 0; } moe;
   auto grow = [](size_t &a, size_t b) { a = std::max(a, b); };
   for (const Layer &L : layers_) {
     const OrionLayerDesc &s = L.d;
     grow(cat, L.cat);
     const std::pair<uint32_t, uint32_t> products[] = {
-        {L.mix_in, (uint32_t)H}, {(uint32_t)H, L.cat}, {s.experts ? s.experts : s.ffn_dim, (uint32_t)H}, {L.w_down ? (uint32_t)H : 0, L.ff_ld}};
+        {L.mix_in, (uint32_t)H}, {(uint32_t)H, L.cat}, {s.experts ? L.moe.outputs() : (L.gated_ffn() ? 2 : 1) * s.ffn_dim, (uint32_t)H}, {L.w_down ? (uint32_t)H : 0, L.ff_ld}};
     for (const auto &[n, k] : products)
       if (n) grow(partial_floats_, gemm_partial_floats(kBf16, (uint32_t)rows, n, k));
     if (L.w_down) grow(cat, L.ff_ld);
@@ -198,6 +264,7 @@ int LayeredModel<T>::init_buffers() {
     if (L.attention()) {
       grow(qcols, (size_t)s.heads * L.kv.head_dim);
       if (s.head_gate) grow(gates, s.heads);
+      if (s.value_gate) grow(value_gates, (size_t)s.heads * s.value_dim);
     }
     if (tuned(L)) grow(qa, (size_t)few * s.heads * L.ls.kv_cols());
     for (uint32_t r = 1; r <= few; ++r) {
@@ -219,13 +286,14 @@ int LayeredModel<T>::init_buffers() {
     }
   }
   ORION_TRY(alloc(&partial_, partial_floats_));
-  if (!sandwich()) {
+  if (parallel()) {
     ORION_TRY(alloc(&conv_m_, rows * H));
     ORION_TRY(alloc(&conv_f_, rows * H));
   }
   ORION_TRY(zeroed(&cat_, rows * cat));  // columns that nobody writes meet zero weights and must be finite
   ORION_TRY(zeroed(&qbuf_, rows * qcols));  // so must the padding of queries, which meets that of the keys
   ORION_TRY(alloc(&gate_, rows * gates));
+  ORION_TRY(alloc(&value_gate_, rows * value_gates));
   ORION_TRY(alloc(&qa_, qa));
   ORION_TRY(zeroed(&scratch_, scratch_floats_));
   if (moe.choices) {
@@ -258,14 +326,19 @@ bool LayeredModel<T>::place(const std::string &name, Place *p) const {
     p->vec = dst, p->rows = 1, p->cols = n, p->matrix = false, p->fill = fill;
     return dst != nullptr && n > 0;
   };
+  if (name == "loop.step") {
+    vector(loop_step_, H, 0.0f);
+    p->rows = d_.loop_times, p->matrix = true;
+    return loop_step_ != nullptr;
+  }
   if (name == "embed") return matrix(embed_, d_.vocab_size, H);
   if (name == "head") return matrix(head_, d_.vocab_size, H);
   if (name == "final.norm") return vector(final_norm_, H);
   unsigned i = 0;
   int used = 0;
-  if (sscanf(name.c_str(), "l%u.%n", &i, &used) != 1 || used == 0 || i >= layers_.size()) return false;
+  if (sscanf(name.c_str(), "l%u.%n", &i, &used) != 1 || used == 0 || i >= first_run_.size()) return false;
   const std::string rest = name.substr((size_t)used);
-  const Layer &L = layers_[i];
+  const Layer &L = layers_[first_run_[i]];
   const OrionLayerDesc &s = L.d;
   if (rest == "norm1") return vector(L.norm, H);
   if (rest == "norm1b") return vector(L.norm_post, H);
@@ -282,7 +355,8 @@ bool LayeredModel<T>::place(const std::string &name, Place *p) const {
       if (part == "down") return matrix(down, H, ffn);
       return false;
     };
-    if (t == "router") return matrix(L.w_router, s.experts, H);
+    if (t == "router") return matrix(L.w_router, L.moe.outputs(), H);
+    if (t == "correction") return vector(L.correction, L.moe.outputs(), 0.0f);
     if (t.compare(0, 7, "shared.") == 0) return expert(t.substr(7), L.s_up, L.s_down, s.shared_dim);
     unsigned e = 0;
     int at = 0;
@@ -291,8 +365,9 @@ bool LayeredModel<T>::place(const std::string &name, Place *p) const {
       return expert(t.substr((size_t)at), L.e_up + e * 2 * s.ffn_dim * H, L.e_down + e * H * s.ffn_dim, s.ffn_dim);
     }
     if (s.experts > 0 || !L.has_ffn()) return false;
+    if (L.gated_ffn() && t != "down") return expert(t, L.w_up, nullptr, s.ffn_dim);
     if (t == "up") return matrix(L.w_up, s.ffn_dim, H);
-    if (t == "down") return sandwich() ? matrix(L.w_down, H, s.ffn_dim, L.ff_ld) : matrix(L.w_out + L.ff_at, H, s.ffn_dim, L.cat);
+    if (t == "down") return parallel() ? matrix(L.w_out + L.ff_at, H, s.ffn_dim, L.cat) : matrix(L.w_down, H, s.ffn_dim, L.ff_ld);
     if (t == "up.b") return vector(L.up_bias, s.ffn_dim, 0.0f);
     if (t == "down.b") return vector(L.down_bias, H, 0.0f);
     return false;
@@ -305,9 +380,13 @@ bool LayeredModel<T>::place(const std::string &name, Place *p) const {
     if (t == "q") return matrix(L.w_mix, nq, H);
     if (t == "k") return matrix(L.w_mix + nq * H, nk, H);
     if (t == "v") return matrix(L.w_mix + (nq + nk) * H, nv, H);
-    if (t == "g") return s.head_gate && matrix(L.w_mix + (nq + nk + nv) * H, s.heads, H);
-    if (t == "q.norm") return vector(L.q_norm, nq);
-    if (t == "k.norm") return vector(L.k_norm, nk);
+    if (t == "g") return (s.head_gate || s.value_gate) && matrix(L.w_mix + (nq + nk + nv) * H, s.value_gate ? s.heads * s.value_dim : s.heads, H);
+    const bool own = s.qk_norm == ORION_QK_NORM_PER_HEAD;
+    if (t == "q.norm") return vector(L.q_norm, own ? s.dim : nq);
+    if (t == "k.norm") return vector(L.k_norm, own ? s.dim : nk);
+    if (t == "q.b") return vector(L.mix_bias, nq, 0.0f);
+    if (t == "k.b") return vector(L.mix_bias ? L.mix_bias + nq : nullptr, nk, 0.0f);
+    if (t == "v.b") return vector(L.mix_bias ? L.mix_bias + nq + nk : nullptr, nv, 0.0f);
     if (t == "sink") return vector(L.sinks, s.heads, 0.0f);
     return false;
   }
@@ -319,6 +398,18 @@ bool LayeredModel<T>::place(const std::string &name, Place *p) const {
     if (t == "dkv.norm") return vector(L.latent_norm, s.kv_rank);
     if (t == "uk") return matrix(L.w_uk, (uint64_t)s.heads * s.dim, s.kv_rank);
     if (t == "uv") return matrix(L.w_uv, (uint64_t)s.heads * s.value_dim, s.kv_rank);
+    return false;
+  }
+  if (L.linear()) {
+    const uint64_t nq = L.gla.q_cols(), nv = L.gla.v_cols();
+    if (t == "q") return matrix(L.w_mix, nq, H);
+    if (t == "k") return matrix(L.w_mix + nq * H, nq, H);
+    if (t == "v") return matrix(L.w_mix + 2 * nq * H, nv, H);
+    if (t == "g") return matrix(L.w_mix + (2 * nq + nv) * H, nv, H);
+    if (t == "a1") return matrix(L.w_mix + (2 * nq + 2 * nv) * H, s.decay_rank, H);
+    if (t == "a2") return matrix(L.w_decay, nq, s.decay_rank);
+    if (t == "a2.b") return vector(L.mix_bias, nq, 3.0f);  // a randomly initialised model forgets slowly
+    if (t == "norm") return vector(L.out_norm, s.value_dim);
     return false;
   }
   if (t == "z") return matrix(L.w_mix, s.width, H);
@@ -335,12 +426,13 @@ std::vector<std::string> LayeredModel<T>::tensor_names() const {
   auto add = [&](const std::string &name) {
     if (uses_tensor(name.c_str())) names.push_back(name);
   };
-  for (const char *n : {"embed", "head", "final.norm"}) add(n);
+  for (const char *n : {"embed", "head", "final.norm", "loop.step"}) add(n);
   for (uint32_t i = 0; i < d_.num_layers; ++i) {
     const std::string l = "l" + std::to_string(i) + ".";
     for (const char *rest : {"norm1", "norm1b", "norm2", "norm2b", "canon1", "canon2", "mlp.up", "mlp.up.b", "mlp.down", "mlp.down.b", "mlp.router",
                              "mlp.shared.gate", "mlp.shared.up", "mlp.shared.down", "mix.o", "mix.q", "mix.k", "mix.v", "mix.q.norm", "mix.k.norm",
-                             "mix.sink", "mix.dkv", "mix.dkv.norm", "mix.uk", "mix.uv", "mix.g", "mix.z", "mix.x", "mix.z.b", "mix.x.b"})
+                             "mix.sink", "mix.dkv", "mix.dkv.norm", "mix.uk", "mix.uv", "mix.g", "mix.z", "mix.x", "mix.z.b", "mix.x.b", "mlp.gate", "mlp.correction", "mix.q.b", "mix.k.b", "mix.v.b", "mix.norm", "mix.a1",
+                             "mix.a2", "mix.a2.b"})
       add(l + rest);
     for (uint32_t e = 0; e < specs_[i].experts; ++e)
       for (const char *part : {".gate", ".up", ".down"}) add(l + "mlp.e" + std::to_string(e) + part);
@@ -360,8 +452,8 @@ int LayeredModel<T>::load_tensor(const char *name, int dtype, const uint64_t *sh
     return set_error(ORION_ERR_MODEL, "tensor `%s` has shape [%llu, %llu], expected [%llu, %llu]", name, (unsigned long long)R,
                      (unsigned long long)C, (unsigned long long)p.rows, (unsigned long long)p.cols);
   finalized_ = false;
-  if (!p.matrix) {
-    ORION_TRY(upload_slice(nullptr, p.vec, data, dtype, C, 0, 1, 0, C));
+  if (p.vec) {
+    ORION_TRY(upload_slice(nullptr, p.vec, data, dtype, C, 0, R, 0, C));
   } else if (p.ld == C && !p.transposed) {
     ORION_TRY(upload_slice(p.dst, nullptr, data, dtype, C, 0, R, 0, C));
   } else {  // a column block of a wider matrix, or filters
@@ -399,8 +491,8 @@ int LayeredModel<T>::init_random(uint64_t seed, float std) {
   for (const std::string &n : tensor_names()) {
     Place p;
     place(n, &p);
-    if (!p.matrix) {
-      ORION_TRY(set_constant(p.vec, p.cols, p.fill));
+    if (p.vec) {
+      ORION_TRY(set_constant(p.vec, p.rows * p.cols, p.fill));
     } else if (p.ld == p.cols) {
       ORION_TRY(fill_random(p.dst, p.rows * p.cols, seed, n.find(".canon") != std::string::npos ? 0.1f : std));
     } else {
@@ -453,7 +545,7 @@ void LayeredModel<T>::fill_extra(const BatchView &b, uint32_t *w) {
   const uint64_t S = b.num_sequences;
   uint32_t *first = w, *read = w + S + 1, *write = read + S, *few = write + S;
   uint64_t row = 0;
-  few_rows_ = portions_ = 0;
+  few_rows_ = portions_ = gla_chunks_ = gla_portions_ = 0;
   for (TileSet &t : tile_sets_) t.count = 0;
   for (uint64_t s = 0; s < S; ++s) {
     first[s] = (uint32_t)row;
@@ -487,6 +579,35 @@ int LayeredModel<T>::fill_tiles(const BatchView &b, uint32_t *t, typename Base::
       row += n;
     }
     at += 4 * ((size_t)b.num_sequences + b.num_tokens / set.positions + 1);
+  }
+  return fill_gla_chunks(b, t, at);
+}
+
+// The sequences that bring more than a few rows, cut into chunks, and scratch for the largest of the layers that take them.
+template <typename T>
+int LayeredModel<T>::fill_gla_chunks(const BatchView &b, uint32_t *t, size_t at) {
+  if (!DTypeOf<T>::is_bf16) return ORION_OK;
+  gla_at_ = at;
+  auto *portions = reinterpret_cast<GlaPortion *>(t + at);
+  auto *chunks = reinterpret_cast<GlaChunk *>(t + at + 4 * b.num_sequences);
+  uint64_t row = 0;
+  for (uint64_t s = 0; s < b.num_sequences; ++s) {
+    const uint64_t n = b.slot_token_counts[s];
+    if (n > kFewRows) {
+      portions[gla_portions_++] = GlaPortion{(uint32_t)s, gla_chunks_, (uint32_t)((n + kGlaChunk - 1) / kGlaChunk), 0};
+      for (uint64_t i = 0; i < n; i += kGlaChunk)
+        chunks[gla_chunks_++] = GlaChunk{(uint32_t)(row + i), (uint32_t)std::min<uint64_t>(kGlaChunk, n - i), 0, 0};
+    }
+    row += n;
+  }
+  size_t need = 0;
+  for (const Layer &L : layers_)
+    if (L.linear() && gla_chunks_ > 0 && gla_chunks_supported(L.gla)) need = std::max(need, gla_scratch_bytes(L.gla, gla_chunks_, (uint32_t)b.num_tokens));
+  if (need > gla_scratch_bytes_) {
+    if (gla_scratch_) cudaFree(gla_scratch_);  // the previous step has ended
+    gla_scratch_ = nullptr, gla_scratch_bytes_ = 0;
+    ORION_CUDA_CHECK("allocate chunk operands", cudaMalloc(&gla_scratch_, need + need / 4));
+    gla_scratch_bytes_ = need + need / 4;
   }
   return ORION_OK;
 }
@@ -557,8 +678,8 @@ template <typename T>
 int LayeredModel<T>::poll_errors() {
   ORION_TRY(Base::poll_errors());
   if (!DTypeOf<T>::is_bf16) return ORION_OK;
-  bool latent = false, attention = false, experts = false;
-  for (const Layer &L : layers_) latent |= L.latent(), attention |= L.attention(), experts |= L.moe.experts > 0;
+  bool latent = false, attention = false, experts = false, linear = false;
+  for (const Layer &L : layers_) latent |= L.latent(), attention |= L.attention(), experts |= L.moe.experts > 0, linear |= L.linear();
   uint32_t code = 0;
   auto poll = [&](int (*read)(uint32_t *), const char *what) -> int {
     ORION_TRY(read(&code));
@@ -574,6 +695,7 @@ int LayeredModel<T>::poll_errors() {
     ORION_TRY(poll(prefill_tc_poll_error, "prefill attention"));
   }
   if (experts) ORION_TRY(poll(moe_poll_error, "mixture of experts"));
+  if (linear) ORION_TRY(poll(gla_poll_error, "gated linear attention"));
   return ORION_OK;
 }
 

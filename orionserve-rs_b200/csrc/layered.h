@@ -1,10 +1,13 @@
 // Layer-list models: decoders whose layers are listed one by one, each with its own token mixer, feed-forward and sizes.
-// Two kinds of block:
+// Three kinds of block:
 //   parallel  h = norm(x); mixer and feed-forward each read h plus a short causal convolution of h; both results are added to
 //             x. They write their activations next to each other into one buffer and their output matrices are stored side by
 //             side along k, so the two sublayers end in a single projection whose accumulator adds them.
 //   sandwich  x += m * norm(mixer(norm(x))), then x += m * norm(feed-forward(norm(x))): one kernel folds a sublayer's output
 //             projection, normalises it, adds it and normalises the sum for the next sublayer.
+//   prenorm   x += m * mixer(norm(x)), then x += m * feed-forward(norm(x)).
+// A run of layers may be passed through several times (prenorm blocks): the passes share the weights, and each has caches and states
+// of its own, so a pass is simply a further layer of the sequence of layer runs that points to the same weights.
 // What a sequence carries from step to step is the paged cache of its attention layers (latents, or keys and values) and, in a
 // state slot, the recurrences' states and the convolutions' last inputs.
 #pragma once
@@ -36,7 +39,7 @@ class LayeredModel final : public StepModel<T> {
   ~LayeredModel() override {
     cudaSetDevice(ordinal_);
     if (stream_) cudaStreamSynchronize(stream_);
-    for (T *p : {ext_latents_, ext_rot_, ext_kv_})
+    for (void *p : {(void *)ext_latents_, (void *)ext_rot_, (void *)ext_kv_, gla_scratch_})
       if (p) cudaFree(p);
   }
 
@@ -52,6 +55,7 @@ class LayeredModel final : public StepModel<T> {
   int read_kv(float *out, uint64_t capacity) override;
   uint32_t num_state_slots() const override { return has_state() ? d_.num_state_slots : 0; }
   bool logical_positions() const override { return true; }
+  float logit_softcap() const override { return (float)d_.logit_softcap; }
   const OrionModelDesc &desc() const override { return desc_; }
 
  private:
@@ -62,6 +66,10 @@ class LayeredModel final : public StepModel<T> {
     KvLayout kv{};
     AttnForm form{};
     bool tuned = false;  // attention: the sizes the tensor-core kernels take
+    GlaShape gla{};
+    // what joins the stream ahead of this run: a vector (may be null), and what entered the model's first layer
+    const float *shift = nullptr;
+    bool restart = false;
     MoeShape moe{};      // experts = 0: dense feed-forward or none
     // joint mixer projection's columns, mixer output, columns of the feed-forward's activations and of the output projection
     uint32_t mix_in = 0, mix_out = 0, ff_at = 0, cat = 0, ff_ld = 0;
@@ -69,13 +77,17 @@ class LayeredModel final : public StepModel<T> {
     float *norm_post = nullptr, *norm2 = nullptr, *norm2_post = nullptr;  // sandwich block
     float *q_norm = nullptr, *k_norm = nullptr, *sinks = nullptr, *up_bias = nullptr, *down_bias = nullptr;
     T *conv1 = nullptr, *conv2 = nullptr, *w_mix = nullptr, *w_up = nullptr, *w_out = nullptr, *w_down = nullptr, *w_uk = nullptr, *w_uv = nullptr;
+    T *w_decay = nullptr;        // gla: [heads * dim][rank], its bias in mix_bias
+    float *out_norm = nullptr, *correction = nullptr;
     T *w_router = nullptr, *e_up = nullptr, *e_down = nullptr, *s_up = nullptr, *s_down = nullptr;
     T *conv_state = nullptr;     // [2 * slots][taps - 1][hidden]
-    float *rec_state = nullptr;  // [2 * slots][width]
+    float *rec_state = nullptr;  // [2 * slots][width, or a matrix per head]
     T *cache = nullptr;          // latents: [blocks][block_size][row_stride]; keys and values: a KvLayout of one layer
     const float *rope_cos = nullptr, *rope_sin = nullptr;
     bool latent() const { return d.mixer == ORION_MIXER_LATENT_ATTENTION; }
     bool attention() const { return d.mixer == ORION_MIXER_ATTENTION; }
+    bool linear() const { return d.mixer == ORION_MIXER_GLA; }
+    bool gated_ffn() const { return d.activation == ORION_ACT_GEGLU_TANH; }
     bool has_ffn() const { return d.ffn_dim > 0; }
     size_t cache_elems() const { return latent() ? (size_t)ls.block_size * ls.row_stride : (attention() ? kv.num_kv_heads * kv.chunk_elems() : 0); }
   };
@@ -91,13 +103,15 @@ class LayeredModel final : public StepModel<T> {
   std::vector<std::string> tensor_names() const;
   int check_layer(uint32_t i) const;
   int init_layer(Layer &L);
+  int init_memory(Layer &L);  // what a layer run keeps of its sequences
   int init_rope(Layer &L);
   int init_buffers();
   bool sandwich() const { return d_.block == ORION_BLOCK_SANDWICH; }
+  bool parallel() const { return d_.block == ORION_BLOCK_PARALLEL; }
   bool has_state() const {
-    if (!sandwich()) return true;
+    if (parallel()) return true;
     for (const OrionLayerDesc &s : specs_)
-      if (s.mixer == ORION_MIXER_MIN_GRU) return true;
+      if (s.mixer == ORION_MIXER_MIN_GRU || s.mixer == ORION_MIXER_GLA) return true;
     return false;
   }
   template <typename U>
@@ -110,9 +124,10 @@ class LayeredModel final : public StepModel<T> {
   int run_step_body(bool want_argmax, int part) override;
   int run_parallel_layers();
   int run_sandwich_layers();
+  int run_prenorm_layers();
   bool graph_eligible() const override {
     return g_step_graph && DTypeOf<T>::is_bf16 && meta_.decode && !meta_.zero_count && !prof_on_ && only_mask_ == 0 &&
-           (sandwich() || residual_norm_conv_supported(d_.hidden_size, d_.conv_taps));
+           (!parallel() || residual_norm_conv_supported(d_.hidden_size, d_.conv_taps));
   }
   void graph_plan(uint32_t *splits, uint32_t *blocks_per_split) const override {
     // the context splits of every attention layer, folded into one word
@@ -132,10 +147,11 @@ class LayeredModel final : public StepModel<T> {
   size_t tile_words(uint64_t seqs, uint64_t rows) const override {
     size_t n = 4 * (2 * seqs + rows / kLatentTileRows + 1);
     for (const TileSet &s : tile_sets_) n += 4 * (seqs + rows / s.positions + 1);
-    return n;
+    return n + 4 * (2 * seqs + rows / kGlaChunk + 1);
   }
   int fill_tiles(const BatchView &b, uint32_t *t, typename Base::Meta &mt) override;
   int fill_latent_tiles(const BatchView &b, uint32_t *t, typename Base::Meta &mt);
+  int fill_gla_chunks(const BatchView &b, uint32_t *t, size_t at);
   bool expands(const Layer &L) const { return DTypeOf<T>::is_bf16 && L.latent() && latent_prefill_supported(L.ls); }
   bool tuned(const Layer &L) const { return DTypeOf<T>::is_bf16 && L.latent() && latent_decode_supported(L.ls); }
   uint32_t context_splits(const Layer &L, uint32_t rows) const {
@@ -160,6 +176,7 @@ class LayeredModel final : public StepModel<T> {
   int mixer(const Layer &L, const T *x);
   int latent_attention(const Layer &L, const GemmPlan &p, size_t slab);
   int attention(const Layer &L, const GemmPlan &p, size_t slab);
+  int linear_attention(const Layer &L, const GemmPlan &p, size_t slab);
   // The up half of a dense feed-forward, activated: x -> act (row stride ld).
   int dense_up(const Layer &L, const T *x, T *act, uint32_t ld);
   int mixture(const Layer &L, const T *x, SublayerOutput *y);
@@ -167,7 +184,9 @@ class LayeredModel final : public StepModel<T> {
   OrionLayeredDesc d_;
   std::vector<OrionLayerDesc> specs_;
   OrionModelDesc desc_;
-  std::vector<Layer> layers_;
+  std::vector<Layer> layers_;         // in the order in which they run
+  std::vector<uint32_t> first_run_;   // of every layer of the list
+  float *loop_step_ = nullptr;        // [passes][hidden]
   std::vector<std::string> got_;
   float *final_norm_ = nullptr;
   T *head_ = nullptr;                        // an output matrix of its own
@@ -176,6 +195,7 @@ class LayeredModel final : public StepModel<T> {
   T *qbuf_ = nullptr;
   T *qa_ = nullptr;           // queries of decoding rows in the latent space
   float *gate_ = nullptr;     // factors of the heads' outputs
+  T *value_gate_ = nullptr;   // factors of their values
   float *scratch_ = nullptr;  // partial results of decode attention per context split
   size_t scratch_floats_ = 0;
   MoeBuffers<T> moe_;
@@ -189,8 +209,12 @@ class LayeredModel final : public StepModel<T> {
     size_t offset;  // words from the start of the tile metadata
   };
   std::vector<TileSet> tile_sets_;
+  // The same portions in chunks for linear attention: counts, place of the lists in the tile metadata, scratch.
+  uint32_t gla_chunks_ = 0, gla_portions_ = 0;
+  size_t gla_at_ = 0, gla_scratch_bytes_ = 0;
+  void *gla_scratch_ = nullptr;
   struct Rope {
-    double base;
+    double base, factor, original, fast, slow;
     uint32_t dims;
     float *cos, *sin;
   };

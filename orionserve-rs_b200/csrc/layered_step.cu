@@ -11,6 +11,7 @@ int LayeredModel<T>::mixer(const Layer &L, const T *x) {
   ORION_TRY(timed(kProfGemm, [&] { return launch_gemm<T>(x, H, L.w_mix, H, partial_, Tn, L.mix_in, H, p, stream_); }));
   if (L.latent()) return latent_attention(L, p, slab);
   if (L.attention()) return attention(L, p, slab);
+  if (L.linear()) return linear_attention(L, p, slab);
   return timed(kProfAttention, [&] { return launch_min_gru<T>(partial_, p.out_slabs, slab, L.mix_bias, L.rec_state, state_batch(), cat_, L.cat, L.d.width, stream_); });
 }
 
@@ -63,9 +64,11 @@ int LayeredModel<T>::attention(const Layer &L, const GemmPlan &p, size_t slab) {
   const AttnBatch ab = attn_batch();
   AttnForm form = L.form;
   form.gate = L.d.head_gate ? gate_ : nullptr;
+  form.value_gate = L.d.value_gate ? value_gate_ : nullptr;
   ORION_TRY(timed(kProfElementwise, [&] {
     return launch_attention_prepare<T>(partial_, p.out_slabs, slab, L.in, ab.query_positions, d_meta_ + meta_.slot_block, d_meta_ + meta_.slot_slot,
-                                       qbuf_, L.cache, L.kv, 0, L.d.head_gate ? gate_ : nullptr, Tn, stream_);
+                                       qbuf_, L.cache, L.kv, 0, L.d.head_gate ? gate_ : nullptr, Tn, stream_,
+                                       L.d.value_gate ? value_gate_ : nullptr);
   }));
   if constexpr (DTypeOf<T>::is_bf16) {
     if (L.tuned) {
@@ -90,10 +93,45 @@ int LayeredModel<T>::attention(const Layer &L, const GemmPlan &p, size_t slab) {
   return timed(kProfAttention, [&] { return launch_paged_attention_generic<T>(qbuf_, L.cache, L.kv, 0, ab, L.d.heads, cat_, stream_, form); });
 }
 
+// Sequences with few rows go token by token, longer portions in chunks.
+template <typename T>
+int LayeredModel<T>::linear_attention(const Layer &L, const GemmPlan &p, size_t slab) {
+  const GlaWeights<T> w{L.w_decay, L.mix_bias, L.out_norm};
+  uint32_t most = UINT32_MAX;
+  if constexpr (DTypeOf<T>::is_bf16) {
+    if (gla_chunks_supported(L.gla)) {
+      most = kFewRows;
+      if (gla_chunks_ > 0) {
+        const uint32_t *lists = d_meta_ + meta_.tiles + gla_at_;
+        const GlaPortions portions{reinterpret_cast<const GlaChunk *>(lists + 4 * meta_.seqs), reinterpret_cast<const GlaPortion *>(lists), gla_chunks_,
+                                   gla_portions_};
+        ORION_TRY(timed(kProfAttention, [&] {
+          return launch_gla_chunks(partial_, p.out_slabs, slab, L.gla, w, L.rec_state, state_batch(), portions, gla_scratch_, cat_, L.cat, stream_);
+        }));
+      }
+      if (few_rows_ == 0) return ORION_OK;
+    }
+  }
+  return timed(kProfAttention, [&] {
+    return launch_gla_steps<T>(partial_, p.out_slabs, slab, L.gla, w, L.rec_state, state_batch(), most, cat_, L.cat, stream_);
+  });
+}
+
 template <typename T>
 int LayeredModel<T>::dense_up(const Layer &L, const T *x, T *act, uint32_t ld) {
   const uint32_t Tn = meta_.rows, H = d_.hidden_size, F = L.d.ffn_dim;
   const bool relu2 = L.d.activation == ORION_ACT_RELU2;
+  if (L.gated_ffn()) {
+    const GemmPlan p = plan_for(Tn, 2 * F, H, H);
+    if constexpr (DTypeOf<T>::is_bf16) {
+      if (p.tensor_core && p.splits == 1)
+        return timed(kProfGemm, [&] { return launch_gemm_act(x, H, L.w_up, H, act, ld, Tn, 2 * F, H, kGemmGeglu, stream_); });
+    }
+    ORION_TRY(timed(kProfGemm, [&] { return launch_gemm<T>(x, H, L.w_up, H, partial_, Tn, 2 * F, H, p, stream_); }));
+    return timed(kProfElementwise, [&] {
+      return launch_gated_act<T>(partial_, p.out_slabs, (size_t)Tn * 2 * F, GatedAct{kGatedGelu, 0.f}, act, ld, Tn, F, stream_);
+    });
+  }
   const GemmPlan p = plan_for(Tn, F, H, H);
   if constexpr (DTypeOf<T>::is_bf16) {
     if (p.tensor_core && p.splits == 1)  // the activation in the GEMM epilogue: no partials, no extra launch
@@ -110,17 +148,19 @@ int LayeredModel<T>::dense_up(const Layer &L, const T *x, T *act, uint32_t ld) {
 // The rows of x through their experts and the shared one; y names the results.
 template <typename T>
 int LayeredModel<T>::mixture(const Layer &L, const T *x, SublayerOutput *y) {
-  const uint32_t Tn = meta_.rows, H = d_.hidden_size, E = L.moe.experts;
+  const uint32_t Tn = meta_.rows, H = d_.hidden_size, E = L.moe.outputs();
   const GemmPlan rp = plan_for(Tn, E, H, H);
   const MoePlan plan = moe_plan(DTypeOf<T>::is_bf16, L.moe, Tn);
   ORION_TRY(timed(kProfGemm, [&] { return launch_gemm<T>(x, H, L.w_router, H, partial_, Tn, E, H, rp, stream_); }));
-  ORION_TRY(timed(kProfElementwise, [&] { return launch_moe_route<T>(partial_, rp.out_slabs, (size_t)Tn * E, x, L.moe, plan, moe_, Tn, stream_); }));
+  ORION_TRY(timed(kProfElementwise, [&] { return launch_moe_route<T>(partial_, rp.out_slabs, (size_t)Tn * E, L.correction, x, L.moe, plan, moe_, Tn, stream_); }));
   ORION_TRY(timed(kProfGemm, [&] {
     return launch_moe_experts<T>(x, L.e_up, L.e_down, L.s_up, L.s_down, L.moe, plan, moe_, partial_, Tn, stream_);
   }));
   if (L.moe.shared_ffn) y->partial = partial_, y->splits = plan.down_splits, y->split_stride = (size_t)Tn * H;
   y->rows = moe_.down, y->place = moe_.place, y->top = L.moe.top;
   y->rows_splits = plan.down_splits, y->rows_stride = (size_t)Tn * L.moe.top * H;
+  if (L.moe.weigh_output) y->weight = moe_.score;
+  y->identity = x;
   return ORION_OK;
 }
 
@@ -204,8 +244,53 @@ int LayeredModel<T>::run_sandwich_layers() {
 }
 
 template <typename T>
+int LayeredModel<T>::run_prenorm_layers() {
+  const uint32_t Tn = meta_.rows, H = d_.hidden_size;
+  const uint32_t *m = d_meta_, *tokens = m + meta_.tokens;
+  const float eps = (float)d_.norm_eps, mult = (float)d_.residual_mult, scale = (float)d_.embed_scale;
+  ORION_TRY(timed(kProfElementwise, [&] {
+    return launch_embed_rmsnorm<T>(embed_, tokens, layers_[0].norm, eps, hidden_, normed_, Tn, H, stream_, scale, layers_[0].shift);
+  }));
+  // Adds a sublayer's output, and ahead of the layer run `next` what belongs there; the sum is normalised for its reader.
+  auto join = [&](const SublayerOutput &y, const float *norm, const Layer *next) -> int {
+    StreamAddition<T> add;
+    if (next) add = StreamAddition<T>{next->restart ? embed_ : nullptr, tokens, scale, next->shift};
+    return timed(kProfElementwise, [&] { return launch_sublayer_residual<T>(y, hidden_, mult, add, norm, eps, normed_, nullptr, Tn, H, stream_); });
+  };
+  auto finish = [&](const SublayerOutput &y) -> int {
+    if (meta_.outs == 0) return ORION_OK;
+    return timed(kProfElementwise, [&] {
+      return launch_sublayer_residual<T>(y, hidden_, mult, StreamAddition<T>{}, final_norm_, eps, tail_, m + meta_.last_rows, meta_.outs, H, stream_);
+    });
+  };
+  auto projected = [&](const T *x, const T *w, uint32_t k, SublayerOutput *y) -> int {
+    const GemmPlan p = plan_for(Tn, H, k, k);
+    y->partial = partial_, y->splits = p.out_slabs, y->split_stride = (size_t)Tn * H;
+    return timed(kProfGemm, [&] { return launch_gemm<T>(x, k, w, k, partial_, Tn, H, k, p, stream_); });
+  };
+  for (size_t l = 0; l < layers_.size(); ++l) {
+    const Layer &L = layers_[l], *next = l + 1 < layers_.size() ? &layers_[l + 1] : nullptr;
+    SublayerOutput y;
+    ORION_TRY(mixer(L, normed_));
+    ORION_TRY(projected(cat_, L.w_out, L.cat, &y));
+    if (L.has_ffn()) {
+      ORION_TRY(join(y, L.norm2, nullptr));
+      y = SublayerOutput{};
+      if (L.moe.experts) {
+        ORION_TRY(mixture(L, normed_, &y));
+      } else {
+        ORION_TRY(dense_up(L, normed_, cat_, L.ff_ld));
+        ORION_TRY(projected(cat_, L.w_down, L.ff_ld, &y));
+      }
+    }
+    ORION_TRY(next ? join(y, next->norm, next) : finish(y));
+  }
+  return ORION_OK;
+}
+
+template <typename T>
 int LayeredModel<T>::run_step_body(bool want_argmax, int part) {
-  if (part != 2) ORION_TRY(sandwich() ? run_sandwich_layers() : run_parallel_layers());
+  if (part != 2) ORION_TRY(parallel() ? run_parallel_layers() : (sandwich() ? run_sandwich_layers() : run_prenorm_layers()));
   if (part == 1 || meta_.outs == 0) return ORION_OK;
   return run_head(want_argmax);
 }

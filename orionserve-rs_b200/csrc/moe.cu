@@ -1,11 +1,11 @@
 // Mixture of experts: the choice of experts, the order of rows by expert, and the grouped products of the f32 build and of
 // sizes the tensor cores do not take (moe_gemm_tc.cu has the others).
-//   moe_choose_kernel  one warp per row: sigmoid scores of the router's logits, the `top` largest (the lower index of equal
+//   moe_choose_kernel  one warp per row: sigmoid or softmax scores of the router's logits, the `top` largest (the lower index of equal
 //                      ones), and a histogram per block of rows
 //   moe_place_kernel   one warp per row: its places in the order by expert (rows of an expert keep their order, so the order
 //                      does not depend on timing), and the row copied there; the first CTA lists the tiles
 //   moe_route_kernel   both for up to 64 rows, in one cluster
-//   moe_simt_kernel    64 rows x 64 columns of one tile, k ascending, optionally with SwiGLU on the scored products
+//   moe_simt_kernel    64 rows x 64 columns of one tile, k ascending, optionally with the gated activation of the scored products
 //   moe_swiglu_kernel  the same activation on k-split products
 #include "kernels.h"
 #include "mma.cuh"
@@ -20,11 +20,14 @@ __host__ __device__ inline uint32_t row_block(uint32_t rows) { return rows <= 51
 constexpr uint32_t kPlaceRows = 8;
 constexpr uint32_t kClusterRows = 64;  // batches of up to this many rows: one kernel, a cluster of a CTA per 8 rows
 
-// One warp: scores of one row in `mine`, its choices to chosen / score, counted in `count` (shared memory).
-__device__ __forceinline__ void choose_row(const float *__restrict__ logits, uint32_t splits, size_t split_stride, uint32_t experts, uint32_t top,
-                                           float *mine, uint32_t *chosen, float *score, uint32_t *count) {
-  const uint32_t lane = threadIdx.x & 31;
-  for (uint32_t e = lane; e < experts; e += 32) {
+// One warp: scores of one row in `mine`, its choices to chosen / score, those that name an expert with weights counted in `count`
+// (shared memory). The correction takes part in the choice only.
+__device__ __forceinline__ void choose_row(const float *__restrict__ logits, uint32_t splits, size_t split_stride,
+                                           const float *__restrict__ correction, const MoeShape &s, float *mine, uint32_t *chosen, float *score,
+                                           uint32_t *count) {
+  const uint32_t lane = threadIdx.x & 31, outputs = s.outputs();
+  float most = -INFINITY;
+  for (uint32_t e = lane; e < outputs; e += 32) {
     float z = 0.f;
     for (uint32_t s0 = 0; s0 < splits; s0 += 8) {  // eight independent loads in flight
       float x[8];
@@ -33,45 +36,56 @@ __device__ __forceinline__ void choose_row(const float *__restrict__ logits, uin
 #pragma unroll
       for (uint32_t s = 0; s < 8; ++s) z += x[s];
     }
-    mine[e] = sigmoid_f(z);
+    mine[e] = s.softmax ? z : sigmoid_f(z);
+    most = fmaxf(most, z);
+  }
+  if (s.softmax) {
+    most = warp_max(most);
+    float sum = 0.f;
+    for (uint32_t e = lane; e < outputs; e += 32) sum += mine[e] = expf(mine[e] - most);
+    sum = warp_sum(sum);
+    for (uint32_t e = lane; e < outputs; e += 32) mine[e] /= sum;
   }
   __syncwarp();
-  for (uint32_t k = 0; k < top; ++k) {
-    float best = -1.f;
+  for (uint32_t k = 0; k < s.top; ++k) {
+    float best = -INFINITY;
     uint32_t at = 0xFFFFFFFFu;
-    for (uint32_t e = lane; e < experts; e += 32)
-      if (mine[e] > best) best = mine[e], at = e;
+    for (uint32_t e = lane; e < outputs; e += 32) {
+      const float v = correction ? mine[e] + correction[e] : mine[e];
+      if (v > best) best = v, at = e;
+    }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
       const float ov = __shfl_xor_sync(0xffffffffu, best, o);
       const uint32_t oi = __shfl_xor_sync(0xffffffffu, at, o);
       if (ov > best || (ov == best && oi < at)) best = ov, at = oi;
     }
-    if (at >= experts) at = k;  // only if scores are not numbers: stay inside the expert list (top <= experts)
+    if (at >= outputs) at = k;  // only if scores are not numbers: stay inside the router's outputs (top is at most as many)
     __syncwarp();
     if (lane == 0) {
-      mine[at] = -2.f;
       chosen[k] = at;
-      score[k] = best;
-      atomicAdd(&count[at], 1u);
+      score[k] = mine[at];
+      mine[at] = -INFINITY;
+      if (at < s.experts) atomicAdd(&count[at], 1u);
     }
     __syncwarp();
   }
 }
 
 __global__ void __launch_bounds__(1024)
-moe_choose_kernel(const float *__restrict__ logits, uint32_t splits, size_t split_stride, uint32_t experts, uint32_t top, uint32_t rows,
-                  uint32_t *__restrict__ chosen, float *__restrict__ score, uint32_t *__restrict__ histogram) {
-  extern __shared__ float smem[];  // [warps][experts] scores, [experts] counts
-  const uint32_t tid = threadIdx.x, warp = tid >> 5, warps = blockDim.x >> 5, block = row_block(rows);
-  uint32_t *count = reinterpret_cast<uint32_t *>(smem + warps * experts);
+moe_choose_kernel(const float *__restrict__ logits, uint32_t splits, size_t split_stride, const float *__restrict__ correction, MoeShape s,
+                  uint32_t rows, uint32_t *__restrict__ chosen, float *__restrict__ score, uint32_t *__restrict__ histogram) {
+  extern __shared__ float smem[];  // [warps][outputs] scores, [experts] counts
+  const uint32_t tid = threadIdx.x, warp = tid >> 5, warps = blockDim.x >> 5, block = row_block(rows), experts = s.experts, top = s.top,
+                 outputs = s.outputs();
+  uint32_t *count = reinterpret_cast<uint32_t *>(smem + warps * outputs);
   pdl_trigger();
   pdl_wait();
   for (uint32_t e = tid; e < experts; e += blockDim.x) count[e] = 0;
   __syncthreads();
   const uint32_t end = min(rows, (blockIdx.x + 1) * block);
   for (uint32_t row = blockIdx.x * block + warp; row < end; row += warps)
-    choose_row(logits + (size_t)row * experts, splits, split_stride, experts, top, smem + warp * experts, chosen + (size_t)row * top,
+    choose_row(logits + (size_t)row * outputs, splits, split_stride, correction, s, smem + warp * outputs, chosen + (size_t)row * top,
                score + (size_t)row * top, count);
   __syncthreads();
   for (uint32_t e = tid; e < experts; e += blockDim.x) histogram[(size_t)blockIdx.x * experts + e] = count[e];
@@ -146,6 +160,10 @@ moe_place_kernel(const uint32_t *__restrict__ chosen, const float *__restrict__ 
   if (row >= rows) return;
   for (uint32_t k = 0; k < top; ++k) {
     const uint32_t at = row * top + k, e = chosen[at];
+    if (e >= E) {  // an identity expert
+      if (lane == 0) place[at] = kNoPlace;
+      continue;
+    }
     uint32_t rank = 0;  // choices of the same expert before this one in the block of rows
     for (uint32_t j = block * per * top; j < at; j += 32) {
       const uint32_t other = j + lane < at ? chosen[j + lane] : 0xFFFFFFFFu;
@@ -171,12 +189,12 @@ __device__ __forceinline__ uint32_t ld_dsmem_u32(const uint32_t *local, uint32_t
 // distributed shared memory.
 template <typename T>
 __global__ void __launch_bounds__(kPlaceRows * 32)
-moe_route_kernel(const float *__restrict__ logits, uint32_t splits, size_t split_stride, const T *__restrict__ x, MoeShape s, uint32_t rows,
-                 uint32_t tile_rows, uint32_t max_tiles, uint32_t *__restrict__ place, float *__restrict__ row_score, MoeTile *__restrict__ tiles,
-                 T *__restrict__ sorted) {
-  extern __shared__ float smem[];  // [8][experts] scores, then words
-  const uint32_t E = s.experts, top = s.top, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  uint32_t *count = reinterpret_cast<uint32_t *>(smem + kPlaceRows * E), *total = count + E, *before = total + E, *first = before + E,
+moe_route_kernel(const float *__restrict__ logits, uint32_t splits, size_t split_stride, const float *__restrict__ correction,
+                 const T *__restrict__ x, MoeShape s, uint32_t rows, uint32_t tile_rows, uint32_t max_tiles, uint32_t *__restrict__ place,
+                 float *__restrict__ row_score, float *__restrict__ weight, MoeTile *__restrict__ tiles, T *__restrict__ sorted) {
+  extern __shared__ float smem[];  // [8][outputs] scores, then words
+  const uint32_t E = s.experts, R = s.outputs(), top = s.top, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  uint32_t *count = reinterpret_cast<uint32_t *>(smem + kPlaceRows * R), *total = count + E, *before = total + E, *first = before + E,
            *tile_at = first + E, *chosen = tile_at + E;
   float *score = reinterpret_cast<float *>(chosen + kPlaceRows * top);
   pdl_trigger();
@@ -185,7 +203,7 @@ moe_route_kernel(const float *__restrict__ logits, uint32_t splits, size_t split
   pdl_wait();
   const uint32_t row = blockIdx.x * kPlaceRows + warp;
   if (row < rows)
-    choose_row(logits + (size_t)row * E, splits, split_stride, E, top, smem + warp * E, chosen + warp * top, score + warp * top, count);
+    choose_row(logits + (size_t)row * R, splits, split_stride, correction, s, smem + warp * R, chosen + warp * top, score + warp * top, count);
   __syncthreads();
   asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
   asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
@@ -208,6 +226,11 @@ moe_route_kernel(const float *__restrict__ logits, uint32_t splits, size_t split
   if (row < rows) {
     for (uint32_t k = 0; k < top; ++k) {
       const uint32_t at = warp * top + k, e = chosen[at];
+      if (weight && lane == 0) weight[row * top + k] = score[at];
+      if (e >= E) {
+        if (lane == 0) place[row * top + k] = kNoPlace;
+        continue;
+      }
       uint32_t rank = 0;
       for (uint32_t j = 0; j < at; j += 32) {
         const uint32_t other = j + lane < at ? chosen[j + lane] : 0xFFFFFFFFu;
@@ -225,12 +248,6 @@ moe_route_kernel(const float *__restrict__ logits, uint32_t splits, size_t split
   asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
 }
 
-// silu(w g) * (w u): the score of a routed row multiplies what the expert reads.
-template <typename T>
-__device__ __forceinline__ float scored_swiglu(float g, float u, float w) {
-  return silu_for<T>(w * g) * (w * u);
-}
-
 constexpr uint32_t BM = 64, BN = 64, BK = 16;
 template <typename T>
 struct SimtFamily {
@@ -238,6 +255,7 @@ struct SimtFamily {
   uint32_t n, k;
   T *act;
   float *out;
+  GatedAct gate;
 };
 template <typename T, bool SWIGLU>
 __global__ void __launch_bounds__(256)
@@ -280,12 +298,12 @@ moe_simt_kernel(SimtFamily<T> routed, SimtFamily<T> shared, uint32_t shared_tile
     const uint32_t r = ty * 4 + i;
     if (r >= t.count) continue;
     const size_t row = t.row + r;
-    const float score = is_shared || !SWIGLU ? 1.f : row_score[row];
+    const float score = is_shared || !SWIGLU || !row_score ? 1.f : row_score[row];  // multiplies what the expert reads
 #pragma unroll
     for (int j = 0; j < 4; j += SWIGLU ? 2 : 1) {
       const uint32_t n = n0 + tx * 4 + j;
       if (n >= f.n) continue;
-      if (SWIGLU) f.act[row * (f.n / 2) + n / 2] = from_f32<T>(scored_swiglu<T>(acc[i][j], acc[i][j + (SWIGLU ? 1 : 0)], score));
+      if (SWIGLU) f.act[row * (f.n / 2) + n / 2] = from_f32<T>(gated<T>(f.gate, score * acc[i][j], score * acc[i][j + (SWIGLU ? 1 : 0)]));
       else f.out[row * f.n + n] = acc[i][j];
     }
   }
@@ -307,7 +325,8 @@ moe_swiglu_kernel(const float *__restrict__ up, uint32_t splits, MoeShape s, uin
       const float2 q = p[k * stride / 2];
       v.x += q.x, v.y += q.y;
     }
-    act[i] = from_f32<T>(scored_swiglu<T>(v.x, v.y, is_shared ? 1.f : row_score[i / s.ffn]));
+    const float w = is_shared || !row_score ? 1.f : row_score[i / s.ffn];
+    act[i] = from_f32<T>(gated<T>(is_shared ? s.shared_act : s.act, w * v.x, w * v.y));
   }
 }
 
@@ -353,25 +372,27 @@ size_t moe_up_floats(bool is_bf16, MoeShape s, uint32_t rows) {
 }
 
 template <typename T>
-int launch_moe_route(const float *logits, uint32_t splits, size_t split_stride, const T *x, MoeShape s, MoePlan plan, MoeBuffers<T> b,
-                     uint32_t rows, cudaStream_t stream) {
+int launch_moe_route(const float *logits, uint32_t splits, size_t split_stride, const float *correction, const T *x, MoeShape s, MoePlan plan,
+                     MoeBuffers<T> b, uint32_t rows, cudaStream_t stream) {
   if (rows == 0) return ORION_OK;
-  if (s.experts == 0 || s.experts > kMoeMaxExperts || s.top == 0 || s.top > s.experts)
-    return set_error(ORION_ERR_INTERNAL, "routing of %u among %u experts is not supported (at most %u)", s.top, s.experts, kMoeMaxExperts);
+  const uint32_t outputs = s.outputs();
+  if (s.experts == 0 || outputs > kMoeMaxExperts || s.top == 0 || s.top > outputs)
+    return set_error(ORION_ERR_INTERNAL, "routing of %u among %u experts is not supported (at most %u)", s.top, outputs, kMoeMaxExperts);
   if (rows <= kClusterRows) {
     const uint32_t ctas = (rows + kPlaceRows - 1) / kPlaceRows;
-    const size_t smem = ((kPlaceRows + 5) * (size_t)s.experts + 2 * kPlaceRows * s.top) * 4;
+    const size_t smem = (kPlaceRows * (size_t)outputs + 5 * (size_t)s.experts + 2 * kPlaceRows * s.top) * 4;
     static bool attr_set[kMaxDeviceOrdinals] = {};
     ORION_CUDA_CHECK("moe_route attr", ensure_dynamic_smem(moe_route_kernel<T>, ((kPlaceRows + 5) + 2 * kPlaceRows) * kMoeMaxExperts * 4, attr_set));
     ORION_CUDA_CHECK("moe_route", launch_pdl_cluster(moe_route_kernel<T>, dim3(ctas), dim3(kPlaceRows * 32), dim3(ctas), smem, stream, logits, splits,
-                                                     split_stride, x, s, rows, plan.tile_rows, plan.tiles, b.place, b.row_score, b.tiles, b.x));
+                                                     split_stride, correction, x, s, rows, plan.tile_rows, plan.tiles, b.place, b.row_score,
+                                                     s.weigh_output ? b.score : nullptr, b.tiles, b.x));
     return after_launch("moe_route");
   }
   const uint32_t block = row_block(rows), threads = block == 8 ? 256 : 1024;
   static bool attr_set[kMaxDeviceOrdinals] = {};
   ORION_CUDA_CHECK("moe_choose attr", ensure_dynamic_smem(moe_choose_kernel, 33 * kMoeMaxExperts * (int)sizeof(float), attr_set));
   ORION_CUDA_CHECK("moe_choose", launch_pdl(moe_choose_kernel, dim3((rows + block - 1) / block), dim3(threads),
-                                            (threads / 32 + 1) * s.experts * sizeof(float), stream, logits, splits, split_stride, s.experts, s.top,
+                                            (threads / 32 * outputs + s.experts) * sizeof(float), stream, logits, splits, split_stride, correction, s,
                                             rows, b.chosen, b.score, b.histogram));
   ORION_TRY(after_launch("moe_choose"));
   ORION_CUDA_CHECK("moe_place", launch_pdl(moe_place_kernel<T>, dim3((rows + kPlaceRows - 1) / kPlaceRows), dim3(kPlaceRows * 32),
@@ -382,12 +403,13 @@ int launch_moe_route(const float *logits, uint32_t splits, size_t split_stride, 
 
 namespace {
 template <typename T>
-int launch_simt(bool swiglu, SimtFamily<T> routed, SimtFamily<T> shared, MoePlan plan, const MoeBuffers<T> &b, uint32_t rows, cudaStream_t stream) {
+int launch_simt(bool swiglu, SimtFamily<T> routed, SimtFamily<T> shared, MoePlan plan, const MoeBuffers<T> &b, const float *row_score, uint32_t rows,
+                cudaStream_t stream) {
   const uint32_t shared_tiles = shared.n ? (rows + BM - 1) / BM : 0;
   const dim3 grid((std::max(routed.n, shared.n) + BN - 1) / BN, shared_tiles + plan.tiles);
   auto kernel = swiglu ? moe_simt_kernel<T, true> : moe_simt_kernel<T, false>;
   ORION_CUDA_CHECK("moe_simt", launch_pdl(kernel, grid, dim3(256), 0, stream, routed, shared, shared_tiles, rows, (const MoeTile *)b.tiles,
-                                          (const float *)b.row_score));
+                                          row_score));
   return after_launch("moe_simt");
 }
 }  // namespace
@@ -397,18 +419,19 @@ int launch_moe_experts(const T *x, const T *w_up, const T *w_down, const T *shar
                        MoeBuffers<T> b, float *shared_out, uint32_t rows, cudaStream_t stream) {
   if (rows == 0) return ORION_OK;
   const size_t sorted = (size_t)rows * s.top;
+  const float *row_score = s.weigh_output ? nullptr : b.row_score;
   T *shared_act = b.act + sorted * s.ffn;
   if constexpr (sizeof(T) == 2) {
     if (plan.tensor_core) {
       const bool fused = plan.up_splits == 1;
       float *shared_up_out = fused ? nullptr : b.up + plan.up_splits * sorted * 2 * s.ffn;
-      MoeProduct p{b.x, w_up, x, shared_up, 2 * s.ffn, s.hidden, 2 * s.shared_ffn, s.hidden, (uint32_t)sorted, rows, s.experts, b.tiles, b.row_score,
-                   b.act, shared_act, fused ? nullptr : b.up, shared_up_out};
+      MoeProduct p{b.x, w_up, x, shared_up, 2 * s.ffn, s.hidden, 2 * s.shared_ffn, s.hidden, (uint32_t)sorted, rows, s.experts, b.tiles, row_score,
+                   b.act, shared_act, fused ? nullptr : b.up, shared_up_out, s.act, s.shared_act};
       ORION_TRY(launch_moe_product_tc(p, fused, plan.up_splits, plan, stream));
       if (!fused) {
         const size_t n = sorted * s.ffn + (size_t)rows * s.shared_ffn;
         ORION_CUDA_CHECK("moe_swiglu", launch_pdl(moe_swiglu_kernel<T>, dim3((uint32_t)std::min<size_t>((n + 255) / 256, 148 * 8)), dim3(256), 0, stream,
-                                                  (const float *)b.up, plan.up_splits, s, rows, (const float *)b.row_score, b.act));
+                                                  (const float *)b.up, plan.up_splits, s, rows, row_score, b.act));
         ORION_TRY(after_launch("moe_swiglu"));
       }
       MoeProduct d{b.act, w_down, shared_act, shared_down, s.hidden, s.ffn, s.shared_ffn ? s.hidden : 0, s.shared_ffn, (uint32_t)sorted, rows, s.experts,
@@ -416,14 +439,14 @@ int launch_moe_experts(const T *x, const T *w_up, const T *w_down, const T *shar
       return launch_moe_product_tc(d, false, plan.down_splits, plan, stream);
     }
   }
-  ORION_TRY(launch_simt<T>(true, {b.x, w_up, 2 * s.ffn, s.hidden, b.act, nullptr}, {x, shared_up, 2 * s.shared_ffn, s.hidden, shared_act, nullptr}, plan,
-                           b, rows, stream));
+  ORION_TRY(launch_simt<T>(true, {b.x, w_up, 2 * s.ffn, s.hidden, b.act, nullptr, s.act},
+                           {x, shared_up, 2 * s.shared_ffn, s.hidden, shared_act, nullptr, s.shared_act}, plan, b, row_score, rows, stream));
   return launch_simt<T>(false, {b.act, w_down, s.hidden, s.ffn, nullptr, b.down},
-                        {shared_act, shared_down, s.shared_ffn ? s.hidden : 0, s.shared_ffn, nullptr, shared_out}, plan, b, rows, stream);
+                        {shared_act, shared_down, s.shared_ffn ? s.hidden : 0, s.shared_ffn, nullptr, shared_out}, plan, b, nullptr, rows, stream);
 }
 
 #define ORION_INSTANTIATE(T)                                                                                                            \
-  template int launch_moe_route<T>(const float *, uint32_t, size_t, const T *, MoeShape, MoePlan, MoeBuffers<T>, uint32_t, cudaStream_t); \
+  template int launch_moe_route<T>(const float *, uint32_t, size_t, const float *, const T *, MoeShape, MoePlan, MoeBuffers<T>, uint32_t, cudaStream_t); \
   template int launch_moe_experts<T>(const T *, const T *, const T *, const T *, const T *, MoeShape, MoePlan, MoeBuffers<T>, float *,    \
                                      uint32_t, cudaStream_t);
 ORION_INSTANTIATE(float)

@@ -7,7 +7,7 @@
 //              preceding kernel has ended; the others once the tile list is there)
 //   warp 2     one lane does the same with the tile's rows
 //   warp 1     allocates tensor memory, one lane issues the MMAs
-//   warps 4-7  epilogue: f32 rows, or silu(w g) * (w u) of neighbouring gate and up rows with the row's score w
+//   warps 4-7  epilogue: f32 rows, or f(w g) * (w u), f a gated activation, of neighbouring gate and up rows with the row's score w
 // Every wait is bounded; a wait that runs out sets the device error word and the CTA still frees its tensor memory.
 #include "kernels.h"
 #include "tcgen05.cuh"
@@ -40,6 +40,7 @@ struct TcArgs {
   const float *row_score;
   bf16 *act, *shared_act;
   float *out, *shared_out;
+  GatedAct f, shared_f;
 };
 
 template <int TOKN, int WST, int XST, int MT, bool SWIGLU>
@@ -164,9 +165,9 @@ moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
             const uint32_t recv = __shfl_xor_sync(0xffffffffu, send, 1);
             const uint32_t r = c + 2 * jj + odd;
             if (r >= tile.count || nn >= n) continue;
-            const float w = shared ? 1.f : a.row_score[tile.row + r];
+            const float w = shared || !a.row_score ? 1.f : a.row_score[tile.row + r];
             const float g = w * __uint_as_float(odd ? recv : rr[b][2 * jj]), u = w * __uint_as_float(odd ? rr[b][2 * jj + 1] : recv);
-            act[(size_t)(tile.row + r) * ffn + f] = __float2bfloat16_rn(silu_for<bf16>(g) * u);
+            act[(size_t)(tile.row + r) * ffn + f] = __float2bfloat16_rn(gated<bf16>(shared ? a.shared_f : a.f, g, u));
           }
         } else if (nn < n) {
 #pragma unroll
@@ -218,7 +219,7 @@ int launch_product(const MoeProduct &p, bool swiglu, uint32_t splits, MoePlan pl
     ORION_TRY(matrix_map(p.shared_x, p.rows, p.shared_k, TOKN, &msx));
   }
   const uint32_t shared_tiles = p.shared_n ? (p.rows + TOKN - 1) / TOKN : 0;
-  const TcArgs a{p.n, p.k, p.shared_n, p.shared_k, shared_tiles, p.rows, p.sorted_rows, splits, p.tiles, p.row_score, p.act, p.shared_act, p.out, p.shared_out};
+  const TcArgs a{p.n, p.k, p.shared_n, p.shared_k, shared_tiles, p.rows, p.sorted_rows, splits, p.tiles, p.row_score, p.act, p.shared_act, p.out, p.shared_out, p.f, p.shared_f};
   const dim3 grid((std::max(p.n, p.shared_n) + MT * kTileN - 1) / (MT * kTileN), shared_tiles + plan.tiles, splits);
   static bool attr_set[2][kMaxDeviceOrdinals] = {};
   auto kernel = swiglu ? moe_gemm_tc_kernel<TOKN, WST, XST, MT, true> : moe_gemm_tc_kernel<TOKN, WST, XST, MT, false>;

@@ -88,6 +88,7 @@ class StepModel : public ModelBase {
   virtual void fill_extra(const BatchView &, uint32_t *) {}
   virtual void step_done(const BatchView &) {}  // the step of a batch was launched and ended without an error
   virtual void step_failed() {}
+  virtual float logit_softcap() const { return 0.f; }  // logits become cap * tanh(logit / cap); 0 = they stay
   virtual bool leader() const { return true; }  // only the leader of a group returns logits (Rank::is_leader)
   virtual bool out_rows_fixed() const { return false; }  // the output buffers cannot move (peers hold their address)
   // Device error words set by bounded waits that ran out.
@@ -389,6 +390,10 @@ int StepModel<T>::run_head(bool want_argmax) {
   GemmPlan hp = gemm_plan(kBf16, S, V, H, H, H);
   hp.splits = hp.out_slabs = 1, hp.cluster_reduce = false;  // logits are written in place, row-major [S][V]
   head_chunks_ = 0;
+  auto cap = [&](uint32_t n0, uint32_t n) -> int {
+    const float c = logit_softcap();
+    return c == 0.f ? ORION_OK : timed(kProfElementwise, [&] { return launch_softcap(logits_ + n0, S, n, V, c, stream_); });
+  };
   if (kBf16 && hp.tensor_core && V >= 4 * 8192 && !want_argmax) {
     // A large vocabulary goes out in column blocks, an event after each: forward() copies block i
     // to the host (copy engine, second stream) while block i + 1 is being computed.
@@ -398,6 +403,7 @@ int StepModel<T>::run_head(bool want_argmax) {
       GemmPlan cp = hp;
       cp.ldc = V;
       ORION_TRY(timed(kProfGemm, [&] { return launch_gemm<T>(tail_, H, lm_head_ + (size_t)n0 * H, H, logits_ + n0, S, nn, H, cp, stream_); }));
+      ORION_TRY(cap(n0, nn));
       ORION_CUDA_CHECK("lm head", cudaEventRecord(head_ev_[c], stream_));
       head_off_[c] = n0;
       head_cols_[c] = nn;
@@ -406,6 +412,7 @@ int StepModel<T>::run_head(bool want_argmax) {
     return ORION_OK;
   }
   ORION_TRY(timed(kProfGemm, [&] { return launch_gemm<T>(tail_, H, lm_head_, H, logits_, S, V, H, hp, stream_); }));
+  ORION_TRY(cap(0, V));
   if (want_argmax) ORION_TRY(timed(kProfElementwise, [&] { return launch_argmax(logits_, S, V, argmax_, stream_); }));
   return ORION_OK;
 }

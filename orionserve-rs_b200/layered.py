@@ -1,31 +1,53 @@
 """``CudaLayeredModel`` — decoders whose configuration lists their layers one by one, each with its own token
-mixer, feed-forward and sizes (``OrionLayeredDesc`` in include/orion_cuda.h) — and the readers of Metapel's and Zulozen's
-``config.json``."""
+mixer, feed-forward and sizes (``OrionLayeredDesc`` in include/orion_cuda.h) — and the readers of Metapel's, Zulozen's and
+Belizen's ``config.json``."""
 from __future__ import annotations
 
 import ctypes as C
 import json
 import os
 from dataclasses import dataclass, field
-from typing import List, Optional
+from typing import Dict, List, Optional, Tuple
 
 import numpy as np
 
 from . import _ffi
 from .backend import CudaBackend
 from .errors import ModelError, check
-from .model import CudaModel
+from .model import CudaModel, safetensors_shapes
 from .types import DType
 
 
-MIXERS = {"mingru": _ffi.MIXER_MIN_GRU, "latent_attention": _ffi.MIXER_LATENT_ATTENTION, "attention": _ffi.MIXER_ATTENTION}
-ACTIVATIONS = {"gelu_tanh": _ffi.ACT_GELU_TANH, "relu2": _ffi.ACT_RELU2}
-BLOCKS = {"parallel": _ffi.BLOCK_PARALLEL, "sandwich": _ffi.BLOCK_SANDWICH}
+MIXERS = {"mingru": _ffi.MIXER_MIN_GRU, "latent_attention": _ffi.MIXER_LATENT_ATTENTION, "attention": _ffi.MIXER_ATTENTION,
+          "gla": _ffi.MIXER_GLA}
+ACTIVATIONS = {"gelu_tanh": _ffi.ACT_GELU_TANH, "relu2": _ffi.ACT_RELU2, "geglu_tanh": _ffi.ACT_GEGLU_TANH}
+BLOCKS = {"parallel": _ffi.BLOCK_PARALLEL, "sandwich": _ffi.BLOCK_SANDWICH, "prenorm": _ffi.BLOCK_PRENORM}
+QK_NORMS = {False: _ffi.QK_NORM_NONE, True: _ffi.QK_NORM_ALL_HEADS, "per_head": _ffi.QK_NORM_PER_HEAD}
+ROUTERS = {"sigmoid_input": _ffi.ROUTER_SIGMOID_INPUT, "softmax": _ffi.ROUTER_SOFTMAX}
+EXPERT_FORMS = {"swiglu": _ffi.EXPERT_SWIGLU, "clamped": _ffi.EXPERT_CLAMPED}
+
+
+@dataclass(frozen=True)
+class Yarn:
+    """Frequencies stretched by ``factor`` where they turn few times within ``original`` positions (``slow`` turns: wholly,
+    ``fast`` turns: not at all)."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+
+@dataclass(frozen=True)
+class Loop:
+    """Layers ``start`` to ``stop - 1`` run ``times`` times in a row; each pass keeps a cache and state of its own."""
+    start: int
+    stop: int
+    times: int
 
 
 @dataclass(frozen=True)
 class LayerSpec:
-    """One layer: its mixer ("mingru", "latent_attention" or "attention"), the mixer's sizes, its feed-forward (0 = none)."""
+    """One layer: its mixer ("mingru", "latent_attention", "attention" or "gla"), the mixer's sizes, its feed-forward (0 = none)."""
     mixer: str
     ffn_dim: int = 0
     # mingru
@@ -43,7 +65,7 @@ class LayerSpec:
     # attention; chunk 0 = no chunks
     kv_heads: int = 0
     chunk: int = 0
-    qk_norm: bool = False
+    qk_norm: object = False  # False, True (over all heads at once) or "per_head"
     sinks: bool = False
     head_gate: bool = False
     # dense feed-forward
@@ -53,13 +75,33 @@ class LayerSpec:
     experts: int = 0
     experts_per_token: int = 0
     shared_dim: int = 0
+    # attention: first positions seen besides the window, pairs of dimensions half the rotated size apart, biases of q, k and v, a
+    # gate per value, soft cap of the scores (0 = none)
+    keep_first: int = 0
+    rope_halves: bool = False
+    qkv_bias: bool = False
+    value_gate: bool = False
+    softcap: float = 0.0
+    yarn: Optional[Yarn] = None
+    # gla (heads, dim and value_dim as above)
+    decay_tau: float = 0.0
+    decay_rank: int = 0
+    # router and experts
+    router: str = "sigmoid_input"
+    router_identity: int = 0
+    expert_form: str = "swiglu"
+    expert_limit: float = 0.0
+    shared_limit: float = 0.0
 
     def _c(self) -> "_ffi.OrionLayerDesc":
         return _ffi.OrionLayerDesc(
             MIXERS[self.mixer], self.ffn_dim, self.width, self.heads, self.dim, self.rot_dim, self.value_dim, self.kv_rank,
-            self.window, self.rope_dims, self.rope_base, self.scale, self.kv_heads, self.chunk, int(self.qk_norm),
+            self.window, self.rope_dims, self.rope_base, self.scale, self.kv_heads, self.chunk, QK_NORMS[self.qk_norm],
             int(self.sinks), int(self.head_gate), ACTIVATIONS[self.activation], int(self.ffn_bias), self.experts,
-            self.experts_per_token, self.shared_dim)
+            self.experts_per_token, self.shared_dim, self.keep_first, int(self.rope_halves), int(self.qkv_bias),
+            int(self.value_gate), self.softcap, *((y.factor, y.original, y.fast, y.slow) if (y := self.yarn) else (0.0,) * 4),
+            self.decay_tau, self.decay_rank, ROUTERS[self.router], self.router_identity, EXPERT_FORMS[self.expert_form],
+            self.expert_limit, self.shared_limit)
 
     def cache_values_per_token(self) -> int:
         if self.mixer == "latent_attention":
@@ -80,23 +122,35 @@ class LayeredMetadata:
     eos_token_ids: List[int] = field(default_factory=list)
     block: str = "parallel"
     untied_lm_head: bool = False
-    residual_mult: float = 1.0  # sandwich blocks
+    residual_mult: float = 1.0  # sandwich and prenorm blocks
+    embed_scale: float = 1.0
+    logit_softcap: float = 0.0
+    loop: Optional[Loop] = None
 
     @property
     def num_layers(self) -> int:
         return len(self.layers)
 
+    def layer_runs(self) -> List[LayerSpec]:
+        """The layers in the order in which they run; a looped layer comes once per pass."""
+        if self.loop is None:
+            return list(self.layers)
+        a, b = self.loop.start, self.loop.stop
+        return self.layers[:a] + self.layers[a:b] * self.loop.times + self.layers[b:]
+
     def cache_values_per_token(self) -> int:
-        """Values the paged cache holds per token, over all layers."""
-        return sum(s.cache_values_per_token() for s in self.layers)
+        """Values the paged cache holds per token, over all layer runs."""
+        return sum(s.cache_values_per_token() for s in self.layer_runs())
 
     @classmethod
-    def from_config(cls, config: dict, name: str = "model") -> "LayeredMetadata":
-        """The ``config.json`` of any design in ``READERS``."""
+    def from_config(cls, config: dict, name: str = "model",
+                    shapes: Optional[Dict[str, Tuple[int, ...]]] = None) -> "LayeredMetadata":
+        """The ``config.json`` of any design in ``READERS``. ``shapes``: the checkpoint's tensors, for the sizes that no
+        configuration gives."""
         try:
             if config["architecture"] not in READERS:
                 raise ModelError(f"unsupported architecture {config['architecture']}")
-            return READERS[config["architecture"]](config, name)
+            return READERS[config["architecture"]](config, name, shapes or {})
         except (KeyError, TypeError, ValueError) as e:
             raise ModelError(f"config.json is malformed: {type(e).__name__}: {e}") from e
 
@@ -110,10 +164,10 @@ class LayeredMetadata:
             raise ModelError(f"{path}: {e}") from e
         except ValueError as e:
             raise ModelError(f"config.json is malformed: {e}") from e
-        return cls.from_config(config, os.path.basename(os.path.normpath(directory)) or "model")
+        return cls.from_config(config, os.path.basename(os.path.normpath(directory)) or "model", safetensors_shapes(directory))
 
 
-def _read_metapel(config: dict, name: str) -> LayeredMetadata:
+def _read_metapel(config: dict, name: str, shapes: dict) -> LayeredMetadata:
     specs = [_metapel_layer(i, entry) for i, entry in enumerate(config["layers"])]
     return LayeredMetadata(architecture=config["architecture"], name=name, hidden_size=int(config["width"]),
                            vocab_size=int(config["vocab"]), layers=specs, norm_eps=float(config["norm"]["eps"]),
@@ -136,7 +190,7 @@ def _metapel_layer(i: int, entry: dict) -> LayerSpec:
     raise ModelError(f"unsupported mixer {kind!r} in layer {i}")
 
 
-def _read_zulozen(config: dict, name: str) -> LayeredMetadata:
+def _read_zulozen(config: dict, name: str, shapes: dict) -> LayeredMetadata:
     specs = [_zulozen_layer(i, entry) for i, entry in enumerate(config["layers"])]
     return LayeredMetadata(architecture=config["architecture"], name=name, hidden_size=int(config["width"]),
                            vocab_size=int(config["vocab"]), layers=specs, norm_eps=float(config["norm"]["eps"]),
@@ -162,12 +216,56 @@ def _zulozen_layer(i: int, entry: dict) -> LayerSpec:
                      qk_norm=True, sinks=True, head_gate=True, **ffn)
 
 
+def _read_belizen(config: dict, name: str, shapes: dict) -> LayeredMetadata:
+    specs = [_belizen_layer(i, entry, shapes) for i, entry in enumerate(config["layers"])]
+    loop = config.get("loop")
+    if loop is not None:
+        loop = Loop(int(loop["start"]), int(loop["stop"]), int(loop["times"]))
+        if not 0 <= loop.start < loop.stop <= len(specs) or loop.times < 1:
+            raise ModelError(f"layers {loop.start} to {loop.stop} of {len(specs)} cannot be looped {loop.times} times")
+    return LayeredMetadata(architecture=config["architecture"], name=name, hidden_size=int(config["width"]),
+                           vocab_size=int(config["vocab"]), layers=specs, norm_eps=float(config["norm"]["eps"]),
+                           block="prenorm", residual_mult=float(config["residual_mult"]),
+                           embed_scale=float(config["embedding"]["scale"]), logit_softcap=float(config.get("logit_softcap") or 0.0),
+                           loop=loop)
+
+
+def _belizen_layer(i: int, entry: dict, shapes: dict) -> LayerSpec:
+    kind, m, mlp = entry["type"], entry["mixer"], entry["mlp"]
+    ffn = {}
+    if mlp is not None and mlp["kind"] == "dense":
+        ffn = dict(ffn_dim=int(mlp["ff"]), activation="geglu_tanh")
+    elif mlp is not None and mlp["kind"] == "moe":
+        router, shared = mlp["router"], mlp.get("shared")
+        ffn = dict(ffn_dim=int(mlp["expert"]["ff"]), experts=int(router["experts"]), experts_per_token=int(router["top"]),
+                   router="softmax", router_identity=int(router.get("identity") or 0), expert_form="clamped",
+                   expert_limit=float(mlp["expert"]["limit"]), shared_dim=int(shared["ff"]) if shared else 0,
+                   shared_limit=float(shared["limit"]) if shared else 0.0)
+    elif mlp is not None:
+        raise ModelError(f"unsupported feed-forward {mlp['kind']!r} in layer {i}")
+    if kind == "gla":
+        if f"l{i}.mix.a1" not in shapes:
+            raise ModelError(f"missing tensor `l{i}.mix.a1`: its rows are the rank of the decays of layer {i}")
+        return LayerSpec("gla", heads=int(m["heads"]), dim=int(m["dim"]), value_dim=int(m["vdim"]), decay_tau=float(m["tau"]),
+                         decay_rank=int(shapes[f"l{i}.mix.a1"][0]), **ffn)
+    if kind != "attention":
+        raise ModelError(f"unsupported mixer {kind!r} in layer {i}")
+    rot, mask = m.get("rot") or {"dims": 0, "base": 1.0}, m.get("mask") or {}
+    yarn = rot.get("scaling")
+    if yarn is not None:
+        yarn = Yarn(float(yarn["factor"]), float(yarn["original"]), float(yarn["fast"]), float(yarn["slow"]))
+    return LayerSpec("attention", heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), value_dim=int(m["vdim"]),
+                     window=_mask_size(m), keep_first=int(mask.get("keep_first") or 0), rope_dims=int(rot["dims"]),
+                     rope_base=float(rot["base"]), yarn=yarn, rope_halves=True, scale=float(m["scale"]),
+                     softcap=float(m.get("softcap") or 0.0), qk_norm="per_head", qkv_bias=True, value_gate=True, **ffn)
+
+
 def _mask_size(mixer: dict) -> int:
     return int(mixer["mask"]["size"]) if mixer.get("mask") else 0
 
 
 #: config.json "architecture" -> reader
-READERS = {"Metapel": _read_metapel, "Zulozen": _read_zulozen}
+READERS = {"Metapel": _read_metapel, "Zulozen": _read_zulozen, "Belizen": _read_belizen}
 
 
 class CudaLayeredModel(CudaModel):
@@ -185,7 +283,8 @@ class CudaLayeredModel(CudaModel):
             meta.hidden_size, meta.vocab_size, meta.num_layers, layers, meta.norm_eps, meta.conv_taps,
             max_positions or num_blocks * block_size,  # no sequence is longer than the whole cache
             num_blocks, block_size, num_state_slots or max_batch_sequences, int(compute_dtype), max_batch_tokens,
-            max_batch_sequences, BLOCKS[meta.block], int(meta.untied_lm_head), meta.residual_mult)
+            max_batch_sequences, BLOCKS[meta.block], int(meta.untied_lm_head), meta.residual_mult, meta.embed_scale,
+            meta.logit_softcap, *((meta.loop.start, meta.loop.stop, meta.loop.times) if meta.loop else (0, 0, 0)))
         check(_ffi.lib().orion_cuda_model_create_layered(backend._h, C.byref(d), C.byref(self._h)))
 
     @classmethod
@@ -203,10 +302,10 @@ class CudaLayeredModel(CudaModel):
         return m
 
     def read_kv(self) -> List[np.ndarray]:
-        """The caches of the attention layers in f32, one after the other: latents as ``[block][slot][kv_rank + rot_dim]``, keys
+        """The caches of the attention layers in f32, one after the other in the order in which they run: latents as ``[block][slot][kv_rank + rot_dim]``, keys
         and values as two arrays ``[block][kv head][slot][dim]``."""
         shapes = []
-        for s in self._meta.layers:
+        for s in self._meta.layer_runs():
             if s.mixer == "latent_attention":
                 shapes.append((self.num_blocks, self.block_size, s.kv_rank + s.rot_dim))
             elif s.mixer == "attention":

@@ -21,24 +21,41 @@ _ST_DTYPES = {"F32": (DType.F32, np.float32), "F16": (DType.F16, np.uint16),
               "BF16": (DType.BF16, np.uint16)}
 
 
-def read_safetensors(path: str) -> Dict[str, Tuple[DType, Tuple[int, ...], np.ndarray]]:
-    """Minimal safetensors reader: 8-byte LE header length, JSON header, raw LE data.
-    Returns name -> (dtype, shape, flat array view); 16-bit floats come back as uint16 bits."""
-    data = np.memmap(path, dtype=np.uint8, mode="r")
-    if data.size < 8:
+def safetensors_header(data: bytes, path: str) -> Tuple[dict, int]:
+    """The JSON header at the start of ``data`` (bytes or a mapping of a whole file) and the offset of the tensors."""
+    if len(data) < 8:
         raise ModelError(f"{path} is malformed: shorter than its header length")
     (hlen,) = struct.unpack("<Q", bytes(data[:8]))
-    if 8 + hlen > data.size:
+    if 8 + hlen > len(data):
         raise ModelError(f"{path} is malformed: header length {hlen} exceeds the file")
     try:
         header = json.loads(bytes(data[8:8 + hlen]).decode("utf-8"))
     except ValueError as e:
         raise ModelError(f"{path} is malformed: {e}") from e
+    return {n: info for n, info in header.items() if n != "__metadata__"}, 8 + hlen
+
+
+def safetensors_shapes(directory: str) -> Dict[str, Tuple[int, ...]]:
+    """The shapes of a checkpoint directory's tensors, from the headers of its files (in name order, the first file wins)."""
+    shapes = {}
+    for f in sorted(os.listdir(directory)):
+        if f.endswith(".safetensors"):
+            path = os.path.join(directory, f)
+            with open(path, "rb") as file:
+                head = file.read(8)
+                head += file.read(int.from_bytes(head, "little")) if len(head) == 8 else b""
+            for name, info in safetensors_header(head, path)[0].items():
+                shapes.setdefault(name, tuple(info["shape"]))
+    return shapes
+
+
+def read_safetensors(path: str) -> Dict[str, Tuple[DType, Tuple[int, ...], np.ndarray]]:
+    """Minimal safetensors reader: 8-byte LE header length, JSON header, raw LE data.
+    Returns name -> (dtype, shape, flat array view); 16-bit floats come back as uint16 bits."""
+    data = np.memmap(path, dtype=np.uint8, mode="r")
+    header, base = safetensors_header(data, path)
     out = {}
-    base = 8 + hlen
     for name, info in header.items():
-        if name == "__metadata__":
-            continue
         if info["dtype"] not in _ST_DTYPES:
             raise ModelError(f"unsupported dtype {info['dtype']} (tensor `{name}`)")  # loader.rs:89-93
         dt, npdt = _ST_DTYPES[info["dtype"]]
