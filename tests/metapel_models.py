@@ -76,7 +76,7 @@ CONFIGS = {"broad_values": BROAD_VALUES, "odd": ODD, "one_tap": ONE_TAP, "tuned"
 
 
 def make_model(pkg, backend, cfg, weights, dtype, blocks=64, tokens=1024, seqs=8):
-    meta = pkg.LayeredMetadata.from_config(cfg, "test")
+    meta = pkg.LayeredMetadata.from_config(cfg, "test", {n: x.shape for n, x in weights.items()})
     return pkg.CudaLayeredModel.new(meta, weights, blocks, 16, backend, compute_dtype=dtype, max_batch_tokens=tokens,
                                     max_batch_sequences=seqs)
 
