@@ -353,8 +353,9 @@ def run_serving(args):
 
 
 # ---------------------------------------------------------------------------------------------
-# Layer-list designs beside the Llama layout at equal size: Metapel (min-GRU and latent attention layers) and Zulozen
-# (chunked attention with sinks, dense and mixture-of-experts feed-forwards)
+# Layer-list designs beside the Llama layout at equal size: Metapel (min-GRU and latent attention layers), Zulozen
+# (chunked attention with sinks, dense and mixture-of-experts feed-forwards) and Belizen (gated linear attention and sliding windows that
+# keep the first tokens, gated dense and mixture-of-experts feed-forwards)
 # ---------------------------------------------------------------------------------------------
 
 # Layer sizes of real models, random weights; the layers alternate min-GRU and latent attention.
@@ -370,6 +371,16 @@ LAYERED_VOCAB = 32768
 ZULOZEN_SHAPES = {
     "2048": dict(hidden=2048, ffn=8192, heads=16, dim=128, rot=64, chunk=2048, experts=16, top=2, expert_ffn=1408, shared=2816),
     "4096": dict(hidden=4096, ffn=16384, heads=32, dim=128, rot=64, chunk=2048, experts=16, top=2, expert_ffn=2816, shared=5632),
+}
+
+
+# Linear attention (key heads half as wide as the stream together) and windows alternate, and with every second layer so do the two
+# feed-forwards; a token's experts (some choices are identity experts) and the shared one are about as large as the dense one.
+BELIZEN_SHAPES = {
+    "2048": dict(hidden=2048, ffn=8192, dense=5504, heads=16, dim=128, rot=64, window=1024, keep=4, gla_dim=64, rank=16, experts=16, identity=2, top=2,
+                 expert_ffn=1408, shared=2816),
+    "4096": dict(hidden=4096, ffn=16384, dense=11008, heads=32, dim=128, rot=64, window=1024, keep=4, gla_dim=64, rank=16, experts=16, identity=2, top=2,
+                 expert_ffn=2816, shared=5632),
 }
 
 
@@ -440,6 +451,50 @@ def zulozen_work(meta, rows, contexts, prompts):
     return w + 2 * LAYERED_VOCAB * H, flops + 2 * outs * LAYERED_VOCAB * H, cache, attn
 
 
+def belizen_meta(pkg, name, layers):
+    z = BELIZEN_SHAPES[name]
+    gla = dict(heads=z["heads"], dim=z["gla_dim"], value_dim=z["dim"], decay_tau=16.0, decay_rank=z["rank"])
+    att = dict(heads=z["heads"], kv_heads=z["heads"] // 4, dim=z["dim"], value_dim=z["dim"], window=z["window"], keep_first=z["keep"],
+               rope_dims=z["rot"], rope_base=10000.0, yarn=pkg.Yarn(4.0, 4096.0, 32.0, 1.0), rope_halves=True, scale=z["dim"] ** -0.5,
+               softcap=30.0, qk_norm="per_head", qkv_bias=True, value_gate=True)
+    dense = dict(ffn_dim=z["dense"], activation="geglu_tanh")
+    mix = dict(ffn_dim=z["expert_ffn"], experts=z["experts"], experts_per_token=z["top"], router="softmax", router_identity=z["identity"],
+               expert_form="clamped", expert_limit=7.0, shared_dim=z["shared"], shared_limit=7.0)
+    specs = [pkg.LayerSpec("attention" if i % 2 else "gla", **(att if i % 2 else gla), **(mix if i % 4 in (1, 2) else dense)) for i in range(layers)]
+    return pkg.LayeredMetadata("Belizen", f"belizen-{name}", z["hidden"], LAYERED_VOCAB, specs, 1e-6, block="prenorm", residual_mult=0.5,
+                               embed_scale=8.0, logit_softcap=30.0)
+
+
+def belizen_work(meta, rows, contexts, prompts):
+    """As ``zulozen_work``, over the layer runs. Linear attention counts as cache traffic the state that a decoding row reads and writes, as
+    attention flops the update and the reading of the state per token."""
+    w = flops = cache = attn = 0
+    H = meta.hidden_size
+    for s in meta.layer_runs():
+        if s.mixer == "gla":
+            k, v = s.heads * s.dim, s.heads * s.value_dim
+            n = H * (2 * k + 2 * v + s.decay_rank) + k * s.decay_rank + v * H
+            cache += len(contexts) * 2 * k * s.value_dim * 4
+            attn += rows * 4 * k * s.value_dim
+        else:
+            n = H * (s.heads * (s.dim + s.value_dim) + s.kv_heads * (s.dim + s.value_dim)) + s.heads * s.value_dim * H
+            most = s.window + s.keep_first if s.window else max(contexts + prompts)
+            seen = [min(c, most) for c in contexts]
+            cache += sum(seen) * s.kv_heads * (s.dim + s.value_dim) * 2
+            attn += (sum(seen) + sum(min(i + 1, most) for p in prompts for i in range(p))) * s.heads * 2 * (s.dim + s.value_dim)
+        if s.experts:
+            outputs = s.experts + s.router_identity
+            fixed, one = H * outputs + 3 * H * s.shared_dim, 3 * H * s.ffn_dim
+            reached = s.experts * (1.0 - (1.0 - s.experts_per_token / outputs) ** rows)
+            w, n = w + 2 * int(reached * one), n + fixed
+            flops += int(2 * s.experts_per_token * s.experts / outputs * one * rows)
+        else:
+            n += 3 * H * s.ffn_dim
+        w, flops = w + 2 * n, flops + 2 * n * rows
+    outs = len(contexts) + len(prompts)
+    return w + 2 * LAYERED_VOCAB * H, flops + 2 * outs * LAYERED_VOCAB * H, cache, attn
+
+
 def llama_work(m, rows, contexts, prompts):
     w = weight_bytes_per_step(m)
     flops = 2 * rows * m["num_layers"] * layer_param_count(m) + 2 * (len(contexts) + len(prompts)) * m["vocab_size"] * m["hidden_size"]
@@ -464,7 +519,8 @@ def run_layered(args):
         tflops = 1400.0
     design = args.workload
     shapes, make_meta, work = {"metapel": (METAPEL_SHAPES, metapel_meta, metapel_work),
-                               "zulozen": (ZULOZEN_SHAPES, zulozen_meta, zulozen_work)}[design]
+                               "zulozen": (ZULOZEN_SHAPES, zulozen_meta, zulozen_work),
+                               "belizen": (BELIZEN_SHAPES, belizen_meta, belizen_work)}[design]
     layers, out = args.layers if args.layers != 32 else 8, []
     batches = [("decode", b, CONTEXT) for b in (1, 16, 64)] + [("prefill", 1, 2048), ("prefill", 4, 2048)]
     with ClockSampler(0) as clocks:
@@ -671,7 +727,7 @@ def tp_parity(pkg, backend, dist, rank, world, dtype_name="BF16", model=None, nu
 def run_ours(args):
     if args.workload in ("serving", "prefix"):
         return run_serving(args)
-    if args.workload in ("metapel", "zulozen"):
+    if args.workload in ("metapel", "zulozen", "belizen"):
         return run_layered(args)
     import __graft_entry__ as ge
 
@@ -887,13 +943,13 @@ def main():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", choices=("ours", "reference"), default="ours")
     ap.add_argument("--no-cpu-baseline", action="store_true")
-    ap.add_argument("--workload", choices=("decode", "serving", "prefix", "metapel", "zulozen"), default="decode",
+    ap.add_argument("--workload", choices=("decode", "serving", "prefix", "metapel", "zulozen", "belizen"), default="decode",
                     help="decode = the headline step (default); serving = continuous batching through the engine "
-                         "loop; prefix = shared-prefix requests on the Qwen2-7B shape through the engine loop; metapel, zulozen = "
+                         "loop; prefix = shared-prefix requests on the Qwen2-7B shape through the engine loop; metapel, zulozen, belizen = "
                          "prefill and decode of that design at a few sizes beside the Llama layout")
-    ap.add_argument("--layered-shapes", "--metapel-shapes", default="2048,4096", help="metapel and zulozen workloads: layer sizes to run")
+    ap.add_argument("--layered-shapes", "--metapel-shapes", default="2048,4096", help="metapel, zulozen and belizen workloads: layer sizes to run")
     ap.add_argument("--layered-only", "--metapel-only", default="",
-                    help="metapel and zulozen workloads: batches to run, for instance decode64,prefill1")
+                    help="metapel, zulozen and belizen workloads: batches to run, for instance decode64,prefill1")
     ap.add_argument("--skip-cached-prefix", action="store_true",
                     help="engine workloads: start prefill after the tokens adopted from the prefix cache "
                          "(an extension; the reference shares the blocks but recomputes them)")

@@ -75,3 +75,19 @@ def test_algorithmic_work_of_a_zulozen_step(pkg):
     assert w == 2 * (2 * mix + dense + fixed + head) + 2 * int(4 * (1 - 0.75 ** 12) * expert)
     assert fl == 2 * (12 * (2 * mix + dense + fixed + expert) + head)
     assert cache == 0 and attn == 2 * (55 + 3) * 4 * 2 * 56
+
+
+def test_algorithmic_work_of_a_belizen_step(pkg):
+    layers = [pkg.LayerSpec("gla", 20, heads=4, dim=8, value_dim=12, decay_rank=3, decay_tau=4.0, activation="geglu_tanh"),
+              pkg.LayerSpec("attention", 12, heads=4, kv_heads=2, dim=32, value_dim=24, window=10, keep_first=2, qk_norm="per_head", experts=3,
+                            router="softmax", router_identity=1, experts_per_token=1, shared_dim=8)]
+    meta = pkg.LayeredMetadata("Belizen", "m", 48, 100, layers, 1e-5, block="prenorm", loop=pkg.Loop(0, 1, 2))
+    lin = 48 * (2 * 32 + 2 * 48 + 3) + 32 * 3 + 48 * 48 + 3 * 48 * 20
+    att = 48 * (4 * 32 + 2 * 56 + 4 * 24) + 4 * 24 * 48 + 4 * 48 + 3 * 48 * 8
+    expert, head = 3 * 48 * 12, bench.LAYERED_VOCAB * 48
+    w, fl, cache, attn = bench.belizen_work(meta, 1, [27], [])  # one row reaches an expert three times out of four
+    assert w == 2 * (2 * lin + att + int(0.75 * expert) + head) and fl == 2 * (2 * lin + att + head) + int(2 * 0.75 * expert)
+    assert cache == 2 * 2 * 32 * 12 * 4 + 12 * 2 * 56 * 2 and attn == 2 * 4 * 32 * 12 + 12 * 4 * 2 * 56
+    w, fl, cache, attn = bench.belizen_work(meta, 14, [], [14])
+    assert w == 2 * (2 * lin + att + head) + 2 * int(3 * (1 - 0.75 ** 14) * expert)
+    assert cache == 0 and attn == 14 * 2 * 4 * 32 * 12 + (78 + 2 * 12) * 4 * 2 * 56
