@@ -56,8 +56,9 @@ __device__ uint32_t g_prefill_tc_error = 0;
 
 __device__ __forceinline__ void softmax_bar() { asm volatile("bar.sync 1, 128;" ::: "memory"); }  // warps 2..5
 
-// FORM: the mask, sinks and gate of `form`; without it those branches and arguments are compiled out.
-template <int DK, int DV, bool FORM>
+// FORM: 1 = the mask, sinks and gate of `form`, 2 = besides them the soft cap, the kept first positions and the gates of values; what
+// is left out is compiled out.
+template <int DK, int DV, int FORM>
 __global__ void __launch_bounds__(kThreads, DV <= 128 ? 2 : 1)
 paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const bf16 *__restrict__ q,
                         KvLayout kv, uint32_t layer, AttnBatch batch, const PrefillTile *__restrict__ tiles, uint32_t q_heads,
@@ -86,8 +87,8 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
   // key tiles start at the block of the first key that the tile's first row sees
   const uint32_t block0 = FORM ? form.range.first(batch.query_positions[tile.row_start]) / kBlk : 0;
   // before them come the blocks of the positions that every row keeps: index i -> logical block
-  const uint32_t kept_blk = FORM ? form.range.kept_blocks(block0, kBlk) : 0;
-  auto logical = [&](uint32_t i) { return !FORM || i < kept_blk ? i : block0 - kept_blk + i; };
+  const uint32_t kept_blk = FORM == 2 ? form.range.kept_blocks(block0, kBlk) : 0;
+  auto logical = [&](uint32_t i) { return FORM == 2 && i < kept_blk ? i : block0 - kept_blk + i; };
   const uint32_t ntiles = (kept_blk + nblocks - block0 + (kKeys / kBlk) - 1) / (kKeys / kBlk);
 
   if (threadIdx.x == 0) {
@@ -137,7 +138,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
 #pragma unroll
         for (uint32_t b = 0; b < kKeys / kBlk; ++b) {
           // a block past the row's context repeats the first one: its keys are masked, its values must be finite
-          const uint32_t lb = FORM ? logical(j * (kKeys / kBlk) + b) : j * (kKeys / kBlk) + b;
+          const uint32_t lb = logical(j * (kKeys / kBlk) + b);
           const uint32_t block = table[lb < nblocks ? lb : block0];
           const int chunk = (int)((chunk0 + block) * kv.num_kv_heads + kvh);
 #pragma unroll
@@ -204,11 +205,21 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     if (threadIdx.x == 64) mbar_arrive(q_ready);
 
     float sl2 = FORM && form.scale != 0.f ? form.scale * 1.4426950408889634f : 1.4426950408889634f / sqrtf((float)DK);
-    const int keep = FORM ? (int)form.range.keep : 0;
-    float cap_in = 0.f, cap_out = 0.f;
-    if (FORM && form.softcap != 0.f) {  // the cap leaves scores in the log2 domain
-      cap_out = form.softcap * 1.4426950408889634f, cap_in = 2.f * sl2 / form.softcap;
+    const int keep = FORM == 2 ? (int)form.range.keep : 0;
+    // A soft cap leaves scores in the log2 domain. Where every score of a warp's tile is at most kTaylor of the cap it is a polynomial, and
+    // unless the cap is very high the exponentials need no running maximum.
+    constexpr float kTaylor = 0.35f;
+    float cap_in = 0.f, cap_out = 0.f, small = 0.f, taylor[5] = {};
+    bool fixed = false;
+    if (FORM == 2 && form.softcap != 0.f) {
+      const float y = (form.scale != 0.f ? form.scale : 1.0f / sqrtf((float)DK)) / form.softcap;  // tanh's argument per unit of q.k
+      cap_out = form.softcap * 1.4426950408889634f, cap_in = 2.f * 1.4426950408889634f * y;
+      small = kTaylor / y;
+      // tanh(x) = x - x^3 / 3 + 2 x^5 / 15 - 17 x^7 / 315 + 62 x^9 / 2835 - ...
+      taylor[0] = cap_out * y, taylor[1] = taylor[0] * y * y * (-1.f / 3.f), taylor[2] = taylor[0] * y * y * y * y * (2.f / 15.f);
+      taylor[3] = taylor[2] * y * y * (-17.f / 42.f), taylor[4] = taylor[3] * y * y * (-62.f / 153.f);
       sl2 = 1.f;
+      fixed = cap_out <= 60.f && !form.sinks;
     }
     float ref = -INFINITY, l = 0.f;
     if (FORM && form.sinks) ref = form.sinks[head] * 1.4426950408889634f, l = 1.f;
@@ -220,20 +231,35 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
       tmem_ld32(taddr, sr[0]);
       tmem_ld32(taddr + 32, sr[1]);
       tmem_ld_wait();
-      const bool straight = !FORM || j * (kKeys / kBlk) >= kept_blk || kept_blk == block0;  // the tile's keys follow one another
-      const int key0 = (int)((FORM ? logical(j * (kKeys / kBlk)) : j * (kKeys / kBlk)) * kBlk);
+      const bool straight = FORM != 2 || j * (kKeys / kBlk) >= kept_blk || kept_blk == block0;  // the tile's keys follow one another
+      const int key0 = (int)(logical(j * (kKeys / kBlk)) * kBlk);
       float mx = -INFINITY;
-      if (FORM && form.softcap != 0.f) {
+      if (FORM == 2 && form.softcap != 0.f) {
+        float most = 0.f;
 #pragma unroll
-        for (int i = 0; i < kKeys; ++i) sr[i >> 5][i & 31] = __float_as_uint(softcap_log2(__uint_as_float(sr[i >> 5][i & 31]), cap_in, cap_out));
+        for (int i = 0; i < kKeys; ++i) most = fmaxf(most, fabsf(__uint_as_float(sr[i >> 5][i & 31])));
+        if (__all_sync(0xffffffffu, most <= small)) {
+#pragma unroll
+          for (int i = 0; i < kKeys; ++i) {
+            const float x = __uint_as_float(sr[i >> 5][i & 31]), x2 = x * x;
+            sr[i >> 5][i & 31] = __float_as_uint(x * fmaf(x2, fmaf(x2, fmaf(x2, fmaf(x2, taylor[4], taylor[3]), taylor[2]), taylor[1]), taylor[0]));
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < kKeys; ++i) sr[i >> 5][i & 31] = __float_as_uint(softcap_log2(__uint_as_float(sr[i >> 5][i & 31]), cap_in, cap_out));
+        }
       }
       // most key tiles are seen whole by every row of a warp (rows past the tile are not stored)
       if (straight && __all_sync(0xffffffffu, !valid || (key0 + kKeys - 1 <= pos && (!FORM || key0 >= low)))) {
+        if (FORM == 2 && fixed) {
+          mx = 0.f;
+        } else {
 #pragma unroll
-        for (int i = 0; i < kKeys; ++i) {
-          const float v = __uint_as_float(sr[i >> 5][i & 31]) * sl2;
-          sr[i >> 5][i & 31] = __float_as_uint(v);
-          mx = fmaxf(mx, v);
+          for (int i = 0; i < kKeys; ++i) {
+            const float v = __uint_as_float(sr[i >> 5][i & 31]) * sl2;
+            sr[i >> 5][i & 31] = __float_as_uint(v);
+            mx = fmaxf(mx, v);
+          }
         }
       } else {
         int from[kKeys / kBlk];  // first key of every block
@@ -242,11 +268,12 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
 #pragma unroll
         for (int i = 0; i < kKeys; ++i) {
           const int key = from[i / kBlk] + i % kBlk;
-          const float v = (key <= pos && (!FORM || key >= low || key < keep)) ? __uint_as_float(sr[i >> 5][i & 31]) * sl2 : -INFINITY;
+          const float v = (key <= pos && (!FORM || key >= low || (FORM == 2 && key < keep))) ? __uint_as_float(sr[i >> 5][i & 31]) * sl2 : -INFINITY;
           sr[i >> 5][i & 31] = __float_as_uint(v);
           mx = fmaxf(mx, v);
         }
       }
+      if (FORM == 2 && fixed) mx = 0.f;  // the reference stays at zero: the exponents are between plus and minus the cap
       // The reference of the exponentials moves only when the maximum runs away from it.
       float corr = 1.0f;
       if (mx > ref + kRescaleThreshold || ref == -INFINITY) {
@@ -295,13 +322,13 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     const uint32_t od = FORM && form.out_dim ? form.out_dim : DV, ldo = FORM && form.ldo ? form.ldo : q_heads * od;
     const bool whole_groups = !FORM || (od % 8 == 0 && ldo % 8 == 0);
     bf16 *dst = out + (size_t)row * ldo + (size_t)head * od;
-    const bf16 *vgate = FORM && form.value_gate ? static_cast<const bf16 *>(form.value_gate) + ((size_t)row * q_heads + head) * od : nullptr;
+    const bf16 *vgate = FORM == 2 && form.value_gate ? static_cast<const bf16 *>(form.value_gate) + ((size_t)row * q_heads + head) * od : nullptr;
 #pragma unroll 1
     for (uint32_t c = 0; c < DV; c += 32) {
       uint32_t orow[32];
       tmem_ld32(taddr + kTmemO + c, orow);
       tmem_ld_wait();
-      if (FORM && vgate && valid) {
+      if (FORM == 2 && vgate && valid) {
 #pragma unroll
         for (int i = 0; i < 32; i += 8) {
           if (c + i >= od) continue;
@@ -376,7 +403,7 @@ int arena_map(const bf16 *arena, KvLayout kv, bool values, const CUtensorMap **o
   return ORION_OK;
 }
 
-template <int DK, int DV, bool FORM>
+template <int DK, int DV, int FORM>
 int launch_prefill_tc(const bf16 *q, const bf16 *arena, KvLayout kv, uint32_t layer, AttnBatch batch, const PrefillTile *tiles,
                       uint32_t num_tiles, uint32_t q_heads, AttnForm form, bf16 *out, cudaStream_t stream) {
   using Cfg = PrefillTcConfig<DK, DV>;
@@ -408,7 +435,7 @@ int launch_paged_attention_prefill_tc(const bf16 *q, const bf16 *arena, KvLayout
   if (num_tiles == 0) return ORION_OK;
   if (!prefill_attention_tc_supported(kv, q_heads, arena))
     return set_error(ORION_ERR_INTERNAL, "tensor-core prefill attention does not cover this shape");
-  return launch_prefill_tc<kHd, kHd, false>(q, arena, kv, layer, batch, tiles, num_tiles, q_heads, AttnForm{}, out, stream);
+  return launch_prefill_tc<kHd, kHd, 0>(q, arena, kv, layer, batch, tiles, num_tiles, q_heads, AttnForm{}, out, stream);
 }
 
 int launch_paged_attention_prefill_form(const bf16 *q, const bf16 *arena, KvLayout kv, uint32_t layer, AttnBatch batch,
@@ -418,9 +445,12 @@ int launch_paged_attention_prefill_form(const bf16 *q, const bf16 *arena, KvLayo
   if (!attention_form_supported(kv, q_heads) || encode_fn() == nullptr)
     return set_error(ORION_ERR_INTERNAL, "tensor-core prefill attention does not cover this shape");
   const uint32_t dk = kv.head_dim, dv = kv.v_dim();
-  auto run = dk == 256 ? launch_prefill_tc<256, 256, true>
-             : dk == 64 ? (dv == 64 ? launch_prefill_tc<64, 64, true> : launch_prefill_tc<64, 128, true>)
-                        : (dv == 64 ? launch_prefill_tc<128, 64, true> : launch_prefill_tc<128, 128, true>);
+  auto pick = [&](auto plain, auto more) { return form.softcap != 0.f || form.range.keep || form.value_gate ? more : plain; };
+  auto run = dk == 256  ? pick(launch_prefill_tc<256, 256, 1>, launch_prefill_tc<256, 256, 2>)
+             : dk == 64 ? (dv == 64 ? pick(launch_prefill_tc<64, 64, 1>, launch_prefill_tc<64, 64, 2>)
+                                    : pick(launch_prefill_tc<64, 128, 1>, launch_prefill_tc<64, 128, 2>))
+                        : (dv == 64 ? pick(launch_prefill_tc<128, 64, 1>, launch_prefill_tc<128, 64, 2>)
+                                    : pick(launch_prefill_tc<128, 128, 1>, launch_prefill_tc<128, 128, 2>));
   return run(q, arena, kv, layer, batch, tiles, num_tiles, q_heads, form, out, stream);
 }
 

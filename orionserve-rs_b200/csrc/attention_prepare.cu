@@ -233,6 +233,77 @@ attention_prepare_heads_kernel(const float *__restrict__ partial, uint32_t split
   }
 }
 
+// The same for heads of at most 128 values (sizes and strides multiples of 4, rotated halves too): a lane holds four columns of each of
+// its warp's HEADS heads, all fetched at once, and pairs meet through shuffles. SLABS as above.
+template <typename T, int HEADS, int SLABS>
+__global__ void __launch_bounds__(kHeadWarps * 32)
+attention_prepare_lanes_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, AttnInputs in,
+                               const uint32_t *__restrict__ positions, const uint32_t *__restrict__ slot_block,
+                               const uint32_t *__restrict__ slot_slot, T *__restrict__ q_out, T *__restrict__ arena, KvLayout kv, uint32_t layer,
+                               T *__restrict__ value_gate) {
+  pdl_trigger();
+  const uint32_t row = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, half = in.rope_dims / 2, d = lane * 4;
+  const uint32_t nq = in.q_heads * in.dim, nk = in.kv_heads * in.dim;
+  const uint32_t pos = positions[row], block = slot_block[row], slot = slot_slot[row];
+  const uint32_t first_v = in.q_heads + in.kv_heads, first_gate = first_v + in.kv_heads, heads = first_gate + (value_gate ? in.q_heads : 0);
+  // angles: the first of a pair adds -sin of the other, the second +sin
+  const float4 one = make_float4(1.f, 1.f, 1.f, 1.f), zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 co = one, si = zero, gq = one, gk = one;
+  uint32_t partner = lane;
+  if (d < 2 * half) {
+    const uint32_t at = d < half ? d : d - half;
+    co = *reinterpret_cast<const float4 *>(in.rope_cos + (size_t)pos * half + at);
+    si = *reinterpret_cast<const float4 *>(in.rope_sin + (size_t)pos * half + at);
+    if (d < half) si = make_float4(-si.x, -si.y, -si.z, -si.w);
+    partner = d < half ? lane + half / 4 : lane - half / 4;
+  }
+  if (in.q_norm && d < in.dim) {
+    gq = *reinterpret_cast<const float4 *>(in.q_norm + d);
+    gk = *reinterpret_cast<const float4 *>(in.k_norm + d);
+  }
+  pdl_wait();
+  float4 v[HEADS];
+#pragma unroll
+  for (int r = 0; r < HEADS; ++r) {
+    const uint32_t t = (blockIdx.y * HEADS + r) * kHeadWarps + warp, n = t < first_v ? in.dim : in.value_dim;
+    v[r] = zero;
+    if (t >= heads || d >= n) continue;
+    const uint32_t at = (t < first_v ? t * in.dim : nq + nk + (t - first_v) * in.value_dim) + d;  // gates follow the values
+    v[r] = sum_slabs4_most<SLABS>(partial + (size_t)row * in.ld + at, splits, split_stride);
+    if (in.bias && t < first_gate) {
+      const float4 b = *reinterpret_cast<const float4 *>(in.bias + at);
+      v[r] = make_float4(v[r].x + b.x, v[r].y + b.y, v[r].z + b.z, v[r].w + b.w);
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < HEADS; ++r) {
+    const uint32_t t = (blockIdx.y * HEADS + r) * kHeadWarps + warp;
+    if (t >= heads) continue;
+    float4 x = v[r];
+    if (t >= first_gate) {
+      x = make_float4(sigmoid_for<T>(x.x), sigmoid_for<T>(x.y), sigmoid_for<T>(x.z), sigmoid_for<T>(x.w));
+      if (d < in.value_dim) store4<T>(value_gate + ((size_t)row * in.q_heads + (t - first_gate)) * in.value_dim + d, x);
+      continue;
+    }
+    if (t >= first_v) {
+      if (d < in.value_dim) store4<T>(arena + kv.row(layer, block, t - first_v, 1, slot) + kv.col(slot, d), x);
+      continue;
+    }
+    const bool is_q = t < in.q_heads;
+    if (in.q_norm) {
+      const float s = 1.0f / sqrtf(warp_sum(x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w) / (float)in.dim + in.eps);
+      const float4 g = is_q ? gq : gk;
+      x = make_float4(x.x * s * g.x, x.y * s * g.y, x.z * s * g.z, x.w * s * g.w);
+    }
+    const float4 o = make_float4(__shfl_sync(0xffffffffu, x.x, partner), __shfl_sync(0xffffffffu, x.y, partner),
+                                 __shfl_sync(0xffffffffu, x.z, partner), __shfl_sync(0xffffffffu, x.w, partner));
+    x = make_float4(x.x * co.x + o.x * si.x, x.y * co.y + o.y * si.y, x.z * co.z + o.z * si.z, x.w * co.w + o.w * si.w);
+    if (d >= in.dim) continue;
+    if (is_q) store4<T>(q_out + ((size_t)row * in.q_heads + t) * kv.head_dim + d, x);
+    else store4<T>(arena + kv.row(layer, block, t - in.q_heads, 0, slot) + kv.col(slot, d), x);
+  }
+}
+
 template <typename T>
 __global__ void arena_rows_kernel(const T *__restrict__ arena, KvLayout kv, uint32_t dim, uint32_t value_dim, float *__restrict__ out) {
   const size_t tokens = (size_t)kv.num_blocks * kv.num_kv_heads * kv.block_size, keys = tokens * dim, all = keys + tokens * value_dim;
@@ -271,7 +342,17 @@ int launch_attention_prepare(const float *partial, uint32_t splits, size_t split
     if (gate) return set_error(ORION_ERR_INTERNAL, "a gate per head is not built for this layout");
     const bool vec = in.dim % 4 == 0 && in.value_dim % 4 == 0 && in.rope_dims % 4 == 0 && in.ld % 4 == 0 && split_stride % 4 == 0 &&
                      kv.head_dim % 4 == 0 && kv.v_dim() % 4 == 0;
-    const uint32_t heads = 2 * in.kv_heads + in.q_heads * (value_gate ? 2 : 1), most = (heads + kHeadWarps - 1) / kHeadWarps;
+    const uint32_t heads = 2 * in.kv_heads + in.q_heads * (value_gate ? 2 : 1);
+    if (vec && in.dim <= 128 && in.value_dim <= 128 && in.halves && in.rope_dims % 8 == 0) {
+      const int slabs = slab_variant(rows, splits);
+      const uint32_t each = slabs == 0 || rows < 296 ? 1 : (slabs == 4 ? 2 : 5);  // heads per warp
+      auto kernel = each == 1 ? attention_prepare_lanes_kernel<T, 1, 0> : (each == 2 ? attention_prepare_lanes_kernel<T, 2, 4> : attention_prepare_lanes_kernel<T, 5, 1>);
+      ORION_CUDA_CHECK("attention_prepare", launch_pdl(kernel, dim3(rows, (heads + each * kHeadWarps - 1) / (each * kHeadWarps)), dim3(kHeadWarps * 32), 0,
+                                                       stream, partial, splits, split_stride, in, positions, slot_block, slot_slot, q_out, arena, kv,
+                                                       layer, value_gate));
+      return after_launch("attention_prepare");
+    }
+    const uint32_t most = (heads + kHeadWarps - 1) / kHeadWarps;
     // decode batches: a warp per head; prompts: a CTA per row
     const uint32_t split = rows >= 1024 ? 1 : (most < 1024 / rows + 1 ? most : 1024 / rows + 1);
     const size_t smem = (size_t)kHeadWarps * in.dim * sizeof(float);

@@ -17,30 +17,52 @@ constexpr uint32_t kThreads = 256;
 template <typename T>
 struct RowInputs {
   float *q, *k, *alpha, *v, *g, *a;
+  T *decay;  // the head's decay weights where they are few, else null
   __device__ RowInputs(float *smem, const GlaShape &s)
-      : q(smem), k(q + s.dim), alpha(k + s.dim), v(alpha + s.dim), g(v + s.value_dim), a(g + s.value_dim) {}
-  static __host__ __device__ size_t floats(const GlaShape &s) { return (3 * (size_t)s.dim + 2 * (size_t)s.value_dim + s.rank + 3) / 4 * 4; }
+      : q(smem), k(q + s.dim), alpha(k + s.dim), v(alpha + s.dim), g(v + s.value_dim), a(g + s.value_dim),
+        decay(held(s) ? reinterpret_cast<T *>(smem + (values(s) + 3) / 4 * 4) : nullptr) {}
+  static __host__ __device__ size_t values(const GlaShape &s) { return 3 * (size_t)s.dim + 2 * (size_t)s.value_dim + s.rank; }
+  static __host__ __device__ size_t held(const GlaShape &s) { return s.dim * s.rank <= 4096 ? s.dim * s.rank : 0; }
+  static __host__ __device__ size_t floats(const GlaShape &s) { return (values(s) + 3) / 4 * 4 + (held(s) * sizeof(T) + 15) / 16 * 4; }
+
+  // Weights: before the kernel waits for the projection.
+  __device__ void fetch_weights(const GlaShape &s, const GlaWeights<T> &w, uint32_t head) const {
+    if (decay)
+      for (uint32_t i = threadIdx.x; i < s.dim * s.rank; i += blockDim.x) decay[i] = w.decay[(size_t)head * s.dim * s.rank + i];
+  }
 
   __device__ void load(const float *p, uint32_t splits, size_t stride, const GlaShape &s, const GlaWeights<T> &w, uint32_t head) const {
     const uint32_t nq = s.q_cols(), nv = s.v_cols(), D = s.dim, V = s.value_dim, all = 2 * D + 2 * V + s.rank;
     const float qs = 1.0f / sqrtf((float)D);
-    for (uint32_t i = threadIdx.x; i < all; i += blockDim.x) {
-      uint32_t at;
-      float *dst;
-      float f = 1.f;
-      if (i < D) at = head * D + i, dst = q + i, f = qs;
-      else if (i < 2 * D) at = nq + head * D + (i - D), dst = k + (i - D);
-      else if (i < 2 * D + V) at = 2 * nq + head * V + (i - 2 * D), dst = v + (i - 2 * D);
-      else if (i < 2 * D + 2 * V) at = 2 * nq + nv + head * V + (i - 2 * D - V), dst = g + (i - 2 * D - V);
-      else at = 2 * nq + 2 * nv + (i - 2 * D - 2 * V), dst = a + (i - 2 * D - 2 * V);
-      *dst = f * fold_slabs(p + at, splits, stride);
+    for (uint32_t i0 = threadIdx.x; i0 < all; i0 += 2 * blockDim.x) {  // two at a time: their loads overlap
+      float x[2], *dst[2];
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        const uint32_t i = i0 + u * blockDim.x;
+        uint32_t at = 0;
+        dst[u] = nullptr;
+        if (i < D) at = head * D + i, dst[u] = q + i;
+        else if (i < 2 * D) at = nq + head * D + (i - D), dst[u] = k + (i - D);
+        else if (i < 2 * D + V) at = 2 * nq + head * V + (i - 2 * D), dst[u] = v + (i - 2 * D);
+        else if (i < 2 * D + 2 * V) at = 2 * nq + nv + head * V + (i - 2 * D - V), dst[u] = g + (i - 2 * D - V);
+        else if (i < all) at = 2 * nq + 2 * nv + (i - 2 * D - 2 * V), dst[u] = a + (i - 2 * D - 2 * V);
+        x[u] = dst[u] ? fold_slabs(p + at, splits, stride) * (i < D ? qs : 1.f) : 0.f;
+      }
+#pragma unroll
+      for (int u = 0; u < 2; ++u)
+        if (dst[u]) *dst[u] = x[u];
     }
     __syncthreads();
-    for (uint32_t d = threadIdx.x; d < D; d += blockDim.x) {
-      const size_t c = (size_t)head * D + d;
-      float z = w.bias[c];
-      for (uint32_t r = 0; r < s.rank; ++r) z = fmaf(to_f32<T>(w.decay[c * s.rank + r]), a[r], z);
-      alpha[d] = expf(log_sigmoid(z) / s.tau);
+    // four lanes per channel, every fourth weight each
+    const T *wd = decay ? decay : w.decay + (size_t)head * D * s.rank;
+    for (uint32_t d0 = 0; d0 < D; d0 += blockDim.x / 4) {
+      const uint32_t d = d0 + threadIdx.x / 4, part = threadIdx.x & 3;
+      float z = 0.f;
+      if (d < D)
+        for (uint32_t r = part; r < s.rank; r += 4) z = fmaf(to_f32<T>(wd[d * s.rank + r]), a[r], z);
+      z += __shfl_xor_sync(0xffffffffu, z, 1);
+      z += __shfl_xor_sync(0xffffffffu, z, 2);
+      if (d < D && part == 0) alpha[d] = expf(log_sigmoid_for<T>(z + w.bias[(size_t)head * D + d]) / s.tau);
     }
     __syncthreads();
   }
@@ -61,7 +83,7 @@ __device__ __forceinline__ void finish_head(const float *o, const float *g, cons
 }
 
 template <typename T, int ROWS>
-__global__ void __launch_bounds__(kThreads)
+__global__ void __launch_bounds__(kThreads, ROWS <= 8 ? 4 : 2)
 gla_step_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, GlaShape s, GlaWeights<T> w, float *__restrict__ state,
                 StateBatch sb, uint32_t most_rows, T *__restrict__ out, uint32_t ldo) {
   extern __shared__ float smem[];
@@ -85,6 +107,7 @@ gla_step_kernel(const float *__restrict__ partial, uint32_t splits, size_t split
                ? *reinterpret_cast<const float4 *>(state + rd * s.state_floats() + at + (size_t)d * s.value_dim)
                : make_float4(0.f, 0.f, 0.f, 0.f);
   }
+  in.fetch_weights(s, w, head);
   pdl_wait();
   for (uint32_t row = first; row < end; ++row) {
     in.load(partial + (size_t)row * s.ld, splits, split_stride, s, w, head);
@@ -125,6 +148,7 @@ gla_generic_kernel(const float *__restrict__ partial, uint32_t splits, size_t sp
   const RowInputs<T> in(smem, s);
   float *sums = smem + RowInputs<T>::floats(s);  // [value_dim]
   pdl_trigger();
+  in.fetch_weights(s, w, blockIdx.x);
   pdl_wait();
   const uint32_t head = blockIdx.x, seq = blockIdx.y, first = sb.first_row[seq], end = sb.first_row[seq + 1], V = s.value_dim;
   if (end - first > most_rows) return;

@@ -7,9 +7,8 @@
 //   gla_scan_kernel     CTA per (head, 32 value columns, sequence), chunk after chunk: S stays in registers as f32 accumulators of
 //                       mma.sync and is read by the products with q as two bf16 parts (value and remainder)
 //   gla_finish_kernel   warp per (row, head): norm over the head, gate
-// A is exact to f32 rounding up to its own storage in bf16: its products take both operands in two bf16 parts, scaled relative to the
-// start of the 16 rows of i, so that only the scale of j inside those 16 rows can exceed one; where a channel decays by more than 2^60
-// within 16 rows, those 16 x 16 pairs are summed one by one instead.
+// The exponents of A's operands are relative to the start of the 16 rows of i, so that only the factor of j inside those 16 rows can
+// exceed one; where a channel decays by more than 2^60 within 16 rows, those 16 x 16 pairs are summed one by one instead.
 #include "gla.cuh"
 #include "mma.cuh"
 
@@ -39,9 +38,10 @@ struct ItemLayout {
 // Row stride of f32 rows whose float2 fragments (8 rows x 4 pairs) fall into different banks.
 __host__ __device__ inline uint32_t float_stride(uint32_t dims) { return dims % 32 ? dims + 24 : dims + 8; }
 
+constexpr uint32_t kRankStride = kC + 4;
 inline size_t prepare_smem(const GlaShape &s) {
   const ItemLayout L(s);
-  return (3 * (size_t)kC * float_stride(L.dims) + kSubs * L.dims + (size_t)kC * s.rank) * sizeof(float);
+  return (3 * (size_t)kC * float_stride(L.dims) + kSubs * L.dims + (size_t)kRankStride * s.rank) * sizeof(float);
 }
 
 // x and y as bf16, and what that leaves out.
@@ -50,10 +50,11 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t &hi, uint32_t 
   lo = pack_bf16x2(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xFFFF0000u));
 }
 
-template <bool VEC>
+// VEC: four columns at once, from at most SLABS slabs (0: any number).
+template <bool VEC, int SLABS>
 __device__ __forceinline__ float4 load_quad(const float *p, uint32_t splits, size_t stride, uint32_t valid) {
   if constexpr (VEC) {
-    return valid ? sum_slabs4(p, splits, stride) : make_float4(0.f, 0.f, 0.f, 0.f);
+    return valid ? sum_slabs4_most<SLABS>(p, splits, stride) : make_float4(0.f, 0.f, 0.f, 0.f);
   } else {
     float v[4];
 #pragma unroll
@@ -61,16 +62,18 @@ __device__ __forceinline__ float4 load_quad(const float *p, uint32_t splits, siz
     return make_float4(v[0], v[1], v[2], v[3]);
   }
 }
+__device__ __forceinline__ float4 exp2_4(float4 x) { return make_float4(fast_exp2(x.x), fast_exp2(x.y), fast_exp2(x.z), fast_exp2(x.w)); }
+__device__ __forceinline__ uint2 pack_product4(float4 a, float4 b) { return make_uint2(pack_bf16x2(a.x * b.x, a.y * b.y), pack_bf16x2(a.z * b.z, a.w * b.w)); }
 
-template <bool VEC>
-__global__ void __launch_bounds__(kThreads, 2)
+template <bool VEC, int SLABS>
+__global__ void __launch_bounds__(kThreads, 3)
 gla_prepare_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, GlaShape s, GlaWeights<bf16> w,
                    const GlaChunk *__restrict__ chunks, uint8_t *__restrict__ items) {
   extern __shared__ __align__(16) float smem[];
   __shared__ uint32_t steep;  // bit I: rows 16 I .. 16 I + 15 decay by more than the limit in some channel
   const ItemLayout L(s);
   const uint32_t SD = float_stride(L.dims), tid = threadIdx.x, head = blockIdx.x;
-  float *q = smem, *k = q + kC * SD, *b = k + kC * SD, *total = b + kC * SD, *a1 = total + kSubs * L.dims;
+  float *q = smem, *k = q + kC * SD, *b = k + kC * SD, *total = b + kC * SD, *a1 = total + kSubs * L.dims;  // a1 [rank][kRankStride]
   uint8_t *item = items + ((size_t)blockIdx.y * s.heads + head) * L.bytes;
   pdl_trigger();
   if (tid == 0) steep = 0;
@@ -79,26 +82,25 @@ gla_prepare_kernel(const float *__restrict__ partial, uint32_t splits, size_t sp
   const uint32_t nq = s.q_cols(), nv = s.v_cols(), quads = L.dims / 4, vquads = L.slices * kSlice / 4;
   const float *p = partial + (size_t)ch.row * s.ld;
   const float qs = 1.0f / sqrtf((float)s.dim);
-#pragma unroll 2
+  for (uint32_t i = tid; i < kC * s.rank; i += kThreads) {
+    const uint32_t t = i / s.rank, r = i % s.rank;
+    const float *src = p + (size_t)t * s.ld + 2 * nq + 2 * nv + r;
+    a1[r * kRankStride + t] = t < ch.count ? (SLABS == 1 ? *src : fold_slabs(src, splits, split_stride)) : 0.f;
+  }
+#pragma unroll 4
   for (uint32_t i = tid; i < kC * quads; i += kThreads) {
     const uint32_t t = i / quads, d = i % quads * 4, valid = t < ch.count && d < s.dim ? s.dim - d : 0;
     const float *src = p + (size_t)t * s.ld + head * s.dim + d;
-    float4 x = load_quad<VEC>(src, splits, split_stride, valid);
-    const float4 y = load_quad<VEC>(src + nq, splits, split_stride, valid);
-    x = make_float4(x.x * qs, x.y * qs, x.z * qs, x.w * qs);
-    *reinterpret_cast<float4 *>(q + t * SD + d) = x;
+    const float4 x = load_quad<VEC, SLABS>(src, splits, split_stride, valid), y = load_quad<VEC, SLABS>(src + nq, splits, split_stride, valid);
+    *reinterpret_cast<float4 *>(q + t * SD + d) = make_float4(x.x * qs, x.y * qs, x.z * qs, x.w * qs);
     *reinterpret_cast<float4 *>(k + t * SD + d) = y;
   }
-#pragma unroll 2
+#pragma unroll 4
   for (uint32_t i = tid; i < kC * vquads; i += kThreads) {
     const uint32_t t = i / vquads, v = i % vquads * 4, valid = t < ch.count && v < s.value_dim ? s.value_dim - v : 0;
-    const float4 x = load_quad<VEC>(p + (size_t)t * s.ld + 2 * nq + head * s.value_dim + v, splits, split_stride, valid);
+    const float4 x = load_quad<VEC, SLABS>(p + (size_t)t * s.ld + 2 * nq + head * s.value_dim + v, splits, split_stride, valid);
     bf16 *dst = reinterpret_cast<bf16 *>(item + L.v + v / kSlice * ItemLayout::slice_bytes()) + t * kVStride + v % kSlice;
     *reinterpret_cast<uint2 *>(dst) = make_uint2(pack_bf16x2(x.x, x.y), pack_bf16x2(x.z, x.w));
-  }
-  for (uint32_t i = tid; i < kC * s.rank; i += kThreads) {
-    const uint32_t t = i / s.rank, r = i % s.rank;
-    a1[i] = t < ch.count ? fold_slabs(p + (size_t)t * s.ld + 2 * nq + 2 * nv + r, splits, split_stride) : 0.f;
   }
   __syncthreads();
 
@@ -108,26 +110,30 @@ gla_prepare_kernel(const float *__restrict__ partial, uint32_t splits, size_t sp
     float z[kSub];
     const bool live = d < s.dim;
     const size_t c = (size_t)head * s.dim + (live ? d : 0);
-    const float bias = w.bias[c];
+    const float bias = w.bias[c], unit = 1.4426950408889634f / s.tau;
 #pragma unroll
     for (uint32_t t = 0; t < kSub; ++t) z[t] = bias;
+#pragma unroll 4
     for (uint32_t r = 0; r < s.rank; ++r) {
       const float wr = __bfloat162float(w.decay[c * s.rank + r]);
+      const float4 *a = reinterpret_cast<const float4 *>(a1 + r * kRankStride + sub * kSub);
 #pragma unroll
-      for (uint32_t t = 0; t < kSub; ++t) z[t] = fmaf(wr, a1[(sub * kSub + t) * s.rank + r], z[t]);
+      for (uint32_t t = 0; t < kSub; t += 4) {
+        const float4 x = a[t / 4];
+        z[t] = fmaf(wr, x.x, z[t]), z[t + 1] = fmaf(wr, x.y, z[t + 1]), z[t + 2] = fmaf(wr, x.z, z[t + 2]), z[t + 3] = fmaf(wr, x.w, z[t + 3]);
+      }
     }
-    const float unit = 1.4426950408889634f / s.tau;
     float sum = 0.f;
 #pragma unroll
     for (uint32_t t = 0; t < kSub; ++t) {
-      if (live && sub * kSub + t < ch.count) sum += log_sigmoid(z[t]) * unit;
+      if (live && sub * kSub + t < ch.count) sum += log_sigmoid_fast(z[t]) * unit;
       b[(sub * kSub + t) * SD + d] = sum;
     }
     total[i] = sum;
     if (!(sum > kMostDecay)) atomicOr(&steep, 1u << sub);
   }
   __syncthreads();
-  for (uint32_t i = tid; i < kSubs * L.dims; i += kThreads) {
+  for (uint32_t i = L.dims + tid; i < kSubs * L.dims; i += kThreads) {
     const uint32_t d = i % L.dims, sub = i / L.dims;
     float before = 0.f;
     for (uint32_t u = 0; u < sub; ++u) before += total[u * L.dims + d];
@@ -138,69 +144,68 @@ gla_prepare_kernel(const float *__restrict__ partial, uint32_t splits, size_t sp
 
   // The operands of the scan.
   const float *last = b + (kC - 1) * SD;
+#pragma unroll 2
   for (uint32_t i = tid; i < kC * quads; i += kThreads) {
     const uint32_t t = i / quads, d = i % quads * 4;
     const float4 x = *reinterpret_cast<const float4 *>(q + t * SD + d), y = *reinterpret_cast<const float4 *>(k + t * SD + d);
     const float4 at = *reinterpret_cast<const float4 *>(b + t * SD + d), e = *reinterpret_cast<const float4 *>(last + d);
     bf16 *dst = reinterpret_cast<bf16 *>(item) + t * L.row + d;
-    *reinterpret_cast<uint2 *>(dst) = make_uint2(pack_bf16x2(x.x * fast_exp2(at.x), x.y * fast_exp2(at.y)), pack_bf16x2(x.z * fast_exp2(at.z), x.w * fast_exp2(at.w)));
-    *reinterpret_cast<uint2 *>(dst + L.k / 2) = make_uint2(pack_bf16x2(y.x * fast_exp2(e.x - at.x), y.y * fast_exp2(e.y - at.y)),
-                                                           pack_bf16x2(y.z * fast_exp2(e.z - at.z), y.w * fast_exp2(e.w - at.w)));
+    *reinterpret_cast<uint2 *>(dst) = pack_product4(x, exp2_4(at));
+    *reinterpret_cast<uint2 *>(dst + L.k / 2) = pack_product4(y, exp2_4(make_float4(e.x - at.x, e.y - at.y, e.z - at.z, e.w - at.w)));
   }
   for (uint32_t d = tid; d < L.dims; d += kThreads) reinterpret_cast<float *>(item + L.decay)[d] = fast_exp2(last[d]);
 
-  // A, a block of 16 x 16 per warp and round; the ten blocks with work come first.
+  // A in blocks of 16 x 16, on and below the diagonal (nothing reads the others): a warp takes one or two of a row of blocks.
+  const uint32_t lane = tid & 31, g = lane >> 2, t2 = (lane & 3) * 2, warp = tid >> 5;
+  constexpr uint32_t kPlan[kWarps] = {0x302, 0x322, 0x202, 0x221, 0x101, 0x111, 0x001, 0};  // I, first J, number of J
+  uint32_t plan = 0;
+#pragma unroll
+  for (uint32_t i = 0; i < kWarps; ++i)
+    if (warp == i) plan = kPlan[i];
+  const uint32_t I = plan >> 8, J0 = plan >> 4 & 15, nJ = plan & 15, i0 = I * kSub;
+  if (nJ == 0) return;
   bf16 *A = reinterpret_cast<bf16 *>(item + L.a);
-  const uint32_t lane = tid & 31, g = lane >> 2, t2 = (lane & 3) * 2;
-  for (uint32_t n = tid >> 5; n < kSubs * kSubs; n += kWarps) {
-    uint32_t I, J;
-    if (n < 10) {
-      I = n < 4 ? 3 : (n < 7 ? 2 : (n < 9 ? 1 : 0));
-      J = n - (n < 4 ? 0 : (n < 7 ? 4 : (n < 9 ? 7 : 9)));
-    } else {
-      const uint32_t u = n - 10;
-      I = u < 3 ? 0 : (u < 5 ? 1 : 2);
-      J = u < 3 ? 1 + u : (u < 5 ? u - 1 : 3);
+  const float *ref = I > 0 ? b + (i0 - 1) * SD : nullptr;
+  auto pair = [&](const float *x, uint32_t row, uint32_t d, float sign, float2 r) {
+    const float2 v = *reinterpret_cast<const float2 *>(x + row * SD + d), at = *reinterpret_cast<const float2 *>(b + row * SD + d);
+    return pack_bf16x2(v.x * fast_exp2(sign * (at.x - r.x)), v.y * fast_exp2(sign * (at.y - r.y)));
+  };
+  float acc[2][2][4] = {};
+  const bool slow = steep >> I & 1u;
+  for (uint32_t d0 = 0; d0 < L.dims; d0 += 16) {
+    uint32_t a[4];
+    float2 r[2];
+#pragma unroll
+    for (uint32_t h = 0; h < 2; ++h) {
+      const uint32_t d = d0 + h * 8 + t2;
+      r[h] = ref ? *reinterpret_cast<const float2 *>(ref + d) : make_float2(0.f, 0.f);
+      a[2 * h] = pair(q, i0 + g, d, 1.f, r[h]);
+      a[2 * h + 1] = pair(q, i0 + g + 8, d, 1.f, r[h]);
     }
-    const uint32_t i0 = I * kSub, j0 = J * kSub;
-    float acc[2][4] = {};
-    if (J == I && (steep >> I & 1u)) {
-#pragma unroll 1
+#pragma unroll
+    for (uint32_t n = 0; n < 2; ++n) {
+      if (n >= nJ || (slow && J0 + n == I)) continue;
+#pragma unroll
+      for (uint32_t nt = 0; nt < 2; ++nt) {
+        uint32_t bk[2];
+#pragma unroll
+        for (uint32_t h = 0; h < 2; ++h) bk[h] = pair(k, (J0 + n) * kSub + nt * 8 + g, d0 + h * 8 + t2, -1.f, r[h]);
+        mma_bf16_16816(acc[n][nt], a, bk[0], bk[1]);
+      }
+    }
+  }
+#pragma unroll
+  for (uint32_t n = 0; n < 2; ++n) {
+    if (n >= nJ) continue;
+    const uint32_t j0 = (J0 + n) * kSub;
+    if (slow && J0 + n == I) {
+#pragma unroll
       for (uint32_t e = 0; e < 8; ++e) {
         const uint32_t i = i0 + g + (e & 2 ? 8 : 0), j = j0 + (e >> 2) * 8 + t2 + (e & 1);
-        if (j > i) continue;
         float sum = 0.f;
-        for (uint32_t d = 0; d < s.dim; ++d) sum += q[i * SD + d] * k[j * SD + d] * fast_exp2(b[i * SD + d] - b[j * SD + d]);
-        acc[e >> 2][e & 3] = sum;
-      }
-    } else if (J <= I) {
-      const float *ref = I > 0 ? b + (i0 - 1) * SD : nullptr;
-      auto pair = [&](const float *x, uint32_t row, uint32_t d, float sign, float2 r, uint32_t &hi, uint32_t &lo) {
-        const float2 v = *reinterpret_cast<const float2 *>(x + row * SD + d), at = *reinterpret_cast<const float2 *>(b + row * SD + d);
-        split2(v.x * fast_exp2(sign * (at.x - r.x)), v.y * fast_exp2(sign * (at.y - r.y)), hi, lo);
-      };
-      for (uint32_t d0 = 0; d0 < L.dims; d0 += 16) {
-        uint32_t ah[4], al[4];
-#pragma unroll
-        for (uint32_t h = 0; h < 2; ++h) {
-          const uint32_t d = d0 + h * 8 + t2;
-          const float2 r = ref ? *reinterpret_cast<const float2 *>(ref + d) : make_float2(0.f, 0.f);
-          pair(q, i0 + g, d, 1.f, r, ah[2 * h], al[2 * h]);
-          pair(q, i0 + g + 8, d, 1.f, r, ah[2 * h + 1], al[2 * h + 1]);
-        }
-#pragma unroll
-        for (uint32_t nt = 0; nt < 2; ++nt) {
-          uint32_t bh[2], bl[2];
-#pragma unroll
-          for (uint32_t h = 0; h < 2; ++h) {
-            const uint32_t d = d0 + h * 8 + t2;
-            const float2 r = ref ? *reinterpret_cast<const float2 *>(ref + d) : make_float2(0.f, 0.f);
-            pair(k, j0 + nt * 8 + g, d, -1.f, r, bh[h], bl[h]);
-          }
-          mma_bf16_16816(acc[nt], al, bh[0], bh[1]);
-          mma_bf16_16816(acc[nt], ah, bl[0], bl[1]);
-          mma_bf16_16816(acc[nt], ah, bh[0], bh[1]);
-        }
+        if (j <= i)
+          for (uint32_t d = 0; d < s.dim; ++d) sum += q[i * SD + d] * k[j * SD + d] * fast_exp2(b[i * SD + d] - b[j * SD + d]);
+        acc[n][e >> 2][e & 3] = sum;
       }
     }
 #pragma unroll
@@ -208,7 +213,7 @@ gla_prepare_kernel(const float *__restrict__ partial, uint32_t splits, size_t sp
 #pragma unroll
       for (uint32_t h = 0; h < 2; ++h) {
         const uint32_t i = i0 + g + 8 * h, j = j0 + nt * 8 + t2;
-        const float x = j <= i ? acc[nt][2 * h] : 0.f, y = j + 1 <= i ? acc[nt][2 * h + 1] : 0.f;
+        const float x = j <= i ? acc[n][nt][2 * h] : 0.f, y = j + 1 <= i ? acc[n][nt][2 * h + 1] : 0.f;
         *reinterpret_cast<uint32_t *>(A + i * kAStride + j) = pack_bf16x2(x, y);
       }
   }
@@ -221,9 +226,10 @@ struct ScanPlan {
   explicit ScanPlan(const GlaShape &s) {
     const ItemLayout L(s);
     const uint32_t stage = L.v + ItemLayout::slice_bytes(), parts = 2 * L.dims * kVStride * 2;
-    for (uint32_t c = 2; c >= 1; --c)
-      for (uint32_t n = 3; n >= 2; --n)
-        if (smem == 0 && n * stage + c * parts + 64 <= 227 * 1024) stages = n, copies = c, smem = n * stage + c * parts + 64;
+    for (uint32_t budget : {113u * 1024, 227u * 1024})  // two CTAs per SM if that can be
+      for (uint32_t c = 2; c >= 1; --c)
+        for (uint32_t n = 3; n >= 2; --n)
+          if (smem == 0 && n * stage + c * parts + 64 <= budget) stages = n, copies = c, smem = n * stage + c * parts + 64;
   }
 };
 
@@ -357,38 +363,47 @@ gla_scan_kernel(const uint8_t *__restrict__ items, GlaShape s, float *__restrict
   if (!ok && lane == 0) atomicOr(&g_gla_error, 1u);
 }
 
-// A warp per (row, head), four heads of a chunk per CTA.
-template <int VEC>
+// Four heads of a chunk per CTA, a warp per row; values of at most 128 (VEC 4): the row's four heads are fetched at once.
+template <int VEC, int SLABS>
 __global__ void __launch_bounds__(kThreads)
 gla_finish_kernel(const float *__restrict__ o, const float *__restrict__ partial, uint32_t splits, size_t split_stride, GlaShape s,
                   const float *__restrict__ norm, const GlaChunk *__restrict__ chunks, bf16 *__restrict__ out, uint32_t ldo) {
   pdl_trigger();
   const GlaChunk ch = chunks[blockIdx.x];
-  const uint32_t lane = threadIdx.x & 31, h0 = blockIdx.y * 4, heads = min(4u, s.heads - h0), g_at = 2 * s.q_cols() + s.v_cols();
+  const uint32_t lane = threadIdx.x & 31, h0 = blockIdx.y * 4, heads = min(4u, s.heads - h0), V = s.value_dim, v4 = lane * 4;
+  const uint32_t g_at = 2 * s.q_cols() + s.v_cols();
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f), w = VEC == 4 && v4 < V ? *reinterpret_cast<const float4 *>(norm + v4) : zero;
   pdl_wait();
-  for (uint32_t n = threadIdx.x >> 5; n < ch.count * heads; n += kWarps) {
-    const uint32_t row = ch.row + n / heads, head = h0 + n % heads;
-    const float *src = o + (size_t)row * s.v_cols() + head * s.value_dim, *gate = partial + (size_t)row * s.ld + g_at + head * s.value_dim;
-    bf16 *dst = out + (size_t)row * ldo + head * s.value_dim;
-    float ss = 0.f;
-    if (VEC == 4) {
-      for (uint32_t v = lane * 4; v < s.value_dim; v += 128) {
-        const float4 x = *reinterpret_cast<const float4 *>(src + v);
-        ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+  for (uint32_t n = threadIdx.x >> 5; n < ch.count; n += kWarps) {
+    const uint32_t row = ch.row + n;
+    const float *src = o + (size_t)row * s.v_cols() + h0 * V, *gate = partial + (size_t)row * s.ld + g_at + h0 * V;
+    bf16 *dst = out + (size_t)row * ldo + h0 * V;
+    if constexpr (VEC == 4) {
+      float4 x[4], g[4];
+#pragma unroll
+      for (uint32_t h = 0; h < 4; ++h) {
+        x[h] = g[h] = zero;
+        if (h >= heads || v4 >= V) continue;
+        x[h] = *reinterpret_cast<const float4 *>(src + h * V + v4);
+        g[h] = sum_slabs4_most<SLABS>(gate + h * V + v4, splits, split_stride);
       }
-      const float scale = 1.0f / sqrtf(warp_sum(ss) / (float)s.value_dim + s.eps);
-      for (uint32_t v = lane * 4; v < s.value_dim; v += 128) {
-        const float4 x = *reinterpret_cast<const float4 *>(src + v), g = sum_slabs4(gate + v, splits, split_stride);
-        const float4 w = *reinterpret_cast<const float4 *>(norm + v);
-        *reinterpret_cast<uint2 *>(dst + v) =
-            make_uint2(pack_bf16x2(x.x * scale * w.x * silu_for<bf16>(g.x), x.y * scale * w.y * silu_for<bf16>(g.y)),
-                       pack_bf16x2(x.z * scale * w.z * silu_for<bf16>(g.z), x.w * scale * w.w * silu_for<bf16>(g.w)));
+#pragma unroll
+      for (uint32_t h = 0; h < 4; ++h) {
+        const float ss = warp_sum(x[h].x * x[h].x + x[h].y * x[h].y + x[h].z * x[h].z + x[h].w * x[h].w);
+        const float scale = 1.0f / sqrtf(ss / (float)V + s.eps);
+        if (h >= heads || v4 >= V) continue;
+        *reinterpret_cast<uint2 *>(dst + h * V + v4) =
+            make_uint2(pack_bf16x2(x[h].x * scale * w.x * silu_for<bf16>(g[h].x), x[h].y * scale * w.y * silu_for<bf16>(g[h].y)),
+                       pack_bf16x2(x[h].z * scale * w.z * silu_for<bf16>(g[h].z), x[h].w * scale * w.w * silu_for<bf16>(g[h].w)));
       }
     } else {
-      for (uint32_t v = lane; v < s.value_dim; v += 32) ss += src[v] * src[v];
-      const float scale = 1.0f / sqrtf(warp_sum(ss) / (float)s.value_dim + s.eps);
-      for (uint32_t v = lane; v < s.value_dim; v += 32)
-        dst[v] = __float2bfloat16_rn(src[v] * scale * norm[v] * silu_for<bf16>(fold_slabs(gate + v, splits, split_stride)));
+      for (uint32_t h = 0; h < heads; ++h) {
+        float ss = 0.f;
+        for (uint32_t v = h * V + lane; v < (h + 1) * V; v += 32) ss += src[v] * src[v];
+        const float scale = 1.0f / sqrtf(warp_sum(ss) / (float)V + s.eps);
+        for (uint32_t v = lane; v < V; v += 32)
+          dst[h * V + v] = __float2bfloat16_rn(src[h * V + v] * scale * norm[v] * silu_for<bf16>(fold_slabs(gate + h * V + v, splits, split_stride)));
+      }
     }
   }
 }
@@ -419,20 +434,23 @@ int launch_gla_chunks(const float *partial, uint32_t splits, size_t split_stride
   auto *items = static_cast<uint8_t *>(scratch);
   auto *o = reinterpret_cast<float *>(items + (size_t)p.num_chunks * s.heads * L.bytes);
   const bool vec = s.dim % 4 == 0 && s.value_dim % 4 == 0 && s.ld % 4 == 0 && split_stride % 4 == 0;
-  static bool attr_set[4][kMaxDeviceOrdinals] = {};
-  auto prepare = vec ? gla_prepare_kernel<true> : gla_prepare_kernel<false>;
-  ORION_CUDA_CHECK("gla_prepare attr", ensure_dynamic_smem(prepare, kPrepareSmem, attr_set[vec]));
+  const int slabs = splits <= 1 ? 1 : (splits <= 4 ? 4 : 0);
+  auto pick = [&](auto any, auto one, auto four) { return slabs == 1 ? one : (slabs == 4 ? four : any); };
+  static bool attr_set[6][kMaxDeviceOrdinals] = {};
+  auto prepare = vec ? pick(gla_prepare_kernel<true, 0>, gla_prepare_kernel<true, 1>, gla_prepare_kernel<true, 4>) : gla_prepare_kernel<false, 0>;
+  ORION_CUDA_CHECK("gla_prepare attr", ensure_dynamic_smem(prepare, kPrepareSmem, attr_set[vec ? (slabs + 1) / 2 : 3]));
   ORION_CUDA_CHECK("gla_prepare", launch_pdl(prepare, dim3(s.heads, p.num_chunks), dim3(kThreads), prepare_smem(s), stream, partial, splits, split_stride,
                                              s, w, p.chunks, items));
   ORION_TRY(after_launch("gla_prepare"));
   const bool wide = L.dims > kWarps * 16;
   auto scan = wide ? gla_scan_kernel<2> : gla_scan_kernel<1>;
-  ORION_CUDA_CHECK("gla_scan attr", ensure_dynamic_smem(scan, 227 * 1024, attr_set[2 + wide]));
+  ORION_CUDA_CHECK("gla_scan attr", ensure_dynamic_smem(scan, 227 * 1024, attr_set[4 + wide]));
   ORION_CUDA_CHECK("gla_scan", launch_pdl(scan, dim3(s.heads * L.slices, p.num_portions), dim3(kThreads), (size_t)plan.smem, stream,
                                           (const uint8_t *)items, s, state, sb, p.chunks, p.portions, o, plan.stages, plan.copies));
   ORION_TRY(after_launch("gla_scan"));
-  const bool quads = vec && ldo % 4 == 0;
-  ORION_CUDA_CHECK("gla_finish", launch_pdl(quads ? gla_finish_kernel<4> : gla_finish_kernel<1>, dim3(p.num_chunks, (s.heads + 3) / 4), dim3(kThreads), 0,
+  auto finish = vec && ldo % 4 == 0 && s.value_dim <= 128 ? pick(gla_finish_kernel<4, 0>, gla_finish_kernel<4, 1>, gla_finish_kernel<4, 4>)
+                                                          : gla_finish_kernel<1, 0>;
+  ORION_CUDA_CHECK("gla_finish", launch_pdl(finish, dim3(p.num_chunks, (s.heads + 3) / 4), dim3(kThreads), 0,
                                             stream, (const float *)o, partial, splits, split_stride, s, w.norm, p.chunks, out, ldo));
   return after_launch("gla_finish");
 }

@@ -43,7 +43,8 @@ struct TcArgs {
   GatedAct f, shared_f;
 };
 
-template <int TOKN, int WST, int XST, int MT, bool SWIGLU>
+// GATED: 0 = f32 products, 1 = SwiGLU, 2 = the gated activations of the arguments.
+template <int TOKN, int WST, int XST, int MT, int GATED>
 __global__ void __launch_bounds__(kThreads)
 moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_sw,
                    const __grid_constant__ CUtensorMap map_sx, TcArgs a) {
@@ -155,7 +156,7 @@ moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
         const int mc = mb + 16 * b;
         const uint32_t c = mc % TOKN, nn = n0 + (mc / TOKN) * kTileN + lq * 32 + lane;  // first row of the tile in this chunk, weight row
         if (c >= tile.count) continue;  // warp-uniform
-        if (SWIGLU) {
+        if (GATED) {
           // lane 2i holds gate f, lane 2i + 1 up f, of the same f for these 16 rows; a pair trades halves and each
           // finishes one row of every two
           const uint32_t odd = lane & 1u, f = nn >> 1, ffn = n >> 1;
@@ -167,7 +168,7 @@ moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
             if (r >= tile.count || nn >= n) continue;
             const float w = shared || !a.row_score ? 1.f : a.row_score[tile.row + r];
             const float g = w * __uint_as_float(odd ? recv : rr[b][2 * jj]), u = w * __uint_as_float(odd ? rr[b][2 * jj + 1] : recv);
-            act[(size_t)(tile.row + r) * ffn + f] = __float2bfloat16_rn(gated<bf16>(shared ? a.shared_f : a.f, g, u));
+            act[(size_t)(tile.row + r) * ffn + f] = __float2bfloat16_rn(GATED == 1 ? silu_for<bf16>(g) * u : gated<bf16>(shared ? a.shared_f : a.f, g, u));
           }
         } else if (nn < n) {
 #pragma unroll
@@ -221,9 +222,10 @@ int launch_product(const MoeProduct &p, bool swiglu, uint32_t splits, MoePlan pl
   const uint32_t shared_tiles = p.shared_n ? (p.rows + TOKN - 1) / TOKN : 0;
   const TcArgs a{p.n, p.k, p.shared_n, p.shared_k, shared_tiles, p.rows, p.sorted_rows, splits, p.tiles, p.row_score, p.act, p.shared_act, p.out, p.shared_out, p.f, p.shared_f};
   const dim3 grid((std::max(p.n, p.shared_n) + MT * kTileN - 1) / (MT * kTileN), shared_tiles + plan.tiles, splits);
-  static bool attr_set[2][kMaxDeviceOrdinals] = {};
-  auto kernel = swiglu ? moe_gemm_tc_kernel<TOKN, WST, XST, MT, true> : moe_gemm_tc_kernel<TOKN, WST, XST, MT, false>;
-  ORION_CUDA_CHECK("moe_gemm attr", ensure_dynamic_smem(kernel, Cfg::kSmemBytes, attr_set[swiglu]));
+  static bool attr_set[3][kMaxDeviceOrdinals] = {};
+  const int form = !swiglu ? 0 : (p.f.kind == kGatedSilu && p.shared_f.kind == kGatedSilu ? 1 : 2);
+  auto kernel = form == 0 ? moe_gemm_tc_kernel<TOKN, WST, XST, MT, 0> : (form == 1 ? moe_gemm_tc_kernel<TOKN, WST, XST, MT, 1> : moe_gemm_tc_kernel<TOKN, WST, XST, MT, 2>);
+  ORION_CUDA_CHECK("moe_gemm attr", ensure_dynamic_smem(kernel, Cfg::kSmemBytes, attr_set[form]));
   ORION_CUDA_CHECK("moe_gemm", launch_pdl(kernel, grid, dim3(kThreads), (size_t)Cfg::kSmemBytes, stream, *mw, *mx, *msw, *msx, a));
   count_launch();
   ORION_CUDA_CHECK("moe_gemm", cudaGetLastError());

@@ -188,7 +188,7 @@ def test_mechanism_alone(pkg, backend, dtype, name):
 def test_tiles_of_experts(pkg, backend, dtype, rows, experts):
     """Every number of rows per tile, experts with no, few and many rows, products that end inside a tile, rows without any expert."""
     cfg = config(128, 64, [gla(1, 8, 8, 4.0, 2, moe(*experts))])
-    w = random_weights(cfg, seed=rows)
+    w = silence(random_weights(cfg, seed=rows), "mix.o")  # a lone head of eight values may all but cancel, whatever computes it
     rng = np.random.default_rng(2)
     t = np.where(rng.random(rows) < 0.7, rng.integers(0, 3, rows), rng.integers(0, 64, rows)).tolist()  # uneven use of the experts
     f = Feeder(pkg, make_model(pkg, backend, cfg, w, dtype))
