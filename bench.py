@@ -377,9 +377,9 @@ ZULOZEN_SHAPES = {
 # Linear attention (key heads half as wide as the stream together) and windows alternate, and with every second layer so do the two
 # feed-forwards; a token's experts (some choices are identity experts) and the shared one are about as large as the dense one.
 BELIZEN_SHAPES = {
-    "2048": dict(hidden=2048, ffn=8192, dense=5504, heads=16, dim=128, rot=64, window=1024, keep=4, gla_dim=64, rank=16, experts=16, identity=2, top=2,
+    "2048": dict(hidden=2048, ffn=8192, dense=5504, heads=16, dim=128, rot=64, window=1024, keep=8, gla_dim=64, rank=16, experts=16, identity=2, top=2,
                  expert_ffn=1408, shared=2816),
-    "4096": dict(hidden=4096, ffn=16384, dense=11008, heads=32, dim=128, rot=64, window=1024, keep=4, gla_dim=64, rank=16, experts=16, identity=2, top=2,
+    "4096": dict(hidden=4096, ffn=16384, dense=11008, heads=32, dim=128, rot=64, window=1024, keep=8, gla_dim=64, rank=16, experts=16, identity=2, top=2,
                  expert_ffn=2816, shared=5632),
 }
 
@@ -453,16 +453,16 @@ def zulozen_work(meta, rows, contexts, prompts):
 
 def belizen_meta(pkg, name, layers):
     z = BELIZEN_SHAPES[name]
-    gla = dict(heads=z["heads"], dim=z["gla_dim"], value_dim=z["dim"], decay_tau=16.0, decay_rank=z["rank"])
+    gla = dict(heads=z["heads"], dim=z["gla_dim"], value_dim=z["dim"], decay_tau=8.0, decay_rank=z["rank"])
     att = dict(heads=z["heads"], kv_heads=z["heads"] // 4, dim=z["dim"], value_dim=z["dim"], window=z["window"], keep_first=z["keep"],
-               rope_dims=z["rot"], rope_base=10000.0, yarn=pkg.Yarn(4.0, 4096.0, 32.0, 1.0), rope_halves=True, scale=z["dim"] ** -0.5,
-               softcap=30.0, qk_norm="per_head", qkv_bias=True, value_gate=True)
+               rope_dims=z["rot"], rope_base=10000.0, yarn=pkg.Yarn(2.0, 4096.0, 32.0, 1.0), rope_halves=True, scale=z["dim"] ** -0.5,
+               softcap=20.0, qk_norm="per_head", qkv_bias=True, value_gate=True)
     dense = dict(ffn_dim=z["dense"], activation="geglu_tanh")
     mix = dict(ffn_dim=z["expert_ffn"], experts=z["experts"], experts_per_token=z["top"], router="softmax", router_identity=z["identity"],
                expert_form="clamped", expert_limit=7.0, shared_dim=z["shared"], shared_limit=7.0)
     specs = [pkg.LayerSpec("attention" if i % 2 else "gla", **(att if i % 2 else gla), **(mix if i % 4 in (1, 2) else dense)) for i in range(layers)]
     return pkg.LayeredMetadata("Belizen", f"belizen-{name}", z["hidden"], LAYERED_VOCAB, specs, 1e-6, block="prenorm", residual_mult=0.5,
-                               embed_scale=8.0, logit_softcap=30.0)
+                               embed_scale=8.0, logit_softcap=25.0)
 
 
 def belizen_work(meta, rows, contexts, prompts):
