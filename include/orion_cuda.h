@@ -128,14 +128,19 @@ void orion_cuda_model_destroy(OrionModel *model);
  * Parallel: h = RMSNorm(x); the mixer and the feed-forward each read h plus a causal per-channel
  * convolution of h over `conv_taps` tokens, and both results are added to x.
  * Sandwich: x += m RMSNorm(mixer(RMSNorm(x))), then x += m RMSNorm(ffn(RMSNorm(x))), m = residual_mult.
+ * Prenorm: x += m mixer(RMSNorm(x)), then x += m ffn(RMSNorm(x)).
+ * Gated post-norm: x += m RMSNorm(g mixer(x)), then x += m RMSNorm(g' ffn(x)); the gates are sigmoids of
+ * projections of the same x, with biases, one per value.
  * The logits are the final norm's output times the embedding table or an output matrix of their own.
- * Metapel is a design with parallel blocks, Zulozen one with sandwich blocks. */
+ * Metapel is a design with parallel blocks, Zulozen one with sandwich blocks, Belizen one with prenorm
+ * blocks, Vusenex one with gated post-norm blocks. */
 enum { ORION_MIXER_MIN_GRU = 0, ORION_MIXER_LATENT_ATTENTION = 1, ORION_MIXER_ATTENTION = 2, ORION_MIXER_GLA = 3 };
-enum { ORION_BLOCK_PARALLEL = 0, ORION_BLOCK_SANDWICH = 1, ORION_BLOCK_PRENORM = 2 };
+enum { ORION_BLOCK_PARALLEL = 0, ORION_BLOCK_SANDWICH = 1, ORION_BLOCK_PRENORM = 2, ORION_BLOCK_GATED_POSTNORM = 3 };
 enum { ORION_ACT_GELU_TANH = 0, ORION_ACT_RELU2 = 1, ORION_ACT_GEGLU_TANH = 2 };
 enum { ORION_QK_NORM_NONE = 0, ORION_QK_NORM_ALL_HEADS = 1, ORION_QK_NORM_PER_HEAD = 2 };
-enum { ORION_ROUTER_SIGMOID_INPUT = 0, ORION_ROUTER_SOFTMAX = 1 };
-enum { ORION_EXPERT_SWIGLU = 0, ORION_EXPERT_CLAMPED = 1 };
+enum { ORION_SINK_NONE = 0, ORION_SINK_LEARNED = 1, ORION_SINK_ZERO = 2 };
+enum { ORION_ROUTER_SIGMOID_INPUT = 0, ORION_ROUTER_SOFTMAX = 1, ORION_ROUTER_SOFTMAX_RENORM = 2 };
+enum { ORION_EXPERT_SWIGLU = 0, ORION_EXPERT_CLAMPED = 1, ORION_EXPERT_GELU = 2 };
 typedef struct OrionLayerDesc {
   uint32_t mixer;    /* ORION_MIXER_* */
   uint32_t ffn_dim;  /* width of the feed-forward, or of each of its experts; 0 = the layer has none */
@@ -149,8 +154,8 @@ typedef struct OrionLayerDesc {
   /* attention: key/value heads (each shared by heads / kv_heads query heads); chunk size (a position sees
    * those before it in its own chunk, chunks counted from position 0; 0 = no chunks); how queries and
    * keys are normalised before the rotation (ORION_QK_NORM_*: RMS over all heads at once, or per head with
-   * gains that the heads share), whether every head has a learned logit in its softmax denominator, and
-   * whether a sigmoid per head gates its output */
+   * gains that the heads share), whether the softmax denominator holds a further logit that carries no value
+   * (ORION_SINK_*: none, a learned one per head, or zero), and whether a sigmoid per head gates its output */
   uint32_t kv_heads, chunk, qk_norm, sinks, head_gate;
   /* dense feed-forward (experts = 0): ORION_ACT_* (the gated one in prenorm blocks only), and whether both
    * projections have biases (sandwich blocks only) */
@@ -173,9 +178,21 @@ typedef struct OrionLayerDesc {
   /* router: ORION_ROUTER_SIGMOID_INPUT (sigmoid of the logits, the score multiplies the expert's input) or
    * ORION_ROUTER_SOFTMAX (over all outputs; the score multiplies the expert's output; a correction per output
    * takes part in the choice only); outputs past the experts whose expert returns its input. Experts:
-   * ORION_EXPERT_*, with the limits of the clamped form */
+   * ORION_EXPERT_*, with the limits of the clamped form. ORION_ROUTER_SOFTMAX_RENORM: softmax without a
+   * correction, the chosen scores divided by their sum. ORION_EXPERT_GELU: W_down gelu(W_up h), no gate, the
+   * exact form */
   uint32_t router, router_identity, expert_form;
   double expert_limit, shared_limit;
+  /* ORION_ROUTER_SOFTMAX_RENORM: the experts form router_groups groups of neighbours, and only those of the
+   * router_keep groups with the largest scores in them can be chosen (0 = any expert) */
+  uint32_t router_groups, router_keep;
+  /* attention: the values are the keys as projected, before their norm (ORION_QK_NORM_ALL_HEADS, no rotation,
+   * value_dim = dim, no v projection; qkv_bias: biases of q and k); a learned multiple per head of the
+   * logarithm of the distance is taken off the scores (with keys_as_values only); the query at position p is
+   * multiplied by 1 + q_temp_coef ln(floor((p + 1) / q_temp_every) + 1) (q_temp_every = 0: not at all) */
+  uint32_t keys_as_values, distance_bias;
+  double q_temp_coef, q_temp_every;
+  uint32_t ungated; /* latent_attention: the output has no gate */
 } OrionLayerDesc;
 typedef struct OrionLayeredDesc {
   uint32_t hidden_size, vocab_size, num_layers;
@@ -196,6 +213,13 @@ typedef struct OrionLayeredDesc {
    * state of its own; ahead of a pass the rows of `loop.step` join the stream, and from the second pass on
    * what entered the first layer of the model. Prenorm blocks only */
   uint32_t loop_start, loop_stop, loop_times;
+  uint32_t scalar_norms;            /* the gain of a norm of the residual stream's width is one number */
+  /* Gated post-norm blocks: the embedding has further tables. `pos`: a row for each of learned_positions
+   * positions (0 = no such table), no sequence is longer. `bigram`: rows chosen by (previous token *
+   * bigram_mul_prev + token * bigram_mul_cur) mod bigram_buckets (0 = no such table), and a last one for a
+   * sequence's first token */
+  uint32_t learned_positions;
+  uint64_t bigram_buckets, bigram_mul_prev, bigram_mul_cur;
 } OrionLayeredDesc;
 int orion_cuda_model_create_layered(OrionBackend *backend, const OrionLayeredDesc *desc, OrionModel **out);
 /* State slots of the model: 0 for models that carry nothing but the KV cache from step to step. */

@@ -14,7 +14,7 @@ from .errors import (BackendError, CacheExhausted, ContextLengthExceeded, CudaUn
 from .types import DType, Device, ForwardBatch, ForwardOutput, ModelMetadata
 from .backend import CudaBackend, device_count, is_available
 from .model import CudaModel, CudaTransformerModel, HfConfig, read_safetensors, write_safetensors
-from .layered import CudaLayeredModel, LayeredMetadata, LayerSpec, Loop, Yarn
+from .layered import Bigram, CudaLayeredModel, LayeredMetadata, LayerSpec, Loop, QueryTemperature, Yarn
 from .registry import load_model, model_class
 from .validate import Tolerance, ValidationReport, validate
 from .distributed import (Collective, CommunicationEstimate, NcclCollective, NcclCollectiveId, ParallelLayout, Rank,
@@ -32,5 +32,5 @@ __all__ = [
     "CommunicationEstimate", "NcclCollective", "NcclCollectiveId", "ParallelLayout", "Rank", "Shard", "ShardStrategy",
     "SingleRank", "shard_dimension", "ops", "PagedAttentionBench", "CacheExhausted", "ContextLengthExceeded",
     "QueueFull", "engine", "errors", "Engine", "KvCacheManager", "SamplingParams", "Scheduler", "SchedulerConfig",
-    "hash_block", "Loop", "Yarn",
+    "hash_block", "Bigram", "Loop", "QueryTemperature", "Yarn",
 ]

@@ -45,7 +45,9 @@ class OrionLayerDesc(C.Structure):
                                           "experts_per_token", "shared_dim", "keep_first", "rope_halves", "qkv_bias", "value_gate")] + \
                [(n, C.c_double) for n in ("softcap", "yarn_factor", "yarn_original", "yarn_fast", "yarn_slow", "decay_tau")] + \
                [(n, C.c_uint32) for n in ("decay_rank", "router", "router_identity", "expert_form")] + \
-               [(n, C.c_double) for n in ("expert_limit", "shared_limit")]
+               [(n, C.c_double) for n in ("expert_limit", "shared_limit")] + \
+               [(n, C.c_uint32) for n in ("router_groups", "router_keep", "keys_as_values", "distance_bias")] + \
+               [(n, C.c_double) for n in ("q_temp_coef", "q_temp_every")] + [("ungated", C.c_uint32)]
 
 
 class OrionLayeredDesc(C.Structure):
@@ -55,15 +57,18 @@ class OrionLayeredDesc(C.Structure):
                 ("num_state_slots", C.c_uint32), ("compute_dtype", C.c_uint32), ("max_batch_tokens", C.c_uint32),
                 ("max_batch_sequences", C.c_uint32), ("block", C.c_uint32), ("untied_lm_head", C.c_uint32),
                 ("residual_mult", C.c_double), ("embed_scale", C.c_double), ("logit_softcap", C.c_double),
-                ("loop_start", C.c_uint32), ("loop_stop", C.c_uint32), ("loop_times", C.c_uint32)]
+                ("loop_start", C.c_uint32), ("loop_stop", C.c_uint32), ("loop_times", C.c_uint32),
+                ("scalar_norms", C.c_uint32), ("learned_positions", C.c_uint32), ("bigram_buckets", C.c_uint64),
+                ("bigram_mul_prev", C.c_uint64), ("bigram_mul_cur", C.c_uint64)]
 
 
 MIXER_MIN_GRU, MIXER_LATENT_ATTENTION, MIXER_ATTENTION, MIXER_GLA = 0, 1, 2, 3
-BLOCK_PARALLEL, BLOCK_SANDWICH, BLOCK_PRENORM = 0, 1, 2
+BLOCK_PARALLEL, BLOCK_SANDWICH, BLOCK_PRENORM, BLOCK_GATED_POSTNORM = 0, 1, 2, 3
 ACT_GELU_TANH, ACT_RELU2, ACT_GEGLU_TANH = 0, 1, 2
 QK_NORM_NONE, QK_NORM_ALL_HEADS, QK_NORM_PER_HEAD = 0, 1, 2
-ROUTER_SIGMOID_INPUT, ROUTER_SOFTMAX = 0, 1
-EXPERT_SWIGLU, EXPERT_CLAMPED = 0, 1
+SINK_NONE, SINK_LEARNED, SINK_ZERO = 0, 1, 2
+ROUTER_SIGMOID_INPUT, ROUTER_SOFTMAX, ROUTER_SOFTMAX_RENORM = 0, 1, 2
+EXPERT_SWIGLU, EXPERT_CLAMPED, EXPERT_GELU = 0, 1, 2
 
 _lib = None
 

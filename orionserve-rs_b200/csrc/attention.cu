@@ -74,6 +74,8 @@ paged_attention_generic_kernel(const T *__restrict__ q, const T *__restrict__ ar
       for (uint32_t d = 0; d < hd; ++d)
         dot = __fadd_rn(dot, __fmul_rn(q_s[d], to_f32<T>(k[kv.col(slot, d)])));
       float s = __fmul_rn(dot, scale);
+      if (kv.factor_elems) s *= *reinterpret_cast<const float *>(arena + kv.factor(layer, table[pos / B], kvh, slot));
+      if (form.dist_mult) s -= form.dist_mult[head] * log1pf(form.dist_rate[head] * (float)(qpos - pos));
       if (form.softcap != 0.f) s = softcap_f(s, form.softcap);
       scores[p] = s;
       cmax = fmaxf(cmax, s);
@@ -145,6 +147,9 @@ constexpr int kMaxGroup = 8;      // query heads per kv head (N of the MMA)
 constexpr int kStashOffset = 512;
 constexpr int chunk_bytes(int dk, int dv) { return kBlk * (dk + dv) * 2; }  // K rows + V rows of one (block, head): 8 KiB at 128
 constexpr uint32_t decode_smem_bytes(int stages, int dk = kHd, int dv = kHd) { return kWarps * stages * chunk_bytes(dk, dv) + 4096; }
+// One set of rows for keys and values and an f32 factor per slot. The ring is at least as large as the merge buffers that reuse it.
+constexpr int joint_chunk_bytes(int d) { return kBlk * d * 2 + kBlk * 4; }
+constexpr uint32_t joint_smem_bytes(int stages, int d) { return kWarps * stages * joint_chunk_bytes(d) + 4096; }
 
 __device__ __forceinline__ float4 ld4(const float *p) { return *reinterpret_cast<const float4 *>(p); }
 __device__ __forceinline__ float4 add4(float4 a, float4 b) {
@@ -174,13 +179,15 @@ __device__ __forceinline__ void store_head_value(const AttnForm &form, uint32_t 
 __device__ uint32_t g_decode_error = 0;
 
 // DK, DV: sizes of the K and V rows. FORM: the mask, sinks, gate and row list of `form` and any number of query heads per
-// kv head (eight to a CTA); without it those branches and arguments are compiled out.
-template <int kStages, int DK, int DV, bool FORM>
+// kv head (eight to a CTA); without it those branches and arguments are compiled out. JOINT: one set of rows for keys and values, with the
+// factors of the keys (KvLayout::factor_elems), and the distance term of `form`.
+template <int kStages, int DK, int DV, bool FORM, bool JOINT = false>
 __global__ void __launch_bounds__(kWarps * 32)
 paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, KvLayout kv,
                     uint32_t layer, AttnBatch batch, uint32_t q_heads, uint32_t splits,
                     DecodeScratch scratch, bf16 *__restrict__ out, FusedQkv fq, AttnForm form) {
-  constexpr int kChunkBytes = chunk_bytes(DK, DV);
+  static_assert(!JOINT || (FORM && DK == DV), "one set of rows has one size");
+  constexpr int kChunkBytes = JOINT ? joint_chunk_bytes(DK) : chunk_bytes(DK, DV);
   extern __shared__ __align__(1024) uint8_t dsmem[];
   uint8_t *ring = dsmem;  // [kWarps][kStages][kChunkBytes]
   uint64_t *bars = reinterpret_cast<uint64_t *>(dsmem + kWarps * kStages * kChunkBytes);
@@ -316,6 +323,14 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
   // (columns 2*(lane%4) and +1), in the log2 domain.
   float sl2 = FORM && form.scale != 0.f ? form.scale * 1.4426950408889634f : 1.4426950408889634f / sqrtf((float)DK);
   float cap_in = 0.f, cap_out = 0.f;
+  float dm[2] = {0.f, 0.f}, dr[2] = {0.f, 0.f};  // distance term of this lane's two heads; its logarithm is to base 2, like the scores
+  if (JOINT && form.dist_mult) {
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      const uint32_t g = (lane & 3) * 2 + k;
+      if (g < group) dm[k] = form.dist_mult[head_first + g], dr[k] = form.dist_rate[head_first + g];
+    }
+  }
   if (FORM && form.softcap != 0.f) {  // the cap leaves scores in the log2 domain
     cap_out = form.softcap * 1.4426950408889634f, cap_in = 2.f * sl2 / form.softcap;
     sl2 = 1.f;
@@ -346,7 +361,7 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
       break;
     }
     const uint32_t kbase = smem_u32(my_ring + stage * kChunkBytes);
-    const uint32_t vbase = kbase + kBlk * DK * 2;
+    const uint32_t vbase = JOINT ? kbase : kbase + kBlk * DK * 2;
     const uint32_t lb = logical(b_begin + warp + i * kWarps);
     const uint32_t valid = min((uint32_t)kBlk, ctx - lb * kBlk);  // tokens of this block in context
     if (!FORM && fq.partial != nullptr && lb == nblocks - 1) {
@@ -383,10 +398,19 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
 #pragma unroll
       for (int k = 0; k < 4; ++k) s[k] = softcap_log2(s[k], cap_in, cap_out);
     }
-    s[0] = see_lo ? s[0] * sl2 : -INFINITY;
-    s[1] = see_lo ? s[1] * sl2 : -INFINITY;
-    s[2] = see_hi ? s[2] * sl2 : -INFINITY;
-    s[3] = see_hi ? s[3] * sl2 : -INFINITY;
+    if (JOINT) {
+      const float *factor = reinterpret_cast<const float *>(my_ring + stage * kChunkBytes + kBlk * DK * 2);
+      const float f_lo = factor[t_lo] * sl2, f_hi = factor[t_hi] * sl2, d_lo = (float)(ctx - 1 - lb * kBlk) - (float)t_lo;
+      s[0] = see_lo ? s[0] * f_lo - dm[0] * __log2f(fmaf(dr[0], d_lo, 1.f)) : -INFINITY;
+      s[1] = see_lo ? s[1] * f_lo - dm[1] * __log2f(fmaf(dr[1], d_lo, 1.f)) : -INFINITY;
+      s[2] = see_hi ? s[2] * f_hi - dm[0] * __log2f(fmaf(dr[0], d_lo - 8.f, 1.f)) : -INFINITY;
+      s[3] = see_hi ? s[3] * f_hi - dm[1] * __log2f(fmaf(dr[1], d_lo - 8.f, 1.f)) : -INFINITY;
+    } else {
+      s[0] = see_lo ? s[0] * sl2 : -INFINITY;
+      s[1] = see_lo ? s[1] * sl2 : -INFINITY;
+      s[2] = see_hi ? s[2] * sl2 : -INFINITY;
+      s[3] = see_hi ? s[3] * sl2 : -INFINITY;
+    }
     float bm0 = fmaxf(s[0], s[2]), bm1 = fmaxf(s[1], s[3]);
 #pragma unroll
     for (int off = 4; off <= 16; off <<= 1) {
@@ -726,23 +750,23 @@ bool attention_form_supported(KvLayout kv, uint32_t q_heads) {
   auto size = [](uint32_t d) { return d == 64 || d == 128; };
   const uint32_t dk = kv.head_dim, dv = kv.v_dim();
   return kv.block_size == kBlk && kv.swizzle == 1 && kv.num_kv_heads > 0 && q_heads % kv.num_kv_heads == 0 &&
-         q_heads / kv.num_kv_heads <= 128 && ((size(dk) && size(dv)) || (dk == 256 && dv == 256)) &&
+         (kv.factor_elems == 0 || (kv.factor_elems == 2 && dk == dv)) && q_heads / kv.num_kv_heads <= 128 && ((size(dk) && size(dv)) || (dk == 256 && dv == 256)) &&
          (uint64_t)kv.num_layers * kv.num_blocks * kv.num_kv_heads < (1ull << 31);
 }
 
 namespace {
 uint32_t group_tiles(KvLayout kv, uint32_t q_heads) { return (q_heads / kv.num_kv_heads + kMaxGroup - 1) / kMaxGroup; }
 
-template <int DK, int DV>
+template <int DK, int DV, bool JOINT>
 int launch_decode_form(const bf16 *q, const bf16 *arena, KvLayout kv, uint32_t layer, AttnBatch batch, uint32_t rows, uint32_t q_heads,
                        uint32_t splits, DecodeScratch scratch, AttnForm form, bf16 *out, cudaStream_t stream) {
   constexpr int kFormStages = 3;
+  constexpr uint32_t kSmem = JOINT ? joint_smem_bytes(kFormStages, DK) : decode_smem_bytes(kFormStages, DK, DV);
   static bool attr_set[kMaxDeviceOrdinals] = {};
-  ORION_CUDA_CHECK("paged_decode attr", ensure_dynamic_smem(paged_decode_kernel<kFormStages, DK, DV, true>,
-                                                            (int)decode_smem_bytes(kFormStages, DK, DV), attr_set));
-  ORION_CUDA_CHECK("paged_decode", launch_pdl(paged_decode_kernel<kFormStages, DK, DV, true>,
+  ORION_CUDA_CHECK("paged_decode attr", ensure_dynamic_smem(paged_decode_kernel<kFormStages, DK, DV, true, JOINT>, (int)kSmem, attr_set));
+  ORION_CUDA_CHECK("paged_decode", launch_pdl(paged_decode_kernel<kFormStages, DK, DV, true, JOINT>,
                                               dim3(kv.num_kv_heads * group_tiles(kv, q_heads), rows, splits), dim3(kWarps * 32),
-                                              (size_t)decode_smem_bytes(kFormStages, DK, DV), stream, q, arena, kv, layer, batch, q_heads,
+                                              (size_t)kSmem, stream, q, arena, kv, layer, batch, q_heads,
                                               splits, scratch, out, FusedQkv{}, form));
   ORION_TRY(after_launch("paged_decode"));
   if (splits == 1) return ORION_OK;
@@ -765,9 +789,11 @@ int launch_paged_attention_decode_form(const bf16 *q, const bf16 *arena, KvLayou
   if (splits > 1 && (scratch.partial_out == nullptr || splits > scratch.max_splits))
     return set_error(ORION_ERR_INTERNAL, "decode attention scratch too small for %u splits", splits);
   const uint32_t dk = kv.head_dim, dv = kv.v_dim();
-  auto run = dk == 256 ? launch_decode_form<256, 256>
-             : dk == 64 ? (dv == 64 ? launch_decode_form<64, 64> : launch_decode_form<64, 128>)
-                        : (dv == 64 ? launch_decode_form<128, 64> : launch_decode_form<128, 128>);
+  if (form.dist_mult && !kv.factor_elems) return set_error(ORION_ERR_INTERNAL, "decode attention takes distance terms where keys and values are one");
+  auto run = kv.factor_elems ? (dk == 256 ? launch_decode_form<256, 256, true> : (dk == 64 ? launch_decode_form<64, 64, true> : launch_decode_form<128, 128, true>))
+             : dk == 256     ? launch_decode_form<256, 256, false>
+             : dk == 64      ? (dv == 64 ? launch_decode_form<64, 64, false> : launch_decode_form<64, 128, false>)
+                             : (dv == 64 ? launch_decode_form<128, 64, false> : launch_decode_form<128, 128, false>);
   return run(q, arena, kv, layer, batch, rows, q_heads, splits, scratch, form, out, stream);
 }
 

@@ -36,18 +36,19 @@ constexpr int kKeys = 64;    // keys per tile
 constexpr int kStages = 2;
 constexpr int kThreads = 192;
 constexpr uint32_t kTmemO = 64;              // S: columns 0..63 of tensor memory, O behind them
-// DK, DV: sizes of the K and V rows, multiples of 64.
-template <int DK, int DV>
+// DK, DV: sizes of the K and V rows, multiples of 64. JOINT: one tile of rows is both K and V.
+template <int DK, int DV, bool JOINT>
 struct PrefillTcConfig {
   static constexpr int kQBytes = DK / 64 * kM * 128;     // 64-dim slabs of [128 rows][128 bytes]
   static constexpr int kKBytes = DK / 64 * kKeys * 128;  // 64-dim slabs of [64 keys][128 bytes]
   static constexpr int kVBytes = DV / 64 * kKeys * 128;
-  static constexpr int kStageBytes = kKBytes + kVBytes;  // K tile, then V tile
-  // P, [128 rows][128 bytes], takes the place of the K tile where that is large enough
-  static constexpr bool kOwnP = kKBytes < kM * 128;
+  static constexpr int kStageBytes = JOINT ? kKBytes : kKBytes + kVBytes;  // K tile, then V tile
+  // P, [128 rows][128 bytes], takes the place of the K tile where that is large enough and not needed any more
+  static constexpr bool kOwnP = JOINT || kKBytes < kM * 128;
   static constexpr int kPOffset = kQBytes + kStages * kStageBytes;
   static constexpr int kBarOffset = kPOffset + (kOwnP ? kM * 128 : 0);
-  static constexpr int kSmem = kBarOffset + 256 + 1024;
+  static constexpr int kFactorOffset = kBarOffset + 256;  // JOINT: the factors of a tile's keys, per stage
+  static constexpr int kSmem = kFactorOffset + (JOINT ? kStages * kKeys * 4 : 0) + 1024;
   static constexpr uint32_t kTmemCols = DV <= 64 ? 128 : (DV <= 128 ? 256 : 512);
 };
 constexpr float kRescaleThreshold = 8.0f;    // log2 units
@@ -57,18 +58,21 @@ __device__ uint32_t g_prefill_tc_error = 0;
 __device__ __forceinline__ void softmax_bar() { asm volatile("bar.sync 1, 128;" ::: "memory"); }  // warps 2..5
 
 // FORM: 1 = the mask, sinks and gate of `form`, 2 = besides them the soft cap, the kept first positions and the gates of values; what
-// is left out is compiled out.
+// is left out is compiled out. 3 = those of 1, one set of rows for keys and values with the factors of the keys
+// (KvLayout::factor_elems), and the distance term.
 template <int DK, int DV, int FORM>
 __global__ void __launch_bounds__(kThreads, DV <= 128 ? 2 : 1)
 paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const bf16 *__restrict__ q,
-                        KvLayout kv, uint32_t layer, AttnBatch batch, const PrefillTile *__restrict__ tiles, uint32_t q_heads,
-                        bf16 *__restrict__ out, AttnForm form) {
-  using Cfg = PrefillTcConfig<DK, DV>;
+                        const bf16 *__restrict__ arena, KvLayout kv, uint32_t layer, AttnBatch batch, const PrefillTile *__restrict__ tiles,
+                        uint32_t q_heads, bf16 *__restrict__ out, AttnForm form) {
+  constexpr bool JOINT = FORM == 3;
+  using Cfg = PrefillTcConfig<DK, DV, JOINT>;
   constexpr int kQBytes = Cfg::kQBytes, kKBytes = Cfg::kKBytes, kStageBytes = Cfg::kStageBytes;
   extern __shared__ uint8_t raw_smem[];
   uint8_t *smem = reinterpret_cast<uint8_t *>((reinterpret_cast<uintptr_t>(raw_smem) + 1023) & ~uintptr_t(1023));
   uint8_t *q_smem = smem;                 // [slab][row 128][128 B]
   uint8_t *ring = smem + kQBytes;         // [stage][K tile | V tile]
+  float *factors = reinterpret_cast<float *>(smem + Cfg::kFactorOffset);  // [stage][key]
   auto p_tile = [&](uint32_t stage) { return Cfg::kOwnP ? smem + Cfg::kPOffset : ring + stage * kStageBytes; };
   uint64_t *kv_full = reinterpret_cast<uint64_t *>(smem + Cfg::kBarOffset);
   uint64_t *kv_empty = kv_full + kStages;
@@ -133,7 +137,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
       for (uint32_t j = 0; j < ntiles; ++j) {
         const uint32_t s = j % kStages, use = j / kStages;
         if (!wait(&kv_empty[s], (use & 1) ^ 1)) { ok = false; break; }
-        mbar_arrive_expect_tx(&kv_full[s], kStageBytes);
+        mbar_arrive_expect_tx(&kv_full[s], kStageBytes + (JOINT ? kKeys * 4 : 0));
         uint8_t *k_dst = ring + s * kStageBytes, *v_dst = k_dst + kKBytes;
 #pragma unroll
         for (uint32_t b = 0; b < kKeys / kBlk; ++b) {
@@ -144,6 +148,10 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
 #pragma unroll
           for (int h = 0; h < DK / 64; ++h)
             tma_load_3d(k_dst + h * (kKeys * 128) + b * (kBlk * 128), &map_k, h * 64, 0, chunk, &kv_full[s]);
+          if (JOINT) {
+            bulk_copy_g2s(factors + s * kKeys + b * kBlk, arena + kv.factor(layer, block, kvh, 0), kBlk * 4, &kv_full[s]);
+            continue;
+          }
 #pragma unroll
           for (int h = 0; h < DV / 64; ++h)
             tma_load_3d(v_dst + h * (kKeys * 128) + b * (kBlk * 128), &map_v, h * 64, 0, chunk, &kv_full[s]);
@@ -160,7 +168,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         const uint32_t s = j % kStages;
         if (!wait(&kv_full[s], (j / kStages) & 1)) { ok = false; break; }
         tc_fence_after();
-        const uint32_t ka = smem_u32(ring + s * kStageBytes), va = ka + kKBytes;
+        const uint32_t ka = smem_u32(ring + s * kStageBytes), va = JOINT ? ka : ka + kKBytes;
         // S = Q K^T: 64-dim slabs, four 16-dim steps each (+32 bytes inside the swizzle atom)
 #pragma unroll
         for (int ks = 0; ks < DK / 16; ++ks) {
@@ -221,6 +229,8 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
       sl2 = 1.f;
       fixed = cap_out <= 60.f && !form.sinks;
     }
+    float dist_mult = 0.f, dist_rate = 0.f;
+    if (JOINT && form.dist_mult) dist_mult = form.dist_mult[head], dist_rate = form.dist_rate[head];
     float ref = -INFINITY, l = 0.f;
     if (FORM && form.sinks) ref = form.sinks[head] * 1.4426950408889634f, l = 1.f;
     for (uint32_t j = 0; j < ntiles; ++j) {
@@ -234,6 +244,21 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
       const bool straight = FORM != 2 || j * (kKeys / kBlk) >= kept_blk || kept_blk == block0;  // the tile's keys follow one another
       const int key0 = (int)(logical(j * (kKeys / kBlk)) * kBlk);
       float mx = -INFINITY;
+      if (JOINT) {
+        if (!__all_sync(0xffffffffu, wait(&kv_full[s], (j / kStages) & 1))) ok = false;  // the factors landed with the tile
+        const float4 *factor = reinterpret_cast<const float4 *>(factors + s * kKeys);
+        const float near = fmaf(dist_rate, (float)(pos - key0), 1.f);  // the logarithm's argument at the tile's first key
+#pragma unroll
+        for (int i = 0; i < kKeys; i += 4) {
+          const float4 f = factor[i / 4];
+          const float fs[4] = {f.x, f.y, f.z, f.w};
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const float v = __uint_as_float(sr[(i + k) >> 5][(i + k) & 31]) * (fs[k] * sl2);
+            sr[(i + k) >> 5][(i + k) & 31] = __float_as_uint(v - dist_mult * __log2f(fmaf(-dist_rate, (float)(i + k), near)));
+          }
+        }
+      }
       if (FORM == 2 && form.softcap != 0.f) {
         float most = 0.f;
 #pragma unroll
@@ -256,7 +281,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         } else {
 #pragma unroll
           for (int i = 0; i < kKeys; ++i) {
-            const float v = __uint_as_float(sr[i >> 5][i & 31]) * sl2;
+            const float v = JOINT ? __uint_as_float(sr[i >> 5][i & 31]) : __uint_as_float(sr[i >> 5][i & 31]) * sl2;
             sr[i >> 5][i & 31] = __float_as_uint(v);
             mx = fmaxf(mx, v);
           }
@@ -268,7 +293,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
 #pragma unroll
         for (int i = 0; i < kKeys; ++i) {
           const int key = from[i / kBlk] + i % kBlk;
-          const float v = (key <= pos && (!FORM || key >= low || (FORM == 2 && key < keep))) ? __uint_as_float(sr[i >> 5][i & 31]) * sl2 : -INFINITY;
+          const float v = (key <= pos && (!FORM || key >= low || (FORM == 2 && key < keep))) ? __uint_as_float(sr[i >> 5][i & 31]) * (JOINT ? 1.f : sl2) : -INFINITY;
           sr[i >> 5][i & 31] = __float_as_uint(v);
           mx = fmaxf(mx, v);
         }
@@ -375,12 +400,12 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
 // no swizzle of its own (the rows are stored pre-permuted).
 int arena_map(const bf16 *arena, KvLayout kv, bool values, const CUtensorMap **out) {
   static std::mutex mu;
-  static std::map<std::tuple<const void *, uint64_t, uint32_t, uint32_t, bool>, CUtensorMap> cache;
+  static std::map<std::tuple<const void *, uint64_t, uint32_t, uint64_t, bool>, CUtensorMap> cache;
   EncodeFn fn = encode_fn();
   if (!fn) return set_error(ORION_ERR_BACKEND, "backend cuda failed at tensor map: driver entry point missing");
   const uint64_t chunks = (uint64_t)kv.num_layers * kv.num_blocks * kv.num_kv_heads;
   std::lock_guard<std::mutex> lock(mu);
-  auto key = std::make_tuple((const void *)arena, chunks, kv.head_dim, kv.v_dim(), values);
+  auto key = std::make_tuple((const void *)arena, chunks, kv.head_dim, (uint64_t)kv.chunk_elems(), values);
   auto it = cache.find(key);
   if (it == cache.end()) {
     if (cache.size() > 4096) cache.clear();
@@ -388,7 +413,7 @@ int arena_map(const bf16 *arena, KvLayout kv, bool values, const CUtensorMap **o
     const cuuint64_t cols = values ? kv.v_dim() : kv.head_dim;
     const cuuint64_t dims[3] = {cols, (cuuint64_t)kBlk, chunks};
     const cuuint64_t strides[2] = {cols * 2, (cuuint64_t)kv.chunk_elems() * 2};
-    bf16 *base = const_cast<bf16 *>(arena) + (values ? (size_t)kBlk * kv.head_dim : 0);
+    bf16 *base = const_cast<bf16 *>(arena) + (values && !kv.factor_elems ? (size_t)kBlk * kv.head_dim : 0);
     const cuuint32_t box[3] = {64, (cuuint32_t)kBlk, 1};
     const cuuint32_t estr[3] = {1, 1, 1};
     const CUresult r = fn(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, base, dims, strides, box, estr,
@@ -406,14 +431,14 @@ int arena_map(const bf16 *arena, KvLayout kv, bool values, const CUtensorMap **o
 template <int DK, int DV, int FORM>
 int launch_prefill_tc(const bf16 *q, const bf16 *arena, KvLayout kv, uint32_t layer, AttnBatch batch, const PrefillTile *tiles,
                       uint32_t num_tiles, uint32_t q_heads, AttnForm form, bf16 *out, cudaStream_t stream) {
-  using Cfg = PrefillTcConfig<DK, DV>;
+  using Cfg = PrefillTcConfig<DK, DV, FORM == 3>;
   const CUtensorMap *mk = nullptr, *mv = nullptr;
   ORION_TRY(arena_map(arena, kv, false, &mk));
   ORION_TRY(arena_map(arena, kv, true, &mv));
   static bool attr_set[kMaxDeviceOrdinals] = {};
   ORION_CUDA_CHECK("paged_prefill_tc attr", ensure_dynamic_smem(paged_prefill_tc_kernel<DK, DV, FORM>, Cfg::kSmem, attr_set));
   ORION_CUDA_CHECK("paged_prefill_tc", launch_pdl(paged_prefill_tc_kernel<DK, DV, FORM>, dim3(kv.num_kv_heads, num_tiles), dim3(kThreads),
-                                                  (size_t)Cfg::kSmem, stream, *mk, *mv, q, kv, layer, batch, tiles, q_heads, out, form));
+                                                  (size_t)Cfg::kSmem, stream, *mk, *mv, q, arena, kv, layer, batch, tiles, q_heads, out, form));
   count_launch();
   ORION_CUDA_CHECK("paged_prefill_tc", cudaGetLastError());
   return ORION_OK;
@@ -445,6 +470,13 @@ int launch_paged_attention_prefill_form(const bf16 *q, const bf16 *arena, KvLayo
   if (!attention_form_supported(kv, q_heads) || encode_fn() == nullptr)
     return set_error(ORION_ERR_INTERNAL, "tensor-core prefill attention does not cover this shape");
   const uint32_t dk = kv.head_dim, dv = kv.v_dim();
+  if (form.dist_mult && !kv.factor_elems) return set_error(ORION_ERR_INTERNAL, "prefill attention takes distance terms where keys and values are one");
+  if (kv.factor_elems) {
+    if (form.softcap != 0.f || form.range.keep || form.value_gate)
+      return set_error(ORION_ERR_INTERNAL, "prefill attention over one set of rows has no soft cap, kept positions or gates of values");
+    auto joint = dk == 256 ? launch_prefill_tc<256, 256, 3> : (dk == 64 ? launch_prefill_tc<64, 64, 3> : launch_prefill_tc<128, 128, 3>);
+    return joint(q, arena, kv, layer, batch, tiles, num_tiles, q_heads, form, out, stream);
+  }
   auto pick = [&](auto plain, auto more) { return form.softcap != 0.f || form.range.keep || form.value_gate ? more : plain; };
   auto run = dk == 256  ? pick(launch_prefill_tc<256, 256, 1>, launch_prefill_tc<256, 256, 2>)
              : dk == 64 ? (dv == 64 ? pick(launch_prefill_tc<64, 64, 1>, launch_prefill_tc<64, 64, 2>)

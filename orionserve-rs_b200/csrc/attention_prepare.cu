@@ -1,6 +1,7 @@
 // What attention with query / key norms, rotation of part of each head and output gates needs between its joint projection
 // and the attention kernels: one pass over the projection's partial sums that normalises, rotates, and leaves queries, cached
-// keys and values, and gates. One CTA per row where a norm spans all heads, one warp per row and head where it does not.
+// keys and values, and gates. One CTA per row where a norm spans all heads, one warp per row and head where it does not. Where the
+// values are the keys before their norm, the cache gets them once, beside the factor of that norm.
 #include "kernels.h"
 #include "mma.cuh"
 
@@ -35,10 +36,11 @@ attention_prepare_kernel(const float *__restrict__ partial, uint32_t splits, siz
   pdl_wait();
   const uint32_t row = blockIdx.x, tid = threadIdx.x, half = in.rope_dims / 2;
   const float *p = partial + (size_t)row * in.ld;
-  const uint32_t nq = in.q_heads * in.dim, nk = in.kv_heads * in.dim, nv = in.kv_heads * in.value_dim;
+  const uint32_t nq = in.q_heads * in.dim, nk = in.kv_heads * in.dim, nv = in.keys_as_values ? 0 : in.kv_heads * in.value_dim;
   float sq = 0.f, sk = 0.f;
+  auto projected = [&](uint32_t i) { return fold(p + i, splits, split_stride) + (in.bias ? in.bias[i] : 0.f); };
   for (uint32_t i = tid; i < nq + nk; i += blockDim.x) {
-    const float v = fold(p + i, splits, split_stride);
+    const float v = projected(i);
     if (i < nq) sq += v * v;
     else sk += v * v;
   }
@@ -46,12 +48,23 @@ attention_prepare_kernel(const float *__restrict__ partial, uint32_t splits, siz
   const float scale_q = 1.0f / sqrtf(ss.x / (float)nq + in.eps), scale_k = 1.0f / sqrtf(ss.y / (float)nk + in.eps);
   const float *cs = in.rope_cos + (size_t)positions[row] * half, *sn = in.rope_sin + (size_t)positions[row] * half;
   const uint32_t block = slot_block[row], slot = slot_slot[row];
+  if (in.keys_as_values) {
+    const float factor = in.q_factor ? in.q_factor[positions[row]] * scale_q : scale_q;
+    for (uint32_t i = tid; i < nq + nk; i += blockDim.x) {
+      const float v = projected(i);
+      const uint32_t c = i < nq ? i : i - nq, head = c / in.dim, d = c % in.dim;
+      if (i < nq) q_out[((size_t)row * in.q_heads + head) * kv.head_dim + d] = from_f32<T>(v * factor * in.q_norm[i]);
+      else arena[kv.row(layer, block, head, 0, slot) + kv.col(slot, d)] = from_f32<T>(v);
+    }
+    for (uint32_t h = tid; h < in.kv_heads; h += blockDim.x) *reinterpret_cast<float *>(arena + kv.factor(layer, block, h, slot)) = scale_k;
+    return;
+  }
   for (uint32_t i = tid; i < nq + nk; i += blockDim.x) {
     const bool is_q = i < nq;
     const uint32_t c = is_q ? i : i - nq, head = c / in.dim, d = c % in.dim;
     const float *w = is_q ? in.q_norm : in.k_norm;
     const float scale = is_q ? scale_q : scale_k;
-    auto value = [&](uint32_t at) { return w ? fold(p + at, splits, split_stride) * scale * w[is_q ? at : at - nq] : fold(p + at, splits, split_stride); };
+    auto value = [&](uint32_t at) { return w ? projected(at) * scale * w[is_q ? at : at - nq] : projected(at); };
     float v = value(i);
     if (d < 2 * half) {
       const float other = value((d & 1) ? i - 1 : i + 1), co = cs[d >> 1], si = sn[d >> 1];
@@ -78,8 +91,9 @@ __device__ __forceinline__ void store4<bf16>(bf16 *p, float4 v) {
 
 // The same, four columns per thread and GROUPS rounds kept in registers, so each partial sum is read once: every size and
 // stride a multiple of four. SLABS: the projection has at most that many (prompts; 0 = any number); gains and angles are then
-// read when they are needed, not while the projection is still running, which leaves registers for more rows per SM.
-template <typename T, int GROUPS, int SLABS>
+// read when they are needed, not while the projection is still running, which leaves registers for more rows per SM. KEYS: keys as
+// values, with biases.
+template <typename T, int GROUPS, int SLABS, bool KEYS>
 __global__ void __launch_bounds__(512, SLABS == 0 ? 1 : (SLABS == 1 ? 3 : 2))
 attention_prepare_vec_kernel(const float *__restrict__ partial, uint32_t splits, size_t split_stride, AttnInputs in,
                              const uint32_t *__restrict__ positions, const uint32_t *__restrict__ slot_block,
@@ -89,12 +103,16 @@ attention_prepare_vec_kernel(const float *__restrict__ partial, uint32_t splits,
   pdl_trigger();
   const uint32_t row = blockIdx.x, tid = threadIdx.x, half = in.rope_dims / 2;
   const float *p = partial + (size_t)row * in.ld;
-  const uint32_t nq = in.q_heads * in.dim, nk = in.kv_heads * in.dim, nv = in.kv_heads * in.value_dim, all = nq + nk + nv;
+  const uint32_t nq = in.q_heads * in.dim, nk = in.kv_heads * in.dim, nv = KEYS ? 0 : in.kv_heads * in.value_dim, all = nq + nk + nv;
   const uint32_t pos = positions[row], block = slot_block[row], slot = slot_slot[row];
   // gain and angles of the four columns from i on
   auto constants = [&](uint32_t i, float4 &gain, float2 &co, float2 &si) {
     gain = make_float4(1.f, 1.f, 1.f, 1.f), co = make_float2(1.f, 1.f), si = make_float2(0.f, 0.f);
     if (i >= nq + nk) return;
+    if (KEYS) {
+      if (i < nq) gain = *reinterpret_cast<const float4 *>(in.q_norm + i);
+      return;
+    }
     if (in.q_norm) gain = *reinterpret_cast<const float4 *>(i < nq ? in.q_norm + i : in.k_norm + (i - nq));
     const uint32_t d = (i < nq ? i : i - nq) % in.dim;
     if (d < in.rope_dims) {
@@ -119,20 +137,29 @@ attention_prepare_vec_kernel(const float *__restrict__ partial, uint32_t splits,
     v[g] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (i >= all) continue;
     v[g] = sum_slabs4_most<SLABS>(p + i, splits, split_stride);
+    if (KEYS && in.bias) {
+      const float4 b = *reinterpret_cast<const float4 *>(in.bias + i);
+      v[g] = make_float4(v[g].x + b.x, v[g].y + b.y, v[g].z + b.z, v[g].w + b.w);
+    }
     const float s = v[g].x * v[g].x + v[g].y * v[g].y + v[g].z * v[g].z + v[g].w * v[g].w;
     if (i < nq) sq += s;
     else if (i < nq + nk) sk += s;
   }
   if (gate && tid < in.q_heads) gate[(size_t)row * in.q_heads + tid] = sigmoid_f(fold(p + all + tid, splits, split_stride));
   const float2 ss = block_sum2(sq, sk, red);
-  const float scale_q = in.q_norm ? 1.0f / sqrtf(ss.x / (float)nq + in.eps) : 1.f;
-  const float scale_k = in.q_norm ? 1.0f / sqrtf(ss.y / (float)nk + in.eps) : 1.f;
+  const float scale_q = (KEYS || in.q_norm ? 1.0f / sqrtf(ss.x / (float)nq + in.eps) : 1.f) * (KEYS && in.q_factor ? in.q_factor[pos] : 1.f);
+  const float scale_k = KEYS || in.q_norm ? 1.0f / sqrtf(ss.y / (float)nk + in.eps) : 1.f;
+  if (KEYS && tid < in.kv_heads) *reinterpret_cast<float *>(arena + kv.factor(layer, block, tid, slot)) = scale_k;
 #pragma unroll
   for (int g = 0; g < GROUPS; ++g) {
     const uint32_t i = (tid + g * blockDim.x) * 4;
     if (i >= all) continue;
     float4 x = v[g];
-    if (i < nq + nk) {
+    if (KEYS) {
+      const int e = kLate ? 0 : g;
+      if (kLate) constants(i, gain[e], co[e], si[e]);
+      if (i < nq) x = make_float4(x.x * scale_q * gain[e].x, x.y * scale_q * gain[e].y, x.z * scale_q * gain[e].z, x.w * scale_q * gain[e].w);
+    } else if (i < nq + nk) {
       const int e = kLate ? 0 : g;
       if (kLate) constants(i, gain[e], co[e], si[e]);
       const float s = i < nq ? scale_q : scale_k;
@@ -306,14 +333,24 @@ attention_prepare_lanes_kernel(const float *__restrict__ partial, uint32_t split
 
 template <typename T>
 __global__ void arena_rows_kernel(const T *__restrict__ arena, KvLayout kv, uint32_t dim, uint32_t value_dim, float *__restrict__ out) {
+  const bool factors = kv.factor_elems > 0;  // in the place of V rows: one value per slot
+  if (factors) value_dim = 1;
   const size_t tokens = (size_t)kv.num_blocks * kv.num_kv_heads * kv.block_size, keys = tokens * dim, all = keys + tokens * value_dim;
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < all; i += (size_t)gridDim.x * blockDim.x) {
     const uint32_t is_v = i >= keys, n = is_v ? value_dim : dim;
     const size_t j = is_v ? i - keys : i, t = j / n;
     const uint32_t slot = t % kv.block_size, head = t / kv.block_size % kv.num_kv_heads;
     const uint32_t block = (uint32_t)(t / kv.block_size / kv.num_kv_heads);
-    out[i] = to_f32<T>(arena[kv.row(0, block, head, is_v, slot) + kv.col(slot, j % n)]);
+    out[i] = factors && is_v ? *reinterpret_cast<const float *>(arena + kv.factor(0, block, head, slot))
+                             : to_f32<T>(arena[kv.row(0, block, head, is_v, slot) + kv.col(slot, j % n)]);
   }
+}
+
+template <typename T>
+__global__ void fill_factors_kernel(T *__restrict__ arena, KvLayout kv, float value) {
+  const size_t tokens = (size_t)kv.num_blocks * kv.num_kv_heads * kv.block_size;
+  for (size_t t = (size_t)blockIdx.x * blockDim.x + threadIdx.x; t < tokens; t += (size_t)gridDim.x * blockDim.x)
+    *reinterpret_cast<float *>(arena + kv.factor(0, (uint32_t)(t / kv.block_size / kv.num_kv_heads), t / kv.block_size % kv.num_kv_heads, t % kv.block_size)) = value;
 }
 
 inline int after_launch(const char *stage) {
@@ -322,13 +359,23 @@ inline int after_launch(const char *stage) {
   return ORION_OK;
 }
 
-template <typename T, int GROUPS, int SLABS>
+template <typename T, int GROUPS, int SLABS, bool KEYS>
 int launch_vec(const float *partial, uint32_t splits, size_t split_stride, AttnInputs in, const uint32_t *positions, const uint32_t *slot_block,
                const uint32_t *slot_slot, T *q_out, T *arena, KvLayout kv, uint32_t layer, float *gate, uint32_t rows, uint32_t threads,
                cudaStream_t stream) {
-  ORION_CUDA_CHECK("attention_prepare", launch_pdl(attention_prepare_vec_kernel<T, GROUPS, SLABS>, dim3(rows), dim3(threads), 0, stream, partial, splits,
+  ORION_CUDA_CHECK("attention_prepare", launch_pdl(attention_prepare_vec_kernel<T, GROUPS, SLABS, KEYS>, dim3(rows), dim3(threads), 0, stream, partial, splits,
                                                    split_stride, in, positions, slot_block, slot_slot, q_out, arena, kv, layer, gate));
   return after_launch("attention_prepare");
+}
+
+// The variant for this many rounds and slabs; null if there is none.
+template <typename T, bool KEYS>
+auto vec_variant(uint32_t rounds, int slabs) {
+  auto pick = [&](auto none, auto one, auto four) { return slabs == 1 ? one : (slabs == 4 ? four : none); };
+  return rounds == 1   ? pick(launch_vec<T, 1, 0, KEYS>, launch_vec<T, 1, 1, KEYS>, launch_vec<T, 1, 4, KEYS>)
+         : rounds == 2 ? pick(launch_vec<T, 2, 0, KEYS>, launch_vec<T, 2, 1, KEYS>, launch_vec<T, 2, 4, KEYS>)
+         : rounds == 4 ? pick(launch_vec<T, 4, 0, KEYS>, launch_vec<T, 4, 1, KEYS>, launch_vec<T, 4, 4, KEYS>)
+                       : launch_vec<T, 8, 0, KEYS>;
 }
 
 }  // namespace
@@ -362,19 +409,18 @@ int launch_attention_prepare(const float *partial, uint32_t splits, size_t split
                                                      slot_slot, q_out, arena, kv, layer, value_gate));
     return after_launch("attention_prepare");
   }
-  if (in.halves || in.bias || value_gate) return set_error(ORION_ERR_INTERNAL, "rotated halves, biases and gates per value come with norms per head");
+  if (in.halves || value_gate || (in.bias && !in.keys_as_values))
+    return set_error(ORION_ERR_INTERNAL, "rotated halves, biases and gates per value come with norms per head");
+  if (in.keys_as_values && (!in.q_norm || in.rope_dims || gate || kv.factor_elems * sizeof(T) != sizeof(float) || in.value_dim != in.dim))
+    return set_error(ORION_ERR_INTERNAL, "keys as values come with norms, without rotation and gates, and one set of rows");
   if ((in.q_norm == nullptr) != (in.k_norm == nullptr)) return set_error(ORION_ERR_INTERNAL, "query and key norms come together");
-  const uint32_t groups = (in.q_heads * in.dim + in.kv_heads * (in.dim + in.value_dim)) / 4;
+  const uint32_t groups = (in.q_heads * in.dim + in.kv_heads * (in.dim + (in.keys_as_values ? 0 : in.value_dim))) / 4;
   const uint32_t rounds = groups <= 256 ? 1 : (groups <= 1024 ? 2 : (groups <= 2048 ? 4 : 8));
   const uint32_t threads = ((groups + rounds - 1) / rounds + 31) / 32 * 32;
   if (in.dim % 4 == 0 && in.value_dim % 4 == 0 && in.rope_dims % 4 == 0 && in.ld % 4 == 0 && split_stride % 4 == 0 && kv.head_dim % 4 == 0 &&
-      kv.v_dim() % 4 == 0 && threads <= 512 && in.q_heads <= threads) {
+      kv.v_dim() % 4 == 0 && threads <= 512 && in.q_heads <= threads && in.kv_heads <= threads) {
     const int slabs = slab_variant(rows, splits);
-    auto pick = [&](auto none, auto one, auto four) { return slabs == 1 ? one : (slabs == 4 ? four : none); };
-    auto run = rounds == 1   ? pick(launch_vec<T, 1, 0>, launch_vec<T, 1, 1>, launch_vec<T, 1, 4>)
-               : rounds == 2 ? pick(launch_vec<T, 2, 0>, launch_vec<T, 2, 1>, launch_vec<T, 2, 4>)
-               : rounds == 4 ? pick(launch_vec<T, 4, 0>, launch_vec<T, 4, 1>, launch_vec<T, 4, 4>)
-                             : launch_vec<T, 8, 0>;
+    auto run = in.keys_as_values ? vec_variant<T, true>(rounds, slabs) : vec_variant<T, false>(rounds, slabs);
     return run(partial, splits, split_stride, in, positions, slot_block, slot_slot, q_out, arena, kv, layer, gate, rows, threads, stream);
   }
   ORION_CUDA_CHECK("attention_prepare", launch_pdl(attention_prepare_kernel<T>, dim3(rows), dim3(256), 0, stream, partial, splits, split_stride, in,
@@ -388,10 +434,17 @@ int launch_arena_rows(const T *arena, KvLayout kv, uint32_t dim, uint32_t value_
   return after_launch("arena_rows");
 }
 
+template <typename T>
+int launch_fill_factors(T *arena, KvLayout kv, float value, cudaStream_t stream) {
+  fill_factors_kernel<T><<<148 * 8, 256, 0, stream>>>(arena, kv, value);
+  return after_launch("fill_factors");
+}
+
 #define ORION_INSTANTIATE(T)                                                                                                            \
   template int launch_attention_prepare<T>(const float *, uint32_t, size_t, AttnInputs, const uint32_t *, const uint32_t *, const uint32_t *, \
                                            T *, T *, KvLayout, uint32_t, float *, uint32_t, cudaStream_t, T *);                         \
-  template int launch_arena_rows<T>(const T *, KvLayout, uint32_t, uint32_t, float *, cudaStream_t);
+  template int launch_arena_rows<T>(const T *, KvLayout, uint32_t, uint32_t, float *, cudaStream_t);                                   \
+  template int launch_fill_factors<T>(T *, KvLayout, float, cudaStream_t);
 ORION_INSTANTIATE(float)
 ORION_INSTANTIATE(bf16)
 

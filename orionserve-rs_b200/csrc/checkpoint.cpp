@@ -243,7 +243,7 @@ int load_checkpoint(ModelBase *model, const char *directory, uint64_t *tensors_l
       else return set_error(ORION_ERR_MODEL, "unsupported dtype %s (tensor `%s`)", t.dtype.c_str(), t.name.c_str());
       uint64_t count = 1;
       for (uint64_t s : t.shape) count *= s;
-      if (t.end > data_size || t.end - t.begin != count * es || t.shape.empty() || t.shape.size() > 2)
+      if (t.end > data_size || t.end - t.begin != count * es || t.shape.size() > 2)
         return set_error(ORION_ERR_MODEL, "malformed checkpoint %s: tensor `%s` does not match its byte range",
                          m.path.c_str(), t.name.c_str());
       ORION_TRY(model->load_tensor(t.name.c_str(), dtype, t.shape.data(), (int)t.shape.size(), bytes + 8 + hlen + t.begin));

@@ -141,12 +141,27 @@ __device__ __forceinline__ float relu2(float x) {
 template <typename T>
 __device__ __forceinline__ float silu_for(float x) { return x * sigmoid_for<T>(x); }
 
+// GELU in its exact form, x times the normal distribution function. For 16-bit results the tail of that function,
+// h = erfc(|x| / sqrt 2) / 2, is formula 7.1.26 of Abramowitz and Stegun's handbook (off by at most 1e-7).
+template <typename T>
+__device__ __forceinline__ float gelu_erf(float x) {
+  if constexpr (sizeof(T) == 2) {
+    const float y = fabsf(x) * 0.7071067811865476f, t = __fdividef(1.f, fmaf(0.3275911f, y, 1.f));
+    const float poly = t * fmaf(t, fmaf(t, fmaf(t, fmaf(t, 1.061405429f, -1.453152027f), 1.421413741f), -0.284496736f), 0.254829592f);
+    const float h = 0.5f * poly * __expf(-y * y);
+    return x >= 0.f ? x - x * h : x * h;
+  } else {
+    return 0.5f * x * (1.f + erff(x * 0.7071067811865476f));
+  }
+}
+
 // Gated feed-forwards, f(gate) * up: SwiGLU, GELU (tanh form), or a clamped form with both inputs limited,
-// g sigmoid(1.702 g) (u + 1) with g at most and |u| at most `limit`.
-enum GatedKind : uint32_t { kGatedSilu = 0, kGatedGelu = 1, kGatedClamped = 2 };
+// g sigmoid(1.702 g) (u + 1) with g at most and |u| at most `limit`. kPlainGelu: no gate, the exact GELU of up.
+enum GatedKind : uint32_t { kGatedSilu = 0, kGatedGelu = 1, kGatedClamped = 2, kPlainGelu = 3 };
 struct GatedAct {
   GatedKind kind = kGatedSilu;
   float limit = 0.f;
+  __host__ __device__ bool plain() const { return kind == kPlainGelu; }
 };
 template <typename T>
 __device__ __forceinline__ float gated(GatedAct f, float g, float u) {

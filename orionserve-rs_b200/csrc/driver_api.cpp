@@ -267,6 +267,8 @@ OrionEngine *orion_engine_create(OrionModel *model, OrionForwardFn forward, void
     return nullptr;
   }
   if (model && model->impl->logical_positions()) cfg.logical_decode_positions = cfg.recompute_on_preempt = true;
+  const size_t longest = model ? (size_t)model->impl->sequence_limit() : 0;
+  if (longest > 0 && (!cfg.max_model_len || *cfg.max_model_len > longest)) cfg.max_model_len = longest;
   if (model) {
     ModelBase *impl = model->impl.get();
     fn = [impl](const HostBatch &b, uint32_t *token_ids) -> int {

@@ -125,6 +125,17 @@ __device__ __forceinline__ void st4<bf16>(bf16 *dst, float4 v) {
   *reinterpret_cast<uint2 *>(dst) = packed;
 }
 
+template <typename T>
+__device__ __forceinline__ float4 load4(const T *p);
+template <>
+__device__ __forceinline__ float4 load4<float>(const float *p) { return ld4(p); }
+template <>
+__device__ __forceinline__ float4 load4<bf16>(const bf16 *p) {
+  const uint2 v = *reinterpret_cast<const uint2 *>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&v.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&v.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+
 // One CTA per output row, up to 1024 threads, CHUNKS float4 groups per thread kept
 // in registers: all loads of a row (residual + every split-K slab) are in flight
 // at once, so a 64-row decode batch costs one memory round trip, not sixteen.
@@ -534,6 +545,61 @@ int launch_embed_rmsnorm(const T *embed, const uint32_t *tokens, const float *no
 }
 
 namespace {
+// One CTA per row. VEC: four columns per thread and round (rows of the tables a multiple of four values).
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(kNormThreads)
+embed_tables_kernel(EmbedTables<T> e, EmbedBatch b, float *__restrict__ hidden, T *__restrict__ out, uint32_t H) {
+  pdl_trigger();
+  pdl_wait();
+  const uint32_t row = blockIdx.x, token = b.tokens[row], pos = b.positions[row], seq = b.seq_of_row[row];
+  size_t pair = e.buckets;
+  if (e.pairs && pos > 0) {
+    uint32_t prev;
+    if (row > 0 && b.seq_of_row[row - 1] == seq) {
+      prev = b.tokens[row - 1];
+    } else {
+      const uint32_t *table = b.tables_flat + b.table_offsets[seq];
+      prev = e.history[(size_t)table[(pos - 1) / e.block_size] * e.block_size + (pos - 1) % e.block_size];
+    }
+    pair = ((uint64_t)prev * e.mul_prev + (uint64_t)token * e.mul_cur) % e.buckets;
+  }
+  if (e.pairs && threadIdx.x == 0) e.history[(size_t)b.slot_block[row] * e.block_size + b.slot_slot[row]] = token;
+  const T *word = e.embed + (size_t)token * H, *more = e.pairs + pair * H, *place = e.places + (size_t)pos * H;
+  float *h = hidden + (size_t)row * H;
+  T *o = out + (size_t)row * H;
+  if (VEC) {
+    for (uint32_t c = threadIdx.x * 4; c < H; c += blockDim.x * 4) {
+      float4 v = load4<T>(word + c);
+      v = make_float4(v.x * e.scale, v.y * e.scale, v.z * e.scale, v.w * e.scale);
+      if (e.pairs) v = add4(v, load4<T>(more + c));
+      if (e.places) v = add4(v, load4<T>(place + c));
+      *reinterpret_cast<float4 *>(h + c) = v;
+      st4<T>(o + c, v);
+    }
+    return;
+  }
+  for (uint32_t c = threadIdx.x; c < H; c += blockDim.x) {
+    float v = to_f32<T>(word[c]) * e.scale;
+    if (e.pairs) v += to_f32<T>(more[c]);
+    if (e.places) v += to_f32<T>(place[c]);
+    h[c] = v;
+    o[c] = from_f32<T>(v);
+  }
+}
+}  // namespace
+
+template <typename T>
+int launch_embed_tables(EmbedTables<T> e, EmbedBatch b, float *hidden, T *out, uint32_t hidden_size, cudaStream_t stream) {
+  if (b.rows == 0) return ORION_OK;
+  if (e.pairs && (e.buckets == 0 || !e.history || e.block_size == 0)) return set_error(ORION_ERR_INTERNAL, "a table of pairs needs buckets and a history");
+  const bool vec = hidden_size % 4 == 0;
+  const uint32_t need = vec ? hidden_size / 4 : hidden_size, threads = need >= (uint32_t)kNormThreads ? kNormThreads : (need + 31) / 32 * 32;
+  ORION_CUDA_CHECK("embed_tables", launch_pdl(vec ? embed_tables_kernel<T, true> : embed_tables_kernel<T, false>, dim3(b.rows), dim3(threads), 0, stream, e,
+                                              b, hidden, out, hidden_size));
+  return after_launch("embed_tables");
+}
+
+namespace {
 template <typename T, int CHUNKS>
 int launch_residual_vec(const float *partial, uint32_t splits, size_t split_stride, float *hidden,
                         const float *norm_w, float eps, T *out, const uint32_t *row_map,
@@ -747,6 +813,11 @@ __device__ __forceinline__ float sublayer_value(const SublayerOutput &y, uint32_
     }
     v += y.weight ? y.weight[(size_t)row * y.top + k] * x : x;
   }
+  if (y.gate) {
+    float g = y.gate_bias[c];
+    for (uint32_t s = 0; s < y.gate_splits; ++s) g += y.gate[s * y.gate_stride + (size_t)row * y.gate_ld + c];
+    v *= sigmoid_for<T>(g);
+  }
   return v;
 }
 
@@ -782,28 +853,20 @@ post_norm_residual_kernel(SublayerOutput y, float *__restrict__ hidden, const fl
     row_cache[c] = v;
     ss += (Acc)v * (Acc)v;
   }
-  const float s2 = norm_scale<Acc>(block_sum<Acc>(ss, red), H, eps);
+  const float s2 = pre_w ? norm_scale<Acc>(block_sum<Acc>(ss, red), H, eps) : 1.f;
   T *o = out + (size_t)blockIdx.x * H;
-  for (uint32_t c = threadIdx.x; c < H; c += blockDim.x) o[c] = from_f32<T>(row_cache[c] * s2 * pre_w[c]);
+  for (uint32_t c = threadIdx.x; c < H; c += blockDim.x) o[c] = from_f32<T>(pre_w ? row_cache[c] * s2 * pre_w[c] : row_cache[c]);
 }
 
 // Row widths that are multiples of 4: a row's values stay in registers between the two norms. SLABS: every sum has
 // at most that many (prompts; 0 = any number); gains are then read when they are needed, which leaves registers for more rows
 // per SM.
-// POST: the output is normalised; otherwise it joins as it is, with the experts' weights, the identity experts and what `add` names.
-template <typename T>
-__device__ __forceinline__ float4 load4(const T *p);
-template <>
-__device__ __forceinline__ float4 load4<float>(const float *p) { return ld4(p); }
-template <>
-__device__ __forceinline__ float4 load4<bf16>(const bf16 *p) {
-  const uint2 v = *reinterpret_cast<const uint2 *>(p);
-  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&v.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162 *>(&v.y));
-  return make_float4(a.x, a.y, b.x, b.y);
-}
+// MODE: the output is normalised (kJoinPost), or it joins as it is, with the experts' weights, the identity experts and what `add` names
+// (kJoinPlain), or it is gated and normalised, with the experts' weights, and the sum need not be normalised (kJoinGated).
+enum JoinMode : int { kJoinPlain = 0, kJoinPost = 1, kJoinGated = 2 };
 __device__ __forceinline__ float4 axpy4(float a, float4 x, float4 y) { return make_float4(a * x.x + y.x, a * x.y + y.y, a * x.z + y.z, a * x.w + y.w); }
 
-template <typename T, int CHUNKS, int SLABS, bool POST>
+template <typename T, int CHUNKS, int SLABS, int MODE>
 __global__ void __launch_bounds__(512, SLABS == 0 ? 1 : (SLABS == 1 && CHUNKS <= 2 ? 3 : 2))
 post_norm_residual_vec_kernel(SublayerOutput y, float *__restrict__ hidden, const float *__restrict__ post_w, float mult, StreamAddition<T> add,
                               const float *__restrict__ pre_w, float eps, T *out, const uint32_t *__restrict__ row_map, uint32_t H) {
@@ -811,7 +874,7 @@ post_norm_residual_vec_kernel(SublayerOutput y, float *__restrict__ hidden, cons
   __shared__ Acc red[32];
   pdl_trigger();
   const uint32_t nvec = H / 4;
-  constexpr bool kLate = SLABS != 0;
+  constexpr bool kLate = SLABS != 0, POST = MODE != kJoinPlain, GATED = MODE == kJoinGated;
   constexpr int kEarly = kLate ? 1 : CHUNKS;
   float4 pw[kEarly], nw[kEarly];
   if (!kLate) {
@@ -821,7 +884,7 @@ post_norm_residual_vec_kernel(SublayerOutput y, float *__restrict__ hidden, cons
       pw[c] = nw[c] = make_float4(0.f, 0.f, 0.f, 0.f);
       if (idx < nvec) {
         if (POST) pw[c] = ld4(post_w + 4 * (size_t)idx);
-        nw[c] = ld4(pre_w + 4 * (size_t)idx);
+        if (!GATED || pre_w) nw[c] = ld4(pre_w + 4 * (size_t)idx);
       }
     }
   }
@@ -841,13 +904,19 @@ post_norm_residual_vec_kernel(SublayerOutput y, float *__restrict__ hidden, cons
     if (y.bias) v[c] = add4(v[c], ld4(y.bias + 4 * (size_t)idx));
     for (uint32_t k = 0; k < y.top; ++k) {
       const uint32_t at = y.place[(size_t)row * y.top + k];
-      if (POST) {
+      if (GATED) {
+        v[c] = axpy4(y.weight ? y.weight[(size_t)row * y.top + k] : 1.f, slabs(y.rows + (size_t)at * H + 4 * (size_t)idx, y.rows_splits, y.rows_stride), v[c]);
+      } else if (POST) {
         v[c] = add4(v[c], slabs(y.rows + (size_t)at * H + 4 * (size_t)idx, y.rows_splits, y.rows_stride));
       } else {
         const float4 e = at == kNoPlace ? load4<T>(static_cast<const T *>(y.identity) + (size_t)row * H + 4 * (size_t)idx)
                                         : slabs(y.rows + (size_t)at * H + 4 * (size_t)idx, y.rows_splits, y.rows_stride);
         v[c] = axpy4(y.weight ? y.weight[(size_t)row * y.top + k] : 1.f, e, v[c]);
       }
+    }
+    if (GATED) {
+      const float4 g = add4(slabs(y.gate + (size_t)row * y.gate_ld + 4 * (size_t)idx, y.gate_splits, y.gate_stride), ld4(y.gate_bias + 4 * (size_t)idx));
+      v[c] = make_float4(v[c].x * sigmoid_for<T>(g.x), v[c].y * sigmoid_for<T>(g.y), v[c].z * sigmoid_for<T>(g.z), v[c].w * sigmoid_for<T>(g.w));
     }
     if (POST) ss += (Acc)v[c].x * (Acc)v[c].x + (Acc)v[c].y * (Acc)v[c].y + (Acc)v[c].z * (Acc)v[c].z + (Acc)v[c].w * (Acc)v[c].w;
   }
@@ -867,8 +936,10 @@ post_norm_residual_vec_kernel(SublayerOutput y, float *__restrict__ hidden, cons
       if (add.shift) x[c] = add4(x[c], ld4(add.shift + 4 * (size_t)idx));
     }
     if (!row_map) *reinterpret_cast<float4 *>(h + 4 * (size_t)idx) = x[c];
+    if (GATED && !pre_w) st4<T>(out + (size_t)blockIdx.x * H + 4 * (size_t)idx, x[c]);
     ss += (Acc)x[c].x * (Acc)x[c].x + (Acc)x[c].y * (Acc)x[c].y + (Acc)x[c].z * (Acc)x[c].z + (Acc)x[c].w * (Acc)x[c].w;
   }
+  if (GATED && !pre_w) return;
   const float s2 = norm_scale<Acc>(block_sum<Acc>(ss, red), H, eps);
   T *o = out + (size_t)blockIdx.x * H;
 #pragma unroll
@@ -881,26 +952,27 @@ post_norm_residual_vec_kernel(SublayerOutput y, float *__restrict__ hidden, cons
 }
 
 namespace {
-template <typename T, int CHUNKS, int SLABS, bool POST>
+template <typename T, int CHUNKS, int SLABS, int MODE>
 int launch_post_norm_vec(SublayerOutput y, float *hidden, const float *post_w, float mult, StreamAddition<T> add, const float *pre_w, float eps,
                          T *out, const uint32_t *row_map, uint32_t out_rows, uint32_t H, uint32_t threads, cudaStream_t stream) {
-  ORION_CUDA_CHECK("sublayer_residual", launch_pdl(post_norm_residual_vec_kernel<T, CHUNKS, SLABS, POST>, dim3(out_rows), dim3(threads), 0, stream, y,
+  ORION_CUDA_CHECK("sublayer_residual", launch_pdl(post_norm_residual_vec_kernel<T, CHUNKS, SLABS, MODE>, dim3(out_rows), dim3(threads), 0, stream, y,
                                                    hidden, post_w, mult, add, pre_w, eps, out, row_map, H));
   return after_launch("sublayer_residual");
 }
 
-template <typename T, bool POST>
+template <typename T, int MODE>
 int launch_join(SublayerOutput y, float *hidden, const float *post_w, float mult, StreamAddition<T> add, const float *pre_w, float eps, T *out,
                 const uint32_t *row_map, uint32_t out_rows, uint32_t H, cudaStream_t stream) {
   if (out_rows == 0) return ORION_OK;
-  if (H % 4 == 0 && H / 4 <= 2048 && y.split_stride % 4 == 0 && y.rows_stride % 4 == 0) {
+  if (H % 4 == 0 && H / 4 <= 2048 && y.split_stride % 4 == 0 && y.rows_stride % 4 == 0 &&
+      (MODE != kJoinGated || (y.gate_ld % 4 == 0 && y.gate_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(y.gate) & 15) == 0))) {
     const uint32_t nvec = H / 4, threads = nvec >= 512 ? 512 : (nvec + 31) / 32 * 32, chunks = (nvec + threads - 1) / threads;
-    const uint32_t a = y.partial ? y.splits : 1, b = y.top ? y.rows_splits : 1;
-    const int slabs = slab_variant(out_rows, a > b ? a : b);
+    const uint32_t a = y.partial ? y.splits : 1, b = y.top ? y.rows_splits : 1, g = MODE == kJoinGated ? y.gate_splits : 1, ab = a > b ? a : b;
+    const int slabs = slab_variant(out_rows, ab > g ? ab : g);
     auto pick = [&](auto none, auto one, auto four) { return slabs == 1 ? one : (slabs == 4 ? four : none); };
-    auto run = chunks == 1   ? pick(launch_post_norm_vec<T, 1, 0, POST>, launch_post_norm_vec<T, 1, 1, POST>, launch_post_norm_vec<T, 1, 4, POST>)
-               : chunks == 2 ? pick(launch_post_norm_vec<T, 2, 0, POST>, launch_post_norm_vec<T, 2, 1, POST>, launch_post_norm_vec<T, 2, 4, POST>)
-                             : pick(launch_post_norm_vec<T, 4, 0, POST>, launch_post_norm_vec<T, 4, 1, POST>, launch_post_norm_vec<T, 4, 4, POST>);
+    auto run = chunks == 1   ? pick(launch_post_norm_vec<T, 1, 0, MODE>, launch_post_norm_vec<T, 1, 1, MODE>, launch_post_norm_vec<T, 1, 4, MODE>)
+               : chunks == 2 ? pick(launch_post_norm_vec<T, 2, 0, MODE>, launch_post_norm_vec<T, 2, 1, MODE>, launch_post_norm_vec<T, 2, 4, MODE>)
+                             : pick(launch_post_norm_vec<T, 4, 0, MODE>, launch_post_norm_vec<T, 4, 1, MODE>, launch_post_norm_vec<T, 4, 4, MODE>);
     return run(y, hidden, post_w, mult, add, pre_w, eps, out, row_map, out_rows, H, threads, stream);
   }
   const size_t smem = (size_t)H * sizeof(float);
@@ -916,12 +988,18 @@ int launch_join(SublayerOutput y, float *hidden, const float *post_w, float mult
 template <typename T>
 int launch_post_norm_residual(SublayerOutput y, float *hidden, const float *post_w, float mult, const float *pre_w, float eps, T *out,
                               const uint32_t *row_map, uint32_t out_rows, uint32_t H, cudaStream_t stream) {
-  return launch_join<T, true>(y, hidden, post_w, mult, StreamAddition<T>{}, pre_w, eps, out, row_map, out_rows, H, stream);
+  return launch_join<T, kJoinPost>(y, hidden, post_w, mult, StreamAddition<T>{}, pre_w, eps, out, row_map, out_rows, H, stream);
 }
 template <typename T>
 int launch_sublayer_residual(SublayerOutput y, float *hidden, float mult, StreamAddition<T> add, const float *pre_w, float eps, T *out,
                              const uint32_t *row_map, uint32_t out_rows, uint32_t H, cudaStream_t stream) {
-  return launch_join<T, false>(y, hidden, nullptr, mult, add, pre_w, eps, out, row_map, out_rows, H, stream);
+  return launch_join<T, kJoinPlain>(y, hidden, nullptr, mult, add, pre_w, eps, out, row_map, out_rows, H, stream);
+}
+template <typename T>
+int launch_gated_post_norm(SublayerOutput y, float *hidden, const float *post_w, float mult, const float *pre_w, float eps, T *out,
+                           const uint32_t *row_map, uint32_t out_rows, uint32_t H, cudaStream_t stream) {
+  if (!y.gate || !y.gate_bias || !post_w) return set_error(ORION_ERR_INTERNAL, "a gated output needs its gate, its bias and its norm");
+  return launch_join<T, kJoinGated>(y, hidden, post_w, mult, StreamAddition<T>{}, pre_w, eps, out, row_map, out_rows, H, stream);
 }
 
 namespace {
@@ -1071,6 +1149,9 @@ int launch_fill_normal(T *dst, size_t n, uint64_t seed, cudaStream_t stream) {
                                             uint32_t, uint32_t, cudaStream_t);                    \
   template int launch_sublayer_residual<T>(SublayerOutput, float *, float, StreamAddition<T>, const float *, float, T *, const uint32_t *, uint32_t, \
                                            uint32_t, cudaStream_t);                               \
+  template int launch_gated_post_norm<T>(SublayerOutput, float *, const float *, float, const float *, float, T *, const uint32_t *, uint32_t, \
+                                         uint32_t, cudaStream_t);                                 \
+  template int launch_embed_tables<T>(EmbedTables<T>, EmbedBatch, float *, T *, uint32_t, cudaStream_t); \
   template int launch_gated_act<T>(const float *, uint32_t, size_t, GatedAct, T *, uint32_t, uint32_t, uint32_t, cudaStream_t); \
   template int launch_convert_from_f32<T>(const float *, T *, size_t, cudaStream_t);              \
   template int launch_convert_to_f32<T>(const T *, float *, size_t, cudaStream_t);                \

@@ -20,8 +20,14 @@ namespace orion {
 struct KvLayout {
   uint32_t num_layers, num_blocks, num_kv_heads, block_size, head_dim, swizzle;
   uint32_t value_dim = 0;  // size of a V row; 0 = head_dim
+  // Not 0: the values are the keys before their norm, which is one factor per token and gains that the queries carry. A chunk
+  // then holds one set of rows, for both, followed by the factor of every slot in f32 (factor_elems elements of storage each).
+  uint32_t factor_elems = 0;
   __host__ __device__ uint32_t v_dim() const { return value_dim ? value_dim : head_dim; }
-  __host__ __device__ size_t chunk_elems() const { return size_t(block_size) * (head_dim + v_dim()); }
+  __host__ __device__ size_t row_elems() const {
+    return factor_elems ? (size_t(block_size) * head_dim + 7) / 8 * 8 : size_t(block_size) * (head_dim + v_dim());
+  }
+  __host__ __device__ size_t chunk_elems() const { return row_elems() + (size_t(block_size) * factor_elems + 7) / 8 * 8; }
   __host__ __device__ size_t layer_elems() const {
     return size_t(num_blocks) * num_kv_heads * chunk_elems();
   }
@@ -29,7 +35,11 @@ struct KvLayout {
   __host__ __device__ size_t row(uint32_t layer, uint32_t block, uint32_t head, uint32_t is_v,
                                  uint32_t slot) const {
     return layer * layer_elems() + (size_t(block) * num_kv_heads + head) * chunk_elems() +
-           (is_v ? size_t(block_size) * head_dim + size_t(slot) * v_dim() : size_t(slot) * head_dim);
+           (is_v && !factor_elems ? size_t(block_size) * head_dim + size_t(slot) * v_dim() : size_t(slot) * head_dim);
+  }
+  // Start of the factor of (layer, block, head, slot).
+  __host__ __device__ size_t factor(uint32_t layer, uint32_t block, uint32_t head, uint32_t slot) const {
+    return layer * layer_elems() + (size_t(block) * num_kv_heads + head) * chunk_elems() + row_elems() + size_t(slot) * factor_elems;
   }
   // Position of logical dim `d` inside the row of `slot`.
   __host__ __device__ uint32_t col(uint32_t slot, uint32_t d) const {
@@ -43,6 +53,25 @@ template <typename T>
 int launch_embed_rmsnorm(const T *embed, const uint32_t *tokens, const float *norm_w, float eps,
                          float *hidden, T *normed, uint32_t rows, uint32_t hidden_size,
                          cudaStream_t stream, float scale = 1.f, const float *shift = nullptr);  // hidden = scale * embed (+ shift, one vector)
+
+// An embedding made of several tables, and its rows in the storage type (not normalised): hidden[r] = scale * embed[token] +
+// pairs[row] + places[position], out[r] = hidden[r]. The row of `pairs` (null: none) is (previous token * mul_prev + token *
+// mul_cur) mod buckets, or `buckets` for a sequence's first token. A token whose predecessor came in an earlier step finds it in
+// `history`, the token of every cache slot ([blocks][block_size], written here). places (null: none) holds a row per position.
+template <typename T>
+struct EmbedTables {
+  const T *embed = nullptr, *pairs = nullptr, *places = nullptr;
+  uint64_t buckets = 0, mul_prev = 0, mul_cur = 0;
+  uint32_t *history = nullptr;
+  uint32_t block_size = 0;
+  float scale = 1.f;
+};
+struct EmbedBatch {
+  const uint32_t *tokens, *positions, *seq_of_row, *slot_block, *slot_slot, *tables_flat, *table_offsets;
+  uint32_t rows;
+};
+template <typename T>
+int launch_embed_tables(EmbedTables<T> e, EmbedBatch b, float *hidden, T *out, uint32_t hidden_size, cudaStream_t stream);
 
 // hidden[r] += sum_s partial[s][r] (+ nothing else); out[i] = rms_norm(hidden[src(i)]) * w,
 // src(i) = row_map ? row_map[i] : i. With row_map the residual is not written
@@ -108,6 +137,10 @@ struct SublayerOutput {
   size_t rows_stride = 0;
   const float *weight = nullptr;   // [rows][top] factors of the experts' rows; null = 1
   const void *identity = nullptr;  // [row][hidden] of T: what a choice with the place kNoPlace contributes
+  // A gate per value, sigmoid(gate + gate_bias), from columns of a projection's slabs (row stride gate_ld). Null: none.
+  const float *gate = nullptr, *gate_bias = nullptr;
+  uint32_t gate_splits = 0, gate_ld = 0;
+  size_t gate_stride = 0;
 };
 constexpr uint32_t kNoPlace = 0xFFFFFFFFu;
 template <typename T>
@@ -125,6 +158,11 @@ struct StreamAddition {
 template <typename T>
 int launch_sublayer_residual(SublayerOutput y, float *hidden, float mult, StreamAddition<T> add, const float *pre_w, float eps, T *out,
                              const uint32_t *row_map, uint32_t out_rows, uint32_t hidden_size, cudaStream_t stream);
+// Post-norm layers: hidden += mult * rms_norm(gated y) * post_w, where the experts' weights and the gate count; out = rms_norm(hidden) *
+// pre_w, or the rows of hidden themselves if pre_w is null.
+template <typename T>
+int launch_gated_post_norm(SublayerOutput y, float *hidden, const float *post_w, float mult, const float *pre_w, float eps, T *out,
+                           const uint32_t *row_map, uint32_t out_rows, uint32_t hidden_size, cudaStream_t stream);
 // x[r * ld + c] = cap * tanh(x[r * ld + c] / cap)
 int launch_softcap(float *x, uint32_t rows, uint32_t cols, uint32_t ld, float cap, cudaStream_t stream);
 
@@ -209,6 +247,9 @@ struct AttnForm {
   const float *gate = nullptr;    // [rows][q_heads] factors of the heads' outputs
   const void *value_gate = nullptr;  // [rows][q_heads * out_dim] of T: factors of the values
   float softcap = 0.f;            // scores become softcap * tanh(score / softcap); 0 = they stay
+  // [q_heads]: dist_mult * ln(1 + dist_rate * (distance to the key)) is taken off every score. Null: nothing. The tuned kernels
+  // take it where keys and values are one (KvLayout::factor_elems).
+  const float *dist_mult = nullptr, *dist_rate = nullptr;
   uint32_t out_dim = 0, ldo = 0;  // values stored per head and row stride of the output; 0 = v_dim() and q_heads * out_dim
   // Decode only: the batch rows that decode (item i of the scratch belongs to row_list[i]), and the first row of every
   // sequence, since several rows of one sequence may decode together. Null: every row, one per sequence.
@@ -230,12 +271,18 @@ int launch_paged_attention_generic(const T *q, const T *arena, KvLayout kv, uint
 // per_head: the other family of layouts. Every head is normalised by itself (gains of dim values, shared by the heads), dimension
 // i rotates with i + rope_dims / 2 if `halves` is set, q, k and v have biases ([q | k | v], may be null), and g has a column per
 // value: sigmoid(g) goes to `value_gate` [rows][q_heads * value_dim] (null: no such columns) instead of `gate`.
+//
+// keys_as_values (norms over all heads, nothing rotates, no gates): the projection holds [q | k] with biases ([q | k]). The cache gets
+// k as projected and the factor of its norm (KvLayout::factor_elems); q_norm holds, per value of the queries, the queries' gain times
+// that of the keys. The queries are also multiplied by q_factor[position] (null: 1).
 struct AttnInputs {
   uint32_t q_heads, kv_heads, dim, value_dim, rope_dims, ld;
   float eps;
   const float *q_norm, *k_norm, *rope_cos, *rope_sin;
   bool per_head = false, halves = false;
   const float *bias = nullptr;
+  bool keys_as_values = false;
+  const float *q_factor = nullptr;
 };
 template <typename T>
 int launch_attention_prepare(const float *partial, uint32_t splits, size_t split_stride, AttnInputs in, const uint32_t *positions,
@@ -244,6 +291,9 @@ int launch_attention_prepare(const float *partial, uint32_t splits, size_t split
 // K and V rows of one layer's arena as f32, [k|v][block][kv head][slot][dim] with dim values of a K row, value_dim of a V row.
 template <typename T>
 int launch_arena_rows(const T *arena, KvLayout kv, uint32_t dim, uint32_t value_dim, float *out, cudaStream_t stream);
+// One value for all factors of an arena (KvLayout::factor_elems).
+template <typename T>
+int launch_fill_factors(T *arena, KvLayout kv, float value, cudaStream_t stream);
 
 // Tuned prefill / mixed-batch path (bf16, head_dim 128, block 16): the batch is cut into
 // tiles of consecutive rows of one sequence (prefill_tile_positions rows at most); one CTA per
@@ -430,12 +480,15 @@ int gla_poll_error(uint32_t *code);
 struct LatentShape {
   uint32_t heads, dim, rot_dim, value_dim, kv_rank, window, rope_dims, block_size, row_stride;
   float scale, eps;
+  bool gated = true;  // the output has a gate per value
+  uint32_t ld = 0;    // row stride of the joint projection (0: its columns)
   __host__ __device__ uint32_t q_dim() const { return dim + rot_dim; }
   // Columns of the joint projection: queries, latent + shared key part, output gate.
   __host__ __device__ uint32_t q_cols() const { return heads * (dim + rot_dim); }
   __host__ __device__ uint32_t kv_cols() const { return kv_rank + rot_dim; }
   __host__ __device__ uint32_t out_cols() const { return heads * value_dim; }
-  __host__ __device__ uint32_t cols() const { return q_cols() + kv_cols() + out_cols(); }
+  __host__ __device__ uint32_t cols() const { return q_cols() + kv_cols() + (gated ? out_cols() : 0); }
+  __host__ __device__ uint32_t row_ld() const { return ld ? ld : cols(); }
   // First position that a query at `pos` sees.
   __host__ __device__ uint32_t first_key(uint32_t pos) const { return KeyRange{window, 0}.first(pos); }
 };
@@ -499,13 +552,22 @@ int latent_prefill_poll_error(uint32_t *code);
 // [experts][hidden][ffn]; the shared expert's the same with one expert.
 // Variants: softmax of the logits for the sigmoid; a correction per output of the router that takes part in the choice only;
 // `identity` further outputs of the router whose experts return their input (they take no part in the products); scores that
-// multiply the experts' outputs (where they are summed: SublayerOutput::weight); other gated activations.
+// multiply the experts' outputs (where they are summed: SublayerOutput::weight); other gated activations. groups: the outputs form
+// that many groups of neighbours, and only those of the `keep` groups with the largest scores in them can be chosen (scores are not
+// negative). renorm: the chosen scores are divided by their sum (+ 1e-20). Experts without a gate (GatedAct::plain) have `up`
+// [experts][ffn][hidden].
 struct MoeShape {
   uint32_t hidden, experts, top, ffn, shared_ffn;
   uint32_t identity = 0;
   bool softmax = false, weigh_output = false;
   GatedAct act{}, shared_act{};
+  uint32_t groups = 0, keep = 0;
+  bool renorm = false;
+  uint32_t logits_ld = 0;  // row stride of the router's partial sums (0: its outputs)
   __host__ __device__ uint32_t outputs() const { return experts + identity; }
+  __host__ __device__ uint32_t row_ld() const { return logits_ld ? logits_ld : outputs(); }
+  __host__ __device__ uint32_t up_cols() const { return act.plain() ? ffn : 2 * ffn; }
+  __host__ __device__ uint32_t shared_up_cols() const { return shared_act.plain() ? shared_ffn : 2 * shared_ffn; }
 };
 struct MoeTile {
   uint32_t expert, row, count;  // sorted rows [row, row + count) go through `expert`; count 0: nothing to do
@@ -544,8 +606,8 @@ template <typename T>
 int launch_moe_experts(const T *x, const T *w_up, const T *w_down, const T *shared_up, const T *shared_down, MoeShape s, MoePlan plan,
                        MoeBuffers<T> b, float *shared_out, uint32_t rows, cudaStream_t stream);
 // One product of the grouped kind on tcgen05: rows of `x` by tile through rows [expert * n, (expert + 1) * n) of `w`, and rows of
-// `shared_x` through `shared_w` (shared_n = 0: none). swiglu: activations to act / shared_act (row stride n / 2, shared_n / 2),
-// the products multiplied by row_score (null = 1); else f32 to out / shared_out, [splits][rows][n].
+// `shared_x` through `shared_w` (shared_n = 0: none). swiglu: activations to act / shared_act (row stride n / 2, shared_n / 2; n, shared_n
+// for experts without a gate), the products multiplied by row_score (null = 1); else f32 to out / shared_out, [splits][rows][n].
 struct MoeProduct {
   const bf16 *x, *w, *shared_x, *shared_w;
   uint32_t n, k, shared_n, shared_k;

@@ -7,7 +7,7 @@
 //   latent_absorb_kernel             rows that decode: their queries taken into the latent space, per head
 //                                    (W_uk^T q on mma.sync)
 //   latent_decode_kernel             rows that decode: scores and weighted latents over the window's cache rows
-//   latent_value_kernel              rows that decode: merges the context splits, W_uv per head, output gate
+//   latent_value_kernel              rows that decode: merges the context splits, W_uv per head, output gate (if the design has one)
 #include "kernels.h"
 #include "mma.cuh"
 
@@ -37,7 +37,7 @@ latent_prepare_kernel(const float *__restrict__ partial, uint32_t splits, size_t
   const uint32_t half = ls.rope_dims / 2;
   const float *cs = rope_cos + (size_t)positions[row] * half, *sn = rope_sin + (size_t)positions[row] * half;
   pdl_wait();
-  const float *p = partial + (size_t)row * ls.cols();
+  const float *p = partial + (size_t)row * ls.row_ld();
   // value `i` of a rotated part whose first column is `at`
   auto rotated = [&](const float *at, uint32_t i) {
     const float v = fold(at + i, splits, split_stride);
@@ -97,7 +97,7 @@ latent_prepare_vec_kernel(const float *__restrict__ partial, uint32_t splits, si
   pdl_trigger();
   const uint32_t row = blockIdx.x, tid = threadIdx.x, half = ls.rope_dims / 2;
   const float *cs = rope_cos + (size_t)positions[row] * half, *sn = rope_sin + (size_t)positions[row] * half;
-  const float *p = partial + (size_t)row * ls.cols();
+  const float *p = partial + (size_t)row * ls.row_ld();
   if (blockIdx.y > 0) {
     const uint32_t i = ((blockIdx.y - 1) * kPrepThreads + tid) * 4, d = i % ls.q_dim();
     const bool live = i < ls.q_cols(), rot = live && d >= ls.dim && d - ls.dim < ls.rope_dims;
@@ -203,14 +203,14 @@ latent_attention_generic_kernel(const T *__restrict__ q, const T *__restrict__ c
     __syncthreads();
   }
   const float inv = 1.0f / l;
-  const float *g = gate + (size_t)row * ls.cols() + ls.q_cols() + ls.kv_cols() + (size_t)head * ls.value_dim;
+  const float *g = gate + (size_t)row * ls.row_ld() + ls.q_cols() + ls.kv_cols() + (size_t)head * ls.value_dim;
   T *o = out + (size_t)row * ldo + (size_t)head * ls.value_dim;
   for (uint32_t v = warp; v < ls.value_dim; v += kGenThreads / 32) {
     const T *w = w_uv + ((size_t)head * ls.value_dim + v) * ls.kv_rank;
     float a = 0.f;
     for (uint32_t r = lane; r < ls.kv_rank; r += 32) a += to_f32<T>(w[r]) * acc[r];
     a = warp_sum(a);
-    if (lane == 0) o[v] = from_f32<T>(a * inv * sigmoid_f(fold(g + v, splits, split_stride)));
+    if (lane == 0) o[v] = from_f32<T>(ls.gated ? a * inv * sigmoid_f(fold(g + v, splits, split_stride)) : a * inv);
   }
 }
 
@@ -521,8 +521,8 @@ latent_value_kernel(const float *__restrict__ part_o, const float *__restrict__ 
 #pragma unroll
   for (uint32_t e = 0; e < 4; ++e) {
     const uint32_t r = rw + (lane & 3) * 2 + (e & 1), v = v0 + vw + (lane >> 2) + (e >> 1) * 8;
-    g[e] = r < n && v < ls.value_dim
-               ? fold(gate + (size_t)row_list[row0 + r] * ls.cols() + ls.q_cols() + ls.kv_cols() + head * ls.value_dim + v, splits, split_stride)
+    g[e] = ls.gated && r < n && v < ls.value_dim
+               ? fold(gate + (size_t)row_list[row0 + r] * ls.row_ld() + ls.q_cols() + ls.kv_cols() + head * ls.value_dim + v, splits, split_stride)
                : 0.f;
   }
   for (uint32_t r = warp; r < n; r += kValueThreads / 32) {  // one warp per row: lane s weighs split s, then all sum
@@ -577,7 +577,8 @@ latent_value_kernel(const float *__restrict__ part_o, const float *__restrict__ 
 #pragma unroll
   for (uint32_t e = 0; e < 4; ++e) {
     const uint32_t r = rw + (lane & 3) * 2 + (e & 1), v = v0 + vw + (lane >> 2) + (e >> 1) * 8;
-    if (r < n && v < ls.value_dim) out[(size_t)row_list[row0 + r] * ldo + head * ls.value_dim + v] = __float2bfloat16_rn(c[e] * sigmoid_f(g[e]));
+    if (r < n && v < ls.value_dim)
+      out[(size_t)row_list[row0 + r] * ldo + head * ls.value_dim + v] = __float2bfloat16_rn(ls.gated ? c[e] * sigmoid_f(g[e]) : c[e]);
   }
 }
 
@@ -594,7 +595,7 @@ int launch_latent_prepare(const float *partial, uint32_t splits, size_t split_st
                           const float *rope_sin, const uint32_t *positions, const uint32_t *slot_block, const uint32_t *slot_slot,
                           T *q, T *cache, LatentShape ls, uint32_t rows, cudaStream_t stream) {
   if (rows == 0) return ORION_OK;
-  if (ls.dim % 4 == 0 && ls.rot_dim % 4 == 0 && ls.rope_dims % 4 == 0 && ls.kv_rank % 4 == 0 && ls.out_cols() % 4 == 0 &&
+  if (ls.dim % 4 == 0 && ls.rot_dim % 4 == 0 && ls.rope_dims % 4 == 0 && ls.kv_rank % 4 == 0 && ls.row_ld() % 4 == 0 &&
       ls.kv_cols() <= 4 * kPrepThreads) {
     const dim3 grid(rows, 1 + (ls.q_cols() / 4 + kPrepThreads - 1) / kPrepThreads);
     ORION_CUDA_CHECK("latent_prepare", launch_pdl(latent_prepare_vec_kernel<T>, grid, dim3(kPrepThreads), 0, stream, partial, splits,

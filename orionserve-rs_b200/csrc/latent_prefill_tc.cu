@@ -253,7 +253,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
     tc_fence_after();
     const float inv = l > 0.f ? 1.0f / l : 0.f;
     bf16 *dst = out + (size_t)row * ldo + (size_t)head * ls.value_dim;
-    const float *g = gate + (size_t)row * ls.cols() + ls.q_cols() + ls.kv_cols() + (size_t)head * ls.value_dim;
+    const float *g = gate + (size_t)row * ls.row_ld() + ls.q_cols() + ls.kv_cols() + (size_t)head * ls.value_dim;
 #pragma unroll 1
     for (uint32_t c = 0; c < ls.value_dim; c += 16) {
       uint32_t o[16];
@@ -263,6 +263,11 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
         float r[16];
 #pragma unroll
         for (uint32_t i = 0; i < 16; i += 4) {
+          if (!ls.gated) {
+#pragma unroll
+            for (uint32_t k = 0; k < 4; ++k) r[i + k] = __uint_as_float(o[i + k]) * inv;
+            continue;
+          }
           const float4 gv = sum_slabs4(g + c + i, splits, split_stride);
           r[i] = __uint_as_float(o[i]) * inv * sigmoid_f(gv.x);
           r[i + 1] = __uint_as_float(o[i + 1]) * inv * sigmoid_f(gv.y);

@@ -28,27 +28,40 @@ int LayeredModel<T>::check_layer(uint32_t i) const {
   const uint32_t rotates = s.mixer == ORION_MIXER_ATTENTION ? s.dim : s.rot_dim;
   if ((s.mixer == ORION_MIXER_ATTENTION || s.mixer == ORION_MIXER_LATENT_ATTENTION) && (s.rope_dims % 2 != 0 || s.rope_dims > rotates))
     return set_error(ORION_ERR_MODEL, "config.json is malformed: layer %u rotates %u of %u dimensions", i, s.rope_dims, rotates);
+  if (s.keys_as_values && (s.mixer != ORION_MIXER_ATTENTION || s.qk_norm != ORION_QK_NORM_ALL_HEADS || s.rope_dims || s.head_gate || s.value_dim != s.dim))
+    return set_error(ORION_ERR_MODEL, "layer %u: keys as values come with norms over all heads, without rotation and gates, and values of the keys' size", i);
+  if ((s.distance_bias || s.q_temp_every != 0) && !s.keys_as_values)
+    return set_error(ORION_ERR_MODEL, "layer %u: distance terms and query factors come with keys as values", i);
+  if (s.sinks > ORION_SINK_ZERO || s.q_temp_every < 0) return set_error(ORION_ERR_MODEL, "config.json is malformed: layer %u has an unknown sink or query factor", i);
   const uint64_t outputs = (uint64_t)s.experts + s.router_identity;
+  if (s.router_groups && (s.router != ORION_ROUTER_SOFTMAX_RENORM || outputs % s.router_groups || s.router_keep == 0 || s.router_keep > s.router_groups ||
+                          s.experts_per_token > outputs / s.router_groups * s.router_keep))
+    return set_error(ORION_ERR_MODEL, "config.json is malformed: layer %u uses %u of %llu experts, of %u of %u groups", i, s.experts_per_token,
+                     (unsigned long long)outputs, s.router_keep, s.router_groups);
   if (s.experts > 0 && (s.ffn_dim == 0 || s.experts_per_token == 0 || s.experts_per_token > outputs || outputs > kMoeMaxExperts))
     return set_error(ORION_ERR_MODEL, "config.json is malformed: layer %u uses %u of %llu experts of width %u (at most %u experts)", i,
                      s.experts_per_token, (unsigned long long)outputs, s.ffn_dim, kMoeMaxExperts);
-  if (s.activation > ORION_ACT_GEGLU_TANH || s.router > ORION_ROUTER_SOFTMAX || s.expert_form > ORION_EXPERT_CLAMPED || s.qk_norm > ORION_QK_NORM_PER_HEAD)
+  if (s.activation > ORION_ACT_GEGLU_TANH || s.router > ORION_ROUTER_SOFTMAX_RENORM || s.expert_form > ORION_EXPERT_GELU || s.qk_norm > ORION_QK_NORM_PER_HEAD)
     return set_error(ORION_ERR_MODEL, "config.json is malformed: layer %u has an unknown activation, router or norm", i);
-  if (s.mixer == ORION_MIXER_ATTENTION && s.qk_norm != ORION_QK_NORM_PER_HEAD && (s.rope_halves || s.qkv_bias || s.value_gate))
+  if (s.mixer == ORION_MIXER_ATTENTION && s.qk_norm != ORION_QK_NORM_PER_HEAD && (s.rope_halves || (s.qkv_bias && !s.keys_as_values) || s.value_gate))
     return set_error(ORION_ERR_MODEL, "layer %u: rotated halves, biases and gates per value come with norms per head", i);
   if (s.mixer == ORION_MIXER_ATTENTION && s.qk_norm == ORION_QK_NORM_PER_HEAD && s.head_gate)
     return set_error(ORION_ERR_MODEL, "layer %u: a gate per head comes with norms over all heads", i);
   if (d_.block == ORION_BLOCK_PARALLEL && (s.experts > 0 || s.ffn_bias))
     return set_error(ORION_ERR_MODEL, "layer %u: a parallel block has a dense feed-forward without biases", i);
-  if (d_.block != ORION_BLOCK_PRENORM && (s.activation == ORION_ACT_GEGLU_TANH || s.router != ORION_ROUTER_SIGMOID_INPUT || s.router_identity))
-    return set_error(ORION_ERR_MODEL, "layer %u: gated dense feed-forwards and softmax routers come with prenorm blocks", i);
+  if (d_.block != ORION_BLOCK_PRENORM && (s.activation == ORION_ACT_GEGLU_TANH || s.router == ORION_ROUTER_SOFTMAX || s.router_identity))
+    return set_error(ORION_ERR_MODEL, "layer %u: gated dense feed-forwards, corrected routers and identity experts come with prenorm blocks", i);
+  if (d_.block == ORION_BLOCK_GATED_POSTNORM && s.mixer == ORION_MIXER_MIN_GRU)
+    return set_error(ORION_ERR_MODEL, "layer %u: a gated post-norm block has no min-GRU", i);
+  if (s.router == ORION_ROUTER_SOFTMAX_RENORM && d_.block != ORION_BLOCK_GATED_POSTNORM && d_.block != ORION_BLOCK_PRENORM)
+    return set_error(ORION_ERR_MODEL, "layer %u: softmax routers come with prenorm and gated post-norm blocks", i);
   return ORION_OK;
 }
 
 template <typename T>
 int LayeredModel<T>::init() {
   const OrionLayeredDesc &d = d_;
-  if (d.hidden_size == 0 || d.vocab_size == 0 || d.num_layers == 0 || d.block > ORION_BLOCK_PRENORM || (parallel() && d.conv_taps == 0))
+  if (d.hidden_size == 0 || d.vocab_size == 0 || d.num_layers == 0 || d.block > ORION_BLOCK_GATED_POSTNORM || (parallel() && d.conv_taps == 0))
     return set_error(ORION_ERR_MODEL, "config.json is malformed: a model dimension is zero");
   if (d.block_size == 0 || d.max_batch_tokens == 0 || d.max_batch_sequences == 0 || d.num_state_slots == 0)
     return set_error(ORION_ERR_INVALID_REQUEST,
@@ -57,6 +70,10 @@ int LayeredModel<T>::init() {
   ORION_TRY(Base::init_step({d.hidden_size, d.vocab_size, d.max_position_embeddings, d.num_blocks, d.block_size, d.max_batch_tokens,
                              d.max_batch_sequences}));
   const size_t H = d.hidden_size;
+  if (!gated_postnorm() && (d.learned_positions || d.bigram_buckets))
+    return set_error(ORION_ERR_MODEL, "learned positions and pairs of tokens come with gated post-norm blocks");
+  if (d.learned_positions && d.max_position_embeddings > d.learned_positions)
+    return set_error(ORION_ERR_MODEL, "%u positions asked for, the model has %u", d.max_position_embeddings, d.learned_positions);
   const bool loop = d.loop_times > 0;
   if (loop && (d.block != ORION_BLOCK_PRENORM || d.loop_start >= d.loop_stop || d.loop_stop > d.num_layers))
     return set_error(ORION_ERR_MODEL, "config.json is malformed: layers %u to %u of %u cannot be looped", d.loop_start, d.loop_stop, d.num_layers);
@@ -87,6 +104,11 @@ int LayeredModel<T>::init() {
   }
   ORION_TRY(alloc(&embed_, (size_t)d.vocab_size * H));
   if (d.untied_lm_head) ORION_TRY(alloc(&head_, (size_t)d.vocab_size * H));
+  if (d.learned_positions) ORION_TRY(alloc(&places_, d.learned_positions * H));
+  if (d.bigram_buckets) {
+    ORION_TRY(alloc(&pairs_, (d.bigram_buckets + 1) * H));
+    ORION_TRY(zeroed(&history_, (size_t)d.num_blocks * d.block_size));
+  }
   ORION_TRY(alloc(&final_norm_, H));
   ORION_TRY(init_buffers());
   slots_.resize(num_state_slots());
@@ -139,6 +161,27 @@ int LayeredModel<T>::init_rope(Layer &L) {
   return ORION_OK;
 }
 
+// Factors of the queries by position, shared by the layers of equal constants.
+template <typename T>
+int LayeredModel<T>::init_query_factors(Layer &L) {
+  const double coef = L.d.q_temp_coef, every = L.d.q_temp_every;
+  if (every == 0) return ORION_OK;
+  const QueryFactors *known = nullptr;
+  for (const QueryFactors &q : query_factors_)
+    if (q.coef == coef && q.every == every) known = &q;
+  if (!known) {
+    std::vector<float> f(d_.max_position_embeddings);
+    for (size_t p = 0; p < f.size(); ++p) f[p] = (float)(1.0 + coef * std::log(std::floor(((double)p + 1.0) / every) + 1.0));
+    QueryFactors fresh{coef, every, nullptr};
+    ORION_TRY(alloc(&fresh.table, f.size()));
+    ORION_CUDA_CHECK("upload query factors", cudaMemcpy(fresh.table, f.data(), f.size() * sizeof(float), cudaMemcpyHostToDevice));
+    query_factors_.push_back(fresh);
+    known = &query_factors_.back();
+  }
+  L.in.q_factor = known->table;
+  return ORION_OK;
+}
+
 template <typename T>
 int LayeredModel<T>::init_layer(Layer &L) {
   const OrionLayeredDesc &d = d_;
@@ -149,7 +192,7 @@ int LayeredModel<T>::init_layer(Layer &L) {
   if (parallel()) ORION_TRY(alloc(&L.conv1, H * d.conv_taps));
   if (L.latent()) {
     L.ls = LatentShape{s.heads, s.dim, s.rot_dim, s.value_dim, s.kv_rank, s.window, s.rope_dims, d.block_size,
-                       odd_groups(s.kv_rank + s.rot_dim), (float)s.scale, (float)d.norm_eps};
+                       odd_groups(s.kv_rank + s.rot_dim), (float)s.scale, (float)d.norm_eps, !s.ungated};
     L.mix_in = L.ls.cols(), L.mix_out = L.ls.out_cols();
     ORION_TRY(alloc(&L.latent_norm, s.kv_rank));
     ORION_TRY(alloc(&L.w_uk, (size_t)s.heads * (s.dim + s.value_dim) * s.kv_rank));  // one matrix for the expansion of prompts
@@ -157,7 +200,7 @@ int LayeredModel<T>::init_layer(Layer &L) {
     ORION_TRY(init_rope(L));
   } else if (L.attention()) {
     // [q | k | v | gate], the rows of the matrix padded so that the partial sums of a row start on 32 bytes
-    const uint32_t qkv = s.heads * s.dim + s.kv_heads * (s.dim + s.value_dim);
+    const uint32_t qkv = s.heads * s.dim + s.kv_heads * (s.dim + (s.keys_as_values ? 0 : s.value_dim));
     L.mix_in = pad8(qkv + (s.head_gate ? s.heads : 0) + (s.value_gate ? s.heads * s.value_dim : 0));
     L.mix_out = s.heads * s.value_dim;
     ORION_TRY(init_rope(L));
@@ -167,18 +210,26 @@ int LayeredModel<T>::init_layer(Layer &L) {
       ORION_TRY(alloc(&L.k_norm, (size_t)(own ? 1 : s.kv_heads) * s.dim));
     }
     if (s.qkv_bias) ORION_TRY(alloc(&L.mix_bias, qkv));
-    if (s.sinks) ORION_TRY(alloc(&L.sinks, s.heads));
+    if (s.sinks) ORION_TRY(zeroed(&L.sinks, s.heads));
+    if (s.keys_as_values) ORION_TRY(alloc(&L.q_gain, (size_t)s.heads * s.dim));
+    if (s.distance_bias) {
+      ORION_TRY(alloc(&L.dist_mult, s.heads));
+      ORION_TRY(alloc(&L.dist_rate, s.heads));
+    }
     // 16-bit caches pad the heads to sizes of the tensor-core kernels where those cover them
     const uint32_t dk = DTypeOf<T>::is_bf16 ? attention_padded_dim(s.dim, s.value_dim) : 0;
     const uint32_t dv = DTypeOf<T>::is_bf16 ? attention_padded_dim(s.value_dim, s.dim) : 0;
-    L.kv = KvLayout{1, d.num_blocks, s.kv_heads, d.block_size, dk ? dk : s.dim, dk ? 1u : 0u, dk ? dv : s.value_dim};
+    L.kv = KvLayout{1, d.num_blocks, s.kv_heads, d.block_size, dk ? dk : s.dim, dk ? 1u : 0u, dk ? dv : s.value_dim,
+                    s.keys_as_values ? (uint32_t)(sizeof(float) / sizeof(T)) : 0};
     L.tuned = DTypeOf<T>::is_bf16 && attention_form_supported(L.kv, s.heads);
-    L.in = AttnInputs{s.heads, s.kv_heads, s.dim, s.value_dim, s.rope_dims, L.mix_in, (float)d.norm_eps, L.q_norm, L.k_norm, L.rope_cos, L.rope_sin,
-                      s.qk_norm == ORION_QK_NORM_PER_HEAD, s.rope_halves != 0, L.mix_bias};
+    L.in = AttnInputs{s.heads, s.kv_heads, s.dim, s.value_dim, s.rope_dims, L.mix_in, (float)d.norm_eps, s.keys_as_values ? L.q_gain : L.q_norm, L.k_norm, L.rope_cos, L.rope_sin,
+                      s.qk_norm == ORION_QK_NORM_PER_HEAD, s.rope_halves != 0, L.mix_bias, s.keys_as_values != 0};
+    ORION_TRY(init_query_factors(L));
     L.form.scale = (float)s.scale;
     L.form.softcap = (float)s.softcap;
     L.form.range = KeyRange{s.window, s.chunk, s.keep_first};
     L.form.sinks = L.sinks;
+    L.form.dist_mult = L.dist_mult, L.form.dist_rate = L.dist_rate;
     L.form.out_dim = s.value_dim;
     if (L.tuned) {
       const uint32_t positions = 128 / (s.heads / s.kv_heads);
@@ -197,6 +248,12 @@ int LayeredModel<T>::init_layer(Layer &L) {
     L.mix_in = 3 * s.width, L.mix_out = s.width;
     ORION_TRY(alloc(&L.mix_bias, 2 * (size_t)s.width));
   }
+  if (gated_postnorm()) {
+    L.gate_at = pad8(L.mix_in);
+    L.mix_in = pad8(L.gate_at + d.hidden_size);
+    L.ls.ld = L.in.ld = L.gla.ld = L.mix_in;
+    ORION_TRY(alloc(&L.gate_bias, H));
+  }
   ORION_TRY(zeroed(&L.w_mix, (size_t)L.mix_in * H));
   // Activations start at multiples of 8 columns; the weights of the columns between them are zero.
   L.ff_at = parallel() ? pad8(L.mix_out) : 0;
@@ -208,21 +265,29 @@ int LayeredModel<T>::init_layer(Layer &L) {
   if (parallel()) ORION_TRY(alloc(&L.conv2, H * d.conv_taps));
   else ORION_TRY(alloc(&L.norm2, H));
   if (sandwich()) ORION_TRY(alloc(&L.norm2_post, H));
+  if (gated_postnorm()) ORION_TRY(alloc(&L.ff_gate_bias, H));
   if (s.experts > 0) {
     L.moe = MoeShape{d.hidden_size, s.experts, s.experts_per_token, s.ffn_dim, s.shared_dim, s.router_identity};
-    L.moe.softmax = L.moe.weigh_output = s.router == ORION_ROUTER_SOFTMAX;
-    const GatedKind kind = s.expert_form == ORION_EXPERT_CLAMPED ? kGatedClamped : kGatedSilu;
+    L.moe.softmax = L.moe.weigh_output = s.router != ORION_ROUTER_SIGMOID_INPUT;
+    L.moe.renorm = s.router == ORION_ROUTER_SOFTMAX_RENORM;
+    L.moe.groups = s.router_groups, L.moe.keep = s.router_keep;
+    const GatedKind kind = s.expert_form == ORION_EXPERT_CLAMPED ? kGatedClamped : (s.expert_form == ORION_EXPERT_GELU ? kPlainGelu : kGatedSilu);
     L.moe.act = GatedAct{kind, (float)s.expert_limit}, L.moe.shared_act = GatedAct{kind, (float)s.shared_limit};
-    ORION_TRY(alloc(&L.w_router, (size_t)L.moe.outputs() * H));
-    if (L.moe.softmax) ORION_TRY(alloc(&L.correction, L.moe.outputs()));
-    ORION_TRY(alloc(&L.e_up, (size_t)s.experts * 2 * s.ffn_dim * H));
+    if (gated_postnorm()) {
+      L.ff_gate_at = pad8(L.moe.outputs());
+      L.moe.logits_ld = pad8(L.ff_gate_at + d.hidden_size);
+    }
+    ORION_TRY(zeroed(&L.w_router, (size_t)L.moe.row_ld() * H));
+    if (s.router == ORION_ROUTER_SOFTMAX) ORION_TRY(alloc(&L.correction, L.moe.outputs()));
+    ORION_TRY(alloc(&L.e_up, (size_t)s.experts * L.moe.up_cols() * H));
     ORION_TRY(alloc(&L.e_down, (size_t)s.experts * H * s.ffn_dim));
     if (s.shared_dim) {
-      ORION_TRY(alloc(&L.s_up, (size_t)2 * s.shared_dim * H));
+      ORION_TRY(alloc(&L.s_up, (size_t)L.moe.shared_up_cols() * H));
       ORION_TRY(alloc(&L.s_down, H * s.shared_dim));
     }
     return ORION_OK;
   }
+  if (gated_postnorm()) ORION_TRY(alloc(&L.w_ff_gate, H * H));
   ORION_TRY(alloc(&L.w_up, (size_t)(L.gated_ffn() ? 2 : 1) * s.ffn_dim * H));
   if (!parallel()) ORION_TRY(zeroed(&L.w_down, H * L.ff_ld));
   if (s.ffn_bias) {
@@ -256,7 +321,8 @@ int LayeredModel<T>::init_buffers() {
     const OrionLayerDesc &s = L.d;
     grow(cat, L.cat);
     const std::pair<uint32_t, uint32_t> products[] = {
-        {L.mix_in, (uint32_t)H}, {(uint32_t)H, L.cat}, {s.experts ? L.moe.outputs() : (L.gated_ffn() ? 2 : 1) * s.ffn_dim, (uint32_t)H}, {L.w_down ? (uint32_t)H : 0, L.ff_ld}};
+        {L.mix_in, (uint32_t)H}, {(uint32_t)H, L.cat}, {s.experts ? L.moe.row_ld() : (L.gated_ffn() ? 2 : 1) * s.ffn_dim, (uint32_t)H}, {L.w_down ? (uint32_t)H : 0, L.ff_ld},
+        {L.w_ff_gate ? (uint32_t)H : 0, (uint32_t)H}};
     for (const auto &[n, k] : products)
       if (n) grow(partial_floats_, gemm_partial_floats(kBf16, (uint32_t)rows, n, k));
     if (L.w_down) grow(cat, L.ff_ld);
@@ -286,6 +352,7 @@ int LayeredModel<T>::init_buffers() {
     }
   }
   ORION_TRY(alloc(&partial_, partial_floats_));
+  if (gated_postnorm()) ORION_TRY(alloc(&out_partial_, partial_floats_));
   if (parallel()) {
     ORION_TRY(alloc(&conv_m_, rows * H));
     ORION_TRY(alloc(&conv_f_, rows * H));
@@ -331,25 +398,39 @@ bool LayeredModel<T>::place(const std::string &name, Place *p) const {
     p->rows = d_.loop_times, p->matrix = true;
     return loop_step_ != nullptr;
   }
+  auto gain = [&](float *dst) {  // of a norm of the residual stream
+    if (!d_.scalar_norms) return vector(dst, H);
+    p->copies = H;
+    return vector(dst, 1);
+  };
   if (name == "embed") return matrix(embed_, d_.vocab_size, H);
+  if (name == "bigram") return matrix(pairs_, d_.bigram_buckets + 1, H);
+  if (name == "pos") return matrix(places_, d_.learned_positions, H);
   if (name == "head") return matrix(head_, d_.vocab_size, H);
-  if (name == "final.norm") return vector(final_norm_, H);
+  if (name == "final.norm") return gain(final_norm_);
   unsigned i = 0;
   int used = 0;
   if (sscanf(name.c_str(), "l%u.%n", &i, &used) != 1 || used == 0 || i >= first_run_.size()) return false;
   const std::string rest = name.substr((size_t)used);
   const Layer &L = layers_[first_run_[i]];
   const OrionLayerDesc &s = L.d;
-  if (rest == "norm1") return vector(L.norm, H);
-  if (rest == "norm1b") return vector(L.norm_post, H);
-  if (rest == "norm2") return vector(L.norm2, H);
-  if (rest == "norm2b") return vector(L.norm2_post, H);
+  if (rest == "norm1") return gain(L.norm);
+  if (rest == "norm1b") return gain(L.norm_post);
+  if (rest == "norm2") return gain(L.norm2);
+  if (rest == "norm2b") return gain(L.norm2_post);
+  if (rest == "rg1") return gated_postnorm() && matrix(L.w_mix + (uint64_t)L.gate_at * H, H, H);
+  if (rest == "rg2") return gated_postnorm() && matrix(L.w_router ? L.w_router + (uint64_t)L.ff_gate_at * H : L.w_ff_gate, H, H);
+  if (rest == "rg1.b") return vector(L.gate_bias, H, 0.0f);
+  if (rest == "rg2.b") return vector(L.ff_gate_bias, H, 0.0f);
   if (rest == "canon1") return L.conv1 && filters(L.conv1);
   if (rest == "canon2") return L.conv2 && filters(L.conv2);
   if (rest.compare(0, 4, "mlp.") == 0) {
     const std::string t = rest.substr(4);
     // an expert's gate and up rows alternate in one matrix
+    const bool plain = s.experts > 0 && L.moe.act.plain();
     auto expert = [&](const std::string &part, T *up, T *down, uint64_t ffn) {
+      if (plain && part == "gate") return false;
+      if (plain && part == "up") return matrix(up, ffn, H);
       if (part == "gate") return matrix(up, ffn, H, 2 * H);
       if (part == "up") return matrix(up ? up + H : nullptr, ffn, H, 2 * H);
       if (part == "down") return matrix(down, H, ffn);
@@ -362,7 +443,7 @@ bool LayeredModel<T>::place(const std::string &name, Place *p) const {
     int at = 0;
     if (sscanf(t.c_str(), "e%u.%n", &e, &at) == 1 && at > 0) {
       if (e >= s.experts) return false;
-      return expert(t.substr((size_t)at), L.e_up + e * 2 * s.ffn_dim * H, L.e_down + e * H * s.ffn_dim, s.ffn_dim);
+      return expert(t.substr((size_t)at), L.e_up + (uint64_t)e * L.moe.up_cols() * H, L.e_down + e * H * s.ffn_dim, s.ffn_dim);
     }
     if (s.experts > 0 || !L.has_ffn()) return false;
     if (L.gated_ffn() && t != "down") return expert(t, L.w_up, nullptr, s.ffn_dim);
@@ -379,22 +460,24 @@ bool LayeredModel<T>::place(const std::string &name, Place *p) const {
     const uint64_t nq = (uint64_t)s.heads * s.dim, nk = (uint64_t)s.kv_heads * s.dim, nv = (uint64_t)s.kv_heads * s.value_dim;
     if (t == "q") return matrix(L.w_mix, nq, H);
     if (t == "k") return matrix(L.w_mix + nq * H, nk, H);
-    if (t == "v") return matrix(L.w_mix + (nq + nk) * H, nv, H);
+    if (t == "v") return !s.keys_as_values && matrix(L.w_mix + (nq + nk) * H, nv, H);
+    if (t == "r1") return vector(L.dist_mult, s.heads, 0.5f);
+    if (t == "r2") return vector(L.dist_rate, s.heads, 0.1f);
     if (t == "g") return (s.head_gate || s.value_gate) && matrix(L.w_mix + (nq + nk + nv) * H, s.value_gate ? s.heads * s.value_dim : s.heads, H);
     const bool own = s.qk_norm == ORION_QK_NORM_PER_HEAD;
     if (t == "q.norm") return vector(L.q_norm, own ? s.dim : nq);
     if (t == "k.norm") return vector(L.k_norm, own ? s.dim : nk);
     if (t == "q.b") return vector(L.mix_bias, nq, 0.0f);
     if (t == "k.b") return vector(L.mix_bias ? L.mix_bias + nq : nullptr, nk, 0.0f);
-    if (t == "v.b") return vector(L.mix_bias ? L.mix_bias + nq + nk : nullptr, nv, 0.0f);
-    if (t == "sink") return vector(L.sinks, s.heads, 0.0f);
+    if (t == "v.b") return !s.keys_as_values && vector(L.mix_bias ? L.mix_bias + nq + nk : nullptr, nv, 0.0f);
+    if (t == "sink") return s.sinks == ORION_SINK_LEARNED && vector(L.sinks, s.heads, 0.0f);
     return false;
   }
   if (L.latent()) {
     const LatentShape &a = L.ls;
     if (t == "q") return matrix(L.w_mix, a.q_cols(), H);
     if (t == "dkv") return matrix(L.w_mix + a.q_cols() * H, a.kv_cols(), H);
-    if (t == "g") return matrix(L.w_mix + (a.q_cols() + a.kv_cols()) * H, a.out_cols(), H);
+    if (t == "g") return a.gated && matrix(L.w_mix + (a.q_cols() + a.kv_cols()) * H, a.out_cols(), H);
     if (t == "dkv.norm") return vector(L.latent_norm, s.kv_rank);
     if (t == "uk") return matrix(L.w_uk, (uint64_t)s.heads * s.dim, s.kv_rank);
     if (t == "uv") return matrix(L.w_uv, (uint64_t)s.heads * s.value_dim, s.kv_rank);
@@ -426,13 +509,13 @@ std::vector<std::string> LayeredModel<T>::tensor_names() const {
   auto add = [&](const std::string &name) {
     if (uses_tensor(name.c_str())) names.push_back(name);
   };
-  for (const char *n : {"embed", "head", "final.norm", "loop.step"}) add(n);
+  for (const char *n : {"embed", "head", "final.norm", "loop.step", "bigram", "pos"}) add(n);
   for (uint32_t i = 0; i < d_.num_layers; ++i) {
     const std::string l = "l" + std::to_string(i) + ".";
     for (const char *rest : {"norm1", "norm1b", "norm2", "norm2b", "canon1", "canon2", "mlp.up", "mlp.up.b", "mlp.down", "mlp.down.b", "mlp.router",
                              "mlp.shared.gate", "mlp.shared.up", "mlp.shared.down", "mix.o", "mix.q", "mix.k", "mix.v", "mix.q.norm", "mix.k.norm",
                              "mix.sink", "mix.dkv", "mix.dkv.norm", "mix.uk", "mix.uv", "mix.g", "mix.z", "mix.x", "mix.z.b", "mix.x.b", "mlp.gate", "mlp.correction", "mix.q.b", "mix.k.b", "mix.v.b", "mix.norm", "mix.a1",
-                             "mix.a2", "mix.a2.b"})
+                             "mix.a2", "mix.a2.b", "rg1", "rg1.b", "rg2", "rg2.b", "mix.r1", "mix.r2"})
       add(l + rest);
     for (uint32_t e = 0; e < specs_[i].experts; ++e)
       for (const char *part : {".gate", ".up", ".down"}) add(l + "mlp.e" + std::to_string(e) + part);
@@ -444,16 +527,21 @@ template <typename T>
 int LayeredModel<T>::load_tensor(const char *name, int dtype, const uint64_t *shape, int ndim, const void *data) {
   ORION_CUDA_CHECK("set device", cudaSetDevice(ordinal_));
   if (dtype_size(dtype) == 0) return set_error(ORION_ERR_MODEL, "unsupported dtype %d (tensor `%s`)", dtype, name);
-  if (!data || ndim < 1 || ndim > 2) return set_error(ORION_ERR_MODEL, "tensor `%s` has rank %d", name, ndim);
+  if (!data || ndim < 0 || ndim > 2) return set_error(ORION_ERR_MODEL, "tensor `%s` has rank %d", name, ndim);
   Place p;
   if (!place(name, &p)) return set_error(ORION_ERR_MODEL, "tensor `%s` is not part of the model", name);
-  const uint64_t R = ndim == 2 ? shape[0] : 1, C = ndim == 2 ? shape[1] : shape[0];
+  const uint64_t R = ndim == 2 ? shape[0] : 1, C = ndim == 0 ? 1 : shape[ndim - 1];
   if (R != p.rows || C != p.cols || (ndim == 2) != p.matrix)
     return set_error(ORION_ERR_MODEL, "tensor `%s` has shape [%llu, %llu], expected [%llu, %llu]", name, (unsigned long long)R,
                      (unsigned long long)C, (unsigned long long)p.rows, (unsigned long long)p.cols);
   finalized_ = false;
   if (p.vec) {
     ORION_TRY(upload_slice(nullptr, p.vec, data, dtype, C, 0, R, 0, C));
+    if (p.copies) {
+      float value = 0.f;
+      ORION_CUDA_CHECK("upload tensor", cudaMemcpy(&value, p.vec, sizeof(float), cudaMemcpyDeviceToHost));
+      ORION_TRY(set_constant(p.vec, p.copies, value));
+    }
   } else if (p.ld == C && !p.transposed) {
     ORION_TRY(upload_slice(p.dst, nullptr, data, dtype, C, 0, R, 0, C));
   } else {  // a column block of a wider matrix, or filters
@@ -478,6 +566,15 @@ int LayeredModel<T>::finalize() {
   std::sort(got.begin(), got.end());
   for (const std::string &n : tensor_names())
     if (!std::binary_search(got.begin(), got.end(), n)) return set_error(ORION_ERR_MODEL, "missing tensor `%s`", n.c_str());
+  for (Layer &L : layers_) {
+    if (!L.q_gain) continue;
+    const size_t nq = (size_t)L.d.heads * L.d.dim, nk = (size_t)L.d.kv_heads * L.d.dim, group = L.d.heads / L.d.kv_heads;
+    std::vector<float> q(nq), k(nk);
+    ORION_CUDA_CHECK("gains", cudaMemcpy(q.data(), L.q_norm, nq * sizeof(float), cudaMemcpyDeviceToHost));
+    ORION_CUDA_CHECK("gains", cudaMemcpy(k.data(), L.k_norm, nk * sizeof(float), cudaMemcpyDeviceToHost));
+    for (size_t i = 0; i < nq; ++i) q[i] *= k[i / L.d.dim / group * L.d.dim + i % L.d.dim];
+    ORION_CUDA_CHECK("gains", cudaMemcpy(L.q_gain, q.data(), nq * sizeof(float), cudaMemcpyHostToDevice));
+  }
   lm_head_ = head_ ? head_ : embed_;
   finalized_ = true;
   return ORION_OK;
@@ -492,7 +589,7 @@ int LayeredModel<T>::init_random(uint64_t seed, float std) {
     Place p;
     place(n, &p);
     if (p.vec) {
-      ORION_TRY(set_constant(p.vec, p.rows * p.cols, p.fill));
+      ORION_TRY(set_constant(p.vec, p.copies ? p.copies : p.rows * p.cols, p.fill));
     } else if (p.ld == p.cols) {
       ORION_TRY(fill_random(p.dst, p.rows * p.cols, seed, n.find(".canon") != std::string::npos ? 0.1f : std));
     } else {
@@ -703,20 +800,23 @@ template <typename T>
 int LayeredModel<T>::fill_kv_random(uint64_t seed, float std) {
   ORION_CUDA_CHECK("set device", cudaSetDevice(ordinal_));
   for (const Layer &L : layers_)
-    if (L.cache) ORION_TRY(fill_random(L.cache, d_.num_blocks * L.cache_elems(), seed, std));
+    if (L.cache) {
+      ORION_TRY(fill_random(L.cache, d_.num_blocks * L.cache_elems(), seed, std));
+      if (L.attention() && L.kv.factor_elems) ORION_TRY(launch_fill_factors<T>(L.cache, L.kv, 1.f, stream_));
+    }
   ORION_CUDA_CHECK("fill_kv_random", cudaStreamSynchronize(stream_));
   return ORION_OK;
 }
 
 // The caches of the attention layers, one after the other: latents as [block][slot][kv_rank + rot_dim], keys and then values as
-// [block][kv head][slot][dim].
+// [block][kv head][slot][dim], where the values are the keys one set of rows and then the factors of the keys.
 template <typename T>
 int LayeredModel<T>::read_kv(float *out, uint64_t capacity) {
   ORION_CUDA_CHECK("set device", cudaSetDevice(ordinal_));
   const size_t tokens = (size_t)d_.num_blocks * d_.block_size;
   for (const Layer &L : layers_) {
     if (!L.cache) continue;
-    const size_t cols = L.latent() ? L.ls.kv_cols() : L.d.kv_heads * (L.d.dim + L.d.value_dim);
+    const size_t cols = L.latent() ? L.ls.kv_cols() : L.d.kv_heads * (L.d.dim + (L.d.keys_as_values ? 1 : L.d.value_dim));
     const size_t stride = L.latent() ? L.ls.row_stride : cols, n = tokens * stride;
     if (capacity < tokens * cols) return set_error(ORION_ERR_INVALID_REQUEST, "KV read-back buffer is too small");
     ORION_TRY(ensure_stage(&stage_f32_, &stage_f32_cap_, n * sizeof(float)));

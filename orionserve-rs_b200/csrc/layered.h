@@ -1,15 +1,19 @@
 // Layer-list models: decoders whose layers are listed one by one, each with its own token mixer, feed-forward and sizes.
-// Three kinds of block:
+// Four kinds of block:
 //   parallel  h = norm(x); mixer and feed-forward each read h plus a short causal convolution of h; both results are added to
 //             x. They write their activations next to each other into one buffer and their output matrices are stored side by
 //             side along k, so the two sublayers end in a single projection whose accumulator adds them.
 //   sandwich  x += m * norm(mixer(norm(x))), then x += m * norm(feed-forward(norm(x))): one kernel folds a sublayer's output
 //             projection, normalises it, adds it and normalises the sum for the next sublayer.
 //   prenorm   x += m * mixer(norm(x)), then x += m * feed-forward(norm(x)).
+//   gated post-norm  x += m * norm(g * mixer(x)), then x += m * norm(g' * feed-forward(x)): the gates are projections of x, stored
+//             below the matrix that the sublayer applies to x first (the mixer's joint projection, the router), so they cost no
+//             launch of their own; the kernel that normalises and adds a sublayer's output reads them from that product.
 // A run of layers may be passed through several times (prenorm blocks): the passes share the weights, and each has caches and states
 // of its own, so a pass is simply a further layer of the sequence of layer runs that points to the same weights.
-// What a sequence carries from step to step is the paged cache of its attention layers (latents, or keys and values) and, in a
-// state slot, the recurrences' states and the convolutions' last inputs.
+// What a sequence carries from step to step is the paged cache of its attention layers (latents, or keys and values; where the
+// embedding looks at the previous token, also the tokens themselves) and, in a state slot, the recurrences' states and the
+// convolutions' last inputs.
 #pragma once
 
 #include <string>
@@ -55,6 +59,7 @@ class LayeredModel final : public StepModel<T> {
   int read_kv(float *out, uint64_t capacity) override;
   uint32_t num_state_slots() const override { return has_state() ? d_.num_state_slots : 0; }
   bool logical_positions() const override { return true; }
+  uint64_t sequence_limit() const override { return d_.learned_positions; }
   float logit_softcap() const override { return (float)d_.logit_softcap; }
   const OrionModelDesc &desc() const override { return desc_; }
 
@@ -73,8 +78,13 @@ class LayeredModel final : public StepModel<T> {
     MoeShape moe{};      // experts = 0: dense feed-forward or none
     // joint mixer projection's columns, mixer output, columns of the feed-forward's activations and of the output projection
     uint32_t mix_in = 0, mix_out = 0, ff_at = 0, cat = 0, ff_ld = 0;
+    // gated post-norm block: first column of a sublayer's gate in the mixer's joint projection, and in the router's
+    uint32_t gate_at = 0, ff_gate_at = 0;
     float *norm = nullptr, *mix_bias = nullptr, *latent_norm = nullptr;
     float *norm_post = nullptr, *norm2 = nullptr, *norm2_post = nullptr;  // sandwich block
+    float *gate_bias = nullptr, *ff_gate_bias = nullptr;                   // gated post-norm block
+    T *w_ff_gate = nullptr;                                                // its gate of a dense feed-forward
+    float *q_gain = nullptr, *dist_mult = nullptr, *dist_rate = nullptr;  // keys as values: gains of queries times those of keys
     float *q_norm = nullptr, *k_norm = nullptr, *sinks = nullptr, *up_bias = nullptr, *down_bias = nullptr;
     T *conv1 = nullptr, *conv2 = nullptr, *w_mix = nullptr, *w_up = nullptr, *w_out = nullptr, *w_down = nullptr, *w_uk = nullptr, *w_uv = nullptr;
     T *w_decay = nullptr;        // gla: [heads * dim][rank], its bias in mix_bias
@@ -98,6 +108,7 @@ class LayeredModel final : public StepModel<T> {
     uint64_t rows = 0, cols = 0, ld = 0;
     bool matrix = true, transposed = false;  // transposed: kept as [cols][rows]
     float fill = 1.0f;                       // a vector's value in a randomly initialised model
+    uint64_t copies = 0;                     // not 0: the tensor is one number, kept as a vector of this size
   };
   bool place(const std::string &name, Place *p) const;
   std::vector<std::string> tensor_names() const;
@@ -105,9 +116,11 @@ class LayeredModel final : public StepModel<T> {
   int init_layer(Layer &L);
   int init_memory(Layer &L);  // what a layer run keeps of its sequences
   int init_rope(Layer &L);
+  int init_query_factors(Layer &L);
   int init_buffers();
   bool sandwich() const { return d_.block == ORION_BLOCK_SANDWICH; }
   bool parallel() const { return d_.block == ORION_BLOCK_PARALLEL; }
+  bool gated_postnorm() const { return d_.block == ORION_BLOCK_GATED_POSTNORM; }
   bool has_state() const {
     if (parallel()) return true;
     for (const OrionLayerDesc &s : specs_)
@@ -125,6 +138,7 @@ class LayeredModel final : public StepModel<T> {
   int run_parallel_layers();
   int run_sandwich_layers();
   int run_prenorm_layers();
+  int run_gated_postnorm_layers();
   bool graph_eligible() const override {
     return g_step_graph && DTypeOf<T>::is_bf16 && meta_.decode && !meta_.zero_count && !prof_on_ && only_mask_ == 0 &&
            (!parallel() || residual_norm_conv_supported(d_.hidden_size, d_.conv_taps));
@@ -172,14 +186,18 @@ class LayeredModel final : public StepModel<T> {
     const uint32_t *m = d_meta_;
     return AttnBatch{m + meta_.positions, m + meta_.seq_of_row, m + meta_.tables, m + meta_.offsets, meta_.rows, meta_.max_position};
   }
-  // The token mixer of one layer: x -> the first mix_out columns of cat_.
-  int mixer(const Layer &L, const T *x);
+  // The token mixer of one layer: x -> the first mix_out columns of cat_. Names the gate of its output in *y (gated post-norm blocks).
+  int mixer(const Layer &L, const T *x, SublayerOutput *y = nullptr);
   int latent_attention(const Layer &L, const GemmPlan &p, size_t slab);
   int attention(const Layer &L, const GemmPlan &p, size_t slab);
   int linear_attention(const Layer &L, const GemmPlan &p, size_t slab);
   // The up half of a dense feed-forward, activated: x -> act (row stride ld).
   int dense_up(const Layer &L, const T *x, T *act, uint32_t ld);
   int mixture(const Layer &L, const T *x, SublayerOutput *y);
+  // y's gate: columns from `at` on of a product of `n` columns in partial_.
+  void set_gate(const GemmPlan &p, uint32_t n, uint32_t at, const float *bias, SublayerOutput *y) const {
+    y->gate = partial_ + at, y->gate_bias = bias, y->gate_splits = p.out_slabs, y->gate_ld = n, y->gate_stride = (size_t)meta_.rows * n;
+  }
 
   OrionLayeredDesc d_;
   std::vector<OrionLayerDesc> specs_;
@@ -187,11 +205,14 @@ class LayeredModel final : public StepModel<T> {
   std::vector<Layer> layers_;         // in the order in which they run
   std::vector<uint32_t> first_run_;   // of every layer of the list
   float *loop_step_ = nullptr;        // [passes][hidden]
+  T *pairs_ = nullptr, *places_ = nullptr;  // further tables of the embedding: [buckets + 1][hidden], [learned_positions][hidden]
+  uint32_t *history_ = nullptr;             // [blocks][block_size]: token of every cache slot
   std::vector<std::string> got_;
   float *final_norm_ = nullptr;
   T *head_ = nullptr;                        // an output matrix of its own
   T *conv_m_ = nullptr, *conv_f_ = nullptr;  // inputs of the mixer and the feed-forward
   T *cat_ = nullptr;                         // their activations, side by side (sandwich: one after the other)
+  float *out_partial_ = nullptr;             // gated post-norm block: products beside those in partial_, which hold the gate
   T *qbuf_ = nullptr;
   T *qa_ = nullptr;           // queries of decoding rows in the latent space
   float *gate_ = nullptr;     // factors of the heads' outputs
@@ -219,6 +240,11 @@ class LayeredModel final : public StepModel<T> {
     float *cos, *sin;
   };
   std::vector<Rope> ropes_;
+  struct QueryFactors {
+    double coef, every;
+    float *table;  // [positions]
+  };
+  std::vector<QueryFactors> query_factors_;
   // What each state slot holds: the number of tokens its state covers and which of its two copies is current.
   struct Slot {
     uint64_t tokens = 0;

@@ -4,11 +4,12 @@
 namespace orion {
 
 template <typename T>
-int LayeredModel<T>::mixer(const Layer &L, const T *x) {
+int LayeredModel<T>::mixer(const Layer &L, const T *x, SublayerOutput *y) {
   const uint32_t Tn = meta_.rows, H = d_.hidden_size;
   const GemmPlan p = plan_for(Tn, L.mix_in, H, H);
   const size_t slab = (size_t)Tn * L.mix_in;
   ORION_TRY(timed(kProfGemm, [&] { return launch_gemm<T>(x, H, L.w_mix, H, partial_, Tn, L.mix_in, H, p, stream_); }));
+  if (L.gate_at && y) set_gate(p, L.mix_in, L.gate_at, L.gate_bias, y);
   if (L.latent()) return latent_attention(L, p, slab);
   if (L.attention()) return attention(L, p, slab);
   if (L.linear()) return linear_attention(L, p, slab);
@@ -148,15 +149,17 @@ int LayeredModel<T>::dense_up(const Layer &L, const T *x, T *act, uint32_t ld) {
 // The rows of x through their experts and the shared one; y names the results.
 template <typename T>
 int LayeredModel<T>::mixture(const Layer &L, const T *x, SublayerOutput *y) {
-  const uint32_t Tn = meta_.rows, H = d_.hidden_size, E = L.moe.outputs();
+  const uint32_t Tn = meta_.rows, H = d_.hidden_size, E = L.moe.row_ld();
+  float *shared_out = out_partial_ ? out_partial_ : partial_;
   const GemmPlan rp = plan_for(Tn, E, H, H);
   const MoePlan plan = moe_plan(DTypeOf<T>::is_bf16, L.moe, Tn);
   ORION_TRY(timed(kProfGemm, [&] { return launch_gemm<T>(x, H, L.w_router, H, partial_, Tn, E, H, rp, stream_); }));
   ORION_TRY(timed(kProfElementwise, [&] { return launch_moe_route<T>(partial_, rp.out_slabs, (size_t)Tn * E, L.correction, x, L.moe, plan, moe_, Tn, stream_); }));
   ORION_TRY(timed(kProfGemm, [&] {
-    return launch_moe_experts<T>(x, L.e_up, L.e_down, L.s_up, L.s_down, L.moe, plan, moe_, partial_, Tn, stream_);
+    return launch_moe_experts<T>(x, L.e_up, L.e_down, L.s_up, L.s_down, L.moe, plan, moe_, shared_out, Tn, stream_);
   }));
-  if (L.moe.shared_ffn) y->partial = partial_, y->splits = plan.down_splits, y->split_stride = (size_t)Tn * H;
+  if (L.ff_gate_at) set_gate(rp, E, L.ff_gate_at, L.ff_gate_bias, y);
+  if (L.moe.shared_ffn) y->partial = shared_out, y->splits = plan.down_splits, y->split_stride = (size_t)Tn * H;
   y->rows = moe_.down, y->place = moe_.place, y->top = L.moe.top;
   y->rows_splits = plan.down_splits, y->rows_stride = (size_t)Tn * L.moe.top * H;
   if (L.moe.weigh_output) y->weight = moe_.score;
@@ -289,8 +292,58 @@ int LayeredModel<T>::run_prenorm_layers() {
 }
 
 template <typename T>
+int LayeredModel<T>::run_gated_postnorm_layers() {
+  const uint32_t Tn = meta_.rows, H = d_.hidden_size;
+  const uint32_t *m = d_meta_;
+  const float eps = (float)d_.norm_eps, mult = (float)d_.residual_mult;
+  ORION_TRY(timed(kProfElementwise, [&] {
+    const EmbedTables<T> e{embed_, pairs_, places_, d_.bigram_buckets, d_.bigram_mul_prev, d_.bigram_mul_cur, history_, d_.block_size, (float)d_.embed_scale};
+    const EmbedBatch b{m + meta_.tokens, m + meta_.positions, m + meta_.seq_of_row, m + meta_.slot_block, m + meta_.slot_slot, m + meta_.tables,
+                       m + meta_.offsets, Tn};
+    return launch_embed_tables<T>(e, b, hidden_, normed_, H, stream_);
+  }));
+  // Gates, normalises and adds a sublayer's output; what reads the sum next takes it as it is, at the end of the model normalised.
+  auto join = [&](const SublayerOutput &y, const float *post, bool end) -> int {
+    if (end && meta_.outs == 0) return ORION_OK;
+    return timed(kProfElementwise, [&] {
+      return end ? launch_gated_post_norm<T>(y, hidden_, post, mult, final_norm_, eps, tail_, m + meta_.last_rows, meta_.outs, H, stream_)
+                 : launch_gated_post_norm<T>(y, hidden_, post, mult, nullptr, eps, normed_, nullptr, Tn, H, stream_);
+    });
+  };
+  // partial_ holds the gate until the output has joined the stream
+  auto projected = [&](const T *x, const T *w, uint32_t k, const float *bias, SublayerOutput *y) -> int {
+    const GemmPlan p = plan_for(Tn, H, k, k);
+    y->partial = out_partial_, y->splits = p.out_slabs, y->split_stride = (size_t)Tn * H, y->bias = bias;
+    return timed(kProfGemm, [&] { return launch_gemm<T>(x, k, w, k, out_partial_, Tn, H, k, p, stream_); });
+  };
+  for (size_t l = 0; l < layers_.size(); ++l) {
+    const Layer &L = layers_[l];
+    const bool end = l + 1 == layers_.size();
+    SublayerOutput y;
+    ORION_TRY(mixer(L, normed_, &y));
+    ORION_TRY(projected(cat_, L.w_out, L.cat, nullptr, &y));
+    ORION_TRY(join(y, L.norm, end && !L.has_ffn()));
+    if (!L.has_ffn()) continue;
+    y = SublayerOutput{};
+    if (L.moe.experts) {
+      ORION_TRY(mixture(L, normed_, &y));
+    } else {
+      ORION_TRY(dense_up(L, normed_, cat_, L.ff_ld));
+      const GemmPlan p = plan_for(Tn, H, H, H);
+      ORION_TRY(timed(kProfGemm, [&] { return launch_gemm<T>(normed_, H, L.w_ff_gate, H, partial_, Tn, H, H, p, stream_); }));
+      set_gate(p, H, 0, L.ff_gate_bias, &y);
+      ORION_TRY(projected(cat_, L.w_down, L.ff_ld, L.down_bias, &y));
+    }
+    ORION_TRY(join(y, L.norm2, end));
+  }
+  return ORION_OK;
+}
+
+template <typename T>
 int LayeredModel<T>::run_step_body(bool want_argmax, int part) {
-  if (part != 2) ORION_TRY(parallel() ? run_parallel_layers() : (sandwich() ? run_sandwich_layers() : run_prenorm_layers()));
+  if (part != 2)
+    ORION_TRY(parallel() ? run_parallel_layers()
+                         : (sandwich() ? run_sandwich_layers() : (gated_postnorm() ? run_gated_postnorm_layers() : run_prenorm_layers())));
   if (part == 1 || meta_.outs == 0) return ORION_OK;
   return run_head(want_argmax);
 }

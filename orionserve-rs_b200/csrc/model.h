@@ -67,6 +67,8 @@ class ModelBase {
   // Whether an engine has to feed every token at its own place in the sequence, and a preempted sequence's generated tokens
   // again (the reference's engine does neither).
   virtual bool logical_positions() const { return false; }
+  // The most tokens a sequence may have, output included (0: the model itself sets no limit).
+  virtual uint64_t sequence_limit() const { return 0; }
   virtual int init_random(uint64_t seed, float std) = 0;
   virtual int finalize() = 0;
   virtual int forward(const BatchView &b, float *logits_out, uint64_t logits_capacity,

@@ -1,12 +1,12 @@
 // Mixture of experts: the choice of experts, the order of rows by expert, and the grouped products of the f32 build and of
 // sizes the tensor cores do not take (moe_gemm_tc.cu has the others).
 //   moe_choose_kernel  one warp per row: sigmoid or softmax scores of the router's logits, the `top` largest (the lower index of equal
-//                      ones), and a histogram per block of rows
+//                      ones; where experts form groups, among the best groups), and a histogram per block of rows
 //   moe_place_kernel   one warp per row: its places in the order by expert (rows of an expert keep their order, so the order
 //                      does not depend on timing), and the row copied there; the first CTA lists the tiles
 //   moe_route_kernel   both for up to 64 rows, in one cluster
 //   moe_simt_kernel    64 rows x 64 columns of one tile, k ascending, optionally with the gated activation of the scored products
-//   moe_swiglu_kernel  the same activation on k-split products
+//   moe_swiglu_kernel  the same activation on k-split products (moe_act_kernel: of experts without a gate)
 #include "kernels.h"
 #include "mma.cuh"
 
@@ -19,6 +19,40 @@ namespace {
 __host__ __device__ inline uint32_t row_block(uint32_t rows) { return rows <= 512 ? 8 : 64; }
 constexpr uint32_t kPlaceRows = 8;
 constexpr uint32_t kClusterRows = 64;  // batches of up to this many rows: one kernel, a cluster of a CTA per 8 rows
+
+// The largest of `value(e)` over the warp's n entries and its place, the lower one of equal ones; at = n or more if there is none.
+template <typename F>
+__device__ __forceinline__ void warp_best(uint32_t n, F value, float &best, uint32_t &at) {
+  best = -INFINITY, at = 0xFFFFFFFFu;
+  for (uint32_t e = threadIdx.x & 31; e < n; e += 32) {
+    const float v = value(e);
+    if (v > best) best = v, at = e;
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+    const uint32_t oi = __shfl_xor_sync(0xffffffffu, at, o);
+    if (ov > best || (ov == best && oi < at)) best = ov, at = oi;
+  }
+}
+
+// Leaves the scores of the `keep` best groups in `mine` and minus infinity for the others. Scores are not negative, so the sign bit can
+// mark the groups that have been taken.
+__device__ __forceinline__ void keep_groups(const MoeShape &s, float *mine) {
+  const uint32_t lane = threadIdx.x & 31, outputs = s.outputs(), per = outputs / s.groups;
+  for (uint32_t k = 0; k < s.keep; ++k) {
+    float best;
+    uint32_t at;
+    warp_best(outputs, [&](uint32_t e) { return signbit(mine[e]) ? -INFINITY : mine[e]; }, best, at);
+    __syncwarp();
+    if (at >= outputs) break;  // only if scores are not numbers
+    const uint32_t first = at / per * per;
+    for (uint32_t e = first + lane; e < first + per; e += 32) mine[e] = -mine[e];
+    __syncwarp();
+  }
+  for (uint32_t e = lane; e < outputs; e += 32) mine[e] = signbit(mine[e]) ? -mine[e] : -INFINITY;
+  __syncwarp();
+}
 
 // One warp: scores of one row in `mine`, its choices to chosen / score, those that name an expert with weights counted in `count`
 // (shared memory). The correction takes part in the choice only.
@@ -47,22 +81,16 @@ __device__ __forceinline__ void choose_row(const float *__restrict__ logits, uin
     for (uint32_t e = lane; e < outputs; e += 32) mine[e] /= sum;
   }
   __syncwarp();
+  if (s.groups && s.keep < s.groups) keep_groups(s, mine);
+  float total = 0.f;
   for (uint32_t k = 0; k < s.top; ++k) {
-    float best = -INFINITY;
-    uint32_t at = 0xFFFFFFFFu;
-    for (uint32_t e = lane; e < outputs; e += 32) {
-      const float v = correction ? mine[e] + correction[e] : mine[e];
-      if (v > best) best = v, at = e;
-    }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-      const uint32_t oi = __shfl_xor_sync(0xffffffffu, at, o);
-      if (ov > best || (ov == best && oi < at)) best = ov, at = oi;
-    }
+    float best;
+    uint32_t at;
+    warp_best(outputs, [&](uint32_t e) { return correction ? mine[e] + correction[e] : mine[e]; }, best, at);
     if (at >= outputs) at = k;  // only if scores are not numbers: stay inside the router's outputs (top is at most as many)
     __syncwarp();
     if (lane == 0) {
+      total += mine[at];
       chosen[k] = at;
       score[k] = mine[at];
       mine[at] = -INFINITY;
@@ -70,6 +98,9 @@ __device__ __forceinline__ void choose_row(const float *__restrict__ logits, uin
     }
     __syncwarp();
   }
+  if (s.renorm && lane == 0)
+    for (uint32_t k = 0; k < s.top; ++k) score[k] /= total + 1e-20f;
+  __syncwarp();
 }
 
 __global__ void __launch_bounds__(1024)
@@ -85,7 +116,7 @@ moe_choose_kernel(const float *__restrict__ logits, uint32_t splits, size_t spli
   __syncthreads();
   const uint32_t end = min(rows, (blockIdx.x + 1) * block);
   for (uint32_t row = blockIdx.x * block + warp; row < end; row += warps)
-    choose_row(logits + (size_t)row * outputs, splits, split_stride, correction, s, smem + warp * outputs, chosen + (size_t)row * top,
+    choose_row(logits + (size_t)row * s.row_ld(), splits, split_stride, correction, s, smem + warp * outputs, chosen + (size_t)row * top,
                score + (size_t)row * top, count);
   __syncthreads();
   for (uint32_t e = tid; e < experts; e += blockDim.x) histogram[(size_t)blockIdx.x * experts + e] = count[e];
@@ -203,7 +234,7 @@ moe_route_kernel(const float *__restrict__ logits, uint32_t splits, size_t split
   pdl_wait();
   const uint32_t row = blockIdx.x * kPlaceRows + warp;
   if (row < rows)
-    choose_row(logits + (size_t)row * R, splits, split_stride, correction, s, smem + warp * R, chosen + warp * top, score + warp * top, count);
+    choose_row(logits + (size_t)row * s.row_ld(), splits, split_stride, correction, s, smem + warp * R, chosen + warp * top, score + warp * top, count);
   __syncthreads();
   asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
   asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
@@ -257,7 +288,8 @@ struct SimtFamily {
   float *out;
   GatedAct gate;
 };
-template <typename T, bool SWIGLU>
+// ACT: 0 = f32 products, 1 = a gated activation of them, 2 = an activation without a gate.
+template <typename T, int ACT>
 __global__ void __launch_bounds__(256)
 moe_simt_kernel(SimtFamily<T> routed, SimtFamily<T> shared, uint32_t shared_tiles, uint32_t rows, const MoeTile *__restrict__ tiles,
                 const float *__restrict__ row_score) {
@@ -298,12 +330,13 @@ moe_simt_kernel(SimtFamily<T> routed, SimtFamily<T> shared, uint32_t shared_tile
     const uint32_t r = ty * 4 + i;
     if (r >= t.count) continue;
     const size_t row = t.row + r;
-    const float score = is_shared || !SWIGLU || !row_score ? 1.f : row_score[row];  // multiplies what the expert reads
+    const float score = is_shared || !ACT || !row_score ? 1.f : row_score[row];  // multiplies what the expert reads
 #pragma unroll
-    for (int j = 0; j < 4; j += SWIGLU ? 2 : 1) {
+    for (int j = 0; j < 4; j += ACT == 1 ? 2 : 1) {
       const uint32_t n = n0 + tx * 4 + j;
       if (n >= f.n) continue;
-      if (SWIGLU) f.act[row * (f.n / 2) + n / 2] = from_f32<T>(gated<T>(f.gate, score * acc[i][j], score * acc[i][j + (SWIGLU ? 1 : 0)]));
+      if (ACT == 1) f.act[row * (f.n / 2) + n / 2] = from_f32<T>(gated<T>(f.gate, score * acc[i][j], score * acc[i][j + (ACT == 1 ? 1 : 0)]));
+      else if (ACT == 2) f.act[row * f.n + n] = from_f32<T>(gelu_erf<T>(score * acc[i][j]));
       else f.out[row * f.n + n] = acc[i][j];
     }
   }
@@ -327,6 +360,23 @@ moe_swiglu_kernel(const float *__restrict__ up, uint32_t splits, MoeShape s, uin
     }
     const float w = is_shared || !row_score ? 1.f : row_score[i / s.ffn];
     act[i] = from_f32<T>(gated<T>(is_shared ? s.shared_act : s.act, w * v.x, w * v.y));
+  }
+}
+
+// The same for experts without a gate: [splits][rows][ffn].
+template <typename T>
+__global__ void __launch_bounds__(256)
+moe_act_kernel(const float *__restrict__ up, uint32_t splits, MoeShape s, uint32_t rows, const float *__restrict__ row_score, T *__restrict__ act) {
+  pdl_trigger();
+  pdl_wait();
+  const size_t routed = (size_t)rows * s.top * s.ffn, all = routed + (size_t)rows * s.shared_ffn;
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < all; i += (size_t)gridDim.x * blockDim.x) {
+    const bool is_shared = i >= routed;
+    const size_t stride = is_shared ? all - routed : routed;
+    const float *p = up + (is_shared ? splits * routed + (i - routed) : i);
+    float v = 0.f;
+    for (uint32_t k = 0; k < splits; ++k) v += p[k * stride];
+    act[i] = from_f32<T>(gelu_erf<T>((is_shared || !row_score ? 1.f : row_score[i / s.ffn]) * v));
   }
 }
 
@@ -360,7 +410,7 @@ MoePlan moe_plan(bool is_bf16, MoeShape s, uint32_t rows) {
       const uint32_t most = std::max(1u, (k + 63) / 64 / 4);
       return (uint32_t)std::max<uint64_t>(1, std::min<uint64_t>({296 / std::max<uint64_t>(1, ctas), most, 8}));
     };
-    p.up_splits = splits(2 * s.ffn, 2 * s.shared_ffn, s.hidden);
+    p.up_splits = splits(s.up_cols(), s.shared_up_cols(), s.hidden);
     p.down_splits = splits(s.hidden, s.shared_ffn ? s.hidden : 0, s.ffn);
   }
   return p;
@@ -368,7 +418,7 @@ MoePlan moe_plan(bool is_bf16, MoeShape s, uint32_t rows) {
 
 size_t moe_up_floats(bool is_bf16, MoeShape s, uint32_t rows) {
   const MoePlan p = moe_plan(is_bf16, s, rows);
-  return p.up_splits == 1 ? 0 : (size_t)p.up_splits * rows * 2 * ((size_t)s.top * s.ffn + s.shared_ffn);
+  return p.up_splits == 1 ? 0 : (size_t)p.up_splits * rows * ((size_t)s.top * s.up_cols() + s.shared_up_cols());
 }
 
 template <typename T>
@@ -378,6 +428,8 @@ int launch_moe_route(const float *logits, uint32_t splits, size_t split_stride, 
   const uint32_t outputs = s.outputs();
   if (s.experts == 0 || outputs > kMoeMaxExperts || s.top == 0 || s.top > outputs)
     return set_error(ORION_ERR_INTERNAL, "routing of %u among %u experts is not supported (at most %u)", s.top, outputs, kMoeMaxExperts);
+  if (s.groups && (!s.softmax || correction || outputs % s.groups || s.keep == 0 || s.keep > s.groups || s.top > outputs / s.groups * s.keep))
+    return set_error(ORION_ERR_INTERNAL, "routing of %u among %u of %u groups of %u experts is not supported", s.top, s.keep, s.groups, outputs);
   if (rows <= kClusterRows) {
     const uint32_t ctas = (rows + kPlaceRows - 1) / kPlaceRows;
     const size_t smem = (kPlaceRows * (size_t)outputs + 5 * (size_t)s.experts + 2 * kPlaceRows * s.top) * 4;
@@ -403,11 +455,11 @@ int launch_moe_route(const float *logits, uint32_t splits, size_t split_stride, 
 
 namespace {
 template <typename T>
-int launch_simt(bool swiglu, SimtFamily<T> routed, SimtFamily<T> shared, MoePlan plan, const MoeBuffers<T> &b, const float *row_score, uint32_t rows,
+int launch_simt(int act, SimtFamily<T> routed, SimtFamily<T> shared, MoePlan plan, const MoeBuffers<T> &b, const float *row_score, uint32_t rows,
                 cudaStream_t stream) {
   const uint32_t shared_tiles = shared.n ? (rows + BM - 1) / BM : 0;
   const dim3 grid((std::max(routed.n, shared.n) + BN - 1) / BN, shared_tiles + plan.tiles);
-  auto kernel = swiglu ? moe_simt_kernel<T, true> : moe_simt_kernel<T, false>;
+  auto kernel = act == 0 ? moe_simt_kernel<T, 0> : (act == 1 ? moe_simt_kernel<T, 1> : moe_simt_kernel<T, 2>);
   ORION_CUDA_CHECK("moe_simt", launch_pdl(kernel, grid, dim3(256), 0, stream, routed, shared, shared_tiles, rows, (const MoeTile *)b.tiles,
                                           row_score));
   return after_launch("moe_simt");
@@ -421,16 +473,18 @@ int launch_moe_experts(const T *x, const T *w_up, const T *w_down, const T *shar
   const size_t sorted = (size_t)rows * s.top;
   const float *row_score = s.weigh_output ? nullptr : b.row_score;
   T *shared_act = b.act + sorted * s.ffn;
+  const uint32_t up_n = s.up_cols(), shared_up_n = s.shared_up_cols();
+  if (s.act.plain() != s.shared_act.plain()) return set_error(ORION_ERR_INTERNAL, "routed and shared experts are of one form");
   if constexpr (sizeof(T) == 2) {
     if (plan.tensor_core) {
       const bool fused = plan.up_splits == 1;
-      float *shared_up_out = fused ? nullptr : b.up + plan.up_splits * sorted * 2 * s.ffn;
-      MoeProduct p{b.x, w_up, x, shared_up, 2 * s.ffn, s.hidden, 2 * s.shared_ffn, s.hidden, (uint32_t)sorted, rows, s.experts, b.tiles, row_score,
+      float *shared_up_out = fused ? nullptr : b.up + plan.up_splits * sorted * up_n;
+      MoeProduct p{b.x, w_up, x, shared_up, up_n, s.hidden, shared_up_n, s.hidden, (uint32_t)sorted, rows, s.experts, b.tiles, row_score,
                    b.act, shared_act, fused ? nullptr : b.up, shared_up_out, s.act, s.shared_act};
       ORION_TRY(launch_moe_product_tc(p, fused, plan.up_splits, plan, stream));
       if (!fused) {
         const size_t n = sorted * s.ffn + (size_t)rows * s.shared_ffn;
-        ORION_CUDA_CHECK("moe_swiglu", launch_pdl(moe_swiglu_kernel<T>, dim3((uint32_t)std::min<size_t>((n + 255) / 256, 148 * 8)), dim3(256), 0, stream,
+        ORION_CUDA_CHECK("moe_swiglu", launch_pdl(s.act.plain() ? moe_act_kernel<T> : moe_swiglu_kernel<T>, dim3((uint32_t)std::min<size_t>((n + 255) / 256, 148 * 8)), dim3(256), 0, stream,
                                                   (const float *)b.up, plan.up_splits, s, rows, row_score, b.act));
         ORION_TRY(after_launch("moe_swiglu"));
       }
@@ -439,9 +493,9 @@ int launch_moe_experts(const T *x, const T *w_up, const T *w_down, const T *shar
       return launch_moe_product_tc(d, false, plan.down_splits, plan, stream);
     }
   }
-  ORION_TRY(launch_simt<T>(true, {b.x, w_up, 2 * s.ffn, s.hidden, b.act, nullptr, s.act},
-                           {x, shared_up, 2 * s.shared_ffn, s.hidden, shared_act, nullptr, s.shared_act}, plan, b, row_score, rows, stream));
-  return launch_simt<T>(false, {b.act, w_down, s.hidden, s.ffn, nullptr, b.down},
+  ORION_TRY(launch_simt<T>(s.act.plain() ? 2 : 1, {b.x, w_up, up_n, s.hidden, b.act, nullptr, s.act},
+                           {x, shared_up, shared_up_n, s.hidden, shared_act, nullptr, s.shared_act}, plan, b, row_score, rows, stream));
+  return launch_simt<T>(0, {b.act, w_down, s.hidden, s.ffn, nullptr, b.down},
                         {shared_act, shared_down, s.shared_ffn ? s.hidden : 0, s.shared_ffn, nullptr, shared_out}, plan, b, nullptr, rows, stream);
 }
 

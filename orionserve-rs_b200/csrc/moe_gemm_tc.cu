@@ -7,7 +7,8 @@
 //              preceding kernel has ended; the others once the tile list is there)
 //   warp 2     one lane does the same with the tile's rows
 //   warp 1     allocates tensor memory, one lane issues the MMAs
-//   warps 4-7  epilogue: f32 rows, or f(w g) * (w u), f a gated activation, of neighbouring gate and up rows with the row's score w
+//   warps 4-7  epilogue: f32 rows, or f(w g) * (w u), f a gated activation, of neighbouring gate and up rows with the row's score w, or
+//              an activation f(w u) without a gate
 // Every wait is bounded; a wait that runs out sets the device error word and the CTA still frees its tensor memory.
 #include "kernels.h"
 #include "tcgen05.cuh"
@@ -43,7 +44,7 @@ struct TcArgs {
   GatedAct f, shared_f;
 };
 
-// GATED: 0 = f32 products, 1 = SwiGLU, 2 = the gated activations of the arguments.
+// GATED: 0 = f32 products, 1 = SwiGLU, 2 = the gated activations of the arguments, 3 = no gate, the exact GELU of every product.
 template <int TOKN, int WST, int XST, int MT, int GATED>
 __global__ void __launch_bounds__(kThreads)
 moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_sw,
@@ -156,7 +157,16 @@ moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
         const int mc = mb + 16 * b;
         const uint32_t c = mc % TOKN, nn = n0 + (mc / TOKN) * kTileN + lq * 32 + lane;  // first row of the tile in this chunk, weight row
         if (c >= tile.count) continue;  // warp-uniform
-        if (GATED) {
+        if (GATED == 3) {
+          if (nn < n) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) {
+              if (c + j >= tile.count) continue;
+              const float w = shared || !a.row_score ? 1.f : a.row_score[tile.row + c + j];
+              act[(size_t)(tile.row + c + j) * n + nn] = __float2bfloat16_rn(gelu_erf<bf16>(w * __uint_as_float(rr[b][j])));
+            }
+          }
+        } else if (GATED) {
           // lane 2i holds gate f, lane 2i + 1 up f, of the same f for these 16 rows; a pair trades halves and each
           // finishes one row of every two
           const uint32_t odd = lane & 1u, f = nn >> 1, ffn = n >> 1;
@@ -222,9 +232,12 @@ int launch_product(const MoeProduct &p, bool swiglu, uint32_t splits, MoePlan pl
   const uint32_t shared_tiles = p.shared_n ? (p.rows + TOKN - 1) / TOKN : 0;
   const TcArgs a{p.n, p.k, p.shared_n, p.shared_k, shared_tiles, p.rows, p.sorted_rows, splits, p.tiles, p.row_score, p.act, p.shared_act, p.out, p.shared_out, p.f, p.shared_f};
   const dim3 grid((std::max(p.n, p.shared_n) + MT * kTileN - 1) / (MT * kTileN), shared_tiles + plan.tiles, splits);
-  static bool attr_set[3][kMaxDeviceOrdinals] = {};
-  const int form = !swiglu ? 0 : (p.f.kind == kGatedSilu && p.shared_f.kind == kGatedSilu ? 1 : 2);
-  auto kernel = form == 0 ? moe_gemm_tc_kernel<TOKN, WST, XST, MT, 0> : (form == 1 ? moe_gemm_tc_kernel<TOKN, WST, XST, MT, 1> : moe_gemm_tc_kernel<TOKN, WST, XST, MT, 2>);
+  static bool attr_set[4][kMaxDeviceOrdinals] = {};
+  const int form = !swiglu ? 0 : (p.f.plain() ? 3 : (p.f.kind == kGatedSilu && p.shared_f.kind == kGatedSilu ? 1 : 2));
+  auto kernel = form == 0   ? moe_gemm_tc_kernel<TOKN, WST, XST, MT, 0>
+                : form == 1 ? moe_gemm_tc_kernel<TOKN, WST, XST, MT, 1>
+                : form == 2 ? moe_gemm_tc_kernel<TOKN, WST, XST, MT, 2>
+                            : moe_gemm_tc_kernel<TOKN, WST, XST, MT, 3>;
   ORION_CUDA_CHECK("moe_gemm attr", ensure_dynamic_smem(kernel, Cfg::kSmemBytes, attr_set[form]));
   ORION_CUDA_CHECK("moe_gemm", launch_pdl(kernel, grid, dim3(kThreads), (size_t)Cfg::kSmemBytes, stream, *mw, *mx, *msw, *msx, a));
   count_launch();

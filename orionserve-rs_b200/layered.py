@@ -1,6 +1,6 @@
 """``CudaLayeredModel`` — decoders whose configuration lists their layers one by one, each with its own token
-mixer, feed-forward and sizes (``OrionLayeredDesc`` in include/orion_cuda.h) — and the readers of Metapel's, Zulozen's and
-Belizen's ``config.json``."""
+mixer, feed-forward and sizes (``OrionLayeredDesc`` in include/orion_cuda.h) — and the readers of Metapel's, Zulozen's,
+Belizen's and Vusenex's ``config.json``."""
 from __future__ import annotations
 
 import ctypes as C
@@ -21,10 +21,12 @@ from .types import DType
 MIXERS = {"mingru": _ffi.MIXER_MIN_GRU, "latent_attention": _ffi.MIXER_LATENT_ATTENTION, "attention": _ffi.MIXER_ATTENTION,
           "gla": _ffi.MIXER_GLA}
 ACTIVATIONS = {"gelu_tanh": _ffi.ACT_GELU_TANH, "relu2": _ffi.ACT_RELU2, "geglu_tanh": _ffi.ACT_GEGLU_TANH}
-BLOCKS = {"parallel": _ffi.BLOCK_PARALLEL, "sandwich": _ffi.BLOCK_SANDWICH, "prenorm": _ffi.BLOCK_PRENORM}
+BLOCKS = {"parallel": _ffi.BLOCK_PARALLEL, "sandwich": _ffi.BLOCK_SANDWICH, "prenorm": _ffi.BLOCK_PRENORM,
+          "gated_postnorm": _ffi.BLOCK_GATED_POSTNORM}
 QK_NORMS = {False: _ffi.QK_NORM_NONE, True: _ffi.QK_NORM_ALL_HEADS, "per_head": _ffi.QK_NORM_PER_HEAD}
-ROUTERS = {"sigmoid_input": _ffi.ROUTER_SIGMOID_INPUT, "softmax": _ffi.ROUTER_SOFTMAX}
-EXPERT_FORMS = {"swiglu": _ffi.EXPERT_SWIGLU, "clamped": _ffi.EXPERT_CLAMPED}
+SINKS = {False: _ffi.SINK_NONE, True: _ffi.SINK_LEARNED, "zero": _ffi.SINK_ZERO}
+ROUTERS = {"sigmoid_input": _ffi.ROUTER_SIGMOID_INPUT, "softmax": _ffi.ROUTER_SOFTMAX, "softmax_renorm": _ffi.ROUTER_SOFTMAX_RENORM}
+EXPERT_FORMS = {"swiglu": _ffi.EXPERT_SWIGLU, "clamped": _ffi.EXPERT_CLAMPED, "gelu": _ffi.EXPERT_GELU}
 
 
 @dataclass(frozen=True)
@@ -43,6 +45,22 @@ class Loop:
     start: int
     stop: int
     times: int
+
+
+@dataclass(frozen=True)
+class Bigram:
+    """A table of embeddings of pairs of tokens: row (previous * ``mul_prev`` + token * ``mul_cur``) mod ``buckets``, and a further row
+    for a sequence's first token."""
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+
+
+@dataclass(frozen=True)
+class QueryTemperature:
+    """Queries are multiplied by 1 + ``coef`` ln(floor((position + 1) / ``every``) + 1)."""
+    coef: float
+    every: float
 
 
 @dataclass(frozen=True)
@@ -66,7 +84,7 @@ class LayerSpec:
     kv_heads: int = 0
     chunk: int = 0
     qk_norm: object = False  # False, True (over all heads at once) or "per_head"
-    sinks: bool = False
+    sinks: object = False  # False, True (a learned logit per head) or "zero"
     head_gate: bool = False
     # dense feed-forward
     activation: str = "gelu_tanh"
@@ -92,20 +110,30 @@ class LayerSpec:
     expert_form: str = "swiglu"
     expert_limit: float = 0.0
     shared_limit: float = 0.0
+    router_groups: int = 0  # 0 = experts form no groups
+    router_keep: int = 0
+    # attention: the values are the keys before their norm; a learned logarithm of the distance is taken off the scores
+    keys_as_values: bool = False
+    distance_bias: bool = False
+    q_temp: Optional[QueryTemperature] = None
+    ungated: bool = False  # latent_attention: no gate on the output
 
     def _c(self) -> "_ffi.OrionLayerDesc":
         return _ffi.OrionLayerDesc(
             MIXERS[self.mixer], self.ffn_dim, self.width, self.heads, self.dim, self.rot_dim, self.value_dim, self.kv_rank,
             self.window, self.rope_dims, self.rope_base, self.scale, self.kv_heads, self.chunk, QK_NORMS[self.qk_norm],
-            int(self.sinks), int(self.head_gate), ACTIVATIONS[self.activation], int(self.ffn_bias), self.experts,
+            SINKS[self.sinks], int(self.head_gate), ACTIVATIONS[self.activation], int(self.ffn_bias), self.experts,
             self.experts_per_token, self.shared_dim, self.keep_first, int(self.rope_halves), int(self.qkv_bias),
             int(self.value_gate), self.softcap, *((y.factor, y.original, y.fast, y.slow) if (y := self.yarn) else (0.0,) * 4),
             self.decay_tau, self.decay_rank, ROUTERS[self.router], self.router_identity, EXPERT_FORMS[self.expert_form],
-            self.expert_limit, self.shared_limit)
+            self.expert_limit, self.shared_limit, self.router_groups, self.router_keep, int(self.keys_as_values),
+            int(self.distance_bias), *((t.coef, t.every) if (t := self.q_temp) else (0.0, 0.0)), int(self.ungated))
 
     def cache_values_per_token(self) -> int:
         if self.mixer == "latent_attention":
             return self.kv_rank + self.rot_dim
+        if self.keys_as_values:
+            return self.kv_heads * self.dim  # besides an f32 factor per head
         return self.kv_heads * (self.dim + self.value_dim) if self.mixer == "attention" else 0
 
 
@@ -126,6 +154,9 @@ class LayeredMetadata:
     embed_scale: float = 1.0
     logit_softcap: float = 0.0
     loop: Optional[Loop] = None
+    scalar_norms: bool = False  # the gain of a norm of the stream's width is one number
+    max_positions: int = 0  # rows of a table of learned positions; 0 = no such table
+    bigram: Optional[Bigram] = None
 
     @property
     def num_layers(self) -> int:
@@ -260,12 +291,44 @@ def _belizen_layer(i: int, entry: dict, shapes: dict) -> LayerSpec:
                      softcap=float(m.get("softcap") or 0.0), qk_norm="per_head", qkv_bias=True, value_gate=True, **ffn)
 
 
+def _read_vusenex(config: dict, name: str, shapes: dict) -> LayeredMetadata:
+    specs = [_vusenex_layer(i, entry) for i, entry in enumerate(config["layers"])]
+    pairs = config["embedding"]["bigram"]
+    return LayeredMetadata(architecture=config["architecture"], name=name, hidden_size=int(config["width"]),
+                           vocab_size=int(config["vocab"]), layers=specs, norm_eps=float(config["norm"]["eps"]),
+                           block="gated_postnorm", untied_lm_head=True, scalar_norms=True, max_positions=int(config["max_positions"]),
+                           bigram=Bigram(int(pairs["buckets"]), int(pairs["mul_prev"]), int(pairs["mul_cur"])))
+
+
+def _vusenex_layer(i: int, entry: dict) -> LayerSpec:
+    kind, m, mlp = entry["type"], entry["mixer"], entry["mlp"]
+    ffn = {}
+    if mlp is not None and mlp["kind"] != "moe":
+        raise ModelError(f"unsupported feed-forward {mlp['kind']!r} in layer {i}")
+    if mlp is not None:
+        router, shared, groups = mlp["router"], mlp.get("shared"), mlp["router"].get("groups") or {"count": 0, "keep": 0}
+        ffn = dict(ffn_dim=int(mlp["expert"]["ff"]), experts=int(router["experts"]), experts_per_token=int(router["top"]),
+                   router="softmax_renorm", router_groups=int(groups["count"]), router_keep=int(groups["keep"]), expert_form="gelu",
+                   shared_dim=int(shared["ff"]) if shared else 0)
+    if kind == "latent_attention":
+        return LayerSpec("latent_attention", heads=int(m["heads"]), dim=int(m["dim"]), value_dim=int(m["vdim"]), kv_rank=int(m["kv_rank"]),
+                         scale=float(m["scale"]), ungated=True, **ffn)
+    if kind != "attention":
+        raise ModelError(f"unsupported mixer {kind!r} in layer {i}")
+    if int(m["vdim"]) != int(m["dim"]):
+        raise ModelError(f"layer {i}: values of {m['vdim']} dimensions cannot be keys of {m['dim']}")
+    temp = m.get("q_temp")
+    return LayerSpec("attention", heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), value_dim=int(m["vdim"]),
+                     scale=float(m["scale"]), qk_norm=True, qkv_bias=True, sinks="zero", keys_as_values=True, distance_bias=True,
+                     q_temp=QueryTemperature(float(temp["coef"]), float(temp["every"])) if temp else None, **ffn)
+
+
 def _mask_size(mixer: dict) -> int:
     return int(mixer["mask"]["size"]) if mixer.get("mask") else 0
 
 
 #: config.json "architecture" -> reader
-READERS = {"Metapel": _read_metapel, "Zulozen": _read_zulozen, "Belizen": _read_belizen}
+READERS = {"Metapel": _read_metapel, "Zulozen": _read_zulozen, "Belizen": _read_belizen, "Vusenex": _read_vusenex}
 
 
 class CudaLayeredModel(CudaModel):
@@ -281,10 +344,12 @@ class CudaLayeredModel(CudaModel):
         layers = (_ffi.OrionLayerDesc * max(1, meta.num_layers))(*[s._c() for s in meta.layers])
         d = _ffi.OrionLayeredDesc(
             meta.hidden_size, meta.vocab_size, meta.num_layers, layers, meta.norm_eps, meta.conv_taps,
-            max_positions or num_blocks * block_size,  # no sequence is longer than the whole cache
+            min(max_positions or num_blocks * block_size,  # no sequence is longer than the whole cache
+                meta.max_positions or 1 << 31),
             num_blocks, block_size, num_state_slots or max_batch_sequences, int(compute_dtype), max_batch_tokens,
             max_batch_sequences, BLOCKS[meta.block], int(meta.untied_lm_head), meta.residual_mult, meta.embed_scale,
-            meta.logit_softcap, *((meta.loop.start, meta.loop.stop, meta.loop.times) if meta.loop else (0, 0, 0)))
+            meta.logit_softcap, *((meta.loop.start, meta.loop.stop, meta.loop.times) if meta.loop else (0, 0, 0)),
+            int(meta.scalar_norms), meta.max_positions, *((b.buckets, b.mul_prev, b.mul_cur) if (b := meta.bigram) else (0, 0, 0)))
         check(_ffi.lib().orion_cuda_model_create_layered(backend._h, C.byref(d), C.byref(self._h)))
 
     @classmethod
@@ -303,13 +368,14 @@ class CudaLayeredModel(CudaModel):
 
     def read_kv(self) -> List[np.ndarray]:
         """The caches of the attention layers in f32, one after the other in the order in which they run: latents as ``[block][slot][kv_rank + rot_dim]``, keys
-        and values as two arrays ``[block][kv head][slot][dim]``."""
+        and values as two arrays ``[block][kv head][slot][dim]``; where the values are the keys, one such array and the keys' factors
+        ``[block][kv head][slot][1]``."""
         shapes = []
         for s in self._meta.layer_runs():
             if s.mixer == "latent_attention":
                 shapes.append((self.num_blocks, self.block_size, s.kv_rank + s.rot_dim))
             elif s.mixer == "attention":
-                shapes += [(self.num_blocks, s.kv_heads, self.block_size, n) for n in (s.dim, s.value_dim)]
+                shapes += [(self.num_blocks, s.kv_heads, self.block_size, n) for n in (s.dim, 1 if s.keys_as_values else s.value_dim)]
         sizes = [int(np.prod(s)) for s in shapes]
         out = np.zeros(max(1, sum(sizes)), np.float32)
         check(_ffi.lib().orion_cuda_model_read_kv(self._h, out.ctypes.data_as(C.POINTER(C.c_float)), out.size))

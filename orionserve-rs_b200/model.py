@@ -69,7 +69,7 @@ def write_safetensors(path: str, tensors: Dict[str, np.ndarray], dtype: DType = 
     """Writes f32 arrays as F32 or (rounded to nearest even) BF16."""
     header, blobs, off = {}, [], 0
     for name, a in tensors.items():
-        a = np.ascontiguousarray(a, dtype=np.float32)
+        a = np.asarray(a, dtype=np.float32, order="C")  # keeps the rank of a single number
         if dtype == DType.BF16:
             bits = a.view(np.uint32)
             rounded = ((bits + 0x7FFF + ((bits >> 16) & 1)) >> 16).astype(np.uint16)
