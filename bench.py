@@ -354,8 +354,9 @@ def run_serving(args):
 
 # ---------------------------------------------------------------------------------------------
 # Layer-list designs beside the Llama layout at equal size: Metapel (min-GRU and latent attention layers), Zulozen
-# (chunked attention with sinks, dense and mixture-of-experts feed-forwards) and Belizen (gated linear attention and sliding windows that
-# keep the first tokens, gated dense and mixture-of-experts feed-forwards)
+# (chunked attention with sinks, dense and mixture-of-experts feed-forwards), Belizen (gated linear attention and sliding windows that
+# keep the first tokens, gated dense and mixture-of-experts feed-forwards) and Vusenex (latent attention and attention whose values are its
+# keys, mixtures of experts in groups, gated residual)
 # ---------------------------------------------------------------------------------------------
 
 # Layer sizes of real models, random weights; the layers alternate min-GRU and latent attention.
@@ -381,6 +382,14 @@ BELIZEN_SHAPES = {
                  expert_ffn=1408, shared=2816),
     "4096": dict(hidden=4096, ffn=16384, dense=11008, heads=32, dim=128, rot=64, window=1024, keep=8, gla_dim=64, rank=16, experts=16, identity=2, top=2,
                  expert_ffn=2816, shared=5632),
+}
+
+
+# Latent attention and attention with keys as values alternate. A token's experts (without gates) and the shared one are about as large as a
+# dense feed-forward of 8192 (16384); `ffn` counts the gates of the two sublayers as well.
+VUSENEX_SHAPES = {
+    "2048": dict(hidden=2048, ffn=10240, heads=16, dim=128, rank=512, experts=16, groups=4, keep=2, top=2, expert_ffn=2112, shared=4224),
+    "4096": dict(hidden=4096, ffn=20480, heads=32, dim=128, rank=512, experts=16, groups=4, keep=2, top=2, expert_ffn=4224, shared=8448),
 }
 
 
@@ -495,6 +504,42 @@ def belizen_work(meta, rows, contexts, prompts):
     return w + 2 * LAYERED_VOCAB * H, flops + 2 * outs * LAYERED_VOCAB * H, cache, attn
 
 
+def vusenex_meta(pkg, name, layers):
+    z = VUSENEX_SHAPES[name]
+    both = dict(ffn_dim=z["expert_ffn"], heads=z["heads"], dim=z["dim"], value_dim=z["dim"], scale=z["dim"] ** -0.5, experts=z["experts"],
+                experts_per_token=z["top"], router="softmax_renorm", router_groups=z["groups"], router_keep=z["keep"], expert_form="gelu",
+                shared_dim=z["shared"])
+    lat = pkg.LayerSpec("latent_attention", kv_rank=z["rank"], ungated=True, **both)
+    att = pkg.LayerSpec("attention", kv_heads=z["heads"] // 4, qk_norm=True, qkv_bias=True, sinks="zero", keys_as_values=True, distance_bias=True,
+                        q_temp=pkg.QueryTemperature(0.1, 512.0), **both)
+    return pkg.LayeredMetadata("Vusenex", f"vusenex-{name}", z["hidden"], LAYERED_VOCAB, [att if i % 2 else lat for i in range(layers)], 1e-6,
+                               block="gated_postnorm", untied_lm_head=True, scalar_norms=True, max_positions=8192,
+                               bigram=pkg.Bigram(32749, 31, 17))
+
+
+def vusenex_work(meta, rows, contexts, prompts):
+    """As ``zulozen_work``, and as ``metapel_work`` for latents. Keys that are values count once, with their factors."""
+    w = flops = cache = attn = 0
+    H = meta.hidden_size
+    keys = sum(contexts) + sum(p * (p + 1) // 2 for p in prompts)
+    for s in meta.layers:
+        q, v = s.heads * s.dim, s.heads * s.value_dim
+        if s.mixer == "latent_attention":
+            n = H * (q + s.kv_rank) + v * H + ((q + v) * s.kv_rank if prompts else 0)
+            cache += sum(contexts) * s.kv_rank * 2
+            attn += sum(contexts) * s.heads * 4 * s.kv_rank + (keys - sum(contexts)) * 2 * (q + v)
+        else:
+            n = H * (q + s.kv_heads * s.dim) + v * H
+            cache += sum(contexts) * s.kv_heads * (2 * s.dim + 4)
+            attn += keys * 2 * (q + v)
+        n += 2 * H * H + H * s.experts + 2 * H * s.shared_dim  # the gates, the router, the shared expert
+        one = 2 * H * s.ffn_dim
+        reached = s.experts * (1.0 - (1.0 - s.experts_per_token / s.experts) ** rows)
+        w, flops = w + 2 * n + 2 * int(reached * one), flops + 2 * (n + s.experts_per_token * one) * rows
+    outs = len(contexts) + len(prompts)
+    return w + 2 * LAYERED_VOCAB * H, flops + 2 * outs * LAYERED_VOCAB * H, cache, attn
+
+
 def llama_work(m, rows, contexts, prompts):
     w = weight_bytes_per_step(m)
     flops = 2 * rows * m["num_layers"] * layer_param_count(m) + 2 * (len(contexts) + len(prompts)) * m["vocab_size"] * m["hidden_size"]
@@ -520,7 +565,8 @@ def run_layered(args):
     design = args.workload
     shapes, make_meta, work = {"metapel": (METAPEL_SHAPES, metapel_meta, metapel_work),
                                "zulozen": (ZULOZEN_SHAPES, zulozen_meta, zulozen_work),
-                               "belizen": (BELIZEN_SHAPES, belizen_meta, belizen_work)}[design]
+                               "belizen": (BELIZEN_SHAPES, belizen_meta, belizen_work),
+                               "vusenex": (VUSENEX_SHAPES, vusenex_meta, vusenex_work)}[design]
     layers, out = args.layers if args.layers != 32 else 8, []
     batches = [("decode", b, CONTEXT) for b in (1, 16, 64)] + [("prefill", 1, 2048), ("prefill", 4, 2048)]
     with ClockSampler(0) as clocks:
@@ -727,7 +773,7 @@ def tp_parity(pkg, backend, dist, rank, world, dtype_name="BF16", model=None, nu
 def run_ours(args):
     if args.workload in ("serving", "prefix"):
         return run_serving(args)
-    if args.workload in ("metapel", "zulozen", "belizen"):
+    if args.workload in ("metapel", "zulozen", "belizen", "vusenex"):
         return run_layered(args)
     import __graft_entry__ as ge
 
@@ -943,13 +989,13 @@ def main():
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", choices=("ours", "reference"), default="ours")
     ap.add_argument("--no-cpu-baseline", action="store_true")
-    ap.add_argument("--workload", choices=("decode", "serving", "prefix", "metapel", "zulozen", "belizen"), default="decode",
+    ap.add_argument("--workload", choices=("decode", "serving", "prefix", "metapel", "zulozen", "belizen", "vusenex"), default="decode",
                     help="decode = the headline step (default); serving = continuous batching through the engine "
-                         "loop; prefix = shared-prefix requests on the Qwen2-7B shape through the engine loop; metapel, zulozen, belizen = "
+                         "loop; prefix = shared-prefix requests on the Qwen2-7B shape through the engine loop; metapel, zulozen, belizen, vusenex = "
                          "prefill and decode of that design at a few sizes beside the Llama layout")
-    ap.add_argument("--layered-shapes", "--metapel-shapes", default="2048,4096", help="metapel, zulozen and belizen workloads: layer sizes to run")
+    ap.add_argument("--layered-shapes", "--metapel-shapes", default="2048,4096", help="workloads named after a design: layer sizes to run")
     ap.add_argument("--layered-only", "--metapel-only", default="",
-                    help="metapel, zulozen and belizen workloads: batches to run, for instance decode64,prefill1")
+                    help="workloads named after a design: batches to run, for instance decode64,prefill1")
     ap.add_argument("--skip-cached-prefix", action="store_true",
                     help="engine workloads: start prefill after the tokens adopted from the prefix cache "
                          "(an extension; the reference shares the blocks but recomputes them)")

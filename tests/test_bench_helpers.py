@@ -91,3 +91,20 @@ def test_algorithmic_work_of_a_belizen_step(pkg):
     w, fl, cache, attn = bench.belizen_work(meta, 14, [], [14])
     assert w == 2 * (2 * lin + att + head) + 2 * int(3 * (1 - 0.75 ** 14) * expert)
     assert cache == 0 and attn == 14 * 2 * 4 * 32 * 12 + (78 + 2 * 12) * 4 * 2 * 56
+
+
+def test_algorithmic_work_of_a_vusenex_step(pkg):
+    moe = dict(ffn_dim=12, experts=4, experts_per_token=1, shared_dim=8, router="softmax_renorm", expert_form="gelu")
+    layers = [pkg.LayerSpec("latent_attention", heads=4, dim=32, value_dim=24, kv_rank=64, ungated=True, **moe),
+              pkg.LayerSpec("attention", heads=4, kv_heads=2, dim=32, value_dim=32, qk_norm=True, keys_as_values=True, **moe)]
+    meta = pkg.LayeredMetadata("Vusenex", "m", 48, 100, layers, 1e-5, block="gated_postnorm")
+    lat, att = 48 * (128 + 64) + 96 * 48, 48 * (128 + 64) + 128 * 48
+    rest, expert, head = 2 * 48 * 48 + 4 * 48 + 2 * 48 * 8, 2 * 48 * 12, bench.LAYERED_VOCAB * 48
+    w, fl, cache, attn = bench.vusenex_work(meta, 1, [27], [])  # one row reaches one expert
+    assert w == 2 * (lat + att + 2 * rest + 2 * expert + head) == fl
+    assert cache == 27 * (64 * 2 + 2 * (32 * 2 + 4)) and attn == 27 * (4 * 4 * 64 + 2 * 2 * 128)
+    w, fl, cache, attn = bench.vusenex_work(meta, 12, [], [12])
+    lat += (128 + 96) * 64
+    assert w == 2 * (lat + att + 2 * rest + head) + 2 * 2 * int(4 * (1 - 0.75 ** 12) * expert)
+    assert fl == 2 * (12 * (lat + att + 2 * rest + 2 * expert) + head)
+    assert cache == 0 and attn == 78 * (2 * (128 + 96) + 2 * 256)
