@@ -760,7 +760,8 @@ uint32_t group_tiles(KvLayout kv, uint32_t q_heads) { return (q_heads / kv.num_k
 template <int DK, int DV, bool JOINT>
 int launch_decode_form(const bf16 *q, const bf16 *arena, KvLayout kv, uint32_t layer, AttnBatch batch, uint32_t rows, uint32_t q_heads,
                        uint32_t splits, DecodeScratch scratch, AttnForm form, bf16 *out, cudaStream_t stream) {
-  constexpr int kFormStages = 3;
+  // as many bytes in flight with one set of rows as with two
+  constexpr int kFormStages = JOINT && DK <= 128 ? 6 : 3;
   constexpr uint32_t kSmem = JOINT ? joint_smem_bytes(kFormStages, DK) : decode_smem_bytes(kFormStages, DK, DV);
   static bool attr_set[kMaxDeviceOrdinals] = {};
   ORION_CUDA_CHECK("paged_decode attr", ensure_dynamic_smem(paged_decode_kernel<kFormStages, DK, DV, true, JOINT>, (int)kSmem, attr_set));

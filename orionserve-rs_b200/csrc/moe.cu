@@ -82,15 +82,19 @@ __device__ __forceinline__ void choose_row(const float *__restrict__ logits, uin
   }
   __syncwarp();
   if (s.groups && s.keep < s.groups) keep_groups(s, mine);
-  float total = 0.f;
+  float total = 0.f, own = 0.f;  // lane k keeps the score of choice k until their sum is known
   for (uint32_t k = 0; k < s.top; ++k) {
     float best;
     uint32_t at;
     warp_best(outputs, [&](uint32_t e) { return correction ? mine[e] + correction[e] : mine[e]; }, best, at);
     if (at >= outputs) at = k;  // only if scores are not numbers: stay inside the router's outputs (top is at most as many)
     __syncwarp();
-    if (lane == 0) {
+    if (s.renorm) {
       total += mine[at];
+      if (lane == k) own = mine[at];
+      __syncwarp();
+    }
+    if (lane == 0) {
       chosen[k] = at;
       score[k] = mine[at];
       mine[at] = -INFINITY;
@@ -98,9 +102,11 @@ __device__ __forceinline__ void choose_row(const float *__restrict__ logits, uin
     }
     __syncwarp();
   }
-  if (s.renorm && lane == 0)
-    for (uint32_t k = 0; k < s.top; ++k) score[k] /= total + 1e-20f;
-  __syncwarp();
+  if (s.renorm) {
+    for (uint32_t k = 32 + lane; k < s.top; k += 32) score[k] /= total + 1e-20f;
+    if (lane < s.top) score[lane] = own / (total + 1e-20f);
+    __syncwarp();
+  }
 }
 
 __global__ void __launch_bounds__(1024)

@@ -7,7 +7,7 @@
 //              preceding kernel has ended; the others once the tile list is there)
 //   warp 2     one lane does the same with the tile's rows
 //   warp 1     allocates tensor memory, one lane issues the MMAs
-//   warps 4-7  epilogue: f32 rows, or f(w g) * (w u), f a gated activation, of neighbouring gate and up rows with the row's score w, or
+//   warps 4-7  epilogue (all eight warps where an activation is computed): f32 rows, or f(w g) * (w u), f a gated activation, of neighbouring gate and up rows with the row's score w, or
 //              an activation f(w u) without a gate
 // Every wait is bounded; a wait that runs out sets the device error word and the CTA still frees its tensor memory.
 #include "kernels.h"
@@ -130,7 +130,12 @@ moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
       }
       umma_commit(acc_ready);
     }
-  } else if (warp >= 4 && live) {
+  }
+  __syncwarp();
+  // The epilogue is on all eight warps where it computes something: the four that may read the same rows of tensor memory share the
+  // chunks of a tile with the four others. Values come before the tests for rows past the end, so that they overlap.
+  constexpr uint32_t kGroups = GATED ? 2 : 1;
+  if (live && (kGroups == 2 || warp >= 4)) {
     const uint32_t lq = warp & 3;
     pdl_wait();  // the results may still be read by the kernel before, and the scores come from one
     if (my_kb > 0 && !mbar_wait(acc_ready, 0)) ok = false;
@@ -138,9 +143,9 @@ moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
     tc_fence_after();
     float *out = shared ? a.shared_out + (size_t)split * a.rows * n : a.out + (size_t)split * a.sorted_rows * n;
     bf16 *act = shared ? a.shared_act : a.act;
-    constexpr int kBatch = TOKN >= 64 ? 4 : TOKN / 16;
+    constexpr int kBatch = TOKN >= 64 ? (GATED ? 2 : 4) : (GATED ? 1 : TOKN / 16);
 #pragma unroll 1
-    for (int mb = 0; mb < MT * TOKN; mb += 16 * kBatch) {
+    for (int mb = kGroups == 2 && warp < 4 ? 16 * kBatch : 0; mb < MT * TOKN; mb += 16 * kBatch * kGroups) {
       uint32_t rr[kBatch][16];
       if (ok && my_kb > 0) {
 #pragma unroll
@@ -158,27 +163,34 @@ moe_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
         const uint32_t c = mc % TOKN, nn = n0 + (mc / TOKN) * kTileN + lq * 32 + lane;  // first row of the tile in this chunk, weight row
         if (c >= tile.count) continue;  // warp-uniform
         if (GATED == 3) {
+          bf16 v[16], *to = act + (size_t)(tile.row + c) * n + nn;
+#pragma unroll
+          for (int j = 0; j < 16; ++j) {
+            const float w = shared || !a.row_score ? 1.f : a.row_score[tile.row + min(c + j, tile.count - 1)];
+            v[j] = __float2bfloat16_rn(gelu_erf<bf16>(w * __uint_as_float(rr[b][j])));
+          }
           if (nn < n) {
 #pragma unroll
-            for (int j = 0; j < 16; ++j) {
-              if (c + j >= tile.count) continue;
-              const float w = shared || !a.row_score ? 1.f : a.row_score[tile.row + c + j];
-              act[(size_t)(tile.row + c + j) * n + nn] = __float2bfloat16_rn(gelu_erf<bf16>(w * __uint_as_float(rr[b][j])));
-            }
+            for (int j = 0; j < 16; ++j, to += n)
+              if (c + j < tile.count) *to = v[j];
           }
         } else if (GATED) {
           // lane 2i holds gate f, lane 2i + 1 up f, of the same f for these 16 rows; a pair trades halves and each
           // finishes one row of every two
           const uint32_t odd = lane & 1u, f = nn >> 1, ffn = n >> 1;
+          bf16 v[8], *to = act + (size_t)(tile.row + c + odd) * ffn + f;
 #pragma unroll
           for (int jj = 0; jj < 8; ++jj) {
             const uint32_t send = odd ? rr[b][2 * jj] : rr[b][2 * jj + 1];
             const uint32_t recv = __shfl_xor_sync(0xffffffffu, send, 1);
-            const uint32_t r = c + 2 * jj + odd;
-            if (r >= tile.count || nn >= n) continue;
-            const float w = shared || !a.row_score ? 1.f : a.row_score[tile.row + r];
+            const float w = shared || !a.row_score ? 1.f : a.row_score[tile.row + min(c + 2 * jj + odd, tile.count - 1)];
             const float g = w * __uint_as_float(odd ? recv : rr[b][2 * jj]), u = w * __uint_as_float(odd ? rr[b][2 * jj + 1] : recv);
-            act[(size_t)(tile.row + r) * ffn + f] = __float2bfloat16_rn(GATED == 1 ? silu_for<bf16>(g) * u : gated<bf16>(shared ? a.shared_f : a.f, g, u));
+            v[jj] = __float2bfloat16_rn(GATED == 1 ? silu_for<bf16>(g) * u : gated<bf16>(shared ? a.shared_f : a.f, g, u));
+          }
+          if (nn < n) {
+#pragma unroll
+            for (int jj = 0; jj < 8; ++jj, to += 2 * (size_t)ffn)
+              if (c + 2 * jj + odd < tile.count) *to = v[jj];
           }
         } else if (nn < n) {
 #pragma unroll
