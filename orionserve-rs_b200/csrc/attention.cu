@@ -401,10 +401,10 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
     if (JOINT) {
       const float *factor = reinterpret_cast<const float *>(my_ring + stage * kChunkBytes + kBlk * DK * 2);
       const float f_lo = factor[t_lo] * sl2, f_hi = factor[t_hi] * sl2, d_lo = (float)(ctx - 1 - lb * kBlk) - (float)t_lo;
-      s[0] = see_lo ? s[0] * f_lo - dm[0] * __log2f(fmaf(dr[0], d_lo, 1.f)) : -INFINITY;
-      s[1] = see_lo ? s[1] * f_lo - dm[1] * __log2f(fmaf(dr[1], d_lo, 1.f)) : -INFINITY;
-      s[2] = see_hi ? s[2] * f_hi - dm[0] * __log2f(fmaf(dr[0], d_lo - 8.f, 1.f)) : -INFINITY;
-      s[3] = see_hi ? s[3] * f_hi - dm[1] * __log2f(fmaf(dr[1], d_lo - 8.f, 1.f)) : -INFINITY;
+      s[0] = see_lo ? s[0] * f_lo - dm[0] * fast_log2(fmaf(dr[0], d_lo, 1.f)) : -INFINITY;
+      s[1] = see_lo ? s[1] * f_lo - dm[1] * fast_log2(fmaf(dr[1], d_lo, 1.f)) : -INFINITY;
+      s[2] = see_hi ? s[2] * f_hi - dm[0] * fast_log2(fmaf(dr[0], d_lo - 8.f, 1.f)) : -INFINITY;
+      s[3] = see_hi ? s[3] * f_hi - dm[1] * fast_log2(fmaf(dr[1], d_lo - 8.f, 1.f)) : -INFINITY;
     } else {
       s[0] = see_lo ? s[0] * sl2 : -INFINITY;
       s[1] = see_lo ? s[1] * sl2 : -INFINITY;

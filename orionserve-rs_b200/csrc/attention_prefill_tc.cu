@@ -10,7 +10,8 @@
 //              sixteen 128-byte rows, and because the arena keeps the 16-byte groups of a row XOR-permuted
 //              by slot & 7, those rows ARE the 128-byte-swizzled operand layout the MMA expects);
 //   warp 1     allocates tensor memory; one lane issues S = Q K^T (M 128, N 64, K 128) and, once the
-//              softmax warps have written P, O (+)= P V (M 128, N 128, K 64; V is the MN-major operand);
+//              softmax warps have written P, O (+)= P V (M 128, N 128, K 64; V is the MN-major operand; keys
+//              that are values as well are one tile for both);
 //   warps 2-5  one thread per row: read the row of S from tensor memory (lane = row, so max and sum
 //              are thread-local), mask by position, exponentiate, write P as bf16 into the shared
 //              memory the K tile has just vacated, and at the end scale O by 1 / sum and store it.
@@ -33,12 +34,15 @@ namespace {
 constexpr int kHd = 128, kBlk = 16;
 constexpr int kM = 128;      // (position, head) rows per CTA
 constexpr int kKeys = 64;    // keys per tile
-constexpr int kStages = 2;
 constexpr int kThreads = 192;
-constexpr uint32_t kTmemO = 64;              // S: columns 0..63 of tensor memory, O behind them
 // DK, DV: sizes of the K and V rows, multiples of 64. JOINT: one tile of rows is both K and V.
 template <int DK, int DV, bool JOINT>
 struct PrefillTcConfig {
+  // Where tensor memory has room for it without costing a CTA, S has two buffers: the scores of the next key tile are computed under
+  // the softmax of this one.
+  static constexpr bool kTwoS = JOINT && DV == 128;
+  static constexpr int kStages = kTwoS ? 3 : 2;
+  static constexpr uint32_t kTmemO = kTwoS ? 128 : 64;  // S: the first columns of tensor memory, O behind them
   static constexpr int kQBytes = DK / 64 * kM * 128;     // 64-dim slabs of [128 rows][128 bytes]
   static constexpr int kKBytes = DK / 64 * kKeys * 128;  // 64-dim slabs of [64 keys][128 bytes]
   static constexpr int kVBytes = DV / 64 * kKeys * 128;
@@ -67,7 +71,9 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                         uint32_t q_heads, bf16 *__restrict__ out, AttnForm form) {
   constexpr bool JOINT = FORM == 3;
   using Cfg = PrefillTcConfig<DK, DV, JOINT>;
-  constexpr int kQBytes = Cfg::kQBytes, kKBytes = Cfg::kKBytes, kStageBytes = Cfg::kStageBytes;
+  constexpr int kQBytes = Cfg::kQBytes, kKBytes = Cfg::kKBytes, kStageBytes = Cfg::kStageBytes, kStages = Cfg::kStages;
+  constexpr uint32_t kTmemO = Cfg::kTmemO;
+  constexpr bool kTwoS = Cfg::kTwoS;
   extern __shared__ uint8_t raw_smem[];
   uint8_t *smem = reinterpret_cast<uint8_t *>((reinterpret_cast<uintptr_t>(raw_smem) + 1023) & ~uintptr_t(1023));
   uint8_t *q_smem = smem;                 // [slab][row 128][128 B]
@@ -78,7 +84,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
   uint64_t *kv_empty = kv_full + kStages;
   uint64_t *q_ready = kv_empty + kStages;
   uint64_t *s_ready = q_ready + 1;
-  uint64_t *p_ready = s_ready + 1;
+  uint64_t *p_ready = s_ready + 2;
   uint64_t *o_ready = p_ready + 1;
   uint32_t *tmem_slot = reinterpret_cast<uint32_t *>(o_ready + 1);
 
@@ -101,7 +107,8 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
       mbar_init(&kv_empty[s], 1);
     }
     mbar_init(q_ready, 1);
-    mbar_init(s_ready, 1);
+    mbar_init(&s_ready[0], 1);
+    mbar_init(&s_ready[1], 1);
     mbar_init(p_ready, 1);
     mbar_init(o_ready, 1);
     mbar_fence_init();
@@ -163,20 +170,28 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     if (lane == 0) {
       constexpr uint32_t idesc_s = idesc(kM, kKeys, false), idesc_o = idesc(kM, DV, true);
       const uint32_t qa = smem_u32(q_smem);
-      if (!wait(q_ready, 0)) ok = false;
-      for (uint32_t j = 0; ok && j < ntiles; ++j) {
+      // S = Q K^T: 64-dim slabs, four 16-dim steps each (+32 bytes inside the swizzle atom)
+      auto scores = [&](uint32_t j) -> bool {
         const uint32_t s = j % kStages;
-        if (!wait(&kv_full[s], (j / kStages) & 1)) { ok = false; break; }
+        if (!wait(&kv_full[s], (j / kStages) & 1)) return false;
         tc_fence_after();
-        const uint32_t ka = smem_u32(ring + s * kStageBytes), va = JOINT ? ka : ka + kKBytes;
-        // S = Q K^T: 64-dim slabs, four 16-dim steps each (+32 bytes inside the swizzle atom)
+        const uint32_t ka = smem_u32(ring + s * kStageBytes), b = kTwoS ? j & 1 : 0;
 #pragma unroll
         for (int ks = 0; ks < DK / 16; ++ks) {
           const uint32_t h = ks >> 2, kk = ks & 3;
-          umma_bf16(tmem_base, desc_k_sw128(qa + h * (kM * 128) + kk * 32), desc_k_sw128(ka + h * (kKeys * 128) + kk * 32),
+          umma_bf16(tmem_base + b * kKeys, desc_k_sw128(qa + h * (kM * 128) + kk * 32), desc_k_sw128(ka + h * (kKeys * 128) + kk * 32),
                     idesc_s, ks > 0 ? 1u : 0u);
         }
-        umma_commit(s_ready);
+        umma_commit(&s_ready[b]);
+        return true;
+      };
+      if (!wait(q_ready, 0)) ok = false;
+      if (kTwoS && ok && ntiles > 0) ok = scores(0);
+      for (uint32_t j = 0; ok && j < ntiles; ++j) {
+        const uint32_t s = j % kStages;
+        // the other buffer's scores have been read: their P came before the product of the tile before
+        if (kTwoS ? j + 1 < ntiles && !scores(j + 1) : !scores(j)) { ok = false; break; }
+        const uint32_t ka = smem_u32(ring + s * kStageBytes), va = JOINT ? ka : ka + kKBytes;
         if (!wait(p_ready, j & 1)) { ok = false; break; }
         tc_fence_after();
         // O (+)= P V: P is [128 rows][64 keys] (where the K tile was, if it fits there); V is [key][dim]: MN-major, 16 keys per step
@@ -235,11 +250,12 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     if (FORM && form.sinks) ref = form.sinks[head] * 1.4426950408889634f, l = 1.f;
     for (uint32_t j = 0; j < ntiles; ++j) {
       const uint32_t s = j % kStages;
-      if (!__all_sync(0xffffffffu, wait(s_ready, j & 1))) ok = false;  // no break: the barriers below stay matched
+      const uint32_t sb = kTwoS ? j & 1 : 0;
+      if (!__all_sync(0xffffffffu, wait(&s_ready[sb], (kTwoS ? j >> 1 : j) & 1))) ok = false;  // no break: the barriers below stay matched
       tc_fence_after();
       uint32_t sr[2][32];
-      tmem_ld32(taddr, sr[0]);
-      tmem_ld32(taddr + 32, sr[1]);
+      tmem_ld32(taddr + sb * kKeys, sr[0]);
+      tmem_ld32(taddr + sb * kKeys + 32, sr[1]);
       tmem_ld_wait();
       const bool straight = FORM != 2 || j * (kKeys / kBlk) >= kept_blk || kept_blk == block0;  // the tile's keys follow one another
       const int key0 = (int)(logical(j * (kKeys / kBlk)) * kBlk);
@@ -247,15 +263,38 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
       if (JOINT) {
         if (!__all_sync(0xffffffffu, wait(&kv_full[s], (j / kStages) & 1))) ok = false;  // the factors landed with the tile
         const float4 *factor = reinterpret_cast<const float4 *>(factors + s * kKeys);
-        const float near = fmaf(dist_rate, (float)(pos - key0), 1.f);  // the logarithm's argument at the tile's first key
+        // The distance term at key i is dist_mult log2(mid + dist_rate t), t = 31.5 - i. Where t is small beside mid / dist_rate for every
+        // row of the warp, it is a polynomial in t: log(1 + x) = x - x^2 / 2 + x^3 / 3 - ... up to x^5 for |x| below 1/8, with
+        // t a constant of each key and the even and odd powers shared by the keys t and -t.
+        const float mid = fmaf(dist_rate, (float)(pos - key0) - 31.5f, 1.f), x1 = __fdividef(dist_rate, mid);
+        if (__all_sync(0xffffffffu, !valid || (mid > 0.f && x1 <= 0.125f / 31.5f))) {
+          const float lead = dist_mult * 1.4426950408889634f, x2 = x1 * x1;
+          const float c0 = dist_mult * fast_log2(mid), c1 = lead * x1, c2 = lead * x2 * -0.5f, c3 = lead * x2 * x1 * (1.f / 3.f),
+                      c4 = lead * x2 * x2 * -0.25f, c5 = lead * x2 * x2 * x1 * 0.2f;
 #pragma unroll
-        for (int i = 0; i < kKeys; i += 4) {
-          const float4 f = factor[i / 4];
-          const float fs[4] = {f.x, f.y, f.z, f.w};
+          for (int i = 0; i < kKeys / 2; i += 4) {
+            const float4 f = factor[i / 4], g = factor[kKeys / 4 - 1 - i / 4];
+            const float fs[4] = {f.x, f.y, f.z, f.w}, gs[4] = {g.w, g.z, g.y, g.x};
 #pragma unroll
-          for (int k = 0; k < 4; ++k) {
-            const float v = __uint_as_float(sr[(i + k) >> 5][(i + k) & 31]) * (fs[k] * sl2);
-            sr[(i + k) >> 5][(i + k) & 31] = __float_as_uint(v - dist_mult * __log2f(fmaf(-dist_rate, (float)(i + k), near)));
+            for (int k = 0; k < 4; ++k) {
+              const int a = i + k, b = kKeys - 1 - a;
+              const float t = 31.5f - (float)a, t2 = t * t;
+              const float even = fmaf(fmaf(c4, t2, c2), t2, c0), odd = fmaf(fmaf(c5, t2, c3), t2, c1);
+              sr[a >> 5][a & 31] = __float_as_uint(fmaf(__uint_as_float(sr[a >> 5][a & 31]), fs[k] * sl2, -fmaf(odd, t, even)));
+              sr[b >> 5][b & 31] = __float_as_uint(fmaf(__uint_as_float(sr[b >> 5][b & 31]), gs[k] * sl2, fmaf(odd, t, -even)));
+            }
+          }
+        } else {
+          const float near = fmaf(dist_rate, (float)(pos - key0), 1.f);  // the logarithm's argument at the tile's first key
+#pragma unroll
+          for (int i = 0; i < kKeys; i += 4) {
+            const float4 f = factor[i / 4];
+            const float fs[4] = {f.x, f.y, f.z, f.w};
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+              const float v = __uint_as_float(sr[(i + k) >> 5][(i + k) & 31]) * (fs[k] * sl2);
+              sr[(i + k) >> 5][(i + k) & 31] = __float_as_uint(v - dist_mult * fast_log2(fmaf(-dist_rate, (float)(i + k), near)));
+            }
           }
         }
       }
@@ -306,9 +345,13 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         corr = (ref == -INFINITY) ? 1.0f : ex2(ref - nref);  // nothing accumulated yet under a reference of -inf
         ref = nref;
       }
+      if (kTwoS && j > 0) {  // P and O belong to the product of the previous tile until it has completed
+        if (!__all_sync(0xffffffffu, wait(o_ready, (j - 1) & 1))) ok = false;
+        tc_fence_after();
+      }
       if (__any_sync(0xffffffffu, corr != 1.0f) && j > 0) {
         // rescale this warp's rows of O in tensor memory (the MMAs of the previous tile have completed:
-        // S of this tile was issued after them)
+        // with one buffer S of this tile was issued after them)
 #pragma unroll 1
         for (uint32_t c = 0; c < DV; c += 32) {
           uint32_t orow[32];

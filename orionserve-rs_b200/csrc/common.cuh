@@ -180,6 +180,13 @@ __device__ __forceinline__ float softcap_log2(float x, float in, float out) {
   return out - __fdividef(2.f * out, 1.f + e);
 }
 
+// Logarithm to base 2 of a normal number, one instruction.
+__device__ __forceinline__ float fast_log2(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -273,7 +273,7 @@ def beacon_model(mixer, width=128, positions=900):
     return cfg, w
 
 
-BEACONS = {"attention": attn(6, 2, 64, temp=(0.2, 100)), "attention, few dimensions": attn(2, 1, 10), "latent attention": latent(3, 32, 32, 64),
+BEACONS = {"attention": attn(6, 2, 64, temp=(0.2, 100)), "attention, few dimensions": attn(2, 1, 10), "attention, many dimensions": attn(8, 2, 112), "latent attention": latent(3, 32, 32, 64),
            "latent attention, few dimensions": latent(2, 6, 10, 12)}
 
 
@@ -316,18 +316,19 @@ def test_a_far_key_among_hundreds(pkg, backend, dtype, name):
         assert worst_error(f.run("p", t, sizes), exp) < tol(dtype), sizes
 
 
-@pytest.mark.parametrize("rate", [0.0, 0.002, 5.0, 300.0])
-def test_distance_terms_of_any_rate(pkg, backend, dtype, rate):
-    """Flat ones, ones that fall slowly, and ones that fall at the first step, with multiples of either sign."""
-    cfg = config(96, 40, [attn(6, 3, 40)])
+@pytest.mark.parametrize("dim", [40, 128, 144])
+@pytest.mark.parametrize("rate", [0.0, 0.002, 0.2, 5.0, 300.0])
+def test_distance_terms_of_any_rate(pkg, backend, dtype, rate, dim):
+    """Flat ones, ones that fall slowly, and ones that fall at the first step, with multiples of either sign, near and far."""
+    cfg = config(96, 40, [attn(6, 3, dim)])
     w = random_weights(cfg, seed=3)
     w["l0.mix.r2"] = bf16(np.full(6, rate))
     w["l0.mix.r1"] = bf16(np.linspace(-0.5, 3.0, 6))
-    t = np.random.default_rng(1).integers(0, 40, 420).tolist()
+    t = np.random.default_rng(1).integers(0, 40, 620).tolist()
     exp = vusenex.forward(t, cfg, w)
     f = Feeder(pkg, make_model(pkg, backend, cfg, w, dtype))
-    assert worst_error(f.run("p", t, [420]), exp) < tol(dtype)
-    assert worst_error(f.run("q", t, [200, 2, 9, 100, 1]), exp) < tol(dtype)
+    assert worst_error(f.run("p", t, [620]), exp) < tol(dtype)
+    assert worst_error(f.run("q", t, [400, 2, 9, 150, 1]), exp) < tol(dtype)
 
 
 def test_pairs_of_tokens_across_steps(pkg, backend, dtype):
