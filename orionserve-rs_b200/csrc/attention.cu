@@ -139,6 +139,7 @@ paged_attention_generic_kernel(const T *__restrict__ q, const T *__restrict__ ar
 constexpr int kHd = 128;          // head_dim
 constexpr int kBlk = 16;          // tokens per KV block
 constexpr int kWarps = 4;         // warps per CTA, each with a private ring
+constexpr int kPlainWarps = kWarps;
 constexpr int kMaxGroup = 8;      // query heads per kv head (N of the MMA)
 // Ring depth per warp is a template parameter: 2 stages = 65 KiB per CTA (3 CTAs per SM),
 // 3 = 97 KiB (2 per SM), 4 = 129 KiB (1 per SM). The merge buffers (16.3 KiB) reuse the ring.
@@ -149,7 +150,9 @@ constexpr int chunk_bytes(int dk, int dv) { return kBlk * (dk + dv) * 2; }  // K
 constexpr uint32_t decode_smem_bytes(int stages, int dk = kHd, int dv = kHd) { return kWarps * stages * chunk_bytes(dk, dv) + 4096; }
 // One set of rows for keys and values and an f32 factor per slot. The ring is at least as large as the merge buffers that reuse it.
 constexpr int joint_chunk_bytes(int d) { return kBlk * d * 2 + kBlk * 4; }
-constexpr uint32_t joint_smem_bytes(int stages, int d) { return kWarps * stages * joint_chunk_bytes(d) + 4096; }
+// A block is half as many bytes as with two sets and as much work, so more warps share a row's blocks.
+constexpr int joint_warps(int d) { return d <= 128 ? 8 : 4; }
+constexpr uint32_t joint_smem_bytes(int stages, int d) { return joint_warps(d) * stages * joint_chunk_bytes(d) + 4096; }
 
 __device__ __forceinline__ float4 ld4(const float *p) { return *reinterpret_cast<const float4 *>(p); }
 __device__ __forceinline__ float4 add4(float4 a, float4 b) {
@@ -182,11 +185,12 @@ __device__ uint32_t g_decode_error = 0;
 // kv head (eight to a CTA); without it those branches and arguments are compiled out. JOINT: one set of rows for keys and values, with the
 // factors of the keys (KvLayout::factor_elems), and the distance term of `form`.
 template <int kStages, int DK, int DV, bool FORM, bool JOINT = false>
-__global__ void __launch_bounds__(kWarps * 32)
+__global__ void __launch_bounds__((JOINT ? joint_warps(DK) : kWarps) * 32)
 paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, KvLayout kv,
                     uint32_t layer, AttnBatch batch, uint32_t q_heads, uint32_t splits,
                     DecodeScratch scratch, bf16 *__restrict__ out, FusedQkv fq, AttnForm form) {
   static_assert(!JOINT || (FORM && DK == DV), "one set of rows has one size");
+  constexpr int kWarps = JOINT ? joint_warps(DK) : kPlainWarps;
   constexpr int kChunkBytes = JOINT ? joint_chunk_bytes(DK) : chunk_bytes(DK, DV);
   extern __shared__ __align__(1024) uint8_t dsmem[];
   uint8_t *ring = dsmem;  // [kWarps][kStages][kChunkBytes]
@@ -479,8 +483,9 @@ paged_decode_kernel(const bf16 *__restrict__ q, const bf16 *__restrict__ arena, 
     }
   }
   __syncthreads();
-  for (uint32_t d = threadIdx.x; d < (uint32_t)DV; d += kWarps * 32) {  // one output dim per thread and round
-    for (uint32_t g = 0; g < group; ++g) {
+  constexpr uint32_t kDims = kWarps * 32 < DV ? kWarps * 32 : DV;  // one output dim per thread and round, heads shared by the rest
+  for (uint32_t d = threadIdx.x % kDims; d < (uint32_t)DV; d += kDims) {
+    for (uint32_t g = threadIdx.x / kDims; g < group; g += kWarps * 32 / kDims) {
       float mall = -INFINITY;
 #pragma unroll
       for (int w = 0; w < kWarps; ++w) mall = fmaxf(mall, mml[(w * kMaxGroup + g) * 2]);
@@ -760,13 +765,12 @@ uint32_t group_tiles(KvLayout kv, uint32_t q_heads) { return (q_heads / kv.num_k
 template <int DK, int DV, bool JOINT>
 int launch_decode_form(const bf16 *q, const bf16 *arena, KvLayout kv, uint32_t layer, AttnBatch batch, uint32_t rows, uint32_t q_heads,
                        uint32_t splits, DecodeScratch scratch, AttnForm form, bf16 *out, cudaStream_t stream) {
-  // as many bytes in flight with one set of rows as with two
-  constexpr int kFormStages = JOINT && DK <= 128 ? 6 : 3;
+  constexpr int kFormStages = 3;
   constexpr uint32_t kSmem = JOINT ? joint_smem_bytes(kFormStages, DK) : decode_smem_bytes(kFormStages, DK, DV);
   static bool attr_set[kMaxDeviceOrdinals] = {};
   ORION_CUDA_CHECK("paged_decode attr", ensure_dynamic_smem(paged_decode_kernel<kFormStages, DK, DV, true, JOINT>, (int)kSmem, attr_set));
   ORION_CUDA_CHECK("paged_decode", launch_pdl(paged_decode_kernel<kFormStages, DK, DV, true, JOINT>,
-                                              dim3(kv.num_kv_heads * group_tiles(kv, q_heads), rows, splits), dim3(kWarps * 32),
+                                              dim3(kv.num_kv_heads * group_tiles(kv, q_heads), rows, splits), dim3((JOINT ? joint_warps(DK) : kWarps) * 32),
                                               (size_t)kSmem, stream, q, arena, kv, layer, batch, q_heads,
                                               splits, scratch, out, FusedQkv{}, form));
   ORION_TRY(after_launch("paged_decode"));
