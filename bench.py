@@ -428,13 +428,14 @@ def metapel_work(meta, rows, contexts, prompts):
     return w + 2 * LAYERED_VOCAB * meta.hidden_size, flops + 2 * outs * LAYERED_VOCAB * meta.hidden_size, cache, attn
 
 
-def zulozen_meta(pkg, name, layers):
+def zulozen_meta(pkg, name, layers, mixtures_only=False):
     z = ZULOZEN_SHAPES[name]
     att = dict(heads=z["heads"], kv_heads=z["heads"] // 4, dim=z["dim"], value_dim=z["dim"], chunk=z["chunk"], rope_dims=z["rot"],
                rope_base=10000.0, scale=z["dim"] ** -0.5, qk_norm=True, sinks=True, head_gate=True)
     dense = pkg.LayerSpec("attention", z["ffn"], activation="relu2", ffn_bias=True, **att)
     mix = pkg.LayerSpec("attention", z["expert_ffn"], experts=z["experts"], experts_per_token=z["top"], shared_dim=z["shared"], **att)
-    return pkg.LayeredMetadata("Zulozen", f"zulozen-{name}", z["hidden"], LAYERED_VOCAB, [mix if i % 2 else dense for i in range(layers)],
+    return pkg.LayeredMetadata("Zulozen", f"zulozen-{name}", z["hidden"], LAYERED_VOCAB,
+                               [mix if i % 2 or mixtures_only else dense for i in range(layers)],
                                1e-6, block="sandwich", untied_lm_head=True, residual_mult=0.5)
 
 
@@ -551,7 +552,7 @@ def llama_work(m, rows, contexts, prompts):
 def run_layered(args):
     """Prefill and decode throughput of a layer-list design at a few layer sizes, and of the Llama layout (same hidden size, head
     count and head size, four query heads per KV head, feed-forward of equal parameter count) on the same
-    batches. Times are CUDA events around whole replayed steps and around one kernel family run back to back."""
+    batches; beside Vusenex also Zulozen with a mixture of equal size in every layer. Times are CUDA events around whole replayed steps and around one kernel family run back to back."""
     import __graft_entry__ as ge
 
     pkg = ge.load_package()
@@ -567,6 +568,9 @@ def run_layered(args):
                                "zulozen": (ZULOZEN_SHAPES, zulozen_meta, zulozen_work),
                                "belizen": (BELIZEN_SHAPES, belizen_meta, belizen_work),
                                "vusenex": (VUSENEX_SHAPES, vusenex_meta, vusenex_work)}[design]
+    kinds = {design: (make_meta, work)}
+    if design == "vusenex":
+        kinds["zulozen"] = (lambda *a: zulozen_meta(*a, mixtures_only=True), zulozen_work)
     layers, out = args.layers if args.layers != 32 else 8, []
     batches = [("decode", b, CONTEXT) for b in (1, 16, 64)] + [("prefill", 1, 2048), ("prefill", 4, 2048)]
     with ClockSampler(0) as clocks:
@@ -576,10 +580,10 @@ def run_layered(args):
                      head_dim=128, vocab_size=LAYERED_VOCAB, ffn_dim=(z["ffn"] * 2 // 3 + 127) // 128 * 128,
                      max_position_embeddings=8192, rope_theta=500000.0, rms_norm_eps=1e-5)
             blocks = max(b * c // BLOCK for _, b, c in batches) + 64
-            for kind in (design, "llama"):
+            for kind in (*kinds, "llama"):
                 kw = dict(compute_dtype=pkg.DType.BF16, max_batch_tokens=8192, max_batch_sequences=64)
-                if kind == design:
-                    meta = make_meta(pkg, name, layers)
+                if kind in kinds:
+                    meta = kinds[kind][0](pkg, name, layers)
                     model = pkg.CudaLayeredModel(meta, blocks, BLOCK, backend, **kw)
                 else:
                     meta = pkg.ModelMetadata(architecture="llama", name="llama", dtype=pkg.DType.BF16, **m)
@@ -610,7 +614,7 @@ def run_layered(args):
                     ms = model.replay(steps) / steps
                     launches = model.last_launch_count()
                     fam = {c: model.replay_categories(steps, c) / steps for c in ("gemm", "attention", "elementwise")}
-                    wb, fl, cb, af = (work(meta, rows, contexts, prompts) if kind == design
+                    wb, fl, cb, af = (kinds[kind][1](meta, rows, contexts, prompts) if kind in kinds
                                       else llama_work(m, rows, contexts, prompts))
                     gemm_s, attn_s = fam["gemm"] / 1e3, fam["attention"] / 1e3
                     out.append({"model": kind, "shape": name, "layers": layers, "mode": mode, "sequences": b, "tokens_each": n,
