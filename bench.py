@@ -515,7 +515,7 @@ def vusenex_meta(pkg, name, layers):
                         q_temp=pkg.QueryTemperature(0.1, 512.0), **both)
     return pkg.LayeredMetadata("Vusenex", f"vusenex-{name}", z["hidden"], LAYERED_VOCAB, [att if i % 2 else lat for i in range(layers)], 1e-6,
                                block="gated_postnorm", untied_lm_head=True, scalar_norms=True, max_positions=8192,
-                               bigram=pkg.Bigram(32749, 31, 17))
+                               bigram=pkg.Bigram(32749, 37, 101))
 
 
 def vusenex_work(meta, rows, contexts, prompts):

@@ -206,7 +206,7 @@ def test_gates_alone(pkg, backend, dtype, part):
 
 
 @pytest.mark.parametrize("rows", [5, 17, 33, 64, 65, 200, 300, 700])
-@pytest.mark.parametrize("experts", [(8, 4, 2, 2, 72, 200), (16, 4, 3, 4, 64, None), (6, 3, 1, 2, 136, 64)])
+@pytest.mark.parametrize("experts", [(8, 4, 2, 2, 72, 200), (16, 8, 5, 4, 64, None), (6, 3, 1, 2, 136, 64)])
 def test_tiles_of_experts(pkg, backend, dtype, rows, experts):
     """Every number of rows per tile, experts with no, few and many rows, products that end inside a tile."""
     cfg = config(128, 64, [latent(1, 16, 16, 16, moe(*experts))])

@@ -123,7 +123,7 @@ def _normed_values(h, w, m, eps):
 
 def _norm_per_head(x, w, eps, real=vusenex.rms_norm):
     """Attention's norms over heads of 48 or 64 instead of all of them at once."""
-    if np.ndim(w) != 1 or w.size not in (704, 192):
+    if np.ndim(w) != 1 or w.size not in (704, 288):
         return real(x, w, eps)
     d = 64 if w.size == 704 else 48
     return real(x.reshape(len(x), -1, d), w.reshape(-1, d), eps).reshape(len(x), -1)
@@ -181,7 +181,7 @@ FAULTS = {
     "gates without bias": ("gated", lambda y, h, m, b: GATED(y, h, m, 0 * b)),
     "weights not renormalised": ("route", lambda h, m, r: (ROUTE(h, m, r)[0], ROUTE(h, m, r)[1] * 0.8)),
     "groups ignored": ("eligible", lambda s, g: np.ones(s.shape, bool)),
-    "groups by the sum of their scores": ("eligible", _group_sum),
+    "groups by the sum of their scores": ("eligible", _group_sum, "broad"),
     "groups of every n-th expert": ("eligible", _strided_groups),
     "silu for gelu": ("gelu", lambda x: x / (1 + np.exp(-x))),
     "shared expert left out": ("mixture", lambda h, w, mlp, real=vusenex.mixture: real(h, w, {**mlp, "shared": None})),

@@ -127,7 +127,7 @@ def _clear_choice(rng, router):
 ODD = config(50, 24, [latent(3, 5, 7, 10, moe(6, 3, 2, 3, 33, 29)), attn(3, 1, 10, moe(5, 5, 3, 2, 37), temp=(1.2, 7)), latent(2, 12, 7, 6, scale=0.1),
                       attn(4, 2, 7, moe(4, 1, 1, 4, 31, 26), temp=None), attn(1, 1, 9, moe(3, 0, 0, 1, 35, 43), temp=(0.35, 1), scale=0.15)], pairs=(23, 1, 1), positions=300)
 # Attention heads that pad to 64, more than eight query heads to a key head, tuned latent sizes, many experts.
-TUNED = config(128, 30, [attn(11, 1, 64, moe(8, 4, 2, 3, 64, 72)), latent(5, 32, 48, 64), attn(4, 2, 48, moe(20, 5, 3, 4, 72), temp=(0.9, 33)),
+TUNED = config(128, 30, [attn(11, 1, 64, moe(8, 4, 2, 3, 64, 72)), latent(5, 32, 48, 64), attn(6, 3, 48, moe(20, 5, 3, 4, 72), temp=(0.9, 33)),
                          latent(12, 16, 32, 96, moe(9, 3, 1, 2, 136, 64))], eps=1e-3, pairs=(101, 1000003, 7919))
 # Heads that pad to 128, long latents, one expert per token.
 WIDE = config(192, 100, [attn(9, 3, 128, moe(6, 2, 1, 1, 192, 136), scale=0.05), latent(20, 64, 64, 192, moe(4, 2, 2, 2, 64, 64)), attn(8, 1, 80)],
